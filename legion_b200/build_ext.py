@@ -24,6 +24,13 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
 ]
+# sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
+PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan"}
+
+
+def _cu_flags(src: Path, verbose: bool) -> list[str]:
+    flags = [f for f in NVCC_FLAGS if f != "--use_fast_math"] if src.stem in PRECISE else list(NVCC_FLAGS)
+    return flags + (["-Xptxas", "-v"] if verbose else [])
 
 
 def _nvcc() -> str:
@@ -47,24 +54,39 @@ def _run(cmd: list[str]) -> str:
     return p.stdout + p.stderr
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
+# the kernels of bf16 / fp32 layer stacks on one GPU: what a model without quantised weights, latent attention,
+# Gated DeltaNet layers or several ranks launches
+CORE_TARGET = ROOT / "_C_core.so"
+CORE = {"gemm_sm100", "moe", "attn_prefill_sm100", "attn_decode_sm100", "attn_decode", "elementwise", "sampling", "spec",
+        "tmap", "conv1d", "hyper", "sgemm", "attn_general", "linear_scan", "linear_scan_sm100", "bindings",
+        "bindings_layers"}
+
+
+def build_core(verbose: bool = False) -> Path:
+    """The subset ``CORE`` as ``legion_b200/_C_core.so``, for a checkout that has not been built: a tool that runs one
+    such model compiles only its kernels. ``ops.sm100.ext`` takes it when ``_C.so`` is absent."""
+    return build(verbose, core=True)
+
+
+def build(verbose: bool = False, force: bool = False, core: bool = False) -> Path:
     import torch
     from torch.utils import cpp_extension
 
     BUILD.mkdir(parents=True, exist_ok=True)
-    cu_files = sorted(CSRC.glob("*.cu"))
-    cpp_files = sorted(CSRC.glob("*.cpp"))
+    cu_files = [f for f in sorted(CSRC.glob("*.cu")) if not core or f.stem in CORE]
+    cpp_files = [f for f in sorted(CSRC.glob("*.cpp")) if not core or f.stem in CORE]
+    target, module = (CORE_TARGET, "_C_core") if core else (TARGET, "_C")
     inc = [f"-I{p}" for p in cpp_extension.include_paths()] + [f"-I{sysconfig.get_paths()['include']}"]
     cuda_home = os.environ.get("CUDA_HOME", "/usr/local/cuda")
     inc.append(f"-I{cuda_home}/include")
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
-    cxx_flags = ["-O2", "-std=c++17", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={abi}", "-DTORCH_EXTENSION_NAME=_C",
-                 "-DTORCH_API_INCLUDE_EXTENSION_H", "-w"]
+    cxx_flags = ["-O2", "-std=c++17", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={abi}", f"-DTORCH_EXTENSION_NAME={module}",
+                 "-DTORCH_API_INCLUDE_EXTENSION_H", "-w"] + (["-DLB_CORE"] if core else [])
 
     jobs = []
     objs = []
     for src in cu_files:
-        flags = NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else [])
+        flags = _cu_flags(src, verbose)
         obj = BUILD / f"{src.stem}.{_hash(src, ' '.join(flags))}.o"
         objs.append(obj)
         if force or not obj.exists():
@@ -86,21 +108,22 @@ def build(verbose: bool = False, force: bool = False) -> Path:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             for name in ex.map(work, jobs):
                 print(f"[build_ext] compiled {name}", file=sys.stderr)
-    # drop stale objects
-    keep = {o.name for o in objs}
+    # drop stale objects of these sources
+    keep = {o.name for o in objs} | {o.name for o in BUILD.glob("bindings*.o") if core}
+    stems = {f.stem for f in cu_files + cpp_files}
     for o in BUILD.glob("*.o"):
-        if o.name not in keep:
+        if o.name not in keep and (not core or o.name.split(".")[0] in stems):
             o.unlink()
 
     newest = max(o.stat().st_mtime for o in objs)
-    if force or jobs or not TARGET.exists() or TARGET.stat().st_mtime < newest:
+    if force or jobs or not target.exists() or target.stat().st_mtime < newest:
         torch_lib = Path(torch.__file__).parent / "lib"
-        link = ["g++", "-shared", "-o", str(TARGET), *map(str, objs), f"-L{torch_lib}", f"-L{cuda_home}/lib64",
+        link = ["g++", "-shared", "-o", str(target), *map(str, objs), f"-L{torch_lib}", f"-L{cuda_home}/lib64",
                 "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-ltorch_python", "-lcudart",
                 f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda_home}/lib64"]
         _run(link)
-        print(f"[build_ext] linked {TARGET}", file=sys.stderr)
-    return TARGET
+        print(f"[build_ext] linked {target}", file=sys.stderr)
+    return target
 
 
 HOST_SRC = ROOT / "csrc_host"

@@ -654,6 +654,10 @@ def make_parser() -> argparse.ArgumentParser:
     s.add_argument("--out", default=None, help=".npz file to write (tokens, logits)")
     s.add_argument("--compare", default=None, help=".npz dump to compare with")
     s.set_defaults(fn=cmd_logits)
+    s = sub.add_parser("trace", help="replay steps of given tokens through a model and write logits")
+    from . import trace
+    trace.add_arguments(s)
+    s.set_defaults(fn=trace.run)
     s = sub.add_parser("tokenize", help="tokenise text with a model's tokenizer")
     s.add_argument("--model", "-m", required=True)
     s.add_argument("text")

@@ -12,6 +12,96 @@ from dataclasses import dataclass, field
 from typing import List, Optional
 
 
+# --------------------------------------------------------------------------------------------------
+# Layer specifications: stacks whose layers each have sizes and constants of their own (``ModelConfig.layers``)
+# --------------------------------------------------------------------------------------------------
+@dataclass
+class AttnSpec:
+    """Grouped-query softmax attention without rotation; values may have a head size of their own."""
+    heads: int
+    kv_heads: int
+    dim: int                           # query / key head size
+    vdim: int                          # value head size
+    scale: float                       # multiplies the scores
+    window: int = 0                    # tokens a position sees, itself included (0 = all)
+    qk_norm: bool = True               # per-head RMS norm of q and k with a plain weight
+    kind: str = "attn"
+
+
+@dataclass
+class LightningSpec:
+    """Linear attention with a constant decay per head, silu on q, k and v, a norm over all heads and an output gate."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: list                        # per head
+    kind: str = "lightning"
+
+
+@dataclass
+class SsdSpec:
+    """Mamba-2 mixer."""
+    heads: int
+    vdim: int                          # head size
+    state: int
+    groups: int = 1                    # B / C groups
+    conv: int = 4                      # taps
+    norm_groups: int = 1               # parts of the gated norm
+    kind: str = "ssd"
+
+
+@dataclass
+class ParallelSpec:
+    """Two mixers side by side over the same input: left_scale * left + right_scale * right."""
+    left: AttnSpec
+    right: SsdSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind: str = "parallel"
+
+
+@dataclass
+class DenseSpec:
+    ff: int
+    act: str = "silu"
+    kind: str = "dense"
+
+
+@dataclass
+class MoeSpec:
+    experts: int
+    top: int
+    ff: int
+    act: str = "silu"
+    router: str = "softmax"            # softmax | sigmoid | softmax_bias (selection by softmax score + correction)
+    correction: bool = False
+    renorm: bool = True
+    n_group: int = 1                   # groups of neighbouring experts, the best keep_group of them stay open
+    keep_group: int = 1
+    group_top: int = 2                 # a group's score sums this many of its best selection scores
+    kind: str = "moe"
+
+
+@dataclass
+class LayerSpec:
+    mixer: object
+    mlp: object = None                 # None: the layer has no feed-forward part
+
+
+_SPECS = {c.__dataclass_fields__["kind"].default: c
+          for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, DenseSpec, MoeSpec)}
+
+
+def spec_from(d):
+    """A specification (or its ``dataclasses.asdict`` form) as the dataclass its ``kind`` names."""
+    if not isinstance(d, dict):
+        return d
+    d = {k: spec_from(v) for k, v in d.items()}
+    if "mixer" in d:
+        return LayerSpec(**d)
+    return _SPECS[d["kind"]](**d)
+
+
 @dataclass
 class ModelConfig:
     arch: str = "qwen3moe"             # registry key (see models.registry)
@@ -57,7 +147,8 @@ class ModelConfig:
     kda_lower: float = -5.0            # lower bound of the log decay: g = lower * sigmoid(-(f(x) + dt_bias) * A)
     # hyper-connections: the residual is ``hyper_streams`` parallel streams mixed before and after every sublayer
     hyper_streams: int = 1
-    hyper_mode: str = "sinkhorn"       # "sinkhorn": per-token pre / post weights and a Sinkhorn-normalised stream mix
+    hyper_mode: str = "sinkhorn"       # "static": per-layer weights that do not depend on the token (stacks with
+                                       # ``layers``). "sinkhorn": per-token pre / post weights and a Sinkhorn-normalised stream mix
                                        # (glm5-next, deepseek41); "gated": a low-rank sigmoid gate per channel mixes
                                        # the normed streams, the block output re-enters every stream with a weight
                                        # of its own, the last mixer is the output norm (qwen4exp)
@@ -111,6 +202,9 @@ class ModelConfig:
     kv_shared_layers: int = 0
     layer_out_scale: bool = False
     ple_dim: int = 0                   # width of the per-layer token embeddings (0 = none)
+    # stacks whose layers have sizes of their own: one LayerSpec per layer. The per-model attention / recurrent / MoE
+    # fields above then only describe the largest layer (memory planning); every layer runs from its specification
+    layers: Optional[List[LayerSpec]] = None
     # multi-token prediction
     mtp_layers: int = 0
     # weights
@@ -118,6 +212,19 @@ class ModelConfig:
     quant: str = "none"                # none | nvfp4 | fp8_block
 
     def __post_init__(self):
+        if self.layers is not None:
+            self.layers = [spec_from(x) for x in self.layers]
+            self.n_layer = len(self.layers)
+            self.layer_kinds = [x.mixer.kind for x in self.layers]
+            attn = [a for a in (self.attn_spec(il) for il in range(self.n_layer)) if a is not None]
+            if attn:
+                big = max(attn, key=lambda a: a.kv_heads * (a.dim + a.vdim))
+                self.n_head, self.n_kv_head, self.head_dim = big.heads, big.kv_heads, big.dim
+            moe = [x.mlp for x in self.layers if isinstance(x.mlp, MoeSpec)]
+            self.n_expert = max([m.experts for m in moe], default=0)
+            self.top_k = max([m.top for m in moe], default=0)
+            self.expert_ff = max([m.ff for m in moe], default=0)
+            self.rope_dim = 0
         if self.rope_dim is None:
             self.rope_dim = self.head_dim if not self.qk_rope_dim else self.qk_rope_dim
         if self.layer_kinds is None:
@@ -131,19 +238,38 @@ class ModelConfig:
         assert len(self.layer_kinds) == self.n_layer
 
     # ---- derived
+    def attn_spec(self, il: int) -> Optional[AttnSpec]:
+        """The softmax-attention part of layer il of a stack with specifications."""
+        m = self.layers[il].mixer
+        return m if isinstance(m, AttnSpec) else (m.left if isinstance(m, ParallelSpec) else None)
+
+    def recurrent_spec(self, il: int):
+        """The part of layer il that carries a recurrent state, of a stack with specifications."""
+        m = self.layers[il].mixer
+        return m if isinstance(m, (LightningSpec, SsdSpec)) else (m.right if isinstance(m, ParallelSpec) else None)
+
     def is_moe_layer(self, il: int) -> bool:
+        if self.layers is not None:
+            return isinstance(self.layers[il].mlp, MoeSpec)
         if self.block_form:
             return il < len(self.layer_kinds) and self.layer_kinds[il] == "moe"
         return self.n_expert > 0 and il >= self.first_dense_layers
 
     def kv_layers(self) -> List[int]:
+        if self.layers is not None:
+            return [i for i in range(self.n_layer) if self.attn_spec(i) is not None]
         return [i for i, k in enumerate(self.layer_kinds) if k in ("attn", "swa", "nope", "mla")]
 
     def recurrent_layers(self) -> List[int]:
+        if self.layers is not None:
+            return [i for i in range(self.n_layer) if self.recurrent_spec(i) is not None]
         return [i for i, k in enumerate(self.layer_kinds) if k in ("gdn", "mamba2", "kda")]
 
     def kv_dims(self, il: int):
         """(n_kv_heads, k_dim, v_dim) stored per token for layer il."""
+        if self.layers is not None:
+            a = self.attn_spec(il)
+            return a.kv_heads, a.dim, a.vdim
         if self.layer_kinds[il] == "mla":
             return 1, self.kv_lora + self.qk_rope_dim, 0
         d, n_kv = self.attn_dims(il)
@@ -336,7 +462,39 @@ def tiny_gemma4() -> ModelConfig:
                        n_expert=8, top_k=2, expert_ff=128, router_mode="softmax", norm_topk=True)
 
 
+def tiny_nisasun() -> ModelConfig:
+    """Nisasun in miniature: linear-attention layers with a constant decay per head beside layers that run windowed
+    attention and a Mamba-2 mixer in parallel, static hyper-connections (3 streams), dense GELU and routed feed-forward
+    parts, one layer without any. Sizes differ from layer to layer."""
+    moe = dict(router="softmax_bias", correction=True, renorm=False, group_top=1)
+    return ModelConfig(
+        arch="nisasun", hidden=160, vocab=640, rms_eps=1e-5, norm_offset=1.0, hyper_streams=3, hyper_mode="static",
+        layers=[LayerSpec(LightningSpec(3, 48, 64, [0.7, 0.95, 0.995]), DenseSpec(192, "gelu_tanh")),
+                LayerSpec(ParallelSpec(AttnSpec(6, 3, 40, 72, 0.17, window=40), SsdSpec(6, 24, 16, 2, 3, 3), 0.6, 0.9),
+                          MoeSpec(10, 3, 56, n_group=5, keep_group=3, **moe)),
+                LayerSpec(ParallelSpec(AttnSpec(4, 1, 64, 32, 0.11, window=75), SsdSpec(2, 48, 40, 1, 5, 2), 1.1, 0.4)),
+                LayerSpec(LightningSpec(5, 32, 24, [0.4, 0.8, 0.9, 0.98, 0.999]), MoeSpec(8, 2, 40, n_group=2,
+                                                                                          keep_group=1, **moe))])
+
+
+def nisasun_3b() -> ModelConfig:
+    """Nisasun with layers the size of a small production model (random weights; speed measurements): 2048 wide, four
+    streams, alternating linear-attention layers (16 heads of 128 x 128) and parallel layers (16 query / 4 key heads of
+    128, window 1024, beside 64 Mamba-2 heads of 64 with state 128), dense and 32-expert feed-forward parts in turn."""
+    decay = [1.0 - 2.0 ** -(2 + 0.5 * h) for h in range(16)]
+    moe = MoeSpec(32, 4, 1024, router="softmax_bias", correction=True, renorm=False, n_group=8, keep_group=4, group_top=1)
+    layers = []
+    for il in range(24):
+        mixer = (ParallelSpec(AttnSpec(16, 4, 128, 128, 128 ** -0.5, window=1024), SsdSpec(64, 64, 128, 8, 4, 8), 0.5, 0.5)
+                 if il % 2 == 0 else LightningSpec(16, 128, 128, decay))
+        layers.append(LayerSpec(mixer, moe if il % 2 else DenseSpec(6144, "gelu_tanh")))
+    return ModelConfig(arch="nisasun", hidden=2048, vocab=65536, rms_eps=1e-5, norm_offset=1.0, hyper_streams=4,
+                       hyper_mode="static", layers=layers)
+
+
 PRESETS = {
+    "tiny-nisasun": tiny_nisasun,
+    "nisasun-3b": nisasun_3b,
     "tiny-muse": tiny_muse,
     "tiny-gemma4": tiny_gemma4,
     "tiny-nemotron-h-moe": tiny_nemotron_h_moe,

@@ -49,26 +49,29 @@ struct DecodeTcArgs {
   int Hq, Hkv, n_splits;
   float scale_log2;
   int window;
-  float* o_part;   // [B, Hq, 2 * n_splits, D]   (part = split * 2 + warpgroup)
+  float* o_part;   // [B, Hq, 2 * n_splits, dv]   (part = split * 2 + warpgroup)
   float* ml_part;  // [B, Hq, 2 * n_splits, 2] (reference maximum in natural-log units, sum)
-  __nv_bfloat16* out;   // [B, Hq, D]
+  int dv;               // value head size (<= DV); the tensor maps end at the head sizes and TMA fills zeros
+  __nv_bfloat16* out;   // [B, Hq, dv]
   int* group_ctr;  // [B * gridDim.x] arrival counters of the splits, zero on entry, left zero on exit
   int* status;
 };
 
-template <int D>
+template <int DK, int DV>
 struct DecodeTcCfg {
   static constexpr int NQ = 16;
   static constexpr int BKV = 128;
-  static constexpr int HALVES = D / 64;
-  static constexpr int KV_BYTES = HALVES * BKV * 128;
+  static constexpr int HALVES = DK / 64;
+  static constexpr int VHALVES = DV / 64;
+  static constexpr int K_BYTES = HALVES * BKV * 128;
+  static constexpr int V_BYTES = VHALVES * BKV * 128;
   static constexpr int Q_BYTES = HALVES * NQ * 128;
   static constexpr int P_BYTES = 2 * NQ * 128;
-  static constexpr int K_STAGES = D <= 64 ? 4 : (D <= 128 ? 3 : 2);
-  static constexpr int V_STAGES = D <= 64 ? 4 : (D <= 128 ? 3 : 1);
-  static constexpr int MT = D <= 128 ? 1 : D / 128;        // 128-row M tiles of O^T
+  static constexpr int K_STAGES = DK <= 64 ? 4 : (DK <= 128 ? 3 : 2);
+  static constexpr int V_STAGES = DV <= 64 ? 4 : (DV <= 128 ? (DK <= 128 ? 3 : 2) : 1);
+  static constexpr int MT = DV <= 128 ? 1 : DV / 128;       // 128-row M tiles of O^T
   static constexpr int TMEM_COLS = (2 * NQ + 2 * MT * NQ <= 64) ? 64 : 128;   // S x 2 + O x 2 (MT x 16 each)
-  static constexpr int SMEM = (K_STAGES + V_STAGES) * KV_BYTES + Q_BYTES + 2 * P_BYTES + 1024 + 1536;
+  static constexpr int SMEM = K_STAGES * K_BYTES + V_STAGES * V_BYTES + Q_BYTES + 2 * P_BYTES + 1024 + 1536;
   static_assert(2 * NQ + 2 * MT * NQ <= TMEM_COLS, "accumulators do not fit the TMEM allocation");
   static_assert(SMEM <= 227 * 1024, "shared memory budget");
 };
@@ -78,18 +81,18 @@ struct DecodeTcCfg {
 // TMEM round trip of the rescale leaves the per-tile critical path.
 static constexpr float DEC_RESCALE_LOG2 = 8.f;
 
-template <int D>
+template <int DK, int DV>
 __global__ void __launch_bounds__(320, 1)
 paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const DecodeTcArgs a) {
-  using Cfg = DecodeTcCfg<D>;
+  using Cfg = DecodeTcCfg<DK, DV>;
   constexpr int NQ = Cfg::NQ, BKV = Cfg::BKV, HALVES = Cfg::HALVES, MT = Cfg::MT;
   constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* k_s = smem;                                   // [KS]
-  uint8_t* v_s = k_s + KS * Cfg::KV_BYTES;               // [VS]
-  uint8_t* q_s = v_s + VS * Cfg::KV_BYTES;
+  uint8_t* v_s = k_s + KS * Cfg::K_BYTES;                // [VS]
+  uint8_t* q_s = v_s + VS * Cfg::V_BYTES;
   uint8_t* p_s = q_s + Cfg::Q_BYTES;                     // [2]
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + 2 * Cfg::P_BYTES);
   uint64_t* q_full = bars;
@@ -114,6 +117,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int b = blockIdx.y;
   const int split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int D = a.dv;
 
   griddep_wait();
   griddep_launch();
@@ -193,13 +197,12 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             ok = false;
             break;
           }
-          uint8_t* dst = (kv ? v_s : k_s) + st * Cfg::KV_BYTES;
-          if (lane == 0) mbar_expect_tx(full, Cfg::KV_BYTES);
+          uint8_t* dst = kv ? v_s + st * Cfg::V_BYTES : k_s + st * Cfg::K_BYTES;
+          if (lane == 0) mbar_expect_tx(full, kv ? Cfg::V_BYTES : Cfg::K_BYTES);
           for (int p = 0; p < ppb; ++p) {
             const int pg = __shfl_sync(0xffffffffu, pg_reg, slot * ppb + p);
             if (lane == 0) {
-#pragma unroll
-              for (int h = 0; h < HALVES; ++h)
+              for (int h = 0; h < (kv ? Cfg::VHALVES : HALVES); ++h)
                 tma_load_3d(dst + h * (BKV * 128) + p * a.page * 128, kv ? &tmV : &tmK, full, h * 64, kvh,
                             pg * a.page);
             }
@@ -216,7 +219,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           const int ks = i % KS;
           if (!mbar_wait(&k_full[ks], (i / KS) & 1, abort_flag)) return false;
           tc_fence_after();
-          const uint32_t ka = smem_u32(k_s + ks * Cfg::KV_BYTES);
+          const uint32_t ka = smem_u32(k_s + ks * Cfg::K_BYTES);
 #pragma unroll
           for (int h = 0; h < HALVES; ++h) {
 #pragma unroll
@@ -244,15 +247,15 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); break;
           }
           tc_fence_after();
-          const uint32_t va = smem_u32(v_s + vs * Cfg::KV_BYTES);
+          const uint32_t va = smem_u32(v_s + vs * Cfg::V_BYTES);
           const uint32_t pa = smem_u32(p_s + wgp * Cfg::P_BYTES);
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
             for (int k = 0; k < BKV / 16; ++k) {
-              // A = V^T rows [mt*128, mt*128+128) of d: two 64-wide MN groups, LBO apart; D = 64 reads the
+              // A = V^T rows [mt*128, mt*128+128) of d: two 64-wide MN groups, LBO apart; DV = 64 reads the
               // only group twice (LBO 0) and the duplicate lanes are never stored.
-              const uint32_t lbo = (D == 64) ? 0u : uint32_t(BKV * 128);
+              const uint32_t lbo = (DV == 64) ? 0u : uint32_t(BKV * 128);
               const uint64_t da = umma_desc_mn_sw128(va + mt * 2 * (BKV * 128) + k * 16 * 128, lbo, 1024);
               const uint64_t db = umma_desc_k_sw128(pa + (k / 4) * (NQ * 128) + (k % 4) * 32);
               umma_f16(tmem_O + (wgp * MT + mt) * NQ, da, db, idesc_o, ((i >> 1) | k) ? 1u : 0u);
@@ -493,11 +496,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 namespace {
 thread_local char g_dec_err[256];
 
-template <int D>
+template <int DK, int DV>
 int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const DecodeTcArgs& a,
                      dim3 grid, cudaStream_t s) {
-  using Cfg = DecodeTcCfg<D>;
-  auto kfn = paged_decode_tc_kernel<D>;
+  using Cfg = DecodeTcCfg<DK, DV>;
+  auto kfn = paged_decode_tc_kernel<DK, DV>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -519,21 +522,24 @@ int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtenso
 const char* paged_decode_tc_last_error() { return g_dec_err; }
 
 // Returns 0 on success, 1 on error, -1 when the shape is outside this kernel (caller falls back).
-int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cache, long n_cells, long cell_stride,
-                           const int* block_table, int table_width, int page, const int* ctx_lens, float scale,
-                           int window, int B, int Hq, int Hkv, int D, int n_splits, float* o_part, float* ml_part,
-                           void* out, int* group_ctr, int n_group_ctr, int* status, cudaStream_t s) {
+int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
+                           long v_cell, const int* block_table, int table_width, int page, const int* ctx_lens,
+                           float scale, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits, float* o_part,
+                           float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status, cudaStream_t s) {
   if (B <= 0) return 0;
-  if ((D != 64 && D != 128 && D != 256) || page <= 0 || 128 % page != 0 || page % 8 != 0 || Hq % Hkv) return -1;
+  if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || k_cell % 8 || v_cell % 8 || page <= 0 ||
+      128 % page != 0 || page % 8 != 0 || Hq % Hkv)
+    return -1;
+  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : 256);
   const int G = Hq / Hkv;
   const int gtiles = (G + 15) / 16;
   if (n_splits < 1 || n_splits > 128 || long(B) * Hkv * gtiles > n_group_ctr) return -1;
-  const CUtensorMap* tq = tmap_3d(q, uint64_t(D), uint64_t(Hq), uint64_t(B), uint64_t(D) * 2, uint64_t(Hq) * D * 2, 64,
+  const CUtensorMap* tq = tmap_3d(q, uint64_t(dk), uint64_t(Hq), uint64_t(B), uint64_t(dk) * 2, uint64_t(Hq) * dk * 2, 64,
                                   16, 1, TM_BF16, true);
-  const CUtensorMap* tk = tmap_3d(k_cache, uint64_t(D), uint64_t(Hkv), uint64_t(n_cells), uint64_t(D) * 2,
-                                  uint64_t(cell_stride) * 2, 64, 1, uint32_t(page), TM_BF16, true);
-  const CUtensorMap* tv = tmap_3d(v_cache, uint64_t(D), uint64_t(Hkv), uint64_t(n_cells), uint64_t(D) * 2,
-                                  uint64_t(cell_stride) * 2, 64, 1, uint32_t(page), TM_BF16, true);
+  const CUtensorMap* tk = tmap_3d(k_cache, uint64_t(dk), uint64_t(Hkv), uint64_t(n_cells), uint64_t(dk) * 2,
+                                  uint64_t(k_cell) * 2, 64, 1, uint32_t(page), TM_BF16, true);
+  const CUtensorMap* tv = tmap_3d(v_cache, uint64_t(dv), uint64_t(Hkv), uint64_t(n_cells), uint64_t(dv) * 2,
+                                  uint64_t(v_cell) * 2, 64, 1, uint32_t(page), TM_BF16, true);
   if (!tq || !tk || !tv) {
     snprintf(g_dec_err, sizeof(g_dec_err), "decode attention: %s", tmap_last_error());
     return 1;
@@ -541,14 +547,14 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   DecodeTcArgs a{};
   a.ctx_lens = ctx_lens; a.block_table = block_table; a.table_width = table_width; a.page = page;
   a.Hq = Hq; a.Hkv = Hkv; a.n_splits = n_splits; a.scale_log2 = scale * 1.4426950408889634f; a.window = window;
-  a.o_part = o_part; a.ml_part = ml_part; a.status = status;
+  a.o_part = o_part; a.ml_part = ml_part; a.status = status; a.dv = dv;
   a.out = static_cast<__nv_bfloat16*>(out); a.group_ctr = group_ctr;
   dim3 grid(Hkv * gtiles, B, n_splits);
-  int rc;
-  if (D == 64) rc = launch_decode_tc<64>(tq, tk, tv, a, grid, s);
-  else if (D == 128) rc = launch_decode_tc<128>(tq, tk, tv, a, grid, s);
-  else rc = launch_decode_tc<256>(tq, tk, tv, a, grid, s);
-  return rc;
+#define LB_DIM(K_, V_) if (DK == K_ && DV == V_) return launch_decode_tc<K_, V_>(tq, tk, tv, a, grid, s);
+  LB_DIM(64, 64) LB_DIM(128, 128) LB_DIM(256, 256) LB_DIM(64, 128) LB_DIM(64, 256) LB_DIM(128, 64) LB_DIM(128, 256)
+  LB_DIM(256, 64) LB_DIM(256, 128)
+#undef LB_DIM
+  return -1;
 }
 
 }  // namespace lb

@@ -92,32 +92,37 @@ struct PrefillArgs {
   float scale_log2;        // softmax scale * log2(e)
   int window;              // 0 = none
   int causal;
-  __nv_bfloat16* out;      // [T, Hq, D]
+  __nv_bfloat16* out;      // [T, Hq, dv]
+  int dk, dv;              // head sizes: at most the template's; the tensor maps end there and TMA fills zeros
   int* status;
 };
 
+template <int N>
+struct IntC { static constexpr int value = N; };
+
 static constexpr float PREFILL_RESCALE_LOG2 = 8.f;
 
-template <int D, int BKV>
+template <int DK, int DV, int BKV>
 struct PrefillCfg {
-  static constexpr bool VSINGLE = false;
-  static constexpr int HALVES = D / 64;               // 64-column (128-byte) halves of a head row
+  static constexpr int HALVES = DK / 64;              // 64-column (128-byte) halves of a query / key row
+  static constexpr int VHALVES = DV / 64;             // of a value row
   static constexpr int Q_BYTES = HALVES * 128 * 128;  // 128 rows x 128 B per half
-  static constexpr int KV_BYTES = HALVES * BKV * 128;
+  static constexpr int K_BYTES = HALVES * BKV * 128;
+  static constexpr int V_BYTES = VHALVES * BKV * 128;
   static constexpr int P_BYTES = (BKV / 64) * 128 * 128;
   static constexpr int STAGES = 3;                      // K stages
   static constexpr int VSTAGES = 2;
   // no alignment slack: the dynamic shared memory of this kernel starts 1024-byte aligned (checked at entry)
-  static constexpr int SMEM = Q_BYTES + (STAGES + VSTAGES) * KV_BYTES + 256;
-  static constexpr int TMEM_RAW = 2 * BKV + D;          // two score buffers + the output accumulator
+  static constexpr int SMEM = Q_BYTES + STAGES * K_BYTES + VSTAGES * V_BYTES + 256;
+  static constexpr int TMEM_RAW = 2 * BKV + DV;         // two score buffers + the output accumulator
   static constexpr int TMEM_COLS = TMEM_RAW <= 128 ? 128 : (TMEM_RAW <= 256 ? 256 : 512);
 };
 
-template <int D, int BKV>
-__global__ void __launch_bounds__(160, (D == 128 && BKV == 64) ? 2 : 1)
+template <int DK, int DV, int BKV>
+__global__ void __launch_bounds__(160, (DK <= 128 && DV <= 128 && BKV == 64) ? 2 : 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const PrefillArgs a) {
-  using Cfg = PrefillCfg<D, BKV>;
+  using Cfg = PrefillCfg<DK, DV, BKV>;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw;
   if (smem_u32(smem_raw) & 1023u) {       // swizzled tiles need 1024-byte alignment; uniform per CTA, before any barrier
@@ -126,8 +131,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
   uint8_t* q_s = smem;
   uint8_t* k_s = q_s + Cfg::Q_BYTES;                       // [STAGES] K tiles
-  uint8_t* v_s = k_s + Cfg::STAGES * Cfg::KV_BYTES;        // [VSTAGES] V tiles
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + Cfg::VSTAGES * Cfg::KV_BYTES);
+  uint8_t* v_s = k_s + Cfg::STAGES * Cfg::K_BYTES;         // [VSTAGES] V tiles
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + Cfg::VSTAGES * Cfg::V_BYTES);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;   // [3]
   uint64_t* v_full = bars + 4;   // [2]
@@ -191,21 +196,25 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 4) {
     if (lane == 0) {
       // ------------------------------------------------------------ loads + MMA issue
-      auto load_tile = [&](const CUtensorMap* tm, uint8_t* dst, uint64_t* bar, int blk) {
+      auto load_tile = [&](const CUtensorMap* tm, uint8_t* dst, uint64_t* bar, int blk, auto halves) {
         const int tok0 = blk * BKV;
-        mbar_expect_tx(bar, Cfg::KV_BYTES);
+        mbar_expect_tx(bar, halves.value * BKV * 128);
         for (int p = 0; p < pages_per_blk; ++p) {
           const int tok = tok0 + p * a.page;
           // pages past the end of the sequence read cell row 0 of a valid page: masked later
           const int pg = (tok < ctx) ? bt[tok / a.page] : bt[0];
           const int cell = pg * a.page;
 #pragma unroll
-          for (int h = 0; h < Cfg::HALVES; ++h)
+          for (int h = 0; h < halves.value; ++h)
             tma_load_3d(dst + h * (BKV * 128) + p * a.page * 128, tm, bar, h * 64, kvh, cell);
         }
       };
-      auto load_k = [&](int blk, int stage) { load_tile(&tmK, k_s + stage * Cfg::KV_BYTES, &k_full[stage], blk); };
-      auto load_v = [&](int blk, int stage) { load_tile(&tmV, v_s + stage * Cfg::KV_BYTES, &v_full[stage], blk); };
+      auto load_k = [&](int blk, int stage) {
+        load_tile(&tmK, k_s + stage * Cfg::K_BYTES, &k_full[stage], blk, IntC<Cfg::HALVES>{});
+      };
+      auto load_v = [&](int blk, int stage) {
+        load_tile(&tmV, v_s + stage * Cfg::V_BYTES, &v_full[stage], blk, IntC<Cfg::VHALVES>{});
+      };
       mbar_expect_tx(q_full, Cfg::Q_BYTES);
 #pragma unroll
       for (int h = 0; h < Cfg::HALVES; ++h)
@@ -215,7 +224,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       load_v(blk_lo, 0);
       if (n_blk > 1) load_v(blk_lo + 1, 1);
       constexpr uint32_t idesc_s = umma_idesc(128, BKV, 1, 1, 0, 0);
-      constexpr uint32_t idesc_o = umma_idesc(128, D, 1, 1, 0, 1);  // B (= V) is MN-major
+      constexpr uint32_t idesc_o = umma_idesc(128, DV, 1, 1, 0, 1);  // B (= V) is MN-major
       bool ok = mbar_wait(q_full, 0, abort_flag);
       if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); }
       const uint32_t qa = smem_u32(q_s);
@@ -226,7 +235,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); return false;
         }
         tc_fence_after();
-        const uint32_t ka = smem_u32(k_s + st * Cfg::KV_BYTES);
+        const uint32_t ka = smem_u32(k_s + st * Cfg::K_BYTES);
         const uint32_t ts = tmem_S + uint32_t(j & 1) * BKV;
 #pragma unroll
         for (int h = 0; h < Cfg::HALVES; ++h) {
@@ -260,7 +269,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); break;
         }
         tc_fence_after();
-        const uint32_t va = smem_u32(v_s + (i & 1) * Cfg::KV_BYTES);
+        const uint32_t va = smem_u32(v_s + (i & 1) * Cfg::V_BYTES);
         const uint32_t tp = tmem_S + uint32_t(i & 1) * BKV;      // P(i) sits over the scores it was computed from
 #pragma unroll
         for (int k = 0; k < BKV / 16; ++k) {
@@ -419,7 +428,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           }
           tc_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < D; c += 32) {
+          for (int c = 0; c < DV; c += 32) {
             uint32_t r[32];
             tmem_ld32(tmem_O + lane_off + c, r);
             tmem_ld_wait();
@@ -451,9 +460,9 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     if (ok) {
       tc_fence_after();
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = a.out + (long(q0 + tile_row0 + row) * a.Hq + head) * D;
+      __nv_bfloat16* orow = a.out + (long(q0 + tile_row0 + row) * a.Hq + head) * a.dv;
 #pragma unroll 1
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < DV; c += 32) {
         uint32_t r[32];
         if (n_blk > 0) {
           tmem_ld32(tmem_O + lane_off + c, r);
@@ -471,7 +480,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             o.y = pack_bf16x2(__uint_as_float(r[8 * v + 2]) * inv, __uint_as_float(r[8 * v + 3]) * inv);
             o.z = pack_bf16x2(__uint_as_float(r[8 * v + 4]) * inv, __uint_as_float(r[8 * v + 5]) * inv);
             o.w = pack_bf16x2(__uint_as_float(r[8 * v + 6]) * inv, __uint_as_float(r[8 * v + 7]) * inv);
-            dst[v] = o;
+            if (c + 8 * v < a.dv) dst[v] = o;
           }
         }
       }
@@ -488,11 +497,11 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 namespace {
 thread_local char g_attn_err[256];
 
-template <int D, int BKV>
+template <int DK, int DV, int BKV>
 int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const PrefillArgs& a,
                    dim3 grid, cudaStream_t s) {
-  using Cfg = PrefillCfg<D, BKV>;
-  auto kfn = prefill_attn_kernel<D, BKV>;
+  using Cfg = PrefillCfg<DK, DV, BKV>;
+  auto kfn = prefill_attn_kernel<DK, DV, BKV>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -513,28 +522,30 @@ int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorM
 
 const char* prefill_attn_last_error() { return g_attn_err; }
 
-int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells,
-                        long cell_stride, const int* cu_q, const int* ctx_lens, const int* block_table,
-                        int table_width, int page, int n_seqs, int max_q_len, int Hq, int Hkv, int D, float scale,
-                        int window, int causal, void* out, int* status, cudaStream_t s) {
+int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
+                        long v_cell, const int* cu_q, const int* ctx_lens, const int* block_table, int table_width,
+                        int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, int window,
+                        int causal, void* out, int* status, cudaStream_t s) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
-  const int BKV = D >= 128 ? 64 : 128;
+  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : 256);
+  const int BKV = (DK >= 128 || DV >= 128) ? 64 : 128;
   if (page <= 0 || BKV % page != 0 || page % 8 != 0) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: page size %d must be a multiple of 8 dividing %d",
              page, BKV);
     return 1;
   }
-  if (D != 64 && D != 128 && D != 256) {
-    snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: head dim %d not supported", D);
+  if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || k_cell % 8 || v_cell % 8) {
+    snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: head sizes %d / %d not supported", dk, dv);
     return 1;
   }
-  // q viewed as [T, Hq, D]; caches as [cells, Hkv, D] with cell pitch cell_stride elements
-  const CUtensorMap* tq = tmap_3d(q, uint64_t(D), uint64_t(Hq), uint64_t(T), uint64_t(D) * 2,
-                                  uint64_t(Hq) * D * 2, 64, 1, 128, TM_BF16, true);
-  const CUtensorMap* tk = tmap_3d(k_cache, uint64_t(D), uint64_t(Hkv), uint64_t(n_cells), uint64_t(D) * 2,
-                                  uint64_t(cell_stride) * 2, 64, 1, uint32_t(page), TM_BF16, true);
-  const CUtensorMap* tv = tmap_3d(v_cache, uint64_t(D), uint64_t(Hkv), uint64_t(n_cells), uint64_t(D) * 2,
-                                  uint64_t(cell_stride) * 2, 64, 1, uint32_t(page), TM_BF16, true);
+  // q viewed as [T, Hq, dk]; caches as [cells, Hkv, dk | dv] with cell pitches in elements. A box that reaches past the
+  // head size reads zeros there, so head sizes between the template sizes need no padding in memory.
+  const CUtensorMap* tq = tmap_3d(q, uint64_t(dk), uint64_t(Hq), uint64_t(T), uint64_t(dk) * 2,
+                                  uint64_t(Hq) * dk * 2, 64, 1, 128, TM_BF16, true);
+  const CUtensorMap* tk = tmap_3d(k_cache, uint64_t(dk), uint64_t(Hkv), uint64_t(n_cells), uint64_t(dk) * 2,
+                                  uint64_t(k_cell) * 2, 64, 1, uint32_t(page), TM_BF16, true);
+  const CUtensorMap* tv = tmap_3d(v_cache, uint64_t(dv), uint64_t(Hkv), uint64_t(n_cells), uint64_t(dv) * 2,
+                                  uint64_t(v_cell) * 2, 64, 1, uint32_t(page), TM_BF16, true);
   if (!tq || !tk || !tv) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: %s", tmap_last_error());
     return 1;
@@ -542,11 +553,13 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
   PrefillArgs a{};
   a.cu_q = cu_q; a.ctx_lens = ctx_lens; a.block_table = block_table; a.table_width = table_width; a.page = page;
   a.Hq = Hq; a.Hkv = Hkv; a.scale_log2 = scale * 1.4426950408889634f; a.window = window; a.causal = causal;
-  a.out = static_cast<__nv_bfloat16*>(out); a.status = status;
+  a.out = static_cast<__nv_bfloat16*>(out); a.dk = dk; a.dv = dv; a.status = status;
   dim3 grid((max_q_len + 127) / 128, Hq, n_seqs);
-  if (D == 64) return launch_prefill<64, 128>(tq, tk, tv, a, grid, s);
-  if (D == 128) return launch_prefill<128, 64>(tq, tk, tv, a, grid, s);
-  return launch_prefill<256, 64>(tq, tk, tv, a, grid, s);
+#define LB_DIM(K_, V_, B_) if (DK == K_ && DV == V_) return launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
+  LB_DIM(64, 64, 128) LB_DIM(128, 128, 64) LB_DIM(256, 256, 64)
+  LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64) LB_DIM(256, 128, 64)
+#undef LB_DIM
+  return 1;
 }
 
 }  // namespace lb

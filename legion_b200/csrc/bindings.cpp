@@ -1,4 +1,5 @@
-// Python bindings (module legion_b200._C): thin checks + pointer extraction around the launchers.
+// Python bindings (module legion_b200._C): thin checks + pointer extraction around the launchers. With LB_CORE only
+// what the bf16 / fp32 layer stack of one GPU needs is bound (build_ext.build_core).
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
@@ -41,7 +42,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
            const OptT& ws, const OptT& counters, Tensor& status, const OptT& tile_group, const OptT& tile_tok0,
            const OptT& tile_ntok, const OptT& meta, int64_t max_tiles, int64_t rows_per_group, int64_t n_tok,
            std::vector<int64_t> out_peer, const OptT& tile_out0, const OptT& w_scales, const OptT& w_gscale,
-           int64_t x_group_col, int64_t k_override) {
+           int64_t x_group_col, int64_t k_override, int64_t act) {
   const bool fp4 = w_scales.has_value();     // w = NVFP4 codes [rows, K/2] uint8, w_scales = e4m3 bytes [rows, K/16]
   if (fp4) {
     TORCH_CHECK(w.scalar_type() == at::kByte && w_scales->is_contiguous() && w_scales->element_size() == 1 &&
@@ -76,7 +77,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
   }
   h.w_scales = fp4 ? w_scales->data_ptr() : nullptr;
   h.w_gscale = optp<float>(w_gscale);
-  h.bn = int(bn); h.dual = dual;
+  h.bn = int(bn); h.dual = dual; h.act = int(act);
   h.tile_group = optp<int>(tile_group); h.tile_tok0 = optp<int>(tile_tok0); h.tile_ntok = optp<int>(tile_ntok);
   h.n_tiles_dev = optp<int>(meta);
   h.tile_out0 = optp<int>(tile_out0);
@@ -329,22 +330,25 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   Tensor& ml_part, Tensor& out, bool use_tc, Tensor& status, Tensor& counters) {
   check_bf16(q, "q");
   c10::cuda::CUDAGuard guard(q.device());
-  const int B = int(q.size(0)), Hq = int(q.size(1)), D = int(q.size(2));
+  const int B = int(q.size(0)), Hq = int(q.size(1)), D = int(q.size(2)), DV = int(v_cache.size(-1));
   const int page = int(k_cache.size(-3)), Hkv = int(k_cache.size(-2));
+  TORCH_CHECK(k_cache.size(-1) == D && out.size(-1) == DV && v_cache.size(-2) == Hkv, "paged_decode: head sizes");
   const int64_t parts = n_splits * (use_tc ? 2 : 1);   // the tensor-core kernel writes two partials per split
-  TORCH_CHECK(o_part.numel() >= int64_t(B) * Hq * parts * D && ml_part.numel() >= int64_t(B) * Hq * parts * 2,
+  TORCH_CHECK(o_part.numel() >= int64_t(B) * Hq * parts * DV && ml_part.numel() >= int64_t(B) * Hq * parts * 2,
               "paged_decode: partial buffers too small");
   if (use_tc && k_cache.is_contiguous() && v_cache.is_contiguous() && q.is_contiguous() && out.is_contiguous()) {
     const long n_cells = k_cache.numel() / (long(Hkv) * D);
     const int rc = lb::paged_decode_tc_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), n_cells,
-                                              long(Hkv) * D, block_table.data_ptr<int>(), int(block_table.size(1)),
-                                              page, ctx_lens.data_ptr<int>(), float(scale), int(window), B, Hq, Hkv,
-                                              D, int(n_splits), o_part.data_ptr<float>(), ml_part.data_ptr<float>(),
-                                              out.data_ptr(), counters.data_ptr<int>(), int(counters.numel()),
-                                              reinterpret_cast<int*>(status.data_ptr()), cur_stream());
+                                              long(Hkv) * D, long(Hkv) * DV, block_table.data_ptr<int>(),
+                                              int(block_table.size(1)), page, ctx_lens.data_ptr<int>(), float(scale),
+                                              int(window), B, Hq, Hkv, D, DV, int(n_splits), o_part.data_ptr<float>(),
+                                              ml_part.data_ptr<float>(), out.data_ptr(), counters.data_ptr<int>(),
+                                              int(counters.numel()), reinterpret_cast<int*>(status.data_ptr()),
+                                              cur_stream());
     TORCH_CHECK(rc <= 0, lb::paged_decode_tc_last_error());
     if (rc == 0) return;
   }
+  TORCH_CHECK(DV == D, "paged_decode: keys and values of different sizes need the tensor-core kernel");
   const int rc = lb::paged_decode_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.stride(-3),
                                          block_table.data_ptr<int>(), int(block_table.size(1)), page,
                                          ctx_lens.data_ptr<int>(), float(scale), int(window), B, Hq, Hkv, D,
@@ -360,19 +364,21 @@ void prefill_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous(), "prefill_attn: q/out must be contiguous [T, Hq, D]");
   c10::cuda::CUDAGuard guard(q.device());
   const long T = q.size(0);
-  const int Hq = int(q.size(1)), D = int(q.size(2));
+  const int Hq = int(q.size(1)), D = int(q.size(2)), DV = int(v_cache.size(-1));
   const int page = int(k_cache.size(-3)), Hkv = int(k_cache.size(-2));
   const long n_cells = k_cache.numel() / (long(Hkv) * D);
+  TORCH_CHECK(k_cache.size(-1) == D && out.size(-1) == DV && v_cache.size(-2) == Hkv, "prefill_attn: head sizes");
   TORCH_CHECK(k_cache.is_contiguous() && v_cache.is_contiguous(), "prefill_attn: caches must be contiguous");
   const int rc = lb::prefill_attn_launch(q.data_ptr(), T, k_cache.data_ptr(), v_cache.data_ptr(), n_cells,
-                                         long(Hkv) * D, cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(),
+                                         long(Hkv) * D, long(Hkv) * DV, cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                          block_table.data_ptr<int>(), int(block_table.size(1)), page,
-                                         int(ctx_lens.numel()), int(max_q_len), Hq, Hkv, D, float(scale), int(window),
+                                         int(ctx_lens.numel()), int(max_q_len), Hq, Hkv, D, DV, float(scale), int(window),
                                          causal ? 1 : 0, out.data_ptr(), reinterpret_cast<int*>(status.data_ptr()),
                                          cur_stream());
   TORCH_CHECK(rc == 0, lb::prefill_attn_last_error());
 }
 
+#ifndef LB_CORE
 void mla_attn(const Tensor& q_abs, const Tensor& cache, const Tensor& cu_q, const Tensor& ctx_lens,
               const Tensor& block_table, int64_t page, int64_t max_q_len, double scale, int64_t n_splits,
               const OptT& o_part, const OptT& ml_part, Tensor& out, Tensor& status) {
@@ -418,15 +424,16 @@ void mla_prep(const Tensor& kva, const Tensor& norm_w, double eps, double w_offs
                                   cache.data_ptr(), 576, q_abs.data_ptr(), int(kva.size(0)), cur_stream()) == 0,
               "mla_prep launch failed");
 }
+#endif
 
 void router_topk(const Tensor& logits, const OptT& bias, int64_t k, int64_t mode, bool renorm, double route_scale,
-                 int64_t n_group, int64_t topk_group, Tensor& ids, Tensor& wts) {
+                 int64_t n_group, int64_t topk_group, Tensor& ids, Tensor& wts, int64_t group_top) {
   TORCH_CHECK(logits.scalar_type() == at::kFloat && logits.stride(1) == 1, "router logits must be float32");
   c10::cuda::CUDAGuard guard(logits.device());
   TORCH_CHECK(lb::router_topk_launch(logits.data_ptr<float>(), logits.stride(0), optp<float>(bias),
                                      int(logits.size(1)), int(k), int(mode), renorm ? 1 : 0, float(route_scale),
-                                     int(n_group), int(topk_group), ids.data_ptr<int>(), wts.data_ptr<float>(),
-                                     int(logits.size(0)), cur_stream()) == 0,
+                                     int(n_group), int(topk_group), int(group_top), ids.data_ptr<int>(),
+                                     wts.data_ptr<float>(), int(logits.size(0)), cur_stream()) == 0,
               "router_topk: unsupported (experts <= 512, k <= 32, groups <= 32)");
 }
 
@@ -435,7 +442,8 @@ void moe_route_small(const Tensor& x, const OptT& norm_w, double eps, double w_o
                      int64_t n_group, int64_t topk_group, Tensor& logits, Tensor& ids, Tensor& wts, int64_t bn,
                      Tensor& tile_group, Tensor& slot_base, Tensor& tile_ntok, Tensor& meta, Tensor& out_rows,
                      Tensor& tok_scale, Tensor& done_ctr, int64_t e_lo, int64_t n_local, const OptT& sh_gate_w,
-                     const OptT& sh_logit, bool shared_slot, Tensor& status, Tensor& active) {
+                     const OptT& sh_logit, bool shared_slot, Tensor& status, Tensor& active,
+                     int64_t group_top) {
   check_bf16(x, "x");
   check_bf16(w, "w");
   const int64_t T = x.size(0), E = w.size(0);
@@ -461,8 +469,8 @@ void moe_route_small(const Tensor& x, const OptT& norm_w, double eps, double w_o
                   x_normed.has_value() ? x_normed->data_ptr() : nullptr,
                   x_normed.has_value() ? x_normed->stride(0) : 0, w.data_ptr(), w.stride(0), int(x.size(1)),
                   logits.data_ptr<float>(), optp<float>(bias), int(E), int(k), int(mode), renorm ? 1 : 0,
-                  float(route_scale), int(n_group), int(topk_group), ids.data_ptr<int>(), wts.data_ptr<float>(),
-                  int(T), int(bn), tile_group.data_ptr<int>(), slot_base.data_ptr<int>(), tile_ntok.data_ptr<int>(),
+                  float(route_scale), int(n_group), int(topk_group), int(group_top), ids.data_ptr<int>(),
+                  wts.data_ptr<float>(), int(T), int(bn), tile_group.data_ptr<int>(), slot_base.data_ptr<int>(), tile_ntok.data_ptr<int>(),
                   meta.data_ptr<int>(), out_rows.data_ptr<int>(), tok_scale.data_ptr<float>(),
                   reinterpret_cast<unsigned int*>(done_ctr.data_ptr()), int(e_lo), int(n_local),
                   sh_gate_w.has_value() ? sh_gate_w->data_ptr() : nullptr, optpm<float>(sh_logit), shared_slot ? 1 : 0,
@@ -578,6 +586,7 @@ void bind_gdn(pybind11::module_& m);
 void bind_comm(pybind11::module_& m);
 void bind_quant(pybind11::module_& m);
 void bind_ep(pybind11::module_& m);
+void bind_layers(pybind11::module_& m);
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("wgemm", &wgemm, pybind11::arg("w"), pybind11::arg("x"), pybind11::arg("out"), pybind11::arg("residual"),
@@ -587,7 +596,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         pybind11::arg("tile_ntok"), pybind11::arg("meta"), pybind11::arg("max_tiles"), pybind11::arg("rows_per_group"),
         pybind11::arg("n_tok"), pybind11::arg("out_peer"), pybind11::arg("tile_out0") = pybind11::none(),
         pybind11::arg("w_scales") = pybind11::none(), pybind11::arg("w_gscale") = pybind11::none(),
-        pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0);
+        pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0, pybind11::arg("act") = 0);
   m.def("wgemm_fp8", &wgemm_fp8);
   m.def("wgemm_fp8_q", &wgemm_fp8_q);
   m.def("wgemm_allreduce", &wgemm_allreduce);
@@ -599,9 +608,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("embed", &embed);
   m.def("paged_decode", &paged_decode);
   m.def("prefill_attn", &prefill_attn);
+#ifndef LB_CORE
   m.def("mla_attn", &mla_attn);
   m.def("mla_prep", &mla_prep);
-  m.def("router_topk", &router_topk);
+#endif
+  m.def("router_topk", &router_topk, pybind11::arg("logits"), pybind11::arg("bias"), pybind11::arg("k"),
+        pybind11::arg("mode"), pybind11::arg("renorm"), pybind11::arg("route_scale"), pybind11::arg("n_group"),
+        pybind11::arg("topk_group"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("group_top") = 2);
+  // group_top: how many of a group's best scores its rank sums up (the other routers of this library sum two)
   m.def("moe_route_small", &moe_route_small);
   m.def("moe_plan", &moe_plan);
   m.def("moe_plan_gather", &moe_plan_gather);
@@ -624,6 +638,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
                                           top_lp.data_ptr<float>(), cur_stream()) == 0,
                 "token_logprobs: at most 20 alternatives");
   });
+#ifndef LB_CORE
   m.def("spec_accept", [](const Tensor& target, const Tensor& cu, const Tensor& draft, const Tensor& n_draft,
                           Tensor& accepted, Tensor& bonus, Tensor& any_rejected) {
     c10::cuda::CUDAGuard guard(target.device());
@@ -633,10 +648,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
                                        accepted.data_ptr<int>(), bonus.data_ptr<int>(), any_rejected.data_ptr<int>(),
                                        cur_stream()) == 0, "spec_accept failed");
   });
+#endif
   m.def("set_pdl", [](bool on) { lb::set_pdl(on); });
   m.def("pdl_enabled", []() { return lb::pdl_enabled(); });
+#ifndef LB_CORE
   bind_gdn(m);
   bind_comm(m);
   bind_quant(m);
   bind_ep(m);
+#endif
+  bind_layers(m);
 }

@@ -1,0 +1,296 @@
+// Bindings of the layer kernels that take bf16 and fp32 activations (layers.h), and of the short convolution.
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/extension.h>
+
+#include "gdn.h"
+#include "layers.h"
+
+namespace {
+using torch::Tensor;
+using OptT = c10::optional<Tensor>;
+
+cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+template <typename T>
+T* optp(const OptT& t) {
+  return t.has_value() ? reinterpret_cast<T*>(t->data_ptr()) : nullptr;
+}
+
+// activation type of a tensor: fp32 or bf16, innermost dimension contiguous
+bool is_f32(const Tensor& t, const char* name) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16), name,
+              " must be a float32 or bfloat16 CUDA tensor");
+  TORCH_CHECK(t.stride(-1) == 1 || t.size(-1) == 1, name, " must be contiguous in its last dimension");
+  return t.scalar_type() == at::kFloat;
+}
+void same(const Tensor& t, bool f32, const char* name) {
+  TORCH_CHECK(is_f32(t, name) == f32, name, " must have the activation type");
+}
+void f32c(const Tensor& t, int64_t n, const char* name) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() >= n, name,
+              " must be a contiguous float32 tensor of at least ", n, " elements");
+}
+
+lb::LinScanArgs scan_args(const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay,
+                          const OptT& dt, const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z,
+                          Tensor& state, const Tensor& cu, const Tensor& slots, int64_t H, int64_t G, int64_t N,
+                          int64_t P, Tensor& out, bool write_state) {
+  const bool f32 = is_f32(q, "q");
+  same(k, f32, "k");
+  same(v, f32, "v");
+  same(out, f32, "out");
+  const int64_t T = q.size(0);
+  TORCH_CHECK(q.dim() == 2 && k.dim() == 2 && v.dim() == 2 && q.size(1) >= G * N && k.size(1) >= G * N && v.size(1) >= H * P &&
+                  k.size(0) == T && v.size(0) == T && out.dim() == 2 && out.size(0) == T && out.size(1) >= H * P,
+              "linear scan: q, k [T, G * N], v and out [T, H * P]");
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == H &&
+                  state.size(2) == P && state.size(3) == N, "linear scan: state [slots, H, P, N] float32");
+  TORCH_CHECK(cu.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && cu.numel() == slots.numel() + 1,
+              "linear scan: int32 sequence bounds and slots");
+  lb::LinScanArgs a{};
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.k = k.data_ptr(); a.ldk = k.stride(0); a.v = v.data_ptr(); a.ldv = v.stride(0);
+  a.silu_in = silu_in;
+  if (decay.has_value()) {
+    f32c(*decay, H, "decay");
+    a.decay = decay->data_ptr<float>();
+  } else {
+    TORCH_CHECK(dt.has_value() && dt_bias.has_value() && A.has_value(), "linear scan: step sizes, their bias and A");
+    same(*dt, f32, "dt");
+    TORCH_CHECK(dt->size(0) == T && dt->size(1) >= H, "linear scan: dt [T, H]");
+    f32c(*dt_bias, H, "dt_bias");
+    f32c(*A, H, "A");
+    a.dt = dt->data_ptr(); a.lddt = dt->stride(0);
+    a.dt_bias = dt_bias->data_ptr<float>(); a.A = A->data_ptr<float>();
+  }
+  if (D.has_value()) {
+    f32c(*D, H, "D");
+    a.D = D->data_ptr<float>();
+  }
+  if (z.has_value()) {
+    same(*z, f32, "z");
+    TORCH_CHECK(z->size(0) == T && z->size(1) >= H * P, "linear scan: z [T, H * P]");
+    a.z = z->data_ptr(); a.ldz = z->stride(0);
+  }
+  a.state = state.data_ptr<float>();
+  a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>();
+  a.n_seqs = int(slots.numel()); a.T = int(T); a.H = int(H); a.G = int(G); a.N = int(N); a.P = int(P);
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  a.write_state = write_state;
+  return a;
+}
+}  // namespace
+
+void bind_layers(pybind11::module_& m) {
+  m.def("hyper_step", [](const OptT& x_in, Tensor& x_out, const OptT& emb, const OptT& ids, const OptT& y0, double c0,
+                         int64_t y_rows, const OptT& y1, double c1, const OptT& mix, const OptT& out_w, const OptT& in_w,
+                         const Tensor& norm_w, double eps, double w_offset, Tensor& h) {
+    const bool f32 = is_f32(h, "h");
+    TORCH_CHECK(x_out.dim() == 3 && x_out.is_contiguous() && x_out.scalar_type() == at::kFloat,
+                "hyper_step: streams are contiguous float32 [rows, streams, width]");
+    const int64_t R = x_out.size(0), S = x_out.size(1), H = x_out.size(2);
+    TORCH_CHECK(h.dim() == 2 && h.size(0) == R && h.size(1) == H, "hyper_step: h [rows, width]");
+    lb::HyperArgs a{};
+    a.x_out = x_out.data_ptr<float>();
+    if (x_in.has_value()) {
+      TORCH_CHECK(x_in->sizes() == x_out.sizes() && x_in->is_contiguous() && x_in->scalar_type() == at::kFloat,
+                  "hyper_step: x_in like x_out");
+      TORCH_CHECK(y0.has_value() && mix.has_value() && out_w.has_value(), "hyper_step: sublayer output and its weights");
+      same(*y0, f32, "y0");
+      TORCH_CHECK(y0->dim() == 2 && y0->size(1) == H && y0->size(0) >= R * y_rows && y_rows >= 1,
+                  "hyper_step: y0 [rows * y_rows, width]");
+      f32c(*mix, S * S, "mix");
+      f32c(*out_w, S, "out_w");
+      a.x_in = x_in->data_ptr<float>();
+      a.y0 = y0->data_ptr(); a.ldy0 = y0->stride(0);
+      if (y1.has_value()) {
+        same(*y1, f32, "y1");
+        TORCH_CHECK(y1->dim() == 2 && y1->size(1) == H && y1->size(0) >= R, "hyper_step: y1 [rows, width]");
+        a.y1 = y1->data_ptr(); a.ldy1 = y1->stride(0);
+      }
+      a.mix = mix->data_ptr<float>(); a.out_w = out_w->data_ptr<float>();
+    } else {
+      TORCH_CHECK(emb.has_value() && emb->dim() == 2 && emb->size(1) == H, "hyper_step: embedding rows");
+      same(*emb, f32, "emb");
+      a.emb = emb->data_ptr(); a.ld_emb = emb->stride(0); a.vocab = int(emb->size(0));
+      if (ids.has_value()) {
+        TORCH_CHECK(ids->scalar_type() == at::kInt && ids->is_contiguous() && ids->numel() == R, "hyper_step: int32 ids");
+        a.ids = ids->data_ptr<int>();
+      } else {
+        TORCH_CHECK(emb->size(0) >= R, "hyper_step: one embedding row per token");
+      }
+    }
+    if (in_w.has_value()) {
+      f32c(*in_w, S, "in_w");
+      a.in_w = in_w->data_ptr<float>();
+    }
+    f32c(norm_w, H, "norm_w");
+    a.norm_w = norm_w.data_ptr<float>(); a.eps = float(eps); a.w_offset = float(w_offset);
+    a.c0 = float(c0); a.c1 = float(c1); a.y_rows = int(y_rows);
+    a.h = h.data_ptr(); a.ldh = h.stride(0); a.rows = int(R); a.S = int(S); a.H = int(H);
+    c10::cuda::CUDAGuard guard(h.device());
+    TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "hyper_step: at most 16 streams of 51200 columns");
+  });
+  m.def("sgemm", [](const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, const OptT& tok_scale,
+                    const OptT& out_rows, int64_t n_feat, bool dual, int64_t dual_offset, int64_t act,
+                    const OptT& tile_group, const OptT& tile_tok0, const OptT& tile_ntok, const OptT& meta,
+                    int64_t max_tiles, int64_t rows_per_group, int64_t n_tok) {
+    const bool f32 = is_f32(x, "x");
+    same(w, f32, "w");
+    TORCH_CHECK(w.dim() == 2 && x.dim() == 2 && out.dim() == 2 && w.size(1) == x.size(1), "sgemm: K mismatch");
+    is_f32(out, "out");
+    TORCH_CHECK(out.size(1) >= n_feat && w.size(0) >= n_feat + (dual ? dual_offset : 0), "sgemm: shapes");
+    lb::SgemmArgs a{};
+    a.x = x.data_ptr(); a.ldx = x.stride(0); a.w = w.data_ptr(); a.ldw = w.stride(0);
+    a.out = out.data_ptr(); a.ldo = out.stride(0); a.out_f32 = out.scalar_type() == at::kFloat;
+    if (residual.has_value()) {
+      same(*residual, f32, "residual");
+      a.residual = residual->data_ptr(); a.ldr = residual->stride(0);
+    }
+    a.tok_scale = optp<float>(tok_scale); a.out_rows = optp<int>(out_rows);
+    a.T = int(n_tok); a.K = int(x.size(1)); a.N = int(n_feat);
+    a.dual = dual; a.dual_offset = dual_offset; a.act = int(act);
+    a.tile_group = optp<int>(tile_group); a.tile_tok0 = optp<int>(tile_tok0); a.tile_ntok = optp<int>(tile_ntok);
+    a.n_tiles = optp<int>(meta); a.max_tiles = int(max_tiles); a.rows_per_group = rows_per_group;
+    TORCH_CHECK(!a.tile_group || (a.tile_tok0 && a.tile_ntok && a.n_tiles), "sgemm: incomplete tile tables");
+    TORCH_CHECK(a.tile_group || x.size(0) >= n_tok, "sgemm: too few rows");
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::sgemm_launch(a, f32, cur_stream()) == 0, "sgemm failed");
+  });
+  m.def("qkv_norm_append", [](const Tensor& q, const Tensor& k, const Tensor& v, const OptT& qw, const OptT& kw, double eps,
+                              const Tensor& slots, Tensor& q_out, Tensor& k_cache, Tensor& v_cache) {
+    const bool f32 = is_f32(q, "q");
+    same(k, f32, "k");
+    same(v, f32, "v");
+    same(k_cache, f32, "k_cache");
+    same(v_cache, f32, "v_cache");
+    same(q_out, f32, "q_out");
+    const int64_t T = q_out.size(0), Hq = q_out.size(1), DK = q_out.size(2), Hkv = k_cache.size(-2), DV = v_cache.size(-1);
+    TORCH_CHECK(q.size(0) == T && q.size(1) == Hq * DK && k.size(1) == Hkv * DK && v.size(1) == Hkv * DV &&
+                    k_cache.size(-1) == DK && v_cache.size(-2) == Hkv, "qkv_norm_append: shapes");
+    TORCH_CHECK(q.stride(0) == k.stride(0) && q.stride(0) == v.stride(0), "qkv_norm_append: column slices of one projection");
+    TORCH_CHECK(slots.scalar_type() == at::kLong && slots.numel() == T, "qkv_norm_append: slots int64 [T]");
+    TORCH_CHECK(q_out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous(), "qkv_norm_append: contiguous");
+    if (qw.has_value()) f32c(*qw, DK, "q norm");
+    if (kw.has_value()) f32c(*kw, DK, "k norm");
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::qkv_norm_append_launch(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), optp<float>(qw),
+                                           optp<float>(kw), float(eps), reinterpret_cast<const long*>(slots.data_ptr()),
+                                           q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
+                                           int(T), int(Hq), int(Hkv), int(DK), int(DV), f32, cur_stream()) == 0,
+                "qkv_norm_append failed");
+  });
+  m.def("paged_attn_general", [](const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
+                                 const Tensor& ctx_lens, const Tensor& block_table, double scale, int64_t window,
+                                 Tensor& out) {
+    const bool f32 = is_f32(q, "q");
+    same(k_cache, f32, "k_cache");
+    same(v_cache, f32, "v_cache");
+    same(out, f32, "out");
+    const int64_t T = q.size(0), Hq = q.size(1), DK = q.size(2), Hkv = k_cache.size(-2), DV = v_cache.size(-1);
+    TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                    k_cache.size(-1) == DK && out.size(0) == T && out.size(1) == Hq && out.size(2) == DV,
+                "paged_attn_general: shapes");
+    TORCH_CHECK(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_table.scalar_type() == at::kInt &&
+                    cu_q.numel() == ctx_lens.numel() + 1 && block_table.stride(1) == 1, "paged_attn_general: int32 tables");
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::paged_attn_general_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
+                                              cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
+                                              int(block_table.stride(0)), int(k_cache.size(-3)), int(ctx_lens.numel()),
+                                              int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), int(window),
+                                              out.data_ptr(), f32, cur_stream()) == 0,
+                "paged_attn_general: value heads of at most 512 columns, key heads of at most 2560");
+  });
+  m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
+                          const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state, const Tensor& cu,
+                          const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& out, bool write_state) {
+    const auto a = scan_args(q, k, v, silu_in, decay, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, write_state);
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::linear_scan_launch(a, q.scalar_type() == at::kFloat, cur_stream()) == 0,
+                "linear scan: at most 512 state columns, heads a multiple of the groups");
+  });
+  m.def("ssd_decode", [](const Tensor& xbc, const Tensor& conv_w, const OptT& conv_b, Tensor& conv_state, const Tensor& dt,
+                         const Tensor& dt_bias, const Tensor& A, const OptT& D, const OptT& z, Tensor& state,
+                         const Tensor& cu, const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& ctr,
+                         Tensor& out) {
+    const int64_t inner = H * P, n = slots.numel();
+    TORCH_CHECK(xbc.dim() == 2 && xbc.size(0) == n && xbc.size(1) == inner + 2 * G * N, "ssd_decode: x | B | C columns");
+    const Tensor x = xbc.narrow(1, 0, inner), B = xbc.narrow(1, inner, G * N), Cm = xbc.narrow(1, inner + G * N, G * N);
+    lb::SsdDecodeArgs a{};
+    a.s = scan_args(Cm, B, x, false, c10::nullopt, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, true);
+    f32c(conv_w, conv_w.numel(), "conv_w");
+    TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == xbc.size(1), "ssd_decode: conv_w [channels, taps]");
+    a.xbc = xbc.data_ptr(); a.ldx = xbc.stride(0);
+    a.conv_w = conv_w.data_ptr<float>(); a.conv_b = optp<float>(conv_b); a.KC = int(conv_w.size(1));
+    TORCH_CHECK(conv_state.scalar_type() == at::kFloat && conv_state.is_contiguous() && conv_state.dim() == 3 &&
+                    conv_state.size(1) == xbc.size(1) && conv_state.size(2) == a.KC - 1, "ssd_decode: history [slots, C, taps - 1]");
+    a.conv_state = conv_state.data_ptr<float>();
+    TORCH_CHECK(ctr.numel() >= n * G && ctr.element_size() == 4 && ctr.is_contiguous(), "ssd_decode: counters [n, G]");
+    a.ctr = reinterpret_cast<unsigned int*>(ctr.data_ptr());
+    c10::cuda::CUDAGuard guard(xbc.device());
+    TORCH_CHECK(lb::ssd_decode_launch(a, xbc.scalar_type() == at::kFloat, cur_stream()) == 0, "ssd_decode: unsupported sizes");
+  });
+  m.def("linear_chunk_ok", [](int64_t N, int64_t P) { return lb::linear_chunk_ok(int(N), int(P)); });
+  m.def("linear_chunk_scratch_bytes", [](int64_t n_chunks, int64_t H, int64_t N, int64_t P) {
+    return int64_t(lb::linear_chunk_scratch_bytes(int(n_chunks), int(H), int(N), int(P)));
+  });
+  m.def("linear_chunk", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
+                           const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state,
+                           const Tensor& cu, const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& out,
+                           bool write_state, const Tensor& tables, int64_t n_chunks, Tensor& scratch, Tensor& status) {
+    const auto a = scan_args(q, k, v, silu_in, decay, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, write_state);
+    TORCH_CHECK(q.scalar_type() == at::kBFloat16, "linear_chunk: bf16 activations");
+    TORCH_CHECK(tables.scalar_type() == at::kInt && tables.is_contiguous() && tables.numel() >= 3 * n_chunks + 2 * a.n_seqs,
+                "linear_chunk: tables = chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk");
+    TORCH_CHECK(size_t(scratch.numel()) * scratch.element_size() >=
+                    lb::linear_chunk_scratch_bytes(int(n_chunks), int(H), int(N), int(P)), "linear_chunk: scratch too small");
+    const int* tb = tables.data_ptr<int>();
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::linear_chunk_launch(a, tb, tb + n_chunks, tb + 2 * n_chunks, int(n_chunks), tb + 3 * n_chunks,
+                                        tb + 3 * n_chunks + a.n_seqs, scratch.data_ptr(),
+                                        reinterpret_cast<int*>(status.data_ptr()), cur_stream()) == 0,
+                "linear_chunk: unsupported sizes");
+  });
+  m.def("group_norm_gate", [](const Tensor& y, const OptT& gate, const Tensor& w, double eps, int64_t groups, Tensor& out) {
+    const bool f32 = is_f32(y, "y");
+    same(out, f32, "out");
+    const int64_t R = y.size(0), C = y.size(1);
+    TORCH_CHECK(y.dim() == 2 && out.size(0) == R && out.size(1) == C && groups > 0 && C % groups == 0, "group_norm_gate: shapes");
+    f32c(w, C, "norm weight");
+    if (gate.has_value()) {
+      same(*gate, f32, "gate");
+      TORCH_CHECK(gate->size(0) == R && gate->size(1) == C, "group_norm_gate: gate like y");
+    }
+    c10::cuda::CUDAGuard guard(y.device());
+    TORCH_CHECK(lb::group_norm_gate_launch(y.data_ptr(), y.stride(0), gate.has_value() ? gate->data_ptr() : nullptr,
+                                           gate.has_value() ? gate->stride(0) : 0, w.data_ptr<float>(), float(eps),
+                                           int(groups), int(C), int(R), out.data_ptr(), out.stride(0), f32, cur_stream()) == 0,
+                "group_norm_gate failed");
+  });
+  m.def("conv1d_silu", [](const Tensor& x, const Tensor& w, const OptT& bias, Tensor& conv_state, const Tensor& cu_seq,
+                          const Tensor& slots, Tensor& out, bool write_state, int64_t max_len) {
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kFloat, "conv1d_silu dtypes");
+    TORCH_CHECK(lb::conv1d_silu_launch(x.data_ptr(), x.stride(0), w.data_ptr<float>(), optp<float>(bias),
+                                       conv_state.data_ptr<float>(), cu_seq.data_ptr<int>(), slots.data_ptr<int>(),
+                                       int(slots.numel()), int(x.size(1)), int(w.size(1)), out.data_ptr(),
+                                       out.stride(0), write_state ? 1 : 0, cur_stream(), int(max_len)) == 0,
+                "conv1d_silu: unsupported kernel width");
+  });
+  m.def("conv_silu_any", [](const Tensor& x, const Tensor& w, const OptT& bias, Tensor& conv_state, const Tensor& cu,
+                            const Tensor& slots, Tensor& out, bool write_state) {
+    const bool f32 = is_f32(x, "x");
+    same(out, f32, "out");
+    const int64_t T = x.size(0), C = x.size(1), KC = w.size(1);
+    TORCH_CHECK(w.size(0) == C && out.size(0) == T && out.size(1) == C && conv_state.is_contiguous() &&
+                    conv_state.size(1) == C && conv_state.size(2) == KC - 1, "conv_silu_any: shapes");
+    f32c(w, C * KC, "conv weight");
+    if (bias.has_value()) f32c(*bias, C, "conv bias");
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::conv_silu_any_launch(x.data_ptr(), x.stride(0), w.data_ptr<float>(), optp<float>(bias),
+                                         conv_state.data_ptr<float>(), cu.data_ptr<int>(), slots.data_ptr<int>(),
+                                         int(slots.numel()), int(T), int(C), int(KC), out.data_ptr(), out.stride(0),
+                                         write_state, f32, cur_stream()) == 0,
+                "conv_silu_any: at most 65535 tokens per step");
+  });
+}

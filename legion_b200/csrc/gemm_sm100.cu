@@ -115,6 +115,11 @@ __device__ __forceinline__ uint32_t bf16x2_to_f16x2(uint32_t v) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
+__device__ __forceinline__ float gate_act(float v, int act) {
+  if (act == 0) return v / (1.f + __expf(-v));
+  return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+}
+
 template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false>
 __global__ void __launch_bounds__(WFP4 ? 448 : 192, 1)
 wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
@@ -584,7 +589,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
-              if (DUAL) v = (v / (1.f + __expf(-v))) * u[j];
+              if (DUAL) v = gate_act(v, a.act) * u[j];
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -674,7 +679,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               if (t < it.ntok) {
                 const int xrow = it.out0 + t;
                 float v = g[j];
-                if (DUAL) v = (v / (1.f + __expf(-v))) * u[j];
+                if (DUAL) v = gate_act(v, a.act) * u[j];
                 if (a.tok_scale) v *= a.tok_scale[xrow];
                 long orow = xrow;
                 if (a.out_rows) orow = a.out_rows[xrow];
@@ -871,7 +876,7 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
   }
   a.tile_group = h.tile_group; a.tile_tok0 = h.tile_tok0; a.tile_out0 = h.tile_out0; a.tile_ntok = h.tile_ntok; a.n_tiles_dev = h.n_tiles_dev;
   a.n_tok_tiles_max = h.n_tok_tiles_max;
-  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset;
+  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act;
   a.x_group_col = h.x_group_col;
   if (h.x_group_col != 0 && (h.x_group_col % 8 != 0 || h.K % BK != 0 || fp8 || fp4 || !h.tile_group)) {
     snprintf(g_gemm_err, sizeof(g_gemm_err),

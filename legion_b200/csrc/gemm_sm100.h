@@ -60,6 +60,7 @@ struct WgemmArgs {
   int x_group_col;                // grouped mode: first activation column of group g is g * x_group_col (per-head
                                   //   projections read their head's slice of a [tokens, heads * width] tensor in place)
   int dual_offset;                // DUAL: rows from a feature's gate row to its up row
+  int act;                        // DUAL: activation of the gate, 0 = silu, 1 = gelu (tanh form)
   int split_k;
   int vec_ok;                     // output rows may be written as aligned 16-byte vectors
   float* ws;                      // split-K partials
@@ -85,7 +86,7 @@ struct WgemmHost {
   const float* tok_scale;
   const int* out_rows;
   int K, n_feat, n_tok;
-  int bn; bool dual;
+  int bn; bool dual; int act;
   const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles_dev;
   const int* tile_out0;
   int n_tok_tiles_max;

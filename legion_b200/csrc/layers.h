@@ -1,0 +1,100 @@
+// Launch interface of the layer kernels that work on bf16 and on fp32 activations (hyper.cu, sgemm.cu, attn_general.cu,
+// linear_scan.cu, linear_scan_sm100.cu). Pointers are device pointers; f32 selects the activation type of the `void*`
+// operands. Every function returns 0 on success and enqueues without synchronising.
+#pragma once
+#include <cuda_runtime.h>
+#include <stddef.h>
+
+namespace lb {
+
+// Hyper-connections with static weights (hyper.cu). X [rows, S, H] fp32.
+struct HyperArgs {
+  const float* x_in;               // streams before the sublayer; nullptr: every stream starts as the embedding row
+  float* x_out;                    // streams after it (may be x_in)
+  const void* emb; const int* ids; // start: embedding table and token ids (ids == nullptr: row t of emb)
+  long ld_emb; int vocab;
+  const void* y0; long ldy0; float c0;   // sublayer output: c0 * (sum of y_rows consecutive rows of y0) + c1 * y1
+  const void* y1; long ldy1; float c1;
+  int y_rows;
+  const float* mix;                // [S from, S to]
+  const float* out_w;              // [S]
+  const float* in_w;               // [S] weights of the next sublayer's input (nullptr: all ones)
+  const float* norm_w; float eps, w_offset;
+  void* h; long ldh;               // norm of the next input, activation type
+  int rows, S, H;
+};
+int hyper_launch(const HyperArgs& a, bool f32, cudaStream_t s);
+
+// Plain FMA GEMM (sgemm.cu): out[t, n] = sum_k x[t, k] w[n, k] in fp32, any sizes and pitches. Token tiles of
+// SGEMM_BN rows; the grouped form takes the tile tables of the tcgen05 GEMM.
+constexpr int SGEMM_BN = 32;
+struct SgemmArgs {
+  const void* x; long ldx;
+  const void* w; long ldw;
+  void* out; long ldo; int out_f32;
+  const void* residual; long ldr;  // activation type
+  const float* tok_scale;          // per activation row (grouped) multiplier
+  const int* out_rows;             // activation row -> output row (negative: drop)
+  int T, K, N;
+  int dual; long dual_offset; int act;   // act(gate) * up, rows dual_offset apart; act 0 silu, 1 gelu (tanh), 2 relu^2 (no up)
+  const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles; int max_tiles;
+  long rows_per_group;
+};
+int sgemm_launch(const SgemmArgs& a, bool f32, cudaStream_t s);
+
+// q / k head norms (optional) and the append of k and v to the paged cache, any head sizes (attn_general.cu)
+int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld, const float* qw, const float* kw,
+                           float eps, const long* slots, void* q_out, void* k_cache, void* v_cache, long k_cell,
+                           long v_cell, int T, int Hq, int Hkv, int DK, int DV, bool f32, cudaStream_t s);
+// Paged causal attention on FMA units, one warp per (token, query head); value heads up to 512 wide
+int paged_attn_general_launch(const void* q, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
+                              const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
+                              int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, int window, void* out,
+                              bool f32, cudaStream_t s);
+
+// Decayed outer-product state S_t = a_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (linear_scan.cu, linear_scan_sm100.cu).
+struct LinScanArgs {
+  const void* q; long ldq;         // [T, G, N]
+  const void* k; long ldk;
+  const void* v; long ldv;         // [T, H, P]
+  int silu_in;                     // q, k and v pass silu first
+  const float* decay;              // [H] constant decay per head, or nullptr: the selective form below
+  const void* dt; long lddt;       // [T, H] raw step sizes: dt = softplus(raw + dt_bias), a = exp(dt * A), v is scaled by dt
+  const float* dt_bias; const float* A;
+  const float* D;                  // [H] skip: o += D v (unscaled v); nullptr: none
+  const void* z; long ldz;         // [T, H, P] gate: o *= silu(z); nullptr: none
+  float* state;                    // [slots, H, P, N] fp32
+  const int* cu; const int* slots;
+  int n_seqs, T, H, G, N, P;
+  void* out; long ldo;
+  int write_state;
+};
+int linear_scan_launch(const LinScanArgs& a, bool f32, cudaStream_t s);
+
+// Chunked form on tcgen05 (bf16): host-side tables of 128-token chunks. chunk_t0 / chunk_n: first token row and valid
+// tokens; seq_chunk0 / seq_nchunk: chunk range of each sequence. scratch: linear_chunk_scratch_bytes, 256-byte aligned.
+bool linear_chunk_ok(int N, int P);
+size_t linear_chunk_scratch_bytes(int n_chunks, int H, int N, int P);
+int linear_chunk_launch(const LinScanArgs& a, const int* chunk_t0, const int* chunk_n, const int* chunk_seq,
+                        int n_chunks, const int* seq_chunk0, const int* seq_nchunk, void* scratch, int* status,
+                        cudaStream_t s);
+
+// One decode step of a Mamba-2 mixer: convolution with history update, step size, state update, skip and gate.
+struct SsdDecodeArgs {
+  const void* xbc; long ldx;       // [n, H * P + 2 * G * N] input projection columns x | B | C
+  const float* conv_w; const float* conv_b; float* conv_state; int KC;
+  LinScanArgs s;                   // q / k / v unused
+  unsigned int* ctr;               // [n, G] zeroed arrival counters, left zero
+};
+int ssd_decode_launch(const SsdDecodeArgs& a, bool f32, cudaStream_t s);
+
+// y normed in `groups` equal parts, times w, times sigmoid(gate) when a gate is given
+int group_norm_gate_launch(const void* y, long ldy, const void* gate, long ldg, const float* w, float eps, int groups,
+                           int C, int rows, void* out, long ldo, bool f32, cudaStream_t s);
+
+// Causal depth-wise convolution + silu with carried history, any number of taps
+int conv_silu_any_launch(const void* x, long ldx, const float* w, const float* bias, float* conv_state,
+                         const int* cu_seq, const int* slots, int n_seqs, int T, int C, int KC, void* out, long ldo,
+                         int write_state, bool f32, cudaStream_t s);
+
+}  // namespace lb

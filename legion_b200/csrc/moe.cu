@@ -14,13 +14,13 @@ namespace lb {
 
 // One warp per token. mode 0: softmax over all experts -> top-k -> renormalise (optional).
 // mode 1: sigmoid scores, selection by score + bias, optional group-limited routing (n_group groups,
-// keep topk_group groups ranked by the sum of their two best biased scores), weights = unbiased
-// scores of the chosen experts, renormalised and multiplied by route_scale.
+// keep topk_group groups ranked by the sum of their group_top (1 or 2) best biased scores), weights = unbiased
+// scores of the chosen experts, renormalised and multiplied by route_scale. mode 2: as mode 1 with softmax scores.
 template <int MAXE>
 __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, const float* __restrict__ bias, int E,
                                                 int k, int mode, int renorm, float route_scale, int n_group,
-                                                int topk_group, int* __restrict__ ids, float* __restrict__ wts,
-                                                int t, int* sm_ids = nullptr, float* sm_wts = nullptr) {
+                                                int topk_group, int group_top, int* __restrict__ ids,
+                                                float* __restrict__ wts, int t, int* sm_ids = nullptr, float* sm_wts = nullptr) {
   constexpr int PER = MAXE / 32;
   const int lane = threadIdx.x & 31;
   float sc[PER], sel[PER];
@@ -32,27 +32,27 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
     mx = fmaxf(mx, sc[j]);
   }
   float inv_sum = 1.f;
+  if (mode == 2 || (mode == 0 && !renorm)) {      // the partition sum of the softmax
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) sum += (lane + 32 * j < E) ? __expf(sc[j] - mx) : 0.f;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    inv_sum = 1.f / sum;
+  }
   if (mode == 0) {
     // selection by the logits themselves (softmax is monotonic); the partition sum is needed only when the chosen
     // weights are not renormalised
 #pragma unroll
     for (int j = 0; j < PER; ++j) sel[j] = sc[j];
-    if (!renorm) {
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      float sum = 0.f;
-#pragma unroll
-      for (int j = 0; j < PER; ++j) sum += (lane + 32 * j < E) ? __expf(sc[j] - mx) : 0.f;
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      inv_sum = 1.f / sum;
-    }
   } else {
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
       const int e = lane + 32 * j;
       if (e < E) {
-        sc[j] = 1.f / (1.f + __expf(-sc[j]));
+        sc[j] = mode == 2 ? __expf(sc[j] - mx) * inv_sum : 1.f / (1.f + __expf(-sc[j]));
         sel[j] = sc[j] + (bias ? bias[e] : 0.f);
       } else {
         sc[j] = 0.f;
@@ -60,7 +60,7 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
       }
     }
     if (n_group > 1 && topk_group < n_group) {
-      // group score = sum of the two best biased scores in the group; groups are contiguous ranges.
+      // group score = sum of the group_top best biased scores in the group; groups are contiguous ranges.
       const int gs = E / n_group;
       float keep_thresh_rank[1];
       (void)keep_thresh_rank;
@@ -85,7 +85,7 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
           const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
           b1 = n1; b2 = n2;
         }
-        if (lane == g) my_gscore = b1 + (b2 == -INFINITY ? 0.f : b2);
+        if (lane == g) my_gscore = b1 + (b2 == -INFINITY || group_top < 2 ? 0.f : b2);
       }
       // rank of each group = number of groups with a better score (ties: lower index wins)
       int rank = 0;
@@ -148,6 +148,7 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
   if (lane < k) {
     const float l = __ldcg(logits + t * ldl + my_id);
     if (mode == 0) w = renorm ? l : __expf(l - mx) * inv_sum;
+    else if (mode == 2) w = __expf(l - mx) * inv_sum;
     else w = 1.f / (1.f + __expf(-l));
   }
   if (mode == 0 && renorm) {
@@ -173,10 +174,11 @@ template <int MAXE>
 __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, long ldl,
                                                           const float* __restrict__ bias, int E, int k, int mode,
                                                           int renorm, float route_scale, int n_group, int topk_group,
-                                                          int* __restrict__ ids, float* __restrict__ wts, int T) {
+                                                          int group_top, int* __restrict__ ids,
+                                                          float* __restrict__ wts, int T) {
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   if (t >= T) return;
-  router_topk_row<MAXE>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group, topk_group, ids, wts, t);
+  router_topk_row<MAXE>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group, topk_group, group_top, ids, wts, t);
 }
 
 // Decode-sized MoE front end in ONE launch (T <= 64 tokens, T * k <= 1024 pairs):
@@ -201,7 +203,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
     const __nv_bfloat16* __restrict__ x, long ldx, const float* __restrict__ norm_w, float eps, float w_offset,
     __nv_bfloat16* __restrict__ x_normed, long ldn, const __nv_bfloat16* __restrict__ w, long ldw, int H,
     float* logits, const float* __restrict__ bias, int E, int k, int mode, int renorm, float route_scale, int n_group,
-    int topk_group, int* ids, float* wts, int T, int bn, int* __restrict__ tile_group, int* __restrict__ slot_base,
+    int topk_group, int group_top, int* ids, float* wts, int T, int bn, int* __restrict__ tile_group, int* __restrict__ slot_base,
     int* __restrict__ tile_ntok, int* __restrict__ meta, int* __restrict__ out_rows, float* __restrict__ tok_scale,
     unsigned int* done_ctr, int e_lo, int n_local, const __nv_bfloat16* __restrict__ sh_gate_w, float* sh_logit,
     int shared_slot, int epc, int tpp, int ksplit, int* status, int* __restrict__ active) {
@@ -369,39 +371,10 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
       l = __ldcg(logits + long(t) * E + e);
       for (int sp = 1; sp < ksplit; ++sp) l += __ldcg(logits + long(sp) * ROUTE_LSTR + long(t) * E + e);
     }
-    float selv = l;
-    if (mode == 1) selv = 1.f / (1.f + __expf(-l)) + (bias && e < E ? bias[e] : 0.f);
     s_logit[e] = l;
-    if (mode == 1 && n_group > 1 && topk_group < n_group) {
-      // group-limited routing: lane g of warp 0 scores group g (the sum of its two best biased scores), the groups
-      // are ranked (ties: lower index first) and the experts of the groups that are not kept drop out
-      const int gs = E / n_group;
-      s_sel[e] = selv;
-      __syncthreads();
-      if (warp == 0) {
-        float gscore = -INFINITY;
-        if (lane < n_group) {
-          float b1 = -INFINITY, b2 = -INFINITY;
-          for (int i = 0; i < gs; ++i) {
-            const float v = s_sel[lane * gs + i];
-            if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
-          }
-          gscore = b1 + (b2 == -INFINITY ? 0.f : b2);
-        }
-        int rank = 0;
-        for (int g = 0; g < n_group; ++g) {
-          const float og = __shfl_sync(0xffffffffu, gscore, g);
-          if (lane < n_group && (og > gscore || (og == gscore && g < lane))) ++rank;
-        }
-        const unsigned keep = __ballot_sync(0xffffffffu, lane < n_group && rank < topk_group);
-        if (lane == 0) s_keep = keep;
-      }
-      __syncthreads();
-      if (e < E && !((s_keep >> (e / gs)) & 1u)) selv = -INFINITY;
-    }
     float mxv = 0.f, inv_sum = 1.f;
-    if (mode == 0 && !renorm) {
-      // softmax weights without renormalisation need the partition sum over all experts
+    if (mode == 2 || (mode == 0 && !renorm)) {
+      // softmax scores need the partition sum over all experts (renormalised weights of mode 0 do not)
       float m = l;
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
@@ -418,6 +391,36 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
       float tot = 0.f;
       for (int i = 0; i < 16; ++i) tot += s_red[i];
       inv_sum = 1.f / tot;
+    }
+    float selv = l;
+    if (mode == 1) selv = 1.f / (1.f + __expf(-l)) + (bias && e < E ? bias[e] : 0.f);
+    else if (mode == 2) selv = __expf(l - mxv) * inv_sum + (bias && e < E ? bias[e] : 0.f);
+    if (mode != 0 && n_group > 1 && topk_group < n_group) {
+      // group-limited routing: lane g of warp 0 scores group g (the sum of its group_top best biased scores), the groups
+      // are ranked (ties: lower index first) and the experts of the groups that are not kept drop out
+      const int gs = E / n_group;
+      s_sel[e] = selv;
+      __syncthreads();
+      if (warp == 0) {
+        float gscore = -INFINITY;
+        if (lane < n_group) {
+          float b1 = -INFINITY, b2 = -INFINITY;
+          for (int i = 0; i < gs; ++i) {
+            const float v = s_sel[lane * gs + i];
+            if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
+          }
+          gscore = b1 + (b2 == -INFINITY || group_top < 2 ? 0.f : b2);
+        }
+        int rank = 0;
+        for (int g = 0; g < n_group; ++g) {
+          const float og = __shfl_sync(0xffffffffu, gscore, g);
+          if (lane < n_group && (og > gscore || (og == gscore && g < lane))) ++rank;
+        }
+        const unsigned keep = __ballot_sync(0xffffffffu, lane < n_group && rank < topk_group);
+        if (lane == 0) s_keep = keep;
+      }
+      __syncthreads();
+      if (e < E && !((s_keep >> (e / gs)) & 1u)) selv = -INFINITY;
     }
     const uint32_t u = __float_as_uint(selv);
     const uint32_t ord = (u & 0x80000000u) ? ~u : (u | 0x80000000u);
@@ -451,6 +454,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
       if (lane < k) {
         const float lg = s_logit[my_id];
         if (mode == 0) w = renorm ? lg : __expf(lg - mxv) * inv_sum;
+        else if (mode == 2) w = __expf(lg - mxv) * inv_sum;
         else w = 1.f / (1.f + __expf(-lg));
       }
       if (mode == 0 && renorm) {
@@ -544,8 +548,8 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
 
 int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float eps, float w_offset, void* x_normed,
                            long ldn, const void* w, long ldw, int H, float* logits, const float* bias, int E, int k,
-                           int mode, int renorm, float route_scale, int n_group, int topk_group, int* ids, float* wts,
-                           int T, int bn, int* tile_group, int* slot_base, int* tile_ntok, int* meta, int* out_rows,
+                           int mode, int renorm, float route_scale, int n_group, int topk_group, int group_top,
+                           int* ids, float* wts, int T, int bn, int* tile_group, int* slot_base, int* tile_ntok, int* meta, int* out_rows,
                            float* tok_scale, unsigned int* done_ctr, int e_lo, int n_local, const void* sh_gate_w,
                            float* sh_logit, int shared_slot, int* status, int* active, cudaStream_t s) {
   if (T <= 0) return 0;
@@ -574,7 +578,7 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
       smem_set = smem;                                                                                              \
     }                                                                                                               \
     launch_pdl(moe_route_small_kernel<MAXE>, dim3(grid), dim3(512), smem, s, xb, ldx, norm_w, eps, w_offset, xn,   \
-               ldn, wb, ldw, H, logits, bias, E, k, mode, renorm, route_scale, n_group, topk_group, ids, wts, T,    \
+               ldn, wb, ldw, H, logits, bias, E, k, mode, renorm, route_scale, n_group, topk_group, group_top, ids, wts, T, \
                bn, tile_group, slot_base, tile_ntok, meta, out_rows, tok_scale, done_ctr, e_lo, n_local, sg,        \
                sh_logit, shared_slot, epc, tpp, ksplit, status, active);                                                    \
   }
@@ -586,19 +590,20 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
 }
 
 int router_topk_launch(const float* logits, long ldl, const float* bias, int E, int k, int mode, int renorm,
-                       float route_scale, int n_group, int topk_group, int* ids, float* wts, int T, cudaStream_t s) {
+                       float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts, int T,
+                       cudaStream_t s) {
   if (T <= 0) return 0;
   if (k > 32 || E > 512 || n_group > 32) return 1;
   const int blocks = (T * 32 + 127) / 128;
   if (E <= 128)
     router_topk_kernel<128><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, T);
   else if (E <= 256)
     router_topk_kernel<256><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, T);
   else
     router_topk_kernel<512><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, T);
   return cudaGetLastError() != cudaSuccess;
 }
 

@@ -184,11 +184,13 @@ class DecodeGraphs:
         o, n = off["block_table"]
         h[o + n_real * e.W:o + n] = 0
 
-    def run(self, rows, B: Optional[int] = None, gather=None) -> Tuple[Optional[List[int]], Optional[torch.Tensor]]:
+    def run(self, rows, B: Optional[int] = None, gather=None,
+            logits: bool = False) -> Tuple[Optional[List[int]], Optional[torch.Tensor]]:
         """rows: [(seq, position, 1)]. Returns (picked token per row, logits [n, V]) or (None, None) when the
         batch does not fit a bucket. ``B`` forces the bucket (data-parallel attention: every rank replays the
         bucket of the fullest rank, possibly with no row of its own) and ``gather=(group, world)`` makes the
-        result the picks of ALL ranks, ``world * B`` values in rank order."""
+        result the picks of ALL ranks, ``world * B`` values in rank order. ``logits``: return the logits even when
+        every row is plain greedy (else they are handed out only where sampling needs them)."""
         n = len(rows)
         B = B or self.bucket(n)
         if B is None:
@@ -209,7 +211,7 @@ class DecodeGraphs:
                 for i, (s, p0, _) in enumerate(rows):
                     if s.media is not None:
                         ps[i] = s.rope_pos(p0)
-            return self._replay(e, rows, n, B, gather)
+            return self._replay(e, rows, n, B, gather, logits)
         off, _ = self._layout(B, e.W)
         h = e.pack_h
         sl = h[off["slots"][0]:off["slots"][0] + 2 * B].view(torch.int64)
@@ -238,9 +240,9 @@ class DecodeGraphs:
         for i in range(n, B):
             e.bt_key[i] = None
         self._fill_padding(e, n)
-        return self._replay(e, rows, n, B, gather)
+        return self._replay(e, rows, n, B, gather, logits)
 
-    def _replay(self, e: _Entry, rows, n: int, B: int, gather=None):
+    def _replay(self, e: _Entry, rows, n: int, B: int, gather=None, logits: bool = False):
         eng = self.eng
         e.pack_d.copy_(e.pack_h, non_blocking=True)
         e.graph.replay()
@@ -262,8 +264,8 @@ class DecodeGraphs:
         self.h2d_bytes += e.n_ints * 4
         self.d2h_bytes += B * 4
         self.replays += 1
-        need_logits = any(not (s.req.sampling.greedy and s.req.sampling.plain and s.constraint is None)
-                          for s, _, _ in rows)
+        need_logits = logits or any(not (s.req.sampling.greedy and s.req.sampling.plain and s.constraint is None)
+                                    for s, _, _ in rows)
         if need_logits and e.logits is None and e.logits_local is not None:
             return e.picks_h[:n].tolist(), eng.model.gather_logits(e.logits_local)[:n]
         return e.picks_h[:n].tolist(), (e.logits[:n] if need_logits else None)

@@ -216,9 +216,9 @@ class LmEngine(Engine):
         self._stop = threading.Event()
         self._thread: Optional[threading.Thread] = None
         self._fail: Optional[str] = None
-        if ("kda" in self.mcfg.layer_kinds) and (drafter is not None or c.spec != "none"):
-            raise ValueError("speculative decoding is not available for models with Kimi-delta-attention layers "
-                             "(their verify steps have no state replay)")
+        if ("kda" in self.mcfg.layer_kinds or self.mcfg.layers is not None) and (drafter is not None or c.spec != "none"):
+            raise ValueError("speculative decoding is not available for models with Kimi-delta-attention layers or "
+                             "layer specifications (their verify steps have no state replay)")
         self._depth_model = None          # spec.depth.DepthModel under the adaptive draft-depth policy
         self._draft_ms_step = 0.0
         self.vision = None                # vision.VisionRuntime once a tower is attached (``attach_vision``)
@@ -299,6 +299,8 @@ class LmEngine(Engine):
         """Mamba-2 layers decode from CUDA graphs when their head shape runs on the scan kernel (the token loop that
         serves other shapes reads sequence bounds on the host)."""
         m = self.mcfg
+        if m.layers is not None:
+            return True           # every kernel of these layers reads lengths and slots on the device
         if "kda" in m.layer_kinds or m.hyper_streams > 1 or m.sandwich_norm or m.block_form:
             return False          # forward paths built from tensor operations (no captured decode step)
         if "mamba2" not in m.layer_kinds:
@@ -1078,9 +1080,10 @@ class LmEngine(Engine):
         b.slots_ring = torch.tensor(cells, dtype=torch.int64, device=self.device)
         b.block_table_ring = table.to(self.device)
 
-    def build_batch_explicit(self, items, all_logits: bool = False) -> StepBatch:
+    def build_batch_explicit(self, items, all_logits: bool = False, logit_rows: Optional[List[int]] = None) -> StepBatch:
         """items = [(seq, first position, token list)]: a batch over the sequences' own block tables with
-        explicit tokens (drafters fill their KV and chain drafts with it). Logits: last row of each item."""
+        explicit tokens (drafters fill their KV and chain drafts with it). Logits: last row of each item, or the
+        given rows of the batch."""
         dev = self.device
         tok, pos, slots, cu, ctx, lrows = [], [], [], [0], [], []
         width = 1
@@ -1102,11 +1105,61 @@ class LmEngine(Engine):
                       cu_q=torch.tensor(cu, **i32), ctx_lens=torch.tensor(ctx, **i32), block_table=bt.to(dev),
                       slots=torch.tensor(slots, dtype=torch.int64, device=dev),
                       state_slots=torch.tensor([s.slot for s, _, _ in items], **i32),
-                      logit_rows=torch.tensor(lrows, dtype=torch.int64, device=dev),
+                      logit_rows=torch.tensor(lrows if logit_rows is None else logit_rows, dtype=torch.int64, device=dev),
                       max_q_len=max(len(t) for _, _, t in items), max_ctx=max(ctx), cu_q_host=cu)
         if self.ring_len:
             self._ring_inputs(b, [(s, p0, len(toks)) for s, p0, toks in items], width)
         return b
+
+    # ------------------------------------------------------------------ steps planned by the caller
+    def open_sequence(self, name: str) -> Seq:
+        """Admits a sequence whose tokens the caller feeds step by step (``feed``): a cleared state slot and an empty
+        block table. For engines whose own scheduler thread is not running."""
+        if not self._free_slots:
+            raise EngineOverloaded("no free state slot")
+        s = Seq(GenerateRequest(prompt_tokens=[], sampling=SamplingParams(temperature=0.0), request_id=name),
+                TokenStream(CancelToken()), [])
+        s.slot = self._free_slots.pop()
+        if self.states is not None:
+            self.states.clear(s.slot)
+        self.running.append(s)
+        return s
+
+    def feed(self, items: Sequence[Tuple[Seq, List[int], List[int]]]) -> Optional[torch.Tensor]:
+        """One step over ``items`` = [(sequence, its next tokens, places among them whose logits are wanted)], all in
+        one batch from the caches and states that earlier steps left. Single tokens that continue a sequence replay
+        the decode graph the generation path uses. Returns logits [wanted, vocab] in the order of the items."""
+        if any(s.slot < 0 or not toks for s, toks, _ in items):
+            raise ValueError("feed: every item needs an open sequence and at least one token")
+        for s, toks, _ in items:
+            s.tokens.extend(toks)
+            s.table.ensure(self.pool, len(s.tokens))
+            s.phase = "decode" if len(toks) == 1 and s.n_computed else "prefill"
+        rows = [(s, s.n_computed, len(toks)) for s, toks, _ in items]
+        want, base = [], 0
+        for _, toks, places in items:
+            want.extend(base + p for p in places)
+            base += len(toks)
+        logits = None
+        done = False
+        if self._graphs is not None and all(s.phase == "decode" for s, _, _ in rows):
+            picks, logits = self._graphs.run(rows, logits=True)
+            done = picks is not None
+            if done:
+                logits = logits[torch.tensor(want, dtype=torch.int64, device=self.device)] if want else None
+        if not done:
+            b = self.build_batch_explicit([(s, p0, toks) for (s, p0, _), (_, toks, _) in zip(rows, items)], logit_rows=want)
+            logits = self.model.forward(b, self.kv, self.states, want_logits=bool(want)).logits
+        for s, p0, n in rows:
+            s.n_computed = s.table.n_tokens = p0 + n
+        self._stats.steps += 1
+        return logits
+
+    def close_sequence(self, s: Seq) -> None:
+        """Gives back the blocks and the state slot of a fed sequence."""
+        s.finished = True
+        self.running.remove(s)
+        self._release(s)
 
     def _own_blocks(self, s: Seq):
         """Data-parallel attention: blocks that enter the prefix cache remember which rank holds their contents."""

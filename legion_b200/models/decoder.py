@@ -14,6 +14,8 @@ Blocks (reference structure in parentheses):
               gated RMS norm -> out-proj (``src/model/core.rs:3484-3984``)
   mla         Multi-head latent attention over a cached [latent | rope-key] row per token
   mamba2      Mamba-2 selective state space layer (``src/model/nemotron_h.rs``)
+  lightning   linear attention with a constant decay per head (stacks with layer specifications)
+  parallel    two mixers over the same input, here windowed attention beside a Mamba-2 mixer
   moe         router -> top-k -> routed experts (+ shared expert, + sigmoid shared gate)
               (``src/model/core.rs:4496-4640``); dense SwiGLU / GELU / ReLU^2 FFN
   mtp         next-token-prediction head: eh_proj([norm(embed) ; norm(hidden)]) -> one block -> shared
@@ -88,7 +90,11 @@ class KvCache:
             layers.append(cfg.n_layer + j)
             kinds[cfg.n_layer + j] = "mla" if cfg.kv_lora > 0 else "attn"
         for il in layers:
-            if kinds[il] == "mla":
+            if cfg.layers is not None:
+                hk, dk, dv = cfg.kv_dims(il)
+                self.k[il] = torch.zeros(n_blocks, page, hk, dk, device=device, dtype=dtype)
+                self.v[il] = torch.zeros(n_blocks, page, hk, dv, device=device, dtype=dtype)
+            elif kinds[il] == "mla":
                 self.k[il] = torch.zeros(n_blocks, page, 1, cfg.kv_lora + cfg.qk_rope_dim, device=device, dtype=dtype)
                 self.v[il] = self.k[il]
             elif cfg.sandwich_norm and il < cfg.n_layer:
@@ -149,7 +155,15 @@ class StatePool:
             if owns is not None and not owns(il):
                 continue
             kind = cfg.layer_kinds[il]
-            if kind == "gdn":
+            if cfg.layers is not None:
+                r = cfg.recurrent_spec(il)
+                N = r.dim if r.kind == "lightning" else r.state
+                # state[head, value column, key column]
+                self.ssm[il] = torch.zeros(n_slots, r.heads, r.vdim, N, device=device, dtype=torch.float32)
+                if r.kind == "ssd":
+                    self.conv[il] = torch.zeros(n_slots, r.heads * r.vdim + 2 * r.groups * N, r.conv - 1, device=device,
+                                                dtype=torch.float32)
+            elif kind == "gdn":
                 C = cfg.gdn_conv_channels() // tp
                 self.conv[il] = torch.zeros(n_slots, C, cfg.gdn_conv - 1, device=device, dtype=torch.float32)
                 self.ssm[il] = torch.zeros(n_slots, cfg.gdn_v_heads // tp, cfg.gdn_k_dim, cfg.gdn_v_dim, device=device,
@@ -314,7 +328,7 @@ class Decoder:
     def __init__(self, cfg: ModelConfig, weights: Dict[str, torch.Tensor], pctx: Optional[ParallelCtx] = None,
                  max_position: Optional[int] = None, pipe=None):
         self.cfg = cfg
-        if cfg.hyper_streams > 1 and pipe is not None:
+        if (cfg.hyper_streams > 1 or cfg.layers is not None) and pipe is not None:
             raise NotImplementedError("hyper-connection models run without pipeline stages")
         self.w = weights
         self.pctx = pctx or ParallelCtx.single()
@@ -332,6 +346,10 @@ class Decoder:
             # sliding-window layers rotate their (own-sized) heads whole with a base of their own
             self.cos_sin_swa = ops.reference.rope_cos_sin(mp, cfg.swa_head_dim or cfg.head_dim,
                                                           cfg.rope_theta_swa or cfg.rope_theta, None, device=dev)
+        self._decay: Dict[int, torch.Tensor] = {}     # linear-attention layers: decay per head
+        for il in range(cfg.n_layer if cfg.layers is not None else 0):
+            if cfg.layers[il].mixer.kind == "lightning":
+                self._decay[il] = torch.tensor(cfg.layers[il].mixer.decay, dtype=torch.float32, device=dev)
         tp = self.pctx.tp
         self.n_head_l = cfg.n_head // tp
         self.n_kv_l = max(1, cfg.n_kv_head // tp)
@@ -916,6 +934,100 @@ class Decoder:
         pc.end_step()
         return out
 
+    # ------------------------------------------------------------------ stacks with layer specifications
+    def _softmax_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache):
+        """Attention part of a layer; ``proj`` starts with its q | k | v columns. Returns (output, columns used)."""
+        cfg, w, a = self.cfg, self.w, self.cfg.attn_spec(il)
+        nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        q = ops.qkv_norm_append(proj[:, :nq], proj[:, nq:nq + nk], proj[:, nq + nk:nq + nk + nv],
+                                w.get(f"{p}.attn.q_norm"), w.get(f"{p}.attn.k_norm"), cfg.rms_eps, b.slots, kv.k[il],
+                                kv.v[il])
+        o = ops.paged_attention(q, kv.k[il], kv.v[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, a.scale,
+                                window=a.window, max_ctx=b.max_ctx or None)
+        return ops.linear(o.reshape(o.shape[0], -1), w[f"{p}.attn.o"]), nq + nk + nv
+
+    def _ssd_mixer(self, p: str, il: int, proj, b: StepBatch, st: StatePool):
+        """Mamba-2 part of a layer; ``proj`` holds its z | x | B | C | dt columns. Decode steps run convolution, state
+        and gate as one launch."""
+        cfg, w, r = self.cfg, self.w, self.cfg.recurrent_spec(il)
+        H, P, N, G = r.heads, r.vdim, r.state, r.groups
+        inner, conv_c = H * P, H * P + 2 * G * N
+        z, xbc, dt = proj[:, :inner], proj[:, inner:inner + conv_c], proj[:, inner + conv_c:inner + conv_c + H]
+        A, D, db = w[f"{p}.ssm.A"], w[f"{p}.ssm.D"], w[f"{p}.ssm.dt_bias"]
+        if proj.is_cuda and b.max_q_len == 1 and b.write_state and proj.shape[0] == b.n_seqs:
+            y = ops.sm100.ssd_decode(xbc, w[f"{p}.ssm.conv_w"], w[f"{p}.ssm.conv_b"], st.conv[il], dt, db, A, D, z,
+                                     st.ssm[il], b.cu_q, b.state_slots, H, G, N, P)
+        else:
+            c = ops.causal_conv1d_silu(xbc, w[f"{p}.ssm.conv_w"], w[f"{p}.ssm.conv_b"], st.conv[il], b.cu_q,
+                                       b.state_slots, write_state=b.write_state, max_len=b.max_q_len)
+            y = ops.linear_scan(c[:, inner + G * N:], c[:, inner:inner + G * N], c[:, :inner], st.ssm[il], b.cu_q,
+                                b.state_slots, H, G, N, P, dt=dt, dt_bias=db, A=A, D=D, z=z,
+                                write_state=b.write_state, max_len=b.max_q_len, cu_host=b.cu_q_host)
+        n = ops.group_norm_gate(y, None, w[f"{p}.ssm.norm"], cfg.rms_eps, r.norm_groups)
+        return ops.linear(n, w[f"{p}.ssm.out"])
+
+    def _lightning_mixer(self, p: str, il: int, h, b: StepBatch, st: StatePool):
+        cfg, w, m = self.cfg, self.w, self.cfg.layers[il].mixer
+        nk, nv = m.heads * m.dim, m.heads * m.vdim
+        proj = ops.linear(h, w[f"{p}.lin.qkvg"])
+        o = ops.linear_scan(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:2 * nk + nv], st.ssm[il], b.cu_q,
+                            b.state_slots, m.heads, m.heads, m.dim, m.vdim, decay=self._decay[il], silu_in=True,
+                            write_state=b.write_state, max_len=b.max_q_len, cu_host=b.cu_q_host)
+        n = ops.group_norm_gate(o, proj[:, 2 * nk + nv:], w[f"{p}.lin.norm"], cfg.rms_eps)
+        return ops.linear(n, w[f"{p}.lin.out"])
+
+    def _spec_mixer(self, p: str, il: int, h, b: StepBatch, kv: KvCache, st: StatePool):
+        """Output of layer il's mixer as [(tensor, scale)]: the terms are summed by the stream update that follows."""
+        m = self.cfg.layers[il].mixer
+        if m.kind == "lightning":
+            return [(self._lightning_mixer(p, il, h, b, st), 1.0)]
+        proj = ops.linear(h, self.w[f"{p}.mix.in"])
+        if m.kind == "ssd":
+            return [(self._ssd_mixer(p, il, proj, b, st), 1.0)]
+        left, used = self._softmax_mixer(p, il, proj, b, kv)
+        if m.kind == "attn":
+            return [(left, 1.0)]
+        return [(left, m.left_scale), (self._ssd_mixer(p, il, proj[:, used:], b, st), m.right_scale)]
+
+    def _spec_ffn(self, p: str, il: int, h):
+        w, f = self.w, self.cfg.layers[il].mlp
+        if f.kind == "dense":
+            return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act), w[f"{p}.mlp.down"]), 1.0)]
+        routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, 1.0, w.get(f"{p}.moe.router_bias"),
+                             f.n_group, f.keep_group, group_top=f.group_top)
+        ids, wts = routing
+        return [(ops.moe_experts(h, ids, wts, w[f"{p}.moe.gate_up"], w[f"{p}.moe.down"], f.ff, f.act, routing=routing,
+                                 defer_combine="pairs"), 1.0)]
+
+    def _forward_streams(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool) -> StepOutput:
+        """Forward pass of a stack with layer specifications and static hyper-connections: fp32 streams, and per
+        sublayer one launch that folds its output into them, mixes the next sublayer's input and applies its norm."""
+        cfg, w = self.cfg, self.w
+        eps, off = cfg.rms_eps, cfg.norm_offset
+        subs = []                                     # (layer, hyper-connection prefix, norm, is mixer)
+        for il, spec in enumerate(cfg.layers):
+            subs.append((il, f"l{il}.hca", f"l{il}.attn_norm", True))
+            if spec.mlp is not None:
+                subs.append((il, f"l{il}.hcf", f"l{il}.ffn_norm", False))
+        table, ids = (w["tok_embd"], b.token_ids) if b.embeds is None else (b.embeds, None)
+        X, h = ops.hyper_start(table, ids, cfg.hyper_streams, w[f"{subs[0][1]}.st_in"], w[subs[0][2]], eps, off)
+        captures: Dict[int, torch.Tensor] = {}
+        for i, (il, hc, _, mixer) in enumerate(subs):
+            p = f"l{il}"
+            terms = self._spec_mixer(p, il, h, b, kv, st) if mixer else self._spec_ffn(p, il, h)
+            last = i + 1 == len(subs)
+            # behind the last sublayer: the plain sum of the streams and the output norm
+            in_w, norm_w = (None, w["output_norm"]) if last else (w[f"{subs[i + 1][1]}.st_in"], w[subs[i + 1][2]])
+            X, h = ops.hyper_step(X, terms, w[f"{hc}.st_mix"], w[f"{hc}.st_out"], in_w, norm_w, eps, off)
+            if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
+                captures[il] = X.sum(1)
+        hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
+        out = StepOutput(hidden=hidden, captures=captures)
+        if want_logits:
+            out.logits = self.logits(hidden)
+        self.pctx.end_step()
+        return out
+
     def _mamba2(self, p: str, il: int, x, b: StepBatch, st: StatePool):
         """Mamba-2 (SSD) layer: on a GPU the recurrence, the D skip and the silu(z) gate are one kernel with the state
         of a (sequence, head) in registers (``csrc/mamba2.cu``); the CPU form is the token-serial reference."""
@@ -1162,6 +1274,8 @@ class Decoder:
     def forward(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool = True) -> StepOutput:
         if self.pipe is not None:
             return self._forward_pipe(b, kv, st, want_logits)
+        if self.cfg.layers is not None:
+            return self._forward_streams(b, kv, st, want_logits)
         if self.cfg.hyper_streams > 1:
             return self._forward_hc(b, kv, st, want_logits)
         if self.cfg.sandwich_norm:

@@ -23,6 +23,8 @@ def layer_weight_shapes(cfg: ModelConfig, il: int, prefix: Optional[str] = None,
     kind = kind or cfg.layer_kinds[il]
     moe = cfg.is_moe_layer(il) if moe is None else moe
     H = cfg.hidden
+    if cfg.layers is not None and prefix is None:
+        return spec_layer_shapes(cfg, il)
     if cfg.block_form and prefix is None:
         # one sub-layer per block: its input norm plus either the mixer's or the feed-forward part's tensors
         if kind in ("ffn", "moe"):
@@ -131,6 +133,58 @@ def _ffn_shapes(cfg: ModelConfig, p: str, moe: bool, s: Dict[str, Tuple[int, ...
     return s
 
 
+def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
+    """A layer of a stack with specifications (``ModelConfig.layers``). What reads the mixer's input is one stacked
+    projection: ``lin.qkvg`` (linear attention: q | k | v | gate), ``mix.in`` (q | k | v of the attention part, then
+    z | x | B | C | dt of the state-space part)."""
+    p, H, spec = f"l{il}", cfg.hidden, cfg.layers[il]
+    s: Dict[str, Tuple[int, ...]] = {f"{p}.attn_norm": (H,)}
+    if spec.mlp is not None:
+        s[f"{p}.ffn_norm"] = (H,)
+    m = spec.mixer
+    if m.kind == "lightning":
+        s[f"{p}.lin.qkvg"] = (2 * m.heads * (m.dim + m.vdim), H)
+        s[f"{p}.lin.norm"] = (m.heads * m.vdim,)
+        s[f"{p}.lin.out"] = (H, m.heads * m.vdim)
+    else:
+        a, r = cfg.attn_spec(il), cfg.recurrent_spec(il)
+        rows = 0
+        if a is not None:
+            rows += (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim
+            if a.qk_norm:
+                s[f"{p}.attn.q_norm"] = (a.dim,)
+                s[f"{p}.attn.k_norm"] = (a.dim,)
+            s[f"{p}.attn.o"] = (H, a.heads * a.vdim)
+        if r is not None:
+            inner, conv_c = r.heads * r.vdim, r.heads * r.vdim + 2 * r.groups * r.state
+            rows += inner + conv_c + r.heads
+            s[f"{p}.ssm.conv_w"] = (conv_c, r.conv)
+            s[f"{p}.ssm.conv_b"] = (conv_c,)
+            for leaf in ("A", "D", "dt_bias"):
+                s[f"{p}.ssm.{leaf}"] = (r.heads,)
+            s[f"{p}.ssm.norm"] = (inner,)
+            s[f"{p}.ssm.out"] = (H, inner)
+        s[f"{p}.mix.in"] = (rows, H)
+    n = cfg.hyper_streams
+    for which in ("hca", "hcf")[:1 if spec.mlp is None else 2]:
+        s[f"{p}.{which}.st_in"] = (n,)                  # streams -> sublayer input
+        s[f"{p}.{which}.st_out"] = (n,)                 # sublayer output -> streams
+        s[f"{p}.{which}.st_mix"] = (n, n)               # stream (row) -> stream (column)
+    if spec.mlp is None:
+        return s
+    f = spec.mlp
+    if f.kind == "moe":
+        s[f"{p}.moe.router"] = (f.experts, H)
+        if f.correction:
+            s[f"{p}.moe.router_bias"] = (f.experts,)
+        s[f"{p}.moe.gate_up"] = (f.experts, 2 * f.ff, H)
+        s[f"{p}.moe.down"] = (f.experts, H, f.ff)
+    else:
+        s[f"{p}.mlp.gate_up"] = (2 * f.ff, H)
+        s[f"{p}.mlp.down"] = (H, f.ff)
+    return s
+
+
 def gemma_layer_shapes(cfg: ModelConfig, il: int, s: Dict[str, Tuple[int, ...]]) -> Dict[str, Tuple[int, ...]]:
     """Gemma-4 layer: q (+ k (+ v)) rows of this layer's head size, post norms, optional routed experts beside the
     dense FFN, output scale, per-layer embedding gate / projection."""
@@ -207,7 +261,7 @@ def is_fp32_weight(name: str) -> bool:
     leaf = name.rsplit(".", 1)[-1]
     return leaf.endswith("norm") or leaf in ("A", "D", "dt_bias", "conv_w", "conv_b", "router_bias", "hc_f", "hc_scale",
                                              "hc_base", "hcg_norm", "hcg_down", "hcg_up", "hcg_inject", "router_scale",
-                                             "out_scale")
+                                             "out_scale", "st_in", "st_out", "st_mix")
 
 
 def layer_of(name: str) -> Optional[int]:
@@ -237,13 +291,19 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=torch.float32, seed: in
         if dropped and (leaf.endswith("norm") or leaf == "D" or (device.type == "cuda" and wd == torch.bfloat16)):
             continue                      # nothing drawn from the host generator for these
         if leaf.endswith("norm"):
-            t = torch.ones(shp, dtype=torch.float32, device=device) - cfg.norm_offset
+            # head norms and the norms behind a recurrent state have plain weights in stacks with specifications
+            plain = cfg.layers is not None and leaf not in ("attn_norm", "ffn_norm", "output_norm")
+            t = torch.ones(shp, dtype=torch.float32, device=device) - (0.0 if plain else cfg.norm_offset)
         elif leaf == "A":
             t = -(torch.rand(shp, generator=g) * 0.9 + 0.1).to(device)
         elif leaf == "D":
             t = torch.ones(shp, dtype=torch.float32, device=device)
         elif leaf in ("dt_bias", "conv_b", "router_bias"):
             t = (torch.randn(shp, generator=g) * 0.1).to(device)
+        elif leaf in ("st_in", "st_out", "st_mix"):
+            n = shp[0]                    # near the plain residual: the streams' mean in, every stream gets the output
+            base = torch.eye(n) if leaf == "st_mix" else torch.full(shp, 1.0 / n if leaf == "st_in" else 1.0)
+            t = (base + torch.randn(shp, generator=g) * 0.05).to(device)
         elif leaf in ("hc_scale", "router_scale", "out_scale"):
             t = torch.ones(shp, dtype=torch.float32, device=device) * (0.9 if leaf == "out_scale" else 1.0)
         elif leaf == "hc_base":
@@ -279,7 +339,7 @@ class Shard:
         if dp_attention:
             self.kv_rep = 1
             return
-        if world > 1 and ("kda" in cfg.layer_kinds or cfg.hyper_streams > 1 or cfg.sandwich_norm or cfg.block_form):
+        if world > 1 and (cfg.layers is not None or "kda" in cfg.layer_kinds or cfg.hyper_streams > 1 or cfg.sandwich_norm or cfg.block_form):
             raise NotImplementedError("Kimi-delta-attention layers, hyper-connections and the Gemma-4 layer form run "
                                       "on one rank (their weights have no tensor-parallel split here)")
         assert cfg.n_head % world == 0, "query heads must divide by the TP degree"

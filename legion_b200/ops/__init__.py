@@ -22,7 +22,7 @@ def _cuda(t) -> bool:
 
 def linear(x, w, residual=None, out_dtype=None, out=None):
     if _cuda(x):
-        return _sm.linear(x, w, residual=residual, out=out, out_dtype=out_dtype or torch.bfloat16)
+        return _sm.linear(x, w, residual=residual, out=out, out_dtype=out_dtype or getattr(x, "dtype", torch.bfloat16))
     y = _ref.linear(x, w, residual=residual, out_dtype=out_dtype)
     if out is not None:
         out.copy_(y)
@@ -32,8 +32,8 @@ def linear(x, w, residual=None, out_dtype=None, out=None):
 
 def gate_up_act(x, w_gate_up, n_ff, act="silu"):
     if _cuda(x):
-        if act == "silu":
-            return _sm.gate_up_act(x, w_gate_up, n_ff)
+        if act == "silu" or (act == "gelu_tanh" and isinstance(w_gate_up, torch.Tensor)):
+            return _sm.gate_up_act(x, w_gate_up, n_ff, act=act)
         h = _sm.linear(x, w_gate_up)
         out = torch.empty(x.shape[0], n_ff, dtype=torch.bfloat16, device=x.device)
         _sm.ext().glu(h, out, n_ff, {"gelu_tanh": 1, "relu2": 2}[act])
@@ -68,8 +68,11 @@ def apply_output_gate(attn, gate, n_q, d):
 
 def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, max_q_len, scale, window=0, causal=True,
                     decode_splits=None, max_ctx=None):
-    """Varlen paged attention; ``max_q_len == 1`` selects the flash-decoding kernel on CUDA."""
+    """Varlen paged attention; ``max_q_len == 1`` selects the flash-decoding kernel on CUDA. fp32 caches and head sizes
+    the tensor-core kernels do not take run on the general kernel (causal only)."""
     if _cuda(q):
+        if not _sm.attn_tc_ok(q, k_cache, v_cache):
+            return _sm.paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal)
         if max_q_len == 1 and causal:
             return _sm.paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window, decode_splits, max_ctx)
         return _sm.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal)
@@ -83,7 +86,7 @@ def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
 
 
 def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
-           e_lo=0, n_local=None, norm=None, **gpu_kw):
+           e_lo=0, n_local=None, norm=None, group_top=2, **gpu_kw):
     """Router projection + top-k. Returns an object that unpacks as ``ids, wts`` ([T, k] int32 / float32); on the
     GPU it may also carry the dense routing tables of a decode-sized step for the experts
     [e_lo, e_lo + n_local) of this rank (pass it on as ``routing=``). With ``norm=(weight, eps, w_offset)`` ``x`` is
@@ -91,12 +94,12 @@ def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
     and the result's ``x_normed`` is the normalised input for the experts."""
     if _cuda(x):
         return _sm.router(x, w_router, k, mode, renorm, route_scale, bias, n_group, topk_group, norm, e_lo, n_local,
-                          **gpu_kw)
+                          group_top=group_top, **gpu_kw)
     xn = None
     if norm is not None:
         xn, _ = _ref.rmsnorm(x, norm[0], norm[1], norm[2])
     logits = _ref.linear(x if xn is None else xn, w_router, out_dtype=torch.float32)
-    ids, wts = _ref.router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group)
+    ids, wts = _ref.router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group, group_top)
     return _sm.Routing(ids, wts, None, xn)
 
 
@@ -146,6 +149,9 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, shared
                 residual=None, out=None, norm=None, routing=None, defer_combine=False):
     """Routed experts (+ optional shared-expert output with sigmoid gate logits, + residual). Returns [T, H];
     with ``norm=(weight, eps, w_offset)`` returns (out, rmsnorm(out)): on the GPU the norm rides on the combine."""
+    if _cuda(x) and isinstance(w_gate_up, torch.Tensor) and not _sm.tma_ok(x, w_gate_up, w_down):
+        return _sm.moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act, e_lo, shared, shared_gate, residual, norm,
+                                     defer_combine)
     if _cuda(x) and act != "silu":
         if act not in ("relu2", "gelu_tanh") or not isinstance(w_gate_up, torch.Tensor):
             raise NotImplementedError("the grouped expert kernels implement SwiGLU experts (squared-ReLU and GELU "
@@ -179,6 +185,8 @@ def argmax(logits):
 
 
 def embed(ids, table):
+    if _cuda(table) and table.dtype == torch.float32:
+        return table.index_select(0, ids.long())
     if _cuda(table):
         return _sm.embed(ids.int(), table)
     return table[ids.long()]
@@ -188,6 +196,41 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, 
     if _cuda(x):
         return _sm.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state, max_len=max_len)
     return _ref.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state)
+
+
+def hyper_start(table, ids, streams, in_w, norm_w, eps, w_offset=0.0):
+    """Hyper-connections with static weights: the streams start as the embedding rows (``ids`` None: the rows are given
+    in ``table``). Returns (streams [T, S, H] float32, normed input of the first sublayer)."""
+    if _cuda(table):
+        return _sm.hyper_start(table, ids, streams, in_w, norm_w, eps, w_offset)
+    return _ref.hyper_start(table if ids is None else table[ids.long()], streams, in_w, norm_w, eps, w_offset)
+
+
+def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset=0.0):
+    """Stream update behind a sublayer, input mix and norm of the next one, in one launch; on CUDA ``X`` is updated in
+    place. ``terms``: [(sublayer output, scale)], at most two; an ``ops.sm100.PendingCombine`` counts as one."""
+    if _cuda(X):
+        return _sm.hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset)
+    return _ref.hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset)
+
+
+def qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache):
+    if _cuda(q):
+        return _sm.qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache)
+    return _ref.qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache)
+
+
+def linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, max_len=None, cu_host=None, **kw):
+    """Decayed linear-attention state (see ``reference.linear_scan``)."""
+    if _cuda(q):
+        return _sm.linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, max_len=max_len, cu_host=cu_host, **kw)
+    return _ref.linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, **kw)
+
+
+def group_norm_gate(y, gate, w, eps, groups=1):
+    if _cuda(y):
+        return _sm.group_norm_gate(y, gate, w, eps, groups)
+    return _ref.group_norm_gate(y, gate, w, eps, groups)
 
 
 def gdn_gates(a, b, A, dt_bias):

@@ -173,11 +173,11 @@ def _gather_kv(cache, table_row, n_tokens):
 def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window: int = 0, causal: bool = True,
                     sinks=None, softcap: float = 0.0):
     """Varlen paged attention. q: [T, Hq, D]; sequence i owns query rows cu_q[i]:cu_q[i+1], which are the
-    LAST rows of its ctx_lens[i] cached tokens. Returns [T, Hq, D]."""
+    LAST rows of its ctx_lens[i] cached tokens. Returns [T, Hq, Dv] (values may have a head size of their own)."""
     T, Hq, D = q.shape
     Hkv = k_cache.shape[2]
     G = Hq // Hkv
-    out = torch.zeros_like(q)
+    out = q.new_zeros(T, Hq, v_cache.shape[3])
     for i in range(len(ctx_lens)):
         q0, q1 = int(cu_q[i]), int(cu_q[i + 1])
         if q1 <= q0:
@@ -210,19 +210,20 @@ def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, win
 
 
 def router_topk(logits, k: int, mode: str = "softmax", renorm: bool = True, route_scale: float = 1.0, bias=None,
-                n_group: int = 1, topk_group: int = 1):
-    """Returns (ids [T, k] int32, weights [T, k] float32); ties go to the lower expert id."""
+                n_group: int = 1, topk_group: int = 1, group_top: int = 2):
+    """Returns (ids [T, k] int32, weights [T, k] float32); ties go to the lower expert id. ``softmax_bias``: selection
+    by softmax score + bias, like the sigmoid mode; ``group_top``: how many scores a group's rank sums up."""
     lf = logits.float()
     T, E = lf.shape
     if mode == "softmax":
         scores = torch.softmax(lf, dim=-1)
         sel = scores.clone()
     else:
-        scores = torch.sigmoid(lf)
+        scores = torch.softmax(lf, dim=-1) if mode == "softmax_bias" else torch.sigmoid(lf)
         sel = scores + (bias.float() if bias is not None else 0.0)
         if n_group > 1 and topk_group < n_group:
             g = sel.view(T, n_group, E // n_group)
-            gscore = g.topk(min(2, g.shape[-1]), dim=-1).values.sum(-1)
+            gscore = g.topk(min(group_top, g.shape[-1]), dim=-1).values.sum(-1)
             order = torch.sort(gscore, dim=-1, descending=True, stable=True).indices[:, :topk_group]
             keep = torch.zeros(T, n_group, dtype=torch.bool, device=lf.device)
             keep.scatter_(1, order, True)
@@ -278,7 +279,7 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool 
         if bias is not None:
             y = y + bias.float()
         out[t0:t1] = F.silu(y).to(x.dtype)
-        if write_state:
+        if write_state and KC > 1:
             conv_state[s] = seq[-(KC - 1):].t().to(conv_state.dtype)
     return out
 
@@ -323,6 +324,83 @@ def gated_rmsnorm(o, z, w, eps: float, act: str = "silu"):
     y = of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps) * w.float()
     zf = z.float()
     return (y * (F.silu(zf) if act == "silu" else torch.sigmoid(zf))).to(o.dtype)
+
+
+def hyper_start(rows, streams: int, in_w, norm_w, eps: float, w_offset: float):
+    """Every stream starts as the embedding row. Returns (streams [T, S, H] float32, h = norm of the mixed input)."""
+    X = rows.float().unsqueeze(1).expand(-1, streams, -1).contiguous()
+    u = torch.einsum("s,tsh->th", in_w, X) if in_w is not None else X.sum(1)
+    return X, _norm32(u, norm_w, eps, w_offset).to(rows.dtype)
+
+
+def _norm32(u, w, eps, w_offset):
+    return u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + w_offset)
+
+
+def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps: float, w_offset: float):
+    """Static hyper-connection around a sublayer: y = sum of scale * tensor over ``terms``; X'_t = sum_s mix[s, t] X_s +
+    out[t] y; returns (X', norm of the next sublayer's input sum_t in[t] X'_t). ``in_w`` None: plain sum."""
+    y = sum(c * t.float() for t, c in terms)
+    Xn = torch.einsum("st,nsh->nth", mix, X) + out_w[None, :, None] * y.unsqueeze(1)
+    u = torch.einsum("s,tsh->th", in_w, Xn) if in_w is not None else Xn.sum(1)
+    return Xn, _norm32(u, norm_w, eps, w_offset).to(terms[0][0].dtype)
+
+
+def qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache):
+    """Head norms and paged append with separate key / value head sizes; returns q [T, Hq, dk]."""
+    n_kv, dk, dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    T = q.shape[0]
+    q, k = q.reshape(T, -1, dk), k.reshape(T, n_kv, dk)
+    if q_norm is not None:
+        q, k = head_rmsnorm(q, q_norm, eps), head_rmsnorm(k, k_norm, eps)
+    ok = slots >= 0
+    k_cache.view(-1, n_kv, dk)[slots[ok].long()] = k[ok].to(k_cache.dtype)
+    v_cache.view(-1, n_kv, dv)[slots[ok].long()] = v.reshape(T, n_kv, dv)[ok].to(v_cache.dtype)
+    return q.contiguous()
+
+
+def linear_scan(q, k, v, state, cu_seq, slots, H: int, G: int, N: int, P: int, decay=None, silu_in: bool = False,
+                dt=None, dt_bias=None, A=None, D=None, z=None, write_state: bool = True):
+    """S_t = a_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, token by token; state [slots, H, P, N] float32. ``decay`` [H]:
+    constant per head; else a_t = exp(dt_t A) with dt_t = softplus(dt + dt_bias), which also scales v. D: skip; z: gate
+    by silu(z). q, k [T, G * N], v [T, H * P]."""
+    T = q.shape[0]
+    qf, kf, vf = q.float().view(T, G, N), k.float().view(T, G, N), v.float().view(T, H, P)
+    if silu_in:
+        qf, kf, vf = F.silu(qf), F.silu(kf), F.silu(vf)
+    qf, kf = qf.repeat_interleave(H // G, 1), kf.repeat_interleave(H // G, 1)
+    if decay is not None:
+        a, vd = decay.float().expand(T, H), vf
+    else:
+        step = F.softplus(dt.float() + dt_bias.float())
+        a, vd = torch.exp(step * A.float()), vf * step.unsqueeze(-1)
+    out = torch.zeros(T, H, P)
+    for i in range(len(slots)):
+        t0, t1, s = int(cu_seq[i]), int(cu_seq[i + 1]), int(slots[i])
+        if t1 <= t0:
+            continue
+        S = state[s].clone()
+        for t in range(t0, t1):
+            S = S * a[t][:, None, None] + vd[t].unsqueeze(2) * kf[t].unsqueeze(1)
+            out[t] = torch.einsum("hpn,hn->hp", S, qf[t])
+        if write_state:
+            state[s] = S
+    if D is not None:
+        out = out + D.float()[:, None] * vf
+    out = out.reshape(T, H * P)
+    if z is not None:
+        out = out * F.silu(z.float())
+    return out.to(q.dtype)
+
+
+def group_norm_gate(y, gate, w, eps: float, groups: int = 1):
+    """RMS norm in ``groups`` equal parts, times w, times sigmoid(gate) when given."""
+    T, C = y.shape
+    yf = y.float().view(T, groups, C // groups)
+    out = (yf / torch.sqrt(yf.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, C) * w.float()
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float())
+    return out.to(y.dtype)
 
 
 def sample(logits, temperature, top_k, top_p, min_p, generator=None):

@@ -83,7 +83,7 @@ def ext():
         with _lock:
             if _C is None and _C_err is None:
                 try:
-                    mod = importlib.import_module("legion_b200._C")
+                    mod = _import_ext()
                     mod.set_pdl(bool(TUNE["pdl"]))
                     _C = _Counting(mod)
                 except BaseException as e:  # missing .so, ABI mismatch, missing libcudart
@@ -93,6 +93,15 @@ def ext():
             "legion_b200._C (the sm_100a extension) is not importable: build it with "
             "`python -m legion_b200.build_ext`") from _C_err
     return _C
+
+
+def _import_ext():
+    """The full extension ``_C``, or the subset ``_C_core`` in a checkout where only that one was built."""
+    from importlib.util import find_spec
+    name = "legion_b200._C"
+    if find_spec(name) is None and find_spec("legion_b200._C_core") is not None:
+        name = "legion_b200._C_core"
+    return importlib.import_module(name)
 
 
 def have_ext() -> bool:
@@ -576,9 +585,32 @@ def _linear_fp8(x, w: "Fp8Weight", residual, out, dual: bool, n_feat: int):
     return out
 
 
+ROUTER_MODES = {"softmax": 0, "sigmoid": 1, "softmax_bias": 2}
+GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
+
+
+def tma_ok(*ts) -> bool:
+    """bf16 operands whose rows TMA can fetch (16-byte aligned base and row pitch)."""
+    return all(t.dtype == torch.bfloat16 and t.shape[-1] % 8 == 0 and t.stride(-2) % 8 == 0 and t.data_ptr() % 16 == 0
+               for t in ts)
+
+
+def sgemm(x, w, residual=None, out=None, out_dtype=None, dual: bool = False, n_ff: int = 0, act: str = "silu"):
+    """x @ w^T in fp32 arithmetic on the FMA units: fp32 models and shapes outside the tcgen05 GEMM's alignment rules.
+    ``dual``: act(x Wg^T) * (x Wu^T) with Wg = w[:n_ff], Wu = w[n_ff:]."""
+    T, N = x.shape[0], (n_ff if dual else w.shape[0])
+    if out is None:
+        out = torch.empty(T, N, dtype=out_dtype or x.dtype, device=x.device)
+    ext().sgemm(w, x, out, residual, None, None, N, dual, n_ff if dual else 0, GATE_ACTS[act] if dual else 0, None, None,
+                None, None, 0, 0, T)
+    return out
+
+
 def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Optional[int] = None, bn=None):
     """out[T, N] = x[T, K] @ w[N, K]^T (+ residual)."""
     C = ext()
+    if isinstance(w, torch.Tensor) and isinstance(x, torch.Tensor) and not tma_ok(x, w):
+        return sgemm(x, w, residual, out, out_dtype)
     if isinstance(x, Fp8Act) and not isinstance(w, Fp8Weight):
         x = x.x
     T, K = x.shape
@@ -613,9 +645,11 @@ def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Opt
     return out
 
 
-def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[int] = None):
-    """silu(x @ Wg^T) * (x @ Wu^T) with Wg = w_gate_up[:n_ff], Wu = w_gate_up[n_ff:]."""
+def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[int] = None, act: str = "silu"):
+    """act(x @ Wg^T) * (x @ Wu^T) with Wg = w_gate_up[:n_ff], Wu = w_gate_up[n_ff:] (GELU: bf16 weights only)."""
     C = ext()
+    if isinstance(w_gate_up, torch.Tensor) and isinstance(x, torch.Tensor) and not tma_ok(x, w_gate_up):
+        return sgemm(x, w_gate_up, None, out, None, True, n_ff, act)
     if isinstance(x, Fp8Act) and not isinstance(w_gate_up, Fp8Weight):
         x = x.x
     T, K = x.shape
@@ -639,7 +673,7 @@ def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[in
     q = isinstance(w_gate_up, QWeight)
     C.wgemm(w_gate_up.codes if q else w_gate_up, x, out, None, None, None, n_ff, True, n_ff, bn, sk,
             ws.splitk if sk > 1 else None, ws.counters if sk > 1 else None, ws.status, None, None, None, None, 0, 0, T,
-            [], None, w_gate_up.scales if q else None, w_gate_up.gscale if q else None)
+            [], None, w_gate_up.scales if q else None, w_gate_up.gscale if q else None, 0, 0, GATE_ACTS[act])
     return out
 
 
@@ -700,16 +734,19 @@ def decode_splits(batch: int, n_kv_heads: int, g_tiles: int, max_ctx: int, head_
 def paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window=0, n_splits=None, max_ctx=None, out=None,
                  impl="tc"):
     C = ext()
-    B, Hq, D = q.shape
-    Hkv = k_cache.shape[2]
+    B, Hq, _ = q.shape
+    Hkv, D = k_cache.shape[2], v_cache.shape[3]
     if n_splits is None:
         G = Hq // Hkv
-        n_splits = decode_splits(B, Hkv, (G + 15) // 16, max_ctx or block_table.shape[1] * k_cache.shape[1], D)
+        span = max_ctx or block_table.shape[1] * k_cache.shape[1]
+        if window > 0:
+            span = min(span, window + 128)            # tiles a window can touch
+        n_splits = decode_splits(B, Hkv, (G + 15) // 16, span, D)
     ws = Workspace.get(q.device)
     o_part = ws.buf("dec_o", (B * Hq * n_splits * 2 * D,), torch.float32)
     ml_part = ws.buf("dec_ml", (B * Hq * n_splits * 2 * 2,), torch.float32)
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty(B, Hq, D, dtype=q.dtype, device=q.device)
     C.paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window, n_splits, o_part, ml_part, out,
                    impl == "tc", ws.status, ws.counters)
     return out
@@ -718,10 +755,35 @@ def paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window=0, n_
 def prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window=0, causal=True, out=None):
     C = ext()
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty(q.shape[0], q.shape[1], v_cache.shape[3], dtype=q.dtype, device=q.device)
     ws = Workspace.get(q.device)
     C.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal, out, ws.status)
     return out
+
+
+def attn_tc_ok(q, k_cache, v_cache) -> bool:
+    """Whether the tcgen05 attention kernels take these caches: bf16, head sizes that are multiples of 8 up to 256."""
+    dk, dv, page = k_cache.shape[3], v_cache.shape[3], k_cache.shape[1]
+    return (q.dtype == torch.bfloat16 and dk % 8 == 0 and dv % 8 == 0 and dk <= 256 and dv <= 256 and page % 8 == 0
+            and 64 % page == 0)
+
+
+def paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window=0, causal=True, out=None):
+    """Paged causal attention for fp32 and for head sizes outside the tensor-core kernels (prompts and decode rows)."""
+    if not causal:
+        raise NotImplementedError("the general attention kernel is causal")
+    if out is None:
+        out = torch.empty(q.shape[0], q.shape[1], v_cache.shape[3], dtype=q.dtype, device=q.device)
+    ext().paged_attn_general(q, k_cache, v_cache, cu_q, ctx_lens, block_table, scale, window, out)
+    return out
+
+
+def qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache):
+    """q, k, v: column slices of one projection. Head norms (plain weights, optional), k and v to their cache cells;
+    returns the queries [T, heads, dk]. Any head sizes, bf16 or fp32."""
+    q_out = torch.empty(q.shape[0], q.shape[1] // k_cache.shape[3], k_cache.shape[3], dtype=q.dtype, device=q.device)
+    ext().qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, q_out, k_cache, v_cache)
+    return q_out
 
 
 def head_linear(x, w2d, n_heads: int, rows_per_group: int, n_feat: int, K: int, x_group_col: int, out2d):
@@ -796,13 +858,13 @@ def mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, 
 
 
 def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
-                ids=None, wts=None):
+                ids=None, wts=None, group_top: int = 2):
     C = ext()
     T = logits.shape[0]
     if ids is None:
         ids = torch.empty(T, k, dtype=torch.int32, device=logits.device)
         wts = torch.empty(T, k, dtype=torch.float32, device=logits.device)
-    C.router_topk(logits, bias, k, 0 if mode == "softmax" else 1, renorm, route_scale, n_group, topk_group, ids, wts)
+    C.router_topk(logits, bias, k, ROUTER_MODES[mode], renorm, route_scale, n_group, topk_group, ids, wts, group_top)
     return ids, wts
 
 
@@ -849,7 +911,7 @@ class DenseRoute:
 
 def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
            norm=None, e_lo: int = 0, n_local: Optional[int] = None, slot_stride: Optional[int] = None, sh_gate=None,
-           shared_slot: bool = False):
+           shared_slot: bool = False, group_top: int = 2):
     """Router logits and top-k selection -> ``Routing``. Decode-sized steps (<= 64 tokens, <= 1024 pairs) run as
     ONE launch that also builds the dense routing tables; with ``norm=(weight, eps, w_offset)`` that launch first
     applies the RMSNorm to ``x`` (the raw residual stream) and ``Routing.x_normed`` is the normalised input.
@@ -857,13 +919,13 @@ def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
     every token uses (weight sigmoid(x . sh_gate) when ``sh_gate`` [1, H] is given, else 1); its output rows are
     the pairs T * k .. T * k + T - 1. Larger steps use the GEMM and the selection kernel."""
     T, E = x.shape[0], w_router.shape[0]
-    small = T <= 64 and T * k <= 1024 and TUNE["fused_router"]
+    small = T <= 64 and T * k <= 1024 and TUNE["fused_router"] and tma_ok(x, w_router)
     if not small:
         xn = None
         if norm is not None:
             xn, _ = rmsnorm(x, norm[0], norm[1], norm[2])
         logits = linear(x if xn is None else xn, w_router, out_dtype=torch.float32)
-        ids, wts = router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group)
+        ids, wts = router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group, group_top=group_top)
         return Routing(ids, wts, None, xn)
     C = ext()
     ws = Workspace.get(x.device)
@@ -884,10 +946,10 @@ def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
     wts = torch.empty(T, k, dtype=torch.float32, device=x.device)
     xn = torch.empty_like(x) if norm is not None else None
     C.moe_route_small(x, norm[0] if norm else None, norm[1] if norm else 0.0, norm[2] if norm else 0.0, xn, w_router,
-                      bias, k, 0 if mode == "softmax" else 1, renorm, route_scale, n_group, topk_group, logits, ids, wts,
+                      bias, k, ROUTER_MODES[mode], renorm, route_scale, n_group, topk_group, logits, ids, wts,
                       stride, dr.tile_group, dr.slot_base, dr.tile_ntok, dr.meta, dr.out_rows, dr.tok_scale, ctr,
                       e_lo, nl, sh_gate.reshape(-1) if sh_gate is not None else None,
-                      dr.sh_logit if sh_gate is not None else None, bool(shared_slot), ws.status, dr.active)
+                      dr.sh_logit if sh_gate is not None else None, bool(shared_slot), ws.status, dr.active, group_top)
     r = Routing(ids, wts, dr, xn, e_lo, nl)
     r.shared_slot = bool(shared_slot)
     return r
@@ -1170,6 +1232,8 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
     C.wgemm(dn2, plan.h_sorted, plan.y_pairs, None, plan.sorted_w, plan.sorted_pair, H, False, 0, bn, 1, None, None,
             ws.status, plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, 0, [], None,
             dn_sc, dn_gs)
+    if defer_combine == "pairs":
+        return PendingCombine(plan.y_pairs, ids, e_lo, e_lo + E_local, None, T, H)
     if out is None:
         out = torch.empty(T, H, dtype=torch.bfloat16, device=x.device)
     if norm is None:
@@ -1179,6 +1243,35 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
     C.moe_combine(plan.y_pairs, ids, e_lo, e_lo + E_local, shared, shared_gate, residual, out, norm[0], norm[1],
                   norm[2], normed)
     return out, normed
+
+
+def moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, shared=None, shared_gate=None,
+                      residual=None, norm=None, defer_combine=False):
+    """Routed experts on the FMA units over the same routing plan (fp32 models, unaligned bf16 shapes; all experts
+    local, gated experts without a shared one). With ``defer_combine`` the weighted pair rows are handed on."""
+    if e_lo or shared is not None or residual is not None or norm is not None or w_gate_up.shape[1] != 2 * n_ff:
+        raise NotImplementedError("plain experts: gated, all local, no shared expert, residual or norm")
+    C = ext()
+    T, H = x.shape
+    k, E = ids.shape[1], w_gate_up.shape[0]
+    P, bn = T * k, 32
+    ws = Workspace.get(x.device)
+    key = ("moe_plan_plain", T, k, E)
+    plan = ws._cache.get(key)
+    if plan is None:
+        plan = ws._cache[key] = MoePlan(T, k, E, bn, x.device)
+    C.moe_plan(ids, wts, 0, E, bn, plan.counts, plan.offsets, plan.sorted_token, plan.sorted_pair, plan.sorted_w,
+               plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta)
+    xs = x.index_select(0, plan.sorted_token)
+    h = torch.empty(P, n_ff, dtype=x.dtype, device=x.device)
+    y = torch.empty(P, H, dtype=x.dtype, device=x.device)
+    C.sgemm(w_gate_up.view(E * 2 * n_ff, H), xs, h, None, None, None, n_ff, True, n_ff, GATE_ACTS[act], plan.tile_group,
+            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, 2 * n_ff, P)
+    C.sgemm(w_down.view(E * H, n_ff), h, y, None, plan.sorted_w, plan.sorted_pair, H, False, 0, 0, plan.tile_group,
+            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, P)
+    if defer_combine:
+        return PendingCombine(y, ids, 0, E, None, T, H)
+    return y.view(T, k, H).sum(1, dtype=torch.float32).to(x.dtype)
 
 
 def _moe_experts_fp8(x, ids, wts, w_gate_up, w_down, n_ff, e_lo, shared, shared_gate, residual, out, norm, routing,
@@ -1301,7 +1394,10 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, 
     sequence) run the token-parallel kernel."""
     C = ext()
     if out is None:
-        out = torch.empty_like(x)
+        out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    if x.dtype != torch.bfloat16 or not 2 <= w.shape[1] <= 8:
+        C.conv_silu_any(x, w, bias, conv_state, cu_seq, slots, out, bool(write_state))
+        return out
     T, n = x.shape[0], max(1, slots.numel())
     if max_len is None:
         max_len = T if T >= 64 * n else 0          # without the host figure: only clearly prompt-sized steps
@@ -1411,6 +1507,97 @@ def mamba2_scan(xbc, dt_raw, z, A, D, dt_bias, state, cu_seq, slots, nh, hd, ng,
         return out
     C.mamba2_scan(xbc, dt_raw, z, A.float(), D.float(), dt_bias.float(), state, cu_seq, slots, nh, hd, ng, ds, out,
                   bool(write_state))
+    return out
+
+
+def hyper_start(table, ids, streams: int, in_w, norm_w, eps, w_offset=0.0):
+    """Streams [T, S, H] fp32 from the embedding and the normed input of the first sublayer, in one launch."""
+    T = table.shape[0] if ids is None else ids.numel()
+    X = torch.empty(T, streams, table.shape[1], dtype=torch.float32, device=table.device)
+    h = torch.empty(T, table.shape[1], dtype=table.dtype, device=table.device)
+    ext().hyper_step(None, X, table, ids, None, 0.0, 1, None, 0.0, None, None, in_w, norm_w, eps, w_offset, h)
+    return X, h
+
+
+def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset=0.0):
+    """X (fp32 streams) updated in place behind a sublayer, and the normed input of the next one. A ``PendingCombine``
+    term is summed over its weighted expert rows inside the launch."""
+    (y0, c0), (y1, c1) = (list(terms) + [(None, 0.0)])[:2]
+    rows = 1
+    if isinstance(y0, PendingCombine):
+        rows, y0 = y0.ids.shape[1], y0.y
+    h = torch.empty(X.shape[0], X.shape[2], dtype=y0.dtype, device=X.device)
+    ext().hyper_step(X, X, None, None, y0, c0, rows, y1, c1, mix, out_w, in_w, norm_w, eps, w_offset, h)
+    return X, h
+
+
+LINEAR_CHUNK_MIN = 48        # longest portion of a step from which the chunked scan runs
+
+
+def _linear_chunk_tables(ws, cu_host, device):
+    """chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk of a step (128-token chunks); kept for the step's other
+    layers."""
+    key = tuple(cu_host)
+    last = ws._cache.get("linear_chunk_tables")
+    if last is not None and last[0] == key:
+        return last[1], last[2]
+    t0, n, sq, first, cnt = [], [], [], [], []
+    for i in range(len(cu_host) - 1):
+        first.append(len(t0))
+        for b in range(cu_host[i], cu_host[i + 1], 128):
+            t0.append(b)
+            n.append(min(128, cu_host[i + 1] - b))
+            sq.append(i)
+        cnt.append(len(t0) - first[-1])
+    tab = torch.tensor(t0 + n + sq + first + cnt, dtype=torch.int32, device=device)
+    ws._cache["linear_chunk_tables"] = (key, tab, len(t0))
+    return tab, len(t0)
+
+
+def linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, decay=None, silu_in=False, dt=None, dt_bias=None, A=None,
+                D=None, z=None, write_state=True, max_len=None, cu_host=None, out=None, chunked=None):
+    """Decayed linear-attention state over the step's tokens (constant or selective decay), state [slots, H, P, N] fp32
+    updated in place. bf16 prompts run in 128-token chunks on the tensor cores (``csrc/linear_scan_sm100.cu``), decode
+    rows, short portions and fp32 on the streaming kernel (``csrc/linear_scan.cu``). ``chunked`` forces the choice."""
+    C = ext()
+    if out is None:
+        out = torch.empty(q.shape[0], H * P, dtype=q.dtype, device=q.device)
+    args = (q, k, v, bool(silu_in), decay, dt, dt_bias, A, D, z, state, cu_seq, slots, H, G, N, P, out, bool(write_state))
+    if chunked is None:
+        chunked = (q.dtype == torch.bfloat16 and cu_host is not None and (max_len or 0) >= LINEAR_CHUNK_MIN
+                   and C.linear_chunk_ok(N, P))
+    if not chunked:
+        C.linear_scan(*args)
+        return out
+    ws = Workspace.get(q.device)
+    tab, n_chunks = _linear_chunk_tables(ws, cu_host if cu_host is not None else cu_seq.tolist(), q.device)
+    need = C.linear_chunk_scratch_bytes(n_chunks, H, N, P)
+    scratch = ws._cache.get("linear_chunk_scratch")
+    if scratch is None or scratch.numel() < need:
+        scratch = ws._cache["linear_chunk_scratch"] = torch.empty(need, dtype=torch.uint8, device=q.device)
+    C.linear_chunk(*args, tab, n_chunks, scratch, ws.status)
+    return out
+
+
+def ssd_decode(xbc, conv_w, conv_b, conv_state, dt, dt_bias, A, D, z, state, cu_seq, slots, H, G, N, P, out=None):
+    """Decode step of a Mamba-2 mixer in one launch (one token per sequence): convolution with history update, step
+    size, state update, skip and silu(z) gate. ``xbc``: x | B | C columns of the input projection."""
+    n = slots.numel()
+    ws = Workspace.get(xbc.device)
+    ctr = ws._cache.get("ssd_ctr")
+    if ctr is None or ctr.numel() < n * G:
+        ctr = ws._cache["ssd_ctr"] = torch.zeros(max(n * G, 4096), dtype=torch.int32, device=xbc.device)
+    if out is None:
+        out = torch.empty(n, H * P, dtype=xbc.dtype, device=xbc.device)
+    ext().ssd_decode(xbc, conv_w, conv_b, conv_state, dt, dt_bias, A, D, z, state, cu_seq, slots, H, G, N, P, ctr, out)
+    return out
+
+
+def group_norm_gate(y, gate, w, eps, groups: int = 1, out=None):
+    """RMS norm of each of ``groups`` equal parts of a row, times w, times sigmoid(gate) when a gate is given."""
+    if out is None:
+        out = torch.empty(y.shape, dtype=y.dtype, device=y.device)
+    ext().group_norm_gate(y, gate, w, eps, groups, out)
     return out
 
 
