@@ -61,9 +61,10 @@ CASES = {
 }
 
 
-def make_weights(cfg, seed=0, dtype=torch.bfloat16):
-    """Random weights by checkpoint name. Head norms are scaled up so that single keys stand out among the scores, and
-    router rows so that no choice is close."""
+def make_weights(cfg, seed=0, dtype=torch.bfloat16, decisive=False):
+    """Random weights by checkpoint name. Head norms are scaled up so that single keys stand out among the scores.
+    ``decisive``: corrections so far apart that rounding cannot change a routing choice (bf16 comparisons of whole
+    models, where one flipped choice would change every later token)."""
     g = torch.Generator().manual_seed(seed)
     r = lambda *s: torch.randn(*s, generator=g)                     # noqa: E731
     u = lambda *s: torch.rand(*s, generator=g)                      # noqa: E731
@@ -113,6 +114,8 @@ def make_weights(cfg, seed=0, dtype=torch.bfloat16):
             parts = [f"{p}.mlp.e{e}" for e in range(E)]
             w[p + ".mlp.router"] = lin(E, W, 3.0)
             w[p + ".mlp.correction"] = r(E) * 0.3 - 0.3          # selection scores of either sign
+            if decisive:
+                w[p + ".mlp.correction"] = 2.0 * torch.randperm(E, generator=g) - E
         for b in parts:
             w[b + ".gate"], w[b + ".up"], w[b + ".down"] = lin(ff, W), lin(ff, W), lin(W, ff)
     return {k: v.to(dtype).contiguous() for k, v in w.items()}

@@ -27,33 +27,35 @@ def check(got, want, dtype, what=""):
     e = nc.errors(got, want)
     if dtype == "float32":
         assert e.max() < 1e-4, (what, float(e.max()), int(e.argmax()))
-    else:                                      # bf16 rounding; a rare routing choice may flip
-        assert e.quantile(0.9) < 0.04 and e.median() < 0.03, (what, float(e.quantile(0.9)), float(e.max()), int(e.argmax()))
+    else:                                      # bf16 rounding (scores of peaked attention reach 50)
+        assert e.max() < 0.2 and e.quantile(0.95) < 0.08 and e.median() < 0.03, (what, float(e.median()), float(e.max()),
+                                                                                int(e.argmax()))
 
 
 @pytest.fixture(scope="module")
 def models(tmp_path_factory):
     out = {}
     for i, (name, cfg) in enumerate(nc.CASES.items()):
-        w = nc.make_weights(cfg, seed=i)
-        out[name] = (cfg, w, nc.write_checkpoint(tmp_path_factory.mktemp(name), cfg, w))
+        for dtype in ("float32", "bfloat16"):
+            w = nc.make_weights(cfg, seed=i, decisive=dtype == "bfloat16")
+            out[name, dtype] = (cfg, w, nc.write_checkpoint(tmp_path_factory.mktemp(name), cfg, w))
     return out
 
 
 _EXPECT = {}
 
 
-def expected(models, name, n, seed):
-    key = (name, n, seed)
+def expected(models, name, dtype, n, seed):
+    key = (name, dtype, n, seed)
     if key not in _EXPECT:
-        cfg, w, _ = models[name]
+        cfg, w, _ = models[name, dtype]
         toks = nc.tokens(cfg, n, seed)
         _EXPECT[key] = (toks, oracle.forward(cfg, w, toks))
     return _EXPECT[key]
 
 
 def replay(models, name, device, dtype, max_tokens):
-    return TraceReplay(replay_engine(models[name][2], getattr(torch, dtype), max_tokens, device))
+    return TraceReplay(replay_engine(models[name, dtype][2], getattr(torch, dtype), max_tokens, device))
 
 
 def test_registry_and_config_round_trip():
@@ -70,7 +72,7 @@ def test_registry_and_config_round_trip():
 
 @pytest.mark.parametrize("name", list(nc.CASES))
 def test_loader_maps_every_tensor(models, name):
-    cfg, w, path = models[name]
+    cfg, w, path = models[name, "float32"]
     mc, lw, _, _ = load_model(path)
     shapes = weight_shapes(mc)
     assert set(shapes) == set(lw) and all(tuple(lw[k].shape) == tuple(v) for k, v in shapes.items())
@@ -83,7 +85,7 @@ def test_loader_maps_every_tensor(models, name):
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("name", list(nc.CASES))
 def test_whole_prompt_layer_by_layer(models, name, device, dtype):
-    cfg, w, path = models[name]
+    cfg, w, path = models[name, dtype]
     toks = nc.tokens(cfg, 70, 1)
     layers = []
     want = oracle.forward(cfg, w, toks, layers_out=layers)
@@ -102,7 +104,7 @@ def test_whole_prompt_layer_by_layer(models, name, device, dtype):
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("name", list(nc.CASES))
 def test_decoding_and_portions_equal_the_whole_prompt(models, name, device, dtype):
-    toks, want = expected(models, name, 210, 2)
+    toks, want = expected(models, name, dtype, 210, 2)
     n = len(toks)
     schedules = {
         "whole": [n],
@@ -128,7 +130,7 @@ def test_unequal_batches_and_used_pages_and_slots(models, name, device, dtype):
     pool that holds no more than the live ones need."""
     seqs, want = {}, {}
     for i, n in enumerate((130, 66, 1, 97, 64, 129, 40)):
-        seqs[f"s{i}"], want[f"s{i}"] = expected(models, name, n, 10 + i)
+        seqs[f"s{i}"], want[f"s{i}"] = expected(models, name, dtype, n, 10 + i)
     schedule = [[("s0", 50), ("s1", 1), ("s2", 1)],
                 [("s0", 1), ("s1", 63), ("s3", 2)],
                 [("s3", 90), ("s0", 78), ("s1", 1)],
@@ -154,7 +156,7 @@ def test_unequal_batches_and_used_pages_and_slots(models, name, device, dtype):
 
 @pytest.mark.parametrize("device,dtype", WHERE)
 def test_long_decoding(models, device, dtype):
-    toks, want = expected(models, "mixed", 330, 40)
+    toks, want = expected(models, "mixed", dtype, 330, 40)
     r = replay(models, "mixed", device, dtype, 330)
     got = nc.run_schedule(r, {"a": toks}, [[("a", 20)]] + [[("a", 1)]] * 310)["a"]
     check(got, want, dtype)
@@ -166,7 +168,7 @@ def test_long_decoding(models, device, dtype):
 def test_greedy_generation_through_the_scheduler(models, device, dtype):
     """Concurrent requests of unequal length, prompts cut into chunks, a resumed prefix: the tokens of the plain
     implementation's greedy continuation."""
-    cfg, w, path = models["mixed"]
+    cfg, w, path = models["mixed", dtype]
     mc, lw, tok, _ = load_model(path, device, getattr(torch, dtype))
     eng = LmEngine(Decoder(mc, lw, None, max_position=264), tok,
                    EngineConfig(ctx_size=256, max_seqs=3, block_size=16, prefill_chunk=24, max_batch_tokens=40,
@@ -232,8 +234,8 @@ def test_sampled_generation_on_gpu():
 @gpu
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 def test_trace_run_program(models, tmp_path, dtype):
-    cfg, w, path = models["mixed"]
-    toks, want = expected(models, "mixed", 66, 11)
+    cfg, w, path = models["mixed", dtype]
+    toks, want = expected(models, "mixed", dtype, 66, 11)
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:40], "want": [0, 39]}], "end": []},
              {"step": 1, "entries": [{"id": "x", "tokens": toks[40:65], "want": []}], "end": []},
