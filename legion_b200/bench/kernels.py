@@ -380,6 +380,128 @@ def bench_gdn(rows):
         print(rows[-1], flush=True)
 
 
+def bench_linear(rows):
+    """Linear-attention state with a scalar decay (constant per head; selective as in Mamba-2) beside the recurrent
+    kernels of the other families, over a prompt and over decode steps. frac_hbm: bytes the operands and the state must
+    move once, over the measured copy bandwidth."""
+    from legion_b200.ops import sm100
+    hbm, _, src = peaks()
+
+    def row(kernel, n_seq, L, ms, byts, launches=None):
+        rows.append(dict(kernel=kernel, n_seq=n_seq, L=L, us=round(ms * 1e3, 2), mbytes=round(byts / 1e6, 1),
+                         frac_hbm=round(byts / ms / 1e6 / hbm, 3), peaks=src))
+        print(rows[-1], flush=True)
+    for n_seq, L in (CASE["attn"] or ((1, 8192), (16, 1), (64, 1))):
+        T = n_seq * L
+        cu = torch.arange(0, (n_seq + 1) * L, L, device="cuda", dtype=torch.int32)
+        cu_host = list(range(0, (n_seq + 1) * L, L))
+        slots = torch.arange(n_seq, device="cuda", dtype=torch.int32)
+        rnd = lambda *s: (torch.randn(*s, device="cuda") * 0.3).bfloat16()          # noqa: E731
+        tm = timeit if L > 1 else timeit_graph
+        # Lightning attention, 16 heads of 128 x 128
+        H, N, P = 16, 128, 128
+        proj = rnd(T, 4 * H * N)
+        st = torch.zeros(n_seq, H, P, N, device="cuda")
+        dec = torch.full((H,), 0.99, device="cuda")
+        q, k, v, g = (proj[:, i * H * N:(i + 1) * H * N] for i in range(4))
+        scan = lambda: sm100.linear_scan(q, k, v, st, cu, slots, H, H, N, P, decay=dec, silu_in=True, max_len=L,   # noqa: E731
+                                         cu_host=cu_host)
+        row("linear_scan constant 16x128x128", n_seq, L, tm(scan), T * 4 * H * N * 2 + st.numel() * 8)
+        o, w = scan(), torch.ones(H * P, device="cuda")
+        row("group_norm_gate 2048", n_seq, L, tm(lambda: sm100.group_norm_gate(o, g, w, 1e-5)), T * H * P * 6)
+        # Mamba-2, 64 heads of 64, state 128, 8 groups
+        H, N, P, G = 64, 128, 64, 8
+        C = H * P + 2 * G * N
+        proj = rnd(T, H * P + C + H)
+        z, xbc, dt = proj[:, :H * P], proj[:, H * P:H * P + C], proj[:, H * P + C:]
+        st = torch.zeros(n_seq, H, P, N, device="cuda")
+        conv = torch.zeros(n_seq, C, 3, device="cuda")
+        cw, cb = torch.randn(C, 4, device="cuda"), torch.zeros(C, device="cuda")
+        A, D, db = (-torch.ones(H, device="cuda") for _ in range(3))
+        ssd_bytes = T * (2 * H * P + C + H) * 2 + st.numel() * 8
+        c = sm100.causal_conv1d_silu(xbc, cw, cb, conv, cu, slots, max_len=L)
+        if L == 1:
+            row("ssd_decode 64x64x128 (with convolution)", n_seq, L,
+                tm(lambda: sm100.ssd_decode(xbc, cw, cb, conv, dt, db, A, D, z, st, cu, slots, H, G, N, P)),
+                ssd_bytes + conv.numel() * 8)
+        else:
+            row("linear_scan selective 64x64x128", n_seq, L,
+                tm(lambda: sm100.linear_scan(c[:, H * P + G * N:], c[:, H * P:H * P + G * N], c[:, :H * P], st, cu, slots,
+                                             H, G, N, P, dt=dt, dt_bias=db, A=A, D=D, z=z, max_len=L, cu_host=cu_host)),
+                ssd_bytes)
+            row("conv1d_silu", n_seq, L, tm(lambda: sm100.causal_conv1d_silu(xbc, cw, cb, conv, cu, slots, max_len=L)),
+                T * C * 4)
+        st2 = torch.zeros(n_seq, H, P, N, device="cuda")
+        row("mamba2_scan 64x64x128 (Nemotron-H)", n_seq, L,
+            tm(lambda: sm100.mamba2_scan(c, dt, z, A, D, db, st2, cu, slots, H, P, G, N)), ssd_bytes)
+        # Gated DeltaNet, 16 heads of 128 x 128
+        H = 16
+        qkv = rnd(T, 3 * H * 128)
+        gg, beta = -torch.rand(T, H, device="cuda") * 0.1, torch.rand(T, H, device="cuda")
+        st = torch.zeros(n_seq, H, 128, 128, device="cuda")
+        gdn_bytes = T * 4 * H * 128 * 2 + st.numel() * 8
+        if L > 1:
+            row("gdn chunked 16x128x128", n_seq, L,
+                tm(lambda: sm100.gdn_recurrent(qkv, gg, beta, st, cu, slots, H, H, 128, 128, False, 128 ** -0.5,
+                                               cu_host=cu_host)), gdn_bytes)
+        else:
+            pj = rnd(T, 4 * H * 128 + 2 * H)
+            cw, hist = torch.randn(3 * H * 128, 4, device="cuda"), torch.zeros(n_seq, 3 * H * 128, 3, device="cuda")
+            one = torch.ones(128, device="cuda")
+            row("gdn_decode_fused 16x128x128 (convolution, norm and gate included)", n_seq, L,
+                tm(lambda: sm100.gdn_decode_fused(pj, cw, hist, -one[:H], one[:H], one, 1e-6, "silu", st, slots, H, H, 128,
+                                                  128, False, 128 ** -0.5)), T * 5 * H * 128 * 2 + st.numel() * 8 + hist.numel() * 8)
+
+
+def bench_hyper(rows):
+    """The stream update of hyper-connections (4 fp32 streams, next input and norm included) beside the residual + RMS
+    norm launch of the other families."""
+    from legion_b200.ops import sm100
+    hbm, _, src = peaks()
+    S, H = 4, 2048
+    for T in CASE["tokens"] or (16, 64, 1024, 8192):
+        X, y = torch.randn(T, S, H, device="cuda"), torch.randn(T, H, device="cuda").bfloat16()
+        mix, v, w = torch.eye(S, device="cuda"), torch.ones(S, device="cuda"), torch.zeros(H, device="cuda")
+        tm = timeit_graph if T <= 64 else timeit
+        for name, fn, byts in (
+                ("hyper_step 4x2048", lambda: sm100.hyper_step(X, [(y, 1.0)], mix, v, v, w, 1e-5, 1.0),
+                 T * H * (S * 8 + 4)),
+                ("residual + rmsnorm 2048", lambda: sm100.rmsnorm(y, w, 1e-5, 1.0, y), T * H * 8)):
+            ms = tm(fn)
+            rows.append(dict(kernel=name, T=T, us=round(ms * 1e3, 2), frac_hbm=round(byts / ms / 1e6 / hbm, 3), peaks=src))
+            print(rows[-1], flush=True)
+
+
+def bench_attn_sizes(rows):
+    """Attention with key and value heads of different sizes, windowed and not, beside equal sizes: prompts by FLOPs of
+    the visible scores, decode by the bytes of the visible keys and values."""
+    from legion_b200.ops import sm100
+    hbm, tf, src = peaks()
+    Hq, Hkv, page = 16, 4, 64
+    for n_seq, L, ctx in ((1, 8192, 8192), (16, 1, 8192)):
+        for dk, dv in ((128, 128), (96, 192), (64, 128), (128, 64)):
+            for window in (0, 1024):
+                nb = n_seq * (ctx // page)
+                kc = torch.randn(nb, page, Hkv, dk, device="cuda").bfloat16()
+                vc = torch.randn(nb, page, Hkv, dv, device="cuda").bfloat16()
+                bt = torch.arange(nb, device="cuda", dtype=torch.int32).view(n_seq, -1)
+                q = torch.randn(n_seq * L, Hq, dk, device="cuda").bfloat16()
+                cl = torch.full((n_seq,), ctx, device="cuda", dtype=torch.int32)
+                seen = ctx if not window else min(window, ctx)
+                r = dict(kernel="prefill_attn" if L > 1 else "paged_decode", n_seq=n_seq, ctx=ctx, heads=(Hq, Hkv, dk, dv),
+                         window=window, peaks=src)
+                if L > 1:
+                    cu = torch.arange(0, (n_seq + 1) * L, L, device="cuda", dtype=torch.int32)
+                    ms = timeit(lambda: sm100.prefill_attn(q, kc, vc, cu, cl, bt, L, dk ** -0.5, window), iters=5)
+                    pairs = L * seen - seen * (seen - 1) / 2 if window else L * (L + 1) / 2
+                    r.update(us=round(ms * 1e3, 1), frac_tflops=round(2.0 * n_seq * pairs * (dk + dv) * Hq / ms / 1e9 / tf, 3))
+                else:
+                    ms = timeit_graph(lambda: sm100.paged_decode(q, kc, vc, bt, cl, dk ** -0.5, window, max_ctx=ctx))
+                    r.update(us=round(ms * 1e3, 1), frac_hbm=round(n_seq * seen * Hkv * (dk + dv) * 2 / ms / 1e6 / hbm, 3))
+                rows.append(r)
+                print(r, flush=True)
+
+
 def bench_gemm(rows):
     from legion_b200.ops import sm100
     hbm, tf, src = peaks()
@@ -476,7 +598,7 @@ def main(argv=None):
     if a.gemm:
         CASE["gemm"] = [tuple(int(y) for y in x.split("x")) for x in a.gemm.split(",")]
     rows = []
-    table = {"moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
+    table = {"linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
     for name in a.only.split(","):
         table[name](rows)
     from legion_b200.ops.sm100 import Workspace

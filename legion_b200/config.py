@@ -492,7 +492,16 @@ def nisasun_3b() -> ModelConfig:
                        hyper_mode="static", layers=layers)
 
 
+def hybrid_4b() -> ModelConfig:
+    """A Gated DeltaNet / gated attention hybrid of the size of ``nisasun_3b``: what that design is compared with."""
+    return ModelConfig(arch="qwen35moe", n_layer=24, hidden=2048, vocab=65536, n_head=16, n_kv_head=4, head_dim=128,
+                       rope_dim=64, full_attention_interval=2, gated_attn=True, gdn_k_heads=16, gdn_v_heads=32,
+                       gdn_k_dim=128, gdn_v_dim=128, first_dense_layers=12, dense_ff=6144, n_expert=32, top_k=4,
+                       expert_ff=1024)
+
+
 PRESETS = {
+    "hybrid-4b": hybrid_4b,
     "tiny-nisasun": tiny_nisasun,
     "nisasun-3b": nisasun_3b,
     "tiny-muse": tiny_muse,
