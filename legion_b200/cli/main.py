@@ -547,7 +547,7 @@ def cmd_ep_place(a):
 
 
 def cmd_completions(a):
-    subs = ["serve", "run", "bench", "chat", "top", "gguf", "st", "info", "tokenize", "logits", "ep-place", "completions",
+    subs = ["serve", "run", "bench", "chat", "top", "gguf", "st", "info", "tokenize", "logits", "trace", "ep-place", "completions",
             "kernel-bench", "comm-bench"]
     if a.shell == "bash":
         print("complete -W '" + " ".join(subs) + "' legion")

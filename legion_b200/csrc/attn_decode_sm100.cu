@@ -67,9 +67,10 @@ struct DecodeTcCfg {
   static constexpr int V_BYTES = VHALVES * BKV * 128;
   static constexpr int Q_BYTES = HALVES * NQ * 128;
   static constexpr int P_BYTES = 2 * NQ * 128;
-  static constexpr int K_STAGES = DK <= 64 ? 4 : (DK <= 128 ? 3 : 2);
-  static constexpr int V_STAGES = DV <= 64 ? 4 : (DV <= 128 ? (DK <= 128 ? 3 : 2) : 1);
-  static constexpr int MT = DV <= 128 ? 1 : DV / 128;       // 128-row M tiles of O^T
+  // as many stages as 224 KB hold, keys and values alike where both fit
+  static constexpr int K_STAGES = DK <= 64 ? 4 : (DK <= 128 ? (DV <= 192 ? 3 : 2) : 2);
+  static constexpr int V_STAGES = DV <= 64 ? 4 : (DV <= 128 ? (DK <= 128 ? 3 : 2) : (DK <= 128 ? 2 : 1));
+  static constexpr int MT = (DV + 127) / 128;       // 128-row M tiles of O^T
   static constexpr int TMEM_COLS = (2 * NQ + 2 * MT * NQ <= 64) ? 64 : 128;   // S x 2 + O x 2 (MT x 16 each)
   static constexpr int SMEM = K_STAGES * K_BYTES + V_STAGES * V_BYTES + Q_BYTES + 2 * P_BYTES + 1024 + 1536;
   static_assert(2 * NQ + 2 * MT * NQ <= TMEM_COLS, "accumulators do not fit the TMEM allocation");
@@ -255,7 +256,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             for (int k = 0; k < BKV / 16; ++k) {
               // A = V^T rows [mt*128, mt*128+128) of d: two 64-wide MN groups, LBO apart; DV = 64 reads the
               // only group twice (LBO 0) and the duplicate lanes are never stored.
-              const uint32_t lbo = (DV == 64) ? 0u : uint32_t(BKV * 128);
+              // (the last tile of an odd number of groups likewise)
+              const uint32_t lbo = (DV < mt * 128 + 128) ? 0u : uint32_t(BKV * 128);
               const uint64_t da = umma_desc_mn_sw128(va + mt * 2 * (BKV * 128) + k * 16 * 128, lbo, 1024);
               const uint64_t db = umma_desc_k_sw128(pa + (k / 4) * (NQ * 128) + (k % 4) * 32);
               umma_f16(tmem_O + (wgp * MT + mt) * NQ, da, db, idesc_o, ((i >> 1) | k) ? 1u : 0u);
@@ -530,7 +532,7 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || k_cell % 8 || v_cell % 8 || page <= 0 ||
       128 % page != 0 || page % 8 != 0 || Hq % Hkv)
     return -1;
-  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : 256);
+  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : (dv <= 192 ? 192 : 256));
   const int G = Hq / Hkv;
   const int gtiles = (G + 15) / 16;
   if (n_splits < 1 || n_splits > 128 || long(B) * Hkv * gtiles > n_group_ctr) return -1;
@@ -552,7 +554,7 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   dim3 grid(Hkv * gtiles, B, n_splits);
 #define LB_DIM(K_, V_) if (DK == K_ && DV == V_) return launch_decode_tc<K_, V_>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64) LB_DIM(128, 128) LB_DIM(256, 256) LB_DIM(64, 128) LB_DIM(64, 256) LB_DIM(128, 64) LB_DIM(128, 256)
-  LB_DIM(256, 64) LB_DIM(256, 128)
+  LB_DIM(256, 64) LB_DIM(256, 128) LB_DIM(64, 192) LB_DIM(128, 192) LB_DIM(256, 192)
 #undef LB_DIM
   return -1;
 }

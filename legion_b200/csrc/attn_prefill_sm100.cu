@@ -241,6 +241,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         for (int h = 0; h < Cfg::HALVES; ++h) {
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
+            if (h * 64 + k * 16 >= a.dk) break;       // the rest of the padded head is zeros
             const uint64_t da = umma_desc_k_sw128(qa + h * (128 * 128) + k * 32);
             const uint64_t db = umma_desc_k_sw128(ka + h * (BKV * 128) + k * 32);
             umma_f16(ts, da, db, idesc_s, (h | k) ? 1u : 0u);
@@ -527,7 +528,7 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
                         int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, int window,
                         int causal, void* out, int* status, cudaStream_t s) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
-  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : 256);
+  const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : (dv <= 192 ? 192 : 256));
   const int BKV = (DK >= 128 || DV >= 128) ? 64 : 128;
   if (page <= 0 || BKV % page != 0 || page % 8 != 0) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: page size %d must be a multiple of 8 dividing %d",
@@ -557,7 +558,8 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
   dim3 grid((max_q_len + 127) / 128, Hq, n_seqs);
 #define LB_DIM(K_, V_, B_) if (DK == K_ && DV == V_) return launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64, 128) LB_DIM(128, 128, 64) LB_DIM(256, 256, 64)
-  LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64) LB_DIM(256, 128, 64)
+  LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64)
+  LB_DIM(64, 192, 64) LB_DIM(128, 192, 64) LB_DIM(256, 192, 64) LB_DIM(256, 128, 64)
 #undef LB_DIM
   return 1;
 }

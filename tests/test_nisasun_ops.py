@@ -96,7 +96,8 @@ def windowed(q, k, v, scale, window):
 
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 96, 128), (6, 3, 40, 72), (2, 2, 64, 256), (3, 1, 136, 24), (2, 1, 13, 19),
-                                       (16, 1, 128, 128), (4, 4, 256, 64)])
+                                       (16, 1, 128, 128), (4, 4, 256, 64), (4, 2, 120, 192), (2, 1, 40, 136),
+                                       (2, 2, 168, 184)])
 def test_windowed_attention_prompts_and_decode(device, dtype, H, G, dk, dv):
     lens, qlens = [200, 64, 1, 131], [70, 64, 1, 2]
     k = [rnd(n, G, dk, seed=i, dtype=dtype) for i, n in enumerate(lens)]
