@@ -10,6 +10,12 @@ namespace {
 using torch::Tensor;
 using OptT = c10::optional<Tensor>;
 
+// text of the launch error behind a failed call, if there is one
+std::string cuda_error() {
+  const cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? std::string() : std::string(" (") + cudaGetErrorString(e) + ")";
+}
+
 cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
 
 template <typename T>
@@ -129,7 +135,7 @@ void bind_layers(pybind11::module_& m) {
     a.c0 = float(c0); a.c1 = float(c1); a.y_rows = int(y_rows);
     a.h = h.data_ptr(); a.ldh = h.stride(0); a.rows = int(R); a.S = int(S); a.H = int(H);
     c10::cuda::CUDAGuard guard(h.device());
-    TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "hyper_step: at most 16 streams of 51200 columns");
+    TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "hyper_step: at most 16 streams of 51200 columns", cuda_error());
   });
   m.def("sgemm", [](const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, const OptT& tok_scale,
                     const OptT& out_rows, int64_t n_feat, bool dual, int64_t dual_offset, int64_t act,
@@ -155,7 +161,7 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(!a.tile_group || (a.tile_tok0 && a.tile_ntok && a.n_tiles), "sgemm: incomplete tile tables");
     TORCH_CHECK(a.tile_group || x.size(0) >= n_tok, "sgemm: too few rows");
     c10::cuda::CUDAGuard guard(x.device());
-    TORCH_CHECK(lb::sgemm_launch(a, f32, cur_stream()) == 0, "sgemm failed");
+    TORCH_CHECK(lb::sgemm_launch(a, f32, cur_stream()) == 0, "sgemm failed", cuda_error());
   });
   m.def("qkv_norm_append", [](const Tensor& q, const Tensor& k, const Tensor& v, const OptT& qw, const OptT& kw, double eps,
                               const Tensor& slots, Tensor& q_out, Tensor& k_cache, Tensor& v_cache) {
@@ -178,7 +184,7 @@ void bind_layers(pybind11::module_& m) {
                                            optp<float>(kw), float(eps), reinterpret_cast<const long*>(slots.data_ptr()),
                                            q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
                                            int(T), int(Hq), int(Hkv), int(DK), int(DV), f32, cur_stream()) == 0,
-                "qkv_norm_append failed");
+                "qkv_norm_append failed", cuda_error());
   });
   m.def("paged_attn_general", [](const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
                                  const Tensor& ctx_lens, const Tensor& block_table, double scale, int64_t window,
@@ -199,7 +205,7 @@ void bind_layers(pybind11::module_& m) {
                                               int(block_table.stride(0)), int(k_cache.size(-3)), int(ctx_lens.numel()),
                                               int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), int(window),
                                               out.data_ptr(), f32, cur_stream()) == 0,
-                "paged_attn_general: value heads of at most 512 columns, key heads of at most 2560");
+                "paged_attn_general: value heads of at most 512 columns, key heads of at most 2560", cuda_error());
   });
   m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
                           const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state, const Tensor& cu,
@@ -207,7 +213,7 @@ void bind_layers(pybind11::module_& m) {
     const auto a = scan_args(q, k, v, silu_in, decay, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, write_state);
     c10::cuda::CUDAGuard guard(q.device());
     TORCH_CHECK(lb::linear_scan_launch(a, q.scalar_type() == at::kFloat, cur_stream()) == 0,
-                "linear scan: at most 512 state columns, heads a multiple of the groups");
+                "linear scan: at most 512 state columns, heads a multiple of the groups", cuda_error());
   });
   m.def("ssd_decode", [](const Tensor& xbc, const Tensor& conv_w, const OptT& conv_b, Tensor& conv_state, const Tensor& dt,
                          const Tensor& dt_bias, const Tensor& A, const OptT& D, const OptT& z, Tensor& state,
@@ -228,7 +234,7 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(ctr.numel() >= n * G && ctr.element_size() == 4 && ctr.is_contiguous(), "ssd_decode: counters [n, G]");
     a.ctr = reinterpret_cast<unsigned int*>(ctr.data_ptr());
     c10::cuda::CUDAGuard guard(xbc.device());
-    TORCH_CHECK(lb::ssd_decode_launch(a, xbc.scalar_type() == at::kFloat, cur_stream()) == 0, "ssd_decode: unsupported sizes");
+    TORCH_CHECK(lb::ssd_decode_launch(a, xbc.scalar_type() == at::kFloat, cur_stream()) == 0, "ssd_decode: unsupported sizes", cuda_error());
   });
   m.def("linear_chunk_ok", [](int64_t N, int64_t P) { return lb::linear_chunk_ok(int(N), int(P)); });
   m.def("linear_chunk_scratch_bytes", [](int64_t n_chunks, int64_t H, int64_t N, int64_t P) {
@@ -249,7 +255,7 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::linear_chunk_launch(a, tb, tb + n_chunks, tb + 2 * n_chunks, int(n_chunks), tb + 3 * n_chunks,
                                         tb + 3 * n_chunks + a.n_seqs, scratch.data_ptr(),
                                         reinterpret_cast<int*>(status.data_ptr()), cur_stream()) == 0,
-                "linear_chunk: unsupported sizes");
+                "linear_chunk: unsupported sizes", cuda_error());
   });
   m.def("group_norm_gate", [](const Tensor& y, const OptT& gate, const Tensor& w, double eps, int64_t groups, Tensor& out) {
     const bool f32 = is_f32(y, "y");
@@ -265,7 +271,7 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::group_norm_gate_launch(y.data_ptr(), y.stride(0), gate.has_value() ? gate->data_ptr() : nullptr,
                                            gate.has_value() ? gate->stride(0) : 0, w.data_ptr<float>(), float(eps),
                                            int(groups), int(C), int(R), out.data_ptr(), out.stride(0), f32, cur_stream()) == 0,
-                "group_norm_gate failed");
+                "group_norm_gate failed", cuda_error());
   });
   m.def("conv1d_silu", [](const Tensor& x, const Tensor& w, const OptT& bias, Tensor& conv_state, const Tensor& cu_seq,
                           const Tensor& slots, Tensor& out, bool write_state, int64_t max_len) {
@@ -291,6 +297,6 @@ void bind_layers(pybind11::module_& m) {
                                          conv_state.data_ptr<float>(), cu.data_ptr<int>(), slots.data_ptr<int>(),
                                          int(slots.numel()), int(T), int(C), int(KC), out.data_ptr(), out.stride(0),
                                          write_state, f32, cur_stream()) == 0,
-                "conv_silu_any: at most 65535 tokens per step");
+                "conv_silu_any: at most 65535 tokens per step", cuda_error());
   });
 }

@@ -10,6 +10,7 @@ Reference counterpart: kept graphs per ``GroupShape`` and stage CUDA graphs with
 """
 from __future__ import annotations
 
+import gc
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -44,7 +45,6 @@ class DecodeGraphs:
 
     def release(self):
         """Destroys every captured graph and its private memory pool."""
-        import gc
         if self.entries and torch.cuda.is_available():
             torch.cuda.synchronize(self.eng.device)
         self.entries.clear()
@@ -154,21 +154,30 @@ class DecodeGraphs:
         torch.cuda.synchronize(dev)
         g = torch.cuda.CUDAGraph()
         side = [torch.cuda.Stream(device=dev) for _ in range(lanes - 1)]
-        with torch.cuda.graph(g):
-            main = torch.cuda.current_stream(dev)
-            if lanes > 1:
-                fork = torch.cuda.Event()
-                fork.record(main)
-            out = run_lane(0)
-            for i, st in enumerate(side):
-                st.wait_event(fork)
-                with torch.cuda.stream(st):
-                    run_lane(i + 1)
-                    join = torch.cuda.Event()
-                    join.record(st)
-                main.wait_event(join)
-            if lanes == 1 and eng.model.head_split is None:
-                e.logits = out.logits
+        # a collection in the middle of the capture could destroy another engine's graphs or pinned buffers, which
+        # invalidates it: collect before, and hold the collector back meanwhile
+        gc.collect()
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(g):
+                main = torch.cuda.current_stream(dev)
+                if lanes > 1:
+                    fork = torch.cuda.Event()
+                    fork.record(main)
+                out = run_lane(0)
+                for i, st in enumerate(side):
+                    st.wait_event(fork)
+                    with torch.cuda.stream(st):
+                        run_lane(i + 1)
+                        join = torch.cuda.Event()
+                        join.record(st)
+                    main.wait_event(join)
+                if lanes == 1 and eng.model.head_split is None:
+                    e.logits = out.logits
+        finally:
+            if collecting:
+                gc.enable()
         e.graph = g
         self.entries[B] = e
         return e
