@@ -9,9 +9,10 @@ Configurations (``--config``):
      DeltaNet to gated attention, 512 experts top-10 + shared expert, 1K-token prompts for the decode rows.
   2  30B-A3B-shape MoE in bf16: 48 layers, 128 experts top-8, 8K-token prompts.
   5  dense 27B-shape model in bf16, 1K-token prompts.
-  6  Nisasun at 3.9B parameters in bf16 (24 layers, hyper-connections, linear attention / attention beside Mamba-2).
+  6  Nisasun at 4B parameters in bf16 (24 layers, hyper-connections, linear attention / attention beside Mamba-2).
   7  the closest hybrid of the other families at that size: 24 layers of Gated DeltaNet and gated attention in turn,
      dense and 32-expert feed-forward parts, bf16 (the comparison for 6).
+  8, 9  the same pair at 13B parameters (20 layers, 4096 columns).
 The ONE parsed number (``value``) is decode tokens/s at 16 users of the selected configuration; the other rows of
 the grid (1 and 64 users, 32K prefill) are under ``extra``.
 
@@ -95,8 +96,10 @@ CONFIGS = {
     4: dict(model="deepseek-671b", prompt_len=1024, weights="fp8",
             dtype="fp8 (block-scaled e4m3 weights, e4m3 activations on the projections and experts), bf16 elsewhere"),
     5: dict(model="dense-27b", prompt_len=1024, weights="bf16", dtype="bf16"),
-    6: dict(model="nisasun-3b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    6: dict(model="nisasun-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
     7: dict(model="hybrid-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    8: dict(model="nisasun-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    9: dict(model="hybrid-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
 }
 
 

@@ -477,33 +477,56 @@ def tiny_nisasun() -> ModelConfig:
                                                                                           keep_group=1, **moe))])
 
 
-def nisasun_3b() -> ModelConfig:
-    """Nisasun with layers the size of a small production model (random weights; speed measurements): 2048 wide, four
-    streams, alternating linear-attention layers (16 heads of 128 x 128) and parallel layers (16 query / 4 key heads of
-    128, window 1024, beside 64 Mamba-2 heads of 64 with state 128), dense and 32-expert feed-forward parts in turn."""
-    decay = [1.0 - 2.0 ** -(2 + 0.5 * h) for h in range(16)]
-    moe = MoeSpec(32, 4, 1024, router="softmax_bias", correction=True, renorm=False, n_group=8, keep_group=4, group_top=1)
+def _nisasun(n_layer: int, hidden: int, heads: int, ssm_heads: int, ff: int, expert_ff: int, attn_dims) -> ModelConfig:
+    """Alternating parallel layers (attention of ``heads`` query heads with window 1024 beside Mamba-2 heads of 64 with
+    state 128) and linear-attention layers (``heads`` heads of 128 x 128), four streams, dense and 32-expert
+    feed-forward parts in turn."""
+    decay = [1.0 - 2.0 ** -(2 + 8.0 * h / heads) for h in range(heads)]
+    moe = MoeSpec(32, 4, expert_ff, router="softmax_bias", correction=True, renorm=False, n_group=8, keep_group=4,
+                  group_top=1)
+    dk, dv = attn_dims
     layers = []
-    for il in range(24):
-        mixer = (ParallelSpec(AttnSpec(16, 4, 128, 128, 128 ** -0.5, window=1024), SsdSpec(64, 64, 128, 8, 4, 8), 0.5, 0.5)
-                 if il % 2 == 0 else LightningSpec(16, 128, 128, decay))
-        layers.append(LayerSpec(mixer, moe if il % 2 else DenseSpec(6144, "gelu_tanh")))
-    return ModelConfig(arch="nisasun", hidden=2048, vocab=65536, rms_eps=1e-5, norm_offset=1.0, hyper_streams=4,
+    for il in range(n_layer):
+        mixer = (ParallelSpec(AttnSpec(heads, heads // 4, dk, dv, dk ** -0.5, window=1024),
+                              SsdSpec(ssm_heads, 64, 128, 8, 4, 8), 0.5, 0.5)
+                 if il % 2 == 0 else LightningSpec(heads, 128, 128, decay))
+        layers.append(LayerSpec(mixer, moe if il % 2 else DenseSpec(ff, "gelu_tanh")))
+    return ModelConfig(arch="nisasun", hidden=hidden, vocab=65536, rms_eps=1e-5, norm_offset=1.0, hyper_streams=4,
                        hyper_mode="static", layers=layers)
 
 
+def nisasun_4b() -> ModelConfig:
+    """Nisasun with layers the size of a small production model (random weights; speed measurements)."""
+    return _nisasun(24, 2048, 16, 64, 6144, 1024, (128, 128))
+
+
+def nisasun_13b() -> ModelConfig:
+    """The same at 4096 columns, with query / key heads of 96 and value heads of 192."""
+    return _nisasun(20, 4096, 32, 128, 12288, 2048, (96, 192))
+
+
+def _hybrid(n_layer: int, hidden: int, heads: int, ff: int, expert_ff: int) -> ModelConfig:
+    """A Gated DeltaNet / gated attention hybrid of the size of a ``_nisasun`` stack: what that design is compared with."""
+    return ModelConfig(arch="qwen35moe", n_layer=n_layer, hidden=hidden, vocab=65536, n_head=heads, n_kv_head=heads // 4,
+                       head_dim=128, rope_dim=64, full_attention_interval=2, gated_attn=True, gdn_k_heads=heads,
+                       gdn_v_heads=2 * heads, gdn_k_dim=128, gdn_v_dim=128, first_dense_layers=n_layer // 2, dense_ff=ff,
+                       n_expert=32, top_k=4, expert_ff=expert_ff)
+
+
 def hybrid_4b() -> ModelConfig:
-    """A Gated DeltaNet / gated attention hybrid of the size of ``nisasun_3b``: what that design is compared with."""
-    return ModelConfig(arch="qwen35moe", n_layer=24, hidden=2048, vocab=65536, n_head=16, n_kv_head=4, head_dim=128,
-                       rope_dim=64, full_attention_interval=2, gated_attn=True, gdn_k_heads=16, gdn_v_heads=32,
-                       gdn_k_dim=128, gdn_v_dim=128, first_dense_layers=12, dense_ff=6144, n_expert=32, top_k=4,
-                       expert_ff=1024)
+    return _hybrid(24, 2048, 16, 6144, 1024)
+
+
+def hybrid_13b() -> ModelConfig:
+    return _hybrid(20, 4096, 32, 12288, 2048)
 
 
 PRESETS = {
     "hybrid-4b": hybrid_4b,
+    "hybrid-13b": hybrid_13b,
     "tiny-nisasun": tiny_nisasun,
-    "nisasun-3b": nisasun_3b,
+    "nisasun-4b": nisasun_4b,
+    "nisasun-13b": nisasun_13b,
     "tiny-muse": tiny_muse,
     "tiny-gemma4": tiny_gemma4,
     "tiny-nemotron-h-moe": tiny_nemotron_h_moe,

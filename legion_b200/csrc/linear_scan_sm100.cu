@@ -53,6 +53,16 @@ struct ChunkArgs {
 
 __device__ __forceinline__ float silu_fast(float z) { return z / (1.f + __expf(-z)); }
 
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+  const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 f = __bfloat1622float2(p[j]);
+    v[2 * j] = f.x;
+    v[2 * j + 1] = f.y;
+  }
+}
+
 // Eight columns of a row as floats (zeros outside), activation applied and rounded to bf16 where the layer has one.
 __device__ __forceinline__ void load8(const __nv_bfloat16* row, int col, int width, bool row_ok, bool vec, bool silu,
                                       float (&v)[8]) {
@@ -60,14 +70,7 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* row, int col, int wid
   for (int j = 0; j < 8; ++j) v[j] = 0.f;
   if (!row_ok || col >= width) return;
   if (vec && col + 8 <= width) {
-    const uint4 u = __ldg(reinterpret_cast<const uint4*>(row + col));
-    const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float2 f = __bfloat1622float2(p[j]);
-      v[2 * j] = f.x;
-      v[2 * j + 1] = f.y;
-    }
+    unpack8(__ldg(reinterpret_cast<const uint4*>(row + col)), v);
   } else {
 #pragma unroll
     for (int j = 0; j < 8; ++j)
@@ -94,17 +97,54 @@ __device__ __forceinline__ uint4 split8(float (&v)[8]) {
   return hi;
 }
 
-// [128 token rows] x [HALVES * 64 columns] into K-major 128-byte-swizzled halves
+// A [128 token rows] x [HALVES * 64 columns] tile, eight columns of a row at a time: put(row, byte offset in the
+// K-major 128-byte-swizzled tile, values). With aligned rows all of a thread's loads are issued before the first is used.
+template <int HALVES, typename Put>
+__device__ __forceinline__ void each8(const __nv_bfloat16* src, long ld, int width, int nval, bool vec, bool silu, Put put) {
+  constexpr int IT = C * HALVES * 8 / 256;
+  auto at = [](int i, int& row, int& c8) {
+    const int e = threadIdx.x + 256 * i;
+    row = e / (HALVES * 8);
+    c8 = e % (HALVES * 8);
+  };
+  auto off = [](int row, int c8) { return (c8 >> 3) * HALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4); };
+  if (vec) {
+    uint4 raw[IT];
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      int row, c8;
+      at(i, row, c8);
+      raw[i] = (row < nval && c8 * 8 < width) ? __ldg(reinterpret_cast<const uint4*>(src + long(row) * ld + c8 * 8))
+                                              : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      int row, c8;
+      at(i, row, c8);
+      float v[8];
+      unpack8(raw[i], v);
+      if (silu) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = silu_fast(v[j]);
+      }
+      put(row, off(row, c8), v);
+    }
+  } else {
+#pragma unroll 1
+    for (int i = 0; i < IT; ++i) {
+      int row, c8;
+      at(i, row, c8);
+      float v[8];
+      load8(src + long(row) * ld, c8 * 8, width, row < nval, false, silu, v);
+      put(row, off(row, c8), v);
+    }
+  }
+}
 template <int HALVES>
 __device__ __forceinline__ void load_tile(uint8_t* dst, const __nv_bfloat16* src, long ld, int width, int nval, bool vec,
                                           bool silu) {
-#pragma unroll 4
-  for (int i = threadIdx.x; i < C * HALVES * 8; i += 256) {
-    const int row = i / (HALVES * 8), c8 = i % (HALVES * 8);
-    float v[8];
-    load8(src + long(row) * ld, c8 * 8, width, row < nval, vec, silu, v);
-    *reinterpret_cast<uint4*>(dst + (c8 >> 3) * HALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4)) = pack8(v);
-  }
+  each8<HALVES>(src, ld, width, nval, vec, silu,
+                [&](int, int off, float (&v)[8]) { *reinterpret_cast<uint4*>(dst + off) = pack8(v); });
 }
 
 // log2 of a constant decay; decays sit close to 1, where log1p keeps the relative accuracy that a plain logarithm loses
@@ -188,18 +228,13 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs a) {
   const auto* vp = static_cast<const __nv_bfloat16*>(L.v) + long(t0) * L.ldv + long(h) * L.P + p0;
   const auto* kp = static_cast<const __nv_bfloat16*>(L.k) + long(t0) * L.ldk + long(g) * L.N;
   load_tile<PH>(v_s, vp, L.ldv, L.P - p0, nval, a.vec_v, L.silu_in);
-#pragma unroll 2
-  for (int i = threadIdx.x; i < C * NH * 8; i += 256) {
-    const int row = i / (NH * 8), c8 = i % (NH * 8);
-    float v[8];
-    load8(kp + long(row) * L.ldk, c8 * 8, L.N, row < nval, a.vec_k, L.silu_in, v);
+  each8<NH>(kp, L.ldk, L.N, nval, a.vec_k, L.silu_in, [&](int row, int off, float (&v)[8]) {
     const float f = exp2f(cC - cs[row]) * ws[row];
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[j] = (L.silu_in ? __bfloat162float(__float2bfloat16(v[j])) : v[j]) * f;
-    const int off = (c8 >> 3) * HALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4);
     *reinterpret_cast<uint4*>(kh_s + off) = split8(v);
     *reinterpret_cast<uint4*>(kl_s + off) = pack8(v);
-  }
+  });
   fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
@@ -371,28 +406,42 @@ __global__ void __launch_bounds__(256) chunk_output_kernel(const ChunkArgs a) {
   load_tile<PH>(v_s, vp, L.ldv, L.P - p0, nval, a.vec_v, L.silu_in);
   {
     const float* S0 = a.dS + ((long(chunk) * L.H + h) * L.P + p0) * L.N;
-#pragma unroll 2
-    for (int i = threadIdx.x; i < PW * NH * 8; i += 256) {
-      const int row = i / (NH * 8), col = (i % (NH * 8)) * 8;
-      float v[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] = 0.f;
-      if (p0 + row < L.P && col < L.N) {
-        const float* src = S0 + long(row) * L.N + col;
-        if (L.N % 4 == 0 && col + 8 <= L.N) {
-          const float4 f0 = *reinterpret_cast<const float4*>(src), f1 = *reinterpret_cast<const float4*>(src + 4);
-          v[0] = f0.x; v[1] = f0.y; v[2] = f0.z; v[3] = f0.w;
-          v[4] = f1.x; v[5] = f1.y; v[6] = f1.z; v[7] = f1.w;
-        } else {
-#pragma unroll
-          for (int j = 0; j < 8; ++j)
-            if (col + j < L.N) v[j] = src[j];
-        }
-      }
-      const int c8 = col >> 3;
+    auto put = [&](int row, int c8, float (&v)[8]) {
       const int off = (c8 >> 3) * SHALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4);
       *reinterpret_cast<uint4*>(sh_s + off) = split8(v);
       *reinterpret_cast<uint4*>(sl_s + off) = pack8(v);
+    };
+    constexpr int IT = PW * NH * 8 / 256, B = IT < 4 ? IT : 4;       // B pieces of 32 bytes in flight per thread
+    if (L.N % 8 == 0) {
+#pragma unroll
+      for (int i0 = 0; i0 < IT; i0 += B) {
+        float4 f[B][2];
+#pragma unroll
+        for (int i = 0; i < B; ++i) {
+          const int e = threadIdx.x + 256 * (i0 + i), row = e / (NH * 8), col = (e % (NH * 8)) * 8;
+          f[i][0] = f[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (p0 + row < L.P && col < L.N) {
+            const float4* src = reinterpret_cast<const float4*>(S0 + long(row) * L.N + col);
+            f[i][0] = src[0];
+            f[i][1] = src[1];
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < B; ++i) {
+          const int e = threadIdx.x + 256 * (i0 + i);
+          float v[8] = {f[i][0].x, f[i][0].y, f[i][0].z, f[i][0].w, f[i][1].x, f[i][1].y, f[i][1].z, f[i][1].w};
+          put(e / (NH * 8), e % (NH * 8), v);
+        }
+      }
+    } else {
+#pragma unroll 1
+      for (int e = threadIdx.x; e < PW * NH * 8; e += 256) {
+        const int row = e / (NH * 8), col = (e % (NH * 8)) * 8;
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = (p0 + row < L.P && col + j < L.N) ? S0[long(row) * L.N + col + j] : 0.f;
+        put(row, col >> 3, v);
+      }
     }
   }
   chunk_decay(a, h, t0, nval, cs, ws, tmp);

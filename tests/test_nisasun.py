@@ -59,7 +59,7 @@ def replay(models, name, device, dtype, max_tokens):
 
 
 def test_registry_and_config_round_trip():
-    for name in ("tiny-nisasun", "nisasun-3b"):
+    for name in ("tiny-nisasun", "nisasun-4b", "nisasun-13b"):
         c = PRESETS[name]()
         assert ModelConfig.from_dict(json.loads(c.to_json())) == c
         assert len(c.layers) == c.n_layer == len(c.layer_kinds)
