@@ -367,6 +367,7 @@ def main(argv=None):
     comm_status = int(pctx.symm.status.item()) if pctx.symm is not None else 0
 
     par = "single GPU" if world == 1 else (f"tp{world}" + ("+ep(experts whole per rank, tokens mirrored)" if ep else ""))
+    extra["tensor_maps_built"] = sm100.ext().tmap_encoded()
     extra.update({"decode": {str(u): rows[u] for u in all_users}, "kernel_status_word": status,
                   "comm_status_word": comm_status, "lm_head": "split by vocabulary rows" if head_split else "whole per rank", "launches_per_step": headline.get("launches_per_step"),
                   "shared_expert": ("stacked behind the routed experts (one slot of the grouped GEMMs)"

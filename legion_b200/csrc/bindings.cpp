@@ -11,6 +11,7 @@
 namespace lb {
 bool pdl_enabled();
 void set_pdl(bool on);
+long tmap_encoded();
 }  // namespace lb
 #include "quant.h"
 
@@ -650,6 +651,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   });
 #endif
   m.def("set_pdl", [](bool on) { lb::set_pdl(on); });
+  m.def("tmap_encoded", []() { return int64_t(lb::tmap_encoded()); });
   m.def("pdl_enabled", []() { return lb::pdl_enabled(); });
 #ifndef LB_CORE
   bind_gdn(m);

@@ -32,8 +32,13 @@ struct KeyHash {
     return size_t(h);
   }
 };
-// Descriptors are handed out by pointer, so entries are never moved once created.
-std::unordered_map<Key, std::unique_ptr<CUtensorMap>, KeyHash> g_cache;
+// Descriptors are handed out by pointer, so entries are never moved once created. A launch looks up several of them
+// before it uses the first: when the cache is full, its entries move to the previous generation and stay valid until
+// the cache has filled up once more (dropping them at once would leave the launch with a dangling descriptor).
+using Cache = std::unordered_map<Key, std::unique_ptr<CUtensorMap>, KeyHash>;
+constexpr size_t CACHE_MAX = 16384;
+Cache g_cache, g_previous;
+long g_encoded = 0;
 
 EncodeTiledFn get_encode() {
   if (g_encode) return g_encode;
@@ -63,7 +68,10 @@ const CUtensorMap* encode(const Key& key, int rank, const void* base, const cuui
   if (it != g_cache.end()) return it->second.get();
   EncodeTiledFn enc = get_encode();
   if (!enc) return nullptr;
-  if (g_cache.size() > 16384) g_cache.clear();
+  if (g_cache.size() >= CACHE_MAX) {
+    g_previous.swap(g_cache);
+    g_cache.clear();
+  }
   uint32_t elem;
   CUtensorMapDataType dt = to_cu(dtype, &elem);
   cuuint32_t estr[5] = {1, 1, 1, 1, 1};
@@ -78,6 +86,7 @@ const CUtensorMap* encode(const Key& key, int rank, const void* base, const cuui
     g_err = buf;
     return nullptr;
   }
+  ++g_encoded;
   const CUtensorMap* p = m.get();
   g_cache.emplace(key, std::move(m));
   return p;
@@ -86,6 +95,10 @@ const CUtensorMap* encode(const Key& key, int rank, const void* base, const cuui
 }  // namespace
 
 const char* tmap_last_error() { return g_err.c_str(); }
+long tmap_encoded() {
+  std::lock_guard<std::mutex> lk(g_mu);
+  return g_encoded;
+}
 
 const CUtensorMap* tmap_2d(const void* base, uint64_t rows, uint64_t cols, uint64_t ld_bytes, uint32_t box_rows,
                            uint32_t box_cols, int dtype, bool swizzle128) {

@@ -23,4 +23,7 @@ const CUtensorMap* tmap_3d(const void* base, uint64_t d0, uint64_t d1, uint64_t 
 
 const char* tmap_last_error();
 
+// descriptors built so far (cache misses)
+long tmap_encoded();
+
 }  // namespace lb

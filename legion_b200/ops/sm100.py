@@ -20,7 +20,7 @@ _lock = threading.Lock()
 
 
 # kernels launched by one call of each binding (for the launch counter)
-KERNELS_PER_CALL = {"moe_plan": 3, "paged_decode": 1, "argmax": 2, "wgemm_workspace_floats": 0, "linear_chunk": 3, "linear_chunk_ok": 0,
+KERNELS_PER_CALL = {"moe_plan": 3, "paged_decode": 1, "argmax": 2, "wgemm_workspace_floats": 0, "linear_chunk": 3, "linear_chunk_ok": 0, "tmap_encoded": 0,
                     "linear_chunk_scratch_bytes": 0, "conv_silu_any": 2}
 LAUNCHES = {"n": 0}
 

@@ -876,3 +876,26 @@ def test_scratch_buffers_keep_their_guard_areas(monkeypatch):
     finally:
         m.Workspace._by_device.clear()
         m.Workspace._by_device.update(saved)
+
+
+def test_more_tensor_maps_than_the_cache_holds():
+    """Every launch with operands at new addresses builds new TMA descriptors; launches on both sides of a full
+    descriptor cache keep working."""
+    from legion_b200.ops import sm100
+    C = sm100.ext()
+    x = torch.randn(18000 * 2, 64, device="cuda").bfloat16()
+    w = torch.randn(128 * 40, 64, device="cuda").bfloat16()
+    want = x.float() @ w[:128].float().t()
+    n0, i = C.tmap_encoded(), 0
+    outs = []
+    while C.tmap_encoded() - n0 < 17500:
+        rows = x[2 * i:2 * i + 2] if i % 2 else x[2 * i:2 * i + 1]
+        k = (i % 39) * 128 if i % 3 else 0
+        outs.append((i, rows.shape[0], k, sm100.linear(rows, w[k:k + 128])))
+        i += 1
+        assert 2 * i + 2 <= x.shape[0]
+    torch.cuda.synchronize()
+    for i, n, k, o in outs[::37] + outs[-1200:]:
+        ref = want[2 * i:2 * i + n] if k == 0 else x[2 * i:2 * i + n].float() @ w[k:k + 128].float().t()
+        assert torch.allclose(o.float(), ref, atol=0.15, rtol=2e-2)
+    assert sm100.Workspace.get("cuda").check() == 0
