@@ -194,7 +194,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           uint64_t* empty = kv ? &v_empty[st] : &k_empty[st];
           uint64_t* full = kv ? &v_full[st] : &k_full[st];
           if (i >= nst && !__all_sync(0xffffffffu, mbar_wait(empty, ((i / nst) - 1) & 1, abort_flag))) {
-            if (lane == 0) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_EMPTY); }
+            if (lane == 0) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_EMPTY | SITE_DECODE_ATTN); }
             ok = false;
             break;
           }
@@ -237,15 +237,15 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         bool ok = mbar_wait(q_full, 0, abort_flag);
         ok = ok && issue_s(0);
         if (ok && n_blk > 1) ok = issue_s(1);
-        if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); }
+        if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_DECODE_ATTN); }
         for (int i = 0; ok && i < n_blk; ++i) {
           const int wgp = i & 1;
           if (!mbar_wait(&p_ready[wgp], (i >> 1) & 1, abort_flag)) {
-            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FLAG); break;
+            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FLAG | SITE_DECODE_ATTN); break;
           }
           const int vs = i % VS;
           if (!mbar_wait(&v_full[vs], (i / VS) & 1, abort_flag)) {
-            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); break;
+            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_DECODE_ATTN); break;
           }
           tc_fence_after();
           const uint32_t va = smem_u32(v_s + vs * Cfg::V_BYTES);
@@ -267,7 +267,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           umma_commit(&v_empty[vs]);
           // the softmax of tile i has read S[wgp]: the scores of tile i+2 go there, two tiles ahead of their use
           if (i + 2 < n_blk && !issue_s(i + 2)) {
-            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); break;
+            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_DECODE_ATTN); break;
           }
         }
       }
@@ -292,7 +292,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // A wait that runs out does not leave the loop: the warp keeps taking part in the named barriers and the
       // p_ready arrivals (without touching TMEM or waiting again), so the other warps can never be left behind.
       bool ok = true;
-      auto fail = [&](int code) { *abort_flag = 1; atomicCAS(a.status, 0, code); ok = false; };
+      auto fail = [&](int code) { *abort_flag = 1; atomicCAS(a.status, 0, code | SITE_DECODE_ATTN); ok = false; };
       int n_mine = 0;
       for (int i = wgp; i < n_blk; i += 2, ++n_mine) {
         const uint32_t ph = (i >> 1) & 1;

@@ -140,8 +140,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* p_ready = bars + 8;  // [2] one per score buffer: with the scores issued a block ahead, a fast softmax warp
                                  //     can finish block i + 1 before a slow one has finished block i; on ONE barrier its
                                  //     second arrival would complete block i's phase early
-  uint64_t* o_done = bars + 10;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 11);
+  uint64_t* o_done = bars + 10;  // [2] P V of even / odd blocks. A softmax warp looks at them only when it rescales and at
+                                 //     the end; on ONE barrier its wait for an old phase could find the barrier two
+                                 //     phases on (same parity) and never return
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 12);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int seq = blockIdx.z;
@@ -165,7 +167,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     mbar_init(&s_full[1], 1);
     mbar_init(&p_ready[0], 128);
     mbar_init(&p_ready[1], 128);
-    mbar_init(o_done, 1);
+    mbar_init(&o_done[0], 1);
+    mbar_init(&o_done[1], 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -226,13 +229,13 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       constexpr uint32_t idesc_s = umma_idesc(128, BKV, 1, 1, 0, 0);
       constexpr uint32_t idesc_o = umma_idesc(128, DV, 1, 1, 0, 1);  // B (= V) is MN-major
       bool ok = mbar_wait(q_full, 0, abort_flag);
-      if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); }
+      if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_PREFILL_ATTN); }
       const uint32_t qa = smem_u32(q_s);
       // S(j) = Q K_j^T into score buffer j & 1, from K stage j % 3
       auto issue_s = [&](int j) -> bool {
         const int st = j % 3;
         if (!mbar_wait(&k_full[st], uint32_t(j / 3) & 1u, abort_flag)) {
-          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); return false;
+          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_PREFILL_ATTN); return false;
         }
         tc_fence_after();
         const uint32_t ka = smem_u32(k_s + st * Cfg::K_BYTES);
@@ -258,16 +261,16 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         if (i + 1 < n_blk && !issue_s(i + 1)) break;
         if (i >= 1 && i + 1 < n_blk) {
           // V stage (i + 1) & 1 held block i - 1: free once that block's P V has completed
-          if (!mbar_wait(o_done, (i - 1) & 1, abort_flag)) {
-            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY); break;
+          if (!mbar_wait(&o_done[(i - 1) & 1], uint32_t((i - 1) >> 1) & 1u, abort_flag)) {
+            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY | SITE_PREFILL_ATTN); break;
           }
           load_v(blk_lo + i + 1, (i + 1) & 1);
         }
         if (!mbar_wait(&p_ready[i & 1], uint32_t(i >> 1) & 1u, abort_flag)) {
-          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FLAG); break;
+          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FLAG | SITE_PREFILL_ATTN); break;
         }
         if (!mbar_wait(&v_full[i & 1], uint32_t(i >> 1) & 1u, abort_flag)) {
-          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL); break;
+          *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_PREFILL_ATTN); break;
         }
         tc_fence_after();
         const uint32_t va = smem_u32(v_s + (i & 1) * Cfg::V_BYTES);
@@ -278,7 +281,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           const uint64_t db = umma_desc_mn_sw128(va + k * 16 * 128, BKV * 128, 1024);
           umma_f16_ts(tmem_O, tp + k * 8, db, idesc_o, (i | k) ? 1u : 0u);
         }
-        umma_commit(o_done);
+        umma_commit(&o_done[i & 1]);
       }
     }
   } else {
@@ -291,7 +294,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     bool ok = true;
     for (int i = 0; i < n_blk; ++i) {
       if (!__all_sync(0xffffffffu, mbar_wait(&s_full[i & 1], uint32_t(i >> 1) & 1u, abort_flag))) {
-        *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); ok = false; break;
+        *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_PREFILL_ATTN); ok = false; break;
       }
       tc_fence_after();
       const uint32_t tmem_Si = tmem_S + uint32_t(i & 1) * BKV;
@@ -424,8 +427,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         // be touched only after the previous block's P V has finished (P itself no longer waits for it: it lives
         // in this block's own score buffer)
         if (__any_sync(0xffffffffu, alpha != 1.f)) {
-          if (!__all_sync(0xffffffffu, mbar_wait(o_done, (i - 1) & 1, abort_flag))) {
-            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY); ok = false; break;
+          if (!__all_sync(0xffffffffu, mbar_wait(&o_done[(i - 1) & 1], uint32_t((i - 1) >> 1) & 1u, abort_flag))) {
+            *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY | SITE_PREFILL_ATTN); ok = false; break;
           }
           tc_fence_after();
 #pragma unroll 1
@@ -445,17 +448,11 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       mbar_arrive(&p_ready[i & 1]);
     }
     // final: O / l -> out
-    if (ok && n_blk > 1) {
-      // a parity wait may be at most one phase behind the barrier: this thread may not have looked at o_done for
-      // many blocks (it waits only when it rescales), so it first catches up with the block before the last (whose
-      // predecessor is known to be complete: it ran before the last block's scores)
-      if (!__all_sync(0xffffffffu, mbar_wait(o_done, (n_blk - 2) & 1, abort_flag))) {
-        *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); ok = false;
-      }
-    }
+    // (P V of the block two before is known to be complete, it ran before this block's scores: at most one phase of
+    // the barrier is open here; the last commit covers every P V)
     if (ok && n_blk > 0) {
-      if (!__all_sync(0xffffffffu, mbar_wait(o_done, (n_blk - 1) & 1, abort_flag))) {
-        *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); ok = false;
+      if (!__all_sync(0xffffffffu, mbar_wait(&o_done[(n_blk - 1) & 1], uint32_t((n_blk - 1) >> 1) & 1u, abort_flag))) {
+        *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_PREFILL_ATTN); ok = false;
       }
     }
     if (ok) {

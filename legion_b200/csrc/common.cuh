@@ -24,6 +24,16 @@ enum : int {
   ST_BAD_ARGS = 6,
 };
 
+// Where a wait gave up, in the bits above the code.
+enum : int {
+  SITE_GEMM = 1 << 8,
+  SITE_PREFILL_ATTN = 2 << 8,
+  SITE_DECODE_ATTN = 3 << 8,
+  SITE_CHUNK_STATES = 4 << 8,
+  SITE_CHUNK_SCORES = 5 << 8,
+  SITE_CHUNK_OUTPUT = 6 << 8,
+};
+
 // Default deadline for in-kernel waits, in nanoseconds of %globaltimer.
 #ifndef LB_WAIT_NS
 #define LB_WAIT_NS 2000000000ull

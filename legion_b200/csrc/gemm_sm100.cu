@@ -257,7 +257,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
         for (int kb = kb0; kb < kb1; ++kb) {
           if (!mbar_wait(&empty[s], ph ^ 1, abort_flag)) {
             *abort_flag = 1;
-            atomicCAS(a.status, 0, ST_TIMEOUT_EMPTY);
+            atomicCAS(a.status, 0, ST_TIMEOUT_EMPTY | SITE_GEMM);
             ok = false;
             break;
           }
@@ -311,7 +311,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
         if (!WFP8) {
           if (!mbar_wait(&tempty[acc], acc_ph ^ 1, abort_flag)) {
             *abort_flag = 1;
-            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY);
+            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY | SITE_GEMM);
             break;
           }
           tc_fence_after();
@@ -319,13 +319,13 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
         for (int kb = kb0; kb < kb1; ++kb) {
           if (!mbar_wait(&full[s], ph, abort_flag) || (WFP4 && !mbar_wait(&wready[s], ph, abort_flag))) {
             *abort_flag = 1;
-            atomicCAS(a.status, 0, ST_TIMEOUT_FULL);
+            atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_GEMM);
             ok = false;
             break;
           }
           if (WFP8 && !mbar_wait(&tempty[acc], acc_ph ^ 1, abort_flag)) {   // this k block's partial accumulator
             *abort_flag = 1;
-            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY);
+            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY | SITE_GEMM);
             ok = false;
             break;
           }
@@ -392,7 +392,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
       for (int kb = kb0; kb < kb1; ++kb) {
         if (ok && !mbar_wait(&full[s], ph, abort_flag)) {
           *abort_flag = 1;
-          atomicCAS(a.status, 0, ST_TIMEOUT_FULL);
+          atomicCAS(a.status, 0, ST_TIMEOUT_FULL | SITE_GEMM);
           ok = false;      // keep arriving so that nobody is left waiting on wready
         }
         uint8_t* st = smem + s * Cfg::STAGE_BYTES;
@@ -466,7 +466,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
         for (int kb = kb0; kb < kb1; ++kb) {
           if (!__all_sync(0xffffffffu, mbar_wait(&tfull[acc], acc_ph, abort_flag))) {
             *abort_flag = 1;
-            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL);
+            atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_GEMM);
             failed = true;
             break;
           }
@@ -496,7 +496,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
       } else {
         if (!__all_sync(0xffffffffu, mbar_wait(&tfull[acc], acc_ph, abort_flag))) {
           *abort_flag = 1;
-          atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL);
+          atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_GEMM);
           break;
         }
         tc_fence_after();

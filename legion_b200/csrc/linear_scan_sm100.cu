@@ -254,7 +254,7 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs a) {
     if (blockIdx.z == 0) a.gC[long(chunk) * L.H + h] = exp2f(cC);
   }
   const bool ok = mbar_wait(done, 0, abort_flag);
-  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); }
+  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_CHUNK_STATES); }
   __syncwarp();
   tc_fence_after();
   if (__all_sync(0xffffffffu, ok)) {
@@ -446,7 +446,7 @@ __global__ void __launch_bounds__(256) chunk_output_kernel(const ChunkArgs a) {
   }
   chunk_decay(a, h, t0, nval, cs, ws, tmp);
   bool ok = mbar_wait(s_done, 0, abort_flag);
-  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); }
+  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_CHUNK_SCORES); }
   __syncwarp();
   tc_fence_after();
   const int row = (warp & 3) * 32 + lane;                 // token of the chunk
@@ -509,7 +509,7 @@ __global__ void __launch_bounds__(256) chunk_output_kernel(const ChunkArgs a) {
   }
   __syncwarp();
   ok = mbar_wait(o_done, 0, abort_flag);
-  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL); }
+  if (!ok) { *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_CHUNK_OUTPUT); }
   __syncwarp();
   tc_fence_after();
   if (__all_sync(0xffffffffu, ok)) {

@@ -104,7 +104,19 @@ def model_bytes_per_step(cfg, n_seqs: int, ctx: int, tp: int = 1, dtype_bytes: i
     dense = 0
     experts = 0
     kv = 0
-    for il, kind in enumerate(cfg.layer_kinds):
+    for il in range(cfg.n_layer if cfg.layers is not None else 0):     # stacks with layer specifications
+        from ..models.weights import layer_weight_shapes
+        for name, shp in layer_weight_shapes(cfg, il).items():
+            if len(shp) == 2 and not name.endswith(("conv_w", "st_mix")):
+                dense += shp[0] * shp[1]
+        a, r, f = cfg.attn_spec(il), cfg.recurrent_spec(il), cfg.layers[il].mlp
+        if a is not None:
+            kv += a.kv_heads * (a.dim + a.vdim) * (min(ctx, a.window) if a.window else ctx) * n_seqs
+        if r is not None:                                               # fp32 state, read and written
+            kv += r.heads * r.vdim * (r.dim if r.kind == "lightning" else r.state) * 4 * n_seqs
+        if f is not None and f.kind == "moe":
+            experts += f.experts * (1.0 - (1.0 - f.top / f.experts) ** n_seqs) * 3 * H * f.ff
+    for il, kind in enumerate(cfg.layer_kinds if cfg.layers is None else []):
         if kind in ("attn", "swa", "nope"):
             qw = cfg.n_head * cfg.head_dim * (2 if cfg.gated_attn else 1)
             dense += (qw + 2 * cfg.n_kv_head * cfg.head_dim) * H + H * cfg.n_head * cfg.head_dim

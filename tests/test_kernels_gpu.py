@@ -899,3 +899,24 @@ def test_more_tensor_maps_than_the_cache_holds():
         ref = want[2 * i:2 * i + n] if k == 0 else x[2 * i:2 * i + n].float() @ w[k:k + 128].float().t()
         assert torch.allclose(o.float(), ref, atol=0.15, rtol=2e-2)
     assert sm100.Workspace.get("cuda").check() == 0
+
+
+@pytest.mark.parametrize("window", [0, 200])
+def test_prefill_attention_many_short_tiles_end_cleanly(window):
+    """Thousands of tiles with few key blocks, launch after launch: no wait of the softmax warps may miss its phase
+    (status word), and the outputs repeat bit for bit."""
+    from legion_b200.ops import sm100
+    g = torch.Generator(device="cuda").manual_seed(0)
+    n, Hq, Hkv, D, ctx = 96, 16, 4, 128, 320
+    q = torch.randn(n * 2, Hq, D, device="cuda", generator=g).bfloat16()
+    kc = torch.randn(n * 5, 64, Hkv, D, device="cuda", generator=g).bfloat16()
+    vc = torch.randn(n * 5, 64, Hkv, D, device="cuda", generator=g).bfloat16()
+    bt = torch.arange(n * 5, device="cuda", dtype=torch.int32).view(n, 5)
+    cu = torch.arange(0, 2 * n + 1, 2, device="cuda", dtype=torch.int32)
+    cl = torch.full((n,), ctx, device="cuda", dtype=torch.int32) - torch.arange(n, device="cuda", dtype=torch.int32) * 3
+    first = sm100.prefill_attn(q, kc, vc, cu, cl, bt, 2, D ** -0.5, window)
+    for _ in range(300):
+        out = sm100.prefill_attn(q, kc, vc, cu, cl, bt, 2, D ** -0.5, window)
+    torch.cuda.synchronize()
+    assert torch.equal(out, first)
+    status_ok()
