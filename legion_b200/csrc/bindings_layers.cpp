@@ -209,8 +209,10 @@ void bind_layers(pybind11::module_& m) {
   });
   m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
                           const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state, const Tensor& cu,
-                          const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& out, bool write_state) {
-    const auto a = scan_args(q, k, v, silu_in, decay, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, write_state);
+                          const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& out, bool write_state,
+                          int64_t max_tokens) {
+    auto a = scan_args(q, k, v, silu_in, decay, dt, dt_bias, A, D, z, state, cu, slots, H, G, N, P, out, write_state);
+    a.max_tokens = int(max_tokens);
     c10::cuda::CUDAGuard guard(q.device());
     TORCH_CHECK(lb::linear_scan_launch(a, q.scalar_type() == at::kFloat, cur_stream()) == 0,
                 "linear scan: at most 512 state columns, heads a multiple of the groups", cuda_error());

@@ -68,6 +68,7 @@ struct LinScanArgs {
   int n_seqs, T, H, G, N, P;
   void* out; long ldo;
   int write_state;
+  int max_tokens;                  // linear_scan: sequences with more tokens are left alone (0: all run)
 };
 int linear_scan_launch(const LinScanArgs& a, bool f32, cudaStream_t s);
 

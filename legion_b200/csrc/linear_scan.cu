@@ -27,7 +27,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const LinScanArgs a) {
   const int h = blockIdx.x / pb, p0 = (blockIdx.x % pb) * RPC + (threadIdx.x >> 5) * RPW;
   const int seq = blockIdx.y, lane = threadIdx.x & 31;
   const int t0 = a.cu[seq], t1 = a.cu[seq + 1], slot = a.slots[seq];
-  if (t1 <= t0 || slot < 0 || p0 >= a.P) return;
+  if (t1 <= t0 || slot < 0 || p0 >= a.P || (a.max_tokens > 0 && t1 - t0 > a.max_tokens)) return;
   const int N = a.N, g = h / (a.H / a.G);
   float* st = a.state + ((long(slot) * a.H + h) * a.P + p0) * N;
   float s[RPW][NJ];

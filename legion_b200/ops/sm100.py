@@ -1533,26 +1533,31 @@ def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset=0.0):
 
 
 LINEAR_CHUNK_MIN = 48        # longest portion of a step from which the chunked scan runs
+LINEAR_CHUNK_SHORT = 8       # ... and up to which its shorter portions stay on the streaming kernel
 
 
 def _linear_chunk_tables(ws, cu_host, device):
-    """chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk of a step (128-token chunks); kept for the step's other
-    layers."""
+    """chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk of a step (128-token chunks; short portions have none);
+    kept for the step's other layers. Returns (tables, chunks, whether there are short portions)."""
     key = tuple(cu_host)
     last = ws._cache.get("linear_chunk_tables")
     if last is not None and last[0] == key:
-        return last[1], last[2]
+        return last[1:]
     t0, n, sq, first, cnt = [], [], [], [], []
     for i in range(len(cu_host) - 1):
         first.append(len(t0))
+        if cu_host[i + 1] - cu_host[i] <= LINEAR_CHUNK_SHORT:
+            cnt.append(0)
+            continue
         for b in range(cu_host[i], cu_host[i + 1], 128):
             t0.append(b)
             n.append(min(128, cu_host[i + 1] - b))
             sq.append(i)
         cnt.append(len(t0) - first[-1])
     tab = torch.tensor(t0 + n + sq + first + cnt, dtype=torch.int32, device=device)
-    ws._cache["linear_chunk_tables"] = (key, tab, len(t0))
-    return tab, len(t0)
+    short = any(c == 0 for c in cnt)
+    ws._cache["linear_chunk_tables"] = (key, tab, len(t0), short)
+    return tab, len(t0), short
 
 
 def linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, decay=None, silu_in=False, dt=None, dt_bias=None, A=None,
@@ -1568,10 +1573,14 @@ def linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, decay=None, silu_in=F
         chunked = (q.dtype == torch.bfloat16 and cu_host is not None and (max_len or 0) >= LINEAR_CHUNK_MIN
                    and C.linear_chunk_ok(N, P))
     if not chunked:
-        C.linear_scan(*args)
+        C.linear_scan(*args, 0)
         return out
     ws = Workspace.get(q.device)
-    tab, n_chunks = _linear_chunk_tables(ws, cu_host if cu_host is not None else cu_seq.tolist(), q.device)
+    tab, n_chunks, short = _linear_chunk_tables(ws, cu_host if cu_host is not None else cu_seq.tolist(), q.device)
+    if short or n_chunks == 0:           # single tokens and the like beside prompts
+        C.linear_scan(*args, LINEAR_CHUNK_SHORT)
+    if n_chunks == 0:
+        return out
     need = C.linear_chunk_scratch_bytes(n_chunks, H, N, P)
     scratch = ws._cache.get("linear_chunk_scratch")
     if scratch is None or scratch.numel() < need:

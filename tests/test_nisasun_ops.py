@@ -229,7 +229,7 @@ def test_linear_state_in_chunks(device, dtype, kind, H, G, N, P):
     more than bf16 accuracy."""
     if kind == "constant":
         G = H
-    lens = [300, 1, 128, 129, 2, 127, 64]
+    lens = [300, 1, 128, 129, 2, 127, 64, 8, 9]
     q, k, v, state, cu, slots, cu_h, kw = scan_case(H, G, N, P, lens, 8, device, dtype, kind)
     want, states = scan_expected(q, k, v, state, cu_h, slots, H, G, N, P, kw)
     got = ops.sm100.linear_scan(q, k, v, state, cu, slots, H, G, N, P, cu_host=cu_h, chunked=True, **kw)
