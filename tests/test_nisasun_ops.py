@@ -95,7 +95,7 @@ def windowed(q, k, v, scale, window):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 96, 128), (6, 3, 40, 72), (2, 2, 64, 256), (3, 1, 136, 24), (2, 1, 13, 19),
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 88, 128), (6, 3, 40, 72), (2, 2, 64, 256), (3, 1, 136, 24), (2, 1, 13, 19),
                                        (16, 1, 128, 128), (4, 4, 256, 64), (4, 2, 120, 192), (2, 1, 40, 136),
                                        (2, 2, 168, 184)])
 def test_windowed_attention_prompts_and_decode(device, dtype, H, G, dk, dv):
@@ -116,7 +116,7 @@ def test_windowed_attention_prompts_and_decode(device, dtype, H, G, dk, dv):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("dk,dv", [(96, 128), (20, 12)])
+@pytest.mark.parametrize("dk,dv", [(112, 160), (20, 12)])
 @pytest.mark.parametrize("window", [1, 8, 64, 65, 127, 128, 129, 300])
 def test_one_key_at_the_window_edge(device, dtype, dk, dv, window):
     """One key scores far above all others and its value is marked: it decides the output exactly as long as it is
@@ -205,7 +205,7 @@ def scan_expected(q, k, v, state, cu, slots, H, G, N, P, kw):
 
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("kind", ["constant", "selective"])
-@pytest.mark.parametrize("H,G,N,P", [(4, 2, 32, 32), (3, 3, 48, 64), (2, 1, 13, 19), (2, 2, 128, 128), (4, 1, 40, 160)])
+@pytest.mark.parametrize("H,G,N,P", [(6, 2, 32, 40), (3, 3, 48, 64), (2, 1, 13, 19), (2, 2, 128, 128), (4, 1, 40, 160)])
 def test_linear_state(device, dtype, kind, H, G, N, P):
     if kind == "constant":
         G = H
@@ -222,7 +222,7 @@ def test_linear_state(device, dtype, kind, H, G, N, P):
 
 @pytest.mark.parametrize("device,dtype", BF16)
 @pytest.mark.parametrize("kind", ["constant", "selective"])
-@pytest.mark.parametrize("H,G,N,P", [(4, 2, 32, 32), (3, 3, 48, 64), (2, 1, 13, 19), (2, 2, 128, 128), (4, 1, 40, 160),
+@pytest.mark.parametrize("H,G,N,P", [(6, 2, 32, 40), (3, 3, 48, 64), (2, 1, 13, 19), (2, 2, 128, 128), (4, 1, 40, 160),
                                      (2, 1, 100, 90)])
 def test_linear_state_in_chunks(device, dtype, kind, H, G, N, P):
     """The tensor-core form: whole chunks, chunk edges, single tokens beside them, carried states; the state keeps far
@@ -242,7 +242,7 @@ def test_linear_state_in_chunks(device, dtype, kind, H, G, N, P):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE[1:])
-@pytest.mark.parametrize("H,G,N,P,K", [(4, 2, 32, 32, 4), (6, 3, 16, 24, 1), (4, 4, 128, 64, 2), (8, 1, 40, 130, 9)])
+@pytest.mark.parametrize("H,G,N,P,K", [(6, 2, 32, 40, 4), (6, 3, 16, 24, 1), (4, 4, 128, 64, 2), (8, 1, 40, 130, 9)])
 def test_ssd_decode_step(device, dtype, H, G, N, P, K):
     """The fused decode launch against convolution and scan one after the other, several steps in a row."""
     n, C = 5, H * P + 2 * G * N
@@ -298,7 +298,7 @@ def test_group_norm_and_gate(device, dtype, C, groups):
 # ------------------------------------------------------------------------------------------- feed-forward parts
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("T", [3, 64, 65, 200])
-@pytest.mark.parametrize("E,top,count,keep", [(12, 4, 4, 3), (8, 2, 2, 1), (5, 1, 1, 1), (64, 6, 8, 3), (6, 3, 6, 4)])
+@pytest.mark.parametrize("E,top,count,keep", [(15, 4, 5, 3), (8, 2, 2, 1), (5, 1, 1, 1), (64, 6, 8, 3), (6, 3, 6, 4)])
 def test_router_groups_and_correction(device, dtype, T, E, top, count, keep):
     W = 64
     h = rnd(T, W, seed=1, dtype=dtype, device=device)
