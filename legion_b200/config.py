@@ -61,10 +61,54 @@ class ParallelSpec:
 
 
 @dataclass
+class RotarySpec:
+    """Rotation of the first ``dims`` columns of a vector, neighbouring columns in pairs. ``original`` > 0: YaRN
+    (frequencies divided by ``factor`` along a ramp between the pairs that turn ``fast`` and ``slow`` times over the
+    original context; cos and sin grow by 0.1 ln(factor) + 1)."""
+    dims: int
+    base: float
+    factor: float = 1.0
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+    kind: str = "rotary"
+
+
+@dataclass
+class LatentSpec:
+    """Latent attention: keys and values of all heads are projections of one cached latent; a rotated key part is shared
+    by the heads. The output is gated by the sigmoid of a projection of the input."""
+    heads: int
+    dim: int                           # query / key columns per head that are not rotated
+    rot_dim: int                       # ... and the rotated part
+    vdim: int
+    kv_rank: int                       # latent size
+    scale: float                       # multiplies the scores
+    rot: RotarySpec
+    gate: str = "channel"              # channel: one gate per output column | head: one per head | none
+    kind: str = "latent"
+
+    def gate_width(self) -> int:
+        return {"channel": self.heads * self.vdim, "head": self.heads, "none": 0}[self.gate]
+
+
+@dataclass
+class RgLruSpec:
+    """Griffin's recurrent block: a short convolution and a real-gated linear recurrent unit beside a GELU branch."""
+    width: int
+    blocks: int                        # equal parts of the width, each with gate matrices of its own
+    conv: int = 4                      # taps
+    kind: str = "rglru"
+
+
+@dataclass
 class DenseSpec:
     ff: int
-    act: str = "silu"
+    act: str = "silu"                  # xielu: un-gated, with two learned numbers per layer
     kind: str = "dense"
+
+    def gated(self) -> bool:
+        return self.act != "xielu"
 
 
 @dataclass
@@ -89,7 +133,7 @@ class LayerSpec:
 
 
 _SPECS = {c.__dataclass_fields__["kind"].default: c
-          for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, DenseSpec, MoeSpec)}
+          for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, RotarySpec, LatentSpec, RgLruSpec, DenseSpec, MoeSpec)}
 
 
 def spec_from(d):
@@ -205,6 +249,11 @@ class ModelConfig:
     # stacks whose layers have sizes of their own: one LayerSpec per layer. The per-model attention / recurrent / MoE
     # fields above then only describe the largest layer (memory planning); every layer runs from its specification
     layers: Optional[List[LayerSpec]] = None
+    # with ``layers`` and ``sandwich_norm``: one fp32 residual stream, every sublayer between two RMS norms that work in
+    # ``norm_groups`` equal parts of the vector; what a sublayer reads first passes h + conv(h), a causal convolution per
+    # channel of ``input_conv`` taps (0: none)
+    norm_groups: int = 1
+    input_conv: int = 0
     # multi-token prediction
     mtp_layers: int = 0
     # weights
@@ -217,6 +266,10 @@ class ModelConfig:
             self.n_layer = len(self.layers)
             self.layer_kinds = [x.mixer.kind for x in self.layers]
             attn = [a for a in (self.attn_spec(il) for il in range(self.n_layer)) if a is not None]
+            lat = [x.mixer for x in self.layers if isinstance(x.mixer, LatentSpec)]
+            if lat:
+                big = max(lat, key=lambda a: a.kv_rank + a.rot_dim)
+                self.n_head, self.n_kv_head, self.head_dim = big.heads, 1, big.kv_rank + big.rot_dim
             if attn:
                 big = max(attn, key=lambda a: a.kv_heads * (a.dim + a.vdim))
                 self.n_head, self.n_kv_head, self.head_dim = big.heads, big.kv_heads, big.dim
@@ -243,10 +296,21 @@ class ModelConfig:
         m = self.layers[il].mixer
         return m if isinstance(m, AttnSpec) else (m.left if isinstance(m, ParallelSpec) else None)
 
+    def latent_spec(self, il: int) -> Optional[LatentSpec]:
+        """The mixer of layer il of a stack with specifications, when it is latent attention."""
+        m = self.layers[il].mixer
+        return m if isinstance(m, LatentSpec) else None
+
     def recurrent_spec(self, il: int):
         """The part of layer il that carries a recurrent state, of a stack with specifications."""
         m = self.layers[il].mixer
-        return m if isinstance(m, (LightningSpec, SsdSpec)) else (m.right if isinstance(m, ParallelSpec) else None)
+        return m if isinstance(m, (LightningSpec, SsdSpec, RgLruSpec)) else (m.right if isinstance(m, ParallelSpec) else None)
+
+    def conv_inputs(self, il: int) -> List[str]:
+        """Sublayers of layer il whose input passes a short convolution (``input_conv``)."""
+        if self.layers is None or self.input_conv < 1:
+            return []
+        return ["attn"] if self.layers[il].mlp is None else ["attn", "ffn"]
 
     def is_moe_layer(self, il: int) -> bool:
         if self.layers is not None:
@@ -257,18 +321,21 @@ class ModelConfig:
 
     def kv_layers(self) -> List[int]:
         if self.layers is not None:
-            return [i for i in range(self.n_layer) if self.attn_spec(i) is not None]
+            return [i for i in range(self.n_layer) if self.attn_spec(i) is not None or self.latent_spec(i) is not None]
         return [i for i, k in enumerate(self.layer_kinds) if k in ("attn", "swa", "nope", "mla")]
 
     def recurrent_layers(self) -> List[int]:
+        """Layers that carry a state from token to token besides the KV cache."""
         if self.layers is not None:
-            return [i for i in range(self.n_layer) if self.recurrent_spec(i) is not None]
+            return [i for i in range(self.n_layer) if self.recurrent_spec(i) is not None or self.conv_inputs(i)]
         return [i for i, k in enumerate(self.layer_kinds) if k in ("gdn", "mamba2", "kda")]
 
     def kv_dims(self, il: int):
         """(n_kv_heads, k_dim, v_dim) stored per token for layer il."""
         if self.layers is not None:
-            a = self.attn_spec(il)
+            a, m = self.attn_spec(il), self.latent_spec(il)
+            if m is not None:                           # one row per token, keys and values alike
+                return 1, -(-(m.kv_rank + m.rot_dim) // 8) * 8, 0
             return a.kv_heads, a.dim, a.vdim
         if self.layer_kinds[il] == "mla":
             return 1, self.kv_lora + self.qk_rope_dim, 0
@@ -521,7 +588,57 @@ def hybrid_13b() -> ModelConfig:
     return _hybrid(20, 4096, 32, 12288, 2048)
 
 
+def tiny_pemezen() -> "ModelConfig":
+    """Pemezen in miniature: latent-attention layers (rotated key parts with YaRN frequencies, output gates per column or
+    per head) and a gated linear recurrent unit, every sublayer between grouped norms behind a short input convolution,
+    xIELU feed-forward parts, one layer without any. Sizes differ from layer to layer."""
+    return ModelConfig(
+        arch="pemezen", hidden=144, vocab=512, rms_eps=1e-5, sandwich_norm=True, norm_groups=3, input_conv=3,
+        embed_scale=2.5, logit_softcap=12.0,
+        layers=[LayerSpec(LatentSpec(6, 40, 24, 32, 72, 0.15, RotarySpec(24, 1e4, 2.0, 256), "head"), DenseSpec(200, "xielu")),
+                LayerSpec(RgLruSpec(120, 3, 5), DenseSpec(88, "xielu")),
+                LayerSpec(LatentSpec(2, 64, 16, 48, 96, 0.11, RotarySpec(16, 5e4, 4.0, 128)), None),
+                LayerSpec(RgLruSpec(64, 1, 3), DenseSpec(136, "xielu"))])
+
+
+def _pemezen(n_layer: int, hidden: int, heads: int, ff: int, rank: int, rot: int) -> ModelConfig:
+    """Two recurrent layers, then a latent-attention layer, in turn; gates per column and per head in turn."""
+    layers = []
+    for il in range(n_layer):
+        mixer = (LatentSpec(heads, 128, rot, 128, rank, (128 + rot) ** -0.5, RotarySpec(rot, 5e5, 4.0, 8192),
+                            "channel" if il % 2 else "head")
+                 if il % 3 == 2 else RgLruSpec(hidden * 5 // 4, hidden // 256 * 5 // 4, 4))
+        layers.append(LayerSpec(mixer, DenseSpec(ff, "xielu")))
+    return ModelConfig(arch="pemezen", hidden=hidden, vocab=65536, rms_eps=1e-5, sandwich_norm=True, norm_groups=4,
+                       input_conv=4, embed_scale=3.0, logit_softcap=15.0, layers=layers)
+
+
+def pemezen_1b() -> ModelConfig:
+    """Pemezen with layers the size of a small production model (random weights; speed measurements)."""
+    return _pemezen(24, 2048, 16, 8192, 512, 64)
+
+
+def pemezen_7b() -> ModelConfig:
+    return _pemezen(30, 4096, 32, 16384, 512, 64)
+
+
+def mla_1b() -> ModelConfig:
+    """A dense latent-attention model of the size of ``pemezen_1b``: what its attention layers are compared with."""
+    return ModelConfig(arch="deepseek_v3", n_layer=24, hidden=2048, vocab=65536, n_head=16, n_kv_head=16, head_dim=192,
+                       kv_lora=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, qk_norm=False, dense_ff=5632)
+
+
+def mla_7b() -> ModelConfig:
+    return ModelConfig(arch="deepseek_v3", n_layer=30, hidden=4096, vocab=65536, n_head=32, n_kv_head=32, head_dim=192,
+                       kv_lora=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, qk_norm=False, dense_ff=11264)
+
+
 PRESETS = {
+    "tiny-pemezen": tiny_pemezen,
+    "pemezen-1b": pemezen_1b,
+    "pemezen-7b": pemezen_7b,
+    "mla-1b": mla_1b,
+    "mla-7b": mla_7b,
     "hybrid-4b": hybrid_4b,
     "hybrid-13b": hybrid_13b,
     "tiny-nisasun": tiny_nisasun,

@@ -15,6 +15,8 @@ Blocks (reference structure in parentheses):
   mla         Multi-head latent attention over a cached [latent | rope-key] row per token
   mamba2      Mamba-2 selective state space layer (``src/model/nemotron_h.rs``)
   lightning   linear attention with a constant decay per head (stacks with layer specifications)
+  latent      latent attention of a layer specification: own sizes, YaRN rotation, output gate
+  rglru       short convolution and a real-gated linear recurrent unit beside a GELU branch
   parallel    two mixers over the same input, here windowed attention beside a Mamba-2 mixer
   moe         router -> top-k -> routed experts (+ shared expert, + sigmoid shared gate)
               (``src/model/core.rs:4496-4640``); dense SwiGLU / GELU / ReLU^2 FFN
@@ -23,6 +25,7 @@ Blocks (reference structure in parentheses):
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
@@ -93,7 +96,8 @@ class KvCache:
             if cfg.layers is not None:
                 hk, dk, dv = cfg.kv_dims(il)
                 self.k[il] = torch.zeros(n_blocks, page, hk, dk, device=device, dtype=dtype)
-                self.v[il] = torch.zeros(n_blocks, page, hk, dv, device=device, dtype=dtype)
+                self.v[il] = (self.k[il] if cfg.latent_spec(il) is not None
+                              else torch.zeros(n_blocks, page, hk, dv, device=device, dtype=dtype))
             elif kinds[il] == "mla":
                 self.k[il] = torch.zeros(n_blocks, page, 1, cfg.kv_lora + cfg.qk_rope_dim, device=device, dtype=dtype)
                 self.v[il] = self.k[il]
@@ -157,6 +161,15 @@ class StatePool:
             kind = cfg.layer_kinds[il]
             if cfg.layers is not None:
                 r = cfg.recurrent_spec(il)
+                for which in cfg.conv_inputs(il):       # last inputs of a sublayer's input convolution, oldest first
+                    self.conv[il, which] = torch.zeros(n_slots, cfg.input_conv - 1, cfg.hidden, device=device,
+                                                       dtype=torch.float32)
+                if r is None:
+                    continue
+                if r.kind == "rglru":
+                    self.ssm[il] = torch.zeros(n_slots, r.width, device=device, dtype=torch.float32)
+                    self.conv[il] = torch.zeros(n_slots, r.width, r.conv - 1, device=device, dtype=torch.float32)
+                    continue
                 N = r.dim if r.kind == "lightning" else r.state
                 # state[head, value column, key column]
                 self.ssm[il] = torch.zeros(n_slots, r.heads, r.vdim, N, device=device, dtype=torch.float32)
@@ -350,6 +363,10 @@ class Decoder:
         for il in range(cfg.n_layer if cfg.layers is not None else 0):
             if cfg.layers[il].mixer.kind == "lightning":
                 self._decay[il] = torch.tensor(cfg.layers[il].mixer.decay, dtype=torch.float32, device=dev)
+        self._rot: Dict[tuple, torch.Tensor] = {}     # latent-attention layers: cos | sin table per rotation
+        for il in range(cfg.n_layer if cfg.layers is not None else 0):
+            if cfg.latent_spec(il) is not None:
+                self.rotary_table(cfg.latent_spec(il).rot, mp)
         tp = self.pctx.tp
         self.n_head_l = cfg.n_head // tp
         self.n_kv_l = max(1, cfg.n_kv_head // tp)
@@ -359,6 +376,15 @@ class Decoder:
         self.head_split = None            # (first row, rows) of this rank's slice of the vocabulary (split_head)
         self.expert_cache: Dict[str, object] = {}     # layer prefix -> residency.ExpertCache (offload modes)
         self._mla_uk: Dict[str, torch.Tensor] = {}    # layer prefix -> W_uk^T per head (absorb projection, K-major)
+
+    def rotary_table(self, r, max_position: int = 0) -> torch.Tensor:
+        """[positions, dims] cos | sin rows of a ``config.RotarySpec``."""
+        key = (r.dims, r.base, r.factor, r.original, r.fast, r.slow)
+        if key not in self._rot:
+            yarn = dict(type="yarn", factor=r.factor, original_max_position_embeddings=r.original, beta_fast=r.fast,
+                        beta_slow=r.slow, attention_factor=0.1 * math.log(r.factor) + 1.0) if r.original > 0 else None
+            self._rot[key] = ops.reference.rope_cos_sin(max_position, r.dims, r.base, yarn, device=self.device)
+        return self._rot[key]
 
     def offload_experts(self, n_slots: int, profile: Optional[dict] = None, ssd_dir: Optional[str] = None,
                         ram_experts: int = 0):
@@ -976,11 +1002,44 @@ class Decoder:
         n = ops.group_norm_gate(o, proj[:, 2 * nk + nv:], w[f"{p}.lin.norm"], cfg.rms_eps)
         return ops.linear(n, w[f"{p}.lin.out"])
 
+    def _latent_mixer(self, p: str, il: int, h, b: StepBatch, kv: KvCache):
+        """Latent attention in its absorbed form: queries moved into the latent space, attention over the cached rows,
+        value projection and output gate, output projection."""
+        cfg, w, m = self.cfg, self.w, self.cfg.layers[il].mixer
+        nq, nl = m.heads * (m.dim + m.rot_dim), m.kv_rank + m.rot_dim
+        proj = ops.linear(h, w[f"{p}.lat.in"])
+        gate = proj[:, nq + nl:nq + nl + m.gate_width()] if m.gate != "none" else None
+        q_abs = ops.latent_queries(proj[:, :nq], proj[:, nq:nq + nl], w[f"{p}.lat.uk"], w[f"{p}.lat.norm"], cfg.rms_eps,
+                                   self.rotary_table(m.rot), b.positions, b.slots, kv.k[il], m.heads, m.dim, m.rot_dim)
+        o = ops.latent_attention(q_abs, kv.k[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, m.scale, m.kv_rank,
+                                 max_ctx=b.max_ctx or None)
+        return ops.linear(ops.latent_values(o, w[f"{p}.lat.uv"], gate), w[f"{p}.lat.o"])
+
+    def _rglru_mixer(self, p: str, il: int, h, b: StepBatch, st: StatePool):
+        """Griffin's recurrent block. Its decode step runs convolution, gates, recurrence and the GELU branch as one
+        launch; prompts run the gates as one block-diagonal product and the recurrence in chunks."""
+        w, m = self.w, self.cfg.layers[il].mixer
+        W = m.width
+        proj = ops.linear(h, w[f"{p}.lru.in"])
+        in_b = w[f"{p}.lru.in_b"]
+        y, x = proj[:, :W], proj[:, W:]
+        u = ops.causal_conv1d_silu(x, w[f"{p}.lru.conv_w"], w[f"{p}.lru.conv_b"], st.conv[il], b.cu_q, b.state_slots,
+                                   write_state=b.write_state, max_len=b.max_q_len, in_bias=in_b[W:], silu=False)
+        gates = ops.block_gates(u, w[f"{p}.lru.gates"], m.blocks)
+        s = ops.gated_recurrence(u, gates, w[f"{p}.lru.gates_b"], w[f"{p}.lru.log_decay"], y, in_b[:W], st.ssm[il],
+                                 b.cu_q, b.state_slots, m.blocks, write_state=b.write_state, max_len=b.max_q_len,
+                                 cu_host=b.cu_q_host)
+        return ops.linear(s, w[f"{p}.lru.out"])
+
     def _spec_mixer(self, p: str, il: int, h, b: StepBatch, kv: KvCache, st: StatePool):
         """Output of layer il's mixer as [(tensor, scale)]: the terms are summed by the stream update that follows."""
         m = self.cfg.layers[il].mixer
         if m.kind == "lightning":
             return [(self._lightning_mixer(p, il, h, b, st), 1.0)]
+        if m.kind == "latent":
+            return [(self._latent_mixer(p, il, h, b, kv), 1.0)]
+        if m.kind == "rglru":
+            return [(self._rglru_mixer(p, il, h, b, st), 1.0)]
         proj = ops.linear(h, self.w[f"{p}.mix.in"])
         if m.kind == "ssd":
             return [(self._ssd_mixer(p, il, proj, b, st), 1.0)]
@@ -991,6 +1050,8 @@ class Decoder:
 
     def _spec_ffn(self, p: str, il: int, h):
         w, f = self.w, self.cfg.layers[il].mlp
+        if f.kind == "dense" and not f.gated():
+            return [(ops.linear(ops.up_act(h, w[f"{p}.mlp.up"], w[f"{p}.mlp.act"]), w[f"{p}.mlp.down"]), 1.0)]
         if f.kind == "dense":
             return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act), w[f"{p}.mlp.down"]), 1.0)]
         routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, 1.0, w.get(f"{p}.moe.router_bias"),
@@ -1021,6 +1082,39 @@ class Decoder:
             X, h = ops.hyper_step(X, terms, w[f"{hc}.st_mix"], w[f"{hc}.st_out"], in_w, norm_w, eps, off)
             if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
                 captures[il] = X.sum(1)
+        hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
+        out = StepOutput(hidden=hidden, captures=captures)
+        if want_logits:
+            out.logits = self.logits(hidden)
+        self.pctx.end_step()
+        return out
+
+    def _forward_sandwich(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool) -> StepOutput:
+        """Forward pass of a stack with layer specifications and one fp32 residual: every sublayer between two grouped
+        norms. Per sublayer one launch adds its normed output to the residual, norms that for the next sublayer and
+        applies the short input convolution with its carried history."""
+        cfg, w = self.cfg, self.w
+        G, eps = cfg.norm_groups, cfg.rms_eps
+        subs = [(il, which) for il, spec in enumerate(cfg.layers) for which in ("attn", "ffn")[:1 if spec.mlp is None else 2]]
+
+        def conv(i):
+            if not cfg.input_conv:
+                return None
+            il, which = subs[i]
+            return w[f"l{il}.{which}_taps"], st.conv[il, which], b.cu_q, b.state_slots, b.write_state
+
+        # rows given in place of the embedding are scaled like it
+        table, ids = (w["tok_embd"], b.token_ids) if b.embeds is None else (b.embeds, None)
+        x, h = ops.resid_start(table, ids, cfg.embed_scale, w["l0.attn_norm"], G, eps, conv(0), max_len=b.max_q_len)
+        captures: Dict[int, torch.Tensor] = {}
+        for i, (il, which) in enumerate(subs):
+            p, last = f"l{il}", i + 1 == len(subs)
+            terms = self._spec_mixer(p, il, h, b, kv, st) if which == "attn" else self._spec_ffn(p, il, h)
+            norm_w = w["output_norm"] if last else w[f"l{subs[i + 1][0]}.{subs[i + 1][1]}_norm"]
+            x, h = ops.resid_step(x, terms[0][0], w[f"{p}.{which}_post_norm"], norm_w, G, eps,
+                                  None if last else conv(i + 1), max_len=b.max_q_len)
+            if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
+                captures[il] = x
         hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
         out = StepOutput(hidden=hidden, captures=captures)
         if want_logits:
@@ -1275,6 +1369,8 @@ class Decoder:
         if self.pipe is not None:
             return self._forward_pipe(b, kv, st, want_logits)
         if self.cfg.layers is not None:
+            if self.cfg.sandwich_norm:
+                return self._forward_sandwich(b, kv, st, want_logits)
             return self._forward_streams(b, kv, st, want_logits)
         if self.cfg.hyper_streams > 1:
             return self._forward_hc(b, kv, st, want_logits)

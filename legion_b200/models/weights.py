@@ -146,6 +146,22 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
         s[f"{p}.lin.qkvg"] = (2 * m.heads * (m.dim + m.vdim), H)
         s[f"{p}.lin.norm"] = (m.heads * m.vdim,)
         s[f"{p}.lin.out"] = (H, m.heads * m.vdim)
+    elif m.kind == "latent":
+        s[f"{p}.lat.in"] = (latent_in_rows(m), H)                               # q | latent | shared key part | gate
+        s[f"{p}.lat.norm"] = (m.kv_rank,)
+        s[f"{p}.lat.uk"] = (m.heads * m.kv_rank, m.dim)                         # per head: key projection, transposed
+        s[f"{p}.lat.uv"] = (m.heads * m.vdim, m.kv_rank)
+        s[f"{p}.lat.o"] = (H, m.heads * m.vdim)
+    elif m.kind == "rglru":
+        d = m.width // m.blocks
+        s[f"{p}.lru.in"] = (2 * m.width, H)                                     # y | x
+        s[f"{p}.lru.in_b"] = (2 * m.width,)
+        s[f"{p}.lru.conv_w"] = (m.width, m.conv)
+        s[f"{p}.lru.conv_b"] = (m.width,)
+        s[f"{p}.lru.gates"] = (m.blocks * 2 * d, d)                             # per block: recurrence | input gate
+        s[f"{p}.lru.gates_b"] = (m.blocks * 2 * d,)
+        s[f"{p}.lru.log_decay"] = (m.width,)                                    # log of the decay at an open gate
+        s[f"{p}.lru.out"] = (H, m.width)
     else:
         a, r = cfg.attn_spec(il), cfg.recurrent_spec(il)
         rows = 0
@@ -166,7 +182,12 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
             s[f"{p}.ssm.out"] = (H, inner)
         s[f"{p}.mix.in"] = (rows, H)
     n = cfg.hyper_streams
-    for which in ("hca", "hcf")[:1 if spec.mlp is None else 2]:
+    if cfg.sandwich_norm:
+        for which in ("attn", "ffn")[:1 if spec.mlp is None else 2]:
+            s[f"{p}.{which}_post_norm"] = (H,)
+            if cfg.input_conv:
+                s[f"{p}.{which}_taps"] = (cfg.input_conv, H)                    # oldest token first
+    for which in () if cfg.sandwich_norm else ("hca", "hcf")[:1 if spec.mlp is None else 2]:
         s[f"{p}.{which}.st_in"] = (n,)                  # streams -> sublayer input
         s[f"{p}.{which}.st_out"] = (n,)                 # sublayer output -> streams
         s[f"{p}.{which}.st_mix"] = (n, n)               # stream (row) -> stream (column)
@@ -179,10 +200,19 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
             s[f"{p}.moe.router_bias"] = (f.experts,)
         s[f"{p}.moe.gate_up"] = (f.experts, 2 * f.ff, H)
         s[f"{p}.moe.down"] = (f.experts, H, f.ff)
+    elif not f.gated():
+        s[f"{p}.mlp.up"] = (f.ff, H)
+        s[f"{p}.mlp.act"] = (2,)
+        s[f"{p}.mlp.down"] = (H, f.ff)
     else:
         s[f"{p}.mlp.gate_up"] = (2 * f.ff, H)
         s[f"{p}.mlp.down"] = (H, f.ff)
     return s
+
+
+def latent_in_rows(m) -> int:
+    """Rows of a latent layer's stacked input projection, padded so that its output rows start on 16-byte boundaries."""
+    return -(-(m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim + m.gate_width()) // 8) * 8
 
 
 def gemma_layer_shapes(cfg: ModelConfig, il: int, s: Dict[str, Tuple[int, ...]]) -> Dict[str, Tuple[int, ...]]:
@@ -261,7 +291,8 @@ def is_fp32_weight(name: str) -> bool:
     leaf = name.rsplit(".", 1)[-1]
     return leaf.endswith("norm") or leaf in ("A", "D", "dt_bias", "conv_w", "conv_b", "router_bias", "hc_f", "hc_scale",
                                              "hc_base", "hcg_norm", "hcg_down", "hcg_up", "hcg_inject", "router_scale",
-                                             "out_scale", "st_in", "st_out", "st_mix")
+                                             "out_scale", "st_in", "st_out", "st_mix", "in_b", "gates_b", "log_decay",
+                                             "act", "attn_taps", "ffn_taps")
 
 
 def layer_of(name: str) -> Optional[int]:
@@ -298,7 +329,11 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=torch.float32, seed: in
             t = -(torch.rand(shp, generator=g) * 0.9 + 0.1).to(device)
         elif leaf == "D":
             t = torch.ones(shp, dtype=torch.float32, device=device)
-        elif leaf in ("dt_bias", "conv_b", "router_bias"):
+        elif leaf == "log_decay":         # decays from 0.9 to 0.999 at a half-open gate
+            t = (2 * torch.log(0.9 + 0.099 * torch.rand(shp, generator=g))).to(device)
+        elif leaf == "act":               # xIELU: softplus(p), 1/2 + softplus(q)
+            t = torch.tensor([0.8, 1.3], device=device)
+        elif leaf in ("dt_bias", "conv_b", "router_bias", "in_b", "gates_b"):
             t = (torch.randn(shp, generator=g) * 0.1).to(device)
         elif leaf in ("st_in", "st_out", "st_mix"):
             n = shp[0]                    # near the plain residual: the streams' mean in, every stream gets the output
@@ -310,7 +345,7 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=torch.float32, seed: in
             t = (torch.randn(shp, generator=g) * 0.5).to(device)
         elif leaf in ("hc_f", "hcg_down", "hcg_up", "hcg_inject"):
             t = (torch.randn(shp, generator=g) * 0.05).to(device)
-        elif leaf == "conv_w":
+        elif leaf in ("conv_w", "attn_taps", "ffn_taps"):
             t = (torch.randn(shp, generator=g) * 0.3).to(device)
         elif device.type == "cuda" and wd == torch.bfloat16:
             from ..ops.sm100 import ext

@@ -192,10 +192,62 @@ def embed(ids, table):
     return table[ids.long()]
 
 
-def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, max_len=None):
+def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, max_len=None, in_bias=None, silu=True):
     if _cuda(x):
-        return _sm.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state, max_len=max_len)
-    return _ref.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state)
+        return _sm.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state, max_len=max_len, in_bias=in_bias,
+                                      silu=silu)
+    return _ref.causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state, in_bias, silu)
+
+
+def up_act(x, w, ab):
+    """Un-gated feed-forward input: xIELU(x w^T) with the activation's two numbers ``ab`` (float32)."""
+    return _sm.up_act(x, w, ab) if _cuda(x) else _ref.up_act(x, w, ab)
+
+
+def resid_start(table, ids, embed_scale, norm_w, groups, eps, conv=None, max_len=None):
+    """Start of a stack with one fp32 residual: x = embedding rows * scale (``ids`` None: rows are given). Returns
+    (x [T, H] float32, input of the first sublayer); ``conv`` as in ``reference.resid_step``."""
+    if _cuda(table):
+        return _sm.resid_step(None, None, None, norm_w, groups, eps, conv, start=(table, ids, embed_scale),
+                              max_len=max_len)
+    x = (table if ids is None else table[ids.long()]).float() * embed_scale
+    return _ref.resid_step(x, None, None, norm_w, groups, eps, table.dtype, conv)
+
+
+def resid_step(x, y, post_w, norm_w, groups, eps, conv=None, max_len=None):
+    """Behind a sublayer with output y: x + norm(y), the norm of that and its input convolution, in one launch.
+    Returns (new x, input of the next sublayer)."""
+    if _cuda(x):
+        return _sm.resid_step(x, y, post_w, norm_w, groups, eps, conv, max_len=max_len)
+    return _ref.resid_step(x, y, post_w, norm_w, groups, eps, y.dtype, conv)
+
+
+def latent_queries(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, heads, dim, rot_dim):
+    f = _sm.latent_queries if _cuda(q) else _ref.latent_queries
+    return f(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, heads, dim, rot_dim)
+
+
+def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, max_ctx=None):
+    if _cuda(q_abs):
+        return _sm.latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, max_ctx)
+    return _ref.latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, scale, rank)
+
+
+def latent_values(o_lat, uv, gate):
+    return _sm.latent_values(o_lat, uv, gate) if _cuda(o_lat) else _ref.latent_values(o_lat, uv, gate)
+
+
+def block_gates(u, w, blocks):
+    """Block-diagonal product, float32 result [T, rows of w]."""
+    return _sm.block_gates(u, w, blocks) if _cuda(u) else _ref.head_linear(u, w, blocks)
+
+
+def gated_recurrence(u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks, write_state=True, max_len=None,
+                     cu_host=None):
+    if _cuda(u):
+        return _sm.gated_recurrence(u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks, write_state,
+                                    max_len, cu_host)
+    return _ref.gated_recurrence(u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks, write_state)
 
 
 def hyper_start(table, ids, streams, in_w, norm_w, eps, w_offset=0.0):

@@ -89,9 +89,7 @@ def rope_cos_sin(max_pos: int, rot: int, theta: float, scaling: Optional[dict] =
             if scaling.get("truncate", True):
                 lo, hi = math.floor(lo), math.ceil(hi)
             lo, hi = max(lo, 0), min(hi, rot - 1)
-            if lo == hi:
-                hi += 0.001
-            ramp = ((torch.arange(half, dtype=torch.float64, device=device) - lo) / (hi - lo)).clamp(0, 1)
+            ramp = ((torch.arange(half, dtype=torch.float64, device=device) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
             inv_freq = inv_freq / factor * ramp + inv_freq * (1 - ramp)
             mag = yarn_attention_factor(scaling)
     pos = torch.arange(max_pos, dtype=torch.float64, device=device)
@@ -263,8 +261,9 @@ def argmax(logits):
     return torch.argmax(logits.float(), dim=-1).int()
 
 
-def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool = True):
-    """x: [T, C]; w: [C, KC]; conv_state: [slots, C, KC-1] float32 (oldest first)."""
+def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool = True, in_bias=None, silu: bool = True):
+    """x: [T, C]; w: [C, KC]; conv_state: [slots, C, KC-1] float32 (oldest first). ``in_bias`` is added to x first (the
+    history holds the sums; before a sequence's start there is zero)."""
     out = torch.empty_like(x)
     KC = w.shape[1]
     for i in range(len(slots)):
@@ -273,12 +272,13 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool 
             continue
         s = int(slots[i])
         hist = conv_state[s].float().t()  # [KC-1, C]
-        seq = torch.cat([hist, x[t0:t1].float()], dim=0)
+        rows = x[t0:t1].float() if in_bias is None else x[t0:t1].float() + in_bias.float()
+        seq = torch.cat([hist, rows], dim=0)
         win = seq.unfold(0, KC, 1)  # [n, C, KC]
         y = (win * w.float()[None]).sum(-1)
         if bias is not None:
             y = y + bias.float()
-        out[t0:t1] = F.silu(y).to(x.dtype)
+        out[t0:t1] = (F.silu(y) if silu else y).to(x.dtype)
         if write_state and KC > 1:
             conv_state[s] = seq[-(KC - 1):].t().to(conv_state.dtype)
     return out
@@ -401,6 +401,111 @@ def group_norm_gate(y, gate, w, eps: float, groups: int = 1):
     if gate is not None:
         out = out * torch.sigmoid(gate.float())
     return out.to(y.dtype)
+
+
+def xielu(z, ab):
+    """a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise; ab = (a, b) float32."""
+    n = z.clamp(max=0)
+    return torch.where(z > 0, ab[0] * z * z, ab[1] * (torch.expm1(n) - n)) + 0.5 * z
+
+
+def up_act(x, w, ab):
+    return xielu(x.float() @ w.float().t(), ab).to(x.dtype)
+
+
+def group_rms(x, w, groups: int, eps: float):
+    """RMS norm in ``groups`` equal parts of a float32 row, times w."""
+    v = x.reshape(*x.shape[:-1], groups, -1)
+    return (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape) * w
+
+
+def resid_step(x, y, post_w, norm_w, groups: int, eps: float, dtype, conv=None):
+    """x [T, H] float32 -> (x + norm(y), h): h = n + conv(n) with n the norm of the new x. y None: x as it is.
+    ``conv`` = (taps [K, H] oldest first, history [slots, K - 1, H], cu_seq, slots, write_state) or None."""
+    if y is not None:
+        x = x + group_rms(y.float(), post_w, groups, eps)
+    n = group_rms(x, norm_w, groups, eps)
+    if conv is None:
+        return x, n.to(dtype)
+    taps, hist, cu, slots, write = conv
+    K = taps.shape[0]
+    h = torch.empty_like(n)
+    for i in range(len(slots)):
+        t0, t1 = int(cu[i]), int(cu[i + 1])
+        if t1 <= t0:
+            continue
+        seq = torch.cat([hist[int(slots[i])], n[t0:t1]], 0)
+        h[t0:t1] = n[t0:t1] + sum(taps[j] * seq[j:j + t1 - t0] for j in range(K))
+        if write and K > 1:
+            hist[int(slots[i])] = seq[seq.shape[0] - (K - 1):]
+    return x, h.to(dtype)
+
+
+def rotate_pairs(x, cos_sin, positions):
+    """x [T, ..., D] float32: neighbouring columns (2i, 2i + 1) of the first cos_sin.shape[1] columns turn."""
+    r = cos_sin.shape[1]
+    cs = cos_sin[positions.long()].view(x.shape[0], *[1] * (x.dim() - 2), r)
+    c, s = cs[..., :r // 2], cs[..., r // 2:]
+    u, v = x[..., 0:r:2], x[..., 1:r:2]
+    out = x.clone()
+    out[..., 0:r:2], out[..., 1:r:2] = u * c - v * s, v * c + u * s
+    return out
+
+
+def latent_queries(q, kv, uk, norm_w, eps: float, cos_sin, positions, slots, cache, heads: int, dim: int, rot_dim: int):
+    """Cache rows [norm(latent) | rotated key part] at the tokens' cells; returns [T, heads, rank + rot_dim]: queries in
+    the latent space and their rotated part."""
+    T, L = q.shape[0], norm_w.numel()
+    kvf = kv.float()
+    c = group_rms(kvf[:, :L], norm_w, 1, eps)
+    row = torch.cat([c, rotate_pairs(kvf[:, L:L + rot_dim], cos_sin, positions)], 1).to(cache.dtype)
+    valid = slots >= 0
+    cache.view(-1, cache.shape[-1])[slots[valid], :L + rot_dim] = row[valid]
+    qh = q.float().reshape(T, heads, dim + rot_dim)
+    qa = torch.einsum("thd,hld->thl", qh[..., :dim], uk.float().view(heads, L, dim))
+    return torch.cat([qa, rotate_pairs(qh[..., dim:], cos_sin, positions)], 2).to(q.dtype)
+
+
+def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, scale: float, rank: int):
+    """Causal attention of q_abs [T, heads, D] over cache rows [D, ...]; values are a row's first ``rank`` columns."""
+    D = q_abs.shape[2]
+    k = cache[..., :D]
+    return paged_attention(q_abs, k, k, block_table, ctx_lens, cu_q, scale)[..., :rank]
+
+
+def latent_values(o_lat, uv, gate):
+    """Per-head value projection and output gate: gate [T, heads * vdim], [T, heads] or None."""
+    T, H, L = o_lat.shape
+    o = torch.einsum("thl,hvl->thv", o_lat.float(), uv.float().view(H, -1, L))
+    if gate is not None:
+        g = torch.sigmoid(gate.float())
+        o = o * (g[:, :, None] if gate.shape[1] == H else g.view(o.shape))
+    return o.reshape(T, -1).to(o_lat.dtype)
+
+
+def head_linear(x, w, heads: int):
+    """x in ``heads`` equal parts, each times its own matrix: w [heads * n, k]; float32 [T, heads * n]."""
+    xh = x.float().view(x.shape[0], heads, -1)
+    return torch.einsum("thk,hnk->thn", xh, w.float().view(heads, -1, xh.shape[2])).reshape(x.shape[0], -1)
+
+
+def gated_recurrence(u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks: int, write_state: bool = True):
+    """RG-LRU over the step's tokens: gates float32 [T, blocks, 2, width / blocks] (recurrence, input; before bias and
+    sigmoid), a = exp(sigmoid(r) log_decay), S = a S + sqrt(1 - a^2) sigmoid(i) u; returns S * gelu(y + y_b)."""
+    T, W = u.shape
+    z = torch.sigmoid((gates.reshape(T, -1) + gates_b).view(T, blocks, 2, -1))
+    r, i = z[:, :, 0].reshape(T, W), z[:, :, 1].reshape(T, W)
+    la = r * log_decay
+    a, b = torch.exp(la), torch.sqrt(-torch.expm1(2 * la)) * i * u.float()
+    out = torch.empty(T, W, dtype=torch.float32, device=u.device)
+    for n in range(len(slots)):
+        S = state[int(slots[n])].clone()
+        for t in range(int(cu_seq[n]), int(cu_seq[n + 1])):
+            S = a[t] * S + b[t]
+            out[t] = S
+        if write_state:
+            state[int(slots[n])] = S
+    return (out * F.gelu(y.float() + y_b, approximate="tanh")).to(u.dtype)
 
 
 def sample(logits, temperature, top_k, top_p, min_p, generator=None):
