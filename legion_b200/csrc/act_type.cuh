@@ -48,6 +48,10 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+  return z > 0.f ? z * fmaf(a, z, 0.5f) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
 __device__ __forceinline__ float warp_sum_f(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

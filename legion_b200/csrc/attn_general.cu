@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(128) qkv_norm_append_kernel(const T* __restric
 // One warp per (token, query head). 32 keys at a time: lane = key for the scores, then lane = value columns.
 template <typename T, int NV>
 __global__ void __launch_bounds__(128) paged_attn_general_kernel(
-    const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, long k_cell, long v_cell,
+    const T* __restrict__ q, long q_row, const T* __restrict__ k_cache, const T* __restrict__ v_cache, long k_cell, long v_cell,
     const int* __restrict__ cu_q, const int* __restrict__ ctx_lens, const int* __restrict__ block_table, int table_width,
     int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, int window, T* __restrict__ out) {
   extern __shared__ float q_sm[];
@@ -83,7 +83,7 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
   const int pos = ctx_lens[seq] - (cu_q[seq + 1] - t);
   const int kvh = h / (Hq / Hkv);
   float* qs = q_sm + warp * DK;
-  for (int d = lane; d < DK; d += 32) qs[d] = ld_f(q + (long(t) * Hq + h) * DK + d);
+  for (int d = lane; d < DK; d += 32) qs[d] = ld_f(q + (long(t) * Hq + h) * q_row + d);
   __syncwarp();
   const int* bt = block_table + long(seq) * table_width;
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;
@@ -137,7 +137,7 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
 }
 
 template <typename T>
-int attn_t(const void* q, const void* k, const void* v, long k_cell, long v_cell, const int* cu_q, const int* ctx_lens,
+int attn_t(const void* q, long q_row, const void* k, const void* v, long k_cell, long v_cell, const int* cu_q, const int* ctx_lens,
            const int* bt, int tw, int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, int window,
            void* out, cudaStream_t s) {
   const long warps = long(nT) * Hq;
@@ -146,10 +146,10 @@ int attn_t(const void* q, const void* k, const void* v, long k_cell, long v_cell
   if (smem > 40 * 1024) return 1;
 #define LB_NV(N)                                                                                                       \
   if (DV <= 32 * N)                                                                                                    \
-    return launch_pdl(paged_attn_general_kernel<T, N>, grid, dim3(128), smem, s, static_cast<const T*>(q),             \
+    return launch_pdl(paged_attn_general_kernel<T, N>, grid, dim3(128), smem, s, static_cast<const T*>(q), q_row,      \
                       static_cast<const T*>(k), static_cast<const T*>(v), k_cell, v_cell, cu_q, ctx_lens, bt, tw,      \
                       page, n_seqs, nT, Hq, Hkv, DK, DV, scale, window, static_cast<T*>(out)) != cudaSuccess;
-  LB_NV(2) LB_NV(4) LB_NV(8) LB_NV(16)
+  LB_NV(2) LB_NV(4) LB_NV(8) LB_NV(16) LB_NV(32)
 #undef LB_NV
   return 1;
 }
@@ -171,15 +171,15 @@ int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld,
 #undef LB_T
 }
 
-int paged_attn_general_launch(const void* q, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
+int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
                               int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, int window, void* out,
                               bool f32, cudaStream_t s) {
   if (T <= 0 || n_seqs <= 0) return 0;
   if (page <= 0 || Hkv <= 0 || Hq % Hkv) return 1;
-  return f32 ? attn_t<float>(q, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page, n_seqs,
+  return f32 ? attn_t<float>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page, n_seqs,
                              T, Hq, Hkv, DK, DV, scale, window, out, s)
-             : attn_t<__nv_bfloat16>(q, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page,
+             : attn_t<__nv_bfloat16>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page,
                                      n_seqs, T, Hq, Hkv, DK, DV, scale, window, out, s);
 }
 

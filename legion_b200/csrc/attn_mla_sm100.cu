@@ -1,11 +1,13 @@
 // Multi-head latent attention (MLA) over the paged latent cache, absorbed form, on tcgen05 for sm_100a.
 //
-// A cache row is [c_kv (512) | k_pe (64)] in bf16: every head of a token reads the SAME row, as key (all 576
-// columns) and as value (the first 512). Queries arrive already absorbed into the latent space,
-// q_abs = [q_nope W_uk | rope(q_pe)] (576 per head), and the kernel returns o_lat = softmax(q_abs . row) . c_kv
-// (512 per head); the caller applies W_uv and the output projection.
+// A cache row is [c_kv (L) | k_pe (R)] in bf16 (512 + 64 in the DeepSeek models): every head of a token reads the SAME
+// row, as key (all L + R columns) and as value (the first L). Queries arrive already absorbed into the latent space,
+// q_abs = [q_nope W_uk | rope(q_pe)] (L + R per head), and the kernel returns o_lat = softmax(q_abs . row) . c_kv
+// (L per head); the caller applies W_uv and the output projection. L up to 512 and L + R up to 576, multiples of 8: the
+// tensor maps end at L + R and TMA fills the rest of the last 64-column half with zeros. Any head count.
 //
-// One CTA = 64 query rows (G heads x 64/G consecutive tokens of one sequence) over one split of the keys:
+// One CTA = up to 64 query rows (G heads x TQ consecutive tokens of one sequence) over one split of the keys. The sizes
+// in this description are those of L + R = 576 (HALVES = 9):
 //   warp 5 (one lane)  TMA producer: Q tile once, then 64-key latent tiles through the block table into a two-stage
 //                      ring (nine 64-column halves per tile, 128-byte swizzle). ONE tile in shared memory serves
 //                      both MMAs: K-major B operand of S = Q K^T and MN-major B operand of O += P V.
@@ -31,16 +33,14 @@ namespace lb {
 
 namespace {
 
-constexpr int MLA_L = 512;                 // latent (value) width
-constexpr int MLA_R = 64;                  // rope width
-constexpr int MLA_DK = MLA_L + MLA_R;      // 576
-constexpr int MLA_HALVES = MLA_DK / 64;    // 9
+constexpr int MLA_L = 512;                 // widths of the append kernel below
+constexpr int MLA_R = 64;
+constexpr int MLA_DK = MLA_L + MLA_R;
 constexpr int MLA_BKV = 64;
 constexpr int MLA_ROWS = 64;
-constexpr int MLA_Q_BYTES = MLA_HALVES * MLA_ROWS * 128;    // 73,728
-constexpr int MLA_KV_BYTES = MLA_HALVES * MLA_BKV * 128;    // 73,728
 constexpr int MLA_P_BYTES = MLA_ROWS * 128;                 // 8,192
-constexpr int MLA_SMEM = MLA_Q_BYTES + 2 * MLA_KV_BYTES + MLA_P_BYTES + 256 + 1024;
+constexpr int mla_tile_bytes(int halves) { return halves * MLA_ROWS * 128; }     // 73,728 for nine halves
+constexpr int mla_smem(int halves) { return 3 * mla_tile_bytes(halves) + MLA_P_BYTES + 256 + 1024; }
 constexpr float MLA_RESCALE_LOG2 = 8.f;
 
 __device__ __forceinline__ void mla_tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
@@ -61,17 +61,21 @@ struct MlaArgs {
   const int* ctx_lens;     // [n_seqs] keys visible after this step
   const int* block_table;  // [n_seqs, table_width]
   int table_width, page;
-  int nh, G, TQ;           // heads, heads per tile, tokens per tile (G * TQ == 64)
+  int nh, G, TQ;           // heads, heads per tile, tokens per tile (G * TQ <= 64)
+  int L;                   // value width
+  int tm_cols;             // TMEM columns: two S buffers and the value width
   int head_blocks, n_splits;
   float scale_log2;
-  __nv_bfloat16* out;      // [T, nh, 512] (n_splits == 1)
-  float* o_part;           // [T * nh, n_splits, 512]
+  __nv_bfloat16* out;      // [T, nh, L] (n_splits == 1)
+  float* o_part;           // [T * nh, n_splits, L]
   float* ml_part;          // [T * nh, n_splits, 2] (max in natural-log units, sum)
   int* status;
 };
 
+template <int MLA_HALVES>
 __global__ void __launch_bounds__(192, 1)
 mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const MlaArgs a) {
+  constexpr int MLA_Q_BYTES = mla_tile_bytes(MLA_HALVES), MLA_KV_BYTES = MLA_Q_BYTES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* q_s = smem;
@@ -110,7 +114,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     mbar_fence_init();
   }
   if (warp == 4) {
-    tmem_alloc(tmem_slot, 512);
+    tmem_alloc(tmem_slot, uint32_t(a.tm_cols));
     tmem_relinquish();
   }
   tc_fence_before();
@@ -134,7 +138,8 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   if (warp == 5) {
     if (lane == 0 && n_blk > 0) {
       // ---------------------------------------------------------------- TMA producer
-      mbar_expect_tx(q_full, MLA_Q_BYTES);
+      // rows past G * TQ stay as they are: they are rows of S and O that nobody reads
+      mbar_expect_tx(q_full, uint32_t(MLA_HALVES * a.G * a.TQ * 128));
 #pragma unroll
       for (int h = 0; h < MLA_HALVES; ++h)
         tma_load_3d(q_s + h * (MLA_ROWS * 128), &tmQ, q_full, h * 64, hb * a.G, q0 + tok0);
@@ -161,7 +166,10 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (lane == 0 && n_blk > 0) {
       // ---------------------------------------------------------------- MMA issue
       constexpr uint32_t idesc_s = umma_idesc(64, MLA_BKV, 1, 1, 0, 0);
-      constexpr uint32_t idesc_o = umma_idesc(64, 256, 1, 1, 0, 1);   // B (= latent tile as V) is MN-major
+      // B (= latent tile as V) is MN-major; the value width in parts of 256 columns, the last rounded up to 16
+      const uint32_t idesc_o = umma_idesc(64, 256, 1, 1, 0, 1);
+      const int n_full = a.L / 256, n_rest = (a.L % 256 + 15) / 16 * 16;
+      const uint32_t idesc_r = umma_idesc(64, uint32_t(n_rest), 1, 1, 0, 1);
       const uint64_t dq0 = umma_desc_k_sw128(smem_u32(q_s));
       const uint64_t dp0 = umma_desc_k_sw128(smem_u32(p_s));
       auto issue_s = [&](int j) {
@@ -179,13 +187,14 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       };
       auto issue_pv = [&](int j) {
         const uint64_t dv0 = umma_desc_mn_sw128(smem_u32(kv_s + (j & 1) * MLA_KV_BYTES), MLA_BKV * 128, 1024);
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
+#pragma unroll 2
+        for (int n = 0; n < n_full + (n_rest > 0); ++n) {
+          const uint32_t idesc = n < n_full ? idesc_o : idesc_r;
 #pragma unroll
           for (int k = 0; k < MLA_BKV / 16; ++k) {
             // A = P (K-major, 16 keys = 32 B per step); B = 256 latent columns (4 halves) of 16 key rows
             const uint64_t db = dv0 + uint64_t((n * 4 * (MLA_BKV * 128) + k * 16 * 128) >> 4);
-            umma_f16(tmem_O + n * 256, dp0 + uint64_t((k * 32) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
+            umma_f16(tmem_O + n * 256, dp0 + uint64_t((k * 32) >> 4), db, idesc, (j | k) ? 1u : 0u);
           }
         }
         umma_commit(&kv_empty[j & 1]);
@@ -311,7 +320,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         tc_fence_after();
         waited = true;
 #pragma unroll 1
-        for (int c = 0; c < MLA_L; c += 32) {
+        for (int c = 0; c < a.L; c += 32) {
           uint32_t o[32];
           tmem_ld32(tmem_base + lane_off + c, o);
           tmem_ld_wait();
@@ -353,12 +362,12 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       tc_fence_after();
       const float m_o = m, l_o = l;
       const long grow = long(q0 + tok0 + tq) * a.nh + head;         // global (token, head) row
-      const bool write = !s_lane && row_ok;
+      const bool write = !s_lane && row_ok && head < a.nh;
       if (a.n_splits == 1) {
         const float inv = l_o > 0.f ? 1.f / l_o : 0.f;
-        __nv_bfloat16* orow = a.out + grow * MLA_L;
+        __nv_bfloat16* orow = a.out + grow * a.L;
 #pragma unroll 1
-        for (int c = 0; c < MLA_L; c += 32) {
+        for (int c = 0; c < a.L; c += 32) {
           uint32_t o[32];
           if (n_blk > 0) {
             tmem_ld32(tmem_base + lane_off + c, o);
@@ -371,6 +380,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             uint4* dst = reinterpret_cast<uint4*>(orow + c);
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
+              if (c + 8 * v >= a.L) break;
               uint4 u;
               u.x = pack_bf16x2(__uint_as_float(o[8 * v + 0]) * inv, __uint_as_float(o[8 * v + 1]) * inv);
               u.y = pack_bf16x2(__uint_as_float(o[8 * v + 2]) * inv, __uint_as_float(o[8 * v + 3]) * inv);
@@ -381,14 +391,14 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           }
         }
       } else {
-        float* orow = a.o_part + (grow * a.n_splits + split) * MLA_L;
+        float* orow = a.o_part + (grow * a.n_splits + split) * a.L;
         if (write) {
           float* ml = a.ml_part + (grow * a.n_splits + split) * 2;
           ml[0] = (n_blk > 0 && m_o != -INFINITY) ? m_o * 0.6931471805599453f : -INFINITY;
           ml[1] = n_blk > 0 ? l_o : 0.f;
         }
 #pragma unroll 1
-        for (int c = 0; c < MLA_L; c += 32) {
+        for (int c = 0; c < a.L; c += 32) {
           uint32_t o[32];
           if (n_blk > 0) {
             tmem_ld32(tmem_base + lane_off + c, o);
@@ -401,7 +411,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             float4* dst = reinterpret_cast<float4*>(orow + c);
 #pragma unroll
             for (int v = 0; v < 8; ++v)
-              dst[v] = make_float4(__uint_as_float(o[4 * v]), __uint_as_float(o[4 * v + 1]),
+              if (c + 4 * v < a.L) dst[v] = make_float4(__uint_as_float(o[4 * v]), __uint_as_float(o[4 * v + 1]),
                                    __uint_as_float(o[4 * v + 2]), __uint_as_float(o[4 * v + 3]));
           }
         }
@@ -412,7 +422,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   __syncthreads();
   if (warp == 4) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
+    tmem_dealloc(tmem_base, uint32_t(a.tm_cols));
   }
 }
 
@@ -467,6 +477,26 @@ mla_prep_kernel(const __nv_bfloat16* __restrict__ kva, long ld_kva, const float*
 
 thread_local char g_mla_err[256];
 
+template <int HALVES>
+int mla_start(const CUtensorMap& tq, const CUtensorMap& tc, const MlaArgs& a, dim3 grid, cudaStream_t s) {
+  constexpr int smem = mla_smem(HALVES);
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(mla_attn_kernel<HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+      snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: cannot set %d bytes of shared memory", smem);
+      return 1;
+    }
+    attr = true;
+  }
+  mla_attn_kernel<HALVES><<<grid, 192, smem, s>>>(tq, tc, a);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) {
+    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention launch: %s", cudaGetErrorString(e));
+    return 1;
+  }
+  return 0;
+}
+
 }  // namespace
 
 int mla_prep_launch(const void* kva, long ld_kva, const float* norm_w, float eps, float w_offset, const void* q,
@@ -483,21 +513,21 @@ int mla_prep_launch(const void* kva, long ld_kva, const float* norm_w, float eps
 
 const char* mla_attn_last_error() { return g_mla_err; }
 
-// q_abs [T, nh, 576] bf16; cache rows [n_cells, 576] bf16 with pitch cell_stride elements; out [T, nh, 512] bf16.
-// o_part / ml_part: workspaces of T * nh * n_splits * 512 and T * nh * n_splits * 2 floats (n_splits > 1).
-int mla_attn_launch(const void* q_abs, long T, const void* cache, long n_cells, long cell_stride, const int* cu_q,
-                    const int* ctx_lens, const int* block_table, int table_width, int page, int n_seqs,
-                    int max_q_len, int nh, float scale, int n_splits, float* o_part, float* ml_part, void* out,
-                    int* status, cudaStream_t s) {
+// q_abs [T, nh, L + R] bf16 with row pitch q_pitch; cache rows [n_cells, L + R] bf16 with pitch cell_stride elements; out
+// [T, nh, L] bf16. o_part / ml_part: workspaces of T * nh * n_splits * L and T * nh * n_splits * 2 floats (n_splits > 1).
+int mla_attn_launch(const void* q_abs, long q_pitch, long T, const void* cache, long n_cells, long cell_stride,
+                    const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page, int n_seqs,
+                    int max_q_len, int nh, int L, int R, float scale, int n_splits, float* o_part, float* ml_part,
+                    void* out, bool merge, int* status, cudaStream_t s) {
   if (n_seqs <= 0 || max_q_len <= 0 || T <= 0) return 0;
   if (page <= 0 || MLA_BKV % page != 0 || page % 8 != 0) {
     snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: page size %d must be a multiple of 8 dividing %d", page,
              MLA_BKV);
     return 1;
   }
-  int G = nh >= 64 ? 64 : nh;
-  if (nh <= 0 || (nh >= 64 && nh % 64 != 0) || (nh < 64 && (64 % nh) != 0)) {
-    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: %d heads (need a divisor or a multiple of 64)", nh);
+  const int DK = L + R, halves = (DK + 63) / 64;
+  if (nh <= 0 || L <= 0 || R < 0 || L > 512 || halves > 9 || L % 8 || (L + 15) / 16 * 16 > halves * 64) {
+    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: %d heads, latent %d, rotated part %d", nh, L, R);
     return 1;
   }
   if (n_splits < 1) n_splits = 1;
@@ -505,41 +535,36 @@ int mla_attn_launch(const void* q_abs, long T, const void* cache, long n_cells, 
     snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: split keys need the partial workspaces");
     return 1;
   }
-  if (cell_stride % 8 != 0) {
-    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: cache row pitch %ld must be a multiple of 8", cell_stride);
+  if (cell_stride % 8 != 0 || q_pitch % 8 != 0) {
+    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: row pitches %ld and %ld must be multiples of 8", cell_stride,
+             q_pitch);
     return 1;
   }
-  const int TQ = 64 / G;
-  const CUtensorMap* tq = tmap_3d(q_abs, uint64_t(MLA_DK), uint64_t(nh), uint64_t(T), uint64_t(MLA_DK) * 2,
-                                  uint64_t(nh) * MLA_DK * 2, 64, uint32_t(G), uint32_t(TQ), TM_BF16, true);
-  const CUtensorMap* tc = tmap_2d(cache, uint64_t(n_cells), uint64_t(MLA_DK), uint64_t(cell_stride) * 2,
+  const int head_blocks = (nh + 63) / 64, G = (nh + head_blocks - 1) / head_blocks, TQ = 64 / G;
+  const CUtensorMap* tq = tmap_3d(q_abs, uint64_t(DK), uint64_t(nh), uint64_t(T), uint64_t(q_pitch) * 2,
+                                  uint64_t(nh) * q_pitch * 2, 64, uint32_t(G), uint32_t(TQ), TM_BF16, true);
+  const CUtensorMap* tc = tmap_2d(cache, uint64_t(n_cells), uint64_t(DK), uint64_t(cell_stride) * 2,
                                   uint32_t(page), 64, TM_BF16, true);
   if (!tq || !tc) {
     snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: %s", tmap_last_error());
     return 1;
   }
-  static bool attr = false;
-  if (!attr) {
-    if (cudaFuncSetAttribute(mla_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MLA_SMEM) != cudaSuccess) {
-      snprintf(g_mla_err, sizeof(g_mla_err), "mla attention: cannot set %d bytes of shared memory", MLA_SMEM);
-      return 1;
-    }
-    attr = true;
-  }
   MlaArgs a{};
   a.cu_q = cu_q; a.ctx_lens = ctx_lens; a.block_table = block_table; a.table_width = table_width; a.page = page;
-  a.nh = nh; a.G = G; a.TQ = TQ; a.head_blocks = nh / G; a.n_splits = n_splits;
+  a.nh = nh; a.G = G; a.TQ = TQ; a.head_blocks = head_blocks; a.n_splits = n_splits;
+  a.L = L;
+  a.tm_cols = L > 256 ? 512 : (L > 128 ? 256 : 128);
   a.scale_log2 = scale * 1.4426950408889634f;
   a.out = static_cast<__nv_bfloat16*>(out); a.o_part = o_part; a.ml_part = ml_part; a.status = status;
   const int q_tiles = (max_q_len + TQ - 1) / TQ;
   dim3 grid(unsigned(q_tiles) * a.head_blocks * n_splits, unsigned(n_seqs));
-  mla_attn_kernel<<<grid, 192, MLA_SMEM, s>>>(*tq, *tc, a);
-  cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) {
-    snprintf(g_mla_err, sizeof(g_mla_err), "mla attention launch: %s", cudaGetErrorString(e));
-    return 1;
-  }
-  if (n_splits > 1) return attn_combine_launch(o_part, ml_part, n_splits, int(T) * nh, MLA_L, out, s);
+  int rc = 1;
+#define LB_HALVES(N) \
+  if (halves == N) rc = mla_start<N>(*tq, *tc, a, grid, s);
+  LB_HALVES(1) LB_HALVES(2) LB_HALVES(3) LB_HALVES(4) LB_HALVES(5) LB_HALVES(6) LB_HALVES(7) LB_HALVES(8) LB_HALVES(9)
+#undef LB_HALVES
+  if (rc) return 1;
+  if (n_splits > 1 && merge) return attn_combine_launch(o_part, ml_part, n_splits, int(T) * nh, L, out, s);
   return 0;
 }
 

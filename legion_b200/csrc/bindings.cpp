@@ -43,7 +43,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
            const OptT& ws, const OptT& counters, Tensor& status, const OptT& tile_group, const OptT& tile_tok0,
            const OptT& tile_ntok, const OptT& meta, int64_t max_tiles, int64_t rows_per_group, int64_t n_tok,
            std::vector<int64_t> out_peer, const OptT& tile_out0, const OptT& w_scales, const OptT& w_gscale,
-           int64_t x_group_col, int64_t k_override, int64_t act) {
+           int64_t x_group_col, int64_t k_override, int64_t act, const OptT& xielu) {
   const bool fp4 = w_scales.has_value();     // w = NVFP4 codes [rows, K/2] uint8, w_scales = e4m3 bytes [rows, K/16]
   if (fp4) {
     TORCH_CHECK(w.scalar_type() == at::kByte && w_scales->is_contiguous() && w_scales->element_size() == 1 &&
@@ -79,6 +79,11 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
   h.w_scales = fp4 ? w_scales->data_ptr() : nullptr;
   h.w_gscale = optp<float>(w_gscale);
   h.bn = int(bn); h.dual = dual; h.act = int(act);
+  if (xielu.has_value()) {
+    TORCH_CHECK(!dual && xielu->scalar_type() == at::kFloat && xielu->is_cuda() && xielu->numel() == 2,
+                "wgemm: xIELU takes two float32 numbers and one weight tile");
+    h.xielu = xielu->data_ptr<float>();
+  }
   h.tile_group = optp<int>(tile_group); h.tile_tok0 = optp<int>(tile_tok0); h.tile_ntok = optp<int>(tile_ntok);
   h.n_tiles_dev = optp<int>(meta);
   h.tile_out0 = optp<int>(tile_out0);
@@ -379,28 +384,31 @@ void prefill_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(rc == 0, lb::prefill_attn_last_error());
 }
 
-#ifndef LB_CORE
 void mla_attn(const Tensor& q_abs, const Tensor& cache, const Tensor& cu_q, const Tensor& ctx_lens,
               const Tensor& block_table, int64_t page, int64_t max_q_len, double scale, int64_t n_splits,
-              const OptT& o_part, const OptT& ml_part, Tensor& out, Tensor& status) {
+              const OptT& o_part, const OptT& ml_part, const OptT& out, int64_t rank, int64_t rot, bool merge,
+              Tensor& status) {
   check_bf16(q_abs, "q_abs");
   check_bf16(cache, "cache");
-  TORCH_CHECK(q_abs.dim() == 3 && q_abs.size(2) == 576 && q_abs.is_contiguous(), "mla_attn: q_abs must be [T, heads, 576]");
-  TORCH_CHECK(cache.size(-1) == 576 && cache.is_contiguous(), "mla_attn: cache rows must be [.., 576]");
-  TORCH_CHECK(out.is_contiguous() && out.size(-1) == 512 && out.numel() == q_abs.size(0) * q_abs.size(1) * 512,
-              "mla_attn: out must be [T, heads, 512]");
+  const int64_t dk = rank + rot;
+  TORCH_CHECK(q_abs.dim() == 3 && q_abs.size(2) >= dk && q_abs.is_contiguous(), "mla_attn: q_abs must be [T, heads, >= ", dk, "]");
+  TORCH_CHECK(cache.size(-1) >= dk && cache.is_contiguous(), "mla_attn: cache rows must be [.., >= ", dk, "]");
   const long T = q_abs.size(0);
   const int nh = int(q_abs.size(1));
+  TORCH_CHECK(n_splits > 1 && !merge ? true : out.has_value() && out->is_contiguous() && out->size(-1) == rank &&
+                                                  out->numel() == T * nh * rank,
+              "mla_attn: out must be [T, heads, ", rank, "]");
   if (n_splits > 1) {
-    TORCH_CHECK(o_part.has_value() && ml_part.has_value() && o_part->numel() >= T * nh * n_splits * 512 &&
+    TORCH_CHECK(o_part.has_value() && ml_part.has_value() && o_part->numel() >= T * nh * n_splits * rank &&
                     ml_part->numel() >= T * nh * n_splits * 2, "mla_attn: partial workspaces too small");
   }
   c10::cuda::CUDAGuard guard(q_abs.device());
-  const int rc = lb::mla_attn_launch(q_abs.data_ptr(), T, cache.data_ptr(), cache.numel() / 576, 576,
-                                     cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
-                                     int(block_table.size(1)), int(page), int(ctx_lens.numel()), int(max_q_len), nh,
-                                     float(scale), int(n_splits), optpm<float>(o_part), optpm<float>(ml_part),
-                                     out.data_ptr(), reinterpret_cast<int*>(status.data_ptr()), cur_stream());
+  const int rc = lb::mla_attn_launch(q_abs.data_ptr(), q_abs.size(2), T, cache.data_ptr(), cache.numel() / cache.size(-1),
+                                     cache.size(-1), cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(),
+                                     block_table.data_ptr<int>(), int(block_table.size(1)), int(page), int(ctx_lens.numel()),
+                                     int(max_q_len), nh, int(rank), int(rot), float(scale), int(n_splits),
+                                     optpm<float>(o_part), optpm<float>(ml_part), out.has_value() ? out->data_ptr() : nullptr,
+                                     merge, reinterpret_cast<int*>(status.data_ptr()), cur_stream());
   TORCH_CHECK(rc == 0, lb::mla_attn_last_error());
 }
 
@@ -425,7 +433,6 @@ void mla_prep(const Tensor& kva, const Tensor& norm_w, double eps, double w_offs
                                   cache.data_ptr(), 576, q_abs.data_ptr(), int(kva.size(0)), cur_stream()) == 0,
               "mla_prep launch failed");
 }
-#endif
 
 void router_topk(const Tensor& logits, const OptT& bias, int64_t k, int64_t mode, bool renorm, double route_scale,
                  int64_t n_group, int64_t topk_group, Tensor& ids, Tensor& wts, int64_t group_top) {
@@ -597,7 +604,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         pybind11::arg("tile_ntok"), pybind11::arg("meta"), pybind11::arg("max_tiles"), pybind11::arg("rows_per_group"),
         pybind11::arg("n_tok"), pybind11::arg("out_peer"), pybind11::arg("tile_out0") = pybind11::none(),
         pybind11::arg("w_scales") = pybind11::none(), pybind11::arg("w_gscale") = pybind11::none(),
-        pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0, pybind11::arg("act") = 0);
+        pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0, pybind11::arg("act") = 0,
+        pybind11::arg("xielu") = pybind11::none());
   m.def("wgemm_fp8", &wgemm_fp8);
   m.def("wgemm_fp8_q", &wgemm_fp8_q);
   m.def("wgemm_allreduce", &wgemm_allreduce);
@@ -609,10 +617,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("embed", &embed);
   m.def("paged_decode", &paged_decode);
   m.def("prefill_attn", &prefill_attn);
-#ifndef LB_CORE
   m.def("mla_attn", &mla_attn);
   m.def("mla_prep", &mla_prep);
-#endif
   m.def("router_topk", &router_topk, pybind11::arg("logits"), pybind11::arg("bias"), pybind11::arg("k"),
         pybind11::arg("mode"), pybind11::arg("renorm"), pybind11::arg("route_scale"), pybind11::arg("n_group"),
         pybind11::arg("topk_group"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("group_top") = 2);

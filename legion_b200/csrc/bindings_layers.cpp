@@ -85,6 +85,29 @@ lb::LinScanArgs scan_args(const Tensor& q, const Tensor& k, const Tensor& v, boo
   a.write_state = write_state;
   return a;
 }
+
+lb::DiagScanArgs diag_args(int64_t T, int64_t W, const Tensor& gates_b, const Tensor& log_decay, const Tensor& y,
+                           const Tensor& y_b, Tensor& state, const Tensor& cu, const Tensor& slots, int64_t blocks,
+                           Tensor& out, bool f32) {
+  same(y, f32, "y");
+  same(out, f32, "out");
+  TORCH_CHECK(blocks >= 1 && W % blocks == 0 && y.dim() == 2 && y.size(0) == T && y.size(1) == W && out.dim() == 2 &&
+                  out.size(0) == T && out.size(1) == W, "diag_scan: y and out [T, W], W in equal blocks");
+  f32c(gates_b, 2 * W, "gate bias");
+  f32c(log_decay, W, "log decay");
+  f32c(y_b, W, "y bias");
+  TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() == 2 && state.size(1) == W,
+              "diag_scan: state [slots, W] float32");
+  TORCH_CHECK(cu.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && cu.numel() == slots.numel() + 1,
+              "diag_scan: int32 sequence bounds and slots");
+  lb::DiagScanArgs a{};
+  a.gates_b = gates_b.data_ptr<float>(); a.log_decay = log_decay.data_ptr<float>();
+  a.y = y.data_ptr(); a.ldy = y.stride(0); a.y_b = y_b.data_ptr<float>();
+  a.state = state.data_ptr<float>(); a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>();
+  a.n_seqs = int(slots.numel()); a.T = int(T); a.W = int(W); a.blocks = int(blocks);
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  return a;
+}
 }  // namespace
 
 void bind_layers(pybind11::module_& m) {
@@ -140,10 +163,12 @@ void bind_layers(pybind11::module_& m) {
   m.def("sgemm", [](const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, const OptT& tok_scale,
                     const OptT& out_rows, int64_t n_feat, bool dual, int64_t dual_offset, int64_t act,
                     const OptT& tile_group, const OptT& tile_tok0, const OptT& tile_ntok, const OptT& meta,
-                    int64_t max_tiles, int64_t rows_per_group, int64_t n_tok) {
+                    int64_t max_tiles, int64_t rows_per_group, int64_t n_tok, const OptT& act_ab) {
     const bool f32 = is_f32(x, "x");
     same(w, f32, "w");
     TORCH_CHECK(w.dim() == 2 && x.dim() == 2 && out.dim() == 2 && w.size(1) == x.size(1), "sgemm: K mismatch");
+    if (act_ab.has_value()) f32c(*act_ab, 2, "activation numbers");
+    TORCH_CHECK(act != 3 || (act_ab.has_value() && !dual), "sgemm: xIELU takes two numbers");
     is_f32(out, "out");
     TORCH_CHECK(out.size(1) >= n_feat && w.size(0) >= n_feat + (dual ? dual_offset : 0), "sgemm: shapes");
     lb::SgemmArgs a{};
@@ -155,7 +180,7 @@ void bind_layers(pybind11::module_& m) {
     }
     a.tok_scale = optp<float>(tok_scale); a.out_rows = optp<int>(out_rows);
     a.T = int(n_tok); a.K = int(x.size(1)); a.N = int(n_feat);
-    a.dual = dual; a.dual_offset = dual_offset; a.act = int(act);
+    a.dual = dual; a.dual_offset = dual_offset; a.act = int(act); a.act_ab = optp<float>(act_ab);
     a.tile_group = optp<int>(tile_group); a.tile_tok0 = optp<int>(tile_tok0); a.tile_ntok = optp<int>(tile_ntok);
     a.n_tiles = optp<int>(meta); a.max_tiles = int(max_tiles); a.rows_per_group = rows_per_group;
     TORCH_CHECK(!a.tile_group || (a.tile_tok0 && a.tile_ntok && a.n_tiles), "sgemm: incomplete tile tables");
@@ -200,12 +225,12 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_table.scalar_type() == at::kInt &&
                     cu_q.numel() == ctx_lens.numel() + 1 && block_table.stride(1) == 1, "paged_attn_general: int32 tables");
     c10::cuda::CUDAGuard guard(q.device());
-    TORCH_CHECK(lb::paged_attn_general_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
+    TORCH_CHECK(lb::paged_attn_general_launch(q.data_ptr(), DK, k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
                                               cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
                                               int(block_table.stride(0)), int(k_cache.size(-3)), int(ctx_lens.numel()),
                                               int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), int(window),
                                               out.data_ptr(), f32, cur_stream()) == 0,
-                "paged_attn_general: value heads of at most 512 columns, key heads of at most 2560", cuda_error());
+                "paged_attn_general: value heads of at most 1024 columns, key heads of at most 2560", cuda_error());
   });
   m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
                           const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state, const Tensor& cu,
@@ -276,18 +301,22 @@ void bind_layers(pybind11::module_& m) {
                 "group_norm_gate failed", cuda_error());
   });
   m.def("conv1d_silu", [](const Tensor& x, const Tensor& w, const OptT& bias, Tensor& conv_state, const Tensor& cu_seq,
-                          const Tensor& slots, Tensor& out, bool write_state, int64_t max_len) {
+                          const Tensor& slots, Tensor& out, bool write_state, int64_t max_len, const OptT& in_bias,
+                          bool silu) {
     c10::cuda::CUDAGuard guard(x.device());
     TORCH_CHECK(x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kFloat, "conv1d_silu dtypes");
+    if (in_bias.has_value()) f32c(*in_bias, x.size(1), "input bias");
     TORCH_CHECK(lb::conv1d_silu_launch(x.data_ptr(), x.stride(0), w.data_ptr<float>(), optp<float>(bias),
                                        conv_state.data_ptr<float>(), cu_seq.data_ptr<int>(), slots.data_ptr<int>(),
                                        int(slots.numel()), int(x.size(1)), int(w.size(1)), out.data_ptr(),
-                                       out.stride(0), write_state ? 1 : 0, cur_stream(), int(max_len)) == 0,
+                                       out.stride(0), write_state ? 1 : 0, cur_stream(), int(max_len),
+                                       optp<float>(in_bias), silu) == 0,
                 "conv1d_silu: unsupported kernel width");
   });
   m.def("conv_silu_any", [](const Tensor& x, const Tensor& w, const OptT& bias, Tensor& conv_state, const Tensor& cu,
-                            const Tensor& slots, Tensor& out, bool write_state) {
+                            const Tensor& slots, Tensor& out, bool write_state, const OptT& in_bias, bool silu) {
     const bool f32 = is_f32(x, "x");
+    if (in_bias.has_value()) f32c(*in_bias, x.size(1), "input bias");
     same(out, f32, "out");
     const int64_t T = x.size(0), C = x.size(1), KC = w.size(1);
     TORCH_CHECK(w.size(0) == C && out.size(0) == T && out.size(1) == C && conv_state.is_contiguous() &&
@@ -298,7 +327,180 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::conv_silu_any_launch(x.data_ptr(), x.stride(0), w.data_ptr<float>(), optp<float>(bias),
                                          conv_state.data_ptr<float>(), cu.data_ptr<int>(), slots.data_ptr<int>(),
                                          int(slots.numel()), int(T), int(C), int(KC), out.data_ptr(), out.stride(0),
-                                         write_state, f32, cur_stream()) == 0,
+                                         write_state, optp<float>(in_bias), silu, f32, cur_stream()) == 0,
                 "conv_silu_any: at most 65535 tokens per step", cuda_error());
+  });
+  // per-head products: out[t, h * out_col + n] = sum_k x[t, h * x_col + k] w[h * rows + n, k]
+  m.def("sgemm_heads", [](const Tensor& w, const Tensor& x, Tensor& out, int64_t heads, int64_t rows, int64_t n_feat, int64_t K,
+                          int64_t x_col, int64_t out_col) {
+    const bool f32 = is_f32(x, "x");
+    same(w, f32, "w");
+    is_f32(out, "out");
+    TORCH_CHECK(heads >= 1 && heads <= 65535 && w.dim() == 2 && x.dim() == 2 && out.dim() == 2 && w.size(1) == K &&
+                    w.size(0) >= (heads - 1) * rows + n_feat && x.size(1) >= (heads - 1) * x_col + K &&
+                    out.size(0) == x.size(0) && out.size(1) >= (heads - 1) * out_col + n_feat, "sgemm_heads: shapes");
+    lb::SgemmArgs a{};
+    a.x = x.data_ptr(); a.ldx = x.stride(0); a.w = w.data_ptr(); a.ldw = w.stride(0);
+    a.out = out.data_ptr(); a.ldo = out.stride(0); a.out_f32 = out.scalar_type() == at::kFloat;
+    a.T = int(x.size(0)); a.K = int(K); a.N = int(n_feat);
+    a.heads = int(heads); a.x_head_col = x_col; a.out_head_col = out_col; a.rows_per_group = rows;
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::sgemm_launch(a, f32, cur_stream()) == 0, "sgemm_heads failed", cuda_error());
+  });
+  m.def("resid_step", [](const OptT& x_in, Tensor& x_out, const OptT& emb, const OptT& ids, double emb_scale, const OptT& y,
+                         const OptT& post_w, const Tensor& norm_w, int64_t groups, double eps, const OptT& taps,
+                         const OptT& hist, const OptT& cu, const OptT& slots, bool write_state, int64_t max_len, int64_t tok,
+                         Tensor& h) {
+    const bool f32 = is_f32(h, "h");
+    TORCH_CHECK(x_out.dim() == 2 && x_out.is_contiguous() && x_out.scalar_type() == at::kFloat,
+                "resid_step: the residual is contiguous float32 [rows, width]");
+    const int64_t R = x_out.size(0), H = x_out.size(1);
+    TORCH_CHECK(h.dim() == 2 && h.size(0) == R && h.size(1) == H, "resid_step: h [rows, width]");
+    TORCH_CHECK(groups >= 1 && H % groups == 0, "resid_step: the width must divide into ", groups, " groups");
+    lb::ResidStepArgs a{};
+    a.x_out = x_out.data_ptr<float>();
+    if (x_in.has_value()) {
+      TORCH_CHECK(x_in->sizes() == x_out.sizes() && x_in->is_contiguous() && x_in->scalar_type() == at::kFloat &&
+                      x_in->data_ptr() != x_out.data_ptr(), "resid_step: x_in like x_out, in a buffer of its own");
+      TORCH_CHECK(y.has_value() && post_w.has_value(), "resid_step: sublayer output and its norm");
+      same(*y, f32, "y");
+      TORCH_CHECK(y->dim() == 2 && y->size(0) == R && y->size(1) == H, "resid_step: y [rows, width]");
+      f32c(*post_w, H, "post norm");
+      a.x_in = x_in->data_ptr<float>();
+      a.y = y->data_ptr(); a.ldy = y->stride(0); a.post_w = post_w->data_ptr<float>();
+    } else {
+      TORCH_CHECK(emb.has_value() && emb->dim() == 2 && emb->size(1) == H, "resid_step: embedding rows");
+      same(*emb, f32, "emb");
+      a.emb = emb->data_ptr(); a.ld_emb = emb->stride(0); a.vocab = int(emb->size(0)); a.emb_scale = float(emb_scale);
+      if (ids.has_value()) {
+        TORCH_CHECK(ids->scalar_type() == at::kInt && ids->is_contiguous() && ids->numel() == R, "resid_step: int32 ids");
+        a.ids = ids->data_ptr<int>();
+      } else {
+        TORCH_CHECK(emb->size(0) >= R, "resid_step: one embedding row per token");
+      }
+    }
+    f32c(norm_w, H, "norm_w");
+    a.norm_w = norm_w.data_ptr<float>(); a.eps = float(eps); a.groups = int(groups);
+    a.rows = int(R); a.H = int(H);
+    a.h = h.data_ptr(); a.ldh = h.stride(0);
+    a.n_seqs = int(R); a.max_len = 1; a.tok = 1;
+    if (taps.has_value()) {
+      TORCH_CHECK(taps->dim() == 2 && taps->size(1) == H && cu.has_value() && slots.has_value() && hist.has_value(),
+                  "resid_step: taps [taps, width], history, bounds and slots");
+      const int64_t K = taps->size(0);
+      f32c(*taps, K * H, "taps");
+      TORCH_CHECK(hist->scalar_type() == at::kFloat && hist->is_contiguous() && hist->dim() == 3 && hist->size(1) == K - 1 &&
+                      hist->size(2) == H, "resid_step: history [slots, taps - 1, width] float32");
+      TORCH_CHECK(cu->scalar_type() == at::kInt && slots->scalar_type() == at::kInt && cu->numel() == slots->numel() + 1,
+                  "resid_step: int32 sequence bounds and slots");
+      a.taps = taps->data_ptr<float>(); a.taps_n = int(K); a.hist = hist->data_ptr<float>();
+      a.cu = cu->data_ptr<int>(); a.slots = slots->data_ptr<int>(); a.n_seqs = int(slots->numel());
+      a.max_len = int(max_len); a.tok = int(tok);
+    }
+    a.write_state = write_state;
+    c10::cuda::CUDAGuard guard(h.device());
+    TORCH_CHECK(lb::resid_step_launch(a, f32, cur_stream()) == 0, "resid_step: width ", H, ", ", groups, " groups, ",
+                a.taps_n, " taps, ", a.tok, " tokens per block", cuda_error());
+  });
+  m.def("latent_prep", [](const Tensor& q, const Tensor& kv, const Tensor& norm_w, double eps, const Tensor& cos_sin,
+                          const Tensor& positions, const Tensor& slots, Tensor& cache, Tensor& q_abs, int64_t dim, int64_t rot) {
+    const bool f32 = is_f32(q, "q");
+    same(kv, f32, "kv");
+    same(cache, f32, "cache");
+    same(q_abs, f32, "q_abs");
+    const int64_t T = q.size(0), H = q_abs.size(1), L = norm_w.numel();
+    TORCH_CHECK(q.dim() == 2 && kv.dim() == 2 && kv.size(0) == T && q.size(1) >= H * (dim + rot) && kv.size(1) >= L + rot,
+                "latent_prep: q [T, heads * (dim + rot)], kv [T, rank + rot]");
+    TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && q_abs.size(0) == T && q_abs.size(2) >= L + rot &&
+                    cache.is_contiguous() && cache.size(-1) >= L + rot, "latent_prep: rows of rank + rot columns");
+    f32c(norm_w, L, "norm");
+    TORCH_CHECK(cos_sin.dim() == 2, "latent_prep: table [positions, rotated columns]");
+    f32c(cos_sin, 0, "cos_sin");
+    TORCH_CHECK(positions.scalar_type() == at::kInt && slots.scalar_type() == at::kLong && positions.numel() == T &&
+                    slots.numel() == T, "latent_prep: positions int32, slots int64");
+    lb::LatentPrepArgs a{};
+    a.q = q.data_ptr(); a.ldq = q.stride(0); a.kv = kv.data_ptr(); a.ldkv = kv.stride(0);
+    a.norm_w = norm_w.data_ptr<float>(); a.eps = float(eps);
+    a.cos_sin = cos_sin.data_ptr<float>(); a.rot = int(cos_sin.size(1));
+    a.positions = positions.data_ptr<int>(); a.slots = reinterpret_cast<const long*>(slots.data_ptr());
+    a.cache = cache.data_ptr(); a.cell = cache.size(-1); a.q_abs = q_abs.data_ptr(); a.q_row = q_abs.size(2);
+    a.T = int(T); a.heads = int(H); a.dim = int(dim); a.R = int(rot); a.L = int(L);
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::latent_prep_launch(a, f32, cur_stream()) == 0, "latent_prep failed", cuda_error());
+  });
+  m.def("latent_attn_general", [](const Tensor& q_abs, const Tensor& cache, const Tensor& cu_q, const Tensor& ctx_lens,
+                                  const Tensor& block_table, double scale, int64_t rank, int64_t rot, Tensor& out) {
+    const bool f32 = is_f32(q_abs, "q_abs");
+    same(cache, f32, "cache");
+    same(out, f32, "out");
+    const int64_t T = q_abs.size(0), H = q_abs.size(1), cell = cache.size(-1);
+    TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && cache.is_contiguous() && cache.dim() == 4 && cell >= rank + rot &&
+                    q_abs.size(2) >= rank + rot && out.is_contiguous() && out.numel() == T * H * rank,
+                "latent_attn_general: rows of rank + rot columns");
+    TORCH_CHECK(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_table.scalar_type() == at::kInt &&
+                    block_table.stride(1) == 1 && cu_q.numel() == ctx_lens.numel() + 1, "latent_attn_general: int32 tables");
+    c10::cuda::CUDAGuard guard(q_abs.device());
+    TORCH_CHECK(lb::paged_attn_general_launch(q_abs.data_ptr(), q_abs.size(2), cache.data_ptr(), cache.data_ptr(), cell, cell,
+                                              cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
+                                              int(block_table.stride(0)), int(cache.size(1)), int(ctx_lens.numel()), int(T),
+                                              int(H), 1, int(rank + rot), int(rank), float(scale), 0, out.data_ptr(), f32,
+                                              cur_stream()) == 0,
+                "latent_attn_general: latents of at most 1024 columns", cuda_error());
+  });
+  m.def("latent_gate", [](Tensor& x, const Tensor& gate, int64_t heads) {
+    const bool f32 = is_f32(x, "x");
+    same(gate, f32, "gate");
+    const int64_t T = x.size(0), N = x.size(1);
+    TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && gate.dim() == 2 && gate.size(0) == T && N % heads == 0 &&
+                    (gate.size(1) == N || gate.size(1) == heads), "latent_gate: one gate per column or per head");
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::latent_gate_launch(x.data_ptr(), gate.data_ptr(), gate.stride(0), gate.size(1) != N, int(N / heads), int(N),
+                                       int(T), f32, cur_stream()) == 0, "latent_gate failed", cuda_error());
+  });
+  m.def("diag_scan", [](const Tensor& u, Tensor& gates, const Tensor& gates_b, const Tensor& log_decay, const Tensor& y,
+                        const Tensor& y_b, Tensor& state, const Tensor& cu, const Tensor& slots, int64_t blocks, Tensor& out,
+                        bool write_state, int64_t max_tokens, const OptT& tables, int64_t n_chunks, const OptT& ends) {
+    const bool f32 = is_f32(u, "u");
+    lb::DiagScanArgs a = diag_args(u.size(0), u.size(1), gates_b, log_decay, y, y_b, state, cu, slots, blocks, out, f32);
+    f32c(gates, u.size(0) * 2 * u.size(1), "gates");
+    a.u = u.data_ptr(); a.ldu = u.stride(0); a.gates = gates.data_ptr<float>();
+    a.write_state = write_state; a.max_tokens = int(max_tokens);
+    c10::cuda::CUDAGuard guard(u.device());
+    if (!tables.has_value()) {
+      TORCH_CHECK(lb::diag_scan_launch(a, f32, cur_stream()) == 0, "diag_scan failed", cuda_error());
+      return;
+    }
+    TORCH_CHECK(tables->scalar_type() == at::kInt && tables->is_contiguous() && tables->numel() == 3 * n_chunks + 2 * a.n_seqs &&
+                    ends.has_value(), "diag_scan: chunk tables");
+    f32c(*ends, n_chunks * 2 * u.size(1), "chunk ends");
+    const int* t = tables->data_ptr<int>();
+    TORCH_CHECK(lb::diag_chunk_launch(a, t, t + n_chunks, int(n_chunks), t + 3 * n_chunks, t + 3 * n_chunks + a.n_seqs,
+                                      ends->data_ptr<float>(), f32, cur_stream()) == 0, "diag_scan failed", cuda_error());
+  });
+  m.def("diag_decode", [](const Tensor& x, const Tensor& in_bias, const Tensor& conv_w, const OptT& conv_b, Tensor& conv_state,
+                          const Tensor& gates_w, const Tensor& gates_b, const Tensor& log_decay, const Tensor& y,
+                          const Tensor& y_b, Tensor& state, const Tensor& cu, const Tensor& slots, int64_t blocks, Tensor& ctr,
+                          Tensor& out) {
+    const bool f32 = is_f32(x, "x");
+    const int64_t n = x.size(0), W = x.size(1), K = conv_w.size(1);
+    TORCH_CHECK(n == slots.numel(), "diag_decode: one token per sequence");
+    lb::DiagDecodeArgs a{};
+    a.s = diag_args(n, W, gates_b, log_decay, y, y_b, state, cu, slots, blocks, out, f32);
+    a.s.write_state = 1;
+    same(gates_w, f32, "gate weights");
+    TORCH_CHECK(gates_w.is_contiguous() && gates_w.numel() == 2 * W * (W / blocks), "diag_decode: gate weights [blocks, 2, d, d]");
+    f32c(conv_w, W * K, "conv weight");
+    f32c(in_bias, W, "input bias");
+    if (conv_b.has_value()) f32c(*conv_b, W, "conv bias");
+    TORCH_CHECK(conv_state.scalar_type() == at::kFloat && conv_state.is_contiguous() && conv_state.dim() == 3 &&
+                    conv_state.size(1) == W && conv_state.size(2) == K - 1, "diag_decode: history [slots, W, taps - 1]");
+    TORCH_CHECK(ctr.scalar_type() == at::kInt && ctr.is_contiguous() &&
+                    ctr.numel() >= (n + lb::DIAG_DECODE_SEQ - 1) / lb::DIAG_DECODE_SEQ * blocks, "diag_decode: counters");
+    a.x = x.data_ptr(); a.ldx = x.stride(0); a.in_bias = in_bias.data_ptr<float>();
+    a.conv_w = conv_w.data_ptr<float>(); a.conv_b = optp<float>(conv_b); a.conv_state = conv_state.data_ptr<float>();
+    a.KC = int(K); a.gates_w = gates_w.data_ptr();
+    a.ctr = reinterpret_cast<unsigned int*>(ctr.data_ptr());
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::diag_decode_launch(a, f32, cur_stream()) == 0, "diag_decode failed", cuda_error());
   });
 }

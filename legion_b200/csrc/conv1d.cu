@@ -15,7 +15,8 @@ __global__ void __launch_bounds__(128) conv1d_silu_kernel(const __nv_bfloat16* _
                                                           float* __restrict__ conv_state,
                                                           const int* __restrict__ cu_seq,
                                                           const int* __restrict__ slots, int C,
-                                                          __nv_bfloat16* __restrict__ out, long ldo, int write_state) {
+                                                          __nv_bfloat16* __restrict__ out, long ldo, int write_state,
+                                                          const float* __restrict__ in_bias, int silu) {
   const int c = blockIdx.x * 128 + threadIdx.x;
   const int seq = blockIdx.y;
   if (c >= C) return;
@@ -27,16 +28,16 @@ __global__ void __launch_bounds__(128) conv1d_silu_kernel(const __nv_bfloat16* _
   float* st = conv_state + (long(slot) * C + c) * (KC - 1);
 #pragma unroll
   for (int j = 0; j < KC - 1; ++j) h[j] = st[j];
-  const float b = bias ? bias[c] : 0.f;
+  const float b = bias ? bias[c] : 0.f, ib = in_bias ? in_bias[c] : 0.f;
   for (int t = t0; t < t1; ++t) {
-    const float xv = __bfloat162float(x[t * ldx + c]);
+    const float xv = __bfloat162float(x[t * ldx + c]) + ib;
     float acc = b + wv[KC - 1] * xv;
 #pragma unroll
     for (int j = 0; j < KC - 1; ++j) acc += wv[j] * h[j];
 #pragma unroll
     for (int j = 0; j < KC - 2; ++j) h[j] = h[j + 1];
     h[KC - 2] = xv;
-    out[t * ldo + c] = __float2bfloat16(acc / (1.f + __expf(-acc)));
+    out[t * ldo + c] = __float2bfloat16(silu ? acc / (1.f + __expf(-acc)) : acc);
   }
   if (write_state) {
 #pragma unroll
@@ -56,7 +57,8 @@ __global__ void __launch_bounds__(128) conv1d_silu_prompt_kernel(const __nv_bflo
                                                                  const int* __restrict__ cu_seq,
                                                                  const int* __restrict__ slots, int C, int tok_per_cta,
                                                                  __nv_bfloat16* __restrict__ out, long ldo,
-                                                                 int write_state) {
+                                                                 int write_state, const float* __restrict__ in_bias,
+                                                                 int silu) {
   const int c = blockIdx.x * 128 + threadIdx.x;
   const int seq = blockIdx.z;
   const int t0 = cu_seq[seq], t1 = cu_seq[seq + 1];
@@ -68,22 +70,22 @@ __global__ void __launch_bounds__(128) conv1d_silu_prompt_kernel(const __nv_bflo
 #pragma unroll
   for (int j = 0; j < KC; ++j) wv[j] = w[c * KC + j];
   float* st = conv_state + (long(slot) * C + c) * (KC - 1);
+  const float b = bias ? bias[c] : 0.f, ib = in_bias ? in_bias[c] : 0.f;
   // h[j] = input of token ta - (KC - 1) + j: from x when that token belongs to this step, else from the history
 #pragma unroll
   for (int j = 0; j < KC - 1; ++j) {
     const int t = ta - (KC - 1) + j;
-    h[j] = t >= t0 ? __bfloat162float(x[long(t) * ldx + c]) : st[(KC - 1) + (t - t0)];
+    h[j] = t >= t0 ? __bfloat162float(x[long(t) * ldx + c]) + ib : st[(KC - 1) + (t - t0)];
   }
-  const float b = bias ? bias[c] : 0.f;
   for (int t = ta; t < tb; ++t) {
-    const float xv = __bfloat162float(x[long(t) * ldx + c]);
+    const float xv = __bfloat162float(x[long(t) * ldx + c]) + ib;
     float acc = b + wv[KC - 1] * xv;
 #pragma unroll
     for (int j = 0; j < KC - 1; ++j) acc += wv[j] * h[j];
 #pragma unroll
     for (int j = 0; j < KC - 2; ++j) h[j] = h[j + 1];
     h[KC - 2] = xv;
-    out[long(t) * ldo + c] = __float2bfloat16(acc / (1.f + __expf(-acc)));
+    out[long(t) * ldo + c] = __float2bfloat16(silu ? acc / (1.f + __expf(-acc)) : acc);
   }
   (void)write_state;   // the history is replaced by conv1d_state_kernel after this kernel
 }
@@ -93,7 +95,8 @@ template <int KC>
 __global__ void __launch_bounds__(128) conv1d_state_kernel(const __nv_bfloat16* __restrict__ x, long ldx,
                                                            float* __restrict__ conv_state,
                                                            const int* __restrict__ cu_seq,
-                                                           const int* __restrict__ slots, int C) {
+                                                           const int* __restrict__ slots, int C,
+                                                           const float* __restrict__ in_bias) {
   const int c = blockIdx.x * 128 + threadIdx.x;
   const int seq = blockIdx.y;
   if (c >= C) return;
@@ -104,7 +107,7 @@ __global__ void __launch_bounds__(128) conv1d_state_kernel(const __nv_bfloat16* 
 #pragma unroll
   for (int j = 0; j < KC - 1; ++j) {
     const int t = t1 - (KC - 1) + j;
-    h[j] = t >= t0 ? __bfloat162float(x[long(t) * ldx + c]) : st[(KC - 1) + (t - t0)];
+    h[j] = t >= t0 ? __bfloat162float(x[long(t) * ldx + c]) + (in_bias ? in_bias[c] : 0.f) : st[(KC - 1) + (t - t0)];
   }
 #pragma unroll
   for (int j = 0; j < KC - 1; ++j) st[j] = h[j];
@@ -112,7 +115,7 @@ __global__ void __launch_bounds__(128) conv1d_state_kernel(const __nv_bfloat16* 
 
 int conv1d_silu_launch(const void* x, long ldx, const float* w, const float* bias, float* conv_state,
                        const int* cu_seq, const int* slots, int n_seqs, int C, int KC, void* out, long ldo,
-                       int write_state, cudaStream_t s, int max_len) {
+                       int write_state, cudaStream_t s, int max_len, const float* in_bias, int silu) {
   if (n_seqs <= 0) return 0;
   auto xb = static_cast<const __nv_bfloat16*>(x);
   auto ob = static_cast<__nv_bfloat16*>(out);
@@ -124,8 +127,8 @@ int conv1d_silu_launch(const void* x, long ldx, const float* w, const float* bia
 #define LB_KCP(K_)                                                                                             \
   if (KC == K_) {                                                                                              \
     conv1d_silu_prompt_kernel<K_><<<grid, 128, 0, s>>>(xb, ldx, w, bias, conv_state, cu_seq, slots, C, tok, ob, \
-                                                       ldo, write_state);                                      \
-    if (write_state) conv1d_state_kernel<K_><<<grid2, 128, 0, s>>>(xb, ldx, conv_state, cu_seq, slots, C);      \
+                                                       ldo, write_state, in_bias, silu);                       \
+    if (write_state) conv1d_state_kernel<K_><<<grid2, 128, 0, s>>>(xb, ldx, conv_state, cu_seq, slots, C, in_bias); \
     return cudaGetLastError() != cudaSuccess;                                                                  \
   }
     LB_KCP(2) LB_KCP(3) LB_KCP(4) LB_KCP(5) LB_KCP(6) LB_KCP(7) LB_KCP(8)
@@ -136,7 +139,7 @@ int conv1d_silu_launch(const void* x, long ldx, const float* w, const float* bia
 #define LB_KC(K_)                                                                                              \
   if (KC == K_) {                                                                                              \
     conv1d_silu_kernel<K_><<<grid, 128, 0, s>>>(xb, ldx, w, bias, conv_state, cu_seq, slots, C, ob, ldo,       \
-                                                write_state);                                                  \
+                                                write_state, in_bias, silu);                                   \
     return cudaGetLastError() != cudaSuccess;                                                                  \
   }
   LB_KC(2) LB_KC(3) LB_KC(4) LB_KC(5) LB_KC(6) LB_KC(7) LB_KC(8)

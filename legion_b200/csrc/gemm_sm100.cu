@@ -23,6 +23,7 @@
 #include <cuda_fp16.h>
 
 #include "comm_dev.cuh"
+#include "act_type.cuh"
 #include "common.cuh"
 #include "gemm_sm100.h"
 #include "nvfp4_dev.cuh"
@@ -547,6 +548,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
       }
 
       if (finalize) {
+        const float xi_a = (!DUAL && a.xielu) ? a.xielu[0] : 0.f, xi_b = (!DUAL && a.xielu) ? a.xielu[1] : 0.f;
         const float* wsb = a.split_k > 1 ? a.ws + size_t(it.tile_id) * a.split_k * (Cfg::ACC_COLS * BM) : nullptr;
 #pragma unroll 1
         for (int c = 0; c < BN; c += 32) {
@@ -590,6 +592,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
               if (DUAL) v = gate_act(v, a.act) * u[j];
+              else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -680,6 +683,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
                 const int xrow = it.out0 + t;
                 float v = g[j];
                 if (DUAL) v = gate_act(v, a.act) * u[j];
+                else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
                 if (a.tok_scale) v *= a.tok_scale[xrow];
                 long orow = xrow;
                 if (a.out_rows) orow = a.out_rows[xrow];
@@ -876,11 +880,12 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
   }
   a.tile_group = h.tile_group; a.tile_tok0 = h.tile_tok0; a.tile_out0 = h.tile_out0; a.tile_ntok = h.tile_ntok; a.n_tiles_dev = h.n_tiles_dev;
   a.n_tok_tiles_max = h.n_tok_tiles_max;
-  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act;
+  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act; a.xielu = h.xielu;
   a.x_group_col = h.x_group_col;
-  if (h.x_group_col != 0 && (h.x_group_col % 8 != 0 || h.K % BK != 0 || fp8 || fp4 || !h.tile_group)) {
+  // (a last K tile that reaches into the next group's columns meets weights that TMA filled with zeros)
+  if (h.x_group_col != 0 && (h.x_group_col % 8 != 0 || h.K % 8 != 0 || fp8 || fp4 || !h.tile_group)) {
     snprintf(g_gemm_err, sizeof(g_gemm_err),
-             "wgemm: per-group activation columns need grouped bf16 mode, K %% 64 == 0 and 16-byte aligned offsets");
+             "wgemm: per-group activation columns need grouped bf16 mode, K %% 8 == 0 and 16-byte aligned offsets");
     return 1;
   }
   a.split_k = h.split_k < 1 ? 1 : h.split_k;

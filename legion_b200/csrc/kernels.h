@@ -43,10 +43,11 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
 const char* prefill_attn_last_error();
 
 // Latent attention (absorbed form) over the paged latent cache: attn_mla_sm100.cu
-int mla_attn_launch(const void* q_abs, long T, const void* cache, long n_cells, long cell_stride, const int* cu_q,
-                    const int* ctx_lens, const int* block_table, int table_width, int page, int n_seqs,
-                    int max_q_len, int nh, float scale, int n_splits, float* o_part, float* ml_part, void* out,
-                    int* status, cudaStream_t s);
+// (merge false: the caller merges the partials of n_splits > 1 itself)
+int mla_attn_launch(const void* q_abs, long q_pitch, long T, const void* cache, long n_cells, long cell_stride,
+                    const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page, int n_seqs,
+                    int max_q_len, int nh, int L, int R, float scale, int n_splits, float* o_part, float* ml_part,
+                    void* out, bool merge, int* status, cudaStream_t s);
 const char* mla_attn_last_error();
 int mla_prep_launch(const void* kva, long ld_kva, const float* norm_w, float eps, float w_offset, const void* q,
                     long ld_q_tok, int q_head_stride, int q_pe_off, int nh, const float* cos_sin,

@@ -25,6 +25,73 @@ struct HyperArgs {
 };
 int hyper_launch(const HyperArgs& a, bool f32, cudaStream_t s);
 
+// One fp32 residual between grouped norms, with the next sublayer's input convolution (resid_step.cu).
+struct ResidStepArgs {
+  const float* x_in;               // [rows, H]; nullptr: start from the embedding
+  float* x_out;                    // [rows, H], not x_in
+  const void* emb; const int* ids; // start: embedding table and token ids (ids == nullptr: row t of emb), times emb_scale
+  long ld_emb; int vocab; float emb_scale;
+  const void* y; long ldy;         // sublayer output, activation type
+  const float* post_w;             // its norm
+  const float* norm_w;             // the next norm
+  float eps; int groups;
+  const float* taps; int taps_n;   // [taps_n, H], oldest token first; nullptr: h = n
+  float* hist;                     // [slots, taps_n - 1, H]
+  const int* cu; const int* slots; // without a convolution cu may be nullptr: every row is a sequence
+  int n_seqs, max_len, tok;        // tok: tokens per CTA, at least taps_n - 1 where sequences are longer than it
+  int write_state;
+  void* h; long ldh;
+  int rows, H;
+  int lanes;                       // set by the launcher
+};
+int resid_step_launch(const ResidStepArgs& a, bool f32, cudaStream_t s);
+
+// Latent attention of any sizes (latent_attn.cu). kv rows: latent [L] | shared key part [R]; q rows: heads of [dim | R].
+struct LatentPrepArgs {
+  const void* q; long ldq;
+  const void* kv; long ldkv;
+  const float* norm_w; float eps;
+  const float* cos_sin; int rot;   // [positions, rot]: cos | sin of rot / 2 pairs of neighbouring columns
+  const int* positions; const long* slots;
+  void* cache; long cell;          // elements between cache cells
+  void* q_abs; long q_row;         // [T, heads] rows of q_row elements; columns [L, L + R) are written here
+  int T, heads, dim, R, L;
+};
+int latent_prep_launch(const LatentPrepArgs& a, bool f32, cudaStream_t s);
+// x[t, n] *= sigmoid(gate[t, per_head ? n / vdim : n]) in place
+int latent_gate_launch(void* x, const void* gate, long ldg, int per_head, int vdim, int N, int T, bool f32, cudaStream_t s);
+
+// Diagonal gated recurrence (diag_scan.cu): a = exp(sigmoid(r) log_decay), S = a S + sqrt(1 - a^2) sigmoid(i) u,
+// out = S gelu(y + y_b). gates: [T, blocks, 2, W / blocks] fp32 before bias and sigmoid.
+struct DiagScanArgs {
+  const void* u; long ldu;
+  float* gates;                    // overwritten by the chunked form
+  const float* gates_b; const float* log_decay;
+  const void* y; long ldy; const float* y_b;
+  float* state;                    // [slots, W]
+  const int* cu; const int* slots;
+  int n_seqs, T, W, blocks;
+  void* out; long ldo;
+  int write_state;
+  int max_tokens;                  // sequential form: sequences with more tokens are left alone (0: all run)
+};
+int diag_scan_launch(const DiagScanArgs& a, bool f32, cudaStream_t s);
+// chunk tables as of linear_chunk_launch; ends: scratch of n_chunks * 2 * W floats
+int diag_chunk_launch(const DiagScanArgs& a, const int* chunk_t0, const int* chunk_n, int n_chunks, const int* seq_chunk0,
+                      const int* seq_nchunk, float* ends, bool f32, cudaStream_t s);
+// One decode step with the convolution and the gate products in front of it
+struct DiagDecodeArgs {
+  const void* x; long ldx;         // [n, W] input of the convolution before in_bias
+  const float* in_bias;
+  const float* conv_w; const float* conv_b; float* conv_state; int KC;   // [W, KC], [slots, W, KC - 1]
+  const void* gates_w;             // [blocks, 2, d, d], activation type
+  DiagScanArgs s;                  // u and gates unused
+  unsigned int* ctr;               // [sequence tiles, blocks] zeroed arrival counters, left zero
+  int vec;                         // set by the launcher
+};
+int diag_decode_launch(const DiagDecodeArgs& a, bool f32, cudaStream_t s);
+constexpr int DIAG_DECODE_SEQ = 4;  // sequences per tile
+
 // Plain FMA GEMM (sgemm.cu): out[t, n] = sum_k x[t, k] w[n, k] in fp32, any sizes and pitches. Token tiles of
 // SGEMM_BN rows; the grouped form takes the tile tables of the tcgen05 GEMM.
 constexpr int SGEMM_BN = 32;
@@ -36,7 +103,11 @@ struct SgemmArgs {
   const float* tok_scale;          // per activation row (grouped) multiplier
   const int* out_rows;             // activation row -> output row (negative: drop)
   int T, K, N;
-  int dual; long dual_offset; int act;   // act(gate) * up, rows dual_offset apart; act 0 silu, 1 gelu (tanh), 2 relu^2 (no up)
+  int dual; long dual_offset; int act;   // act(gate) * up, rows dual_offset apart; act 0 silu, 1 gelu (tanh), 2 relu^2
+                                         // (no up), 3 xIELU (no up) with act_ab
+  const float* act_ab;             // [2]
+  int heads; long x_head_col, out_head_col;  // heads > 1: head z reads x columns from z * x_head_col and weight rows from
+                                             // z * rows_per_group, and writes output columns from z * out_head_col
   const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles; int max_tiles;
   long rows_per_group;
 };
@@ -46,8 +117,9 @@ int sgemm_launch(const SgemmArgs& a, bool f32, cudaStream_t s);
 int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld, const float* qw, const float* kw,
                            float eps, const long* slots, void* q_out, void* k_cache, void* v_cache, long k_cell,
                            long v_cell, int T, int Hq, int Hkv, int DK, int DV, bool f32, cudaStream_t s);
-// Paged causal attention on FMA units, one warp per (token, query head); value heads up to 512 wide
-int paged_attn_general_launch(const void* q, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
+// Paged causal attention on FMA units, one warp per (token, query head); value heads up to 1024 wide; q_row: elements
+// between query heads
+int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
                               int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, int window, void* out,
                               bool f32, cudaStream_t s);
@@ -93,9 +165,9 @@ int ssd_decode_launch(const SsdDecodeArgs& a, bool f32, cudaStream_t s);
 int group_norm_gate_launch(const void* y, long ldy, const void* gate, long ldg, const float* w, float eps, int groups,
                            int C, int rows, void* out, long ldo, bool f32, cudaStream_t s);
 
-// Causal depth-wise convolution + silu with carried history, any number of taps
+// Causal depth-wise convolution (+ silu) with carried history, any number of taps; in_bias is added to x first
 int conv_silu_any_launch(const void* x, long ldx, const float* w, const float* bias, float* conv_state,
                          const int* cu_seq, const int* slots, int n_seqs, int T, int C, int KC, void* out, long ldo,
-                         int write_state, bool f32, cudaStream_t s);
+                         int write_state, const float* in_bias, int silu, bool f32, cudaStream_t s);
 
 }  // namespace lb

@@ -1,0 +1,321 @@
+// One fp32 residual whose sublayers run between two RMS norms, with a short causal convolution in front of each:
+//   x' = x + norm(y) * post_w            (y: the sublayer's output; the first launch of a step starts from the embedding)
+//   n  = norm(x') * norm_w               (the next sublayer's norm; both norms work in `groups` equal parts of the row)
+//   h_t = n_t + sum_j taps[j] n_(t - K + 1 + j)                     (per channel; n before the sequence's start is zero)
+// in one launch per sublayer, so that the residual and the sublayer output are read once. The last K - 1 rows of n are a
+// sequence's history; the launch reads and replaces it.
+//
+// A CTA walks up to `tok` consecutive tokens of one sequence with the previous rows of n in registers. A tile in the
+// middle of a sequence recomputes n of the K - 1 tokens in front of it from x and y (the new residual goes to a second
+// buffer, so these are still there). Only the first tile of a sequence touches the history: it reads it, and replaces it
+// with the rows of the sequence's last tokens, recomputed when they lie in another tile. So no launch waits and no two
+// CTAs meet in the state.
+#include <algorithm>
+
+#include "act_type.cuh"
+#include "common.cuh"
+#include "layers.h"
+
+namespace lb {
+namespace {
+
+struct Tile { int seq, t0, t1, ta; };
+
+// The sequence and first token of tile `idx` when every sequence is cut into tiles of `tok` tokens (warp-wide; seq < 0:
+// no such tile).
+__device__ __forceinline__ Tile find_tile(const int* __restrict__ cu, int n_seqs, int tok, int idx) {
+  const int lane = threadIdx.x & 31;
+  int before = 0;
+  for (int b = 0; b < n_seqs; b += 32) {
+    const int s = b + lane;
+    const int c0 = s < n_seqs ? cu[s] : 0, c1 = s < n_seqs ? cu[s + 1] : 0;
+    const int n = (c1 - c0 + tok - 1) / tok;
+    int inc = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += v;
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, before + inc > idx);
+    if (hit) {
+      const int l = __ffs(hit) - 1;
+      const int first = before + __shfl_sync(0xffffffffu, inc - n, l);
+      Tile t;
+      t.seq = b + l;
+      t.t0 = __shfl_sync(0xffffffffu, c0, l);
+      t.t1 = __shfl_sync(0xffffffffu, c1, l);
+      t.ta = t.t0 + (idx - first) * tok;
+      return t;
+    }
+    before += __shfl_sync(0xffffffffu, inc, 31);
+  }
+  return Tile{-1, 0, 0, 0};
+}
+
+template <typename T, int VEC, int NC, int KMAX>
+__global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) {
+  extern __shared__ float part_s[];                       // two buffers of partial sums of squares
+  griddep_wait();
+  griddep_launch();
+  const int tid = threadIdx.x, nt = blockDim.x, H = a.H;
+  Tile tl;
+  if (a.tok >= a.max_len) {
+    tl.seq = blockIdx.x;
+    tl.t0 = tl.ta = a.cu ? a.cu[tl.seq] : int(blockIdx.x);
+    tl.t1 = a.cu ? a.cu[tl.seq + 1] : tl.t0 + 1;
+  } else {
+    tl = find_tile(a.cu, a.n_seqs, a.tok, blockIdx.x);
+  }
+  if (tl.seq < 0 || tl.ta >= tl.t1) return;
+  const int tb = min(tl.t1, tl.ta + a.tok);
+  const int gs = H / a.groups, W = a.lanes, ppg = gs / (VEC * W), n_part = H / (VEC * W);
+  const float gs_inv = 1.f / float(gs);
+  const bool start = a.x_in == nullptr;
+
+  float xv[NC][VEC], yv[NC][VEC];
+  auto load = [&](int t) {
+    const T* er = nullptr;
+    if (start) {
+      long row = t;
+      if (a.ids) {
+        const int id = a.ids[t];
+        row = (id < 0 || id >= a.vocab) ? 0 : id;
+      }
+      er = static_cast<const T*>(a.emb) + row * a.ld_emb;
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = (c * nt + tid) * VEC;
+      if (d < H) {
+        if (start) {
+          ld_vec<VEC>(er + d, xv[c]);
+        } else {
+          ld_vec<VEC>(a.x_in + long(t) * H + d, xv[c]);
+          ld_vec<VEC>(static_cast<const T*>(a.y) + long(t) * a.ldy + d, yv[c]);
+        }
+      }
+    }
+  };
+  // 1 / rms of the group that holds each of this thread's vectors
+  auto group_inv = [&](const float (&v)[NC][VEC], float* part, float (&inv)[NC]) {
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = (c * nt + tid) * VEC;
+      float ss = 0.f;
+      if (d < H) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss = fmaf(v[c][j], v[c][j], ss);
+      }
+      for (int o = W >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (d < H && (tid & (W - 1)) == 0) part[d / (VEC * W)] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = (c * nt + tid) * VEC;
+      inv[c] = 0.f;
+      if (d < H) {
+        const float* p = part + (d / gs) * ppg;
+        float s = 0.f;
+        for (int i = 0; i < ppg; ++i) s += p[i];
+        inv[c] = 1.f / sqrtf(s * gs_inv + a.eps);
+      }
+    }
+  };
+  // n of the token whose x and y are loaded; the new residual is written when the token is this tile's own
+  float n[NC][VEC];
+  auto advance = [&](int t, bool own) {
+    float inv[NC];
+    if (start) {
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) n[c][j] = xv[c][j] * a.emb_scale;
+    } else {
+      group_inv(yv, part_s, inv);
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const int d = (c * nt + tid) * VEC;
+        if (d < H) {
+          float pw[VEC];
+          ld_vec<VEC>(a.post_w + d, pw);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) n[c][j] = xv[c][j] + yv[c][j] * inv[c] * pw[j];
+        }
+      }
+    }
+    if (own) {
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const int d = (c * nt + tid) * VEC;
+        if (d < H) st_vec<VEC>(a.x_out + long(t) * H + d, n[c]);
+      }
+    }
+    group_inv(n, part_s + n_part, inv);
+    if (start) __syncthreads();                            // the one buffer in use is written again by the next token
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = (c * nt + tid) * VEC;
+      if (d < H) {
+        float nw[VEC];
+        ld_vec<VEC>(a.norm_w + d, nw);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) n[c][j] *= inv[c] * nw[j];
+      }
+    }
+  };
+
+  // hist[KMAX - 2] is the row before the current token; rows older than K - 1 are not used
+  constexpr int R = KMAX > 1 ? KMAX - 1 : 1;
+  float hist[R][NC][VEC];
+  const int K1 = KMAX > 1 ? a.taps_n - 1 : 0;
+  auto push = [&]() {
+    if constexpr (KMAX > 1) {
+#pragma unroll
+      for (int i = 0; i + 1 < R; ++i)
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) hist[i][c][j] = hist[i + 1][c][j];
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) hist[R - 1][c][j] = n[c][j];
+    }
+  };
+  float* st = (KMAX > 1 && a.hist) ? a.hist + long(a.slots[tl.seq]) * K1 * H : nullptr;
+  const bool first = tl.ta == tl.t0;
+  if constexpr (KMAX > 1) {
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) hist[i][c][j] = 0.f;
+    if (first) {
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int r = i - (R - K1);
+        if (r >= 0) {
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            const int d = (c * nt + tid) * VEC;
+            if (d < H) ld_vec<VEC>(st + long(r) * H + d, hist[i][c]);
+          }
+        }
+      }
+    } else {
+      for (int t = tl.ta - K1; t < tl.ta; ++t) {
+        load(t);
+        advance(t, false);
+        push();
+      }
+    }
+  }
+  load(tl.ta);
+  for (int t = tl.ta; t < tb; ++t) {
+    advance(t, true);
+    if (t + 1 < tb) load(t + 1);
+    T* hr = static_cast<T*>(a.h) + long(t) * a.ldh;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = (c * nt + tid) * VEC;
+      if (d < H) {
+        float o[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) o[j] = n[c][j];
+        if (a.taps) {
+          float w[VEC];
+          ld_vec<VEC>(a.taps + long(K1) * H + d, w);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], n[c][j], o[j]);
+          if constexpr (KMAX > 1) {
+#pragma unroll
+            for (int i = 0; i < R; ++i) {
+              const int r = i - (R - K1);
+              if (r >= 0) {
+                ld_vec<VEC>(a.taps + long(r) * H + d, w);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], hist[i][c][j], o[j]);
+              }
+            }
+          }
+        }
+        st_vec<VEC>(hr + d, o);
+      }
+    }
+    push();
+  }
+  if constexpr (KMAX > 1) {
+    if (first && a.write_state && K1 > 0) {
+      if (tb < tl.t1) {                                    // the sequence's last tokens lie in another tile
+        for (int t = tl.t1 - K1; t < tl.t1; ++t) {
+          load(t);
+          advance(t, false);
+          push();
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int r = i - (R - K1);
+        if (r >= 0) {
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            const int d = (c * nt + tid) * VEC;
+            if (d < H) st_vec<VEC>(st + long(r) * H + d, hist[i][c]);
+          }
+        }
+      }
+    }
+  }
+}
+
+template <typename T, int VEC, int NC>
+int launch_k(const ResidStepArgs& a, int nt, dim3 grid, cudaStream_t s) {
+  const size_t smem = size_t(2) * (a.H / (VEC * a.lanes)) * 4;
+  if (smem > 48 * 1024) return 1;
+  const int K = a.taps ? a.taps_n : 1;
+#define LB_K(N)                                                                                                        \
+  if (K <= N) return launch_pdl(resid_step_kernel<T, VEC, NC, N>, grid, dim3(nt), smem, s, a) != cudaSuccess;
+  LB_K(1) LB_K(4) LB_K(16)
+#undef LB_K
+  return 1;
+}
+
+template <typename T>
+int dispatch(ResidStepArgs a, cudaStream_t s) {
+  const size_t es = sizeof(T);
+  auto al = [&](const void* p, size_t n) { return p == nullptr || reinterpret_cast<uintptr_t>(p) % n == 0; };
+  const int gs = a.H / a.groups;
+  const bool v4 = gs % 4 == 0 && al(a.x_in, 16) && al(a.x_out, 16) && al(a.emb, 4 * es) && al(a.y, 4 * es) &&
+                  al(a.h, 4 * es) && al(a.post_w, 16) && al(a.norm_w, 16) && al(a.taps, 16) && al(a.hist, 16) &&
+                  a.ld_emb % 4 == 0 && a.ldy % 4 == 0 && a.ldh % 4 == 0;
+  const int vec = v4 ? 4 : 1;
+  a.lanes = 1;
+  while (a.lanes < 32 && gs % (vec * a.lanes * 2) == 0) a.lanes *= 2;
+  const int need = (a.H + vec - 1) / vec;                 // threads for one vector each
+  const int nt = std::min(512, (need + 31) / 32 * 32), nc = (need + nt - 1) / nt;
+  const int tiles = a.tok >= a.max_len ? (a.cu ? a.n_seqs : a.rows) : a.rows / a.tok + a.n_seqs;
+  const dim3 grid(tiles);
+  if (vec == 4) {
+    if (nc <= 1) return launch_k<T, 4, 1>(a, nt, grid, s);
+    if (nc <= 2) return launch_k<T, 4, 2>(a, nt, grid, s);
+    if (nc <= 4) return launch_k<T, 4, 4>(a, nt, grid, s);
+    if (nc <= 8) return launch_k<T, 4, 8>(a, nt, grid, s);
+  } else {
+    if (nc <= 1) return launch_k<T, 1, 1>(a, nt, grid, s);
+    if (nc <= 8) return launch_k<T, 1, 8>(a, nt, grid, s);
+  }
+  return 1;
+}
+
+}  // namespace
+
+int resid_step_launch(const ResidStepArgs& a, bool f32, cudaStream_t s) {
+  if (a.rows <= 0) return 0;
+  if (a.groups < 1 || a.H < 1 || a.H % a.groups || a.tok < 1) return 1;
+  if (a.taps && (a.taps_n < 1 || a.tok < (a.tok >= a.max_len ? 1 : a.taps_n - 1))) return 1;
+  return f32 ? dispatch<float>(a, s) : dispatch<__nv_bfloat16>(a, s);
+}
+
+}  // namespace lb

@@ -2,7 +2,8 @@
 // shapes the TMA-fed tcgen05 GEMM does not take (row pitches that are not multiples of 16 bytes). 64 features x 32
 // tokens per CTA, 16-wide k steps through shared memory, 2 x 4 outputs per thread; the next k step's operands are
 // fetched into registers while the current one is multiplied. The grouped form walks the same tile tables as
-// gemm_sm100.cu (tile -> expert, first row, rows), so routed experts run on the same routing plan.
+// gemm_sm100.cu (tile -> expert, first row, rows), so routed experts run on the same routing plan. A third grid dimension
+// serves per-head products (each head's own slice of x, weights and output).
 #include "act_type.cuh"
 #include "common.cuh"
 #include "layers.h"
@@ -31,8 +32,9 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const SgemmArgs a) {
     ntok = min(TN, a.tile_ntok[blockIdx.y]);
   }
   const int n0 = blockIdx.x * TM;
-  const T* w = static_cast<const T*>(a.w) + long(group) * a.rows_per_group * a.ldw;
-  const T* x = static_cast<const T*>(a.x);
+  const T* w = static_cast<const T*>(a.w) + long(group + blockIdx.z) * a.rows_per_group * a.ldw;
+  const T* x = static_cast<const T*>(a.x) + blockIdx.z * a.x_head_col;
+  const long out_col = blockIdx.z * a.out_head_col;
   const int tid = threadIdx.x;
   const int lk = tid % TK, lr = tid / TK;          // loader: k within the step, row 0..15
   float wr[DUAL ? 2 : 1][4], xr[2];
@@ -97,10 +99,11 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const SgemmArgs a) {
       float v = acc[0][i][j];
       if constexpr (DUAL) v = act_of<T>(v, a.act) * acc[1][i][j];
       else if (a.act == 2) { v = fmaxf(v, 0.f); v *= v; }
+      else if (a.act == 3) v = xielu_f(v, a.act_ab[0], a.act_ab[1]);
       v *= sc;
       if (a.residual) v += ld_f(static_cast<const T*>(a.residual) + orow * a.ldr + n);
-      if (a.out_f32) static_cast<float*>(a.out)[orow * a.ldo + n] = v;
-      else st_f(static_cast<T*>(a.out) + orow * a.ldo + n, v);
+      if (a.out_f32) static_cast<float*>(a.out)[orow * a.ldo + out_col + n] = v;
+      else st_f(static_cast<T*>(a.out) + orow * a.ldo + out_col + n, v);
     }
   }
 }
@@ -108,7 +111,7 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const SgemmArgs a) {
 template <typename T>
 int launch_t(const SgemmArgs& a, cudaStream_t s) {
   const int tiles = a.tile_group ? a.max_tiles : (a.T + TN - 1) / TN;
-  const dim3 grid((a.N + TM - 1) / TM, tiles);
+  const dim3 grid((a.N + TM - 1) / TM, tiles, a.heads > 1 ? a.heads : 1);
   if (tiles <= 0) return 0;
   if (tiles > 65535) return 1;
   return (a.dual ? launch_pdl(sgemm_kernel<T, true>, grid, dim3(256), 0, s, a)

@@ -1012,7 +1012,7 @@ class Decoder:
         q_abs = ops.latent_queries(proj[:, :nq], proj[:, nq:nq + nl], w[f"{p}.lat.uk"], w[f"{p}.lat.norm"], cfg.rms_eps,
                                    self.rotary_table(m.rot), b.positions, b.slots, kv.k[il], m.heads, m.dim, m.rot_dim)
         o = ops.latent_attention(q_abs, kv.k[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, m.scale, m.kv_rank,
-                                 max_ctx=b.max_ctx or None)
+                                 m.rot_dim, max_ctx=b.max_ctx or None)
         return ops.linear(ops.latent_values(o, w[f"{p}.lat.uv"], gate), w[f"{p}.lat.o"])
 
     def _rglru_mixer(self, p: str, il: int, h, b: StepBatch, st: StatePool):
@@ -1023,6 +1023,11 @@ class Decoder:
         proj = ops.linear(h, w[f"{p}.lru.in"])
         in_b = w[f"{p}.lru.in_b"]
         y, x = proj[:, :W], proj[:, W:]
+        if proj.is_cuda and b.max_q_len == 1 and b.write_state and proj.shape[0] == b.n_seqs:
+            s = ops.sm100.rglru_decode(x, in_b[W:], w[f"{p}.lru.conv_w"], w[f"{p}.lru.conv_b"], st.conv[il],
+                                       w[f"{p}.lru.gates"], w[f"{p}.lru.gates_b"], w[f"{p}.lru.log_decay"], y, in_b[:W],
+                                       st.ssm[il], b.cu_q, b.state_slots, m.blocks)
+            return ops.linear(s, w[f"{p}.lru.out"])
         u = ops.causal_conv1d_silu(x, w[f"{p}.lru.conv_w"], w[f"{p}.lru.conv_b"], st.conv[il], b.cu_q, b.state_slots,
                                    write_state=b.write_state, max_len=b.max_q_len, in_bias=in_b[W:], silu=False)
         gates = ops.block_gates(u, w[f"{p}.lru.gates"], m.blocks)

@@ -227,9 +227,9 @@ def latent_queries(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, hea
     return f(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, heads, dim, rot_dim)
 
 
-def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, max_ctx=None):
+def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, rot_dim, max_ctx=None):
     if _cuda(q_abs):
-        return _sm.latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, max_ctx)
+        return _sm.latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank, rot_dim, max_ctx)
     return _ref.latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, scale, rank)
 
 

@@ -596,22 +596,30 @@ def tma_ok(*ts) -> bool:
                for t in ts)
 
 
-def sgemm(x, w, residual=None, out=None, out_dtype=None, dual: bool = False, n_ff: int = 0, act: str = "silu"):
+def sgemm(x, w, residual=None, out=None, out_dtype=None, dual: bool = False, n_ff: int = 0, act: str = "silu",
+          act_ab=None):
     """x @ w^T in fp32 arithmetic on the FMA units: fp32 models and shapes outside the tcgen05 GEMM's alignment rules.
     ``dual``: act(x Wg^T) * (x Wu^T) with Wg = w[:n_ff], Wu = w[n_ff:]."""
     T, N = x.shape[0], (n_ff if dual else w.shape[0])
     if out is None:
         out = torch.empty(T, N, dtype=out_dtype or x.dtype, device=x.device)
-    ext().sgemm(w, x, out, residual, None, None, N, dual, n_ff if dual else 0, GATE_ACTS[act] if dual else 0, None, None,
-                None, None, 0, 0, T)
+    ext().sgemm(w, x, out, residual, None, None, N, dual, n_ff if dual else 0,
+                3 if act_ab is not None else GATE_ACTS[act] if dual else 0, None, None, None, None, 0, 0, T, act_ab)
     return out
 
 
-def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Optional[int] = None, bn=None):
+def up_act(x, w, ab):
+    """xIELU(x @ w^T) with the activation in the epilogue; ``ab``: its two numbers, float32."""
+    return linear(x, w, out_dtype=x.dtype, xielu=ab)
+
+
+def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Optional[int] = None, bn=None, xielu=None):
     """out[T, N] = x[T, K] @ w[N, K]^T (+ residual)."""
     C = ext()
     if isinstance(w, torch.Tensor) and isinstance(x, torch.Tensor) and not tma_ok(x, w):
-        return sgemm(x, w, residual, out, out_dtype)
+        return sgemm(x, w, residual, out, out_dtype, act_ab=xielu)
+    if xielu is not None and not isinstance(w, torch.Tensor):
+        raise ValueError("xIELU runs in the epilogue of bf16 and fp32 weights")
     if isinstance(x, Fp8Act) and not isinstance(w, Fp8Weight):
         x = x.x
     T, K = x.shape
@@ -642,7 +650,7 @@ def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Opt
             sk = 1
     C.wgemm(w.codes if q else w, x, out, residual, None, None, N, False, 0, bn, sk, ws.splitk if sk > 1 else None,
             ws.counters if sk > 1 else None, ws.status, None, None, None, None, 0, 0, T, [], None,
-            w.scales if q else None, w.gscale if q else None)
+            w.scales if q else None, w.gscale if q else None, xielu=xielu)
     return out
 
 
@@ -795,6 +803,10 @@ def head_linear(x, w2d, n_heads: int, rows_per_group: int, n_feat: int, K: int, 
     go through a row map, so nothing is transposed or copied."""
     C = ext()
     T = x.shape[0]
+    if not (tma_ok(x, w2d) and x_group_col % 8 == 0):
+        # fp32 and unaligned shapes: the FMA kernel
+        C.sgemm_heads(w2d, x, out2d.view(T, -1), n_heads, rows_per_group, n_feat, K, x_group_col, out2d.shape[1])
+        return out2d
     ws = Workspace.get(x.device)
     bn = pick_bn(T, False)
     key = ("head_linear", T, n_heads, bn)
@@ -840,8 +852,10 @@ def mla_prep(kva, norm_w, eps, w_offset, q, q_pe_off, cos_sin, positions, slots,
     ext().mla_prep(kva, norm_w, eps, w_offset, q, q_pe_off, cos_sin, positions, slots, cache, q_abs)
 
 
-def mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, n_splits=None, max_ctx=None, out=None):
-    """Latent attention, absorbed form: q_abs [T, heads, 576], cache rows [.., 576] -> [T, heads, 512]."""
+def mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, n_splits=None, max_ctx=None, out=None,
+             rank: int = 512, rot: int = 64):
+    """Latent attention, absorbed form: q_abs [T, heads, rank + rot], cache rows [.., rank + rot] (either with padding
+    columns behind) -> [T, heads, rank]."""
     C = ext()
     T, nh, _ = q_abs.shape
     if n_splits is None:
@@ -849,12 +863,50 @@ def mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, 
     ws = Workspace.get(q_abs.device)
     o_part = ml_part = None
     if n_splits > 1:
-        o_part = ws.buf("mla_o", (T * nh * n_splits * 512,), torch.float32)
+        o_part = ws.buf("mla_o", (T * nh * n_splits * rank,), torch.float32)
         ml_part = ws.buf("mla_ml", (T * nh * n_splits * 2,), torch.float32)
     if out is None:
-        out = torch.empty(T, nh, 512, dtype=torch.bfloat16, device=q_abs.device)
-    C.mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, n_splits, o_part, ml_part, out,
-               ws.status)
+        out = torch.empty(T, nh, rank, dtype=torch.bfloat16, device=q_abs.device)
+    C.mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, max_q_len, scale, n_splits, o_part, ml_part, out, rank, rot,
+               True, ws.status)
+    return out
+
+
+def latent_tc_ok(q_abs, cache, rank: int, rot: int) -> bool:
+    """Whether the tcgen05 latent-attention kernel takes these rows."""
+    page = cache.shape[1]
+    return (q_abs.dtype == torch.bfloat16 and rank % 8 == 0 and (rank + rot) % 8 == 0 and rank <= 512 and rank + rot <= 576
+            and q_abs.shape[2] % 8 == 0 and cache.shape[-1] % 8 == 0 and page % 8 == 0 and 64 % page == 0)
+
+
+def latent_queries(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, heads: int, dim: int, rot_dim: int):
+    """Cache rows of the step's tokens and the queries in the latent space, [T, heads, rank + rot_dim] (rows padded to
+    multiples of 8 columns)."""
+    T, L = q.shape[0], norm_w.numel()
+    q_abs = torch.empty(T, heads, -(-(L + rot_dim) // 8) * 8, dtype=q.dtype, device=q.device)
+    head_linear(q, uk, heads, L, L, dim, dim + rot_dim, q_abs.view(T * heads, -1))
+    ext().latent_prep(q, kv, norm_w, eps, cos_sin, positions, slots, cache, q_abs, dim, rot_dim)
+    return q_abs
+
+
+def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank: int, rot: int, max_ctx=None):
+    """Causal attention over cached latent rows, [T, heads, rank]: tcgen05 in bf16, FMA units for fp32 and other sizes."""
+    if latent_tc_ok(q_abs, cache, rank, rot):
+        return mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, cache.shape[1], max_q_len, scale, max_ctx=max_ctx, rank=rank,
+                        rot=rot)
+    out = torch.empty(q_abs.shape[0], q_abs.shape[1], rank, dtype=q_abs.dtype, device=q_abs.device)
+    ext().latent_attn_general(q_abs, cache, cu_q, ctx_lens, block_table, scale, rank, rot, out)
+    return out
+
+
+def latent_values(o_lat, uv, gate):
+    """Per-head value projection of the attended latents and the output gate: [T, heads * vdim]."""
+    T, H, L = o_lat.shape
+    vdim = uv.shape[0] // H
+    out = torch.empty(T, H * vdim, dtype=o_lat.dtype, device=o_lat.device)
+    head_linear(o_lat.view(T, H * L), uv, H, vdim, vdim, L, L, out.view(T * H, vdim))
+    if gate is not None:
+        ext().latent_gate(out, gate, H)
     return out
 
 
@@ -1390,19 +1442,21 @@ def sample(logits, temperature, top_k, top_p, min_p, seeds, steps, out=None):
     return out
 
 
-def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, out=None, max_len=None):
+def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, out=None, max_len=None, in_bias=None,
+                       silu: bool = True):
     """``max_len``: longest sequence of the step when known on the host; prompt-sized steps (>= 64 rows per
     sequence) run the token-parallel kernel."""
     C = ext()
     if out is None:
         out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     if x.dtype != torch.bfloat16 or not 2 <= w.shape[1] <= 8:
-        C.conv_silu_any(x, w, bias, conv_state, cu_seq, slots, out, bool(write_state))
+        C.conv_silu_any(x, w, bias, conv_state, cu_seq, slots, out, bool(write_state), in_bias, bool(silu))
         return out
     T, n = x.shape[0], max(1, slots.numel())
     if max_len is None:
         max_len = T if T >= 64 * n else 0          # without the host figure: only clearly prompt-sized steps
-    C.conv1d_silu(x, w, bias, conv_state, cu_seq, slots, out, write_state, int(max_len) if max_len >= 64 else 0)
+    C.conv1d_silu(x, w, bias, conv_state, cu_seq, slots, out, write_state, int(max_len) if max_len >= 64 else 0, in_bias,
+                  bool(silu))
     return out
 
 
@@ -1536,11 +1590,12 @@ LINEAR_CHUNK_MIN = 48        # longest portion of a step from which the chunked 
 LINEAR_CHUNK_SHORT = 8       # ... and up to which its shorter portions stay on the streaming kernel
 
 
-def _linear_chunk_tables(ws, cu_host, device):
-    """chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk of a step (128-token chunks; short portions have none);
-    kept for the step's other layers. Returns (tables, chunks, whether there are short portions)."""
+def _linear_chunk_tables(ws, cu_host, device, size: int = 128):
+    """chunk_t0 | chunk_n | chunk_seq | seq_chunk0 | seq_nchunk of a step (chunks of ``size`` tokens; short portions have
+    none); kept for the step's other layers. Returns (tables, chunks, whether there are short portions)."""
     key = tuple(cu_host)
-    last = ws._cache.get("linear_chunk_tables")
+    name = ("linear_chunk_tables", size)
+    last = ws._cache.get(name)
     if last is not None and last[0] == key:
         return last[1:]
     t0, n, sq, first, cnt = [], [], [], [], []
@@ -1549,14 +1604,14 @@ def _linear_chunk_tables(ws, cu_host, device):
         if cu_host[i + 1] - cu_host[i] <= LINEAR_CHUNK_SHORT:
             cnt.append(0)
             continue
-        for b in range(cu_host[i], cu_host[i + 1], 128):
+        for b in range(cu_host[i], cu_host[i + 1], size):
             t0.append(b)
-            n.append(min(128, cu_host[i + 1] - b))
+            n.append(min(size, cu_host[i + 1] - b))
             sq.append(i)
         cnt.append(len(t0) - first[-1])
     tab = torch.tensor(t0 + n + sq + first + cnt, dtype=torch.int32, device=device)
     short = any(c == 0 for c in cnt)
-    ws._cache["linear_chunk_tables"] = (key, tab, len(t0), short)
+    ws._cache[name] = (key, tab, len(t0), short)
     return tab, len(t0), short
 
 
@@ -1608,6 +1663,85 @@ def group_norm_gate(y, gate, w, eps, groups: int = 1, out=None):
     if out is None:
         out = torch.empty(y.shape, dtype=y.dtype, device=y.device)
     ext().group_norm_gate(y, gate, w, eps, groups, out)
+    return out
+
+
+def resid_tokens(rows: int, max_len: int) -> int:
+    """Tokens per CTA of ``resid_step``: long runs share the recomputed rows in front of a tile, short ones fill the SMs."""
+    if max_len <= 1:
+        return 1
+    return 16 if rows >= 16 * NUM_SMS else 8
+
+
+def resid_step(x, y, post_w, norm_w, groups: int, eps: float, conv=None, start=None, max_len=None):
+    """x + norm(y) into a new buffer, its norm and the input convolution behind it, in one launch. ``start`` = (embedding
+    table, ids or None, scale) begins a step. Returns (x, input of the next sublayer)."""
+    if start is None:
+        table = ids = None
+        scale, xo, h = 1.0, torch.empty_like(x), torch.empty(x.shape, dtype=y.dtype, device=x.device)
+    else:
+        table, ids, scale = start
+        T = table.shape[0] if ids is None else ids.numel()
+        xo = torch.empty(T, table.shape[1], dtype=torch.float32, device=table.device)
+        h = torch.empty(T, table.shape[1], dtype=table.dtype, device=table.device)
+    taps, hist, cu, slots, write = conv if conv is not None else (None, None, None, None, False)
+    rows = xo.shape[0]
+    max_len = rows if max_len is None else max_len
+    tok = 1 if taps is None else max(resid_tokens(rows, max_len), min(taps.shape[0] - 1, max_len))
+    ext().resid_step(x, xo, table, ids, float(scale), y, post_w, norm_w, groups, eps, taps, hist, cu, slots, bool(write),
+                     int(max_len), tok, h)
+    return xo, h
+
+
+def block_gates(u, w, blocks: int):
+    """Block-diagonal product of u [T, W] with w [blocks * n, W / blocks], float32 [T, blocks * n]."""
+    T, d, n = u.shape[0], w.shape[1], w.shape[0] // blocks
+    out = torch.empty(T * blocks, n, dtype=torch.float32, device=u.device)
+    return head_linear(u, w, blocks, n, n, d, d, out).view(T, blocks * n)
+
+
+DIAG_CHUNK = 64              # tokens per chunk of the diagonal recurrence
+
+
+def gated_recurrence(u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks: int, write_state=True, max_len=None,
+                     cu_host=None, out=None, chunked=None):
+    """RG-LRU over the step's tokens (``reference.gated_recurrence``). Prompts run in chunks, short portions token by
+    token; ``chunked`` forces the choice. The chunked form overwrites ``gates``."""
+    C = ext()
+    if out is None:
+        out = torch.empty(u.shape, dtype=u.dtype, device=u.device)
+    args = (u, gates, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks, out, bool(write_state))
+    if chunked is None:
+        chunked = cu_host is not None and (max_len or 0) >= LINEAR_CHUNK_MIN
+    if not chunked:
+        C.diag_scan(*args, 0, None, 0, None)
+        return out
+    ws = Workspace.get(u.device)
+    tab, n_chunks, short = _linear_chunk_tables(ws, cu_host if cu_host is not None else cu_seq.tolist(), u.device, DIAG_CHUNK)
+    if short or n_chunks == 0:
+        C.diag_scan(*args, LINEAR_CHUNK_SHORT, None, 0, None)
+    if n_chunks:
+        need = n_chunks * 2 * u.shape[1]
+        ends = ws._cache.get("diag_chunk_ends")
+        if ends is None or ends.numel() < need:
+            ends = ws._cache["diag_chunk_ends"] = torch.empty(need, dtype=torch.float32, device=u.device)
+        C.diag_scan(*args, 0, tab, n_chunks, ends)
+    return out
+
+
+def rglru_decode(x, in_bias, conv_w, conv_b, conv_state, gates_w, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks: int,
+                 out=None):
+    """Decode step of a gated linear recurrent unit in one launch (one token per sequence): convolution with history
+    update, block-diagonal gates, recurrence and the GELU branch."""
+    n = slots.numel()
+    ws = Workspace.get(x.device)
+    ctr = ws._cache.get("diag_ctr")
+    if ctr is None or ctr.numel() < n * blocks:
+        ctr = ws._cache["diag_ctr"] = torch.zeros(max(n * blocks, 4096), dtype=torch.int32, device=x.device)
+    if out is None:
+        out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    ext().diag_decode(x, in_bias, conv_w, conv_b, conv_state, gates_w, gates_b, log_decay, y, y_b, state, cu_seq, slots, blocks,
+                      ctr, out)
     return out
 
 
