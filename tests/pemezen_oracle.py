@@ -64,13 +64,13 @@ def frequencies(rot):
 def rotate(x, positions, rot):
     """x [T, ..., >= dims]: neighbouring pairs of the first ``dims`` dimensions turn with the position."""
     f, m = frequencies(rot)
+    angle = torch.as_tensor(list(positions), dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
+    c, s = torch.cos(angle) * m, torch.sin(angle) * m
     y = x.clone()
-    for t, p in enumerate(positions):
-        for i, fi in enumerate(f):
-            c, s = math.cos(p * fi) * m, math.sin(p * fi) * m
-            u, v = x[t, ..., 2 * i], x[t, ..., 2 * i + 1]
-            y[t, ..., 2 * i] = u * c - v * s
-            y[t, ..., 2 * i + 1] = v * c + u * s
+    for i in range(len(f)):
+        u, v = x[..., 2 * i].transpose(0, -1), x[..., 2 * i + 1].transpose(0, -1)   # tokens last
+        y[..., 2 * i] = (u * c[:, i] - v * s[:, i]).transpose(0, -1)
+        y[..., 2 * i + 1] = (v * c[:, i] + u * s[:, i]).transpose(0, -1)
     return y
 
 

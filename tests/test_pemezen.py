@@ -1,0 +1,265 @@
+"""The Pemezen design against the plain implementation in ``pemezen_oracle``: whole prompts, decoding, portions, mixed
+batches, used pages and slots, long decoding, and greedy generation through the engine's own scheduler."""
+import json
+import os
+import subprocess
+import sys
+
+import pytest
+import torch
+
+import nisasun_case as nc
+import pemezen_case as pc
+import pemezen_oracle as oracle
+from legion_b200.config import PRESETS, LatentSpec, ModelConfig
+from legion_b200.engine.lm import EngineConfig, LmEngine, build_engine
+from legion_b200.engine.replay import TraceReplay, replay_engine
+from legion_b200.engine.types import GenerateRequest, SamplingParams
+from legion_b200.kv.blocks import OutOfBlocks
+from legion_b200.loaders.model import load_model
+from legion_b200.models.decoder import Decoder
+from legion_b200.models.weights import weight_shapes
+
+gpu = pytest.mark.gpu
+WHERE = [pytest.param("cpu", "float32", id="cpu"), pytest.param("cuda:0", "float32", id="gpu-f32", marks=gpu),
+         pytest.param("cuda:0", "bfloat16", id="gpu-bf16", marks=gpu)]
+
+
+def check(got, want, dtype, what=""):
+    e = nc.errors(got, want)
+    if dtype == "float32":
+        assert e.max() < 1e-4, (what, float(e.max()), int(e.argmax()))
+    else:                                      # bf16 rounding
+        assert e.max() < 0.2 and e.quantile(0.95) < 0.08 and e.median() < 0.03, (what, float(e.median()), float(e.max()),
+                                                                                int(e.argmax()))
+
+
+@pytest.fixture(scope="module")
+def models(tmp_path_factory):
+    out = {}
+    for i, (name, cfg) in enumerate(pc.CASES.items()):
+        w = pc.make_weights(cfg, seed=i)
+        out[name] = (cfg, w, nc.write_checkpoint(tmp_path_factory.mktemp(name), cfg, w))
+    return out
+
+
+_EXPECT = {}
+
+
+def expected(models, name, n, seed):
+    key = (name, n, seed)
+    if key not in _EXPECT:
+        cfg, w, _ = models[name]
+        toks = nc.tokens(cfg, n, seed)
+        _EXPECT[key] = (toks, oracle.forward(cfg, w, toks))
+    return _EXPECT[key]
+
+
+def replay(models, name, device, dtype, max_tokens):
+    return TraceReplay(replay_engine(models[name][2], getattr(torch, dtype), max_tokens, device))
+
+
+def test_registry_and_config_round_trip():
+    for name in ("tiny-pemezen", "pemezen-1b", "pemezen-7b"):
+        c = PRESETS[name]()
+        assert ModelConfig.from_dict(json.loads(c.to_json())) == c
+        assert len(c.layers) == c.n_layer == len(c.layer_kinds)
+    c = PRESETS["tiny-pemezen"]()
+    assert c.kv_layers() == [0, 2] and c.recurrent_layers() == [0, 1, 2, 3]
+    assert c.kv_dims(0) == (1, 96, 0) and isinstance(c.layers[0].mixer, LatentSpec) and c.layers[0].mixer.gate == "head"
+    assert "l2.ffn_norm" not in weight_shapes(c) and "l2.ffn_taps" not in weight_shapes(c)
+    c.layers[0].mlp = None
+    assert c.conv_inputs(0) == ["attn"]
+
+
+@pytest.mark.parametrize("name", list(pc.CASES))
+def test_loader_maps_every_tensor(models, name):
+    cfg, w, path = models[name]
+    mc, lw, _, _ = load_model(path)
+    shapes = weight_shapes(mc)
+    assert set(shapes) == set(lw) and all(tuple(lw[k].shape) == tuple(v) for k, v in shapes.items())
+    pad = 0
+    for i, layer in enumerate(cfg["layers"]):
+        if layer["type"] == "rglru":
+            lam = w[f"l{i}.mix.lam"].double()
+            assert torch.allclose(lw[f"l{i}.lru.log_decay"].double(), -8 * oracle.softplus(lam))
+        else:
+            m = layer["mixer"]
+            rows = sum(w[f"l{i}.mix.{x}"].shape[0] for x in ("q", "dkv", "g"))
+            pad += (lw[f"l{i}.lat.in"].shape[0] - rows) * cfg["width"]
+            assert mc.layers[i].mixer.gate == ("head" if layer["type"].endswith("_2") else "channel")
+            uk = lw[f"l{i}.lat.uk"].view(m["heads"], m["kv_rank"], m["dim"]).transpose(1, 2).reshape(-1, m["kv_rank"])
+            assert torch.equal(uk, w[f"l{i}.mix.uk"].float())
+    assert sum(t.numel() for t in lw.values()) == sum(t.numel() for t in w.values()) + pad
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+@pytest.mark.parametrize("name", list(pc.CASES))
+def test_whole_prompt_layer_by_layer(models, name, device, dtype):
+    cfg, w, path = models[name]
+    toks = nc.tokens(cfg, 70, 1)
+    layers = []
+    want = oracle.forward(cfg, w, toks, layers_out=layers)
+    eng = replay_engine(path, getattr(torch, dtype), 128, device)
+    s = eng.open_sequence("a")
+    s.tokens, s.phase = list(toks), "prefill"
+    s.table.ensure(eng.pool, len(toks))
+    b = eng.build_batch_explicit([(s, 0, toks)], all_logits=True)
+    b.capture_layers = list(range(len(cfg["layers"])))
+    out = eng.model.forward(b, eng.kv, eng.states)
+    for i, x in enumerate(layers):
+        check(out.captures[i].cpu(), x, dtype, f"layer {i}")
+    check(out.logits.cpu(), want, dtype)
+    assert float(out.logits.abs().max()) < cfg["logit_softcap"]
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+@pytest.mark.parametrize("name", list(pc.CASES))
+def test_decoding_and_portions_equal_the_whole_prompt(models, name, device, dtype):
+    toks, want = expected(models, name, 210, 2)
+    n = len(toks)
+    schedules = {
+        "whole": [n],
+        "decoded": [150] + [1] * (n - 150),
+        "token by token": [1] * 72 + [n - 72],
+        "twos": [2] * 20 + [60] + [2] * 10 + [n - 120],
+        "odd": [63, 1, 65, 3, 64, n - 196],
+        "chunk edges": [127, 2, 1, n - 130],
+        "sevens": [7] * 30,
+    }
+    for what, cuts in schedules.items():
+        assert sum(cuts) == n
+        r = replay(models, name, device, dtype, n)
+        got = nc.run_schedule(r, {"a": toks}, [[("a", c)] for c in cuts])["a"]
+        check(got, want, dtype, f"{name}: {what}")
+        assert r.engine.pool.used == 0 and len(r.engine._free_slots) == 4
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+@pytest.mark.parametrize("name", list(pc.CASES))
+def test_unequal_batches_and_used_pages_and_slots(models, name, device, dtype):
+    """Portions beside single tokens in one step; later sequences run in pages and slots that earlier ones left, in a
+    pool that holds no more than the live ones need."""
+    seqs, want = {}, {}
+    for i, n in enumerate((130, 66, 1, 97, 64, 129, 40)):
+        seqs[f"s{i}"], want[f"s{i}"] = expected(models, name, n, 10 + i)
+    schedule = [[("s0", 50), ("s1", 1), ("s2", 1)],
+                [("s0", 1), ("s1", 63), ("s3", 2)],
+                [("s3", 90), ("s0", 78), ("s1", 1)],
+                [("s1", 1), ("s0", 1), ("s3", 1), ("s4", 64)],          # s0, s1 and s4 end
+                [("s3", 1), ("s5", 1)], [("s3", 1), ("s5", 1)],          # two decoded together
+                [("s5", 120), ("s6", 3)], [("s5", 1), ("s6", 36), ("s3", 1)],
+                [("s5", 1), ("s3", 1), ("s6", 1)]] + [[("s5", 1)]] * 5
+    r = replay(models, name, device, dtype, 8 * 64)
+    for turn in range(2):                                                # the second turn only sees used pages
+        got = nc.run_schedule(r, seqs, schedule)
+        for k in seqs:
+            check(got[k], want[k], dtype, f"{name} {k} turn {turn}")
+        assert r.engine.pool.used == 0
+    with pytest.raises(OutOfBlocks):
+        r.step([{"id": "big", "tokens": [0] * (8 * 64 + 1), "want": []}], [])
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+def test_long_prompt_in_long_portions(models, device, dtype):
+    """Hundreds of tokens a step: tiles that recompute the rows in front of them, chunks of the recurrence, key splits."""
+    toks, want = expected(models, "wide", 900, 30)
+    for cuts in ([900], [400, 1, 499], [513, 2, 2, 383]):
+        r = replay(models, "wide", device, dtype, 900)
+        check(nc.run_schedule(r, {"a": toks}, [[("a", c)] for c in cuts])["a"], want, dtype, str(cuts))
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+def test_long_decoding(models, device, dtype):
+    toks, want = expected(models, "mixed", 330, 40)
+    r = replay(models, "mixed", device, dtype, 330)
+    got = nc.run_schedule(r, {"a": toks}, [[("a", 20)]] + [[("a", 1)]] * 310)["a"]
+    check(got, want, dtype)
+    if device != "cpu":
+        assert r.engine._graphs.replays == 310                           # decode steps replay the captured graph
+
+
+@pytest.mark.parametrize("device,dtype", WHERE[:2])
+def test_greedy_generation_through_the_scheduler(models, device, dtype):
+    """Concurrent requests of unequal length, prompts cut into chunks, a resumed prefix: the tokens of the plain
+    implementation's greedy continuation."""
+    cfg, w, path = models["mixed"]
+    mc, lw, tok, _ = load_model(path, device, getattr(torch, dtype))
+    eng = LmEngine(Decoder(mc, lw, None, max_position=264), tok,
+                   EngineConfig(ctx_size=256, max_seqs=3, block_size=16, prefill_chunk=24, max_batch_tokens=40,
+                                prefix_cache=True, device=device))
+
+    def greedy(prompt, n):
+        t = list(prompt)
+        for _ in range(n):
+            t.append(int(oracle.forward(cfg, w, t)[-1].argmax()))
+        return t[len(prompt):]
+    prompts = [nc.tokens(cfg, n, 60 + n) for n in (5, 61, 33, 90)]
+    want = [greedy(p, 6) for p in prompts]
+    streams = [eng.generate(GenerateRequest(prompt_tokens=list(p), sampling=SamplingParams(
+        temperature=0.0, max_tokens=6, ignore_eos=True))) for p in prompts]
+    assert [s.collect().token_ids for s in streams] == want
+    # a longer conversation over the cached prefix: pages and the states come back
+    follow = prompts[3] + want[3] + nc.tokens(cfg, 9, 77)
+    out = eng.generate_text(tokens=follow, temperature=0.0, max_tokens=4, ignore_eos=True)
+    assert out.token_ids == greedy(follow, 4) and out.usage.cached_tokens > 0
+    eng.shutdown()
+
+
+def test_preempted_sequences_are_recomputed():
+    c = PRESETS["tiny-pemezen"]()
+    prompts = [torch.randint(0, 256, (n,), generator=torch.Generator().manual_seed(n)).tolist() for n in (40, 33, 50)]
+
+    def run(**kw):
+        eng = build_engine(c, engine_cfg=EngineConfig(ctx_size=128, max_seqs=3, block_size=16, prefill_chunk=32,
+                                                      prefix_cache=False, **kw))
+        ss = [eng.generate(GenerateRequest(prompt_tokens=p, sampling=SamplingParams(temperature=0.0, max_tokens=40,
+                                                                                   ignore_eos=True))) for p in prompts]
+        out = [s.collect().token_ids for s in ss]
+        n = eng.stats().kv_preemptions
+        eng.shutdown()
+        return out, n
+    plain, _ = run()
+    for extra in ({}, {"kv_swap_gib": 0.1}):
+        tight, n = run(kv_admission="on-demand", kv_cache_tokens=12 * 16, **extra)
+        assert tight == plain and n > 0
+
+
+def test_speculation_and_ranks_are_refused():
+    from legion_b200.models.weights import Shard
+    c = PRESETS["tiny-pemezen"]()
+    with pytest.raises(ValueError, match="speculative"):
+        build_engine(c, engine_cfg=EngineConfig(ctx_size=64, max_seqs=1, spec="ngram"), start=False)
+    with pytest.raises(NotImplementedError):
+        Shard(c, 0, 2)
+
+
+@gpu
+def test_sampled_generation_on_gpu():
+    c = PRESETS["tiny-pemezen"]()
+    eng = build_engine(c, device="cuda:0", engine_cfg=EngineConfig(ctx_size=256, max_seqs=4, block_size=64))
+    a = eng.generate_text(tokens=list(range(70)), temperature=0.8, top_k=20, max_tokens=12, seed=3, ignore_eos=True)
+    b = eng.generate_text(tokens=list(range(70)), temperature=0.8, top_k=20, max_tokens=12, seed=3, ignore_eos=True)
+    assert a.error is None and len(a.token_ids) == 12 and a.token_ids == b.token_ids
+    eng.shutdown()
+
+
+@gpu
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+def test_trace_run_program(models, tmp_path, dtype):
+    cfg, w, path = models["mixed"]
+    toks, want = expected(models, "mixed", 66, 11)
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:40], "want": [0, 39]}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": toks[40:65], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "x", "tokens": toks[65:], "want": [0]}], "end": ["x"]}]
+    p = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", path, "--dtype", dtype, "--out",
+                        str(tmp_path), "--max-tokens", "128"], input="\n".join(json.dumps(s) for s in steps) + "\n",
+                       capture_output=True, text=True, timeout=240)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert [x for x in p.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2"]
+    assert not (tmp_path / "1.f32").exists()
+    for n, places in ((0, [0, 39]), (2, [65])):
+        got = torch.frombuffer(bytearray((tmp_path / f"{n}.f32").read_bytes()), dtype=torch.float32).view(len(places), -1)
+        e = nc.errors(got, want[places])
+        assert e.max() < (1e-4 if dtype == "float32" else 0.06), e
