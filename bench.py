@@ -13,6 +13,9 @@ Configurations (``--config``):
   7  the closest hybrid of the other families at that size: 24 layers of Gated DeltaNet and gated attention in turn,
      dense and 32-expert feed-forward parts, bf16 (the comparison for 6).
   8, 9  the same pair at 13B parameters (20 layers, 4096 columns).
+  10 Pemezen at 1B parameters in bf16 (24 layers: two RG-LRU layers and a latent-attention layer in turn).
+  11 the closest model of the other families at that size: dense latent attention in every layer (DeepSeek form).
+  12, 13  the same pair at 7B parameters (30 layers, 4096 columns).
 The ONE parsed number (``value``) is decode tokens/s at 16 users of the selected configuration; the other rows of
 the grid (1 and 64 users, 32K prefill) are under ``extra``.
 
@@ -100,6 +103,10 @@ CONFIGS = {
     7: dict(model="hybrid-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
     8: dict(model="nisasun-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
     9: dict(model="hybrid-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    10: dict(model="pemezen-1b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    11: dict(model="mla-1b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    12: dict(model="pemezen-7b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    13: dict(model="mla-7b", prompt_len=2048, weights="bf16", dtype="bf16"),
 }
 
 

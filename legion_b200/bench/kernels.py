@@ -472,6 +472,113 @@ def bench_hyper(rows):
             print(rows[-1], flush=True)
 
 
+def bench_resid(rows):
+    """The residual step between grouped norms (input convolution of four taps and history included) beside the residual +
+    RMS norm launch and the hyper-connection step of the other families."""
+    from legion_b200.ops import sm100
+    hbm, _, src = peaks()
+    for T, n_seq in ((1, 1), (16, 16), (64, 64), (1024, 1), (8192, 1), (8192, 8)):
+        for H in (2048, 4096):
+            x, y = torch.randn(T, H, device="cuda"), torch.randn(T, H, device="cuda").bfloat16()
+            w, taps, hist = torch.ones(H, device="cuda"), torch.randn(4, H, device="cuda"), torch.zeros(n_seq, 3, H, device="cuda")
+            L = T // n_seq
+            cu = torch.arange(0, T + 1, L, device="cuda", dtype=torch.int32)
+            slots = torch.arange(n_seq, device="cuda", dtype=torch.int32)
+            tm = timeit_graph if T <= 64 else timeit
+            for name, fn, byts in (
+                    (f"resid_step {H}", lambda: sm100.resid_step(x, y, w, w, 4, 1e-5, (taps, hist, cu, slots, True), max_len=L),
+                     T * H * 12 + hist.numel() * 8),
+                    (f"residual + rmsnorm {H}", lambda: sm100.rmsnorm(y, w, 1e-5, 0.0, y), T * H * 8)):
+                ms = tm(fn)
+                rows.append(dict(kernel=name, T=T, n_seq=n_seq, us=round(ms * 1e3, 2), frac_hbm=round(byts / ms / 1e6 / hbm, 3),
+                                 peaks=src))
+                print(rows[-1], flush=True)
+
+
+def bench_diag(rows):
+    """RG-LRU (2560 channels, 10 blocks): decode launch (convolution, gates, recurrence, GELU branch) and the launches of a
+    prompt. frac_hbm: bytes that must move once."""
+    from legion_b200.ops import sm100
+    hbm, tf, src = peaks()
+    W, nb, KC = 2560, 10, 4
+    d = W // nb
+    f = lambda *s: torch.randn(*s, device="cuda")                                    # noqa: E731
+    in_b, cw, cb, gb, ld, yb = f(W), f(W, KC), f(W), f(2 * W), -torch.rand(W, device="cuda"), f(W)
+    gw = (f(2 * W, d) * d ** -0.5).bfloat16()
+    for n, L in ((1, 1), (16, 1), (64, 1), (1, 8192), (8, 1024)):
+        T = n * L
+        cu, cu_host = torch.arange(0, T + 1, L, device="cuda", dtype=torch.int32), list(range(0, T + 1, L))
+        slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        proj = f(T, 2 * W).bfloat16()
+        y, x = proj[:, :W], proj[:, W:]
+        conv, st = torch.zeros(n, W, KC - 1, device="cuda"), torch.zeros(n, W, device="cuda")
+        if L == 1:
+            parts = [("rglru_decode", lambda: sm100.rglru_decode(x, in_b, cw, cb, conv, gw, gb, ld, y, yb, st, cu, slots, nb),
+                      T * W * 6 + st.numel() * 8 + conv.numel() * 8 + gw.numel() * 2)]
+        else:
+            cv = lambda: sm100.causal_conv1d_silu(x, cw, cb, conv, cu, slots, max_len=L, in_bias=in_b, silu=False)   # noqa: E731
+            u = cv()
+            gates = sm100.block_gates(u, gw, nb)
+            scan = lambda: sm100.gated_recurrence(u, gates, gb, ld, y, yb, st, cu, slots, nb, max_len=L, cu_host=cu_host)  # noqa: E731
+
+            def whole():
+                v = cv()
+                sm100.gated_recurrence(v, sm100.block_gates(v, gw, nb), gb, ld, y, yb, st, cu, slots, nb, max_len=L,
+                                       cu_host=cu_host)
+            parts = [("conv1d", cv, T * W * 4), ("block_gates", lambda: sm100.block_gates(u, gw, nb), T * W * 10 + gw.numel() * 2),
+                     ("gated_recurrence", scan, T * W * 14), ("rglru all", whole, T * W * 6)]
+        for name, fn, byts in parts:
+            ms = (timeit_graph if L == 1 else timeit)(fn)
+            rows.append(dict(kernel=name, n_seq=n, L=L, us=round(ms * 1e3, 2), frac_hbm=round(byts / ms / 1e6 / hbm, 3), peaks=src))
+            print(rows[-1], flush=True)
+
+
+def bench_latent(rows):
+    """Latent attention of two sizes: the pieces of a decode step and of a prompt. Attention by the bytes of the latents
+    (decode) or the FLOPs of the per-head form, 2 (dim + rot + vdim) per visible pair and head (prompts)."""
+    from legion_b200.ops import sm100
+    hbm, tf, src = peaks()
+    for H, dim, R, L, V in ((16, 128, 64, 512, 128), (32, 128, 64, 512, 128), (16, 64, 32, 256, 64)):
+        for n, q_len, ctx in ((1, 1, 8192), (16, 1, 2048), (16, 1, 8192), (64, 1, 8192), (1, 8192, 8192), (1, 2048, 16384)):
+            T, page = n * q_len, 64
+            f = lambda *s: (torch.randn(*s, device="cuda") * 0.5).bfloat16()        # noqa: E731
+            nb = n * ctx // page
+            cache, bt = f(nb, page, 1, L + R), torch.arange(nb, device="cuda", dtype=torch.int32).view(n, -1)
+            proj = f(T, H * (dim + R) + L + R + H * V)
+            nq = H * (dim + R)
+            q, kv, gate = proj[:, :nq], proj[:, nq:nq + L + R], proj[:, nq + L + R:]
+            uk, uv = f(H * L, dim), f(H * V, L)
+            w = torch.ones(L, device="cuda")
+            cs = torch.randn(ctx, R, device="cuda")
+            pos = torch.arange(ctx - q_len, ctx, device="cuda", dtype=torch.int32).repeat(n)
+            slots = torch.cat([torch.arange(ctx - q_len, ctx, device="cuda") + i * ctx for i in range(n)])
+            cu = torch.arange(0, T + 1, q_len, device="cuda", dtype=torch.int32)
+            cl = torch.full((n,), ctx, device="cuda", dtype=torch.int32)
+            pairs = n * (q_len * ctx - q_len * (q_len - 1) / 2)
+            for name, fn in latent_parts(sm100, q, kv, gate, uk, uv, w, cs, pos, slots, cache, bt, cl, cu, q_len, H, dim, R, L, ctx):
+                ms = (timeit_graph if q_len == 1 else timeit)(fn)
+                r = dict(kernel=name, heads=H, dims=(dim, R, L, V), n_seq=n, q_len=q_len, ctx=ctx, us=round(ms * 1e3, 2), peaks=src)
+                if "attention" in name or "all" in name:
+                    if q_len == 1:
+                        r["frac_hbm"] = round(n * ctx * (L + R) * 2 / ms / 1e6 / hbm, 3)
+                    else:
+                        r["frac_tflops"] = round(2.0 * H * pairs * (dim + R + V) / ms / 1e9 / tf, 3)
+                rows.append(r)
+                print(r, flush=True)
+
+
+def latent_parts(sm100, q, kv, gate, uk, uv, w, cs, pos, slots, cache, bt, cl, cu, q_len, H, dim, R, L, ctx):
+    qa = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
+    o = sm100.latent_attention(qa, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx)
+
+    def whole():
+        a = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
+        sm100.latent_values(sm100.latent_attention(a, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx), uv, gate)
+    return [("latent_queries", lambda: sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)),
+            ("latent_attention", lambda: sm100.latent_attention(qa, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx)),
+            ("latent_values", lambda: sm100.latent_values(o, uv, gate)), ("latent all", whole)]
+
+
 def bench_attn_sizes(rows):
     """Attention with key and value heads of different sizes, windowed and not, beside equal sizes: prompts by FLOPs of
     the visible scores, decode by the bytes of the visible keys and values."""
@@ -598,7 +705,7 @@ def main(argv=None):
     if a.gemm:
         CASE["gemm"] = [tuple(int(y) for y in x.split("x")) for x in a.gemm.split(",")]
     rows = []
-    table = {"linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
+    table = {"resid": bench_resid, "diag": bench_diag, "latent": bench_latent, "linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
     for name in a.only.split(","):
         table[name](rows)
     from legion_b200.ops.sm100 import Workspace

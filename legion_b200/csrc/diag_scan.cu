@@ -290,11 +290,145 @@ __global__ void __launch_bounds__(256) diag_decode_kernel(const DiagDecodeArgs a
   }
 }
 
+// The same step for bf16 and blocks of 32 to 256 channels (multiples of 32): the d / 32 CTAs of a block form a cluster.
+// Each evaluates u of its own 32 channels - so it owns their history - and hands it to the others through distributed
+// shared memory; its gate weights are on the way before the launch in front of this one has finished.
+template <int NK>
+__global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDecodeArgs a, const int d) {
+  __shared__ float u_s[DEC_SEQ][256];
+  __shared__ float z_s[2][DEC_SEQ][DEC_CH];
+  using T = __nv_bfloat16;
+  const DiagScanArgs& r = a.s;
+  const int parts = d / DEC_CH, b = blockIdx.x / parts, part = blockIdx.x % parts;
+  const int s0 = blockIdx.y * DEC_SEQ, ns = min(DEC_SEQ, r.n_seqs - s0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+  // warp w multiplies rows 8 w .. 8 w + 7 of the 2 x 32 gate rows of this CTA's channels; a lane holds 4 columns of every 128
+  const T* gw = static_cast<const T*>(a.gates_w) + long(b) * 2 * d * d;
+  uint2 w[8][NK];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int row = warp * 8 + i;
+    const T* wr = gw + (long(row / DEC_CH) * d + part * DEC_CH + row % DEC_CH) * d;
+#pragma unroll
+    for (int n = 0; n < NK; ++n) {
+      const int k = n * 128 + lane * 4;
+      w[i][n] = k < d ? *reinterpret_cast<const uint2*>(wr + k) : make_uint2(0u, 0u);
+    }
+  }
+  // threads 0..127: one (sequence, channel) each
+  const int q = threadIdx.x >> 5, c = b * d + part * DEC_CH + lane, K1 = a.KC - 1;
+  const bool mine = threadIdx.x < DEC_SEQ * DEC_CH && q < ns;
+  const Chan g = gate_of(c, d);
+  float br = 0.f, bi = 0.f, ld = 0.f, yb = 0.f, ib = 0.f, cb = 0.f;
+  if (mine) {
+    br = r.gates_b[g.r]; bi = r.gates_b[g.i]; ld = r.log_decay[c]; yb = r.y_b[c]; ib = a.in_bias[c];
+    cb = a.conv_b ? a.conv_b[c] : 0.f;
+  }
+  griddep_wait();
+  griddep_launch();
+  float u = 0.f, S = 0.f, yv = 0.f;
+  float* st = nullptr;
+  if (mine) {
+    const int seq = s0 + q, slot = r.slots[seq];
+    float* h = a.conv_state + (long(slot) * r.W + c) * K1;
+    const float* cw = a.conv_w + long(c) * a.KC;
+    st = r.state + long(slot) * r.W + c;
+    const float xv = ld_f(static_cast<const T*>(a.x) + seq * a.ldx + c) + ib;
+    S = *st;
+    yv = ld_f(static_cast<const T*>(r.y) + seq * r.ldy + c) + yb;
+    float acc = cb;
+    for (int j = 0; j < K1; ++j) {
+      const float hv = h[j];
+      acc = fmaf(cw[j], hv, acc);
+      if (j > 0) h[j - 1] = hv;
+    }
+    if (K1 > 0) h[K1 - 1] = xv;
+    u = __bfloat162float(__float2bfloat16(fmaf(cw[K1], xv, acc)));
+  }
+  asm volatile("barrier.cluster.wait.aligned;" ::: "memory");        // every CTA of the cluster has started
+  if (threadIdx.x < DEC_SEQ * DEC_CH) {
+    const uint32_t local = smem_u32(&u_s[q][part * DEC_CH + lane]);
+    for (int p = 0; p < parts; ++p) {
+      uint32_t remote;
+      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(p));
+      asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(u) : "memory");
+    }
+  }
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+  float v[32];
+#pragma unroll
+  for (int i = 0; i < 32; ++i) v[i] = 0.f;
+#pragma unroll
+  for (int n = 0; n < NK; ++n) {
+    const int k = n * 128 + lane * 4;
+    if (k < d) {
+      float4 uu[DEC_SEQ];
+#pragma unroll
+      for (int s = 0; s < DEC_SEQ; ++s) uu[s] = *reinterpret_cast<const float4*>(&u_s[s][k]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float2 w0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].x));
+        const float2 w1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].y));
+#pragma unroll
+        for (int s = 0; s < DEC_SEQ; ++s)
+          v[i * DEC_SEQ + s] = fmaf(w0.x, uu[s].x, fmaf(w0.y, uu[s].y, fmaf(w1.x, uu[s].z, fmaf(w1.y, uu[s].w,
+                                                                                              v[i * DEC_SEQ + s]))));
+      }
+    }
+  }
+  // sum over the lanes: lane l ends up with value l (row l / 4, sequence l % 4)
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  const int row = warp * 8 + lane / DEC_SEQ;
+  z_s[row / DEC_CH][lane % DEC_SEQ][row % DEC_CH] = v[0];
+  __syncthreads();
+  if (mine) {
+    const float2 ab = recur_terms<T>(z_s[0][q][lane] + br, z_s[1][q][lane] + bi, u, ld);
+    S = fmaf(ab.x, S, ab.y);
+    *st = S;
+    st_f(static_cast<T*>(r.out) + (s0 + q) * r.ldo + c, S * gelu_branch<T>(yv));
+  }
+}
+
+template <int NK>
+int decode_cluster(const DiagDecodeArgs& a, int d, cudaStream_t s) {
+  const int parts = d / DEC_CH;
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3(a.s.blocks * parts, (a.s.n_seqs + DEC_SEQ - 1) / DEC_SEQ);
+  cfg.blockDim = dim3(256);
+  cfg.stream = s;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = parts;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  cfg.numAttrs = 1;
+  if (pdl_enabled()) {
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.numAttrs = 2;
+  }
+  cfg.attrs = attr;
+  return cudaLaunchKernelEx(&cfg, diag_decode_cluster_kernel<NK>, a, d) != cudaSuccess;
+}
+
 template <typename T>
 int decode_t(DiagDecodeArgs a, cudaStream_t s) {
   const int d = a.s.W / a.s.blocks, parts = (d + DEC_CH - 1) / DEC_CH;
   const size_t smem = size_t(DEC_SEQ) * d * 4;
   a.vec = d % 4 == 0 && reinterpret_cast<uintptr_t>(a.gates_w) % (4 * sizeof(T)) == 0;
+  if constexpr (sizeof(T) == 2) {
+    if (d % DEC_CH == 0 && d <= 256 && a.s.write_state && reinterpret_cast<uintptr_t>(a.gates_w) % 8 == 0)
+      return d <= 128 ? decode_cluster<1>(a, d, s) : decode_cluster<2>(a, d, s);
+  }
   if (smem > 200 * 1024) return 1;
   auto k = diag_decode_kernel<T>;
   if (smem > 40 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess) return 1;

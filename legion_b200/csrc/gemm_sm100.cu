@@ -675,6 +675,37 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               }
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
+          } else if (OUT_F32 && a.vec_ok) {
+            // fp32 rows leave as 16-byte stores too: a warp writes one token's 128 features, 4 token rows per pass
+            const int etid = threadIdx.x - 64;
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              float v = g[j];
+              if (DUAL) v = gate_act(v, a.act) * u[j];
+              else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
+              stage[j * BM + row] = v;
+            }
+            asm volatile("bar.sync 2, 128;" ::: "memory");
+            const int f4 = (etid & 31) * 4;
+            const int feat4 = it.feat0 + f4;
+#pragma unroll
+            for (int pass = 0; pass < 8; ++pass) {
+              const int j = pass * 4 + (etid >> 5);
+              const int t = c + j;
+              if (t < it.ntok && feat4 < a.n_feat) {
+                const int xrow = it.out0 + t;
+                const long orow = a.out_rows ? a.out_rows[xrow] : xrow;
+                if (orow >= 0) {
+                  float4 v = *reinterpret_cast<const float4*>(&stage[j * BM + f4]);
+                  if (a.tok_scale) {
+                    const float sc = a.tok_scale[xrow];
+                    v.x *= sc; v.y *= sc; v.z *= sc; v.w *= sc;
+                  }
+                  *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.out) + orow * a.ldo + feat4) = v;
+                }
+              }
+            }
+            asm volatile("bar.sync 2, 128;" ::: "memory");
           } else if (feat_ok) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
@@ -895,6 +926,9 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
   a.vec_ok = (!h.out_f32 && h.n_feat % 8 == 0 && h.ldo % 8 == 0 && (reinterpret_cast<uintptr_t>(h.out) & 15) == 0 &&
               (!h.residual || (h.ldr % 8 == 0 && (reinterpret_cast<uintptr_t>(h.residual) & 15) == 0)))
                  ? 1 : 0;
+  if (h.out_f32 && h.n_feat % 4 == 0 && h.ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(h.out) & 15) == 0 && !h.residual &&
+      h.n_out_peer == 0)
+    a.vec_ok = 1;
   if (h.q8_out) a.vec_ok = 1;     // the encoded rows always leave through the staged write-out
   const int num_kb = fp8 ? h.K / 128 : (h.K + BK - 1) / BK;
   if (a.split_k > num_kb) a.split_k = num_kb;

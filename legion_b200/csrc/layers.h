@@ -42,7 +42,6 @@ struct ResidStepArgs {
   int write_state;
   void* h; long ldh;
   int rows, H;
-  int lanes;                       // set by the launcher
 };
 int resid_step_launch(const ResidStepArgs& a, bool f32, cudaStream_t s);
 

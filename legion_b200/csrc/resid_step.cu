@@ -5,11 +5,12 @@
 // in one launch per sublayer, so that the residual and the sublayer output are read once. The last K - 1 rows of n are a
 // sequence's history; the launch reads and replaces it.
 //
-// A CTA walks up to `tok` consecutive tokens of one sequence with the previous rows of n in registers. A tile in the
-// middle of a sequence recomputes n of the K - 1 tokens in front of it from x and y (the new residual goes to a second
-// buffer, so these are still there). Only the first tile of a sequence touches the history: it reads it, and replaces it
-// with the rows of the sequence's last tokens, recomputed when they lie in another tile. So no launch waits and no two
-// CTAs meet in the state.
+// A norm never leaves its group, so a CTA takes one group of columns and walks up to `tok` consecutive tokens of one
+// sequence with the previous rows of n in registers: one warp for groups of up to 512 columns (no barrier at all), several
+// for wider ones. A tile in the middle of a sequence recomputes n of the K - 1 tokens in front of it from x and y (the new
+// residual goes to a second buffer, so these are still there). Only the first tile of a sequence touches the history: it
+// reads it, and replaces it with the rows of the sequence's last tokens, recomputed when they lie in another tile. So no
+// launch waits and no two CTAs meet in the state.
 #include <algorithm>
 
 #include "act_type.cuh"
@@ -52,28 +53,40 @@ __device__ __forceinline__ Tile find_tile(const int* __restrict__ cu, int n_seqs
   return Tile{-1, 0, 0, 0};
 }
 
-template <typename T, int VEC, int NC, int KMAX>
-__global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) {
-  extern __shared__ float part_s[];                       // two buffers of partial sums of squares
+template <typename T, int VEC, int NC, int KMAX, bool ONE_WARP>
+__global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 16 && KMAX <= 4 ? 12 : 1)
+    resid_step_kernel(const ResidStepArgs a) {
+  __shared__ float part_s[2][16];
+  const int tid = threadIdx.x, nt = blockDim.x, H = a.H, gs = H / a.groups;
+  const int tile = blockIdx.x / a.groups, col0 = (blockIdx.x % a.groups) * gs;
+  constexpr int R = KMAX > 1 ? KMAX - 1 : 1;
+  const int K1 = KMAX > 1 ? a.taps_n - 1 : 0;
+  const bool start = a.x_in == nullptr;
+  // this thread's columns
+  bool on[NC];
+  int col[NC];
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int d = (c * nt + tid) * VEC;
+    on[c] = d < gs;
+    col[c] = col0 + d;
+  }
   griddep_wait();
   griddep_launch();
-  const int tid = threadIdx.x, nt = blockDim.x, H = a.H;
   Tile tl;
   if (a.tok >= a.max_len) {
-    tl.seq = blockIdx.x;
-    tl.t0 = tl.ta = a.cu ? a.cu[tl.seq] : int(blockIdx.x);
+    tl.seq = tile;
+    tl.t0 = tl.ta = a.cu ? a.cu[tl.seq] : tile;
     tl.t1 = a.cu ? a.cu[tl.seq + 1] : tl.t0 + 1;
   } else {
-    tl = find_tile(a.cu, a.n_seqs, a.tok, blockIdx.x);
+    tl = find_tile(a.cu, a.n_seqs, a.tok, tile);
   }
   if (tl.seq < 0 || tl.ta >= tl.t1) return;
   const int tb = min(tl.t1, tl.ta + a.tok);
-  const int gs = H / a.groups, W = a.lanes, ppg = gs / (VEC * W), n_part = H / (VEC * W);
   const float gs_inv = 1.f / float(gs);
-  const bool start = a.x_in == nullptr;
 
-  float xv[NC][VEC], yv[NC][VEC];
-  auto load = [&](int t) {
+  struct Row { float x[NC][VEC], y[NC][VEC]; };
+  auto load = [&](int t, Row& r) {
     const T* er = nullptr;
     if (start) {
       long row = t;
@@ -84,91 +97,69 @@ __global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) 
       er = static_cast<const T*>(a.emb) + row * a.ld_emb;
     }
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int d = (c * nt + tid) * VEC;
-      if (d < H) {
+    for (int c = 0; c < NC; ++c)
+      if (on[c]) {
         if (start) {
-          ld_vec<VEC>(er + d, xv[c]);
+          ld_vec<VEC>(er + col[c], r.x[c]);
         } else {
-          ld_vec<VEC>(a.x_in + long(t) * H + d, xv[c]);
-          ld_vec<VEC>(static_cast<const T*>(a.y) + long(t) * a.ldy + d, yv[c]);
+          ld_vec<VEC>(static_cast<const T*>(a.y) + long(t) * a.ldy + col[c], r.y[c]);
+          ld_vec<VEC>(a.x_in + long(t) * H + col[c], r.x[c]);
         }
       }
-    }
   };
-  // 1 / rms of the group that holds each of this thread's vectors
-  auto group_inv = [&](const float (&v)[NC][VEC], float* part, float (&inv)[NC]) {
+  auto inv_rms = [&](const float (&v)[NC][VEC], int buf) {
+    float ss = 0.f;
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int d = (c * nt + tid) * VEC;
-      float ss = 0.f;
-      if (d < H) {
+    for (int c = 0; c < NC; ++c)
+      if (on[c]) {
 #pragma unroll
         for (int j = 0; j < VEC; ++j) ss = fmaf(v[c][j], v[c][j], ss);
       }
-      for (int o = W >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      if (d < H && (tid & (W - 1)) == 0) part[d / (VEC * W)] = ss;
+    ss = warp_sum_f(ss);
+    if constexpr (!ONE_WARP) {
+      if ((tid & 31) == 0) part_s[buf][tid >> 5] = ss;
+      __syncthreads();
+      ss = 0.f;
+      for (int i = 0; i < nt / 32; ++i) ss += part_s[buf][i];
     }
-    __syncthreads();
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int d = (c * nt + tid) * VEC;
-      inv[c] = 0.f;
-      if (d < H) {
-        const float* p = part + (d / gs) * ppg;
-        float s = 0.f;
-        for (int i = 0; i < ppg; ++i) s += p[i];
-        inv[c] = 1.f / sqrtf(s * gs_inv + a.eps);
-      }
-    }
+    return 1.f / sqrtf(ss * gs_inv + a.eps);
   };
-  // n of the token whose x and y are loaded; the new residual is written when the token is this tile's own
+  // n of a token; the new residual is written when the token is this tile's own
   float n[NC][VEC];
-  auto advance = [&](int t, bool own) {
-    float inv[NC];
+  auto advance = [&](int t, const Row& r, bool own) {
     if (start) {
+      if constexpr (!ONE_WARP) __syncthreads();            // with one norm per token its buffer is written every time
 #pragma unroll
       for (int c = 0; c < NC; ++c)
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) n[c][j] = xv[c][j] * a.emb_scale;
+        for (int j = 0; j < VEC; ++j) n[c][j] = r.x[c][j] * a.emb_scale;
     } else {
-      group_inv(yv, part_s, inv);
+      const float inv = inv_rms(r.y, 0);
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
-        const int d = (c * nt + tid) * VEC;
-        if (d < H) {
-          float pw[VEC];
-          ld_vec<VEC>(a.post_w + d, pw);
+        float w[VEC];
+        if (on[c]) ld_vec<VEC>(a.post_w + col[c], w);
 #pragma unroll
-          for (int j = 0; j < VEC; ++j) n[c][j] = xv[c][j] + yv[c][j] * inv[c] * pw[j];
-        }
+        for (int j = 0; j < VEC; ++j) n[c][j] = r.x[c][j] + r.y[c][j] * inv * w[j];
       }
     }
     if (own) {
 #pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        const int d = (c * nt + tid) * VEC;
-        if (d < H) st_vec<VEC>(a.x_out + long(t) * H + d, n[c]);
-      }
+      for (int c = 0; c < NC; ++c)
+        if (on[c]) st_vec<VEC>(a.x_out + long(t) * H + col[c], n[c]);
     }
-    group_inv(n, part_s + n_part, inv);
-    if (start) __syncthreads();                            // the one buffer in use is written again by the next token
+    const float inv = inv_rms(n, 1);
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
-      const int d = (c * nt + tid) * VEC;
-      if (d < H) {
-        float nw[VEC];
-        ld_vec<VEC>(a.norm_w + d, nw);
+      float w[VEC];
+      if (on[c]) ld_vec<VEC>(a.norm_w + col[c], w);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) n[c][j] *= inv[c] * nw[j];
-      }
+      for (int j = 0; j < VEC; ++j) n[c][j] *= inv * w[j];
     }
   };
 
-  // hist[KMAX - 2] is the row before the current token; rows older than K - 1 are not used
-  constexpr int R = KMAX > 1 ? KMAX - 1 : 1;
+  // hist[R - 1] is the row before the current token; rows older than K - 1 are not used
   float hist[R][NC][VEC];
-  const int K1 = KMAX > 1 ? a.taps_n - 1 : 0;
   auto push = [&]() {
     if constexpr (KMAX > 1) {
 #pragma unroll
@@ -185,6 +176,7 @@ __global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) 
   };
   float* st = (KMAX > 1 && a.hist) ? a.hist + long(a.slots[tl.seq]) * K1 * H : nullptr;
   const bool first = tl.ta == tl.t0;
+  Row cur;
   if constexpr (KMAX > 1) {
 #pragma unroll
     for (int i = 0; i < R; ++i)
@@ -198,60 +190,56 @@ __global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) 
         const int r = i - (R - K1);
         if (r >= 0) {
 #pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            const int d = (c * nt + tid) * VEC;
-            if (d < H) ld_vec<VEC>(st + long(r) * H + d, hist[i][c]);
-          }
+          for (int c = 0; c < NC; ++c)
+            if (on[c]) ld_vec<VEC>(st + long(r) * H + col[c], hist[i][c]);
         }
-      }
-    } else {
-      for (int t = tl.ta - K1; t < tl.ta; ++t) {
-        load(t);
-        advance(t, false);
-        push();
       }
     }
   }
-  load(tl.ta);
-  for (int t = tl.ta; t < tb; ++t) {
-    advance(t, true);
-    if (t + 1 < tb) load(t + 1);
-    T* hr = static_cast<T*>(a.h) + long(t) * a.ldh;
+  const int tw = first ? tl.ta : tl.ta - K1;                // rows in front of the tile come first
+  load(tw, cur);
+  for (int t = tw; t < tb; ++t) {
+    Row next;
+    if (t + 1 < tb) load(t + 1, next);
+    const bool own = t >= tl.ta;
+    advance(t, cur, own);
+    if (own) {
+      T* hr = static_cast<T*>(a.h) + long(t) * a.ldh;
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int d = (c * nt + tid) * VEC;
-      if (d < H) {
-        float o[VEC];
+      for (int c = 0; c < NC; ++c)
+        if (on[c]) {
+          float o[VEC];
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) o[j] = n[c][j];
-        if (a.taps) {
-          float w[VEC];
-          ld_vec<VEC>(a.taps + long(K1) * H + d, w);
+          for (int j = 0; j < VEC; ++j) o[j] = n[c][j];
+          if (a.taps) {
+            float w[VEC];
+            ld_vec<VEC>(a.taps + long(K1) * H + col[c], w);
 #pragma unroll
-          for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], n[c][j], o[j]);
-          if constexpr (KMAX > 1) {
+            for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], n[c][j], o[j]);
+            if constexpr (KMAX > 1) {
 #pragma unroll
-            for (int i = 0; i < R; ++i) {
-              const int r = i - (R - K1);
-              if (r >= 0) {
-                ld_vec<VEC>(a.taps + long(r) * H + d, w);
+              for (int i = 0; i < R; ++i) {
+                const int r = i - (R - K1);
+                if (r >= 0) {
+                  ld_vec<VEC>(a.taps + long(r) * H + col[c], w);
 #pragma unroll
-                for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], hist[i][c][j], o[j]);
+                  for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], hist[i][c][j], o[j]);
+                }
               }
             }
           }
+          st_vec<VEC>(hr + col[c], o);
         }
-        st_vec<VEC>(hr + d, o);
-      }
     }
     push();
+    cur = next;
   }
   if constexpr (KMAX > 1) {
     if (first && a.write_state && K1 > 0) {
-      if (tb < tl.t1) {                                    // the sequence's last tokens lie in another tile
+      if (tb < tl.t1) {                                     // the sequence's last tokens lie in another tile
         for (int t = tl.t1 - K1; t < tl.t1; ++t) {
-          load(t);
-          advance(t, false);
+          load(t, cur);
+          advance(t, cur, false);
           push();
         }
       }
@@ -260,51 +248,46 @@ __global__ void __launch_bounds__(512) resid_step_kernel(const ResidStepArgs a) 
         const int r = i - (R - K1);
         if (r >= 0) {
 #pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            const int d = (c * nt + tid) * VEC;
-            if (d < H) st_vec<VEC>(st + long(r) * H + d, hist[i][c]);
-          }
+          for (int c = 0; c < NC; ++c)
+            if (on[c]) st_vec<VEC>(st + long(r) * H + col[c], hist[i][c]);
         }
       }
     }
   }
 }
 
-template <typename T, int VEC, int NC>
+template <typename T, int VEC, int NC, bool ONE>
 int launch_k(const ResidStepArgs& a, int nt, dim3 grid, cudaStream_t s) {
-  const size_t smem = size_t(2) * (a.H / (VEC * a.lanes)) * 4;
-  if (smem > 48 * 1024) return 1;
   const int K = a.taps ? a.taps_n : 1;
 #define LB_K(N)                                                                                                        \
-  if (K <= N) return launch_pdl(resid_step_kernel<T, VEC, NC, N>, grid, dim3(nt), smem, s, a) != cudaSuccess;
+  if (K <= N) return launch_pdl(resid_step_kernel<T, VEC, NC, N, ONE>, grid, dim3(nt), 0, s, a) != cudaSuccess;
   LB_K(1) LB_K(4) LB_K(16)
 #undef LB_K
   return 1;
 }
 
 template <typename T>
-int dispatch(ResidStepArgs a, cudaStream_t s) {
+int dispatch(const ResidStepArgs& a, cudaStream_t s) {
   const size_t es = sizeof(T);
   auto al = [&](const void* p, size_t n) { return p == nullptr || reinterpret_cast<uintptr_t>(p) % n == 0; };
   const int gs = a.H / a.groups;
   const bool v4 = gs % 4 == 0 && al(a.x_in, 16) && al(a.x_out, 16) && al(a.emb, 4 * es) && al(a.y, 4 * es) &&
                   al(a.h, 4 * es) && al(a.post_w, 16) && al(a.norm_w, 16) && al(a.taps, 16) && al(a.hist, 16) &&
                   a.ld_emb % 4 == 0 && a.ldy % 4 == 0 && a.ldh % 4 == 0;
-  const int vec = v4 ? 4 : 1;
-  a.lanes = 1;
-  while (a.lanes < 32 && gs % (vec * a.lanes * 2) == 0) a.lanes *= 2;
-  const int need = (a.H + vec - 1) / vec;                 // threads for one vector each
-  const int nt = std::min(512, (need + 31) / 32 * 32), nc = (need + nt - 1) / nt;
-  const int tiles = a.tok >= a.max_len ? (a.cu ? a.n_seqs : a.rows) : a.rows / a.tok + a.n_seqs;
-  const dim3 grid(tiles);
-  if (vec == 4) {
-    if (nc <= 1) return launch_k<T, 4, 1>(a, nt, grid, s);
-    if (nc <= 2) return launch_k<T, 4, 2>(a, nt, grid, s);
-    if (nc <= 4) return launch_k<T, 4, 4>(a, nt, grid, s);
-    if (nc <= 8) return launch_k<T, 4, 8>(a, nt, grid, s);
+  const long tiles = a.tok >= a.max_len ? (a.cu ? a.n_seqs : a.rows) : a.rows / a.tok + a.n_seqs;
+  if (tiles * a.groups > 0x7fffffffL) return 1;
+  const dim3 grid(static_cast<unsigned>(tiles * a.groups));
+  const int need = v4 ? gs / 4 : gs;                        // threads with one vector each
+  const int nt = std::min(512, (need + 127) / 128 * 32), nc = (need + nt - 1) / nt;     // up to 4 vectors per thread
+  if (v4) {
+    if (need <= 32) return launch_k<T, 4, 1, true>(a, 32, grid, s);
+    if (nt == 32) return launch_k<T, 4, 4, true>(a, 32, grid, s);
+    if (nc <= 4) return launch_k<T, 4, 4, false>(a, nt, grid, s);
+    if (nc <= 8) return launch_k<T, 4, 8, false>(a, nt, grid, s);
   } else {
-    if (nc <= 1) return launch_k<T, 1, 1>(a, nt, grid, s);
-    if (nc <= 8) return launch_k<T, 1, 8>(a, nt, grid, s);
+    if (nt == 32) return launch_k<T, 1, 4, true>(a, 32, grid, s);
+    if (nc <= 4) return launch_k<T, 1, 4, false>(a, nt, grid, s);
+    if (nc <= 8) return launch_k<T, 1, 8, false>(a, nt, grid, s);
   }
   return 1;
 }

@@ -1666,11 +1666,13 @@ def group_norm_gate(y, gate, w, eps, groups: int = 1, out=None):
     return out
 
 
-def resid_tokens(rows: int, max_len: int) -> int:
-    """Tokens per CTA of ``resid_step``: long runs share the recomputed rows in front of a tile, short ones fill the SMs."""
+def resid_tokens(rows: int, max_len: int, width: int, groups: int) -> int:
+    """Tokens per CTA of ``resid_step``: as few as give one wave of CTAs (about 12 warps per SM, a warp per 512 columns of
+    a group), so that the rows recomputed in front of a tile cost little in long runs and short ones still fill the SMs."""
     if max_len <= 1:
         return 1
-    return 16 if rows >= 16 * NUM_SMS else 8
+    warps = groups * -(-(width // groups) // 512)
+    return max(4, min(32, -(-rows * warps // (12 * NUM_SMS))))
 
 
 def resid_step(x, y, post_w, norm_w, groups: int, eps: float, conv=None, start=None, max_len=None):
@@ -1687,7 +1689,9 @@ def resid_step(x, y, post_w, norm_w, groups: int, eps: float, conv=None, start=N
     taps, hist, cu, slots, write = conv if conv is not None else (None, None, None, None, False)
     rows = xo.shape[0]
     max_len = rows if max_len is None else max_len
-    tok = 1 if taps is None else max(resid_tokens(rows, max_len), min(taps.shape[0] - 1, max_len))
+    tok = 1
+    if taps is not None:
+        tok = max(resid_tokens(rows, max_len, xo.shape[1], groups), min(taps.shape[0] - 1, max_len))
     ext().resid_step(x, xo, table, ids, float(scale), y, post_w, norm_w, groups, eps, taps, hist, cu, slots, bool(write),
                      int(max_len), tok, h)
     return xo, h
