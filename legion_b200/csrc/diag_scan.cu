@@ -293,14 +293,16 @@ __global__ void __launch_bounds__(256) diag_decode_kernel(const DiagDecodeArgs a
 // The same step for bf16 and blocks of 32 to 256 channels (multiples of 32): the d / 32 CTAs of a block form a cluster.
 // Each evaluates u of its own 32 channels - so it owns their history - and hands it to the others through distributed
 // shared memory; its gate weights are on the way before the launch in front of this one has finished.
-template <int NK>
+// SEQ sequences per CTA, four at a time through the products.
+template <int NK, int SEQ>
 __global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDecodeArgs a, const int d) {
-  __shared__ float u_s[DEC_SEQ][256];
-  __shared__ float z_s[2][DEC_SEQ][DEC_CH];
+  constexpr int PER = (SEQ * DEC_CH + 255) / 256;        // (sequence, channel) pairs per thread: sequence q + 8 p
+  __shared__ float u_s[SEQ][256];
+  __shared__ float z_s[2][SEQ][DEC_CH];
   using T = __nv_bfloat16;
   const DiagScanArgs& r = a.s;
   const int parts = d / DEC_CH, b = blockIdx.x / parts, part = blockIdx.x % parts;
-  const int s0 = blockIdx.y * DEC_SEQ, ns = min(DEC_SEQ, r.n_seqs - s0);
+  const int s0 = blockIdx.y * SEQ, ns = min(SEQ, r.n_seqs - s0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
   // warp w multiplies rows 8 w .. 8 w + 7 of the 2 x 32 gate rows of this CTA's channels; a lane holds 4 columns of every 128
@@ -316,94 +318,105 @@ __global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDeco
       w[i][n] = k < d ? *reinterpret_cast<const uint2*>(wr + k) : make_uint2(0u, 0u);
     }
   }
-  // threads 0..127: one (sequence, channel) each
-  const int q = threadIdx.x >> 5, c = b * d + part * DEC_CH + lane, K1 = a.KC - 1;
-  const bool mine = threadIdx.x < DEC_SEQ * DEC_CH && q < ns;
+  const int c = b * d + part * DEC_CH + lane, K1 = a.KC - 1;
   const Chan g = gate_of(c, d);
-  float br = 0.f, bi = 0.f, ld = 0.f, yb = 0.f, ib = 0.f, cb = 0.f;
-  if (mine) {
-    br = r.gates_b[g.r]; bi = r.gates_b[g.i]; ld = r.log_decay[c]; yb = r.y_b[c]; ib = a.in_bias[c];
-    cb = a.conv_b ? a.conv_b[c] : 0.f;
-  }
+  const float br = r.gates_b[g.r], bi = r.gates_b[g.i], ld = r.log_decay[c], yb = r.y_b[c], ib = a.in_bias[c];
+  const float cb = a.conv_b ? a.conv_b[c] : 0.f;
   griddep_wait();
   griddep_launch();
-  float u = 0.f, S = 0.f, yv = 0.f;
-  float* st = nullptr;
-  if (mine) {
-    const int seq = s0 + q, slot = r.slots[seq];
-    float* h = a.conv_state + (long(slot) * r.W + c) * K1;
-    const float* cw = a.conv_w + long(c) * a.KC;
-    st = r.state + long(slot) * r.W + c;
-    const float xv = ld_f(static_cast<const T*>(a.x) + seq * a.ldx + c) + ib;
-    S = *st;
-    yv = ld_f(static_cast<const T*>(r.y) + seq * r.ldy + c) + yb;
-    float acc = cb;
-    for (int j = 0; j < K1; ++j) {
-      const float hv = h[j];
-      acc = fmaf(cw[j], hv, acc);
-      if (j > 0) h[j - 1] = hv;
+  float u[PER], S[PER], yv[PER];
+  float* st[PER];
+#pragma unroll
+  for (int p = 0; p < PER; ++p) {
+    const int q = warp + 8 * p;
+    u[p] = 0.f;
+    st[p] = nullptr;
+    if (q < ns) {
+      const int seq = s0 + q, slot = r.slots[seq];
+      float* h = a.conv_state + (long(slot) * r.W + c) * K1;
+      const float* cw = a.conv_w + long(c) * a.KC;
+      st[p] = r.state + long(slot) * r.W + c;
+      const float xv = ld_f(static_cast<const T*>(a.x) + seq * a.ldx + c) + ib;
+      S[p] = *st[p];
+      yv[p] = ld_f(static_cast<const T*>(r.y) + seq * r.ldy + c) + yb;
+      float acc = cb;
+      for (int j = 0; j < K1; ++j) {
+        const float hv = h[j];
+        acc = fmaf(cw[j], hv, acc);
+        if (j > 0) h[j - 1] = hv;
+      }
+      if (K1 > 0) h[K1 - 1] = xv;
+      u[p] = __bfloat162float(__float2bfloat16(fmaf(cw[K1], xv, acc)));
     }
-    if (K1 > 0) h[K1 - 1] = xv;
-    u = __bfloat162float(__float2bfloat16(fmaf(cw[K1], xv, acc)));
   }
   asm volatile("barrier.cluster.wait.aligned;" ::: "memory");        // every CTA of the cluster has started
-  if (threadIdx.x < DEC_SEQ * DEC_CH) {
-    const uint32_t local = smem_u32(&u_s[q][part * DEC_CH + lane]);
-    for (int p = 0; p < parts; ++p) {
-      uint32_t remote;
-      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(p));
-      asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(u) : "memory");
+#pragma unroll
+  for (int p = 0; p < PER; ++p) {
+    const int q = warp + 8 * p;
+    if (q < SEQ) {
+      const uint32_t local = smem_u32(&u_s[q][part * DEC_CH + lane]);
+      for (int k = 0; k < parts; ++k) {
+        uint32_t remote;
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(k));
+        asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(u[p]) : "memory");
+      }
     }
   }
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-  float v[32];
+#pragma unroll 1
+  for (int q0 = 0; q0 < ns; q0 += 4) {
+    float v[32];
 #pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = 0.f;
+    for (int i = 0; i < 32; ++i) v[i] = 0.f;
 #pragma unroll
-  for (int n = 0; n < NK; ++n) {
-    const int k = n * 128 + lane * 4;
-    if (k < d) {
-      float4 uu[DEC_SEQ];
+    for (int n = 0; n < NK; ++n) {
+      const int k = n * 128 + lane * 4;
+      if (k < d) {
+        float4 uu[4];
 #pragma unroll
-      for (int s = 0; s < DEC_SEQ; ++s) uu[s] = *reinterpret_cast<const float4*>(&u_s[s][k]);
+        for (int s = 0; s < 4; ++s) uu[s] = *reinterpret_cast<const float4*>(&u_s[q0 + s][k]);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const float2 w0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].x));
-        const float2 w1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].y));
+        for (int i = 0; i < 8; ++i) {
+          const float2 w0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].x));
+          const float2 w1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].y));
 #pragma unroll
-        for (int s = 0; s < DEC_SEQ; ++s)
-          v[i * DEC_SEQ + s] = fmaf(w0.x, uu[s].x, fmaf(w0.y, uu[s].y, fmaf(w1.x, uu[s].z, fmaf(w1.y, uu[s].w,
-                                                                                              v[i * DEC_SEQ + s]))));
+          for (int s = 0; s < 4; ++s)
+            v[i * 4 + s] = fmaf(w0.x, uu[s].x, fmaf(w0.y, uu[s].y, fmaf(w1.x, uu[s].z, fmaf(w1.y, uu[s].w, v[i * 4 + s]))));
+        }
       }
     }
-  }
-  // sum over the lanes: lane l ends up with value l (row l / 4, sequence l % 4)
+    // sum over the lanes: lane l ends up with value l (row l / 4, sequence l % 4)
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const bool up = lane & o;
+    for (int o = 16; o > 0; o >>= 1) {
+      const bool up = lane & o;
 #pragma unroll
-    for (int i = 0; i < o; ++i) {
-      const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
-      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      for (int i = 0; i < o; ++i) {
+        const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      }
     }
+    const int row = warp * 8 + lane / 4;
+    z_s[row / DEC_CH][q0 + lane % 4][row % DEC_CH] = v[0];
   }
-  const int row = warp * 8 + lane / DEC_SEQ;
-  z_s[row / DEC_CH][lane % DEC_SEQ][row % DEC_CH] = v[0];
   __syncthreads();
-  if (mine) {
-    const float2 ab = recur_terms<T>(z_s[0][q][lane] + br, z_s[1][q][lane] + bi, u, ld);
-    S = fmaf(ab.x, S, ab.y);
-    *st = S;
-    st_f(static_cast<T*>(r.out) + (s0 + q) * r.ldo + c, S * gelu_branch<T>(yv));
+#pragma unroll
+  for (int p = 0; p < PER; ++p) {
+    const int q = warp + 8 * p;
+    if (q < ns) {
+      const float2 ab = recur_terms<T>(z_s[0][q][lane] + br, z_s[1][q][lane] + bi, u[p], ld);
+      const float Sn = fmaf(ab.x, S[p], ab.y);
+      *st[p] = Sn;
+      st_f(static_cast<T*>(r.out) + (s0 + q) * r.ldo + c, Sn * gelu_branch<T>(yv[p]));
+    }
   }
 }
 
-template <int NK>
+template <int NK, int SEQ>
 int decode_cluster(const DiagDecodeArgs& a, int d, cudaStream_t s) {
   const int parts = d / DEC_CH;
   cudaLaunchConfig_t cfg{};
-  cfg.gridDim = dim3(a.s.blocks * parts, (a.s.n_seqs + DEC_SEQ - 1) / DEC_SEQ);
+  cfg.gridDim = dim3(a.s.blocks * parts, (a.s.n_seqs + SEQ - 1) / SEQ);
   cfg.blockDim = dim3(256);
   cfg.stream = s;
   cudaLaunchAttribute attr[2];
@@ -417,7 +430,15 @@ int decode_cluster(const DiagDecodeArgs& a, int d, cudaStream_t s) {
     cfg.numAttrs = 2;
   }
   cfg.attrs = attr;
-  return cudaLaunchKernelEx(&cfg, diag_decode_cluster_kernel<NK>, a, d) != cudaSuccess;
+  return cudaLaunchKernelEx(&cfg, diag_decode_cluster_kernel<NK, SEQ>, a, d) != cudaSuccess;
+}
+template <int NK>
+int decode_cluster_n(const DiagDecodeArgs& a, int d, cudaStream_t s) {
+  // as many sequences per CTA as leave about one wave of two CTAs per SM
+  const long ctas = long(a.s.W / DEC_CH) * ((a.s.n_seqs + 3) / 4);
+  if (ctas <= 296) return decode_cluster<NK, 4>(a, d, s);
+  if (ctas <= 592) return decode_cluster<NK, 8>(a, d, s);
+  return decode_cluster<NK, 16>(a, d, s);
 }
 
 template <typename T>
@@ -427,7 +448,7 @@ int decode_t(DiagDecodeArgs a, cudaStream_t s) {
   a.vec = d % 4 == 0 && reinterpret_cast<uintptr_t>(a.gates_w) % (4 * sizeof(T)) == 0;
   if constexpr (sizeof(T) == 2) {
     if (d % DEC_CH == 0 && d <= 256 && a.s.write_state && reinterpret_cast<uintptr_t>(a.gates_w) % 8 == 0)
-      return d <= 128 ? decode_cluster<1>(a, d, s) : decode_cluster<2>(a, d, s);
+      return d <= 128 ? decode_cluster_n<1>(a, d, s) : decode_cluster_n<2>(a, d, s);
   }
   if (smem > 200 * 1024) return 1;
   auto k = diag_decode_kernel<T>;

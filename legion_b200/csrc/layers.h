@@ -42,6 +42,7 @@ struct ResidStepArgs {
   int write_state;
   void* h; long ldh;
   int rows, H;
+  int direct;                      // set by the launcher
 };
 int resid_step_launch(const ResidStepArgs& a, bool f32, cudaStream_t s);
 

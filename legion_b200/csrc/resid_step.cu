@@ -22,6 +22,13 @@ namespace {
 
 struct Tile { int seq, t0, t1, ta; };
 
+constexpr int RING = 4;          // tokens whose rows are on the way to shared memory
+
+template <int BYTES>
+__device__ __forceinline__ void copy_async(void* smem, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(smem)), "l"(src), "n"(BYTES) : "memory");
+}
+
 // The sequence and first token of tile `idx` when every sequence is cut into tiles of `tok` tokens (warp-wide; seq < 0:
 // no such tile).
 __device__ __forceinline__ Tile find_tile(const int* __restrict__ cu, int n_seqs, int tok, int idx) {
@@ -85,7 +92,53 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
   const int tb = min(tl.t1, tl.ta + a.tok);
   const float gs_inv = 1.f / float(gs);
 
+  // Four columns at a time: a token's rows come through a ring in shared memory, every thread copying what it reads itself
+  extern __shared__ __align__(16) uint8_t ring_s[];
+  constexpr bool ASYNC = VEC == 4;
+  constexpr int YB = 4 * int(sizeof(T));
+  auto ring_x = [&](int stage, int c) { return ring_s + size_t((stage * NC + c) * nt + tid) * 16; };
+  auto ring_y = [&](int stage, int c) { return ring_s + size_t(RING * NC * nt) * 16 + size_t((stage * NC + c) * nt + tid) * YB; };
+  auto issue = [&](int t, int t_end, int stage) {
+    if constexpr (ASYNC) {
+      if (t < t_end && !a.direct) {
+        if (start) {
+          long row = t;
+          if (a.ids) {
+            const int id = a.ids[t];
+            row = (id < 0 || id >= a.vocab) ? 0 : id;
+          }
+          const T* er = static_cast<const T*>(a.emb) + row * a.ld_emb;
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+            if (on[c]) copy_async<YB>(ring_y(stage, c), er + col[c]);
+        } else {
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+            if (on[c]) {
+              copy_async<YB>(ring_y(stage, c), static_cast<const T*>(a.y) + long(t) * a.ldy + col[c]);
+              copy_async<16>(ring_x(stage, c), a.x_in + long(t) * H + col[c]);
+            }
+        }
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+  };
   struct Row { float x[NC][VEC], y[NC][VEC]; };
+  auto take = [&](int stage, Row& r) {
+    if constexpr (ASYNC) {
+      asm volatile("cp.async.wait_group %0;" ::"n"(RING - 1) : "memory");
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+        if (on[c]) {
+          if (start) {
+            ld_vec<VEC>(reinterpret_cast<const T*>(ring_y(stage, c)), r.x[c]);
+          } else {
+            ld_vec<VEC>(reinterpret_cast<const T*>(ring_y(stage, c)), r.y[c]);
+            ld_vec<VEC>(reinterpret_cast<const float*>(ring_x(stage, c)), r.x[c]);
+          }
+        }
+    }
+  };
   auto load = [&](int t, Row& r) {
     const T* er = nullptr;
     if (start) {
@@ -197,11 +250,19 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
     }
   }
   const int tw = first ? tl.ta : tl.ta - K1;                // rows in front of the tile come first
-  load(tw, cur);
-  for (int t = tw; t < tb; ++t) {
-    Row next;
-    if (t + 1 < tb) load(t + 1, next);
-    const bool own = t >= tl.ta;
+  // rows [tw, tb), and behind them, where this tile owns the history, the sequence's last rows
+  const bool tail = KMAX > 1 && first && a.write_state && K1 > 0 && tb < tl.t1;
+  const int n_rows = tb - tw, n_all = n_rows + (tail ? K1 : 0);
+  auto row_at = [&](int i) { return i < n_rows ? tw + i : tl.t1 - K1 + (i - n_rows); };
+#pragma unroll
+  for (int i = 0; i < RING - 1; ++i) issue(i < n_all ? row_at(i) : 0, i < n_all ? 0x7fffffff : 0, i);
+  for (int i = 0; i < n_all; ++i) {
+    const int t = row_at(i);
+    const int ahead = i + RING - 1;
+    issue(ahead < n_all ? row_at(ahead) : 0, ahead < n_all ? 0x7fffffff : 0, ahead % RING);
+    if (ASYNC && !a.direct) take(i % RING, cur);
+    else load(t, cur);
+    const bool own = i < n_rows && t >= tl.ta;
     advance(t, cur, own);
     if (own) {
       T* hr = static_cast<T*>(a.h) + long(t) * a.ldh;
@@ -232,17 +293,9 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
         }
     }
     push();
-    cur = next;
   }
   if constexpr (KMAX > 1) {
     if (first && a.write_state && K1 > 0) {
-      if (tb < tl.t1) {                                     // the sequence's last tokens lie in another tile
-        for (int t = tl.t1 - K1; t < tl.t1; ++t) {
-          load(t, cur);
-          advance(t, cur, false);
-          push();
-        }
-      }
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         const int r = i - (R - K1);
@@ -256,11 +309,112 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
   }
 }
 
-template <typename T, int VEC, int NC, bool ONE>
-int launch_k(const ResidStepArgs& a, int nt, dim3 grid, cudaStream_t s) {
+// Decode: one token per sequence, everything a CTA reads is asked for at once. A thread holds one vector of columns.
+template <typename T, int VEC, int K>
+__global__ void __launch_bounds__(1024) resid_token_kernel(const ResidStepArgs a) {
+  __shared__ float part_s[2][32];
+  const int tid = threadIdx.x, H = a.H, gs = H / a.groups;
+  const int seq = blockIdx.x / a.groups, d = (blockIdx.x % a.groups) * gs + tid * VEC;
+  const bool on = tid * VEC < gs, start = a.x_in == nullptr;
+  constexpr int K1 = K - 1;
+  float nw[VEC], pw[VEC], w[K][VEC];
+  if (on) {                                                 // weights do not depend on the launches before
+    ld_vec<VEC>(a.norm_w + d, nw);
+    if (!start) ld_vec<VEC>(a.post_w + d, pw);
+    if (a.taps) {
+#pragma unroll
+      for (int j = 0; j < K; ++j) ld_vec<VEC>(a.taps + long(j) * H + d, w[j]);
+    }
+  }
+  griddep_wait();
+  griddep_launch();
+  const int t = a.cu ? a.cu[seq] : seq;
+  if (a.cu && a.cu[seq + 1] <= t) return;
+  float* st = a.hist ? a.hist + long(a.slots[seq]) * K1 * H + d : nullptr;
+  float x[VEC], y[VEC], h[K][VEC];
+  if (on) {
+    if (start) {
+      long row = t;
+      if (a.ids) {
+        const int id = a.ids[t];
+        row = (id < 0 || id >= a.vocab) ? 0 : id;
+      }
+      ld_vec<VEC>(static_cast<const T*>(a.emb) + row * a.ld_emb + d, x);
+    } else {
+      ld_vec<VEC>(a.x_in + long(t) * H + d, x);
+      ld_vec<VEC>(static_cast<const T*>(a.y) + long(t) * a.ldy + d, y);
+    }
+    if (a.taps) {
+#pragma unroll
+      for (int j = 0; j < K1; ++j) ld_vec<VEC>(st + long(j) * H, h[j]);
+    }
+  }
+  auto inv_rms = [&](const float (&v)[VEC], float* part) {
+    float ss = 0.f;
+    if (on) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
+    }
+    ss = warp_sum_f(ss);
+    if (blockDim.x > 32) {
+      if ((tid & 31) == 0) part[tid >> 5] = ss;
+      __syncthreads();
+      ss = 0.f;
+      for (int i = 0; i < int(blockDim.x) / 32; ++i) ss += part[i];
+    }
+    return 1.f / sqrtf(ss / float(gs) + a.eps);
+  };
+  if (start) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) x[j] *= a.emb_scale;
+  } else {
+    const float inv = inv_rms(y, part_s[0]);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) x[j] += y[j] * inv * pw[j];
+  }
+  if (on) st_vec<VEC>(a.x_out + long(t) * H + d, x);
+  const float inv = inv_rms(x, part_s[1]);
+  if (!on) return;
+  float o[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) o[j] = h[K1][j] = x[j] * inv * nw[j];
+  if (a.taps) {
+#pragma unroll
+    for (int i = 0; i < K; ++i)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[i][j], h[i][j], o[j]);
+    if (a.write_state) {
+#pragma unroll
+      for (int i = 0; i < K1; ++i) st_vec<VEC>(st + long(i) * H, h[i + 1]);
+    }
+  }
+  st_vec<VEC>(static_cast<T*>(a.h) + long(t) * a.ldh + d, o);
+}
+
+template <typename T, int VEC>
+int launch_token(const ResidStepArgs& a, int nt, dim3 grid, cudaStream_t s) {
   const int K = a.taps ? a.taps_n : 1;
 #define LB_K(N)                                                                                                        \
-  if (K <= N) return launch_pdl(resid_step_kernel<T, VEC, NC, N, ONE>, grid, dim3(nt), 0, s, a) != cudaSuccess;
+  if (K == N) return launch_pdl(resid_token_kernel<T, VEC, N>, grid, dim3(nt), 0, s, a) != cudaSuccess;
+  LB_K(1) LB_K(2) LB_K(3) LB_K(4) LB_K(5)
+#undef LB_K
+  return -1;
+}
+
+template <typename T, int VEC, int NC, bool ONE>
+int launch_k(ResidStepArgs a, int nt, dim3 grid, cudaStream_t s) {
+  const int K = a.taps ? a.taps_n : 1;
+  size_t smem = VEC == 4 ? size_t(RING) * NC * nt * (16 + 4 * sizeof(T)) : 0;
+  a.direct = smem > 200 * 1024;                             // groups too wide for the ring: plain loads
+  if (a.direct) smem = 0;
+#define LB_K(N)                                                                                                        \
+  if (K <= N) {                                                                                                        \
+    auto k = resid_step_kernel<T, VEC, NC, N, ONE>;                                                                    \
+    if (smem > 40 * 1024 &&                                                                                            \
+        cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess)                \
+      return 1;                                                                                                        \
+    return launch_pdl(k, grid, dim3(nt), smem, s, a) != cudaSuccess;                                                   \
+  }
   LB_K(1) LB_K(4) LB_K(16)
 #undef LB_K
   return 1;
@@ -279,6 +433,10 @@ int dispatch(const ResidStepArgs& a, cudaStream_t s) {
   const dim3 grid(static_cast<unsigned>(tiles * a.groups));
   const int need = v4 ? gs / 4 : gs;                        // threads with one vector each
   const int nt = std::min(512, (need + 127) / 128 * 32), nc = (need + nt - 1) / nt;     // up to 4 vectors per thread
+  if (a.max_len <= 1 && need <= 1024) {
+    const int rc = v4 ? launch_token<T, 4>(a, (need + 31) / 32 * 32, grid, s) : launch_token<T, 1>(a, (need + 31) / 32 * 32, grid, s);
+    if (rc >= 0) return rc;
+  }
   if (v4) {
     if (need <= 32) return launch_k<T, 4, 1, true>(a, 32, grid, s);
     if (nt == 32) return launch_k<T, 4, 4, true>(a, 32, grid, s);
