@@ -484,7 +484,7 @@ def bench_resid(rows):
             L = T // n_seq
             cu = torch.arange(0, T + 1, L, device="cuda", dtype=torch.int32)
             slots = torch.arange(n_seq, device="cuda", dtype=torch.int32)
-            tm = timeit_graph if T <= 64 else timeit
+            tm = timeit_graph
             for name, fn, byts in (
                     (f"resid_step {H}", lambda: sm100.resid_step(x, y, w, w, 4, 1e-5, (taps, hist, cu, slots, True), max_len=L),
                      T * H * 12 + hist.numel() * 8),
@@ -533,6 +533,13 @@ def bench_diag(rows):
             print(rows[-1], flush=True)
 
 
+class Batch:
+    """The fields of a step that a planner reads."""
+
+    def __init__(self, **kw):
+        self.__dict__.update(kw)
+
+
 def bench_latent(rows):
     """Latent attention of two sizes: the pieces of a decode step and of a prompt. Attention by the bytes of the latents
     (decode) or the FLOPs of the per-head form, 2 (dim + rot + vdim) per visible pair and head (prompts)."""
@@ -555,28 +562,38 @@ def bench_latent(rows):
             cu = torch.arange(0, T + 1, q_len, device="cuda", dtype=torch.int32)
             cl = torch.full((n,), ctx, device="cuda", dtype=torch.int32)
             pairs = n * (q_len * ctx - q_len * (q_len - 1) / 2)
-            for name, fn in latent_parts(sm100, q, kv, gate, uk, uv, w, cs, pos, slots, cache, bt, cl, cu, q_len, H, dim, R, L, ctx):
+            args = (uv, w, 1e-5, cs)
+            if q_len == 1:
+                qa = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
+                fns = [("latent_attention", lambda: sm100.latent_attention(qa, cache, bt, cl, cu, 1, 0.07, L, R, max_ctx=ctx)),
+                       ("latent_decode (queries, append, attention, values, gate)", lambda: sm100.latent_decode(
+                           q, kv, gate, uk, *args, pos, slots, cache, bt, cl, cu, 0.07, H, dim, R, ctx))]
+            else:
+                part = sm100.latent_parts(Batch(cu_q=cu, ctx_lens=cl, block_table=bt, positions=pos, slots=slots, token_ids=pos,
+                                                n_seqs=n, max_q_len=q_len, max_ctx=ctx, cu_q_host=list(range(0, T + 1, q_len)),
+                                                ctx_host=[ctx] * n, latent_parts=None), page)[0]
+                rows_uk = f(H * dim, L)
+
+                def latent_space():
+                    qs = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
+                    sm100.latent_values(sm100.latent_attention(qs, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx), uv, gate)
+                fns = [("latent space, all", latent_space),
+                       ("latent_prompt (per head), all", lambda: sm100.latent_prompt(q, kv, gate, rows_uk, *args, cache, part, 0.07,
+                                                                                     H, dim, R))]
+                if R == 64:
+                    kc, vc = f(nb, page, H, dim + R), f(nb, page, H, V)
+                    qq = f(T, H, dim + R)
+                    fns.append(("prefill_attn (its attention alone)",
+                                lambda: sm100.prefill_attn(qq, kc, vc, cu, cl, bt, q_len, 0.07)))
+            for name, fn in fns:
                 ms = (timeit_graph if q_len == 1 else timeit)(fn)
                 r = dict(kernel=name, heads=H, dims=(dim, R, L, V), n_seq=n, q_len=q_len, ctx=ctx, us=round(ms * 1e3, 2), peaks=src)
-                if "attention" in name or "all" in name:
-                    if q_len == 1:
-                        r["frac_hbm"] = round(n * ctx * (L + R) * 2 / ms / 1e6 / hbm, 3)
-                    else:
-                        r["frac_tflops"] = round(2.0 * H * pairs * (dim + R + V) / ms / 1e9 / tf, 3)
+                if q_len == 1:
+                    r["frac_hbm"] = round(n * ctx * (L + R) * 2 / ms / 1e6 / hbm, 3)
+                else:
+                    r["frac_tflops"] = round(2.0 * H * pairs * (dim + R + V) / ms / 1e9 / tf, 3)
                 rows.append(r)
                 print(r, flush=True)
-
-
-def latent_parts(sm100, q, kv, gate, uk, uv, w, cs, pos, slots, cache, bt, cl, cu, q_len, H, dim, R, L, ctx):
-    qa = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
-    o = sm100.latent_attention(qa, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx)
-
-    def whole():
-        a = sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)
-        sm100.latent_values(sm100.latent_attention(a, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx), uv, gate)
-    return [("latent_queries", lambda: sm100.latent_queries(q, kv, uk, w, 1e-5, cs, pos, slots, cache, H, dim, R)),
-            ("latent_attention", lambda: sm100.latent_attention(qa, cache, bt, cl, cu, q_len, 0.07, L, R, max_ctx=ctx)),
-            ("latent_values", lambda: sm100.latent_values(o, uv, gate)), ("latent all", whole)]
 
 
 def bench_attn_sizes(rows):

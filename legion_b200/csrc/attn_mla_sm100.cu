@@ -92,6 +92,8 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 11);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
+  griddep_wait();
+  griddep_launch();
   const int seq = blockIdx.y;
   int w = blockIdx.x;
   const int split = w % a.n_splits; w /= a.n_splits;
@@ -488,8 +490,7 @@ int mla_start(const CUtensorMap& tq, const CUtensorMap& tc, const MlaArgs& a, di
     }
     attr = true;
   }
-  mla_attn_kernel<HALVES><<<grid, 192, smem, s>>>(tq, tc, a);
-  const cudaError_t e = cudaGetLastError();
+  const cudaError_t e = launch_pdl(mla_attn_kernel<HALVES>, grid, dim3(192), smem, s, tq, tc, a);
   if (e != cudaSuccess) {
     snprintf(g_mla_err, sizeof(g_mla_err), "mla attention launch: %s", cudaGetErrorString(e));
     return 1;

@@ -402,8 +402,11 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::resid_step_launch(a, f32, cur_stream()) == 0, "resid_step: width ", H, ", ", groups, " groups, ",
                 a.taps_n, " taps, ", a.tok, " tokens per block", cuda_error());
   });
+  // the cache append and the queries: rot part only (latent space rows), with uk also their way into the latent space;
+  // prompt: q_abs takes the queries themselves, [T, heads, dim + rot]
   m.def("latent_prep", [](const Tensor& q, const Tensor& kv, const Tensor& norm_w, double eps, const Tensor& cos_sin,
-                          const Tensor& positions, const Tensor& slots, Tensor& cache, Tensor& q_abs, int64_t dim, int64_t rot) {
+                          const Tensor& positions, const Tensor& slots, Tensor& cache, Tensor& q_abs, int64_t dim, int64_t rot,
+                          const OptT& uk, bool prompt) {
     const bool f32 = is_f32(q, "q");
     same(kv, f32, "kv");
     same(cache, f32, "cache");
@@ -411,10 +414,11 @@ void bind_layers(pybind11::module_& m) {
     const int64_t T = q.size(0), H = q_abs.size(1), L = norm_w.numel();
     TORCH_CHECK(q.dim() == 2 && kv.dim() == 2 && kv.size(0) == T && q.size(1) >= H * (dim + rot) && kv.size(1) >= L + rot,
                 "latent_prep: q [T, heads * (dim + rot)], kv [T, rank + rot]");
-    TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && q_abs.size(0) == T && q_abs.size(2) >= L + rot &&
-                    cache.is_contiguous() && cache.size(-1) >= L + rot, "latent_prep: rows of rank + rot columns");
+    TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && q_abs.size(0) == T &&
+                    (prompt ? q_abs.size(2) == dim + rot : q_abs.size(2) >= L + rot) && cache.is_contiguous() &&
+                    cache.size(-1) >= L + rot, "latent_prep: rows of rank + rot columns");
     f32c(norm_w, L, "norm");
-    TORCH_CHECK(cos_sin.dim() == 2, "latent_prep: table [positions, rotated columns]");
+    TORCH_CHECK(cos_sin.dim() == 2 && cos_sin.size(1) <= rot && cos_sin.size(1) % 2 == 0, "latent_prep: table [positions, rotated columns]");
     f32c(cos_sin, 0, "cos_sin");
     TORCH_CHECK(positions.scalar_type() == at::kInt && slots.scalar_type() == at::kLong && positions.numel() == T &&
                     slots.numel() == T, "latent_prep: positions int32, slots int64");
@@ -426,7 +430,60 @@ void bind_layers(pybind11::module_& m) {
     a.cache = cache.data_ptr(); a.cell = cache.size(-1); a.q_abs = q_abs.data_ptr(); a.q_row = q_abs.size(2);
     a.T = int(T); a.heads = int(H); a.dim = int(dim); a.R = int(rot); a.L = int(L);
     c10::cuda::CUDAGuard guard(q.device());
-    TORCH_CHECK(lb::latent_prep_launch(a, f32, cur_stream()) == 0, "latent_prep failed", cuda_error());
+    if (uk.has_value()) {
+      TORCH_CHECK(!f32 && !is_f32(*uk, "uk") && uk->is_contiguous() && uk->numel() == H * L * dim, "latent_prep: uk [heads * rank, dim]");
+      TORCH_CHECK(lb::latent_decode_q_launch(a, uk->data_ptr(), cur_stream()) == 0, "latent decode queries failed", cuda_error());
+    } else if (prompt) {
+      TORCH_CHECK(!f32, "latent_prep: the prompt form is bf16");
+      TORCH_CHECK(lb::latent_prompt_prep_launch(a, cur_stream()) == 0, "latent prompt queries failed", cuda_error());
+    } else {
+      TORCH_CHECK(lb::latent_prep_launch(a, f32, cur_stream()) == 0, "latent_prep failed", cuda_error());
+    }
+  });
+  m.def("latent_gather", [](const Tensor& cache, const Tensor& block_table, const Tensor& ctx_lens, const Tensor& pages,
+                            Tensor& lat, Tensor& k, int64_t dim, int64_t rot) {
+    TORCH_CHECK(!is_f32(cache, "cache") && !is_f32(lat, "lat") && !is_f32(k, "k"), "latent_gather: bf16");
+    const int64_t n = pages.size(1), L = lat.size(1), H = k.size(1);
+    TORCH_CHECK(pages.scalar_type() == at::kInt && pages.is_contiguous() && pages.size(0) == 2 && lat.is_contiguous() &&
+                    k.is_contiguous() && lat.size(0) == n * 64 && k.size(0) == n * 64 && k.size(2) == dim + rot &&
+                    cache.is_contiguous() && cache.dim() == 4 && cache.size(3) >= L + rot, "latent_gather: shapes");
+    TORCH_CHECK(block_table.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_table.stride(1) == 1,
+                "latent_gather: int32 tables");
+    lb::LatentGatherArgs a{};
+    a.cache = cache.data_ptr(); a.cell = cache.size(3); a.page = int(cache.size(1));
+    a.block_table = block_table.data_ptr<int>(); a.table_width = int(block_table.stride(0)); a.ctx_lens = ctx_lens.data_ptr<int>();
+    a.page_seq = pages.data_ptr<int>(); a.page_pos = pages.data_ptr<int>() + n;
+    a.lat = lat.data_ptr(); a.k = k.data_ptr();
+    a.pages = int(n); a.heads = int(H); a.dim = int(dim); a.R = int(rot); a.L = int(L);
+    c10::cuda::CUDAGuard guard(cache.device());
+    TORCH_CHECK(lb::latent_gather_launch(a, cur_stream()) == 0, "latent_gather failed", cuda_error());
+  });
+  m.def("latent_decode_v", [](const OptT& o_part, const OptT& ml_part, int64_t n_splits, const OptT& o_lat, const Tensor& uv,
+                              const OptT& gate, int64_t heads, int64_t L, Tensor& out) {
+    TORCH_CHECK(!is_f32(uv, "uv") && !is_f32(out, "out") && uv.is_contiguous() && uv.size(1) == L && out.is_contiguous() &&
+                    uv.size(0) % heads == 0 && out.size(1) == uv.size(0), "latent_decode_v: uv [heads * V, rank], out [T, heads * V]");
+    const int64_t T = out.size(0), V = uv.size(0) / heads;
+    lb::LatentValueArgs a{};
+    a.n_splits = int(n_splits);
+    if (n_splits > 1) {
+      TORCH_CHECK(o_part.has_value() && ml_part.has_value(), "latent_decode_v: partials");
+      f32c(*o_part, T * heads * n_splits * L, "o_part");
+      f32c(*ml_part, T * heads * n_splits * 2, "ml_part");
+      a.o_part = o_part->data_ptr<float>(); a.ml_part = ml_part->data_ptr<float>();
+    } else {
+      TORCH_CHECK(o_lat.has_value() && !is_f32(*o_lat, "o_lat") && o_lat->is_contiguous() && o_lat->numel() == T * heads * L,
+                  "latent_decode_v: o_lat [T, heads, rank]");
+      a.o_lat = o_lat->data_ptr();
+    }
+    a.uv = uv.data_ptr();
+    if (gate.has_value()) {
+      TORCH_CHECK(!is_f32(*gate, "gate") && gate->dim() == 2 && gate->size(0) == T && (gate->size(1) == heads * V || gate->size(1) == heads),
+                  "latent_decode_v: one gate per column or per head");
+      a.gate = gate->data_ptr(); a.ldg = gate->stride(0); a.per_head = gate->size(1) != heads * V;
+    }
+    a.out = out.data_ptr(); a.T = int(T); a.heads = int(heads); a.L = int(L); a.V = int(V);
+    c10::cuda::CUDAGuard guard(out.device());
+    TORCH_CHECK(lb::latent_decode_v_launch(a, cur_stream()) == 0, "latent_decode_v failed", cuda_error());
   });
   m.def("latent_attn_general", [](const Tensor& q_abs, const Tensor& cache, const Tensor& cu_q, const Tensor& ctx_lens,
                                   const Tensor& block_table, double scale, int64_t rank, int64_t rot, Tensor& out) {

@@ -58,6 +58,29 @@ struct LatentPrepArgs {
   int T, heads, dim, R, L;
 };
 int latent_prep_launch(const LatentPrepArgs& a, bool f32, cudaStream_t s);
+// Prompts in the per-head form (bf16): q_abs takes [T, heads, dim + R] with the last R columns rotated; cache as above
+int latent_prompt_prep_launch(const LatentPrepArgs& a, cudaStream_t s);
+struct LatentGatherArgs {
+  const void* cache; long cell;
+  const int* block_table; int table_width, page; const int* ctx_lens;
+  const int* page_seq; const int* page_pos;   // [pages] of 64 expanded rows: sequence and first position
+  void* lat;                       // [pages * 64, L]
+  void* k;                         // [pages * 64, heads, dim + R]; columns [dim, dim + R) are written
+  int pages, heads, dim, R, L;
+};
+int latent_gather_launch(const LatentGatherArgs& a, cudaStream_t s);
+// Decode (bf16): latent_prep and the queries' way into the latent space, uk [heads, L, dim], in one launch
+int latent_decode_q_launch(const LatentPrepArgs& a, const void* uk, cudaStream_t s);
+// Decode (bf16): merge of the key splits (n_splits > 1) or attended latents, value projection and gate
+struct LatentValueArgs {
+  const float* o_part; const float* ml_part; int n_splits;   // [T * heads, n_splits, L], [.., 2]
+  const void* o_lat;               // n_splits == 1: [T, heads, L]
+  const void* uv;                  // [heads, V, L]
+  const void* gate; long ldg; int per_head;                  // nullptr: none
+  void* out;                       // [T, heads * V]
+  int T, heads, L, V;
+};
+int latent_decode_v_launch(const LatentValueArgs& a, cudaStream_t s);
 // x[t, n] *= sigmoid(gate[t, per_head ? n / vdim : n]) in place
 int latent_gate_launch(void* x, const void* gate, long ldg, int per_head, int vdim, int N, int T, bool f32, cudaStream_t s);
 

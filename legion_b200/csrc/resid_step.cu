@@ -60,24 +60,17 @@ __device__ __forceinline__ Tile find_tile(const int* __restrict__ cu, int n_seqs
   return Tile{-1, 0, 0, 0};
 }
 
-template <typename T, int VEC, int NC, int KMAX, bool ONE_WARP>
-__global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 16 && KMAX <= 4 ? 12 : 1)
+// K: taps; 0: any number up to 16 (a.taps_n). FULL: the group is exactly VEC * NC columns per thread.
+template <typename T, int VEC, int NC, int K, bool ONE_WARP, bool FULL>
+__global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 16 && K > 0 ? 12 : 1)
     resid_step_kernel(const ResidStepArgs a) {
   __shared__ float part_s[2][16];
-  const int tid = threadIdx.x, nt = blockDim.x, H = a.H, gs = H / a.groups;
-  const int tile = blockIdx.x / a.groups, col0 = (blockIdx.x % a.groups) * gs;
-  constexpr int R = KMAX > 1 ? KMAX - 1 : 1;
-  const int K1 = KMAX > 1 ? a.taps_n - 1 : 0;
+  const int tid = threadIdx.x, nt = ONE_WARP ? 32 : blockDim.x, H = a.H, gs = FULL ? nt * NC * VEC : H / a.groups;
+  const int tile = blockIdx.x / a.groups, col0 = (blockIdx.x % a.groups) * gs + tid * VEC;
+  constexpr int R = K > 0 ? (K > 1 ? K - 1 : 1) : 15;     // rows of history in registers
+  const int K1 = K > 0 ? K - 1 : a.taps_n - 1;
   const bool start = a.x_in == nullptr;
-  // this thread's columns
-  bool on[NC];
-  int col[NC];
-#pragma unroll
-  for (int c = 0; c < NC; ++c) {
-    const int d = (c * nt + tid) * VEC;
-    on[c] = d < gs;
-    col[c] = col0 + d;
-  }
+  auto on = [&](int c) { return FULL || (c * nt + tid) * VEC < gs; };
   griddep_wait();
   griddep_launch();
   Tile tl;
@@ -91,80 +84,68 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
   if (tl.seq < 0 || tl.ta >= tl.t1) return;
   const int tb = min(tl.t1, tl.ta + a.tok);
   const float gs_inv = 1.f / float(gs);
+  const int step = nt * VEC;                              // columns between a thread's vectors
 
   // Four columns at a time: a token's rows come through a ring in shared memory, every thread copying what it reads itself
   extern __shared__ __align__(16) uint8_t ring_s[];
   constexpr bool ASYNC = VEC == 4;
   constexpr int YB = 4 * int(sizeof(T));
-  auto ring_x = [&](int stage, int c) { return ring_s + size_t((stage * NC + c) * nt + tid) * 16; };
-  auto ring_y = [&](int stage, int c) { return ring_s + size_t(RING * NC * nt) * 16 + size_t((stage * NC + c) * nt + tid) * YB; };
-  auto issue = [&](int t, int t_end, int stage) {
+  uint8_t* ring_x = ring_s + tid * 16;
+  uint8_t* ring_y = ring_s + size_t(RING * NC * nt) * 16 + tid * YB;
+  auto emb_row = [&](int t) {
+    long row = t;
+    if (a.ids) {
+      const int id = a.ids[t];
+      row = (id < 0 || id >= a.vocab) ? 0 : id;
+    }
+    return static_cast<const T*>(a.emb) + row * a.ld_emb + col0;
+  };
+  auto issue = [&](int t, bool real, int stage) {
     if constexpr (ASYNC) {
-      if (t < t_end && !a.direct) {
-        if (start) {
-          long row = t;
-          if (a.ids) {
-            const int id = a.ids[t];
-            row = (id < 0 || id >= a.vocab) ? 0 : id;
-          }
-          const T* er = static_cast<const T*>(a.emb) + row * a.ld_emb;
+      if (real && !a.direct) {
+        const T* yp = start ? emb_row(t) : static_cast<const T*>(a.y) + long(t) * a.ldy + col0;
+        uint8_t* sy = ring_y + stage * (NC * nt * YB);
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+          if (on(c)) copy_async<YB>(sy + c * (nt * YB), yp + c * step);
+        if (!start) {
+          const float* xp = a.x_in + long(t) * H + col0;
+          uint8_t* sx = ring_x + stage * (NC * nt * 16);
 #pragma unroll
           for (int c = 0; c < NC; ++c)
-            if (on[c]) copy_async<YB>(ring_y(stage, c), er + col[c]);
-        } else {
-#pragma unroll
-          for (int c = 0; c < NC; ++c)
-            if (on[c]) {
-              copy_async<YB>(ring_y(stage, c), static_cast<const T*>(a.y) + long(t) * a.ldy + col[c]);
-              copy_async<16>(ring_x(stage, c), a.x_in + long(t) * H + col[c]);
-            }
+            if (on(c)) copy_async<16>(sx + c * (nt * 16), xp + c * step);
         }
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
     }
   };
-  struct Row { float x[NC][VEC], y[NC][VEC]; };
-  auto take = [&](int stage, Row& r) {
-    if constexpr (ASYNC) {
-      asm volatile("cp.async.wait_group %0;" ::"n"(RING - 1) : "memory");
+  // the token's rows: embedding in x, or residual in x and sublayer output in y
+  float x[NC][VEC], y[NC][VEC];
+  auto take = [&](int t, int stage) {
+    const bool ring = ASYNC && !a.direct;
+    if constexpr (ASYNC) asm volatile("cp.async.wait_group %0;" ::"n"(RING - 1) : "memory");
+    const T* yp = ring ? reinterpret_cast<const T*>(ring_y + stage * (NC * nt * YB))
+                       : (start ? emb_row(t) : static_cast<const T*>(a.y) + long(t) * a.ldy + col0);
+    const int ys = ring ? nt * 4 : step;
+    if (start) {
 #pragma unroll
       for (int c = 0; c < NC; ++c)
-        if (on[c]) {
-          if (start) {
-            ld_vec<VEC>(reinterpret_cast<const T*>(ring_y(stage, c)), r.x[c]);
-          } else {
-            ld_vec<VEC>(reinterpret_cast<const T*>(ring_y(stage, c)), r.y[c]);
-            ld_vec<VEC>(reinterpret_cast<const float*>(ring_x(stage, c)), r.x[c]);
-          }
-        }
+        if (on(c)) ld_vec<VEC>(yp + c * ys, x[c]);
+      return;
     }
-  };
-  auto load = [&](int t, Row& r) {
-    const T* er = nullptr;
-    if (start) {
-      long row = t;
-      if (a.ids) {
-        const int id = a.ids[t];
-        row = (id < 0 || id >= a.vocab) ? 0 : id;
-      }
-      er = static_cast<const T*>(a.emb) + row * a.ld_emb;
-    }
+    const float* xp = ring ? reinterpret_cast<const float*>(ring_x + stage * (NC * nt * 16)) : a.x_in + long(t) * H + col0;
 #pragma unroll
     for (int c = 0; c < NC; ++c)
-      if (on[c]) {
-        if (start) {
-          ld_vec<VEC>(er + col[c], r.x[c]);
-        } else {
-          ld_vec<VEC>(static_cast<const T*>(a.y) + long(t) * a.ldy + col[c], r.y[c]);
-          ld_vec<VEC>(a.x_in + long(t) * H + col[c], r.x[c]);
-        }
+      if (on(c)) {
+        ld_vec<VEC>(yp + c * ys, y[c]);
+        ld_vec<VEC>(xp + c * ys, x[c]);
       }
   };
   auto inv_rms = [&](const float (&v)[NC][VEC], int buf) {
     float ss = 0.f;
 #pragma unroll
     for (int c = 0; c < NC; ++c)
-      if (on[c]) {
+      if (on(c)) {
 #pragma unroll
         for (int j = 0; j < VEC; ++j) ss = fmaf(v[c][j], v[c][j], ss);
       }
@@ -175,136 +156,123 @@ __global__ void __launch_bounds__(ONE_WARP ? 32 : 512, ONE_WARP && NC * VEC <= 1
       ss = 0.f;
       for (int i = 0; i < nt / 32; ++i) ss += part_s[buf][i];
     }
-    return 1.f / sqrtf(ss * gs_inv + a.eps);
+    return rsqrtf(fmaf(ss, gs_inv, a.eps));
   };
-  // n of a token; the new residual is written when the token is this tile's own
-  float n[NC][VEC];
-  auto advance = [&](int t, const Row& r, bool own) {
+  // x becomes n; the new residual is written when the token is this tile's own
+  const float* post_w = a.post_w + col0;
+  const float* norm_w = a.norm_w + col0;
+  auto advance = [&](int t, bool own) {
     if (start) {
       if constexpr (!ONE_WARP) __syncthreads();            // with one norm per token its buffer is written every time
 #pragma unroll
       for (int c = 0; c < NC; ++c)
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) n[c][j] = r.x[c][j] * a.emb_scale;
+        for (int j = 0; j < VEC; ++j) x[c][j] *= a.emb_scale;
     } else {
-      const float inv = inv_rms(r.y, 0);
+      const float inv = inv_rms(y, 0);
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
         float w[VEC];
-        if (on[c]) ld_vec<VEC>(a.post_w + col[c], w);
+        if (on(c)) ld_vec<VEC>(post_w + c * step, w);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) n[c][j] = r.x[c][j] + r.y[c][j] * inv * w[j];
+        for (int j = 0; j < VEC; ++j) x[c][j] = fmaf(y[c][j] * inv, w[j], x[c][j]);
       }
     }
     if (own) {
+      float* xo = a.x_out + long(t) * H + col0;
 #pragma unroll
       for (int c = 0; c < NC; ++c)
-        if (on[c]) st_vec<VEC>(a.x_out + long(t) * H + col[c], n[c]);
+        if (on(c)) st_vec<VEC>(xo + c * step, x[c]);
     }
-    const float inv = inv_rms(n, 1);
+    const float inv = inv_rms(x, 1);
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       float w[VEC];
-      if (on[c]) ld_vec<VEC>(a.norm_w + col[c], w);
+      if (on(c)) ld_vec<VEC>(norm_w + c * step, w);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) n[c][j] *= inv * w[j];
+      for (int j = 0; j < VEC; ++j) x[c][j] *= inv * w[j];
     }
   };
 
-  // hist[R - 1] is the row before the current token; rows older than K - 1 are not used
+  // hist[R - 1] is the row before the current token; with K == 0 rows older than K1 are not used
   float hist[R][NC][VEC];
+  auto used = [&](int i) { return K > 1 || (K == 0 && i >= R - K1); };
   auto push = [&]() {
-    if constexpr (KMAX > 1) {
-#pragma unroll
-      for (int i = 0; i + 1 < R; ++i)
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) hist[i][c][j] = hist[i + 1][c][j];
+    if constexpr (K != 1) {
 #pragma unroll
       for (int c = 0; c < NC; ++c)
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) hist[R - 1][c][j] = n[c][j];
+        for (int j = 0; j < VEC; ++j) {
+#pragma unroll
+          for (int i = 0; i + 1 < R; ++i) hist[i][c][j] = hist[i + 1][c][j];
+          hist[R - 1][c][j] = x[c][j];
+        }
     }
   };
-  float* st = (KMAX > 1 && a.hist) ? a.hist + long(a.slots[tl.seq]) * K1 * H : nullptr;
+  float* st = (K != 1 && a.hist) ? a.hist + long(a.slots[tl.seq]) * K1 * H + col0 : nullptr;
   const bool first = tl.ta == tl.t0;
-  Row cur;
-  if constexpr (KMAX > 1) {
+  if constexpr (K != 1) {
 #pragma unroll
     for (int i = 0; i < R; ++i)
 #pragma unroll
-      for (int c = 0; c < NC; ++c)
+      for (int c = 0; c < NC; ++c) {
 #pragma unroll
         for (int j = 0; j < VEC; ++j) hist[i][c][j] = 0.f;
-    if (first) {
-#pragma unroll
-      for (int i = 0; i < R; ++i) {
-        const int r = i - (R - K1);
-        if (r >= 0) {
-#pragma unroll
-          for (int c = 0; c < NC; ++c)
-            if (on[c]) ld_vec<VEC>(st + long(r) * H + col[c], hist[i][c]);
-        }
+        if (first && used(i) && on(c)) ld_vec<VEC>(st + long(i - (R - K1)) * H + c * step, hist[i][c]);
       }
-    }
   }
   const int tw = first ? tl.ta : tl.ta - K1;                // rows in front of the tile come first
   // rows [tw, tb), and behind them, where this tile owns the history, the sequence's last rows
-  const bool tail = KMAX > 1 && first && a.write_state && K1 > 0 && tb < tl.t1;
+  const bool tail = K != 1 && first && a.write_state && K1 > 0 && tb < tl.t1;
   const int n_rows = tb - tw, n_all = n_rows + (tail ? K1 : 0);
   auto row_at = [&](int i) { return i < n_rows ? tw + i : tl.t1 - K1 + (i - n_rows); };
-#pragma unroll
-  for (int i = 0; i < RING - 1; ++i) issue(i < n_all ? row_at(i) : 0, i < n_all ? 0x7fffffff : 0, i);
+#pragma unroll 1
+  for (int i = 0; i < RING - 1; ++i) issue(row_at(i), i < n_all, i);
+#pragma unroll 1
   for (int i = 0; i < n_all; ++i) {
     const int t = row_at(i);
-    const int ahead = i + RING - 1;
-    issue(ahead < n_all ? row_at(ahead) : 0, ahead < n_all ? 0x7fffffff : 0, ahead % RING);
-    if (ASYNC && !a.direct) take(i % RING, cur);
-    else load(t, cur);
+    issue(row_at(i + RING - 1), i + RING - 1 < n_all, (i + RING - 1) % RING);
+    take(t, i % RING);
     const bool own = i < n_rows && t >= tl.ta;
-    advance(t, cur, own);
+    advance(t, own);
     if (own) {
-      T* hr = static_cast<T*>(a.h) + long(t) * a.ldh;
+      T* hr = static_cast<T*>(a.h) + long(t) * a.ldh + col0;
 #pragma unroll
       for (int c = 0; c < NC; ++c)
-        if (on[c]) {
+        if (on(c)) {
           float o[VEC];
 #pragma unroll
-          for (int j = 0; j < VEC; ++j) o[j] = n[c][j];
+          for (int j = 0; j < VEC; ++j) o[j] = x[c][j];
           if (a.taps) {
+            const float* tp = a.taps + col0 + c * step;
             float w[VEC];
-            ld_vec<VEC>(a.taps + long(K1) * H + col[c], w);
+            ld_vec<VEC>(tp + long(K1) * H, w);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], n[c][j], o[j]);
-            if constexpr (KMAX > 1) {
+            for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], x[c][j], o[j]);
+            if constexpr (K != 1) {
 #pragma unroll
-              for (int i = 0; i < R; ++i) {
-                const int r = i - (R - K1);
-                if (r >= 0) {
-                  ld_vec<VEC>(a.taps + long(r) * H + col[c], w);
+              for (int i2 = 0; i2 < R; ++i2)
+                if (used(i2)) {
+                  ld_vec<VEC>(tp + long(i2 - (R - K1)) * H, w);
 #pragma unroll
-                  for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], hist[i][c][j], o[j]);
+                  for (int j = 0; j < VEC; ++j) o[j] = fmaf(w[j], hist[i2][c][j], o[j]);
                 }
-              }
             }
           }
-          st_vec<VEC>(hr + col[c], o);
+          st_vec<VEC>(hr + c * step, o);
         }
     }
     push();
   }
-  if constexpr (KMAX > 1) {
+  if constexpr (K != 1) {
     if (first && a.write_state && K1 > 0) {
 #pragma unroll
-      for (int i = 0; i < R; ++i) {
-        const int r = i - (R - K1);
-        if (r >= 0) {
+      for (int i = 0; i < R; ++i)
+        if (used(i)) {
 #pragma unroll
           for (int c = 0; c < NC; ++c)
-            if (on[c]) st_vec<VEC>(st + long(r) * H + col[c], hist[i][c]);
+            if (on(c)) st_vec<VEC>(st + long(i - (R - K1)) * H + c * step, hist[i][c]);
         }
-      }
     }
   }
 }
@@ -362,7 +330,7 @@ __global__ void __launch_bounds__(1024) resid_token_kernel(const ResidStepArgs a
       ss = 0.f;
       for (int i = 0; i < int(blockDim.x) / 32; ++i) ss += part[i];
     }
-    return 1.f / sqrtf(ss / float(gs) + a.eps);
+    return rsqrtf(fmaf(ss, 1.f / float(gs), a.eps));
   };
   if (start) {
 #pragma unroll
@@ -401,23 +369,29 @@ int launch_token(const ResidStepArgs& a, int nt, dim3 grid, cudaStream_t s) {
   return -1;
 }
 
-template <typename T, int VEC, int NC, bool ONE>
+template <typename T, int VEC, int NC, bool ONE, bool FULL = false>
 int launch_k(ResidStepArgs a, int nt, dim3 grid, cudaStream_t s) {
   const int K = a.taps ? a.taps_n : 1;
   size_t smem = VEC == 4 ? size_t(RING) * NC * nt * (16 + 4 * sizeof(T)) : 0;
   a.direct = smem > 200 * 1024;                             // groups too wide for the ring: plain loads
   if (a.direct) smem = 0;
+  if (!a.taps) a.taps_n = 1;
 #define LB_K(N)                                                                                                        \
-  if (K <= N) {                                                                                                        \
-    auto k = resid_step_kernel<T, VEC, NC, N, ONE>;                                                                    \
+  if (K == N || (N == 0 && K <= 16)) {                                                                                 \
+    auto k = resid_step_kernel<T, VEC, NC, N, ONE, FULL>;                                                              \
     if (smem > 40 * 1024 &&                                                                                            \
         cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess)                \
       return 1;                                                                                                        \
     return launch_pdl(k, grid, dim3(nt), smem, s, a) != cudaSuccess;                                                   \
   }
-  LB_K(1) LB_K(4) LB_K(16)
+  if constexpr (FULL) {
+    LB_K(1) LB_K(3) LB_K(4)
+    return launch_k<T, VEC, NC, ONE, false>(a, nt, grid, s);
+  } else {
+    LB_K(1) LB_K(4) LB_K(0)
+    return 1;
+  }
 #undef LB_K
-  return 1;
 }
 
 template <typename T>
@@ -439,7 +413,10 @@ int dispatch(const ResidStepArgs& a, cudaStream_t s) {
   }
   if (v4) {
     if (need <= 32) return launch_k<T, 4, 1, true>(a, 32, grid, s);
+    if (gs == 256) return launch_k<T, 4, 2, true, true>(a, 32, grid, s);
+    if (gs == 512) return launch_k<T, 4, 4, true, true>(a, 32, grid, s);
     if (nt == 32) return launch_k<T, 4, 4, true>(a, 32, grid, s);
+    if (nt * 16 == gs) return launch_k<T, 4, 4, false, true>(a, nt, grid, s);
     if (nc <= 4) return launch_k<T, 4, 4, false>(a, nt, grid, s);
     if (nc <= 8) return launch_k<T, 4, 8, false>(a, nt, grid, s);
   } else {

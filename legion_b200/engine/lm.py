@@ -1059,7 +1059,7 @@ class LmEngine(Engine):
             slots=torch.tensor(slots, dtype=torch.int64, device=dev),
             state_slots=torch.tensor([s.slot for s, _, _ in rows], **i32),
             logit_rows=torch.tensor(logit_rows, dtype=torch.int64, device=dev),
-            max_q_len=max(n for _, _, n in rows), max_ctx=max(ctx), write_state=write_state, cu_q_host=cu)
+            max_q_len=max(n for _, _, n in rows), max_ctx=max(ctx), write_state=write_state, cu_q_host=cu, ctx_host=ctx)
         if any(s.media is not None and s.phase != "decode" for s, _, _ in rows):
             self._media_inputs(b, rows, tok)
         if self.ring_len:
@@ -1106,7 +1106,7 @@ class LmEngine(Engine):
                       slots=torch.tensor(slots, dtype=torch.int64, device=dev),
                       state_slots=torch.tensor([s.slot for s, _, _ in items], **i32),
                       logit_rows=torch.tensor(lrows if logit_rows is None else logit_rows, dtype=torch.int64, device=dev),
-                      max_q_len=max(len(t) for _, _, t in items), max_ctx=max(ctx), cu_q_host=cu)
+                      max_q_len=max(len(t) for _, _, t in items), max_ctx=max(ctx), cu_q_host=cu, ctx_host=ctx)
         if self.ring_len:
             self._ring_inputs(b, [(s, p0, len(toks)) for s, p0, toks in items], width)
         return b

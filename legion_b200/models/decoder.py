@@ -53,6 +53,8 @@ class StepBatch:
     embeds: Optional[torch.Tensor] = None       # input rows instead of the token embedding
     capture_layers: Optional[List[int]] = None  # layer outputs to return (EAGLE-3 features)
     cu_q_host: Optional[List[int]] = None
+    ctx_host: Optional[List[int]] = None         # ctx_lens on the host
+    latent_parts: Optional[list] = None          # ops.sm100.latent_parts of this step
     decode_splits: Optional[int] = None
     replay: Optional[dict] = None                # verify steps: per-layer recurrent inputs kept for commit
     rope_table: Optional[torch.Tensor] = None    # [T, rot] per-token cos | sin rows (multi-section rotary positions of
@@ -363,6 +365,7 @@ class Decoder:
         for il in range(cfg.n_layer if cfg.layers is not None else 0):
             if cfg.layers[il].mixer.kind == "lightning":
                 self._decay[il] = torch.tensor(cfg.layers[il].mixer.decay, dtype=torch.float32, device=dev)
+        self._latent_uk: Dict[str, torch.Tensor] = {} # layer prefix -> key projection of the per-head form
         self._rot: Dict[tuple, torch.Tensor] = {}     # latent-attention layers: cos | sin table per rotation
         for il in range(cfg.n_layer if cfg.layers is not None else 0):
             if cfg.latent_spec(il) is not None:
@@ -1003,17 +1006,44 @@ class Decoder:
         return ops.linear(n, w[f"{p}.lin.out"])
 
     def _latent_mixer(self, p: str, il: int, h, b: StepBatch, kv: KvCache):
-        """Latent attention in its absorbed form: queries moved into the latent space, attention over the cached rows,
-        value projection and output gate, output projection."""
-        cfg, w, m = self.cfg, self.w, self.cfg.layers[il].mixer
-        nq, nl = m.heads * (m.dim + m.rot_dim), m.kv_rank + m.rot_dim
+        """Input projection, latent attention, output projection."""
+        w, m = self.w, self.cfg.layers[il].mixer
         proj = ops.linear(h, w[f"{p}.lat.in"])
+        if not proj.is_cuda:
+            o = self._latent_part(p, il, proj, b, kv)
+        elif b.max_q_len == 1:
+            o = self._latent_part(p, il, proj, b, kv, decode=proj.shape[0] == b.n_seqs)
+        else:
+            parts = ops.sm100.latent_parts(b, kv.page)
+            if len(parts) == 1:
+                o = self._latent_part(p, il, proj, parts[0], kv)
+            else:
+                o = torch.empty(proj.shape[0], m.heads * m.vdim, dtype=proj.dtype, device=proj.device)
+                for part in parts:
+                    o.index_copy_(0, part.rows, self._latent_part(p, il, proj.index_select(0, part.rows), part, kv))
+        return ops.linear(o, w[f"{p}.lat.o"])
+
+    def _latent_part(self, p: str, il: int, proj, b, kv: KvCache, decode: bool = False):
+        """Latent attention over ``proj`` (q | latent | key part | gate columns), the rows of a batch or of a part of one:
+        fused launches for decode rows, keys and values per head for long portions, the latent space otherwise."""
+        cfg, w, m = self.cfg, self.w, self.cfg.layers[il].mixer
+        H, L, R = m.heads, m.kv_rank, m.rot_dim
+        nq, nl = H * (m.dim + R), L + R
+        q, lat = proj[:, :nq], proj[:, nq:nq + nl]
         gate = proj[:, nq + nl:nq + nl + m.gate_width()] if m.gate != "none" else None
-        q_abs = ops.latent_queries(proj[:, :nq], proj[:, nq:nq + nl], w[f"{p}.lat.uk"], w[f"{p}.lat.norm"], cfg.rms_eps,
-                                   self.rotary_table(m.rot), b.positions, b.slots, kv.k[il], m.heads, m.dim, m.rot_dim)
-        o = ops.latent_attention(q_abs, kv.k[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, m.scale, m.kv_rank,
-                                 m.rot_dim, max_ctx=b.max_ctx or None)
-        return ops.linear(ops.latent_values(o, w[f"{p}.lat.uv"], gate), w[f"{p}.lat.o"])
+        uk, uv, norm, rot, cache = w[f"{p}.lat.uk"], w[f"{p}.lat.uv"], w[f"{p}.lat.norm"], self.rotary_table(m.rot), kv.k[il]
+        max_ctx = b.max_ctx or None
+        if decode and ops.sm100.latent_decode_ok(q, cache, H, m.dim, R, L, m.vdim):
+            return ops.sm100.latent_decode(q, lat, gate, uk, uv, norm, cfg.rms_eps, rot, b.positions, b.slots, cache,
+                                           b.block_table, b.ctx_lens, b.cu_q, m.scale, H, m.dim, R, max_ctx)
+        if isinstance(b, ops.sm100.LatentPart) and ops.sm100.latent_expand_ok(q, cache, b, H, m.dim, R, m.rot.dims, L, m.vdim):
+            rows = self._latent_uk.get(p)
+            if rows is None:          # the key projection as stored, [heads * dim, rank]
+                rows = self._latent_uk[p] = uk.view(H, L, m.dim).transpose(1, 2).reshape(H * m.dim, L).contiguous()
+            return ops.sm100.latent_prompt(q, lat, gate, rows, uv, norm, cfg.rms_eps, rot, cache, b, m.scale, H, m.dim, R)
+        q_abs = ops.latent_queries(q, lat, uk, norm, cfg.rms_eps, rot, b.positions, b.slots, cache, H, m.dim, R)
+        o = ops.latent_attention(q_abs, cache, b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, m.scale, L, R, max_ctx=max_ctx)
+        return ops.latent_values(o, uv, gate)
 
     def _rglru_mixer(self, p: str, il: int, h, b: StepBatch, st: StatePool):
         """Griffin's recurrent block. Its decode step runs convolution, gates, recurrence and the GELU branch as one

@@ -797,7 +797,8 @@ def qkv_norm_append(q, k, v, q_norm, k_norm, eps, slots, k_cache, v_cache):
 
 def head_linear(x, w2d, n_heads: int, rows_per_group: int, n_feat: int, K: int, x_group_col: int, out2d):
     """Per-head projections read and written in place: for every head h
-    ``out2d[t * n_heads + h, :n_feat] = W_h @ x[t, h * x_group_col : h * x_group_col + K]`` with
+    ``out2d[t * n_heads + h, :n_feat] = W_h @ x[t, h * x_group_col : h * x_group_col + K]`` (0: every head reads the
+    same K columns) with
     ``W_h = w2d[h * rows_per_group : h * rows_per_group + n_feat]``. One grouped launch of the tcgen05 GEMM (group =
     head); the activation tile of a head is fetched from its column slice of ``x`` by the TMA load, the output rows
     go through a row map, so nothing is transposed or copied."""
@@ -827,7 +828,7 @@ def head_linear(x, w2d, n_heads: int, rows_per_group: int, n_feat: int, K: int, 
         ws._cache[key] = tab
     tile_group, tile_tok0, tile_ntok, tile_out0, out_rows, meta, n_tiles = tab
     C.wgemm(w2d, x, out2d, None, None, out_rows, n_feat, False, 0, bn, 1, None, None, ws.status, tile_group, tile_tok0,
-            tile_ntok, meta, n_tiles, rows_per_group, 0, [], tile_out0, None, None, x_group_col, K)
+            tile_ntok, meta, n_tiles, rows_per_group, 0, [], tile_out0, None, None, x_group_col, K if x_group_col else 0)
     return out2d
 
 
@@ -879,14 +880,137 @@ def latent_tc_ok(q_abs, cache, rank: int, rot: int) -> bool:
             and q_abs.shape[2] % 8 == 0 and cache.shape[-1] % 8 == 0 and page % 8 == 0 and 64 % page == 0)
 
 
+def latent_row(rank: int, rot: int) -> int:
+    """Columns of a query row in the latent space, padded so that rows start on 16-byte boundaries."""
+    return -(-(rank + rot) // 8) * 8
+
+
 def latent_queries(q, kv, uk, norm_w, eps, cos_sin, positions, slots, cache, heads: int, dim: int, rot_dim: int):
     """Cache rows of the step's tokens and the queries in the latent space, [T, heads, rank + rot_dim] (rows padded to
     multiples of 8 columns)."""
     T, L = q.shape[0], norm_w.numel()
-    q_abs = torch.empty(T, heads, -(-(L + rot_dim) // 8) * 8, dtype=q.dtype, device=q.device)
+    q_abs = torch.empty(T, heads, latent_row(L, rot_dim), dtype=q.dtype, device=q.device)
     head_linear(q, uk, heads, L, L, dim, dim + rot_dim, q_abs.view(T * heads, -1))
-    ext().latent_prep(q, kv, norm_w, eps, cos_sin, positions, slots, cache, q_abs, dim, rot_dim)
+    ext().latent_prep(q, kv, norm_w, eps, cos_sin, positions, slots, cache, q_abs, dim, rot_dim, None, False)
     return q_abs
+
+
+LATENT_DECODE_ROWS = 64      # most rows of a step on the fused decode launches
+
+
+def latent_decode_ok(q, cache, heads: int, dim: int, rot: int, rank: int, vdim: int) -> bool:
+    """Whether a decode step runs on the fused launches around the tcgen05 latent attention."""
+    page = cache.shape[1]
+    return (q.dtype == torch.bfloat16 and q.shape[0] <= LATENT_DECODE_ROWS and rank % 8 == 0 and (rank + rot) % 8 == 0
+            and rank <= 512 and rank + rot <= 576 and dim % 4 == 0 and dim <= 256 and (dim + rot) % 4 == 0
+            and q.stride(0) % 4 == 0 and q.data_ptr() % 8 == 0 and page % 8 == 0 and 64 % page == 0)
+
+
+def latent_decode(q, kv, gate, uk, uv, norm_w, eps, cos_sin, positions, slots, cache, block_table, ctx_lens, cu_q, scale,
+                  heads: int, dim: int, rot: int, max_ctx=None):
+    """One token per sequence: queries into the latent space with the cache append | attention over the latents in key
+    splits | merge, value projection and output gate. [T, heads * vdim]."""
+    C = ext()
+    T, L, page = q.shape[0], norm_w.numel(), cache.shape[1]
+    ws = Workspace.get(q.device)
+    bf = dict(dtype=torch.bfloat16, device=q.device)
+    q_abs = torch.empty(T, heads, latent_row(L, rot), **bf)
+    C.latent_prep(q, kv, norm_w, eps, cos_sin, positions, slots, cache, q_abs, dim, rot, uk, False)
+    n = mla_splits(int(ctx_lens.numel()), 1, heads, max_ctx or block_table.shape[1] * page)
+    o_part = ml_part = o_lat = None
+    if n > 1:
+        o_part = ws.buf("mla_o", (T * heads * n * L,), torch.float32)
+        ml_part = ws.buf("mla_ml", (T * heads * n * 2,), torch.float32)
+    else:
+        o_lat = torch.empty(T, heads, L, **bf)
+    C.mla_attn(q_abs, cache, cu_q, ctx_lens, block_table, page, 1, scale, n, o_part, ml_part, o_lat, L, rot, False, ws.status)
+    out = torch.empty(T, uv.shape[0], **bf)
+    C.latent_decode_v(o_part, ml_part, n, o_lat, uv, gate, heads, L, out)
+    return out
+
+
+LATENT_EXPAND_MIN = 192      # portions from this many tokens attend in the per-head form
+LATENT_EXPAND_BYTES = 2 << 30    # ... while the expanded keys and values stay below this
+
+
+class LatentPart:
+    """Sequences of a step that run in one form of latent attention. ``rows``: their rows in the step (None: all of it)."""
+    __slots__ = ("expand", "rows", "positions", "slots", "cu_q", "ctx_lens", "block_table", "max_q_len", "max_ctx", "pages",
+                 "table")
+
+
+def latent_parts(b, page: int) -> list:
+    """Splits a step's sequences into long portions (per-head form) and the rest (latent space); kept with the batch for
+    its other layers. Without host copies of the lengths everything runs in the latent space."""
+    if b.latent_parts is not None:
+        return b.latent_parts
+    cu, ctx, dev = b.cu_q_host, b.ctx_host, b.token_ids.device
+    lens = [cu[i + 1] - cu[i] for i in range(len(cu) - 1)] if cu is not None else []
+    long = [i for i, n in enumerate(lens) if n >= LATENT_EXPAND_MIN] if ctx is not None else []
+    rest = [i for i, n in enumerate(lens) if i not in set(long) and n > 0]
+
+    def part(seqs, expand):
+        p = LatentPart()
+        p.expand, p.pages, p.table = expand, None, None
+        if len(seqs) == b.n_seqs:
+            p.rows, p.positions, p.slots, p.cu_q, p.ctx_lens, p.block_table = (None, b.positions, b.slots, b.cu_q, b.ctx_lens,
+                                                                               b.block_table)
+            p.max_q_len, p.max_ctx = b.max_q_len, b.max_ctx
+        else:
+            p.rows = torch.tensor([r for i in seqs for r in range(cu[i], cu[i + 1])], dtype=torch.int64, device=dev)
+            at = [0]
+            for i in seqs:
+                at.append(at[-1] + lens[i])
+            sel = torch.tensor(seqs, dtype=torch.int64, device=dev)
+            p.positions, p.slots = b.positions.index_select(0, p.rows), b.slots.index_select(0, p.rows)
+            p.cu_q = torch.tensor(at, dtype=torch.int32, device=dev)
+            p.ctx_lens, p.block_table = b.ctx_lens.index_select(0, sel), b.block_table.index_select(0, sel)
+            p.max_q_len = max(lens[i] for i in seqs)
+            p.max_ctx = max(ctx[i] for i in seqs) if ctx is not None else b.max_ctx
+        if expand:
+            n = [-(-ctx[i] // 64) for i in seqs]
+            p.pages = torch.tensor([[j for j, k in enumerate(n) for _ in range(k)], [64 * x for k in n for x in range(k)]],
+                                   dtype=torch.int32, device=dev)
+            t, first = torch.zeros(len(seqs), max(n), dtype=torch.int32), 0
+            for j, k in enumerate(n):
+                t[j, :k] = torch.arange(first, first + k)
+                first += k
+            p.table = t.to(dev)
+        return p
+    if not long:
+        p = part(list(range(b.n_seqs)), False)
+        parts = [p]
+    else:
+        parts = [part(long, True)] + ([part(rest, False)] if rest else [])
+    b.latent_parts = parts
+    return parts
+
+
+def latent_expand_ok(q, cache, p: LatentPart, heads: int, dim: int, rot: int, rot_cols: int, rank: int, vdim: int) -> bool:
+    return (p.expand and q.dtype == torch.bfloat16 and dim % 8 == 0 and rot % 8 == 0 and rot_cols == rot and rank % 8 == 0
+            and vdim % 8 == 0 and dim + rot <= 256 and vdim <= 256 and cache.shape[-1] % 8 == 0 and q.stride(0) % 8 == 0
+            and q.data_ptr() % 16 == 0 and p.pages.shape[1] * 64 * heads * (dim + rot + vdim) * 2 <= LATENT_EXPAND_BYTES)
+
+
+def latent_prompt(q, kv, gate, uk_rows, uv, norm_w, eps, cos_sin, cache, p: LatentPart, scale, heads: int, dim: int, rot: int):
+    """Long portions: the sequences' cached latents become keys and values of every head (one product each), attended by
+    the prefill kernel. Per visible pair that is dim + rot + vdim products instead of 2 rank + rot in the latent space.
+    ``uk_rows`` [heads * dim, rank]. [T, heads * vdim]."""
+    C = ext()
+    T, L, n = q.shape[0], norm_w.numel(), p.pages.shape[1]
+    V = uv.shape[0] // heads
+    bf = dict(dtype=torch.bfloat16, device=q.device)
+    qf = torch.empty(T, heads, dim + rot, **bf)
+    C.latent_prep(q, kv, norm_w, eps, cos_sin, p.positions, p.slots, cache, qf, dim, rot, None, True)
+    lat, k = torch.empty(n * 64, L, **bf), torch.empty(n * 64, heads, dim + rot, **bf)
+    C.latent_gather(cache, p.block_table, p.ctx_lens, p.pages, lat, k, dim, rot)
+    head_linear(lat, uk_rows, heads, dim, dim, L, 0, k.view(n * 64 * heads, dim + rot))
+    v = linear(lat, uv)
+    o = prefill_attn(qf, k.view(n, 64, heads, dim + rot), v.view(n, 64, heads, V), p.cu_q, p.ctx_lens, p.table, p.max_q_len,
+                     scale).view(T, heads * V)
+    if gate is not None:
+        C.latent_gate(o, gate, heads)
+    return o
 
 
 def latent_attention(q_abs, cache, block_table, ctx_lens, cu_q, max_q_len, scale, rank: int, rot: int, max_ctx=None):

@@ -172,7 +172,7 @@ def latent_case(H, dim, R, L, V, lens, qlens, page, device, dtype, loud=None, se
                 H=H, dim=dim, R=R, L=L, V=V)
 
 
-def latent_run(c, lens, qlens, gates, device, decode_first=False):
+def latent_run(c, lens, qlens, gates, device, append_only=False):
     """The last qlens rows of every sequence through the ops, the rows before them appended in a first call."""
     H, dim, R, L = c["H"], c["dim"], c["R"], c["L"]
     slot = lambda i, p: int(c["bt"][i, p // c["page"]]) * c["page"] + p % c["page"]                     # noqa: E731
@@ -187,6 +187,8 @@ def latent_run(c, lens, qlens, gates, device, decode_first=False):
     before = [(i, 0, n - m) for i, (n, m) in enumerate(zip(lens, qlens)) if n > m]
     if before:
         feed(before)
+    if append_only:
+        return None
     q_abs = feed([(i, n - m, n) for i, (n, m) in enumerate(zip(lens, qlens))])
     cu = i32([0] + torch.tensor(qlens).cumsum(0).tolist(), device)
     o = ops.latent_attention(q_abs, c["cache"], c["bt"], i32(lens, device), cu, max(qlens), c["scale"], L, R, max_ctx=max(lens))
@@ -241,6 +243,63 @@ def test_far_keys_at_page_and_split_borders(device, dtype, H, dim, R, L, V):
             for t in range(0, m, 13):                                       # the key decides every row that sees it
                 off = float((want[t] - far).norm() / far.norm())
                 assert off < 0.4 if p <= n - m + t else off > 0.6
+    status_ok(device)
+
+
+@gpu
+@pytest.mark.parametrize("H,dim,R,L,V", [(4, 64, 32, 128, 64), (16, 128, 64, 512, 128), (3, 40, 24, 72, 32), (5, 64, 64, 256, 96),
+                                         (2, 192, 64, 320, 256), (6, 48, 16, 136, 40)])
+@pytest.mark.parametrize("page", [64, 16])
+def test_fused_decode_and_per_head_prompts(H, dim, R, L, V, page):
+    """The fused launches of decode steps, and steps whose long portions attend with keys and values per head beside short
+    ones in the latent space; a loud key decides at page borders."""
+    device, dtype = "cuda:0", torch.bfloat16
+    bench = type("B", (), {})
+    for lens, qlens in (([200, 64, 1, 131, 65], [1] * 5), ([700, 30], [1, 1]), ([300, 64, 700, 131, 1], [300, 64, 250, 1, 1]),
+                        ([260], [200]), ([500, 193], [192, 193])):
+        for loud in (None, (0, 63), (0, lens[0] - qlens[0])):
+            c = latent_case(H, dim, R, L, V, lens, qlens, page, device, dtype, loud=loud)
+            want = latent_want(c, lens, qlens, None)
+            gates = [None, rnd(sum(qlens), H, seed=9, dtype=dtype), rnd(sum(qlens), H * V, seed=9, dtype=dtype)]
+            latent_run(c, lens, qlens, None, device, append_only=True)
+            q = torch.cat([x[1][n - m:].reshape(m, -1) for x, n, m in zip(c["seqs"], lens, qlens)]).to(device)
+            kv = torch.cat([x[0][n - m:] for x, n, m in zip(c["seqs"], lens, qlens)]).to(device)
+            uk_t = c["uk"].view(H, dim, L).transpose(1, 2).reshape(H * L, dim).contiguous().to(device)
+            uk, uv, nw = c["uk"].to(device), c["uv"].to(device), c["nw"].to(device)
+            host = [0] + torch.tensor(qlens).cumsum(0).tolist()
+            b = bench()
+            b.positions = i32([p for n, m in zip(lens, qlens) for p in range(n - m, n)], device)
+            b.slots = torch.tensor([int(c["bt"][i, p // page]) * page + p % page for i, (n, m) in enumerate(zip(lens, qlens))
+                                    for p in range(n - m, n)], device=device)
+            b.cu_q, b.ctx_lens, b.block_table, b.token_ids = i32(host, device), i32(lens, device), c["bt"], b.positions
+            b.n_seqs, b.max_q_len, b.max_ctx, b.cu_q_host, b.ctx_host, b.latent_parts = (len(lens), max(qlens), max(lens), host, lens,
+                                                                                        None)
+            for g in gates:
+                gd = None if g is None else g.to(device)
+                if max(qlens) == 1:
+                    assert ops.sm100.latent_decode_ok(q, c["cache"], H, dim, R, L, V)
+                    o = ops.sm100.latent_decode(q, kv, gd, uk_t, uv, nw, c["eps"], c["tab"], b.positions, b.slots, c["cache"],
+                                                b.block_table, b.ctx_lens, b.cu_q, c["scale"], H, dim, R, max(lens))
+                else:
+                    o = torch.zeros(sum(qlens), H * V, dtype=dtype, device=device)
+                    parts = ops.sm100.latent_parts(b, page)
+                    assert [p.expand for p in parts] == ([True, False] if min(qlens) < 192 else [True])
+                    for p in parts:
+                        sel = (lambda t: t) if p.rows is None else (lambda t: t.index_select(0, p.rows))      # noqa: E731
+                        qp, kvp, gp = sel(q), sel(kv), None if gd is None else sel(gd)
+                        if p.expand:
+                            assert ops.sm100.latent_expand_ok(qp, c["cache"], p, H, dim, R, R, L, V)
+                            r = ops.sm100.latent_prompt(qp, kvp, gp, uk, uv, nw, c["eps"], c["tab"], c["cache"], p, c["scale"], H, dim, R)
+                        else:
+                            qa = ops.latent_queries(qp, kvp, uk_t, nw, c["eps"], c["tab"], p.positions, p.slots, c["cache"], H, dim, R)
+                            r = ops.latent_values(ops.latent_attention(qa, c["cache"], p.block_table, p.ctx_lens, p.cu_q, p.max_q_len,
+                                                                       c["scale"], L, R, max_ctx=p.max_ctx), uv, gp)
+                        o = r if p.rows is None else o.index_copy_(0, p.rows, r)
+                x = want
+                if g is not None:
+                    s = oracle.sigmoid(d(g))
+                    x = (want.view(-1, H, V) * (s[:, :, None] if g.shape[1] == H else s.view(-1, H, V))).reshape(want.shape)
+                close(o, x, dtype, 2e-5, 2e-2)
     status_ok(device)
 
 
