@@ -25,7 +25,7 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
-PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan"}
+PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:
@@ -58,7 +58,7 @@ def _run(cmd: list[str]) -> str:
 # layers or several ranks launches
 CORE_TARGET = ROOT / "_C_core.so"
 CORE = {"gemm_sm100", "moe", "attn_prefill_sm100", "attn_decode_sm100", "attn_decode", "elementwise", "sampling", "spec",
-        "tmap", "conv1d", "hyper", "sgemm", "attn_general", "linear_scan", "linear_scan_sm100", "attn_mla_sm100", "resid_step", "latent_attn", "diag_scan", "bindings",
+        "tmap", "conv1d", "hyper", "sgemm", "attn_general", "linear_scan", "linear_scan_sm100", "attn_mla_sm100", "resid_step", "latent_attn", "diag_scan", "logits", "bindings",
         "bindings_layers"}
 
 

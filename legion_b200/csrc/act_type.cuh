@@ -52,6 +52,15 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 __device__ __forceinline__ float xielu_f(float z, float a, float b) {
   return z > 0.f ? z * fmaf(a, z, 0.5f) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
+// The same for results that are rounded to bf16: exp(z) - 1 - z by its series where the difference would cancel
+// (|error| < 2e-6 of it for z > -0.5), by the hardware exponential elsewhere.
+__device__ __forceinline__ float xielu_fast(float z, float a, float b) {
+  const float n = fminf(z, 0.f);
+  const float series = n * n * fmaf(n, fmaf(n, fmaf(n, fmaf(n, fmaf(n, 1.f / 5040.f, 1.f / 720.f), 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f);
+  const float e = n > -0.5f ? series : __expf(n) - 1.f - n;
+  const float p = fmaxf(z, 0.f);
+  return fmaf(a * p, p, fmaf(b, e, 0.5f * z));
+}
 __device__ __forceinline__ float warp_sum_f(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

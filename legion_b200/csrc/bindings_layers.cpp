@@ -560,4 +560,10 @@ void bind_layers(pybind11::module_& m) {
     c10::cuda::CUDAGuard guard(x.device());
     TORCH_CHECK(lb::diag_decode_launch(a, f32, cur_stream()) == 0, "diag_decode failed", cuda_error());
   });
+  m.def("softcap", [](Tensor& x, double scale, double cap) {
+    f32c(x, 0, "logits");
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::softcap_launch(x.data_ptr<float>(), float(scale), float(cap), x.numel(), cur_stream()) == 0, "softcap failed",
+                cuda_error());
+  });
 }

@@ -340,12 +340,24 @@ __global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDeco
       S[p] = *st[p];
       yv[p] = ld_f(static_cast<const T*>(r.y) + seq * r.ldy + c) + yb;
       float acc = cb;
-      for (int j = 0; j < K1; ++j) {
-        const float hv = h[j];
-        acc = fmaf(cw[j], hv, acc);
-        if (j > 0) h[j - 1] = hv;
+      if (K1 <= 4) {                                     // all loads before the first store
+        float hv[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) hv[j] = j < K1 ? h[j] : 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (j < K1) {
+            acc = fmaf(cw[j], hv[j], acc);
+            h[j] = j + 1 < K1 ? hv[(j + 1) & 3] : xv;
+          }
+      } else {
+        for (int j = 0; j < K1; ++j) {
+          const float hv = h[j];
+          acc = fmaf(cw[j], hv, acc);
+          if (j > 0) h[j - 1] = hv;
+        }
+        h[K1 - 1] = xv;
       }
-      if (K1 > 0) h[K1 - 1] = xv;
       u[p] = __bfloat162float(__float2bfloat16(fmaf(cw[K1], xv, acc)));
     }
   }
@@ -438,7 +450,8 @@ int decode_cluster_n(const DiagDecodeArgs& a, int d, cudaStream_t s) {
   const long ctas = long(a.s.W / DEC_CH) * ((a.s.n_seqs + 3) / 4);
   if (ctas <= 296) return decode_cluster<NK, 4>(a, d, s);
   if (ctas <= 592) return decode_cluster<NK, 8>(a, d, s);
-  return decode_cluster<NK, 16>(a, d, s);
+  if (ctas <= 1184) return decode_cluster<NK, 16>(a, d, s);
+  return decode_cluster<NK, 32>(a, d, s);
 }
 
 template <typename T>

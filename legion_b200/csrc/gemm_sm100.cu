@@ -588,11 +588,18 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             // Staged write-out: fp32 values go through shared memory so that every token row leaves as
             // 16-byte stores covering 256 contiguous bytes per 16 lanes (8 token rows per pass).
             const int etid = threadIdx.x - 64;  // 0..127 over the four epilogue warps
+            // output rows of this thread's passes, asked for before the first store could be in their way
+            long orows[4];
+#pragma unroll
+            for (int pass = 0; pass < 4; ++pass) {
+              const int t = c + pass * 8 + (etid >> 4);
+              orows[pass] = t < it.ntok ? (a.out_rows ? long(a.out_rows[it.out0 + t]) : long(it.out0 + t)) : -1;
+            }
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
               if (DUAL) v = gate_act(v, a.act) * u[j];
-              else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
+              else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -639,10 +646,9 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             for (int pass = 0; pass < 4; ++pass) {
               const int j = pass * 8 + (etid >> 4);
               const int t = c + j;
-              if (t < it.ntok && feat8 < a.n_feat) {
+              if (feat8 < a.n_feat) {
                 const int xrow = it.out0 + t;
-                long orow = xrow;
-                if (a.out_rows) orow = a.out_rows[xrow];
+                long orow = orows[pass];
                 if (orow >= 0) {
                   __nv_bfloat16* obase = reinterpret_cast<__nv_bfloat16*>(a.out);
                   if (a.n_out_peer > 0) {
@@ -678,11 +684,17 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
           } else if (OUT_F32 && a.vec_ok) {
             // fp32 rows leave as 16-byte stores too: a warp writes one token's 128 features, 4 token rows per pass
             const int etid = threadIdx.x - 64;
+            long orows[8];
+#pragma unroll
+            for (int pass = 0; pass < 8; ++pass) {
+              const int t = c + pass * 4 + (etid >> 5);
+              orows[pass] = t < it.ntok ? (a.out_rows ? long(a.out_rows[it.out0 + t]) : long(it.out0 + t)) : -1;
+            }
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
               if (DUAL) v = gate_act(v, a.act) * u[j];
-              else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
+              else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -692,9 +704,9 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             for (int pass = 0; pass < 8; ++pass) {
               const int j = pass * 4 + (etid >> 5);
               const int t = c + j;
-              if (t < it.ntok && feat4 < a.n_feat) {
+              if (feat4 < a.n_feat) {
                 const int xrow = it.out0 + t;
-                const long orow = a.out_rows ? a.out_rows[xrow] : xrow;
+                const long orow = orows[pass];
                 if (orow >= 0) {
                   float4 v = *reinterpret_cast<const float4*>(&stage[j * BM + f4]);
                   if (a.tok_scale) {
@@ -714,7 +726,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
                 const int xrow = it.out0 + t;
                 float v = g[j];
                 if (DUAL) v = gate_act(v, a.act) * u[j];
-                else if (a.xielu) v = xielu_f(v, xi_a, xi_b);
+                else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
                 if (a.tok_scale) v *= a.tok_scale[xrow];
                 long orow = xrow;
                 if (a.out_rows) orow = a.out_rows[xrow];

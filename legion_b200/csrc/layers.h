@@ -193,4 +193,7 @@ int conv_silu_any_launch(const void* x, long ldx, const float* w, const float* b
                          const int* cu_seq, const int* slots, int n_seqs, int T, int C, int KC, void* out, long ldo,
                          int write_state, const float* in_bias, int silu, bool f32, cudaStream_t s);
 
+// x = cap * tanh(x * scale / cap) in place (logits.cu)
+int softcap_launch(float* x, float scale, float cap, long n, cudaStream_t s);
+
 }  // namespace lb

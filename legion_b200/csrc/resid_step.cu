@@ -416,6 +416,7 @@ int dispatch(const ResidStepArgs& a, cudaStream_t s) {
     if (gs == 256) return launch_k<T, 4, 2, true, true>(a, 32, grid, s);
     if (gs == 512) return launch_k<T, 4, 4, true, true>(a, 32, grid, s);
     if (nt == 32) return launch_k<T, 4, 4, true>(a, 32, grid, s);
+    if (gs % 256 == 0 && gs <= 4096) return launch_k<T, 4, 2, false, true>(a, gs / 8, grid, s);
     if (nt * 16 == gs) return launch_k<T, 4, 4, false, true>(a, nt, grid, s);
     if (nc <= 4) return launch_k<T, 4, 4, false>(a, nt, grid, s);
     if (nc <= 8) return launch_k<T, 4, 8, false>(a, nt, grid, s);

@@ -1142,15 +1142,19 @@ class Decoder:
         table, ids = (w["tok_embd"], b.token_ids) if b.embeds is None else (b.embeds, None)
         x, h = ops.resid_start(table, ids, cfg.embed_scale, w["l0.attn_norm"], G, eps, conv(0), max_len=b.max_q_len)
         captures: Dict[int, torch.Tensor] = {}
+        rows = b.logit_rows                           # behind the last sublayer only the wanted rows are normed
         for i, (il, which) in enumerate(subs):
             p, last = f"l{il}", i + 1 == len(subs)
             terms = self._spec_mixer(p, il, h, b, kv, st) if which == "attn" else self._spec_ffn(p, il, h)
             norm_w = w["output_norm"] if last else w[f"l{subs[i + 1][0]}.{subs[i + 1][1]}_norm"]
-            x, h = ops.resid_step(x, terms[0][0], w[f"{p}.{which}_post_norm"], norm_w, G, eps,
+            y = terms[0][0]
+            if last and not b.capture_layers and rows is not None:
+                x, y, rows = x.index_select(0, rows), y.index_select(0, rows), None
+            x, h = ops.resid_step(x, y, w[f"{p}.{which}_post_norm"], norm_w, G, eps,
                                   None if last else conv(i + 1), max_len=b.max_q_len)
             if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
                 captures[il] = x
-        hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
+        hidden = h if rows is None else h.index_select(0, rows)
         out = StepOutput(hidden=hidden, captures=captures)
         if want_logits:
             out.logits = self.logits(hidden)
@@ -1476,6 +1480,8 @@ class Decoder:
 
     def _local_logits(self, hidden):
         lg = ops.linear(hidden, self.lm_head, out_dtype=torch.float32)
+        if lg.is_cuda and self.cfg.logit_softcap > 0:
+            return ops.sm100.softcap(lg, self.cfg.logit_scale, self.cfg.logit_softcap)
         if self.cfg.logit_scale != 1.0:
             lg = lg * self.cfg.logit_scale
         if self.cfg.logit_softcap > 0:

@@ -415,7 +415,7 @@ def up_act(x, w, ab):
 
 def group_rms(x, w, groups: int, eps: float):
     """RMS norm in ``groups`` equal parts of a float32 row, times w."""
-    v = x.reshape(*x.shape[:-1], groups, -1)
+    v = x.reshape(*x.shape[:-1], groups, x.shape[-1] // groups)
     return (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape) * w
 
 

@@ -1443,9 +1443,9 @@ def moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, 
     h = torch.empty(P, n_ff, dtype=x.dtype, device=x.device)
     y = torch.empty(P, H, dtype=x.dtype, device=x.device)
     C.sgemm(w_gate_up.view(E * 2 * n_ff, H), xs, h, None, None, None, n_ff, True, n_ff, GATE_ACTS[act], plan.tile_group,
-            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, 2 * n_ff, P)
+            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, 2 * n_ff, P, None)
     C.sgemm(w_down.view(E * H, n_ff), h, y, None, plan.sorted_w, plan.sorted_pair, H, False, 0, 0, plan.tile_group,
-            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, P)
+            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, P, None)
     if defer_combine:
         return PendingCombine(y, ids, 0, E, None, T, H)
     return y.view(T, k, H).sum(1, dtype=torch.float32).to(x.dtype)
@@ -1790,6 +1790,12 @@ def group_norm_gate(y, gate, w, eps, groups: int = 1, out=None):
     return out
 
 
+def softcap(logits, scale: float, cap: float):
+    """cap * tanh(logits * scale / cap) in place, float32."""
+    ext().softcap(logits, float(scale), float(cap))
+    return logits
+
+
 def resid_tokens(rows: int, max_len: int, width: int, groups: int) -> int:
     """Tokens per CTA of ``resid_step``: as few as give one wave of CTAs (about 12 warps per SM, a warp per 512 columns of
     a group), so that the rows recomputed in front of a tile cost little in long runs and short ones still fill the SMs."""
@@ -1812,6 +1818,8 @@ def resid_step(x, y, post_w, norm_w, groups: int, eps: float, conv=None, start=N
         h = torch.empty(T, table.shape[1], dtype=table.dtype, device=table.device)
     taps, hist, cu, slots, write = conv if conv is not None else (None, None, None, None, False)
     rows = xo.shape[0]
+    if rows == 0:
+        return xo, h
     max_len = rows if max_len is None else max_len
     tok = 1
     if taps is not None:
