@@ -8,6 +8,7 @@ what changed.  Run ``python -m legion_b200.build_ext`` (add ``-v`` for ptxas res
 from __future__ import annotations
 
 import hashlib
+import json
 import os
 import subprocess
 import sys
@@ -25,7 +26,7 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
-PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits"}
+PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:
@@ -54,27 +55,46 @@ def _run(cmd: list[str]) -> str:
     return p.stdout + p.stderr
 
 
-# the kernels of bf16 / fp32 layer stacks on one GPU: what a model without quantised weights, Gated DeltaNet
-# layers or several ranks launches
+# A checkout that has not been built compiles only the kernels of the model it is asked to run (bf16 / fp32 on one GPU):
+# those every model launches, and those of its layer kinds. The binding files name all kernels; the subset is linked and
+# loaded with lazy binding, so the absent ones do not matter until something calls them.
 CORE_TARGET = ROOT / "_C_core.so"
-CORE = {"gemm_sm100", "moe", "attn_prefill_sm100", "attn_decode_sm100", "attn_decode", "elementwise", "sampling", "spec",
-        "tmap", "conv1d", "hyper", "sgemm", "attn_general", "linear_scan", "linear_scan_sm100", "attn_mla_sm100", "resid_step", "latent_attn", "diag_scan", "logits", "bindings",
-        "bindings_layers"}
+CORE = {"gemm_sm100", "sgemm", "elementwise", "sampling", "spec", "tmap", "logits", "bindings", "bindings_layers"}
+_ATTN = {"attn_prefill_sm100", "attn_decode_sm100", "attn_decode", "attn_general"}
+_SCAN = {"linear_scan", "linear_scan_sm100", "conv1d", "conv_any"}
+KIND_KERNELS = {
+    "attn": _ATTN, "lightning": _SCAN, "ssd": _SCAN, "parallel": _ATTN | _SCAN,
+    "latent": {"attn_mla_sm100", "latent_attn", "attn_prefill_sm100", "attn_decode", "attn_general"},
+    "rglru": {"diag_scan", "conv1d", "conv_any"},
+}
 
 
-def build_core(verbose: bool = False) -> Path:
-    """The subset ``CORE`` as ``legion_b200/_C_core.so``, for a checkout that has not been built: a tool that runs one
-    such model compiles only its kernels. ``ops.sm100.ext`` takes it when ``_C.so`` is absent."""
-    return build(verbose, core=True)
+def kernels_of(cfg) -> set:
+    """Source files (without suffix) a ``ModelConfig`` needs beside ``CORE``."""
+    if cfg.layers is None:
+        return _ATTN | {"moe", "attn_mla_sm100"}
+    need = set().union(*(KIND_KERNELS[x.mixer.kind] for x in cfg.layers)) | {"resid_step" if cfg.sandwich_norm else "hyper"}
+    return need | {"moe"} if cfg.n_expert else need
 
 
-def build(verbose: bool = False, force: bool = False, core: bool = False) -> Path:
+def build_core(cfg, verbose: bool = False) -> Path:
+    """The kernels of ``cfg``, beside those of models built before, as ``legion_b200/_C_core.so``. ``ops.sm100.ext`` takes
+    it when ``_C.so`` is absent."""
+    stamp = BUILD / "core.json"
+    have = set(json.loads(stamp.read_text())) if stamp.exists() else set()
+    need = have | kernels_of(cfg)
+    out = build(verbose, core=CORE | need, force_link=need != have)
+    stamp.write_text(json.dumps(sorted(need)))
+    return out
+
+
+def build(verbose: bool = False, force: bool = False, core: set = frozenset(), force_link: bool = False) -> Path:
     import torch
     from torch.utils import cpp_extension
 
     BUILD.mkdir(parents=True, exist_ok=True)
-    cu_files = [f for f in sorted(CSRC.glob("*.cu")) if not core or f.stem in CORE]
-    cpp_files = [f for f in sorted(CSRC.glob("*.cpp")) if not core or f.stem in CORE]
+    cu_files = [f for f in sorted(CSRC.glob("*.cu")) if not core or f.stem in core]
+    cpp_files = [f for f in sorted(CSRC.glob("*.cpp")) if not core or f.stem in core]
     target, module = (CORE_TARGET, "_C_core") if core else (TARGET, "_C")
     inc = [f"-I{p}" for p in cpp_extension.include_paths()] + [f"-I{sysconfig.get_paths()['include']}"]
     cuda_home = os.environ.get("CUDA_HOME", "/usr/local/cuda")
@@ -116,11 +136,11 @@ def build(verbose: bool = False, force: bool = False, core: bool = False) -> Pat
             o.unlink()
 
     newest = max(o.stat().st_mtime for o in objs)
-    if force or jobs or not target.exists() or target.stat().st_mtime < newest:
+    if force or force_link or jobs or not target.exists() or target.stat().st_mtime < newest:
         torch_lib = Path(torch.__file__).parent / "lib"
         link = ["g++", "-shared", "-o", str(target), *map(str, objs), f"-L{torch_lib}", f"-L{cuda_home}/lib64",
                 "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-ltorch_python", "-lcudart",
-                f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda_home}/lib64"]
+                f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda_home}/lib64"] + (["-Wl,-z,lazy"] if core else [])
         _run(link)
         print(f"[build_ext] linked {target}", file=sys.stderr)
     return target

@@ -24,18 +24,20 @@ def add_arguments(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
 
 
-def ensure_built() -> None:
-    """Brings the extension up to date; a checkout that was never built compiles the core kernels only."""
+def ensure_built(model: str) -> None:
+    """Brings the extension up to date; a checkout that was never built compiles the kernels of this model only."""
     from .. import build_ext
     if build_ext.TARGET.exists():
         build_ext.build()
-    else:
-        build_ext.build_core()
+        return
+    from ..loaders.hf_map import config_from_hf
+    with open(os.path.join(model, "config.json")) as f:
+        build_ext.build_core(config_from_hf(json.load(f)))
 
 
 def run(a) -> int:
     import torch
-    ensure_built()
+    ensure_built(a.model)
     from ..engine.replay import TraceReplay, replay_engine
     torch.backends.cuda.matmul.allow_tf32 = False
     replay = TraceReplay(replay_engine(a.model, getattr(torch, a.dtype), a.max_tokens))

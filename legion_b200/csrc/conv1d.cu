@@ -1,5 +1,5 @@
 // Causal depth-wise convolution + SiLU with carried history, bf16 activations, 2 to 8 taps (the recurrent layers' short
-// convolution; fp32 activations and other tap counts: linear_scan.cu).
+// convolution; fp32 activations and other tap counts: conv_any.cu).
 //
 // Counterpart in the reference: src/cuda/fused.cu (conv_silu_kernel).
 #include "common.cuh"

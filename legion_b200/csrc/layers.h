@@ -188,7 +188,7 @@ int ssd_decode_launch(const SsdDecodeArgs& a, bool f32, cudaStream_t s);
 int group_norm_gate_launch(const void* y, long ldy, const void* gate, long ldg, const float* w, float eps, int groups,
                            int C, int rows, void* out, long ldo, bool f32, cudaStream_t s);
 
-// Causal depth-wise convolution (+ silu) with carried history, any number of taps; in_bias is added to x first
+// Causal depth-wise convolution (+ silu) with carried history, any number of taps (conv_any.cu); in_bias is added to x first
 int conv_silu_any_launch(const void* x, long ldx, const float* w, const float* bias, float* conv_state,
                          const int* cu_seq, const int* slots, int n_seqs, int T, int C, int KC, void* out, long ldo,
                          int write_state, const float* in_bias, int silu, bool f32, cudaStream_t s);

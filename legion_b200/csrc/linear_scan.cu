@@ -2,8 +2,8 @@
 //   S_t = a_t S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t        (S: N x P, fp32, kept transposed as [P, N])
 // Two forms share the kernels: a constant decay per head with silu on q, k and v (Lightning attention), and the
 // selective form a_t = exp(dt_t A), v scaled by dt_t = softplus(raw + bias), skip D v and gate silu(z) (Mamba-2).
-// Beside it: the one-launch decode step of a Mamba-2 mixer, the norms that follow the state (whole row or equal parts,
-// optional sigmoid gate) and the short convolution for any number of taps.
+// Beside it: the one-launch decode step of a Mamba-2 mixer and the norms that follow the state (whole row or equal parts,
+// optional sigmoid gate).
 //
 // The scan kernel owns 32 state rows (value columns) of one head per CTA: a warp holds four rows across its lanes, so
 // a decode step streams the state once with 128-byte accesses, and a portion of several tokens keeps it in registers.
@@ -265,69 +265,6 @@ int group_norm_t(const void* y, long ldy, const void* gate, long ldg, const floa
                     ldo) != cudaSuccess;
 }
 
-// ---------------------------------------------------------------------------------------------------------------
-template <typename T>
-__global__ void __launch_bounds__(128) conv_silu_any_kernel(const T* __restrict__ x, long ldx, const float* __restrict__ w,
-                                                            const float* __restrict__ bias,
-                                                            const float* __restrict__ conv_state,
-                                                            const int* __restrict__ cu, const int* __restrict__ slots,
-                                                            int n_seqs, int C, int KC, T* __restrict__ out, long ldo,
-                                                            const float* __restrict__ in_bias, int silu) {
-  griddep_wait();
-  griddep_launch();
-  const int c = blockIdx.x * 128 + threadIdx.x, t = blockIdx.y;
-  if (c >= C) return;
-  int lo = 0, hi = n_seqs;
-  while (hi - lo > 1) {
-    const int m = (lo + hi) >> 1;
-    if (cu[m] <= t) lo = m; else hi = m;
-  }
-  const int t0 = cu[lo];
-  const float* st = conv_state + (long(slots[lo]) * C + c) * (KC - 1);
-  float acc = bias ? bias[c] : 0.f;
-  const float ib = in_bias ? in_bias[c] : 0.f;
-  for (int j = 0; j < KC; ++j) {
-    const int s = t - (KC - 1) + j;
-    const float v = s >= t0 ? ld_f(x + long(s) * ldx + c) + ib : st[(KC - 1) + (s - t0)];
-    acc = fmaf(w[long(c) * KC + j], v, acc);
-  }
-  st_f(out + long(t) * ldo + c, silu ? silu_f(acc) : acc);
-}
-
-// history update: reads of the old history happen in the kernel before (stream order)
-template <typename T>
-__global__ void __launch_bounds__(128) conv_history_kernel(const T* __restrict__ x, long ldx, float* conv_state,
-                                                           const int* __restrict__ cu, const int* __restrict__ slots,
-                                                           int C, int KC, const float* __restrict__ in_bias) {
-  griddep_wait();
-  griddep_launch();
-  const int c = blockIdx.x * 128 + threadIdx.x, seq = blockIdx.y;
-  if (c >= C) return;
-  const int t0 = cu[seq], t1 = cu[seq + 1];
-  if (t1 <= t0) return;
-  float* st = conv_state + (long(slots[seq]) * C + c) * (KC - 1);
-  for (int j = 0; j < KC - 1; ++j) {           // position j takes what was j + n places later: never read after written
-    const int s = t1 - (KC - 1) + j;
-    st[j] = s >= t0 ? ld_f(x + long(s) * ldx + c) + (in_bias ? in_bias[c] : 0.f) : st[(KC - 1) + (s - t0)];
-  }
-}
-
-template <typename T>
-int conv_t(const void* x, long ldx, const float* w, const float* bias, float* conv_state, const int* cu, const int* slots,
-           int n_seqs, int T_, int C, int KC, void* out, long ldo, int write_state, const float* in_bias, int silu,
-           cudaStream_t s) {
-  if (T_ > 65535) return 1;
-  const int cb = (C + 127) / 128;
-  if (launch_pdl(conv_silu_any_kernel<T>, dim3(cb, T_), dim3(128), 0, s, static_cast<const T*>(x), ldx, w, bias,
-                 static_cast<const float*>(conv_state), cu, slots, n_seqs, C, KC, static_cast<T*>(out), ldo, in_bias,
-                 silu) != cudaSuccess)
-    return 1;
-  if (write_state && KC > 1)
-    return launch_pdl(conv_history_kernel<T>, dim3(cb, n_seqs), dim3(128), 0, s, static_cast<const T*>(x), ldx, conv_state,
-                      cu, slots, C, KC, in_bias) != cudaSuccess;
-  return 0;
-}
-
 }  // namespace
 
 int linear_scan_launch(const LinScanArgs& a, bool f32, cudaStream_t s) {
@@ -348,17 +285,6 @@ int group_norm_gate_launch(const void* y, long ldy, const void* gate, long ldg, 
   if (groups <= 0 || C % groups) return 1;
   return f32 ? group_norm_t<float>(y, ldy, gate, ldg, w, eps, groups, C, rows, out, ldo, s)
              : group_norm_t<__nv_bfloat16>(y, ldy, gate, ldg, w, eps, groups, C, rows, out, ldo, s);
-}
-
-int conv_silu_any_launch(const void* x, long ldx, const float* w, const float* bias, float* conv_state,
-                         const int* cu_seq, const int* slots, int n_seqs, int T, int C, int KC, void* out, long ldo,
-                         int write_state, const float* in_bias, int silu, bool f32, cudaStream_t s) {
-  if (n_seqs <= 0 || T <= 0) return 0;
-  if (KC < 1) return 1;
-  return f32 ? conv_t<float>(x, ldx, w, bias, conv_state, cu_seq, slots, n_seqs, T, C, KC, out, ldo, write_state, in_bias,
-                             silu, s)
-             : conv_t<__nv_bfloat16>(x, ldx, w, bias, conv_state, cu_seq, slots, n_seqs, T, C, KC, out, ldo, write_state,
-                                     in_bias, silu, s);
 }
 
 }  // namespace lb

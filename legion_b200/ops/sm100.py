@@ -97,11 +97,18 @@ def ext():
 
 
 def _import_ext():
-    """The full extension ``_C``, or the subset ``_C_core`` in a checkout where only that one was built."""
+    """The full extension ``_C``, or the subset ``_C_core`` in a checkout where only that one was built (its absent kernels
+    stay unresolved)."""
+    import sys
     from importlib.util import find_spec
     name = "legion_b200._C"
     if find_spec(name) is None and find_spec("legion_b200._C_core") is not None:
-        name = "legion_b200._C_core"
+        flags = sys.getdlopenflags()
+        sys.setdlopenflags(os.RTLD_LAZY)
+        try:
+            return importlib.import_module("legion_b200._C_core")
+        finally:
+            sys.setdlopenflags(flags)
     return importlib.import_module(name)
 
 
