@@ -293,30 +293,36 @@ __global__ void __launch_bounds__(256) diag_decode_kernel(const DiagDecodeArgs a
 // The same step for bf16 and blocks of 32 to 256 channels (multiples of 32): the d / 32 CTAs of a block form a cluster.
 // Each evaluates u of its own 32 channels - so it owns their history - and hands it to the others through distributed
 // shared memory; its gate weights are on the way before the launch in front of this one has finished.
-// SEQ sequences per CTA, four at a time through the products.
+// SEQ sequences per CTA, eight at a time through the products, which run on mma.sync (u is rounded to bf16 anyway): four
+// tiles of 16 of the CTA's 64 gate rows, each shared by two warps that take half of the columns.
+__device__ __forceinline__ void mma_16x8x16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
 template <int NK, int SEQ>
 __global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDecodeArgs a, const int d) {
   constexpr int PER = (SEQ * DEC_CH + 255) / 256;        // (sequence, channel) pairs per thread: sequence q + 8 p
-  __shared__ float u_s[SEQ][256];
-  __shared__ float z_s[2][SEQ][DEC_CH];
+  constexpr int KS = 4 * NK;                             // steps of 16 columns per warp, at most
+  constexpr int PITCH = 128 * NK + 8;                    // so that the eight rows of a fragment lie in different banks
+  constexpr int ROWS = SEQ < 8 ? 8 : SEQ;
+  __shared__ __align__(16) __nv_bfloat16 u_s[ROWS][PITCH];
+  __shared__ float z_s[2][2 * DEC_CH][ROWS + 1];         // column half, gate row, sequence
   using T = __nv_bfloat16;
   const DiagScanArgs& r = a.s;
   const int parts = d / DEC_CH, b = blockIdx.x / parts, part = blockIdx.x % parts;
   const int s0 = blockIdx.y * SEQ, ns = min(SEQ, r.n_seqs - s0);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
   asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
-  // warp w multiplies rows 8 w .. 8 w + 7 of the 2 x 32 gate rows of this CTA's channels; a lane holds 4 columns of every 128
   const T* gw = static_cast<const T*>(a.gates_w) + long(b) * 2 * d * d;
-  uint2 w[8][NK];
+  const int half = d / 2, k0 = (warp >> 2) * half, row0 = (warp & 3) * 16;
+  uint32_t w[KS][4];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const int row = warp * 8 + i;
-    const T* wr = gw + (long(row / DEC_CH) * d + part * DEC_CH + row % DEC_CH) * d;
+  for (int i = 0; i < 4; ++i) {                          // fragment i: rows + 8 for odd i, columns + 8 for i >= 2
+    const int row = row0 + g4 + (i & 1) * 8;
+    const T* wr = gw + (long(row / DEC_CH) * d + part * DEC_CH + row % DEC_CH) * d + k0 + (i >> 1) * 8 + 2 * t4;
 #pragma unroll
-    for (int n = 0; n < NK; ++n) {
-      const int k = n * 128 + lane * 4;
-      w[i][n] = k < d ? *reinterpret_cast<const uint2*>(wr + k) : make_uint2(0u, 0u);
-    }
+    for (int n = 0; n < KS; ++n) w[n][i] = n * 16 < half ? *reinterpret_cast<const uint32_t*>(wr + n * 16) : 0u;
   }
   const int c = b * d + part * DEC_CH + lane, K1 = a.KC - 1;
   const Chan g = gate_of(c, d);
@@ -364,59 +370,41 @@ __global__ void __launch_bounds__(256) diag_decode_cluster_kernel(const DiagDeco
   asm volatile("barrier.cluster.wait.aligned;" ::: "memory");        // every CTA of the cluster has started
 #pragma unroll
   for (int p = 0; p < PER; ++p) {
-    const int q = warp + 8 * p;
-    if (q < SEQ) {
+    const int q = warp + 8 * p;                          // rows past the last sequence hold zeros
+    const uint32_t two = pack_bf16x2(u[p], __shfl_down_sync(0xffffffffu, u[p], 1));
+    if (q < ROWS && !(lane & 1)) {
       const uint32_t local = smem_u32(&u_s[q][part * DEC_CH + lane]);
       for (int k = 0; k < parts; ++k) {
         uint32_t remote;
         asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(k));
-        asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(u[p]) : "memory");
+        asm volatile("st.shared::cluster.u32 [%0], %1;" ::"r"(remote), "r"(two) : "memory");
       }
     }
   }
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-#pragma unroll 1
-  for (int q0 = 0; q0 < ns; q0 += 4) {
-    float v[32];
 #pragma unroll
-    for (int i = 0; i < 32; ++i) v[i] = 0.f;
+  for (int q0 = 0; q0 < ROWS; q0 += 8) {
+    if (q0 >= ns) break;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const T* ub = &u_s[q0 + g4][k0 + 2 * t4];
 #pragma unroll
-    for (int n = 0; n < NK; ++n) {
-      const int k = n * 128 + lane * 4;
-      if (k < d) {
-        float4 uu[4];
-#pragma unroll
-        for (int s = 0; s < 4; ++s) uu[s] = *reinterpret_cast<const float4*>(&u_s[q0 + s][k]);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float2 w0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].x));
-          const float2 w1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i][n].y));
-#pragma unroll
-          for (int s = 0; s < 4; ++s)
-            v[i * 4 + s] = fmaf(w0.x, uu[s].x, fmaf(w0.y, uu[s].y, fmaf(w1.x, uu[s].z, fmaf(w1.y, uu[s].w, v[i * 4 + s]))));
-        }
-      }
-    }
-    // sum over the lanes: lane l ends up with value l (row l / 4, sequence l % 4)
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const bool up = lane & o;
-#pragma unroll
-      for (int i = 0; i < o; ++i) {
-        const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
-        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-      }
-    }
-    const int row = warp * 8 + lane / 4;
-    z_s[row / DEC_CH][q0 + lane % 4][row % DEC_CH] = v[0];
+    for (int n = 0; n < KS; ++n)
+      if (n * 16 < half)
+        mma_16x8x16(acc, w[n], *reinterpret_cast<const uint32_t*>(ub + n * 16), *reinterpret_cast<const uint32_t*>(ub + n * 16 + 8));
+    float (*z)[ROWS + 1] = z_s[warp >> 2];
+    z[row0 + g4][q0 + 2 * t4] = acc[0];
+    z[row0 + g4][q0 + 2 * t4 + 1] = acc[1];
+    z[row0 + g4 + 8][q0 + 2 * t4] = acc[2];
+    z[row0 + g4 + 8][q0 + 2 * t4 + 1] = acc[3];
   }
   __syncthreads();
 #pragma unroll
   for (int p = 0; p < PER; ++p) {
     const int q = warp + 8 * p;
     if (q < ns) {
-      const float2 ab = recur_terms<T>(z_s[0][q][lane] + br, z_s[1][q][lane] + bi, u[p], ld);
+      const float zr = z_s[0][lane][q] + z_s[1][lane][q], zi = z_s[0][DEC_CH + lane][q] + z_s[1][DEC_CH + lane][q];
+      const float2 ab = recur_terms<T>(zr + br, zi + bi, u[p], ld);
       const float Sn = fmaf(ab.x, S[p], ab.y);
       *st[p] = Sn;
       st_f(static_cast<T*>(r.out) + (s0 + q) * r.ldo + c, Sn * gelu_branch<T>(yv[p]));
@@ -447,10 +435,9 @@ int decode_cluster(const DiagDecodeArgs& a, int d, cudaStream_t s) {
 template <int NK>
 int decode_cluster_n(const DiagDecodeArgs& a, int d, cudaStream_t s) {
   // as many sequences per CTA as leave about one wave of two CTAs per SM
-  const long ctas = long(a.s.W / DEC_CH) * ((a.s.n_seqs + 3) / 4);
-  if (ctas <= 296) return decode_cluster<NK, 4>(a, d, s);
-  if (ctas <= 592) return decode_cluster<NK, 8>(a, d, s);
-  if (ctas <= 1184) return decode_cluster<NK, 16>(a, d, s);
+  const long ctas = long(a.s.W / DEC_CH) * ((a.s.n_seqs + 7) / 8);
+  if (ctas <= 296) return decode_cluster<NK, 8>(a, d, s);
+  if (ctas <= 592) return decode_cluster<NK, 16>(a, d, s);
   return decode_cluster<NK, 32>(a, d, s);
 }
 

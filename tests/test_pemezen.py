@@ -72,6 +72,15 @@ def test_registry_and_config_round_trip():
     assert c.conv_inputs(0) == ["attn"]
 
 
+def test_fresh_checkouts_compile_the_kernels_of_the_model_only():
+    from legion_b200 import build_ext
+    for name in ("tiny-pemezen", "tiny-nisasun", "tiny-dense"):
+        need = build_ext.CORE | build_ext.kernels_of(PRESETS[name]())
+        assert all(any((build_ext.CSRC / (k + x)).exists() for x in (".cu", ".cpp")) for k in need)
+    mine = build_ext.kernels_of(PRESETS["tiny-pemezen"]())
+    assert {"latent_attn", "diag_scan", "resid_step"} <= mine and not mine & {"moe", "hyper", "linear_scan", "gdn"}
+
+
 @pytest.mark.parametrize("name", list(pc.CASES))
 def test_loader_maps_every_tensor(models, name):
     cfg, w, path = models[name]

@@ -323,7 +323,8 @@ def lru_weights(W, blocks, K, dtype):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("W,blocks,K", [(96, 3, 4), (640, 5, 4), (21, 1, 1), (35, 35, 3), (512, 1, 2), (90, 2, 9), (256, 2, 4)])
+@pytest.mark.parametrize("W,blocks,K", [(96, 3, 4), (640, 5, 4), (21, 1, 1), (35, 35, 3), (512, 1, 2), (90, 2, 9), (256, 2, 4), (512, 2, 4),
+                                        (192, 3, 7)])
 def test_gated_recurrence_prompts_portions_and_decode(device, dtype, W, blocks, K):
     """Convolution, gates, recurrence and GELU branch; every portion size, states of other slots untouched."""
     w, dd = lru_weights(W, blocks, K, dtype), W // blocks
@@ -367,6 +368,35 @@ def test_gated_recurrence_prompts_portions_and_decode(device, dtype, W, blocks, 
             close(state[slots[i]], want[i][1], dtype, 2e-5, 1.5e-2)
         assert bool((state[[0, 3]] == 9.0).all()) and bool((conv[[0, 3]] == 9.0).all()), name
     status_ok(device)
+
+
+@gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("W,blocks,n", [(2560, 10, 64), (1280, 5, 70), (640, 20, 9), (256, 1, 17), (96, 1, 33)])
+def test_gated_recurrence_decode_of_many_sequences(dtype, W, blocks, n):
+    """One token of each of n sequences from random histories and states, in slots in no order."""
+    device, K = "cuda:0", 4
+    w, dd = lru_weights(W, blocks, K, dtype), W // blocks
+    conv, state = rnd(n + 3, W, K - 1, seed=31), rnd(n + 3, W, seed=32)
+    x, y = rnd(n, W, seed=33, dtype=dtype), rnd(n, W, seed=34, dtype=dtype)
+    slots = torch.randperm(n + 3, generator=torch.Generator().manual_seed(35))[:n]
+    win = torch.cat([d(conv)[slots], (d(x) + d(w["in_b"]))[:, :, None]], 2)
+    u = (win * d(w["conv_w"])).sum(2) + d(w["conv_b"])
+    u = u.bfloat16().double() if dtype == torch.bfloat16 else u
+    r, i = (oracle.sigmoid(oracle.block_product(u, d(w[k]), d(w[k + "_b"]))) for k in ("ra", "ri"))
+    S = torch.stack([oracle.gated_recurrence(u[j:j + 1], r[j:j + 1], i[j:j + 1], d(w["lam"]), d(state)[slots[j]])[1] for j in range(n)])
+    g = {k: v.to(device) for k, v in w.items()}
+    gw = torch.stack([g["ra"], g["ri"]], 1).reshape(-1, dd).contiguous()
+    gb = torch.stack([g["ra_b"], g["ri_b"]], 1).reshape(-1).contiguous()
+    ld = (-8 * torch.nn.functional.softplus(g["lam"].double())).float()
+    cv, st = conv.to(device), state.to(device)
+    o = ops.sm100.rglru_decode(x.to(device), g["in_b"], g["conv_w"], g["conv_b"], cv, gw, gb, ld, y.to(device), g["y_b"], st,
+                               i32(list(range(n + 1)), device), slots.int().to(device), blocks)
+    close(o, S * oracle.gelu_tanh(d(y) + d(w["y_b"])), dtype, 2e-5, 1.5e-2)
+    close(st[slots.to(device)], S, dtype, 2e-5, 1.5e-2)
+    close(cv[slots.to(device)], win[:, :, 1:], torch.float32, 1e-6)
+    rest = [j for j in range(n + 3) if j not in set(slots.tolist())]
+    assert torch.equal(st[rest].cpu(), state[rest]) and torch.equal(cv[rest].cpu(), conv[rest])
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
