@@ -605,12 +605,12 @@ def _pemezen(n_layer: int, hidden: int, heads: int, ff: int, rank: int, rot: int
     """Two recurrent layers, then a latent-attention layer, in turn; gates per column and per head in turn."""
     layers = []
     for il in range(n_layer):
-        mixer = (LatentSpec(heads, 128, rot, 128, rank, (128 + rot) ** -0.5, RotarySpec(rot, 5e5, 4.0, 8192),
+        mixer = (LatentSpec(heads, 128, rot, 128, rank, (128 + rot) ** -0.5, RotarySpec(rot, 1e6, 8.0, 8192),
                             "channel" if il % 2 else "head")
                  if il % 3 == 2 else RgLruSpec(hidden * 5 // 4, hidden // 256 * 5 // 4, 4))
         layers.append(LayerSpec(mixer, DenseSpec(ff, "xielu")))
     return ModelConfig(arch="pemezen", hidden=hidden, vocab=65536, rms_eps=1e-5, sandwich_norm=True, norm_groups=4,
-                       input_conv=4, embed_scale=3.0, logit_softcap=15.0, layers=layers)
+                       input_conv=4, embed_scale=2.0, logit_softcap=20.0, layers=layers)
 
 
 def pemezen_1b() -> ModelConfig:

@@ -119,7 +119,7 @@ def test_residual_step_without_writing_the_history(device, dtype):
 
 # ------------------------------------------------------------------------------------------- rotation
 @pytest.mark.parametrize("dims,base,factor,original,fast,slow", [
-    (32, 5e5, 4.0, 1024, 32.0, 1.0), (16, 2e4, 8.0, 4096, 32.0, 1.0), (64, 1e4, 40.0, 4096, 32.0, 1.0), (2, 1e4, 2.0, 64, 8.0, 2.0),
+    (40, 3e5, 6.0, 2048, 24.0, 1.5), (20, 7e4, 8.0, 4096, 32.0, 1.0), (64, 1e4, 40.0, 4096, 32.0, 1.0), (2, 1e4, 2.0, 64, 8.0, 2.0),
     (8, 1e4, 1.0, 100, 32.0, 1.0), (24, 100.0, 3.0, 10, 32.0, 1.0), (24, 100.0, 3.0, 2, 32.0, 1.0), (12, 30.0, 0.5, 10 ** 7, 4.0, 2.0)])
 def test_rotation_frequencies(dims, base, factor, original, fast, slow):
     """The table of a rotation with YaRN scaling, also where the ramp's ends meet or cross."""
@@ -211,7 +211,7 @@ def latent_want(c, lens, qlens, gates):
     return torch.cat(out)
 
 
-SIZES = [(4, 64, 32, 128, 64), (16, 128, 64, 512, 128), (3, 40, 24, 72, 32), (1, 13, 6, 19, 11), (6, 48, 16, 136, 40),
+SIZES = [(4, 96, 32, 128, 80), (16, 128, 64, 512, 128), (3, 40, 24, 72, 32), (1, 13, 6, 19, 11), (6, 48, 16, 136, 40),
          (70, 16, 8, 64, 8), (5, 64, 64, 256, 96), (2, 32, 8, 320, 24), (128, 8, 16, 48, 16), (9, 24, 40, 504, 16)]
 
 
@@ -229,7 +229,7 @@ def test_latent_attention_prompts_and_decode(device, dtype, H, dim, R, L, V, pag
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("H,dim,R,L,V", [(4, 64, 32, 128, 64), (3, 128, 64, 512, 128), (3, 40, 24, 72, 32)])
+@pytest.mark.parametrize("H,dim,R,L,V", [(4, 96, 32, 128, 80), (3, 128, 64, 512, 128), (3, 40, 24, 72, 32)])
 def test_far_keys_at_page_and_split_borders(device, dtype, H, dim, R, L, V):
     """One key that outshines hundreds, at every border of pages and key splits: seen from prompts and from decode rows,
     and not seen by the rows in front of it."""
@@ -247,7 +247,7 @@ def test_far_keys_at_page_and_split_borders(device, dtype, H, dim, R, L, V):
 
 
 @gpu
-@pytest.mark.parametrize("H,dim,R,L,V", [(4, 64, 32, 128, 64), (16, 128, 64, 512, 128), (3, 40, 24, 72, 32), (5, 64, 64, 256, 96),
+@pytest.mark.parametrize("H,dim,R,L,V", [(4, 96, 32, 128, 80), (16, 128, 64, 512, 128), (3, 40, 24, 72, 32), (5, 64, 64, 256, 96),
                                          (2, 192, 64, 320, 256), (6, 48, 16, 136, 40)])
 @pytest.mark.parametrize("page", [64, 16])
 def test_fused_decode_and_per_head_prompts(H, dim, R, L, V, page):
@@ -305,11 +305,11 @@ def test_fused_decode_and_per_head_prompts(H, dim, R, L, V, page):
 
 @pytest.mark.parametrize("device,dtype", WHERE)
 def test_padding_rows_leave_the_cache_alone(device, dtype):
-    c = latent_case(4, 64, 32, 128, 64, [70], [1], 64, device, dtype)
+    c = latent_case(4, 96, 32, 128, 80, [70], [1], 64, device, dtype)
     before = c["cache"].clone()
     q, kv = c["seqs"][0][1].reshape(70, -1)[:2].to(device), c["seqs"][0][0][:2].to(device)
-    ops.latent_queries(q, kv, rnd(4 * 128, 64, dtype=dtype, device=device), c["nw"].to(device), 1e-5, c["tab"], i32([0, 0], device),
-                       torch.tensor([-1, -1], device=device), c["cache"], 4, 64, 32)
+    ops.latent_queries(q, kv, rnd(4 * 128, 96, dtype=dtype, device=device), c["nw"].to(device), 1e-5, c["tab"], i32([0, 0], device),
+                       torch.tensor([-1, -1], device=device), c["cache"], 4, 96, 32)
     assert torch.equal(before, c["cache"])
 
 
