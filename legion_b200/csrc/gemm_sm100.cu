@@ -121,7 +121,10 @@ __device__ __forceinline__ float gate_act(float v, int act) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
 }
 
-template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false>
+// XIELU: the output passes xIELU with the two numbers of WgemmArgs::xielu. A variant of its own, as is the lookahead of
+// output rows for wide token tiles: decode-sized launches run the epilogue once, and code they skip still costs them
+// instruction fetches.
+template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false, bool XIELU = false>
 __global__ void __launch_bounds__(WFP4 ? 448 : 192, 1)
 wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
              const __grid_constant__ CUtensorMap tmS, const WgemmArgs a) {
@@ -548,7 +551,6 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
       }
 
       if (finalize) {
-        const float xi_a = (!DUAL && a.xielu) ? a.xielu[0] : 0.f, xi_b = (!DUAL && a.xielu) ? a.xielu[1] : 0.f;
         const float* wsb = a.split_k > 1 ? a.ws + size_t(it.tile_id) * a.split_k * (Cfg::ACC_COLS * BM) : nullptr;
 #pragma unroll 1
         for (int c = 0; c < BN; c += 32) {
@@ -584,22 +586,28 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               if (DUAL) u[j] *= gs1;
             }
           }
+          if constexpr (XIELU) {
+            const float xi_a = a.xielu[0], xi_b = a.xielu[1];
+#pragma unroll
+            for (int j = 0; j < 32; ++j) g[j] = xielu_fast(g[j], xi_a, xi_b);
+          }
           if (!OUT_F32 && a.vec_ok) {
             // Staged write-out: fp32 values go through shared memory so that every token row leaves as
             // 16-byte stores covering 256 contiguous bytes per 16 lanes (8 token rows per pass).
             const int etid = threadIdx.x - 64;  // 0..127 over the four epilogue warps
             // output rows of this thread's passes, asked for before the first store could be in their way
             long orows[4];
+            if constexpr (BN > 32) {
 #pragma unroll
-            for (int pass = 0; pass < 4; ++pass) {
-              const int t = c + pass * 8 + (etid >> 4);
-              orows[pass] = t < it.ntok ? (a.out_rows ? long(a.out_rows[it.out0 + t]) : long(it.out0 + t)) : -1;
+              for (int pass = 0; pass < 4; ++pass) {
+                const int t = c + pass * 8 + (etid >> 4);
+                orows[pass] = t < it.ntok ? (a.out_rows ? long(a.out_rows[it.out0 + t]) : long(it.out0 + t)) : -1;
+              }
             }
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
               if (DUAL) v = gate_act(v, a.act) * u[j];
-              else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -646,9 +654,11 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             for (int pass = 0; pass < 4; ++pass) {
               const int j = pass * 8 + (etid >> 4);
               const int t = c + j;
-              if (feat8 < a.n_feat) {
+              if (t < it.ntok && feat8 < a.n_feat) {
                 const int xrow = it.out0 + t;
-                long orow = orows[pass];
+                long orow = xrow;
+                if constexpr (BN > 32) orow = orows[pass];
+                else if (a.out_rows) orow = a.out_rows[xrow];
                 if (orow >= 0) {
                   __nv_bfloat16* obase = reinterpret_cast<__nv_bfloat16*>(a.out);
                   if (a.n_out_peer > 0) {
@@ -681,7 +691,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               }
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
-          } else if (OUT_F32 && a.vec_ok) {
+          } else if (OUT_F32 && BN > 32 && a.vec_ok) {      // (few tokens: plain stores of what there is)
             // fp32 rows leave as 16-byte stores too: a warp writes one token's 128 features, 4 token rows per pass
             const int etid = threadIdx.x - 64;
             long orows[8];
@@ -694,7 +704,6 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             for (int j = 0; j < 32; ++j) {
               float v = g[j];
               if (DUAL) v = gate_act(v, a.act) * u[j];
-              else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
               stage[j * BM + row] = v;
             }
             asm volatile("bar.sync 2, 128;" ::: "memory");
@@ -726,7 +735,6 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
                 const int xrow = it.out0 + t;
                 float v = g[j];
                 if (DUAL) v = gate_act(v, a.act) * u[j];
-                else if (a.xielu) v = xielu_fast(v, xi_a, xi_b);
                 if (a.tok_scale) v *= a.tok_scale[xrow];
                 long orow = xrow;
                 if (a.out_rows) orow = a.out_rows[xrow];
@@ -820,11 +828,11 @@ namespace {
 
 thread_local char g_gemm_err[512];
 
-template <int BN, bool DUAL, bool OUT_F32, bool WFP4 = false, bool WFP8 = false>
+template <int BN, bool DUAL, bool OUT_F32, bool WFP4 = false, bool WFP8 = false, bool XIELU = false>
 int launch(const CUtensorMap* tmW, const CUtensorMap* tmX, const CUtensorMap* tmS, const WgemmArgs& a, int grid,
            cudaStream_t stream) {
   using Cfg = WgemmCfg<BN, DUAL, WFP4, WFP8>;
-  auto kfn = wgemm_kernel<BN, DUAL, OUT_F32, WFP4, WFP8>;
+  auto kfn = wgemm_kernel<BN, DUAL, OUT_F32, WFP4, WFP8, XIELU>;
   static bool attr_set = false;  // per instantiation
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
@@ -942,6 +950,10 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
       h.n_out_peer == 0)
     a.vec_ok = 1;
   if (h.q8_out) a.vec_ok = 1;     // the encoded rows always leave through the staged write-out
+  if (h.xielu && (h.dual || fp4 || fp8 || h.out_f32)) {
+    snprintf(g_gemm_err, sizeof(g_gemm_err), "wgemm: xIELU comes with bf16 weights and bf16 output, one weight tile");
+    return 1;
+  }
   const int num_kb = fp8 ? h.K / 128 : (h.K + BK - 1) / BK;
   if (a.split_k > num_kb) a.split_k = num_kb;
   while (a.split_k > 1 && (a.split_k - 1) * ((num_kb + a.split_k - 1) / a.split_k) >= num_kb) --a.split_k;
@@ -959,6 +971,9 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
     if (fp4) return launch<BN_, DUAL_, false, true>(tmW, tmX, tmS, a, grid, stream);            \
     if (fp8) {                                                                                  \
       if constexpr (BN_ <= 64) return launch<BN_, DUAL_, false, false, true>(tmW, tmX, tmS, a, grid, stream); \
+    }                                                                                           \
+    if constexpr (!DUAL_) {                                                                     \
+      if (h.xielu) return launch<BN_, false, false, false, false, true>(tmW, tmX, tmS, a, grid, stream); \
     }                                                                                           \
     return h.out_f32 ? launch<BN_, DUAL_, true>(tmW, tmX, tmS, a, grid, stream)                 \
                      : launch<BN_, DUAL_, false>(tmW, tmX, tmS, a, grid, stream);               \
