@@ -17,15 +17,25 @@ from typing import List, Optional
 # --------------------------------------------------------------------------------------------------
 @dataclass
 class AttnSpec:
-    """Grouped-query softmax attention without rotation; values may have a head size of their own."""
+    """Grouped-query softmax attention; values may have a head size of their own. Between projection and scores, all
+    optional and in this order: a bias, a short causal convolution per channel of q, k and v, a norm of q and k, rotation."""
     heads: int
     kv_heads: int
     dim: int                           # query / key head size
     vdim: int                          # value head size
     scale: float                       # multiplies the scores
     window: int = 0                    # tokens a position sees, itself included (0 = all)
-    qk_norm: bool = True               # per-head RMS norm of q and k with a plain weight
+    qk_norm: bool = True               # RMS norm of q and k with a plain weight
+    norm_over: str = "head"            # each head by itself | all: the whole of q (of k) at once, a weight per column
+    bias: bool = False                 # of the q, k and v projections
+    conv: int = 0                      # taps of the short convolution (0: none)
+    rot: Optional["RotarySpec"] = None
+    softcap: float = 0.0               # cap * tanh(score / cap)
     kind: str = "attn"
+
+    def direct(self) -> bool:
+        """Whether q, k and v come straight from the projection, up to head norms."""
+        return not (self.conv or self.rot or self.bias or (self.qk_norm and self.norm_over != "head"))
 
 
 @dataclass
@@ -62,15 +72,20 @@ class ParallelSpec:
 
 @dataclass
 class RotarySpec:
-    """Rotation of the first ``dims`` columns of a vector, neighbouring columns in pairs. ``original`` > 0: YaRN
+    """Rotation of the first ``dims`` columns of a vector. ``original`` > 0 stretches the low frequencies: ``yarn``
     (frequencies divided by ``factor`` along a ramp between the pairs that turn ``fast`` and ``slow`` times over the
-    original context; cos and sin grow by 0.1 ln(factor) + 1)."""
+    original context; cos and sin grow by 0.1 ln(factor) + 1) or ``llama3`` (wavelengths above original / low divided by
+    ``factor``, those below original / high kept, a blend between)."""
     dims: int
     base: float
     factor: float = 1.0
     original: float = 0.0
     fast: float = 32.0
     slow: float = 1.0
+    scaling: str = "yarn"
+    low: float = 1.0
+    high: float = 4.0
+    layout: str = "pairs"              # neighbouring columns | half: column i with column i + dims / 2
     kind: str = "rotary"
 
 
@@ -102,6 +117,42 @@ class RgLruSpec:
 
 
 @dataclass
+class ChannelDeltaSpec:
+    """Gated delta rule with a decay per head and key channel: q, k and v behind a short convolution and silu, unit q and
+    k per head, decay and output gate from low-rank projections, an RMS norm per head in front of the gate."""
+    heads: int
+    kv_heads: int                      # q / k heads, each shared by heads / kv_heads state heads
+    dim: int                           # query / key head size
+    vdim: int
+    conv: int = 4                      # taps
+    rank: int = 8                      # width of the low-rank projections (the wider one, a multiple of 8)
+    kind: str = "channel_delta"
+
+    def in_columns(self) -> dict:
+        """First column of each part of the stacked input projection, and its width (``end``). The low-rank parts start on
+        16-byte boundaries."""
+        up8 = lambda n: -(-n // 8) * 8                               # noqa: E731
+        k = self.kv_heads * self.dim
+        b = 2 * k + self.heads * self.vdim
+        a1 = up8(b + self.heads)
+        return {"q": 0, "k": k, "v": 2 * k, "b": b, "a1": a1, "g1": a1 + self.rank, "end": a1 + 2 * self.rank}
+
+
+@dataclass
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row with the same weights; each pass begins with a projection of
+    [stream, embedding output] and has caches and states of its own."""
+    start: int
+    stop: int
+    times: int
+    kind: str = "loop"
+
+    def expand(self, layers: list) -> list:
+        """One entry per layer run."""
+        return layers[:self.start] + layers[self.start:self.stop] * self.times + layers[self.stop:]
+
+
+@dataclass
 class DenseSpec:
     ff: int
     act: str = "silu"                  # xielu: un-gated, with two learned numbers per layer
@@ -119,11 +170,22 @@ class MoeSpec:
     act: str = "silu"
     router: str = "softmax"            # softmax | sigmoid | softmax_bias (selection by softmax score + correction)
     correction: bool = False
-    renorm: bool = True
+    renorm: object = True              # chosen weights divided by their sum (held away from zero); "sum": by the plain sum
+    scale: float = 1.0                 # ... and multiplied by this
     n_group: int = 1                   # groups of neighbouring experts, the best keep_group of them stay open
     keep_group: int = 1
     group_top: int = 2                 # a group's score sums this many of its best selection scores
+    shared_ff: int = 0                 # width of the shared expert (0: none)
+    shared_gate: bool = False          # its output times the sigmoid of one more row of the router projection
     kind: str = "moe"
+
+    def gated(self) -> bool:
+        return self.act != "relu2"
+
+    def shared_slots(self) -> int:
+        """Un-gated experts add up over parts of their width, so the shared expert is stored as this many more experts of
+        width ``ff`` (the last one padded with zeros) behind the routed ones."""
+        return -(-self.shared_ff // self.ff)
 
 
 @dataclass
@@ -133,7 +195,8 @@ class LayerSpec:
 
 
 _SPECS = {c.__dataclass_fields__["kind"].default: c
-          for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, RotarySpec, LatentSpec, RgLruSpec, DenseSpec, MoeSpec)}
+          for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, RotarySpec, LatentSpec, RgLruSpec, ChannelDeltaSpec, LoopSpec,
+                    DenseSpec, MoeSpec)}
 
 
 def spec_from(d):
@@ -254,6 +317,10 @@ class ModelConfig:
     # channel of ``input_conv`` taps (0: none)
     norm_groups: int = 1
     input_conv: int = 0
+    # with ``layers``, one stream and no sandwich norms: pre-norm layers on one fp32 residual, x + residual_mult * f(norm(x))
+    residual_mult: float = 1.0
+    embed_norm: bool = False           # the embedding rows pass the model's norm first
+    loop: Optional[LoopSpec] = None    # ``layers`` then has one entry per layer run (``LoopSpec.expand``)
     # multi-token prediction
     mtp_layers: int = 0
     # weights
@@ -262,7 +329,7 @@ class ModelConfig:
 
     def __post_init__(self):
         if self.layers is not None:
-            self.layers = [spec_from(x) for x in self.layers]
+            self.layers, self.loop = [spec_from(x) for x in self.layers], spec_from(self.loop)
             self.n_layer = len(self.layers)
             self.layer_kinds = [x.mixer.kind for x in self.layers]
             attn = [a for a in (self.attn_spec(il) for il in range(self.n_layer)) if a is not None]
@@ -304,7 +371,37 @@ class ModelConfig:
     def recurrent_spec(self, il: int):
         """The part of layer il that carries a recurrent state, of a stack with specifications."""
         m = self.layers[il].mixer
-        return m if isinstance(m, (LightningSpec, SsdSpec, RgLruSpec)) else (m.right if isinstance(m, ParallelSpec) else None)
+        if isinstance(m, (LightningSpec, SsdSpec, RgLruSpec, ChannelDeltaSpec)):
+            return m
+        return m.right if isinstance(m, ParallelSpec) else None
+
+    def attn_history(self, il: int):
+        """(channels, tokens) of the projected q, k and v that the short convolution of an attention layer keeps, or None."""
+        a = self.attn_spec(il)
+        if a is None or a.conv < 2:
+            return None
+        return (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim, a.conv - 1
+
+    def state_floats(self, il: int) -> int:
+        """float32 numbers of recurrent state (without convolution histories) per sequence of layer il."""
+        r = self.recurrent_spec(il)
+        if r is None:
+            return 0
+        return r.width if r.kind == "rglru" else r.heads * r.vdim * (r.state if r.kind == "ssd" else r.dim)
+
+    # layer runs of a looped stack: caches and states belong to a run, weights to a layer
+    def weight_layer(self, il: int) -> int:
+        """Index of the weights of layer run il."""
+        lo = self.loop
+        if lo is None or il < lo.start:
+            return il
+        n = lo.stop - lo.start
+        return lo.start + (il - lo.start) % n if il < lo.start + n * lo.times else il - n * (lo.times - 1)
+
+    def begins_pass(self, il: int) -> bool:
+        lo = self.loop
+        n = 0 if lo is None else lo.stop - lo.start
+        return n > 0 and lo.start <= il < lo.start + n * lo.times and (il - lo.start) % n == 0
 
     def conv_inputs(self, il: int) -> List[str]:
         """Sublayers of layer il whose input passes a short convolution (``input_conv``)."""
@@ -327,7 +424,8 @@ class ModelConfig:
     def recurrent_layers(self) -> List[int]:
         """Layers that carry a state from token to token besides the KV cache."""
         if self.layers is not None:
-            return [i for i in range(self.n_layer) if self.recurrent_spec(i) is not None or self.conv_inputs(i)]
+            return [i for i in range(self.n_layer) if self.recurrent_spec(i) is not None or self.conv_inputs(i)
+                    or self.attn_history(i) is not None]
         return [i for i, k in enumerate(self.layer_kinds) if k in ("gdn", "mamba2", "kda")]
 
     def kv_dims(self, il: int):

@@ -109,13 +109,13 @@ def model_bytes_per_step(cfg, n_seqs: int, ctx: int, tp: int = 1, dtype_bytes: i
         for name, shp in layer_weight_shapes(cfg, il).items():
             if len(shp) == 2 and not name.endswith(("conv_w", "st_mix")):
                 dense += shp[0] * shp[1]
-        a, r, f = cfg.attn_spec(il), cfg.recurrent_spec(il), cfg.layers[il].mlp
+        a, f = cfg.attn_spec(il), cfg.layers[il].mlp
         if a is not None:
             kv += a.kv_heads * (a.dim + a.vdim) * (min(ctx, a.window) if a.window else ctx) * n_seqs
-        if r is not None:                                               # fp32 state, read and written
-            kv += r.heads * r.vdim * (r.dim if r.kind == "lightning" else r.state) * 4 * n_seqs
+        kv += cfg.state_floats(il) * 4 * n_seqs                         # fp32 state, read and written
         if f is not None and f.kind == "moe":
-            experts += f.experts * (1.0 - (1.0 - f.top / f.experts) ** n_seqs) * 3 * H * f.ff
+            experts += f.experts * (1.0 - (1.0 - f.top / f.experts) ** n_seqs) * (3 if f.gated() else 2) * H * f.ff
+            dense += 2 * H * f.shared_ff
     for il, kind in enumerate(cfg.layer_kinds if cfg.layers is None else []):
         if kind in ("attn", "swa", "nope"):
             qw = cfg.n_head * cfg.head_dim * (2 if cfg.gated_attn else 1)

@@ -17,6 +17,7 @@ Blocks (reference structure in parentheses):
   lightning   linear attention with a constant decay per head (stacks with layer specifications)
   latent      latent attention of a layer specification: own sizes, YaRN rotation, output gate
   rglru       short convolution and a real-gated linear recurrent unit beside a GELU branch
+  channel_delta  gated delta rule with a decay per key channel, low-rank decay and gate projections
   parallel    two mixers over the same input, here windowed attention beside a Mamba-2 mixer
   moe         router -> top-k -> routed experts (+ shared expert, + sigmoid shared gate)
               (``src/model/core.rs:4496-4640``); dense SwiGLU / GELU / ReLU^2 FFN
@@ -166,7 +167,14 @@ class StatePool:
                 for which in cfg.conv_inputs(il):       # last inputs of a sublayer's input convolution, oldest first
                     self.conv[il, which] = torch.zeros(n_slots, cfg.input_conv - 1, cfg.hidden, device=device,
                                                        dtype=torch.float32)
+                if cfg.attn_history(il) is not None:            # projected q | k | v in front of the short convolution
+                    self.conv[il] = torch.zeros(n_slots, *cfg.attn_history(il), device=device, dtype=torch.float32)
                 if r is None:
+                    continue
+                if r.kind == "channel_delta":
+                    self.ssm[il] = torch.zeros(n_slots, r.heads, r.vdim, r.dim, device=device, dtype=torch.float32)
+                    self.conv[il] = torch.zeros(n_slots, 2 * r.kv_heads * r.dim + r.heads * r.vdim, r.conv - 1, device=device,
+                                                dtype=torch.float32)
                     continue
                 if r.kind == "rglru":
                     self.ssm[il] = torch.zeros(n_slots, r.width, device=device, dtype=torch.float32)
@@ -366,10 +374,15 @@ class Decoder:
             if cfg.layers[il].mixer.kind == "lightning":
                 self._decay[il] = torch.tensor(cfg.layers[il].mixer.decay, dtype=torch.float32, device=dev)
         self._latent_uk: Dict[str, torch.Tensor] = {} # layer prefix -> key projection of the per-head form
-        self._rot: Dict[tuple, torch.Tensor] = {}     # latent-attention layers: cos | sin table per rotation
+        self._shared_down: Dict[str, torch.Tensor] = {}   # layer prefix -> shared expert's down projection as one matrix
+        self._logit_rows: Optional[torch.Tensor] = None   # logit scale, one per row
+        self._rot: Dict[tuple, torch.Tensor] = {}     # layers with a rotation of their own: cos | sin table per rotation
         for il in range(cfg.n_layer if cfg.layers is not None else 0):
             if cfg.latent_spec(il) is not None:
                 self.rotary_table(cfg.latent_spec(il).rot, mp)
+            a = cfg.attn_spec(il)
+            if a is not None and a.rot is not None:
+                self.rotary_table(a.rot, mp)
         tp = self.pctx.tp
         self.n_head_l = cfg.n_head // tp
         self.n_kv_l = max(1, cfg.n_kv_head // tp)
@@ -382,11 +395,16 @@ class Decoder:
 
     def rotary_table(self, r, max_position: int = 0) -> torch.Tensor:
         """[positions, dims] cos | sin rows of a ``config.RotarySpec``."""
-        key = (r.dims, r.base, r.factor, r.original, r.fast, r.slow)
+        key = (r.dims, r.base, r.factor, r.original, r.fast, r.slow, r.scaling, r.low, r.high)
         if key not in self._rot:
-            yarn = dict(type="yarn", factor=r.factor, original_max_position_embeddings=r.original, beta_fast=r.fast,
-                        beta_slow=r.slow, attention_factor=0.1 * math.log(r.factor) + 1.0) if r.original > 0 else None
-            self._rot[key] = ops.reference.rope_cos_sin(max_position, r.dims, r.base, yarn, device=self.device)
+            scaling = None
+            if r.original > 0 and r.scaling == "llama3":
+                scaling = dict(type="llama3", factor=r.factor, original_max_position_embeddings=r.original,
+                               low_freq_factor=r.low, high_freq_factor=r.high)
+            elif r.original > 0:
+                scaling = dict(type="yarn", factor=r.factor, original_max_position_embeddings=r.original, beta_fast=r.fast,
+                               beta_slow=r.slow, attention_factor=0.1 * math.log(r.factor) + 1.0)
+            self._rot[key] = ops.reference.rope_cos_sin(max_position, r.dims, r.base, scaling, device=self.device)
         return self._rot[key]
 
     def offload_experts(self, n_slots: int, profile: Optional[dict] = None, ssd_dir: Optional[str] = None,
@@ -964,15 +982,23 @@ class Decoder:
         return out
 
     # ------------------------------------------------------------------ stacks with layer specifications
-    def _softmax_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache):
+    def _softmax_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache, st: StatePool):
         """Attention part of a layer; ``proj`` starts with its q | k | v columns. Returns (output, columns used)."""
         cfg, w, a = self.cfg, self.w, self.cfg.attn_spec(il)
         nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
-        q = ops.qkv_norm_append(proj[:, :nq], proj[:, nq:nq + nk], proj[:, nq + nk:nq + nk + nv],
-                                w.get(f"{p}.attn.q_norm"), w.get(f"{p}.attn.k_norm"), cfg.rms_eps, b.slots, kv.k[il],
-                                kv.v[il])
+        if a.direct():
+            q = ops.qkv_norm_append(proj[:, :nq], proj[:, nq:nq + nk], proj[:, nq + nk:nq + nk + nv],
+                                    w.get(f"{p}.attn.q_norm"), w.get(f"{p}.attn.k_norm"), cfg.rms_eps, b.slots, kv.k[il],
+                                    kv.v[il])
+        else:
+            q = ops.qkv_conv_append(proj[:, :nq + nk + nv], w.get(f"{p}.attn.in_b"), w.get(f"{p}.attn.conv_w"),
+                                    st.conv[il] if a.conv > 1 else None, b.cu_q, b.state_slots, w.get(f"{p}.attn.q_norm"),
+                                    w.get(f"{p}.attn.k_norm"), a.norm_over, cfg.rms_eps,
+                                    self.rotary_table(a.rot) if a.rot is not None else None,
+                                    a.rot.layout if a.rot is not None else "half", b.positions, b.slots, kv.k[il], kv.v[il],
+                                    a.heads, write_state=b.write_state, max_len=b.max_q_len)
         o = ops.paged_attention(q, kv.k[il], kv.v[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, a.scale,
-                                window=a.window, max_ctx=b.max_ctx or None)
+                                window=a.window, max_ctx=b.max_ctx or None, softcap=a.softcap)
         return ops.linear(o.reshape(o.shape[0], -1), w[f"{p}.attn.o"]), nq + nk + nv
 
     def _ssd_mixer(self, p: str, il: int, proj, b: StepBatch, st: StatePool):
@@ -1066,6 +1092,22 @@ class Decoder:
                                  cu_host=b.cu_q_host)
         return ops.linear(s, w[f"{p}.lru.out"])
 
+    def _channel_delta_mixer(self, p: str, il: int, h, b: StepBatch, st: StatePool):
+        """Decode steps run convolution, decays, delta rule, norm and gate as one launch behind the projections."""
+        cfg, w, m = self.cfg, self.w, self.cfg.layers[il].mixer
+        col, nk, nv = m.in_columns(), m.heads * m.dim, m.heads * m.vdim
+        proj = ops.linear(h, w[f"{p}.cd.in"])
+        a_raw, gate = ops.low_rank_pair(proj[:, col["a1"]:col["end"]], w[f"{p}.cd.low"], nk, m.rank)
+        qkv, b_raw = proj[:, :col["b"]], proj[:, col["b"]:col["b"] + m.heads]
+        args = (qkv, w[f"{p}.cd.conv_w"], st.conv[il], a_raw, w[f"{p}.cd.A"], w[f"{p}.cd.dt_bias"], b_raw, st.ssm[il], b.cu_q,
+                b.state_slots, m.heads, m.kv_heads, m.dim, m.vdim)
+        if proj.is_cuda and b.max_q_len == 1 and b.write_state and proj.shape[0] == b.n_seqs:
+            n = ops.sm100.channel_delta_decode(*args, gate, w[f"{p}.cd.norm"], cfg.rms_eps)
+        else:
+            o = ops.channel_delta(*args, write_state=b.write_state, max_len=b.max_q_len, cu_host=b.cu_q_host)
+            n = ops.head_norm_gate(o, gate, w[f"{p}.cd.norm"], cfg.rms_eps, m.heads)
+        return ops.linear(n, w[f"{p}.cd.out"])
+
     def _spec_mixer(self, p: str, il: int, h, b: StepBatch, kv: KvCache, st: StatePool):
         """Output of layer il's mixer as [(tensor, scale)]: the terms are summed by the stream update that follows."""
         m = self.cfg.layers[il].mixer
@@ -1075,10 +1117,12 @@ class Decoder:
             return [(self._latent_mixer(p, il, h, b, kv), 1.0)]
         if m.kind == "rglru":
             return [(self._rglru_mixer(p, il, h, b, st), 1.0)]
+        if m.kind == "channel_delta":
+            return [(self._channel_delta_mixer(p, il, h, b, st), 1.0)]
         proj = ops.linear(h, self.w[f"{p}.mix.in"])
         if m.kind == "ssd":
             return [(self._ssd_mixer(p, il, proj, b, st), 1.0)]
-        left, used = self._softmax_mixer(p, il, proj, b, kv)
+        left, used = self._softmax_mixer(p, il, proj, b, kv, st)
         if m.kind == "attn":
             return [(left, 1.0)]
         return [(left, m.left_scale), (self._ssd_mixer(p, il, proj[:, used:], b, st), m.right_scale)]
@@ -1089,11 +1133,20 @@ class Decoder:
             return [(ops.linear(ops.up_act(h, w[f"{p}.mlp.up"], w[f"{p}.mlp.act"]), w[f"{p}.mlp.down"]), 1.0)]
         if f.kind == "dense":
             return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act), w[f"{p}.mlp.down"]), 1.0)]
-        routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, 1.0, w.get(f"{p}.moe.router_bias"),
-                             f.n_group, f.keep_group, group_top=f.group_top)
+        routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, f.scale, w.get(f"{p}.moe.router_bias"),
+                             f.n_group, f.keep_group, n_local=f.experts, group_top=f.group_top, gate_row=f.shared_gate,
+                             shared_slots=f.shared_slots())
         ids, wts = routing
-        return [(ops.moe_experts(h, ids, wts, w[f"{p}.moe.gate_up"], w[f"{p}.moe.down"], f.ff, f.act, routing=routing,
-                                 defer_combine="pairs"), 1.0)]
+        up, down, E = w[f"{p}.moe.gate_up"], w[f"{p}.moe.down"], f.experts
+        if f.shared_ff and routing.dense is None:
+            # the shared expert as a dense feed-forward part of its own (decode steps: a slot of the grouped products)
+            sd = self._shared_down.get(p)
+            if sd is None:
+                sd = self._shared_down[p] = down[E:].transpose(0, 1).reshape(self.cfg.hidden, -1).contiguous()
+            hs = ops.up_relu2(h, up[E:].reshape(-1, up.shape[2]))
+            y = ops.moe_experts(h, ids, wts, up[:E], down[:E], f.ff, f.act, routing=routing, defer_combine="pairs")
+            return [(y, 1.0), (ops.linear(hs, sd, tok_scale=routing.gate), 1.0)]
+        return [(ops.moe_experts(h, ids, wts, up, down, f.ff, f.act, routing=routing, defer_combine="pairs"), 1.0)]
 
     def _forward_streams(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool) -> StepOutput:
         """Forward pass of a stack with layer specifications and static hyper-connections: fp32 streams, and per
@@ -1155,6 +1208,43 @@ class Decoder:
             if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
                 captures[il] = x
         hidden = h if rows is None else h.index_select(0, rows)
+        out = StepOutput(hidden=hidden, captures=captures)
+        if want_logits:
+            out.logits = self.logits(hidden)
+        self.pctx.end_step()
+        return out
+
+    def _forward_prenorm(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool) -> StepOutput:
+        """Forward pass of a stack with layer specifications and pre-norm sublayers on one fp32 residual: one launch behind
+        every sublayer adds its output and norms the next one's input. A pass of the loop first maps
+        [stream, embedding output] back to the stream."""
+        cfg, w = self.cfg, self.w
+        H, eps, off = cfg.hidden, cfg.rms_eps, cfg.norm_offset
+        subs = [(il, which) for il, spec in enumerate(cfg.layers) for which in ("attn", "ffn")[:1 if spec.mlp is None else 2]]
+        norm_of = lambda i: w[f"l{cfg.weight_layer(subs[i][0])}.{subs[i][1]}_norm"]              # noqa: E731
+        enters = lambda i: subs[i][1] == "attn" and cfg.begins_pass(subs[i][0])                  # noqa: E731
+        table, ids = (w["tok_embd"], b.token_ids) if b.embeds is None else (b.embeds, None)
+        T = table.shape[0] if ids is None else ids.numel()
+        both = torch.empty(T, 2 * H, dtype=table.dtype, device=table.device) if cfg.loop is not None else None
+        x, h = ops.prenorm_start(table, ids, w.get("embed_norm"), None if enters(0) else norm_of(0), eps, off,
+                                 raw=None if both is None else both[:, H:])
+        if enters(0):
+            both[:, :H].copy_(both[:, H:])
+        captures: Dict[int, torch.Tensor] = {}
+        for i, (il, which) in enumerate(subs):
+            p, last = f"l{cfg.weight_layer(il)}", i + 1 == len(subs)
+            if enters(i):
+                x = ops.linear(both, w["loop_in"], out_dtype=torch.float32)
+                x, h = ops.prenorm_step(x, (), 1.0, norm_of(i), eps, off, dtype=table.dtype)
+            terms = self._spec_mixer(p, il, h, b, kv, st) if which == "attn" else self._spec_ffn(p, il, h)
+            if not last and enters(i + 1):
+                x, h = ops.prenorm_step(x, terms, cfg.residual_mult, None, eps, off, raw=both[:, :H], dtype=table.dtype)
+            else:
+                x, h = ops.prenorm_step(x, terms, cfg.residual_mult, w["output_norm"] if last else norm_of(i + 1), eps, off,
+                                        dtype=table.dtype)
+            if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
+                captures[il] = x.clone()
+        hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
         out = StepOutput(hidden=hidden, captures=captures)
         if want_logits:
             out.logits = self.logits(hidden)
@@ -1410,7 +1500,9 @@ class Decoder:
         if self.cfg.layers is not None:
             if self.cfg.sandwich_norm:
                 return self._forward_sandwich(b, kv, st, want_logits)
-            return self._forward_streams(b, kv, st, want_logits)
+            if self.cfg.hyper_mode == "static":
+                return self._forward_streams(b, kv, st, want_logits)
+            return self._forward_prenorm(b, kv, st, want_logits)
         if self.cfg.hyper_streams > 1:
             return self._forward_hc(b, kv, st, want_logits)
         if self.cfg.sandwich_norm:
@@ -1479,6 +1571,12 @@ class Decoder:
         return True
 
     def _local_logits(self, hidden):
+        if hidden.is_cuda and self.cfg.layers is not None and self.cfg.logit_scale != 1.0 and self.cfg.logit_softcap <= 0:
+            rows = self._logit_rows                 # one size for good: captured graphs hold its address
+            if rows is None:
+                rows = self._logit_rows = torch.full((65536,), self.cfg.logit_scale, device=hidden.device)
+            if hidden.shape[0] <= rows.numel():
+                return ops.linear(hidden, self.lm_head, out_dtype=torch.float32, tok_scale=rows)
         lg = ops.linear(hidden, self.lm_head, out_dtype=torch.float32)
         if lg.is_cuda and self.cfg.logit_softcap > 0:
             return ops.sm100.softcap(lg, self.cfg.logit_scale, self.cfg.logit_softcap)

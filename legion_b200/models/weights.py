@@ -136,8 +136,8 @@ def _ffn_shapes(cfg: ModelConfig, p: str, moe: bool, s: Dict[str, Tuple[int, ...
 def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
     """A layer of a stack with specifications (``ModelConfig.layers``). What reads the mixer's input is one stacked
     projection: ``lin.qkvg`` (linear attention: q | k | v | gate), ``mix.in`` (q | k | v of the attention part, then
-    z | x | B | C | dt of the state-space part)."""
-    p, H, spec = f"l{il}", cfg.hidden, cfg.layers[il]
+    z | x | B | C | dt of the state-space part), ``cd.in`` (``ChannelDeltaSpec.in_columns``)."""
+    p, H, spec = f"l{cfg.weight_layer(il)}", cfg.hidden, cfg.layers[il]
     s: Dict[str, Tuple[int, ...]] = {f"{p}.attn_norm": (H,)}
     if spec.mlp is not None:
         s[f"{p}.ffn_norm"] = (H,)
@@ -162,14 +162,28 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
         s[f"{p}.lru.gates_b"] = (m.blocks * 2 * d,)
         s[f"{p}.lru.log_decay"] = (m.width,)                                    # log of the decay at an open gate
         s[f"{p}.lru.out"] = (H, m.width)
+    elif m.kind == "channel_delta":
+        nk, nv = m.kv_heads * m.dim, m.heads * m.vdim
+        s[f"{p}.cd.in"] = (m.in_columns()["end"], H)                            # q | k | v | b | a1 | g1
+        s[f"{p}.cd.conv_w"] = (2 * nk + nv, m.conv)
+        s[f"{p}.cd.low"] = (m.heads * m.dim + nv, m.rank)                       # decay | output gate, from a1 and g1
+        s[f"{p}.cd.A"] = (m.heads,)
+        s[f"{p}.cd.dt_bias"] = (m.heads * m.dim,)
+        s[f"{p}.cd.norm"] = (m.vdim,)
+        s[f"{p}.cd.out"] = (H, nv)
     else:
         a, r = cfg.attn_spec(il), cfg.recurrent_spec(il)
         rows = 0
         if a is not None:
             rows += (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim
             if a.qk_norm:
-                s[f"{p}.attn.q_norm"] = (a.dim,)
-                s[f"{p}.attn.k_norm"] = (a.dim,)
+                whole = a.norm_over == "all"
+                s[f"{p}.attn.q_norm"] = (a.heads * a.dim if whole else a.dim,)
+                s[f"{p}.attn.k_norm"] = (a.kv_heads * a.dim if whole else a.dim,)
+            if a.bias:
+                s[f"{p}.attn.in_b"] = (rows,)
+            if a.conv:
+                s[f"{p}.attn.conv_w"] = (rows, a.conv)
             s[f"{p}.attn.o"] = (H, a.heads * a.vdim)
         if r is not None:
             inner, conv_c = r.heads * r.vdim, r.heads * r.vdim + 2 * r.groups * r.state
@@ -187,7 +201,7 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
             s[f"{p}.{which}_post_norm"] = (H,)
             if cfg.input_conv:
                 s[f"{p}.{which}_taps"] = (cfg.input_conv, H)                    # oldest token first
-    for which in () if cfg.sandwich_norm else ("hca", "hcf")[:1 if spec.mlp is None else 2]:
+    for which in () if cfg.hyper_mode != "static" else ("hca", "hcf")[:1 if spec.mlp is None else 2]:
         s[f"{p}.{which}.st_in"] = (n,)                  # streams -> sublayer input
         s[f"{p}.{which}.st_out"] = (n,)                 # sublayer output -> streams
         s[f"{p}.{which}.st_mix"] = (n, n)               # stream (row) -> stream (column)
@@ -195,11 +209,12 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
         return s
     f = spec.mlp
     if f.kind == "moe":
-        s[f"{p}.moe.router"] = (f.experts, H)
+        n = f.experts + f.shared_slots()
+        s[f"{p}.moe.router"] = (f.experts + int(f.shared_gate), H)              # its last row gates the shared expert
         if f.correction:
             s[f"{p}.moe.router_bias"] = (f.experts,)
-        s[f"{p}.moe.gate_up"] = (f.experts, 2 * f.ff, H)
-        s[f"{p}.moe.down"] = (f.experts, H, f.ff)
+        s[f"{p}.moe.gate_up"] = (n, 2 * f.ff if f.gated() else f.ff, H)
+        s[f"{p}.moe.down"] = (n, H, f.ff)
     elif not f.gated():
         s[f"{p}.mlp.up"] = (f.ff, H)
         s[f"{p}.mlp.act"] = (2,)
@@ -269,6 +284,10 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
         s.update(gated_mixer_shapes(cfg, "out_hc", inject=False))
     if not cfg.tie_embeddings:
         s["output"] = (cfg.vocab, cfg.hidden)
+    if cfg.embed_norm:
+        s["embed_norm"] = (cfg.hidden,)
+    if cfg.loop is not None:
+        s["loop_in"] = (cfg.hidden, 2 * cfg.hidden)     # [stream, embedding output] -> stream of a pass
     for il in range(cfg.n_layer):
         s.update(layer_weight_shapes(cfg, il))
     for j in range(cfg.mtp_layers):
@@ -323,7 +342,7 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=torch.float32, seed: in
             continue                      # nothing drawn from the host generator for these
         if leaf.endswith("norm"):
             # head norms and the norms behind a recurrent state have plain weights in stacks with specifications
-            plain = cfg.layers is not None and leaf not in ("attn_norm", "ffn_norm", "output_norm")
+            plain = cfg.layers is not None and leaf not in ("attn_norm", "ffn_norm", "output_norm", "embed_norm")
             t = torch.ones(shp, dtype=torch.float32, device=device) - (0.0 if plain else cfg.norm_offset)
         elif leaf == "A":
             t = -(torch.rand(shp, generator=g) * 0.9 + 0.1).to(device)

@@ -20,10 +20,14 @@ def _cuda(t) -> bool:
     return t.is_cuda
 
 
-def linear(x, w, residual=None, out_dtype=None, out=None):
+def linear(x, w, residual=None, out_dtype=None, out=None, tok_scale=None):
+    """x @ w^T, each row times its ``tok_scale`` (float32 [T]), plus the residual."""
     if _cuda(x):
-        return _sm.linear(x, w, residual=residual, out=out, out_dtype=out_dtype or getattr(x, "dtype", torch.bfloat16))
-    y = _ref.linear(x, w, residual=residual, out_dtype=out_dtype)
+        return _sm.linear(x, w, residual=residual, out=out, out_dtype=out_dtype or getattr(x, "dtype", torch.bfloat16),
+                          tok_scale=tok_scale)
+    y = _ref.linear(x, w, residual=residual, out_dtype=out_dtype if tok_scale is None else torch.float32)
+    if tok_scale is not None:
+        y = (y * tok_scale[:, None]).to(out_dtype or x.dtype)
     if out is not None:
         out.copy_(y)
         return out
@@ -67,16 +71,20 @@ def apply_output_gate(attn, gate, n_q, d):
 
 
 def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, max_q_len, scale, window=0, causal=True,
-                    decode_splits=None, max_ctx=None):
+                    decode_splits=None, max_ctx=None, softcap=0.0):
     """Varlen paged attention; ``max_q_len == 1`` selects the flash-decoding kernel on CUDA. fp32 caches and head sizes
-    the tensor-core kernels do not take run on the general kernel (causal only)."""
+    the tensor-core kernels do not take run on the general kernel (causal only). ``softcap`` > 0: scores become
+    softcap * tanh(score / softcap)."""
     if _cuda(q):
         if not _sm.attn_tc_ok(q, k_cache, v_cache):
-            return _sm.paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal)
+            return _sm.paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal,
+                                          softcap=softcap)
         if max_q_len == 1 and causal:
-            return _sm.paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window, decode_splits, max_ctx)
-        return _sm.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal)
-    return _ref.paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal)
+            return _sm.paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window, decode_splits, max_ctx,
+                                    softcap=softcap)
+        return _sm.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal,
+                                softcap=softcap)
+    return _ref.paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal, softcap=softcap)
 
 
 def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1):
@@ -86,21 +94,28 @@ def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
 
 
 def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
-           e_lo=0, n_local=None, norm=None, group_top=2, **gpu_kw):
+           e_lo=0, n_local=None, norm=None, group_top=2, gate_row=False, shared_slots=0, **gpu_kw):
     """Router projection + top-k. Returns an object that unpacks as ``ids, wts`` ([T, k] int32 / float32); on the
     GPU it may also carry the dense routing tables of a decode-sized step for the experts
     [e_lo, e_lo + n_local) of this rank (pass it on as ``routing=``). With ``norm=(weight, eps, w_offset)`` ``x`` is
     the raw residual stream: the RMSNorm runs first (inside the routing launch for decode-sized steps on the GPU)
-    and the result's ``x_normed`` is the normalised input for the experts."""
+    and the result's ``x_normed`` is the normalised input for the experts. ``gate_row``: the last row of ``w_router``
+    gates the shared expert; the result's ``gate`` is its sigmoid [T] (None where the shared expert, stored as
+    ``shared_slots`` experts behind the routed ones, rides in the dense routing tables)."""
     if _cuda(x):
         return _sm.router(x, w_router, k, mode, renorm, route_scale, bias, n_group, topk_group, norm, e_lo, n_local,
-                          group_top=group_top, **gpu_kw)
+                          group_top=group_top, gate_row=gate_row, shared_slots=shared_slots, **gpu_kw)
     xn = None
     if norm is not None:
         xn, _ = _ref.rmsnorm(x, norm[0], norm[1], norm[2])
     logits = _ref.linear(x if xn is None else xn, w_router, out_dtype=torch.float32)
+    gate = None
+    if gate_row:
+        logits, gate = logits[:, :-1], torch.sigmoid(logits[:, -1])
     ids, wts = _ref.router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group, group_top)
-    return _sm.Routing(ids, wts, None, xn)
+    r = _sm.Routing(ids, wts, None, xn)
+    r.gate = gate
+    return r
 
 
 def _moe_experts_ungated(x, ids, wts, w_up, w_down, e_lo, shared, shared_gate, residual, norm, act="relu2", n_ff=None):
@@ -202,6 +217,67 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state=True, 
 def up_act(x, w, ab):
     """Un-gated feed-forward input: xIELU(x w^T) with the activation's two numbers ``ab`` (float32)."""
     return _sm.up_act(x, w, ab) if _cuda(x) else _ref.up_act(x, w, ab)
+
+
+def up_relu2(x, w):
+    """Un-gated feed-forward input: relu(x w^T)^2."""
+    return _sm.linear(x, w, out_dtype=x.dtype, unary="relu2") if _cuda(x) else _ref.gate_up_act(x, w, w.shape[0], "relu2")
+
+
+def prenorm_start(table, ids, pre_w, norm_w, eps, w_offset=0.0, raw=None):
+    """Start of a pre-norm stack on one fp32 residual: x = embedding rows (``ids`` None: rows are given), normed with
+    ``pre_w`` when given. Returns (x [T, H] float32, norm of x or None without ``norm_w``); ``raw`` takes x in the
+    activation type."""
+    if _cuda(table):
+        return _sm.prenorm_step(None, (), 1.0, norm_w, eps, w_offset, raw, start=(table, ids, pre_w))
+    x, h = _ref.prenorm_start(table if ids is None else table[ids.long()], pre_w, norm_w, eps, w_offset)
+    if raw is not None:
+        raw.copy_(x)
+    return x, h
+
+
+def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, dtype=None):
+    """Behind a sublayer: x + mult * (sum of its output ``terms`` [(tensor or ops.sm100.PendingCombine, scale)]) and the
+    norm of that for the next one, in one launch; on CUDA ``x`` is updated in place. No terms: only the norm."""
+    if _cuda(x):
+        return _sm.prenorm_step(x, terms, mult, norm_w, eps, w_offset, raw, dtype=dtype)
+    x, h = _ref.prenorm_step(x, terms, mult, norm_w, eps, w_offset, dtype)
+    if raw is not None:
+        raw.copy_(x)
+    return x, h
+
+
+def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout, positions,
+                    slots, k_cache, v_cache, heads, write_state=True, max_len=None):
+    """What lies between the q | k | v projection and the scores (see ``reference.qkv_conv_append``)."""
+    args = (proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout, positions, slots,
+            k_cache, v_cache, heads, write_state)
+    return _sm.qkv_conv_append(*args, max_len=max_len) if _cuda(proj) else _ref.qkv_conv_append(*args)
+
+
+def channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, write_state=True,
+                  max_len=None, cu_host=None):
+    """Gated delta rule with a decay per key channel (see ``reference.channel_delta``)."""
+    args = (qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, write_state)
+    return _sm.channel_delta(*args, max_len=max_len, cu_host=cu_host) if _cuda(qkv) else _ref.channel_delta(*args)
+
+
+def low_rank_pair(x, w, n0, rank):
+    """x [T, 2 * rank] = a | g times w = [W_a (n0 rows); W_g]: (a W_a^T [T, n0], g W_g^T)."""
+    if _cuda(x) and w.shape[0] == 2 * n0:
+        y = torch.empty(x.shape[0] * 2, n0, dtype=x.dtype, device=x.device)
+        _sm.head_linear(x, w, 2, n0, n0, rank, rank, y)
+        y = y.view(x.shape[0], 2 * n0)
+        return y[:, :n0], y[:, n0:]
+    return linear(x[:, :rank], w[:n0]), linear(x[:, rank:], w[n0:])
+
+
+def head_norm_gate(o, gate, w, eps, heads):
+    """RMS norm of each head of o [T, heads * d], times w [d], times sigmoid(gate)."""
+    if _cuda(o):
+        return _sm.head_norm_gate(o, gate, w, eps, heads)
+    return _ref.gated_rmsnorm(o.view(o.shape[0], heads, -1), gate.reshape(o.shape[0], heads, -1), w, eps,
+                              "sigmoid").reshape(o.shape)
 
 
 def resid_start(table, ids, embed_scale, norm_w, groups, eps, conv=None, max_len=None):

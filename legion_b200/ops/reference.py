@@ -209,7 +209,8 @@ def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, win
 
 def router_topk(logits, k: int, mode: str = "softmax", renorm: bool = True, route_scale: float = 1.0, bias=None,
                 n_group: int = 1, topk_group: int = 1, group_top: int = 2):
-    """Returns (ids [T, k] int32, weights [T, k] float32); ties go to the lower expert id. ``softmax_bias``: selection
+    """Returns (ids [T, k] int32, weights [T, k] float32); ties go to the lower expert id. ``renorm``: True holds the sum
+    of the chosen weights away from zero, "sum" divides by it as it is. ``softmax_bias``: selection
     by softmax score + bias, like the sigmoid mode; ``group_top``: how many scores a group's rank sums up."""
     lf = logits.float()
     T, E = lf.shape
@@ -228,7 +229,9 @@ def router_topk(logits, k: int, mode: str = "softmax", renorm: bool = True, rout
             sel = g.masked_fill(~keep[:, :, None], float("-inf")).reshape(T, E)
     order = torch.sort(sel, dim=-1, descending=True, stable=True).indices[:, :k]
     w = scores.gather(1, order)
-    if renorm:
+    if renorm == "sum":
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    elif renorm:
         w = w / w.sum(-1, keepdim=True).clamp_min(6.1e-5)
     return order.int(), (w * route_scale).float()
 
@@ -282,6 +285,57 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool 
         if write_state and KC > 1:
             conv_state[s] = seq[-(KC - 1):].t().to(conv_state.dtype)
     return out
+
+
+def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout,
+                    positions, slots, k_cache, v_cache, heads: int, write_state: bool = True):
+    """``proj`` [T, q | k | v]: bias, short convolution with carried history, norm of q and k over each head or the whole,
+    rotation, k and v to their cache cells. Everything behind the projection is optional (None). Returns q [T, heads, dk]
+    in the activation type; the values between are float32."""
+    n_kv, dk, dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    T, nq, nk = proj.shape[0], heads * dk, n_kv * dk
+    u = proj.float() if in_b is None else proj.float() + in_b
+    if conv_w is not None:
+        u = causal_conv1d_silu(u, conv_w, None, conv_state, cu_seq, state_slots, write_state, None, False)
+    q, k, v = u[:, :nq], u[:, nq:nq + nk], u[:, nq + nk:nq + nk + n_kv * dv]
+    if q_norm is not None and norm_over == "all":
+        q, k = _norm32(q, q_norm, eps, 0.0), _norm32(k, k_norm, eps, 0.0)
+    q, k = q.reshape(T, heads, dk), k.reshape(T, n_kv, dk)
+    if q_norm is not None and norm_over == "head":
+        q, k = _norm32(q, q_norm, eps, 0.0), _norm32(k, k_norm, eps, 0.0)
+    if rot is not None:
+        turn = rotate_pairs if layout == "pairs" else (lambda x, cs, p: apply_rope(x, cs, p, cs.shape[1]))
+        q, k = turn(q, rot, positions), turn(k, rot, positions)
+    ok = slots >= 0
+    k_cache.view(-1, n_kv, dk)[slots[ok].long()] = k[ok].to(k_cache.dtype)
+    v_cache.view(-1, n_kv, dv)[slots[ok].long()] = v.reshape(T, n_kv, dv)[ok].to(v_cache.dtype)
+    return q.to(proj.dtype).contiguous()
+
+
+def channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H: int, G: int, dk: int, dv: int,
+                  write_state: bool = True):
+    """Gated delta rule with a decay per key channel. ``qkv`` [T, q | k | v] in front of the short convolution, ``a_raw``
+    [T, H * dk] and ``b_raw`` [T, H] before their activations, state [slots, H, dv, dk] float32. Per head
+    S = g S (key channels), S += k (beta (v - S^T k))^T, o = S^T q. Returns o [T, H * dv]."""
+    T = qkv.shape[0]
+    u = causal_conv1d_silu(qkv, conv_w, None, conv_state, cu_seq, slots, write_state).float()
+    unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)                  # noqa: E731
+    q = unit(u[:, :G * dk].reshape(T, G, dk)).repeat_interleave(H // G, 1) * dk ** -0.5
+    k = unit(u[:, G * dk:2 * G * dk].reshape(T, G, dk)).repeat_interleave(H // G, 1)
+    v = u[:, 2 * G * dk:].reshape(T, H, dv)
+    g = torch.exp(A.float()[:, None] * F.softplus(a_raw.float() + dt_bias).view(T, H, dk))
+    beta = torch.sigmoid(b_raw.float())
+    out = torch.empty(T, H, dv, dtype=torch.float32, device=qkv.device)
+    for i in range(len(slots)):
+        S = state[int(slots[i])].clone()
+        for t in range(int(cu_seq[i]), int(cu_seq[i + 1])):
+            S = S * g[t].unsqueeze(1)
+            d = beta[t].unsqueeze(1) * (v[t] - torch.einsum("hvk,hk->hv", S, k[t]))
+            S = S + d.unsqueeze(2) * k[t].unsqueeze(1)
+            out[t] = torch.einsum("hvk,hk->hv", S, q[t])
+        if write_state:
+            state[int(slots[i])] = S
+    return out.reshape(T, H * dv).to(qkv.dtype)
 
 
 def gdn_gates(a, b, A, dt_bias):
@@ -401,6 +455,19 @@ def group_norm_gate(y, gate, w, eps: float, groups: int = 1):
     if gate is not None:
         out = out * torch.sigmoid(gate.float())
     return out.to(y.dtype)
+
+
+def prenorm_start(rows, pre_w, norm_w, eps: float, w_offset: float):
+    """x [T, H] float32: the rows, normed with ``pre_w`` when given; and its norm (``norm_w`` None: none)."""
+    x = rows.float() if pre_w is None else _norm32(rows.float(), pre_w, eps, w_offset)
+    return x, None if norm_w is None else _norm32(x, norm_w, eps, w_offset).to(rows.dtype)
+
+
+def prenorm_step(x, terms, mult: float, norm_w, eps: float, w_offset: float, dtype):
+    """x + mult * (sum of scale * tensor over ``terms``) and the norm of that (``norm_w`` None: none)."""
+    if terms:
+        x = x + mult * sum(c * t.float() for t, c in terms)
+    return x, None if norm_w is None else _norm32(x, norm_w, eps, w_offset).to(dtype)
 
 
 def xielu(z, ab):

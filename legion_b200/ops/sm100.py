@@ -1055,13 +1055,15 @@ def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
 class Routing:
     """Router result of one step: ``ids`` / ``wts`` [T, k] and, for decode-sized steps, the dense routing tables
     (``dense``) that let the expert GEMMs run without a gather. Unpacks as ``ids, wts = routing``."""
-    __slots__ = ("ids", "wts", "dense", "x_normed", "e_lo", "n_local", "shared_slot", "xq")
+    __slots__ = ("ids", "wts", "dense", "x_normed", "e_lo", "n_local", "shared_slot", "xq", "gate", "shared_rows")
 
     def __init__(self, ids, wts, dense=None, x_normed=None, e_lo=0, n_local=None):
         self.ids, self.wts, self.dense, self.x_normed = ids, wts, dense, x_normed
         self.e_lo, self.n_local = e_lo, n_local      # expert range the dense tables were built for
         self.shared_slot = False                     # the shared expert has a slot of its own in the dense tables
         self.xq = None                               # the experts' input already NVFP4-encoded (Nv4Act)
+        self.gate = None                             # [T] sigmoid gate of a shared expert that runs by itself
+        self.shared_rows = 0                         # always-chosen experts in the dense tables, behind a token's pairs
 
     def __iter__(self):
         yield self.ids
