@@ -16,6 +16,9 @@ Configurations (``--config``):
   10 Pemezen at 1B parameters in bf16 (24 layers: two RG-LRU layers and a latent-attention layer in turn).
   11 the closest model of the other families at that size: dense latent attention in every layer (DeepSeek form).
   12, 13  the same pair at 7B parameters (30 layers, 4096 columns).
+  14 Gurozen at 4B parameters in bf16 (24 layer runs: delta-rule layers with a decay per key channel and soft-capped
+     attention in turn, dense and 32-expert feed-forward parts); compared with 7.
+  15 the same at 13B (20 layer runs, 4096 columns); compared with 9.
 The ONE parsed number (``value``) is decode tokens/s at 16 users of the selected configuration; the other rows of
 the grid (1 and 64 users, 32K prefill) are under ``extra``.
 
@@ -107,6 +110,8 @@ CONFIGS = {
     11: dict(model="mla-1b", prompt_len=2048, weights="bf16", dtype="bf16"),
     12: dict(model="pemezen-7b", prompt_len=2048, weights="bf16", dtype="bf16"),
     13: dict(model="mla-7b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    14: dict(model="gurozen-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    15: dict(model="gurozen-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
 }
 
 

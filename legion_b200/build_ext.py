@@ -26,7 +26,8 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
-PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any"}
+PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any",
+           "channel_delta", "qkv_conv"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:
@@ -66,6 +67,7 @@ KIND_KERNELS = {
     "attn": _ATTN, "lightning": _SCAN, "ssd": _SCAN, "parallel": _ATTN | _SCAN,
     "latent": {"attn_mla_sm100", "latent_attn", "attn_prefill_sm100", "attn_decode", "attn_general"},
     "rglru": {"diag_scan", "conv1d", "conv_any"},
+    "channel_delta": {"channel_delta"},
 }
 
 
@@ -74,6 +76,8 @@ def kernels_of(cfg) -> set:
     if cfg.layers is None:
         return _ATTN | {"moe", "attn_mla_sm100"}
     need = set().union(*(KIND_KERNELS[x.mixer.kind] for x in cfg.layers)) | {"resid_step" if cfg.sandwich_norm else "hyper"}
+    if any(a is not None and not a.direct() for a in map(cfg.attn_spec, range(cfg.n_layer))):
+        need |= {"qkv_conv"}
     return need | {"moe"} if cfg.n_expert else need
 
 

@@ -731,7 +731,54 @@ def mla_7b() -> ModelConfig:
                        kv_lora=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, qk_norm=False, dense_ff=11264)
 
 
+def tiny_gurozen() -> "ModelConfig":
+    """Gurozen in miniature: gated delta rule layers with a decay per key channel beside soft-capped attention behind short
+    convolutions, pre-norm sublayers on one scaled residual, squared-ReLU experts with a gated shared one, a dense layer,
+    one layer without feed-forward part, and a loop of three layers that runs twice."""
+    moe = dict(act="relu2", router="sigmoid", renorm="sum", shared_gate=True)
+    rot = dict(scaling="llama3", layout="half")
+    loop = LoopSpec(1, 4, 2)
+    layers = [LayerSpec(ChannelDeltaSpec(4, 2, 40, 32, 4, 16), DenseSpec(200)),
+              LayerSpec(AttnSpec(6, 2, 32, 48, 0.15, norm_over="all", bias=True, conv=3, rot=RotarySpec(24, 1e4, 4.0, 128, **rot),
+                                 softcap=20.0), MoeSpec(10, 3, 56, scale=1.5, n_group=5, keep_group=2, shared_ff=112, **moe)),
+              LayerSpec(ChannelDeltaSpec(3, 3, 24, 56, 2, 8), None),
+              LayerSpec(AttnSpec(4, 1, 64, 32, 0.11, norm_over="all", bias=True, conv=4, rot=RotarySpec(64, 5e4, 8.0, 64, **rot),
+                                 softcap=15.0), DenseSpec(96)),
+              LayerSpec(ChannelDeltaSpec(2, 1, 64, 64, 3, 24), MoeSpec(8, 2, 40, scale=2.0, n_group=2, keep_group=1, shared_ff=72,
+                                                                        **moe))]
+    return ModelConfig(arch="gurozen", hidden=144, vocab=512, rms_eps=1e-5, norm_offset=1.0, tie_embeddings=True, embed_norm=True,
+                       residual_mult=0.7, logit_scale=1.5, layers=loop.expand(layers), loop=loop)
+
+
+def _gurozen(n_layer: int, hidden: int, heads: int, ff: int, expert_ff: int) -> ModelConfig:
+    """``n_layer`` runs of alternating delta-rule and attention layers, four of them a second pass over the same weights;
+    the first half dense, then 32 squared-ReLU experts and a shared one."""
+    rot = RotarySpec(64, 1e6, 8.0, 8192, scaling="llama3", layout="half")
+    moe = MoeSpec(32, 4, expert_ff, "relu2", router="sigmoid", renorm="sum", scale=2.0, n_group=8, keep_group=4,
+                  shared_ff=expert_ff, shared_gate=True)
+    layers = []
+    for il in range(n_layer - 4):
+        mixer = (AttnSpec(heads, heads // 4, 128, 128, 128 ** -0.5, norm_over="all", bias=True, conv=4, rot=rot, softcap=30.0)
+                 if il % 2 else ChannelDeltaSpec(2 * heads, heads, 128, 128, 4, 128))
+        layers.append(LayerSpec(mixer, moe if il >= (n_layer - 4) // 2 else DenseSpec(ff)))
+    loop = LoopSpec(n_layer // 2 - 4, n_layer // 2, 2)
+    return ModelConfig(arch="gurozen", hidden=hidden, vocab=65536, rms_eps=1e-5, norm_offset=1.0, tie_embeddings=True,
+                       embed_norm=True, residual_mult=0.5, logit_scale=1.0, layers=loop.expand(layers), loop=loop)
+
+
+def gurozen_4b() -> ModelConfig:
+    """Gurozen with layers the size of a small production model (random weights; speed measurements)."""
+    return _gurozen(24, 2048, 16, 6144, 1536)
+
+
+def gurozen_13b() -> ModelConfig:
+    return _gurozen(20, 4096, 32, 12288, 3072)
+
+
 PRESETS = {
+    "tiny-gurozen": tiny_gurozen,
+    "gurozen-4b": gurozen_4b,
+    "gurozen-13b": gurozen_13b,
     "tiny-pemezen": tiny_pemezen,
     "pemezen-1b": pemezen_1b,
     "pemezen-7b": pemezen_7b,

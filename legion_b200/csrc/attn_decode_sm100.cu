@@ -47,7 +47,8 @@ struct DecodeTcArgs {
   const int* block_table;
   int table_width, page;
   int Hq, Hkv, n_splits;
-  float scale_log2;
+  float scale_log2;     // softmax scale * log2(e); soft-capped scores: 2 cap log2(e)
+  float cap_k;          // soft-capped scores: see softcap_r
   int window;
   float* o_part;   // [B, Hq, 2 * n_splits, dv]   (part = split * 2 + warpgroup)
   float* ml_part;  // [B, Hq, 2 * n_splits, 2] (reference maximum in natural-log units, sum)
@@ -82,7 +83,8 @@ struct DecodeTcCfg {
 // TMEM round trip of the rescale leaves the per-tile critical path.
 static constexpr float DEC_RESCALE_LOG2 = 8.f;
 
-template <int DK, int DV>
+// CAP: the scores pass a soft cap on their way out of tensor memory
+template <int DK, int DV, bool CAP>
 __global__ void __launch_bounds__(320, 1)
 paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const DecodeTcArgs a) {
@@ -317,6 +319,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int q = 0; q < NQ; ++q) {
           s[q] = -INFINITY;
           if (q < gn) {
+            if constexpr (CAP) r[q] = __float_as_uint(softcap_r(__uint_as_float(r[q]), a.cap_k));
             s[q] = valid ? __uint_as_float(r[q]) * a.scale_log2 : -INFINITY;
             over |= s[q] > m_ref[q] + DEC_RESCALE_LOG2;
           }
@@ -498,11 +501,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 namespace {
 thread_local char g_dec_err[256];
 
-template <int DK, int DV>
+template <int DK, int DV, bool CAP>
 int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const DecodeTcArgs& a,
                      dim3 grid, cudaStream_t s) {
   using Cfg = DecodeTcCfg<DK, DV>;
-  auto kfn = paged_decode_tc_kernel<DK, DV>;
+  auto kfn = paged_decode_tc_kernel<DK, DV, CAP>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -526,8 +529,9 @@ const char* paged_decode_tc_last_error() { return g_dec_err; }
 // Returns 0 on success, 1 on error, -1 when the shape is outside this kernel (caller falls back).
 int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                            long v_cell, const int* block_table, int table_width, int page, const int* ctx_lens,
-                           float scale, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits, float* o_part,
-                           float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status, cudaStream_t s) {
+                           float scale, float softcap, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits,
+                           float* o_part, float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status,
+                           cudaStream_t s) {
   if (B <= 0) return 0;
   if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || k_cell % 8 || v_cell % 8 || page <= 0 ||
       128 % page != 0 || page % 8 != 0 || Hq % Hkv)
@@ -549,10 +553,17 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   DecodeTcArgs a{};
   a.ctx_lens = ctx_lens; a.block_table = block_table; a.table_width = table_width; a.page = page;
   a.Hq = Hq; a.Hkv = Hkv; a.n_splits = n_splits; a.scale_log2 = scale * 1.4426950408889634f; a.window = window;
+  const bool cap = softcap > 0.f;
+  if (cap) {
+    a.cap_k = 2.f * 1.4426950408889634f * scale / softcap;
+    a.scale_log2 = 2.f * 1.4426950408889634f * softcap;
+  }
   a.o_part = o_part; a.ml_part = ml_part; a.status = status; a.dv = dv;
   a.out = static_cast<__nv_bfloat16*>(out); a.group_ctr = group_ctr;
   dim3 grid(Hkv * gtiles, B, n_splits);
-#define LB_DIM(K_, V_) if (DK == K_ && DV == V_) return launch_decode_tc<K_, V_>(tq, tk, tv, a, grid, s);
+#define LB_DIM(K_, V_)                                                                                    \
+  if (DK == K_ && DV == V_)                                                                               \
+    return cap ? launch_decode_tc<K_, V_, true>(tq, tk, tv, a, grid, s) : launch_decode_tc<K_, V_, false>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64) LB_DIM(128, 128) LB_DIM(256, 256) LB_DIM(64, 128) LB_DIM(64, 256) LB_DIM(128, 64) LB_DIM(128, 256)
   LB_DIM(256, 64) LB_DIM(256, 128) LB_DIM(64, 192) LB_DIM(128, 192) LB_DIM(256, 192)
 #undef LB_DIM

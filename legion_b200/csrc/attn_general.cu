@@ -66,7 +66,7 @@ template <typename T, int NV>
 __global__ void __launch_bounds__(128) paged_attn_general_kernel(
     const T* __restrict__ q, long q_row, const T* __restrict__ k_cache, const T* __restrict__ v_cache, long k_cell, long v_cell,
     const int* __restrict__ cu_q, const int* __restrict__ ctx_lens, const int* __restrict__ block_table, int table_width,
-    int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, int window, T* __restrict__ out) {
+    int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, float cap, int window, T* __restrict__ out) {
   extern __shared__ float q_sm[];
   griddep_wait();
   griddep_launch();
@@ -105,6 +105,7 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
       }
       if (d < DK) a0 = fmaf(qs[d], ld_f(kr + d), a0);
       s = (a0 + a1) * scale;
+      if (cap > 0.f) s = cap * tanhf(s / cap);
     }
     float mx = s;
 #pragma unroll
@@ -138,8 +139,8 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
 
 template <typename T>
 int attn_t(const void* q, long q_row, const void* k, const void* v, long k_cell, long v_cell, const int* cu_q, const int* ctx_lens,
-           const int* bt, int tw, int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, int window,
-           void* out, cudaStream_t s) {
+           const int* bt, int tw, int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, float cap,
+           int window, void* out, cudaStream_t s) {
   const long warps = long(nT) * Hq;
   const dim3 grid(unsigned((warps + 3) / 4));
   const size_t smem = size_t(4) * DK * 4;
@@ -148,7 +149,7 @@ int attn_t(const void* q, long q_row, const void* k, const void* v, long k_cell,
   if (DV <= 32 * N)                                                                                                    \
     return launch_pdl(paged_attn_general_kernel<T, N>, grid, dim3(128), smem, s, static_cast<const T*>(q), q_row,      \
                       static_cast<const T*>(k), static_cast<const T*>(v), k_cell, v_cell, cu_q, ctx_lens, bt, tw,      \
-                      page, n_seqs, nT, Hq, Hkv, DK, DV, scale, window, static_cast<T*>(out)) != cudaSuccess;
+                      page, n_seqs, nT, Hq, Hkv, DK, DV, scale, cap, window, static_cast<T*>(out)) != cudaSuccess;
   LB_NV(2) LB_NV(4) LB_NV(8) LB_NV(16) LB_NV(32)
 #undef LB_NV
   return 1;
@@ -173,14 +174,14 @@ int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld,
 
 int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
-                              int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, int window, void* out,
-                              bool f32, cudaStream_t s) {
+                              int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, float softcap, int window,
+                              void* out, bool f32, cudaStream_t s) {
   if (T <= 0 || n_seqs <= 0) return 0;
   if (page <= 0 || Hkv <= 0 || Hq % Hkv) return 1;
   return f32 ? attn_t<float>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page, n_seqs,
-                             T, Hq, Hkv, DK, DV, scale, window, out, s)
+                             T, Hq, Hkv, DK, DV, scale, softcap, window, out, s)
              : attn_t<__nv_bfloat16>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page,
-                                     n_seqs, T, Hq, Hkv, DK, DV, scale, window, out, s);
+                                     n_seqs, T, Hq, Hkv, DK, DV, scale, softcap, window, out, s);
 }
 
 }  // namespace lb

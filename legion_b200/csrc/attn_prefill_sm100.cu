@@ -89,7 +89,8 @@ struct PrefillArgs {
   const int* block_table;  // [n_seqs, table_width]
   int table_width, page;
   int Hq, Hkv;
-  float scale_log2;        // softmax scale * log2(e)
+  float scale_log2;        // softmax scale * log2(e); soft-capped scores: 2 cap log2(e)
+  float cap_k;             // soft-capped scores: see softcap_r
   int window;              // 0 = none
   int causal;
   __nv_bfloat16* out;      // [T, Hq, dv]
@@ -118,7 +119,8 @@ struct PrefillCfg {
   static constexpr int TMEM_COLS = TMEM_RAW <= 128 ? 128 : (TMEM_RAW <= 256 ? 256 : 512);
 };
 
-template <int DK, int DV, int BKV>
+// CAP: the scores pass a soft cap on their way out of tensor memory
+template <int DK, int DV, int BKV, bool CAP>
 __global__ void __launch_bounds__(160, (DK <= 128 && DV <= 128 && BKV == 64) ? 2 : 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const PrefillArgs a) {
@@ -313,6 +315,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
         for (int c = 0; c < BKV; c += 32) tmem_ld32(tmem_Si + lane_off + c, *reinterpret_cast<uint32_t(*)[32]>(&r[c]));
         tmem_ld_wait();
+        if constexpr (CAP) {
+#pragma unroll
+          for (int j = 0; j < BKV; ++j) r[j] = __float_as_uint(softcap_r(__uint_as_float(r[j]), a.cap_k));
+        }
         float mx = -INFINITY;
         if (full_blk) {
           // four independent chains: a single one is 64 dependent operations with only two warps per scheduler
@@ -495,11 +501,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 namespace {
 thread_local char g_attn_err[256];
 
-template <int DK, int DV, int BKV>
+template <int DK, int DV, int BKV, bool CAP = false>
 int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const PrefillArgs& a,
                    dim3 grid, cudaStream_t s) {
   using Cfg = PrefillCfg<DK, DV, BKV>;
-  auto kfn = prefill_attn_kernel<DK, DV, BKV>;
+  static_assert(!CAP || BKV <= 64, "the soft cap is applied to a row of scores in registers");
+  auto kfn = prefill_attn_kernel<DK, DV, BKV, CAP>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -522,11 +529,12 @@ const char* prefill_attn_last_error() { return g_attn_err; }
 
 int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                         long v_cell, const int* cu_q, const int* ctx_lens, const int* block_table, int table_width,
-                        int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, int window,
-                        int causal, void* out, int* status, cudaStream_t s) {
+                        int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, float softcap,
+                        int window, int causal, void* out, int* status, cudaStream_t s) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
   const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : (dv <= 192 ? 192 : 256));
-  const int BKV = (DK >= 128 || DV >= 128) ? 64 : 128;
+  const bool cap = softcap > 0.f;
+  const int BKV = (DK >= 128 || DV >= 128 || cap) ? 64 : 128;
   if (page <= 0 || BKV % page != 0 || page % 8 != 0) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: page size %d must be a multiple of 8 dividing %d",
              page, BKV);
@@ -551,9 +559,15 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
   PrefillArgs a{};
   a.cu_q = cu_q; a.ctx_lens = ctx_lens; a.block_table = block_table; a.table_width = table_width; a.page = page;
   a.Hq = Hq; a.Hkv = Hkv; a.scale_log2 = scale * 1.4426950408889634f; a.window = window; a.causal = causal;
+  if (cap) {
+    a.cap_k = 2.f * 1.4426950408889634f * scale / softcap;
+    a.scale_log2 = 2.f * 1.4426950408889634f * softcap;
+  }
   a.out = static_cast<__nv_bfloat16*>(out); a.dk = dk; a.dv = dv; a.status = status;
   dim3 grid((max_q_len + 127) / 128, Hq, n_seqs);
-#define LB_DIM(K_, V_, B_) if (DK == K_ && DV == V_) return launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
+#define LB_DIM(K_, V_, B_)                                                                   \
+  if (DK == K_ && DV == V_)                                                                  \
+    return cap ? launch_prefill<K_, V_, 64, true>(tq, tk, tv, a, grid, s) : launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64, 128) LB_DIM(128, 128, 64) LB_DIM(256, 256, 64)
   LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64)
   LB_DIM(64, 192, 64) LB_DIM(128, 192, 64) LB_DIM(256, 192, 64) LB_DIM(256, 128, 64)

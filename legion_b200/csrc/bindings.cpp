@@ -43,7 +43,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
            const OptT& ws, const OptT& counters, Tensor& status, const OptT& tile_group, const OptT& tile_tok0,
            const OptT& tile_ntok, const OptT& meta, int64_t max_tiles, int64_t rows_per_group, int64_t n_tok,
            std::vector<int64_t> out_peer, const OptT& tile_out0, const OptT& w_scales, const OptT& w_gscale,
-           int64_t x_group_col, int64_t k_override, int64_t act, const OptT& xielu) {
+           int64_t x_group_col, int64_t k_override, int64_t act, const OptT& xielu, bool relu2) {
   const bool fp4 = w_scales.has_value();     // w = NVFP4 codes [rows, K/2] uint8, w_scales = e4m3 bytes [rows, K/16]
   if (fp4) {
     TORCH_CHECK(w.scalar_type() == at::kByte && w_scales->is_contiguous() && w_scales->element_size() == 1 &&
@@ -84,6 +84,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
                 "wgemm: xIELU takes two float32 numbers and one weight tile");
     h.xielu = xielu->data_ptr<float>();
   }
+  h.relu2 = relu2;
   h.tile_group = optp<int>(tile_group); h.tile_tok0 = optp<int>(tile_tok0); h.tile_ntok = optp<int>(tile_ntok);
   h.n_tiles_dev = optp<int>(meta);
   h.tile_out0 = optp<int>(tile_out0);
@@ -333,7 +334,7 @@ void embed(const Tensor& ids, const Tensor& table, Tensor& out) {
 
 void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_table,
                   const Tensor& ctx_lens, double scale, int64_t window, int64_t n_splits, Tensor& o_part,
-                  Tensor& ml_part, Tensor& out, bool use_tc, Tensor& status, Tensor& counters) {
+                  Tensor& ml_part, Tensor& out, bool use_tc, Tensor& status, Tensor& counters, double softcap) {
   check_bf16(q, "q");
   c10::cuda::CUDAGuard guard(q.device());
   const int B = int(q.size(0)), Hq = int(q.size(1)), D = int(q.size(2)), DV = int(v_cache.size(-1));
@@ -347,13 +348,14 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
     const int rc = lb::paged_decode_tc_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), n_cells,
                                               long(Hkv) * D, long(Hkv) * DV, block_table.data_ptr<int>(),
                                               int(block_table.size(1)), page, ctx_lens.data_ptr<int>(), float(scale),
-                                              int(window), B, Hq, Hkv, D, DV, int(n_splits), o_part.data_ptr<float>(),
+                                              float(softcap), int(window), B, Hq, Hkv, D, DV, int(n_splits), o_part.data_ptr<float>(),
                                               ml_part.data_ptr<float>(), out.data_ptr(), counters.data_ptr<int>(),
                                               int(counters.numel()), reinterpret_cast<int*>(status.data_ptr()),
                                               cur_stream());
     TORCH_CHECK(rc <= 0, lb::paged_decode_tc_last_error());
     if (rc == 0) return;
   }
+  TORCH_CHECK(softcap <= 0, "paged_decode: soft-capped scores need the tensor-core kernel");
   TORCH_CHECK(DV == D, "paged_decode: keys and values of different sizes need the tensor-core kernel");
   const int rc = lb::paged_decode_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.stride(-3),
                                          block_table.data_ptr<int>(), int(block_table.size(1)), page,
@@ -365,7 +367,7 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
 
 void prefill_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
                   const Tensor& ctx_lens, const Tensor& block_table, int64_t max_q_len, double scale, int64_t window,
-                  bool causal, Tensor& out, Tensor& status) {
+                  bool causal, Tensor& out, Tensor& status, double softcap) {
   check_bf16(q, "q");
   TORCH_CHECK(q.is_contiguous() && out.is_contiguous(), "prefill_attn: q/out must be contiguous [T, Hq, D]");
   c10::cuda::CUDAGuard guard(q.device());
@@ -378,7 +380,8 @@ void prefill_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   const int rc = lb::prefill_attn_launch(q.data_ptr(), T, k_cache.data_ptr(), v_cache.data_ptr(), n_cells,
                                          long(Hkv) * D, long(Hkv) * DV, cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(),
                                          block_table.data_ptr<int>(), int(block_table.size(1)), page,
-                                         int(ctx_lens.numel()), int(max_q_len), Hq, Hkv, D, DV, float(scale), int(window),
+                                         int(ctx_lens.numel()), int(max_q_len), Hq, Hkv, D, DV, float(scale),
+                                         float(softcap), int(window),
                                          causal ? 1 : 0, out.data_ptr(), reinterpret_cast<int*>(status.data_ptr()),
                                          cur_stream());
   TORCH_CHECK(rc == 0, lb::prefill_attn_last_error());
@@ -434,31 +437,35 @@ void mla_prep(const Tensor& kva, const Tensor& norm_w, double eps, double w_offs
               "mla_prep launch failed");
 }
 
-void router_topk(const Tensor& logits, const OptT& bias, int64_t k, int64_t mode, bool renorm, double route_scale,
-                 int64_t n_group, int64_t topk_group, Tensor& ids, Tensor& wts, int64_t group_top) {
+void router_topk(const Tensor& logits, const OptT& bias, int64_t k, int64_t mode, int64_t renorm, double route_scale,
+                 int64_t n_group, int64_t topk_group, Tensor& ids, Tensor& wts, int64_t group_top, const OptT& gate) {
   TORCH_CHECK(logits.scalar_type() == at::kFloat && logits.stride(1) == 1, "router logits must be float32");
+  // with a gate output the last column gates the shared expert
+  const int64_t E = logits.size(1) - (gate.has_value() ? 1 : 0);
+  TORCH_CHECK(!gate.has_value() || (gate->scalar_type() == at::kFloat && gate->is_contiguous() && gate->numel() >= logits.size(0)),
+              "router_topk: float32 gate [tokens]");
   c10::cuda::CUDAGuard guard(logits.device());
   TORCH_CHECK(lb::router_topk_launch(logits.data_ptr<float>(), logits.stride(0), optp<float>(bias),
-                                     int(logits.size(1)), int(k), int(mode), renorm ? 1 : 0, float(route_scale),
+                                     int(E), int(k), int(mode), int(renorm), float(route_scale),
                                      int(n_group), int(topk_group), int(group_top), ids.data_ptr<int>(),
-                                     wts.data_ptr<float>(), int(logits.size(0)), cur_stream()) == 0,
+                                     wts.data_ptr<float>(), optpm<float>(gate), int(logits.size(0)), cur_stream()) == 0,
               "router_topk: unsupported (experts <= 512, k <= 32, groups <= 32)");
 }
 
 void moe_route_small(const Tensor& x, const OptT& norm_w, double eps, double w_offset, const OptT& x_normed,
-                     const Tensor& w, const OptT& bias, int64_t k, int64_t mode, bool renorm, double route_scale,
+                     const Tensor& w, const OptT& bias, int64_t k, int64_t mode, int64_t renorm, double route_scale,
                      int64_t n_group, int64_t topk_group, Tensor& logits, Tensor& ids, Tensor& wts, int64_t bn,
                      Tensor& tile_group, Tensor& slot_base, Tensor& tile_ntok, Tensor& meta, Tensor& out_rows,
                      Tensor& tok_scale, Tensor& done_ctr, int64_t e_lo, int64_t n_local, const OptT& sh_gate_w,
                      const OptT& sh_logit, bool shared_slot, Tensor& status, Tensor& active,
-                     int64_t group_top) {
+                     int64_t group_top, int64_t shared_rows) {
   check_bf16(x, "x");
   check_bf16(w, "w");
   const int64_t T = x.size(0), E = w.size(0);
   if (sh_gate_w.has_value()) {
     check_bf16(*sh_gate_w, "sh_gate_w");
     TORCH_CHECK(sh_gate_w->numel() == x.size(1) && sh_gate_w->is_contiguous() && sh_logit.has_value() &&
-                    sh_logit->scalar_type() == at::kFloat && sh_logit->numel() >= 4 * 64 && shared_slot,
+                    sh_logit->scalar_type() == at::kFloat && sh_logit->numel() >= 4 * 64 && (shared_slot || shared_rows > 0),
                 "moe_route_small: the shared gate is one row of the hidden width with a float [4 * 64] scratch");
   }
   TORCH_CHECK(x.size(1) == w.size(1) && x.stride(1) == 1 && w.stride(1) == 1, "moe_route_small: shape mismatch");
@@ -467,7 +474,7 @@ void moe_route_small(const Tensor& x, const OptT& norm_w, double eps, double w_o
               "moe_route_small: the logit scratch holds four planes of 64 x 512 floats (one per column split)");
   TORCH_CHECK(done_ctr.numel() >= 2 && done_ctr.element_size() == 4, "moe_route_small: two int32 counters");
   TORCH_CHECK(active.scalar_type() == at::kInt && active.numel() >= n_local, "moe_route_small: active flags [n_local]");
-  const int64_t max_slots = std::min<int64_t>(E, n_local) + (shared_slot ? 1 : 0);
+  const int64_t max_slots = std::min<int64_t>(E, n_local) + (shared_rows > 0 ? shared_rows : (shared_slot ? 1 : 0));
   TORCH_CHECK(tile_group.numel() >= max_slots && slot_base.numel() >= max_slots && tile_ntok.numel() >= max_slots &&
                   meta.numel() >= 2 && out_rows.numel() >= max_slots * bn && tok_scale.numel() >= max_slots * bn,
               "moe_route_small: tables too small");
@@ -476,12 +483,12 @@ void moe_route_small(const Tensor& x, const OptT& norm_w, double eps, double w_o
                   x.data_ptr(), x.stride(0), optp<float>(norm_w), float(eps), float(w_offset),
                   x_normed.has_value() ? x_normed->data_ptr() : nullptr,
                   x_normed.has_value() ? x_normed->stride(0) : 0, w.data_ptr(), w.stride(0), int(x.size(1)),
-                  logits.data_ptr<float>(), optp<float>(bias), int(E), int(k), int(mode), renorm ? 1 : 0,
+                  logits.data_ptr<float>(), optp<float>(bias), int(E), int(k), int(mode), int(renorm),
                   float(route_scale), int(n_group), int(topk_group), int(group_top), ids.data_ptr<int>(),
                   wts.data_ptr<float>(), int(T), int(bn), tile_group.data_ptr<int>(), slot_base.data_ptr<int>(), tile_ntok.data_ptr<int>(),
                   meta.data_ptr<int>(), out_rows.data_ptr<int>(), tok_scale.data_ptr<float>(),
                   reinterpret_cast<unsigned int*>(done_ctr.data_ptr()), int(e_lo), int(n_local),
-                  sh_gate_w.has_value() ? sh_gate_w->data_ptr() : nullptr, optpm<float>(sh_logit), shared_slot ? 1 : 0,
+                  sh_gate_w.has_value() ? sh_gate_w->data_ptr() : nullptr, optpm<float>(sh_logit), shared_slot ? 1 : 0, int(shared_rows),
                   reinterpret_cast<int*>(status.data_ptr()), active.data_ptr<int>(), cur_stream()) == 0,
               "moe_route_small: unsupported (tokens <= 64 and <= bn, pairs <= 1024, experts <= 512, k <= 32)");
 }
@@ -605,7 +612,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         pybind11::arg("n_tok"), pybind11::arg("out_peer"), pybind11::arg("tile_out0") = pybind11::none(),
         pybind11::arg("w_scales") = pybind11::none(), pybind11::arg("w_gscale") = pybind11::none(),
         pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0, pybind11::arg("act") = 0,
-        pybind11::arg("xielu") = pybind11::none());
+        pybind11::arg("xielu") = pybind11::none(), pybind11::arg("relu2") = false);
   m.def("wgemm_fp8", &wgemm_fp8);
   m.def("wgemm_fp8_q", &wgemm_fp8_q);
   m.def("wgemm_allreduce", &wgemm_allreduce);
@@ -615,13 +622,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sigmoid_gate", &sigmoid_gate);
   m.def("glu", &glu);
   m.def("embed", &embed);
-  m.def("paged_decode", &paged_decode);
+  m.def("paged_decode", &paged_decode);      // softcap > 0: scores become softcap * tanh(score / softcap)
   m.def("prefill_attn", &prefill_attn);
   m.def("mla_attn", &mla_attn);
   m.def("mla_prep", &mla_prep);
   m.def("router_topk", &router_topk, pybind11::arg("logits"), pybind11::arg("bias"), pybind11::arg("k"),
         pybind11::arg("mode"), pybind11::arg("renorm"), pybind11::arg("route_scale"), pybind11::arg("n_group"),
-        pybind11::arg("topk_group"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("group_top") = 2);
+        pybind11::arg("topk_group"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("group_top") = 2,
+        pybind11::arg("gate") = pybind11::none());
   // group_top: how many of a group's best scores its rank sums up (the other routers of this library sum two)
   m.def("moe_route_small", &moe_route_small);
   m.def("moe_plan", &moe_plan);

@@ -3,6 +3,8 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include <cmath>
+
 #include "gdn.h"
 #include "layers.h"
 
@@ -108,6 +110,38 @@ lb::DiagScanArgs diag_args(int64_t T, int64_t W, const Tensor& gates_b, const Te
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   return a;
 }
+
+lb::ChannelDeltaArgs delta_args(const Tensor& qkv, const Tensor& conv_w, Tensor& conv_state, const Tensor& a_raw, const Tensor& A,
+                                const Tensor& dt_bias, const Tensor& b_raw, Tensor& state, const Tensor& cu, const Tensor& slots,
+                                int64_t H, int64_t G, int64_t DK, int64_t DV, Tensor& out, bool f32) {
+  const int64_t T = qkv.size(0), C = 2 * G * DK + H * DV;
+  same(a_raw, f32, "decay projection");
+  same(b_raw, f32, "beta projection");
+  same(out, f32, "out");
+  TORCH_CHECK(G >= 1 && H % G == 0 && qkv.dim() == 2 && qkv.size(1) == C && a_raw.size(0) == T && a_raw.size(1) == H * DK &&
+                  b_raw.size(0) == T && b_raw.size(1) == H && out.size(0) == T && out.size(1) == H * DV,
+              "channel_delta: q | k | v [T, columns], decays [T, H * DK], beta [T, H], out [T, H * DV]");
+  f32c(conv_w, 0, "conv_w");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C, "channel_delta: conv_w [columns, taps]");
+  TORCH_CHECK(conv_state.scalar_type() == at::kFloat && conv_state.is_contiguous() && conv_state.dim() == 3 &&
+                  conv_state.size(1) == C && conv_state.size(2) == conv_w.size(1) - 1, "channel_delta: history [slots, columns, taps - 1]");
+  f32c(A, H, "A");
+  f32c(dt_bias, H * DK, "dt_bias");
+  TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() == 4 && state.size(1) == H &&
+                  state.size(2) == DV && state.size(3) == DK, "channel_delta: state [slots, H, DV, DK] float32");
+  TORCH_CHECK(cu.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && cu.numel() == slots.numel() + 1,
+              "channel_delta: int32 sequence bounds and slots");
+  lb::ChannelDeltaArgs a{};
+  a.qkv = qkv.data_ptr(); a.ld = qkv.stride(0);
+  a.conv_w = conv_w.data_ptr<float>(); a.KC = int(conv_w.size(1)); a.conv_state = conv_state.data_ptr<float>();
+  a.a = a_raw.data_ptr(); a.lda = a_raw.stride(0); a.A = A.data_ptr<float>(); a.dt_bias = dt_bias.data_ptr<float>();
+  a.b = b_raw.data_ptr(); a.ldb = b_raw.stride(0);
+  a.state = state.data_ptr<float>(); a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>();
+  a.n_seqs = int(slots.numel()); a.T = int(T); a.H = int(H); a.G = int(G); a.DK = int(DK); a.DV = int(DV);
+  a.scale = 1.f / std::sqrt(float(DK)); a.l2_eps = 1e-6f;
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  return a;
+}
 }  // namespace
 
 void bind_layers(pybind11::module_& m) {
@@ -159,6 +193,165 @@ void bind_layers(pybind11::module_& m) {
     a.h = h.data_ptr(); a.ldh = h.stride(0); a.rows = int(R); a.S = int(S); a.H = int(H);
     c10::cuda::CUDAGuard guard(h.device());
     TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "hyper_step: at most 16 streams of 51200 columns", cuda_error());
+  });
+  m.def("prenorm_step", [](const OptT& x_in, Tensor& x_out, const OptT& emb, const OptT& ids, const OptT& pre_w, const OptT& y0,
+                           double c0, int64_t y_rows, const OptT& y1, double c1, const OptT& norm_w, double eps, double w_offset,
+                           const OptT& h, const OptT& raw) {
+    // one stream of the hyper-connection launch without mix weights
+    TORCH_CHECK(h.has_value() || raw.has_value(), "prenorm_step: nothing to write for the next sublayer");
+    const bool f32 = is_f32(h.has_value() ? *h : *raw, "h");
+    TORCH_CHECK(x_out.dim() == 2 && x_out.is_contiguous() && x_out.scalar_type() == at::kFloat,
+                "prenorm_step: the stream is contiguous float32 [rows, width]");
+    const int64_t R = x_out.size(0), H = x_out.size(1);
+    lb::HyperArgs a{};
+    a.x_out = x_out.data_ptr<float>();
+    a.y_rows = 1;
+    if (x_in.has_value()) {
+      TORCH_CHECK(x_in->sizes() == x_out.sizes() && x_in->is_contiguous() && x_in->scalar_type() == at::kFloat,
+                  "prenorm_step: x_in like x_out");
+      a.x_in = x_in->data_ptr<float>();
+      if (y0.has_value()) {
+        same(*y0, f32, "y0");
+        TORCH_CHECK(y0->dim() == 2 && y0->size(1) == H && y_rows >= 1 && y0->size(0) >= R * y_rows, "prenorm_step: y0 [rows * y_rows, width]");
+        a.y0 = y0->data_ptr(); a.ldy0 = y0->stride(0); a.y_rows = int(y_rows);
+      }
+      if (y1.has_value()) {
+        same(*y1, f32, "y1");
+        TORCH_CHECK(y1->dim() == 2 && y1->size(1) == H && y1->size(0) >= R, "prenorm_step: y1 [rows, width]");
+        a.y1 = y1->data_ptr(); a.ldy1 = y1->stride(0);
+      }
+    } else {
+      TORCH_CHECK(emb.has_value() && emb->dim() == 2 && emb->size(1) == H, "prenorm_step: embedding rows");
+      same(*emb, f32, "emb");
+      a.emb = emb->data_ptr(); a.ld_emb = emb->stride(0); a.vocab = int(emb->size(0));
+      if (ids.has_value()) {
+        TORCH_CHECK(ids->scalar_type() == at::kInt && ids->is_contiguous() && ids->numel() == R, "prenorm_step: int32 ids");
+        a.ids = ids->data_ptr<int>();
+      } else {
+        TORCH_CHECK(emb->size(0) >= R, "prenorm_step: one embedding row per token");
+      }
+      if (pre_w.has_value()) {
+        f32c(*pre_w, H, "pre_w");
+        a.pre_w = pre_w->data_ptr<float>();
+      }
+    }
+    if (h.has_value()) {
+      TORCH_CHECK(norm_w.has_value() && h->dim() == 2 && h->size(0) == R && h->size(1) == H, "prenorm_step: h [rows, width] and its norm");
+      f32c(*norm_w, H, "norm_w");
+      a.norm_w = norm_w->data_ptr<float>();
+      a.h = h->data_ptr(); a.ldh = h->stride(0);
+    }
+    if (raw.has_value()) {
+      same(*raw, f32, "raw");
+      TORCH_CHECK(raw->dim() == 2 && raw->size(0) == R && raw->size(1) == H, "prenorm_step: raw [rows, width]");
+      a.raw = raw->data_ptr(); a.ldraw = raw->stride(0);
+    }
+    a.c0 = float(c0); a.c1 = float(c1); a.eps = float(eps); a.w_offset = float(w_offset);
+    a.rows = int(R); a.S = 1; a.H = int(H);
+    c10::cuda::CUDAGuard guard(x_out.device());
+    TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "prenorm_step: rows of at most 51200 columns", cuda_error());
+  });
+  m.def("qkv_conv_append", [](const Tensor& x, const OptT& in_b, const OptT& conv_w, const OptT& conv_state, const Tensor& cu,
+                              const Tensor& state_slots, const OptT& qw, const OptT& kw, bool norm_all, double eps,
+                              const OptT& cos_sin, bool rot_half, const Tensor& positions, const Tensor& slots, Tensor& q_out,
+                              Tensor& k_cache, Tensor& v_cache, int64_t max_len, bool write_state) {
+    const bool f32 = is_f32(x, "x");
+    same(q_out, f32, "q_out");
+    same(k_cache, f32, "k_cache");
+    same(v_cache, f32, "v_cache");
+    lb::QkvConvArgs a{};
+    const int64_t T = q_out.size(0), Hq = q_out.size(1), DK = q_out.size(2), Hkv = k_cache.size(-2), DV = v_cache.size(-1);
+    const int64_t C = (Hq + Hkv) * DK + Hkv * DV;
+    TORCH_CHECK(x.dim() == 2 && x.size(0) == T && x.size(1) == C && k_cache.size(-1) == DK && v_cache.size(-2) == Hkv &&
+                    q_out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous(), "qkv_conv_append: q | k | v columns");
+    TORCH_CHECK(cu.scalar_type() == at::kInt && state_slots.scalar_type() == at::kInt && cu.numel() == state_slots.numel() + 1 &&
+                    positions.scalar_type() == at::kInt && positions.numel() == T && slots.scalar_type() == at::kLong &&
+                    slots.numel() == T, "qkv_conv_append: int32 bounds, slots and positions, int64 cells");
+    a.x = x.data_ptr(); a.ld = x.stride(0);
+    if (in_b.has_value()) {
+      f32c(*in_b, C, "bias");
+      a.in_b = in_b->data_ptr<float>();
+    }
+    a.KC = 1;
+    if (conv_w.has_value()) {
+      f32c(*conv_w, 0, "conv_w");
+      TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(0) == C, "qkv_conv_append: conv_w [columns, taps]");
+      a.conv_w = conv_w->data_ptr<float>();
+      a.KC = int(conv_w->size(1));
+      if (a.KC > 1) {
+        TORCH_CHECK(conv_state.has_value() && conv_state->scalar_type() == at::kFloat && conv_state->is_contiguous() &&
+                        conv_state->dim() == 3 && conv_state->size(1) == C && conv_state->size(2) == a.KC - 1,
+                    "qkv_conv_append: history [slots, columns, taps - 1]");
+        a.conv_state = conv_state->data_ptr<float>();
+      }
+    }
+    a.cu = cu.data_ptr<int>(); a.state_slots = state_slots.data_ptr<int>(); a.n_seqs = int(state_slots.numel());
+    TORCH_CHECK(qw.has_value() == kw.has_value(), "qkv_conv_append: norms of q and k go together");
+    if (qw.has_value()) {
+      f32c(*qw, norm_all ? Hq * DK : DK, "q norm");
+      f32c(*kw, norm_all ? Hkv * DK : DK, "k norm");
+      a.qw = qw->data_ptr<float>(); a.kw = kw->data_ptr<float>();
+    }
+    a.norm_all = norm_all; a.eps = float(eps);
+    if (cos_sin.has_value()) {
+      f32c(*cos_sin, 0, "cos_sin");
+      a.cos_sin = cos_sin->data_ptr<float>();
+      a.rot = int(cos_sin->size(1));
+    }
+    a.rot_half = rot_half;
+    a.positions = positions.data_ptr<int>(); a.slots = reinterpret_cast<const long*>(slots.data_ptr());
+    a.q_out = q_out.data_ptr(); a.k_cache = k_cache.data_ptr(); a.v_cache = v_cache.data_ptr();
+    a.k_cell = Hkv * DK; a.v_cell = Hkv * DV;
+    a.T = int(T); a.Hq = int(Hq); a.Hkv = int(Hkv); a.DK = int(DK); a.DV = int(DV);
+    a.max_len = int(max_len); a.write_state = write_state;
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::qkv_conv_append_launch(a, f32, cur_stream()) == 0,
+                "qkv_conv_append: at most 51200 query and key columns, rotation within a head", cuda_error());
+  });
+  m.def("channel_delta_record_floats", [](int64_t H, int64_t DK, int64_t DV) {
+    return int64_t(lb::channel_delta_record_floats(int(H), int(DK), int(DV)));
+  });
+  m.def("channel_delta", [](const Tensor& qkv, const Tensor& conv_w, Tensor& conv_state, const Tensor& a_raw, const Tensor& A,
+                            const Tensor& dt_bias, const Tensor& b_raw, Tensor& state, const Tensor& cu, const Tensor& slots,
+                            int64_t H, int64_t G, int64_t DK, int64_t DV, Tensor& out, bool write_state, const Tensor& rec,
+                            Tensor& status) {
+    const bool f32 = is_f32(qkv, "qkv");
+    auto a = delta_args(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu, slots, H, G, DK, DV, out, f32);
+    a.write_state = write_state;
+    f32c(rec, 0, "scratch");
+    c10::cuda::CUDAGuard guard(qkv.device());
+    TORCH_CHECK(lb::channel_delta_launch(a, rec.data_ptr<float>(), rec.numel(), reinterpret_cast<int*>(status.data_ptr()), f32,
+                                         cur_stream()) == 0,
+                "channel_delta: key heads of at most 256 columns, heads a multiple of the key heads", cuda_error());
+  });
+  m.def("channel_delta_decode", [](const Tensor& qkv, const Tensor& conv_w, Tensor& conv_state, const Tensor& a_raw, const Tensor& A,
+                                   const Tensor& dt_bias, const Tensor& b_raw, Tensor& state, const Tensor& cu,
+                                   const Tensor& slots, int64_t H, int64_t G, int64_t DK, int64_t DV, const Tensor& gate,
+                                   const Tensor& norm_w, double eps, Tensor& ctr, Tensor& out) {
+    const bool f32 = is_f32(qkv, "qkv");
+    auto a = delta_args(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu, slots, H, G, DK, DV, out, f32);
+    a.write_state = 1;
+    same(gate, f32, "gate");
+    f32c(norm_w, DV, "norm weight");
+    TORCH_CHECK(qkv.size(0) == slots.numel() && gate.size(0) == qkv.size(0) && gate.size(1) == H * DV && ctr.element_size() == 4 &&
+                    ctr.numel() >= slots.numel() * G, "channel_delta_decode: one token per sequence, gate like the output");
+    c10::cuda::CUDAGuard guard(qkv.device());
+    TORCH_CHECK(lb::channel_delta_decode_launch(a, gate.data_ptr(), gate.stride(0), norm_w.data_ptr<float>(), float(eps),
+                                                reinterpret_cast<unsigned int*>(ctr.data_ptr()), f32, cur_stream()) == 0,
+                "channel_delta_decode: key heads of at most 256 columns, heads a multiple of the key heads", cuda_error());
+  });
+  m.def("head_norm_gate", [](const Tensor& o, const Tensor& gate, const Tensor& w, double eps, int64_t H, Tensor& out) {
+    const bool f32 = is_f32(o, "o");
+    same(gate, f32, "gate");
+    same(out, f32, "out");
+    const int64_t R = o.size(0), C = o.size(1);
+    TORCH_CHECK(H > 0 && C % H == 0 && gate.size(0) == R && gate.size(1) == C && out.size(0) == R && out.size(1) == C,
+                "head_norm_gate: o, gate and out [rows, heads * d]");
+    f32c(w, C / H, "norm weight");
+    c10::cuda::CUDAGuard guard(o.device());
+    TORCH_CHECK(lb::head_norm_gate_launch(o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), w.data_ptr<float>(),
+                                          float(eps), int(H), int(C / H), int(R), out.data_ptr(), out.stride(0), f32,
+                                          cur_stream()) == 0, "head_norm_gate failed", cuda_error());
   });
   m.def("sgemm", [](const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, const OptT& tok_scale,
                     const OptT& out_rows, int64_t n_feat, bool dual, int64_t dual_offset, int64_t act,
@@ -213,7 +406,7 @@ void bind_layers(pybind11::module_& m) {
   });
   m.def("paged_attn_general", [](const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
                                  const Tensor& ctx_lens, const Tensor& block_table, double scale, int64_t window,
-                                 Tensor& out) {
+                                 Tensor& out, double softcap) {
     const bool f32 = is_f32(q, "q");
     same(k_cache, f32, "k_cache");
     same(v_cache, f32, "v_cache");
@@ -228,8 +421,8 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::paged_attn_general_launch(q.data_ptr(), DK, k_cache.data_ptr(), v_cache.data_ptr(), Hkv * DK, Hkv * DV,
                                               cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
                                               int(block_table.stride(0)), int(k_cache.size(-3)), int(ctx_lens.numel()),
-                                              int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), int(window),
-                                              out.data_ptr(), f32, cur_stream()) == 0,
+                                              int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), float(softcap),
+                                              int(window), out.data_ptr(), f32, cur_stream()) == 0,
                 "paged_attn_general: value heads of at most 1024 columns, key heads of at most 2560", cuda_error());
   });
   m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
@@ -500,7 +693,7 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::paged_attn_general_launch(q_abs.data_ptr(), q_abs.size(2), cache.data_ptr(), cache.data_ptr(), cell, cell,
                                               cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
                                               int(block_table.stride(0)), int(cache.size(1)), int(ctx_lens.numel()), int(T),
-                                              int(H), 1, int(rank + rot), int(rank), float(scale), 0, out.data_ptr(), f32,
+                                              int(H), 1, int(rank + rot), int(rank), float(scale), 0.f, 0, out.data_ptr(), f32,
                                               cur_stream()) == 0,
                 "latent_attn_general: latents of at most 1024 columns", cuda_error());
   });

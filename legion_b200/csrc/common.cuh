@@ -32,6 +32,7 @@ enum : int {
   SITE_CHUNK_STATES = 4 << 8,
   SITE_CHUNK_SCORES = 5 << 8,
   SITE_CHUNK_OUTPUT = 6 << 8,
+  SITE_DELTA_SCAN = 7 << 8,
 };
 
 // Default deadline for in-kernel waits, in nanoseconds of %globaltimer.
@@ -291,6 +292,16 @@ __host__ __device__ constexpr uint32_t umma_idesc(uint32_t M, uint32_t N, uint32
          | (a_fmt << 7) | (b_fmt << 10)
          | (a_mn_major << 15) | (b_mn_major << 16)
          | ((N >> 3) << 17) | ((M >> 4) << 24);
+}
+
+// Soft cap of attention scores, cap * tanh(x / cap) = cap + 2 cap r with r = -1 / (1 + exp(2 x / cap)): a softmax does not
+// see the constant, so its kernels work on r with 2 cap in place of the score scale. k = 2 log2(e) scale / cap takes the raw
+// score in; about 2^-22 of the cap.
+__device__ __forceinline__ float softcap_r(float raw, float k) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * k));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return -r;
 }
 
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {

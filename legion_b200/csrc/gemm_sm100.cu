@@ -121,10 +121,11 @@ __device__ __forceinline__ float gate_act(float v, int act) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
 }
 
-// XIELU: the output passes xIELU with the two numbers of WgemmArgs::xielu. A variant of its own, as is the lookahead of
-// output rows for wide token tiles: decode-sized launches run the epilogue once, and code they skip still costs them
-// instruction fetches.
-template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false, bool XIELU = false>
+// UNARY: the output passes xIELU with the two numbers of WgemmArgs::xielu, or max(., 0)^2. Variants of their own, as is the
+// lookahead of output rows for wide token tiles: decode-sized launches run the epilogue once, and code they skip still
+// costs them instruction fetches.
+enum : int { UN_NONE = 0, UN_XIELU = 1, UN_RELU2 = 2 };
+template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false, int UNARY = UN_NONE>
 __global__ void __launch_bounds__(WFP4 ? 448 : 192, 1)
 wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
              const __grid_constant__ CUtensorMap tmS, const WgemmArgs a) {
@@ -586,7 +587,14 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               if (DUAL) u[j] *= gs1;
             }
           }
-          if constexpr (XIELU) {
+          if constexpr (UNARY == UN_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              const float p = fmaxf(g[j], 0.f);
+              g[j] = p * p;
+            }
+          }
+          if constexpr (UNARY == UN_XIELU) {
             const float xi_a = a.xielu[0], xi_b = a.xielu[1];
 #pragma unroll
             for (int j = 0; j < 32; ++j) g[j] = xielu_fast(g[j], xi_a, xi_b);
@@ -828,11 +836,11 @@ namespace {
 
 thread_local char g_gemm_err[512];
 
-template <int BN, bool DUAL, bool OUT_F32, bool WFP4 = false, bool WFP8 = false, bool XIELU = false>
+template <int BN, bool DUAL, bool OUT_F32, bool WFP4 = false, bool WFP8 = false, int UNARY = UN_NONE>
 int launch(const CUtensorMap* tmW, const CUtensorMap* tmX, const CUtensorMap* tmS, const WgemmArgs& a, int grid,
            cudaStream_t stream) {
   using Cfg = WgemmCfg<BN, DUAL, WFP4, WFP8>;
-  auto kfn = wgemm_kernel<BN, DUAL, OUT_F32, WFP4, WFP8, XIELU>;
+  auto kfn = wgemm_kernel<BN, DUAL, OUT_F32, WFP4, WFP8, UNARY>;
   static bool attr_set = false;  // per instantiation
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
@@ -950,8 +958,8 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
       h.n_out_peer == 0)
     a.vec_ok = 1;
   if (h.q8_out) a.vec_ok = 1;     // the encoded rows always leave through the staged write-out
-  if (h.xielu && (h.dual || fp4 || fp8 || h.out_f32)) {
-    snprintf(g_gemm_err, sizeof(g_gemm_err), "wgemm: xIELU comes with bf16 weights and bf16 output, one weight tile");
+  if ((h.xielu || h.relu2) && (h.dual || fp4 || fp8 || h.out_f32 || (h.xielu && h.relu2))) {
+    snprintf(g_gemm_err, sizeof(g_gemm_err), "wgemm: unary activations come with bf16 weights and bf16 output, one weight tile");
     return 1;
   }
   const int num_kb = fp8 ? h.K / 128 : (h.K + BK - 1) / BK;
@@ -973,7 +981,8 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
       if constexpr (BN_ <= 64) return launch<BN_, DUAL_, false, false, true>(tmW, tmX, tmS, a, grid, stream); \
     }                                                                                           \
     if constexpr (!DUAL_) {                                                                     \
-      if (h.xielu) return launch<BN_, false, false, false, false, true>(tmW, tmX, tmS, a, grid, stream); \
+      if (h.xielu) return launch<BN_, false, false, false, false, UN_XIELU>(tmW, tmX, tmS, a, grid, stream); \
+      if (h.relu2) return launch<BN_, false, false, false, false, UN_RELU2>(tmW, tmX, tmS, a, grid, stream); \
     }                                                                                           \
     return h.out_f32 ? launch<BN_, DUAL_, true>(tmW, tmX, tmS, a, grid, stream)                 \
                      : launch<BN_, DUAL_, false>(tmW, tmX, tmS, a, grid, stream);               \

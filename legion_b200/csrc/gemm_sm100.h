@@ -61,7 +61,7 @@ struct WgemmArgs {
                                   //   projections read their head's slice of a [tokens, heads * width] tensor in place)
   int dual_offset;                // DUAL: rows from a feature's gate row to its up row
   int act;                        // DUAL: activation of the gate, 0 = silu, 1 = gelu (tanh form)
-  const float* xielu;             // not DUAL: the output passes xIELU with these two numbers (act_type.cuh); may be null
+  const float* xielu;             // not DUAL, xIELU variant: its two numbers (act_type.cuh)
   int split_k;
   int vec_ok;                     // output rows may be written as aligned 16-byte vectors
   float* ws;                      // split-K partials
@@ -88,7 +88,8 @@ struct WgemmHost {
   const int* out_rows;
   int K, n_feat, n_tok;
   int bn; bool dual; int act;
-  const float* xielu;
+  const float* xielu;             // not dual: the output passes xIELU with these two numbers (null: not)
+  bool relu2;                     // not dual: the output is max(., 0)^2
   const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles_dev;
   const int* tile_out0;
   int n_tok_tiles_max;

@@ -4,8 +4,9 @@
 //   X'_t = sum_s mix[s, t] X_s + out[t] * y                      (all streams at once from the old ones)
 //   u    = sum_t in[t] X'_t,   h = u / sqrt(mean(u^2) + eps) * (w_offset + w)
 // so the stream update, the next sublayer's input mix and its norm read and write the streams once. The first launch of
-// a step starts from the embedding rows instead (X_s = embedding for every s). One CTA per token; u is kept in shared
-// memory between the sum of squares and the write of h.
+// a step starts from the embedding rows instead (X_s = embedding for every s), normed first where a model has that. One CTA
+// per token; u is kept in shared memory between the sum of squares and the write of h. With one stream, no mix weights and
+// y scaled, this is the pre-norm residual step x + m y; without y only the norm.
 #include "act_type.cuh"
 #include "common.cuh"
 #include "layers.h"
@@ -24,10 +25,10 @@ __global__ void __launch_bounds__(256) hyper_kernel(const HyperArgs a) {
   const int H = a.H, Sr = a.S, nt = blockDim.x;
   for (int i = threadIdx.x; i < S * S; i += nt) {
     const int f = i / S, to = i % S;
-    mix_s[i] = (!START && f < Sr && to < Sr) ? a.mix[f * Sr + to] : 0.f;
+    mix_s[i] = (!START && f < Sr && to < Sr) ? (a.mix ? a.mix[f * Sr + to] : float(f == to)) : 0.f;
   }
   if (threadIdx.x < S) {
-    out_s[threadIdx.x] = (!START && threadIdx.x < Sr) ? a.out_w[threadIdx.x] : 0.f;
+    out_s[threadIdx.x] = (!START && threadIdx.x < Sr) ? (a.out_w ? a.out_w[threadIdx.x] : 1.f) : 0.f;
     in_s[threadIdx.x] = threadIdx.x < Sr ? (a.in_w ? a.in_w[threadIdx.x] : 1.f) : 0.f;
   }
   __syncthreads();
@@ -43,11 +44,32 @@ __global__ void __launch_bounds__(256) hyper_kernel(const HyperArgs a) {
   const float* xi = START ? nullptr : a.x_in + long(t) * Sr * H;
   float* xo = a.x_out + long(t) * Sr * H;
   float ss = 0.f;
+  float pre_inv = 1.f;
+  if (START && a.pre_w) {
+    float es = 0.f;
+    for (int d = threadIdx.x * VEC; d < H; d += nt * VEC) {
+      float e[VEC];
+      ld_vec<VEC>(er + d, e);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) es = fmaf(e[j], e[j], es);
+    }
+    es = warp_sum_f(es);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = es;
+    __syncthreads();
+    es = 0.f;
+    for (int i = 0; i < nt / 32; ++i) es += red[i];
+    pre_inv = 1.f / sqrtf(es / float(H) + a.eps);
+    __syncthreads();
+  }
   for (int d = threadIdx.x * VEC; d < H; d += nt * VEC) {
     float xn[S][VEC];
     if constexpr (START) {
       float e[VEC];
       ld_vec<VEC>(er + d, e);
+      if (a.pre_w) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) e[j] = e[j] * pre_inv * (a.w_offset + a.pre_w[d + j]);
+      }
 #pragma unroll
       for (int s = 0; s < S; ++s)
 #pragma unroll
@@ -57,16 +79,20 @@ __global__ void __launch_bounds__(256) hyper_kernel(const HyperArgs a) {
 #pragma unroll
       for (int s = 0; s < S; ++s)
         if (s < Sr) ld_vec<VEC>(xi + long(s) * H + d, xv[s]);
-      const T* y0 = static_cast<const T*>(a.y0) + long(t) * a.y_rows * a.ldy0 + d;
-      ld_vec<VEC>(y0, y);
-      for (int r = 1; r < a.y_rows; ++r) {
-        float yr[VEC];
-        ld_vec<VEC>(y0 + r * a.ldy0, yr);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) y[j] += yr[j];
+      for (int j = 0; j < VEC; ++j) y[j] = 0.f;
+      if (a.y0) {
+        const T* y0 = static_cast<const T*>(a.y0) + long(t) * a.y_rows * a.ldy0 + d;
+        ld_vec<VEC>(y0, y);
+        for (int r = 1; r < a.y_rows; ++r) {
+          float yr[VEC];
+          ld_vec<VEC>(y0 + r * a.ldy0, yr);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) y[j] += yr[j];
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] *= a.c0;
       }
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) y[j] *= a.c0;
       if (a.y1) {
         ld_vec<VEC>(static_cast<const T*>(a.y1) + long(t) * a.ldy1 + d, y1);
 #pragma unroll
@@ -100,7 +126,9 @@ __global__ void __launch_bounds__(256) hyper_kernel(const HyperArgs a) {
       ss = fmaf(u[j], u[j], ss);
       u_s[d + j] = u[j];
     }
+    if (a.raw) st_vec<VEC>(static_cast<T*>(a.raw) + long(t) * a.ldraw + d, u);
   }
+  if (!a.h) return;
   ss = warp_sum_f(ss);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
@@ -134,7 +162,7 @@ int launch_s(const HyperArgs& a, cudaStream_t s) {
 bool vec4_ok(const HyperArgs& a, size_t es) {
   auto al = [&](const void* p, size_t n) { return p == nullptr || reinterpret_cast<uintptr_t>(p) % n == 0; };
   return a.H % 4 == 0 && al(a.x_in, 16) && al(a.x_out, 16) && al(a.emb, 4 * es) && al(a.y0, 4 * es) &&
-         al(a.y1, 4 * es) && al(a.h, 4 * es) && a.ld_emb % 4 == 0 && a.ldy0 % 4 == 0 && a.ldy1 % 4 == 0 && a.ldh % 4 == 0;
+         al(a.y1, 4 * es) && al(a.h, 4 * es) && al(a.raw, 4 * es) && a.ldraw % 4 == 0 && a.ld_emb % 4 == 0 && a.ldy0 % 4 == 0 && a.ldy1 % 4 == 0 && a.ldh % 4 == 0;
 }
 
 template <typename T>

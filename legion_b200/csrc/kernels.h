@@ -32,14 +32,15 @@ int attn_combine_launch(const float* o_part, const float* ml_part, int n_splits,
 // Value heads may have a size of their own (dk, dv: multiples of 8 up to 256); k_cell / v_cell: elements between cells
 int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                            long v_cell, const int* block_table, int table_width, int page, const int* ctx_lens,
-                           float scale, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits, float* o_part,
-                           float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status, cudaStream_t s);
+                           float scale, float softcap, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits,
+                           float* o_part, float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status,
+                           cudaStream_t s);
 const char* paged_decode_tc_last_error();
 
 int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                         long v_cell, const int* cu_q, const int* ctx_lens, const int* block_table, int table_width,
-                        int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, int window,
-                        int causal, void* out, int* status, cudaStream_t s);
+                        int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, float softcap,
+                        int window, int causal, void* out, int* status, cudaStream_t s);
 const char* prefill_attn_last_error();
 
 // Latent attention (absorbed form) over the paged latent cache: attn_mla_sm100.cu
@@ -55,8 +56,8 @@ int mla_prep_launch(const void* kva, long ld_kva, const float* norm_w, float eps
                     cudaStream_t s);
 
 int router_topk_launch(const float* logits, long ldl, const float* bias, int E, int k, int mode, int renorm,
-                       float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts, int T,
-                       cudaStream_t s);
+                       float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts,
+                       float* gate, int T, cudaStream_t s);   // gate: sigmoid of the logit behind the experts', or nullptr
 
 int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float eps, float w_offset, void* x_normed,
                            long ldn, const void* w, long ldw, int H, float* logits, const float* bias, int E, int k,
@@ -64,7 +65,7 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
                            int* ids, float* wts,
                            int T, int bn, int* tile_group, int* slot_base, int* tile_ntok, int* meta, int* out_rows,
                            float* tok_scale, unsigned int* done_ctr, int e_lo, int n_local, const void* sh_gate_w, float* sh_logit,
-                           int shared_slot, int* status, int* active, cudaStream_t s);
+                           int shared_slot, int shared_rows, int* status, int* active, cudaStream_t s);
 int moe_plan_gather_small_launch(const int* ids, const float* wts, int n_tokens, int k, int e_lo, int n_local, int bn,
                                  int* counts, int* offsets, int* sorted_token, int* sorted_pair, float* sorted_w,
                                  int* tile_group, int* tile_tok0, int* tile_ntok, int max_tiles, int* meta,

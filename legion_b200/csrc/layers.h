@@ -10,17 +10,20 @@ namespace lb {
 // Hyper-connections with static weights (hyper.cu). X [rows, S, H] fp32.
 struct HyperArgs {
   const float* x_in;               // streams before the sublayer; nullptr: every stream starts as the embedding row
+                                   // (normed with pre_w, if given)
   float* x_out;                    // streams after it (may be x_in)
   const void* emb; const int* ids; // start: embedding table and token ids (ids == nullptr: row t of emb)
   long ld_emb; int vocab;
   const void* y0; long ldy0; float c0;   // sublayer output: c0 * (sum of y_rows consecutive rows of y0) + c1 * y1
   const void* y1; long ldy1; float c1;
   int y_rows;
-  const float* mix;                // [S from, S to]
-  const float* out_w;              // [S]
+  const float* mix;                // [S from, S to]; nullptr: identity
+  const float* out_w;              // [S]; nullptr: all ones
   const float* in_w;               // [S] weights of the next sublayer's input (nullptr: all ones)
   const float* norm_w; float eps, w_offset;
-  void* h; long ldh;               // norm of the next input, activation type
+  void* h; long ldh;               // norm of the next input, activation type; nullptr: none
+  const float* pre_w;              // start: norm of the embedding rows, nullptr: none
+  void* raw; long ldraw;           // next input without the norm, activation type; nullptr: none
   int rows, S, H;
 };
 int hyper_launch(const HyperArgs& a, bool f32, cudaStream_t s);
@@ -140,12 +143,55 @@ int sgemm_launch(const SgemmArgs& a, bool f32, cudaStream_t s);
 int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld, const float* qw, const float* kw,
                            float eps, const long* slots, void* q_out, void* k_cache, void* v_cache, long k_cell,
                            long v_cell, int T, int Hq, int Hkv, int DK, int DV, bool f32, cudaStream_t s);
+// What lies between a q | k | v projection and the scores (qkv_conv.cu): bias, short causal convolution with carried
+// history, RMS norm of q and k over each head or the whole, rotation, append of k and v. All but the append optional.
+struct QkvConvArgs {
+  const void* x; long ld;          // [T, Hq * DK | Hkv * DK | Hkv * DV]
+  const float* in_b;               // [columns]; the history holds x + in_b
+  const float* conv_w; int KC;     // [columns, KC]; nullptr: none
+  float* conv_state;               // [slots, columns, KC - 1]
+  const int* cu; const int* state_slots; int n_seqs;
+  const float* qw; const float* kw; int norm_all; float eps;   // weights [DK], or [Hq * DK] / [Hkv * DK] with norm_all
+  const float* cos_sin; int rot; int rot_half;                 // [positions, rot]; rot_half: column i turns with i + rot / 2
+  const int* positions; const long* slots;
+  void* q_out; void* k_cache; void* v_cache; long k_cell, v_cell;
+  int T, Hq, Hkv, DK, DV;
+  int max_len;                     // longest sequence of the step
+  int write_state;
+  int tok, one;                    // set by the launcher: tokens per CTA; every sequence has one token
+};
+int qkv_conv_append_launch(QkvConvArgs a, bool f32, cudaStream_t s);
+
+// Gated delta rule with a decay per key channel (channel_delta.cu)
+struct ChannelDeltaArgs {
+  const void* qkv; long ld;        // [T, G * DK | G * DK | H * DV] in front of the convolution
+  const float* conv_w; int KC; float* conv_state;              // [columns, KC], [slots, columns, KC - 1]
+  const void* a; long lda;         // [T, H * DK]: decay exp(A softplus(a + dt_bias))
+  const float* A; const float* dt_bias;                        // [H], [H * DK]
+  const void* b; long ldb;         // [T, H]: beta = sigmoid(b)
+  float* state;                    // [slots, H, DV, DK]
+  const int* cu; const int* slots;
+  int n_seqs, T, H, G, DK, DV;
+  float scale, l2_eps;
+  void* out; long ldo;             // [T, H * DV]
+  int write_state;
+};
+// floats of scratch per four tokens (and per sequence); rec: 128-byte aligned, for at least n_seqs + 1 of them
+long channel_delta_record_floats(int H, int DK, int DV);
+int channel_delta_launch(const ChannelDeltaArgs& a, float* rec, long rec_floats, int* status, bool f32, cudaStream_t s);
+// One decode step with the norm per head (times norm_w, times sigmoid(gate)) behind it; ctr: [n_seqs, G] zeroed arrival
+// counters, left zero
+int channel_delta_decode_launch(const ChannelDeltaArgs& a, const void* gate, long ldg, const float* norm_w, float eps,
+                                unsigned int* ctr, bool f32, cudaStream_t s);
+int head_norm_gate_launch(const void* o, long ldo, const void* gate, long ldg, const float* w, float eps, int H, int D, int rows,
+                          void* out, long ldout, bool f32, cudaStream_t s);
+
 // Paged causal attention on FMA units, one warp per (token, query head); value heads up to 1024 wide; q_row: elements
 // between query heads
 int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
-                              int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, int window, void* out,
-                              bool f32, cudaStream_t s);
+                              int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, float softcap, int window,
+                              void* out, bool f32, cudaStream_t s);
 
 // Decayed outer-product state S_t = a_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (linear_scan.cu, linear_scan_sm100.cu).
 struct LinScanArgs {

@@ -16,6 +16,7 @@ namespace lb {
 // mode 1: sigmoid scores, selection by score + bias, optional group-limited routing (n_group groups,
 // keep topk_group groups ranked by the sum of their group_top (1 or 2) best biased scores), weights = unbiased
 // scores of the chosen experts, renormalised and multiplied by route_scale. mode 2: as mode 1 with softmax scores.
+// renorm 1: by the sum of the chosen weights, held away from zero; 2: by the sum + 1e-20.
 template <int MAXE>
 __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, const float* __restrict__ bias, int E,
                                                 int k, int mode, int renorm, float route_scale, int n_group,
@@ -160,7 +161,7 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) wsum += __shfl_xor_sync(0xffffffffu, wsum, o);
   if (lane < k) {
-    if (renorm) w = w / fmaxf(wsum, 6.1e-5f);
+    if (renorm) w = w / (renorm == 2 ? wsum + 1e-20f : fmaxf(wsum, 6.1e-5f));
     ids[t * k + lane] = my_id;
     wts[t * k + lane] = w * route_scale;
     if (sm_ids) {     // copy for a caller that goes on working on the selection in shared memory
@@ -175,10 +176,12 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
                                                           const float* __restrict__ bias, int E, int k, int mode,
                                                           int renorm, float route_scale, int n_group, int topk_group,
                                                           int group_top, int* __restrict__ ids,
-                                                          float* __restrict__ wts, int T) {
+                                                          float* __restrict__ wts, float* __restrict__ gate, int T) {
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   if (t >= T) return;
   router_topk_row<MAXE>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group, topk_group, group_top, ids, wts, t);
+  // the logit behind the experts' gates the shared expert
+  if (gate && (threadIdx.x & 31) == 0) gate[t] = 1.f / (1.f + __expf(-logits[t * ldl + E]));
 }
 
 // Decode-sized MoE front end in ONE launch (T <= 64 tokens, T * k <= 1024 pairs):
@@ -206,7 +209,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
     int topk_group, int group_top, int* ids, float* wts, int T, int bn, int* __restrict__ tile_group, int* __restrict__ slot_base,
     int* __restrict__ tile_ntok, int* __restrict__ meta, int* __restrict__ out_rows, float* __restrict__ tok_scale,
     unsigned int* done_ctr, int e_lo, int n_local, const __nv_bfloat16* __restrict__ sh_gate_w, float* sh_logit,
-    int shared_slot, int epc, int tpp, int ksplit, int* status, int* __restrict__ active) {
+    int shared_slot, int shared_rows, int epc, int tpp, int ksplit, int* status, int* __restrict__ active) {
   extern __shared__ uint4 xs_rows[];          // [tpp][H / 8 / ksplit] this CTA's columns of the pass's token rows
   __shared__ int s_last;
   __shared__ float s_logit[512];
@@ -465,7 +468,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) wsum += __shfl_xor_sync(0xffffffffu, wsum, o);
       if (lane < k) {
-        if (renorm) w = w / fmaxf(wsum, 6.1e-5f);
+        if (renorm) w = w / (renorm == 2 ? wsum + 1e-20f : fmaxf(wsum, 6.1e-5f));
         ids[t * k + lane] = my_id;
         wts[t * k + lane] = w * route_scale;
       }
@@ -475,13 +478,13 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
   // ---- dense routing tables, indexed by local expert: rows e * bn + t of the intermediate belong to expert e and
   // token t. Each token CTA writes its token's column of out_rows / tok_scale (pair index t * k + c where the
   // token chose the expert, -1 elsewhere) and marks the experts it chose as active.
-  const int P = T * k;
+  const int P = T * k, kp = k + shared_rows;
   for (int t = blockIdx.x; t < T; t += gridDim.x) {
     s_chosen[tid] = -1;
     __syncthreads();
     if (tid < k) {
       const int e = ids[t * k + tid];                   // written by this CTA above
-      s_chosen[e] = t * k + tid;
+      s_chosen[e] = t * kp + tid;
       s_logit[e] = wts[t * k + tid];
     }
     __syncthreads();
@@ -494,14 +497,16 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
         active[local] = 1;
       }
     }
-    if (shared_slot && tid == 0) {
+    if (tid < shared_rows || (shared_slot && tid == 0)) {
       // the shared expert (stacked behind this rank's routed experts as group n_local) is used by every token:
       // its output rows are the pairs P .. P + T - 1, weighted by the sigmoid of its gate (or 1)
-      out_rows[n_local * bn + t] = P + t;
+      // (shared_rows: the shared expert as that many groups, its output rows behind the token's own pairs)
+      const int slot = n_local + (shared_rows ? tid : 0);
+      out_rows[slot * bn + t] = shared_rows ? t * kp + k + tid : P + t;
       float gl = 0.f;
       if (sh_gate_w)
         for (int sp = 0; sp < ksplit; ++sp) gl += __ldcg(&sh_logit[sp * 64 + t]);
-      tok_scale[n_local * bn + t] = sh_gate_w ? 1.f / (1.f + __expf(-gl)) : 1.f;
+      tok_scale[slot * bn + t] = sh_gate_w ? 1.f / (1.f + __expf(-gl)) : 1.f;
     }
     __syncthreads();
   }
@@ -535,12 +540,13 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
     tile_ntok[slot] = T;
   }
   if (tid == 0) {
-    if (shared_slot) {
-      tile_group[n_active] = n_local;
-      slot_base[n_active] = n_local * bn;
-      tile_ntok[n_active] = T;
+    const int n_shared = shared_rows ? shared_rows : (shared_slot ? 1 : 0);
+    for (int i = 0; i < n_shared; ++i) {
+      tile_group[n_active + i] = n_local + i;
+      slot_base[n_active + i] = (n_local + i) * bn;
+      tile_ntok[n_active + i] = T;
     }
-    const int n_slots = n_active + (shared_slot ? 1 : 0);
+    const int n_slots = n_active + n_shared;
     meta[0] = n_slots;
     meta[1] = n_slots * bn;
   }
@@ -551,10 +557,11 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
                            int mode, int renorm, float route_scale, int n_group, int topk_group, int group_top,
                            int* ids, float* wts, int T, int bn, int* tile_group, int* slot_base, int* tile_ntok, int* meta, int* out_rows,
                            float* tok_scale, unsigned int* done_ctr, int e_lo, int n_local, const void* sh_gate_w,
-                           float* sh_logit, int shared_slot, int* status, int* active, cudaStream_t s) {
+                           float* sh_logit, int shared_slot, int shared_rows, int* status, int* active, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (k > 32 || E > 512 || n_group > 32 || H % 8 || T > 64 || T * k > 1024 || T > bn) return 1;
-  if (sh_gate_w && (!sh_logit || !shared_slot)) return 1;
+  if (k > 32 || E > 512 || n_group > 32 || H % 8 || T > 64 || T * k > 1024 || T > bn || shared_rows < 0 || shared_rows > 64)
+    return 1;
+  if (sh_gate_w && (!sh_logit || !(shared_slot || shared_rows))) return 1;
   auto sg = static_cast<const __nv_bfloat16*>(sh_gate_w);
   auto xb = static_cast<const __nv_bfloat16*>(x);
   auto xn = static_cast<__nv_bfloat16*>(x_normed);
@@ -580,7 +587,7 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
     launch_pdl(moe_route_small_kernel<MAXE>, dim3(grid), dim3(512), smem, s, xb, ldx, norm_w, eps, w_offset, xn,   \
                ldn, wb, ldw, H, logits, bias, E, k, mode, renorm, route_scale, n_group, topk_group, group_top, ids, wts, T, \
                bn, tile_group, slot_base, tile_ntok, meta, out_rows, tok_scale, done_ctr, e_lo, n_local, sg,        \
-               sh_logit, shared_slot, epc, tpp, ksplit, status, active);                                                    \
+               sh_logit, shared_slot, shared_rows, epc, tpp, ksplit, status, active);                                                    \
   }
   if (E <= 128) LB_ROUTE(128)
   else if (E <= 256) LB_ROUTE(256)
@@ -590,20 +597,20 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
 }
 
 int router_topk_launch(const float* logits, long ldl, const float* bias, int E, int k, int mode, int renorm,
-                       float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts, int T,
-                       cudaStream_t s) {
+                       float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts, float* gate,
+                       int T, cudaStream_t s) {
   if (T <= 0) return 0;
   if (k > 32 || E > 512 || n_group > 32) return 1;
   const int blocks = (T * 32 + 127) / 128;
   if (E <= 128)
     router_topk_kernel<128><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, group_top, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, gate, T);
   else if (E <= 256)
     router_topk_kernel<256><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, group_top, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, gate, T);
   else
     router_topk_kernel<512><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,
-                                                   topk_group, group_top, ids, wts, T);
+                                                   topk_group, group_top, ids, wts, gate, T);
   return cudaGetLastError() != cudaSuccess;
 }
 

@@ -1133,11 +1133,11 @@ class Decoder:
             return [(ops.linear(ops.up_act(h, w[f"{p}.mlp.up"], w[f"{p}.mlp.act"]), w[f"{p}.mlp.down"]), 1.0)]
         if f.kind == "dense":
             return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act), w[f"{p}.mlp.down"]), 1.0)]
-        routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, f.scale, w.get(f"{p}.moe.router_bias"),
-                             f.n_group, f.keep_group, n_local=f.experts, group_top=f.group_top, gate_row=f.shared_gate,
-                             shared_slots=f.shared_slots())
-        ids, wts = routing
         up, down, E = w[f"{p}.moe.gate_up"], w[f"{p}.moe.down"], f.experts
+        routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, f.scale, w.get(f"{p}.moe.router_bias"),
+                             f.n_group, f.keep_group, n_local=E, group_top=f.group_top, gate_row=f.shared_gate,
+                             shared_slots=f.shared_slots(), dense=ops.sm100.tma_ok(h, up, down))
+        ids, wts = routing
         if f.shared_ff and routing.dense is None:
             # the shared expert as a dense feed-forward part of its own (decode steps: a slot of the grouped products)
             sd = self._shared_down.get(p)

@@ -167,6 +167,9 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, shared
     if _cuda(x) and isinstance(w_gate_up, torch.Tensor) and not _sm.tma_ok(x, w_gate_up, w_down):
         return _sm.moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act, e_lo, shared, shared_gate, residual, norm,
                                      defer_combine)
+    if _cuda(x) and act == "relu2" and defer_combine == "pairs" and isinstance(w_gate_up, torch.Tensor):
+        return _sm.moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo, None, shared, shared_gate, residual, out, norm,
+                               routing if isinstance(routing, _sm.Routing) else None, defer_combine=defer_combine, act=act)
     if _cuda(x) and act != "silu":
         if act not in ("relu2", "gelu_tanh") or not isinstance(w_gate_up, torch.Tensor):
             raise NotImplementedError("the grouped expert kernels implement SwiGLU experts (squared-ReLU and GELU "

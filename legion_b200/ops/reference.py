@@ -295,7 +295,9 @@ def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm,
     n_kv, dk, dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
     T, nq, nk = proj.shape[0], heads * dk, n_kv * dk
     u = proj.float() if in_b is None else proj.float() + in_b
-    if conv_w is not None:
+    if conv_w is not None and conv_w.shape[1] == 1:
+        u = u * conv_w[:, 0]
+    elif conv_w is not None:
         u = causal_conv1d_silu(u, conv_w, None, conv_state, cu_seq, state_slots, write_state, None, False)
     q, k, v = u[:, :nq], u[:, nq:nq + nk], u[:, nq + nk:nq + nk + n_kv * dv]
     if q_norm is not None and norm_over == "all":

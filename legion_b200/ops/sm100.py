@@ -594,6 +594,7 @@ def _linear_fp8(x, w: "Fp8Weight", residual, out, dual: bool, n_feat: int):
 
 
 ROUTER_MODES = {"softmax": 0, "sigmoid": 1, "softmax_bias": 2}
+RENORM = {False: 0, True: 1, "sum": 2}       # see config.MoeSpec.renorm
 GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
 
 
@@ -604,14 +605,14 @@ def tma_ok(*ts) -> bool:
 
 
 def sgemm(x, w, residual=None, out=None, out_dtype=None, dual: bool = False, n_ff: int = 0, act: str = "silu",
-          act_ab=None):
+          act_ab=None, unary: Optional[str] = None, tok_scale=None):
     """x @ w^T in fp32 arithmetic on the FMA units: fp32 models and shapes outside the tcgen05 GEMM's alignment rules.
     ``dual``: act(x Wg^T) * (x Wu^T) with Wg = w[:n_ff], Wu = w[n_ff:]."""
     T, N = x.shape[0], (n_ff if dual else w.shape[0])
     if out is None:
         out = torch.empty(T, N, dtype=out_dtype or x.dtype, device=x.device)
-    ext().sgemm(w, x, out, residual, None, None, N, dual, n_ff if dual else 0,
-                3 if act_ab is not None else GATE_ACTS[act] if dual else 0, None, None, None, None, 0, 0, T, act_ab)
+    ext().sgemm(w, x, out, residual, tok_scale, None, N, dual, n_ff if dual else 0,
+                3 if act_ab is not None else GATE_ACTS[unary] if unary else GATE_ACTS[act] if dual else 0, None, None, None, None, 0, 0, T, act_ab)
     return out
 
 
@@ -620,13 +621,14 @@ def up_act(x, w, ab):
     return linear(x, w, out_dtype=x.dtype, xielu=ab)
 
 
-def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Optional[int] = None, bn=None, xielu=None):
-    """out[T, N] = x[T, K] @ w[N, K]^T (+ residual)."""
+def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Optional[int] = None, bn=None, xielu=None,
+           unary: Optional[str] = None, tok_scale=None):
+    """out[T, N] = x[T, K] @ w[N, K]^T (+ residual). ``unary``: "relu2"; ``tok_scale`` (float32): a factor per row."""
     C = ext()
     if isinstance(w, torch.Tensor) and isinstance(x, torch.Tensor) and not tma_ok(x, w):
-        return sgemm(x, w, residual, out, out_dtype, act_ab=xielu)
-    if xielu is not None and not isinstance(w, torch.Tensor):
-        raise ValueError("xIELU runs in the epilogue of bf16 and fp32 weights")
+        return sgemm(x, w, residual, out, out_dtype, act_ab=xielu, unary=unary, tok_scale=tok_scale)
+    if (xielu is not None or unary is not None or tok_scale is not None) and not isinstance(w, torch.Tensor):
+        raise ValueError("activations and row factors run in the epilogue of bf16 and fp32 weights")
     if isinstance(x, Fp8Act) and not isinstance(w, Fp8Weight):
         x = x.x
     T, K = x.shape
@@ -655,9 +657,9 @@ def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Opt
         need = C.wgemm_workspace_floats(bn, False, n_tt, ft, sk)
         if need > ws.splitk.numel() or n_tt * ft > ws.counters.numel():
             sk = 1
-    C.wgemm(w.codes if q else w, x, out, residual, None, None, N, False, 0, bn, sk, ws.splitk if sk > 1 else None,
+    C.wgemm(w.codes if q else w, x, out, residual, tok_scale, None, N, False, 0, bn, sk, ws.splitk if sk > 1 else None,
             ws.counters if sk > 1 else None, ws.status, None, None, None, None, 0, 0, T, [], None,
-            w.scales if q else None, w.gscale if q else None, xielu=xielu)
+            w.scales if q else None, w.gscale if q else None, xielu=xielu, relu2=unary == "relu2")
     return out
 
 
@@ -748,7 +750,7 @@ def decode_splits(batch: int, n_kv_heads: int, g_tiles: int, max_ctx: int, head_
 
 
 def paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window=0, n_splits=None, max_ctx=None, out=None,
-                 impl="tc"):
+                 impl="tc", softcap=0.0):
     C = ext()
     B, Hq, _ = q.shape
     Hkv, D = k_cache.shape[2], v_cache.shape[3]
@@ -764,16 +766,18 @@ def paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window=0, n_
     if out is None:
         out = torch.empty(B, Hq, D, dtype=q.dtype, device=q.device)
     C.paged_decode(q, k_cache, v_cache, block_table, ctx_lens, scale, window, n_splits, o_part, ml_part, out,
-                   impl == "tc", ws.status, ws.counters)
+                   impl == "tc", ws.status, ws.counters, float(softcap))
     return out
 
 
-def prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window=0, causal=True, out=None):
+def prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window=0, causal=True, out=None,
+                 softcap=0.0):
     C = ext()
     if out is None:
         out = torch.empty(q.shape[0], q.shape[1], v_cache.shape[3], dtype=q.dtype, device=q.device)
     ws = Workspace.get(q.device)
-    C.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal, out, ws.status)
+    C.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal, out, ws.status,
+                   float(softcap))
     return out
 
 
@@ -784,13 +788,13 @@ def attn_tc_ok(q, k_cache, v_cache) -> bool:
             and 64 % page == 0)
 
 
-def paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window=0, causal=True, out=None):
+def paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window=0, causal=True, out=None, softcap=0.0):
     """Paged causal attention for fp32 and for head sizes outside the tensor-core kernels (prompts and decode rows)."""
     if not causal:
         raise NotImplementedError("the general attention kernel is causal")
     if out is None:
         out = torch.empty(q.shape[0], q.shape[1], v_cache.shape[3], dtype=q.dtype, device=q.device)
-    ext().paged_attn_general(q, k_cache, v_cache, cu_q, ctx_lens, block_table, scale, window, out)
+    ext().paged_attn_general(q, k_cache, v_cache, cu_q, ctx_lens, block_table, scale, window, out, float(softcap))
     return out
 
 
@@ -1042,13 +1046,15 @@ def latent_values(o_lat, uv, gate):
 
 
 def router_topk(logits, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
-                ids=None, wts=None, group_top: int = 2):
+                ids=None, wts=None, group_top: int = 2, gate=None):
+    """``gate`` (float32 [T]) takes the sigmoid of the logits' last column, which then is no expert."""
     C = ext()
     T = logits.shape[0]
     if ids is None:
         ids = torch.empty(T, k, dtype=torch.int32, device=logits.device)
         wts = torch.empty(T, k, dtype=torch.float32, device=logits.device)
-    C.router_topk(logits, bias, k, ROUTER_MODES[mode], renorm, route_scale, n_group, topk_group, ids, wts, group_top)
+    C.router_topk(logits, bias, k, ROUTER_MODES[mode], RENORM[renorm], route_scale, n_group, topk_group, ids, wts, group_top,
+                  gate)
     return ids, wts
 
 
@@ -1097,22 +1103,31 @@ class DenseRoute:
 
 def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=None, n_group=1, topk_group=1,
            norm=None, e_lo: int = 0, n_local: Optional[int] = None, slot_stride: Optional[int] = None, sh_gate=None,
-           shared_slot: bool = False, group_top: int = 2):
+           shared_slot: bool = False, group_top: int = 2, gate_row: bool = False, shared_slots: int = 0,
+           dense: bool = True):
     """Router logits and top-k selection -> ``Routing``. Decode-sized steps (<= 64 tokens, <= 1024 pairs) run as
     ONE launch that also builds the dense routing tables; with ``norm=(weight, eps, w_offset)`` that launch first
     applies the RMSNorm to ``x`` (the raw residual stream) and ``Routing.x_normed`` is the normalised input.
     ``shared_slot``: the shared expert is stacked behind the local routed experts and gets a slot of its own that
     every token uses (weight sigmoid(x . sh_gate) when ``sh_gate`` [1, H] is given, else 1); its output rows are
-    the pairs T * k .. T * k + T - 1. Larger steps use the GEMM and the selection kernel."""
-    T, E = x.shape[0], w_router.shape[0]
-    small = T <= 64 and T * k <= 1024 and TUNE["fused_router"] and tma_ok(x, w_router)
+    the pairs T * k .. T * k + T - 1. Larger steps use the GEMM and the selection kernel. ``gate_row`` /
+    ``shared_slots``: the last row of ``w_router`` gates a shared expert stored as that many experts behind the routed ones;
+    decode-sized steps give each a slot whose output rows follow the token's own pairs, larger ones return the gate.
+    ``dense`` False: no dense tables (experts that do not run on the grouped GEMM)."""
+    T, E = x.shape[0], w_router.shape[0] - int(gate_row)
+    small = dense and T <= 64 and T * k <= 1024 and TUNE["fused_router"] and tma_ok(x, w_router)
     if not small:
         xn = None
         if norm is not None:
             xn, _ = rmsnorm(x, norm[0], norm[1], norm[2])
         logits = linear(x if xn is None else xn, w_router, out_dtype=torch.float32)
-        ids, wts = router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group, group_top=group_top)
-        return Routing(ids, wts, None, xn)
+        gate = torch.empty(T, dtype=torch.float32, device=x.device) if gate_row else None
+        ids, wts = router_topk(logits, k, mode, renorm, route_scale, bias, n_group, topk_group, group_top=group_top, gate=gate)
+        r = Routing(ids, wts, None, xn)
+        r.gate = gate
+        return r
+    if gate_row:
+        w_router, sh_gate = w_router[:E], w_router[E]
     C = ext()
     ws = Workspace.get(x.device)
     logits = ws.buf("router_logits", (4 * 64 * 512,), torch.float32)    # one plane per column split
@@ -1123,7 +1138,7 @@ def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
     bn = 32 if T <= 32 else 64
     stride = slot_stride or bn
     nl = E if n_local is None else n_local
-    n_slots = nl + (1 if shared_slot else 0)
+    n_slots = nl + (shared_slots or (1 if shared_slot else 0))
     dr = ws._cache.get(("dense_route", n_slots, bn, stride))
     if dr is None:
         dr = DenseRoute(n_slots, bn, x.device, stride)
@@ -1132,12 +1147,13 @@ def router(x, w_router, k, mode="softmax", renorm=True, route_scale=1.0, bias=No
     wts = torch.empty(T, k, dtype=torch.float32, device=x.device)
     xn = torch.empty_like(x) if norm is not None else None
     C.moe_route_small(x, norm[0] if norm else None, norm[1] if norm else 0.0, norm[2] if norm else 0.0, xn, w_router,
-                      bias, k, ROUTER_MODES[mode], renorm, route_scale, n_group, topk_group, logits, ids, wts,
+                      bias, k, ROUTER_MODES[mode], RENORM[renorm], route_scale, n_group, topk_group, logits, ids, wts,
                       stride, dr.tile_group, dr.slot_base, dr.tile_ntok, dr.meta, dr.out_rows, dr.tok_scale, ctr,
                       e_lo, nl, sh_gate.reshape(-1) if sh_gate is not None else None,
-                      dr.sh_logit if sh_gate is not None else None, bool(shared_slot), ws.status, dr.active, group_top)
+                      dr.sh_logit if sh_gate is not None else None, bool(shared_slot), ws.status, dr.active, group_top,
+                      shared_slots)
     r = Routing(ids, wts, dr, xn, e_lo, nl)
-    r.shared_slot = bool(shared_slot)
+    r.shared_slot, r.shared_rows = bool(shared_slot), shared_slots
     return r
 
 
@@ -1165,7 +1181,8 @@ class MoePlan:
 
 def _dense_ok(routing, n_groups: int, e_lo: int, ids) -> bool:
     return (routing is not None and routing.dense is not None and routing.e_lo == e_lo and routing.ids is ids
-            and routing.n_local + int(routing.shared_slot) == n_groups and bool(TUNE["dense_route"]))
+            and routing.n_local + (routing.shared_rows or int(routing.shared_slot)) == n_groups
+            and (routing.shared_rows > 0 or bool(TUNE["dense_route"])))
 
 
 def _dense_pairs(dr: DenseRoute, P: int, T: int, k: int, H: int, device):
@@ -1179,10 +1196,11 @@ class PendingCombine:
     """The weighted pair rows of a decode-sized MoE layer whose per-token sum has not run yet: the rank-partial
     result of an expert-parallel layer, handed to the reduction that follows so that it sums them inside its own
     launch (``parallel.symm.SymmComm.all_reduce_add_norm``). ``materialize`` runs the combine kernel instead."""
-    __slots__ = ("y", "ids", "e_lo", "e_hi", "shared", "T", "H")
+    __slots__ = ("y", "ids", "e_lo", "e_hi", "shared", "T", "H", "rows")
 
-    def __init__(self, y, ids, e_lo, e_hi, shared, T, H):
+    def __init__(self, y, ids, e_lo, e_hi, shared, T, H, rows=None):
         self.y, self.ids, self.e_lo, self.e_hi, self.shared, self.T, self.H = y, ids, e_lo, e_hi, shared, T, H
+        self.rows = rows or ids.shape[1]             # consecutive rows of ``y`` that make up a token
 
     def materialize(self, out=None):
         if out is None:
@@ -1332,12 +1350,12 @@ NV4_H_AMAX = 32.0
 
 def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[MoePlan] = None, shared=None,
                 shared_gate=None, residual=None, out=None, norm=None, routing: Optional[Routing] = None,
-                defer_combine: bool = False):
+                defer_combine: bool = False, act: str = "silu"):
     """Routed experts over the device routing plan: plan -> gather -> grouped gate/up (+SwiGLU) ->
     grouped down (x routing weight) -> combine (+ shared expert, + residual).
 
-    w_gate_up: [E_local, 2*n_ff, H]; w_down: [E_local, H, n_ff]; ids/wts: [T, k]. Returns bf16 [T, H]; with
-    ``norm=(weight, eps, w_offset)`` the combine also applies that RMSNorm and (out, normed) is returned."""
+    w_gate_up: [E_local, 2*n_ff, H] (``act`` "relu2": un-gated, [E_local, n_ff, H]); w_down: [E_local, H, n_ff]; ids/wts:
+    [T, k]. Returns bf16 [T, H]; with ``norm=(weight, eps, w_offset)`` the combine also applies that RMSNorm and (out, normed) is returned."""
     C = ext()
     T, H = x.shape
     k = ids.shape[1]
@@ -1359,6 +1377,10 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
         w_gate_up, w_down = w_gate_up.as_qweight(), w_down.as_qweight()
     if routing is not None and routing.shared_slot and not _dense_ok(routing, E_local, e_lo, ids):
         raise ValueError("the routing carries a shared-expert slot that these expert weights do not have")
+    gated = act != "relu2"
+    n_gu = (2 if gated else 1) * n_ff                # rows of an expert in w_gate_up
+    if routing is not None and routing.shared_rows and not _dense_ok(routing, E_local, e_lo, ids):
+        raise ValueError("the routing carries shared experts that these expert weights do not have")
     if routing is None or not routing.shared_slot:
         n_routed = E_local
     else:
@@ -1367,7 +1389,7 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
     if isinstance(w_gate_up, QWeight):
         (gu2, gu_sc), gu_gs = w_gate_up.view2d(), w_gate_up.gscale
     else:
-        gu2, gu_sc, gu_gs = w_gate_up.view(E_local * 2 * n_ff, H), None, None
+        gu2, gu_sc, gu_gs = w_gate_up.view(E_local * n_gu, H), None, None
     if isinstance(w_down, QWeight):
         (dn2, dn_sc), dn_gs = w_down.view2d(), w_down.gscale
     else:
@@ -1378,13 +1400,18 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
         P = T * k
         if dr.h_all is None or dr.h_all.shape[1] != n_ff:
             dr.h_all = torch.zeros(dr.n_slots * dr.stride, n_ff, dtype=torch.bfloat16, device=x.device)
-        y_pairs = _dense_pairs(dr, P, T, k, H, x.device)
-        C.wgemm(gu2, x, dr.h_all, None, None, None, n_ff, True, n_ff, dr.bn, 1,
-                None, None, ws.status, dr.tile_group, dr.zeros, dr.tile_ntok, dr.meta, dr.n_slots, 2 * n_ff, 0, [],
-                dr.slot_base, gu_sc, gu_gs)
+        kp = k + routing.shared_rows
+        y_pairs = _dense_pairs(dr, T * kp, T, kp, H, x.device)
+        C.wgemm(gu2, x, dr.h_all, None, None, None, n_ff, gated, n_ff if gated else 0, dr.bn, 1,
+                None, None, ws.status, dr.tile_group, dr.zeros, dr.tile_ntok, dr.meta, dr.n_slots, n_gu, 0, [],
+                dr.slot_base, gu_sc, gu_gs, relu2=not gated)
         C.wgemm(dn2, dr.h_all, y_pairs, None, dr.tok_scale, dr.out_rows, H, False, 0,
                 dr.bn, 1, None, None, ws.status, dr.tile_group, dr.slot_base, dr.tile_ntok, dr.meta, dr.n_slots, H, 0, [],
                 None, dn_sc, dn_gs)
+        if routing.shared_rows:
+            if not defer_combine or shared is not None or residual is not None or norm is not None:
+                raise NotImplementedError("shared experts among a token's pairs are summed by the step that follows")
+            return PendingCombine(y_pairs[:T * kp], ids, e_lo, e_lo + routing.n_local, None, T, H, kp)
         return _dense_combine(dr, routing, ids, e_lo, T, k, H, shared, shared_gate, residual, out, norm, x.device,
                               defer_combine)
     E_local = n_routed
@@ -1412,9 +1439,9 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
         C.moe_plan(ids, wts, e_lo, E_local, bn, plan.counts, plan.offsets, plan.sorted_token, plan.sorted_pair,
                    plan.sorted_w, plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta)
         C.gather_rows(x, plan.sorted_token, plan.meta[1:2], plan.x_sorted[:P])
-    C.wgemm(gu2, plan.x_sorted, plan.h_sorted, None, None, None, n_ff, True, n_ff, bn, 1, None, None, ws.status,
-            plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, 2 * n_ff, 0, [], None,
-            gu_sc, gu_gs)
+    C.wgemm(gu2, plan.x_sorted, plan.h_sorted, None, None, None, n_ff, gated, n_ff if gated else 0, bn, 1, None, None, ws.status,
+            plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, n_gu, 0, [], None,
+            gu_sc, gu_gs, relu2=not gated)
     C.wgemm(dn2, plan.h_sorted, plan.y_pairs, None, plan.sorted_w, plan.sorted_pair, H, False, 0, bn, 1, None, None,
             ws.status, plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, 0, [], None,
             dn_sc, dn_gs)
@@ -1434,9 +1461,11 @@ def moe_experts(x, ids, wts, w_gate_up, w_down, n_ff, e_lo=0, plan: Optional[Moe
 def moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, shared=None, shared_gate=None,
                       residual=None, norm=None, defer_combine=False):
     """Routed experts on the FMA units over the same routing plan (fp32 models, unaligned bf16 shapes; all experts
-    local, gated experts without a shared one). With ``defer_combine`` the weighted pair rows are handed on."""
-    if e_lo or shared is not None or residual is not None or norm is not None or w_gate_up.shape[1] != 2 * n_ff:
-        raise NotImplementedError("plain experts: gated, all local, no shared expert, residual or norm")
+    local, without a shared one). With ``defer_combine`` the weighted pair rows are handed on."""
+    gated = act != "relu2"
+    n_gu = (2 if gated else 1) * n_ff
+    if e_lo or shared is not None or residual is not None or norm is not None or w_gate_up.shape[1] != n_gu:
+        raise NotImplementedError("plain experts: all local, no shared expert, residual or norm")
     C = ext()
     T, H = x.shape
     k, E = ids.shape[1], w_gate_up.shape[0]
@@ -1451,8 +1480,8 @@ def moe_experts_plain(x, ids, wts, w_gate_up, w_down, n_ff, act="silu", e_lo=0, 
     xs = x.index_select(0, plan.sorted_token)
     h = torch.empty(P, n_ff, dtype=x.dtype, device=x.device)
     y = torch.empty(P, H, dtype=x.dtype, device=x.device)
-    C.sgemm(w_gate_up.view(E * 2 * n_ff, H), xs, h, None, None, None, n_ff, True, n_ff, GATE_ACTS[act], plan.tile_group,
-            plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, 2 * n_ff, P, None)
+    C.sgemm(w_gate_up.view(E * n_gu, H), xs, h, None, None, None, n_ff, gated, n_ff if gated else 0, GATE_ACTS[act],
+            plan.tile_group, plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, n_gu, P, None)
     C.sgemm(w_down.view(E * H, n_ff), h, y, None, plan.sorted_w, plan.sorted_pair, H, False, 0, 0, plan.tile_group,
             plan.tile_tok0, plan.tile_ntok, plan.meta, plan.max_tiles, H, P, None)
     if defer_combine:
@@ -1713,10 +1742,92 @@ def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset=0.0):
     (y0, c0), (y1, c1) = (list(terms) + [(None, 0.0)])[:2]
     rows = 1
     if isinstance(y0, PendingCombine):
-        rows, y0 = y0.ids.shape[1], y0.y
+        rows, y0 = y0.rows, y0.y
     h = torch.empty(X.shape[0], X.shape[2], dtype=y0.dtype, device=X.device)
     ext().hyper_step(X, X, None, None, y0, c0, rows, y1, c1, mix, out_w, in_w, norm_w, eps, w_offset, h)
     return X, h
+
+
+def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None, dtype=None):
+    """x (fp32 [T, H]) updated in place by mult * (sum of scale * tensor over ``terms``), and its norm in the activation type
+    (``norm_w`` None: none); ``raw`` takes x itself in the activation type. ``start`` = (embedding table, ids or None, norm
+    weight or None) begins a step. Returns (x, norm)."""
+    table = ids = pre_w = None
+    x_in = x
+    if start is not None:
+        table, ids, pre_w = start
+        T = table.shape[0] if ids is None else ids.numel()
+        x, dtype = torch.empty(T, table.shape[1], dtype=torch.float32, device=table.device), table.dtype
+    (y0, c0), (y1, c1) = (list(terms) + [(None, 0.0), (None, 0.0)])[:2]
+    rows = 1
+    if isinstance(y0, PendingCombine):
+        rows, y0 = y0.rows, y0.y
+    h = torch.empty(x.shape, dtype=dtype, device=x.device) if norm_w is not None else None
+    if x.shape[0]:
+        ext().prenorm_step(x_in, x, table, ids, pre_w, y0, c0 * mult, rows, y1, c1 * mult, norm_w, eps, w_offset, h, raw)
+    return x, h
+
+
+def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout, positions,
+                    slots, k_cache, v_cache, heads: int, write_state=True, max_len=None):
+    """Bias, short convolution, norms, rotation of a q | k | v projection and the append to the cache (``csrc/qkv_conv.cu``);
+    returns the queries [T, heads, dk]."""
+    T = proj.shape[0]
+    q = torch.empty(T, heads, k_cache.shape[3], dtype=proj.dtype, device=proj.device)
+    ext().qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over == "all", eps, rot,
+                          layout == "half", positions, slots, q, k_cache, v_cache, T if max_len is None else int(max_len),
+                          bool(write_state))
+    return q
+
+
+DELTA_SCRATCH = 256 << 20    # bytes of block records a slice of a long step may take
+
+
+def channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, write_state=True,
+                  max_len=None, cu_host=None, out=None):
+    """Gated delta rule with a decay per key channel over the step's tokens, convolution included
+    (``csrc/channel_delta.cu``); state [slots, H, dv, dk] fp32 updated in place. Returns [T, H * dv]."""
+    C = ext()
+    T, n = qkv.shape[0], slots.numel()
+    if out is None:
+        out = torch.empty(T, H * dv, dtype=qkv.dtype, device=qkv.device)
+    if T == 0:
+        return out
+    ws = Workspace.get(qkv.device)
+    per = C.channel_delta_record_floats(H, dk, dv)
+    need = (T + 3) // 4 + n                        # records of the whole step
+    if write_state:                                # a long step may run in slices of at least 64 tokens
+        need = min(need, max(DELTA_SCRATCH // (4 * per), n + 16))
+    rec = ws._cache.get("channel_delta_rec")
+    if rec is None or rec.numel() < need * per:
+        rec = ws._cache["channel_delta_rec"] = torch.empty(need * per, dtype=torch.float32, device=qkv.device)
+    C.channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, out, bool(write_state),
+                    rec, ws.status)
+    return out
+
+
+def channel_delta_decode(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, gate, norm_w, eps,
+                         out=None):
+    """Decode step of ``channel_delta`` (one token per sequence) with the norm per head and sigmoid(gate) behind it, in one
+    launch."""
+    n = slots.numel()
+    ws = Workspace.get(qkv.device)
+    ctr = ws._cache.get("delta_ctr")
+    if ctr is None or ctr.numel() < n * G:
+        ctr = ws._cache["delta_ctr"] = torch.zeros(max(n * G, 16384), dtype=torch.int32, device=qkv.device)
+    if out is None:
+        out = torch.empty(n, H * dv, dtype=qkv.dtype, device=qkv.device)
+    ext().channel_delta_decode(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H, G, dk, dv, gate, norm_w,
+                               eps, ctr, out)
+    return out
+
+
+def head_norm_gate(o, gate, w, eps, heads: int, out=None):
+    """RMS norm of each head of o [T, heads * d], times w [d], times sigmoid(gate)."""
+    if out is None:
+        out = torch.empty(o.shape, dtype=o.dtype, device=o.device)
+    ext().head_norm_gate(o, gate, w, eps, heads, out)
+    return out
 
 
 LINEAR_CHUNK_MIN = 48        # longest portion of a step from which the chunked scan runs
