@@ -533,6 +533,100 @@ def bench_diag(rows):
             print(rows[-1], flush=True)
 
 
+def bench_delta(rows):
+    """Gurozen: delta rule with a decay per key channel, what lies between the attention projections and the scores, soft-capped
+    attention, squared-ReLU experts and the residual step, each beside the like kernel of the other families. frac_hbm: bytes
+    that must move once; frac_tc: FLOPs over measured cuBLAS bf16 (attention, experts)."""
+    from legion_b200.ops import sm100
+    hbm, tf, src = peaks()
+    f = lambda *s: (torch.randn(*s, device="cuda") * 0.5).bfloat16()                 # noqa: E731
+
+    def row(kernel, n, L, ms, byts=None, flops=None):
+        r = dict(kernel=kernel, n_seq=n, L=L, us=round(ms * 1e3, 2), peaks=src)
+        if byts:
+            r["frac_hbm"] = round(byts / ms / 1e6 / hbm, 3)
+        if flops:
+            r["frac_tc"] = round(flops / ms / 1e9 / tf, 3)
+        rows.append(r)
+        print(r, flush=True)
+    H, D, KC = 16, 128, 4
+    C = 3 * H * D
+    cw, A, db, one = torch.randn(KC, C, device="cuda"), -torch.ones(H, device="cuda"), torch.zeros(H * D, device="cuda"), torch.ones(D, device="cuda")
+    for n, L in (CASE["attn"] or ((1, 1), (16, 1), (64, 1), (1, 8192), (4, 2048))):
+        T = n * L
+        cu, cu_host = torch.arange(0, T + 1, L, device="cuda", dtype=torch.int32), list(range(0, T + 1, L))
+        slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        tm = timeit if L > 1 else timeit_graph
+        qkv, araw, braw, gate = f(T, C), f(T, H * D), f(T, H), f(T, H * D)
+        st, hist = torch.zeros(n, H, D, D, device="cuda"), torch.zeros(n, KC - 1, C, device="cuda")
+        args = (qkv, cw, hist, araw, A, db, braw, st, cu, slots, H, H, D, D)
+        byts = T * 5 * H * D * 2 + st.numel() * 8 + hist.numel() * 8
+        cwg, histg = torch.randn(C, KC, device="cuda"), torch.zeros(n, C, KC - 1, device="cuda")      # Gated DeltaNet's layout
+        gg, beta = -torch.rand(T, H, device="cuda") * 0.1, torch.rand(T, H, device="cuda")
+        if L == 1:
+            row("channel_delta_decode 16x128x128 (convolution, norm and gate included)", n, L,
+                tm(lambda: sm100.channel_delta_decode(*args, gate, one, 1e-6)), byts + T * H * D * 2)
+            pj = f(T, 4 * H * D + 2 * H)
+            row("gdn_decode_fused, same size", n, L, tm(lambda: sm100.gdn_decode_fused(
+                pj, cwg, histg, -one[:H], one[:H], one, 1e-6, "silu", st, slots, H, H, D, D, False, D ** -0.5)), byts)
+        else:
+            row("channel_delta 16x128x128 (convolution included)", n, L, tm(lambda: sm100.channel_delta(*args, max_len=L)), byts)
+            c = sm100.causal_conv1d_silu(qkv, cwg, None, histg, cu, slots, max_len=L)
+            row("gdn chunked, same size", n, L, tm(lambda: sm100.gdn_recurrent(c, gg, beta, st, cu, slots, H, H, D, D, False, D ** -0.5,
+                                                                             cu_host=cu_host)), byts)
+            row("conv1d_silu in front of it", n, L, tm(lambda: sm100.causal_conv1d_silu(qkv, cwg, None, histg, cu, slots, max_len=L)), T * C * 4)
+            o = f(T, H * D)
+            row("head_norm_gate 16x128", n, L, tm(lambda: sm100.head_norm_gate(o, gate, one, 1e-6, H)), T * H * D * 6)
+            row("gated_rmsnorm (Gated DeltaNet)", n, L, tm(lambda: sm100.gated_rmsnorm(o.view(T, H, D), gate, one, 1e-6)), T * H * D * 6)
+        # attention: 16 query heads over 4 kv heads of 128
+        G, page = 4, 64
+        nb, ctx = max(1, -(-L // page)), max(L, 2048)
+        nb = ctx // page
+        kc, vc = f(n * nb, page, G, D), f(n * nb, page, G, D)
+        bt = torch.arange(n * nb, device="cuda", dtype=torch.int32).view(n, nb)
+        pos = torch.arange(ctx - L, ctx, device="cuda", dtype=torch.int32).repeat(n)
+        cells = (bt.long()[:, :, None] * page + torch.arange(page, device="cuda")).view(n, -1)[:, ctx - L:].reshape(-1).contiguous()
+        proj, cs = f(T, (H + 2 * G) * D), torch.randn(ctx, 64, device="cuda")
+        Cq = proj.shape[1]
+        aw, ab, ah = torch.randn(KC, Cq, device="cuda"), torch.randn(Cq, device="cuda"), torch.zeros(n, KC - 1, Cq, device="cuda")
+        qn, kn = torch.ones(H * D, device="cuda"), torch.ones(G * D, device="cuda")
+        row("qkv_conv_append 16/4 heads of 128", n, L, tm(lambda: sm100.qkv_conv_append(
+            proj, ab, aw, ah, cu, slots, qn, kn, "all", 1e-6, cs, "half", pos, cells, kc, vc, H, max_len=L)), T * Cq * 4)
+        row("qk_norm_rope_append, same size", n, L, tm(lambda: sm100.qk_norm_rope_append(
+            proj, H, G, D, one, one, 1e-6, 0.0, cs, 64, pos, cells, kc, vc)), T * Cq * 4)
+        q, cl = f(T, H, D), torch.full((n,), ctx, device="cuda", dtype=torch.int32)
+        for cap in (30.0, 0.0):
+            name = "soft-capped attention" if cap else "attention"
+            if L == 1:
+                row(f"{name}, decode at {ctx}", n, L, tm(lambda: sm100.paged_decode(q, kc, vc, bt, cl, D ** -0.5, max_ctx=ctx, softcap=cap)),
+                    n * ctx * G * D * 4)
+            else:
+                row(f"{name}, prompt", n, L, tm(lambda: sm100.prefill_attn(q, kc, vc, cu, cl, bt, L, D ** -0.5, softcap=cap)),
+                    flops=n * L * L / 2 * H * D * 4)
+        # residual step of 2048 columns
+        W = 2048
+        x, y, nw = torch.randn(T, W, device="cuda"), f(T, W), torch.zeros(W, device="cuda")
+        row("prenorm_step 2048", n, L, tm(lambda: sm100.prenorm_step(x, [(y, 1.0)], 0.5, nw, 1e-6, 1.0, dtype=torch.bfloat16)), T * W * 12)
+        xb = f(T, W)
+        row("residual + RMS norm 2048", n, L, tm(lambda: sm100.rmsnorm(y, nw, 1e-6, 1.0, residual=xb)), T * W * 8)
+        # experts: 32 of 1536 (squared ReLU), of 1024 (gated), top 4
+        E, k = 32, 4
+        rw = f(E + 1, W)
+        for act, ff in (("relu2", 1536), ("silu", 1024)):
+            up, dn = f(E + 1, ff if act == "relu2" else 2 * ff, W), f(E + 1, W, ff)
+            sh = act == "relu2"
+
+            def experts():
+                r = sm100.router(y, rw if sh else rw[:E], k, "sigmoid", "sum", 2.0, None, 8, 4, n_local=E, gate_row=sh, shared_slots=int(sh))
+                m = E + int(sh and r.dense is not None)
+                return sm100.moe_experts(y, r.ids, r.wts, up[:m], dn[:m], ff, 0, routing=r, defer_combine="pairs", act=act)
+            slots_used = k + (1 if sh and T <= 64 else 0)
+            seen = min(E, E * (1 - (1 - k / E) ** T)) + (1 if sh and T <= 64 else 0)
+            row(f"router + experts {act} {ff}", n, L, tm(experts), byts=seen * (up[0].numel() + dn[0].numel()) * 2 + T * W * 2 * (2 + slots_used),
+                flops=2.0 * T * slots_used * (up[0].numel() + dn[0].numel()))
+            del up, dn
+
+
 class Batch:
     """The fields of a step that a planner reads."""
 
@@ -722,7 +816,7 @@ def main(argv=None):
     if a.gemm:
         CASE["gemm"] = [tuple(int(y) for y in x.split("x")) for x in a.gemm.split(",")]
     rows = []
-    table = {"resid": bench_resid, "diag": bench_diag, "latent": bench_latent, "linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
+    table = {"delta": bench_delta, "resid": bench_resid, "diag": bench_diag, "latent": bench_latent, "linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
     for name in a.only.split(","):
         table[name](rows)
     from legion_b200.ops.sm100 import Workspace

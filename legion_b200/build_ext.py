@@ -27,7 +27,7 @@ NVCC_FLAGS = [
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
 PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any",
-           "channel_delta", "qkv_conv"}
+           "channel_delta", "channel_delta_mma", "qkv_conv"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:
@@ -67,7 +67,7 @@ KIND_KERNELS = {
     "attn": _ATTN, "lightning": _SCAN, "ssd": _SCAN, "parallel": _ATTN | _SCAN,
     "latent": {"attn_mla_sm100", "latent_attn", "attn_prefill_sm100", "attn_decode", "attn_general"},
     "rglru": {"diag_scan", "conv1d", "conv_any"},
-    "channel_delta": {"channel_delta"},
+    "channel_delta": {"channel_delta", "channel_delta_mma"},
 }
 
 

@@ -376,11 +376,11 @@ class ModelConfig:
         return m.right if isinstance(m, ParallelSpec) else None
 
     def attn_history(self, il: int):
-        """(channels, tokens) of the projected q, k and v that the short convolution of an attention layer keeps, or None."""
+        """(tokens, channels) of the projected q, k and v that the short convolution of an attention layer keeps, or None."""
         a = self.attn_spec(il)
         if a is None or a.conv < 2:
             return None
-        return (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim, a.conv - 1
+        return a.conv - 1, (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim
 
     def state_floats(self, il: int) -> int:
         """float32 numbers of recurrent state (without convolution histories) per sequence of layer il."""

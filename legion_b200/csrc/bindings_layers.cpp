@@ -122,9 +122,9 @@ lb::ChannelDeltaArgs delta_args(const Tensor& qkv, const Tensor& conv_w, Tensor&
                   b_raw.size(0) == T && b_raw.size(1) == H && out.size(0) == T && out.size(1) == H * DV,
               "channel_delta: q | k | v [T, columns], decays [T, H * DK], beta [T, H], out [T, H * DV]");
   f32c(conv_w, 0, "conv_w");
-  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C, "channel_delta: conv_w [columns, taps]");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(1) == C, "channel_delta: conv_w [taps, columns]");
   TORCH_CHECK(conv_state.scalar_type() == at::kFloat && conv_state.is_contiguous() && conv_state.dim() == 3 &&
-                  conv_state.size(1) == C && conv_state.size(2) == conv_w.size(1) - 1, "channel_delta: history [slots, columns, taps - 1]");
+                  conv_state.size(2) == C && conv_state.size(1) == conv_w.size(0) - 1, "channel_delta: history [slots, taps - 1, columns]");
   f32c(A, H, "A");
   f32c(dt_bias, H * DK, "dt_bias");
   TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() == 4 && state.size(1) == H &&
@@ -133,7 +133,7 @@ lb::ChannelDeltaArgs delta_args(const Tensor& qkv, const Tensor& conv_w, Tensor&
               "channel_delta: int32 sequence bounds and slots");
   lb::ChannelDeltaArgs a{};
   a.qkv = qkv.data_ptr(); a.ld = qkv.stride(0);
-  a.conv_w = conv_w.data_ptr<float>(); a.KC = int(conv_w.size(1)); a.conv_state = conv_state.data_ptr<float>();
+  a.conv_w = conv_w.data_ptr<float>(); a.KC = int(conv_w.size(0)); a.conv_state = conv_state.data_ptr<float>();
   a.a = a_raw.data_ptr(); a.lda = a_raw.stride(0); a.A = A.data_ptr<float>(); a.dt_bias = dt_bias.data_ptr<float>();
   a.b = b_raw.data_ptr(); a.ldb = b_raw.stride(0);
   a.state = state.data_ptr<float>(); a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>();
@@ -275,13 +275,13 @@ void bind_layers(pybind11::module_& m) {
     a.KC = 1;
     if (conv_w.has_value()) {
       f32c(*conv_w, 0, "conv_w");
-      TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(0) == C, "qkv_conv_append: conv_w [columns, taps]");
+      TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(1) == C, "qkv_conv_append: conv_w [taps, columns]");
       a.conv_w = conv_w->data_ptr<float>();
-      a.KC = int(conv_w->size(1));
+      a.KC = int(conv_w->size(0));
       if (a.KC > 1) {
         TORCH_CHECK(conv_state.has_value() && conv_state->scalar_type() == at::kFloat && conv_state->is_contiguous() &&
-                        conv_state->dim() == 3 && conv_state->size(1) == C && conv_state->size(2) == a.KC - 1,
-                    "qkv_conv_append: history [slots, columns, taps - 1]");
+                        conv_state->dim() == 3 && conv_state->size(2) == C && conv_state->size(1) == a.KC - 1,
+                    "qkv_conv_append: history [slots, taps - 1, columns]");
         a.conv_state = conv_state->data_ptr<float>();
       }
     }
@@ -308,8 +308,8 @@ void bind_layers(pybind11::module_& m) {
     TORCH_CHECK(lb::qkv_conv_append_launch(a, f32, cur_stream()) == 0,
                 "qkv_conv_append: at most 51200 query and key columns, rotation within a head", cuda_error());
   });
-  m.def("channel_delta_record_floats", [](int64_t H, int64_t DK, int64_t DV) {
-    return int64_t(lb::channel_delta_record_floats(int(H), int(DK), int(DV)));
+  m.def("channel_delta_record_floats", [](int64_t H, int64_t DK, int64_t DV, bool f32) {
+    return int64_t(lb::channel_delta_record_floats(int(H), int(DK), int(DV), f32));
   });
   m.def("channel_delta", [](const Tensor& qkv, const Tensor& conv_w, Tensor& conv_state, const Tensor& a_raw, const Tensor& A,
                             const Tensor& dt_bias, const Tensor& b_raw, Tensor& state, const Tensor& cu, const Tensor& slots,

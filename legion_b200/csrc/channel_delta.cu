@@ -13,11 +13,11 @@
 // norms, decays, the decayed vectors and the 16 inner products. SCAN walks the blocks of a sequence; columns of the state are
 // independent, so a warp owns four of them (eight lanes per column) with the state in registers, and the records stream
 // through shared memory by bulk copies. Steps whose records would not fit the scratch run in slices of tokens.
+// This file's form serves fp32 and head sizes of any kind; bf16 prompts run the same algebra with blocks of eight tokens and
+// the products on tensor cores (channel_delta_mma.cu).
 //
 // Decode steps are one launch: history and convolution, decays, update, RMS norm per head and output gate.
-#include "act_type.cuh"
-#include "common.cuh"
-#include "layers.h"
+#include "channel_delta.cuh"
 
 namespace lb {
 namespace {
@@ -32,54 +32,17 @@ __host__ __device__ constexpr int pad_dk(int dk) { return dk <= 32 ? 32 : dk <= 
 __host__ __device__ constexpr int pad_dv(int dv) { return (dv + COLS - 1) / COLS * COLS; }
 __host__ __device__ constexpr long record_floats(int dkp, int dvp) { return long(NVEC) * dkp + NSCAL + BT * dvp; }
 
-// Blocks of a slice [lo, hi) of the step's rows: sequence i begins at block (rows of the slice in front of it) / 4 + i, which
-// leaves room for every sequence's last, partial block. Returns false where a block number has no tokens.
-struct Block { int seq, t0, n, seq0; };  // sequence, first row, tokens, first row of the sequence
-__device__ __forceinline__ int clamp_i(int v, int lo, int hi) { return v < lo ? lo : v > hi ? hi : v; }
-__device__ __forceinline__ bool find_block(const int* cu, int n_seqs, int lo, int hi, int blk, Block& b) {
-  int a = 0, z = n_seqs;                 // last sequence whose first block is <= blk
-  while (z - a > 1) {
-    const int m = (a + z) >> 1;
-    if ((clamp_i(cu[m], lo, hi) - lo) / BT + m <= blk) a = m; else z = m;
-  }
-  const int s0 = clamp_i(cu[a], lo, hi), s1 = clamp_i(cu[a + 1], lo, hi);
-  const int t0 = s0 + (blk - ((s0 - lo) / BT + a)) * BT;
-  if (t0 >= s1) return false;
-  b.seq = a; b.t0 = t0; b.n = min(BT, s1 - t0); b.seq0 = cu[a];
-  return true;
-}
-
-template <typename T>
-__device__ __forceinline__ float silu_t(float z) {
-  if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
-  else return silu_f(z);
-}
-template <typename T>
-__device__ __forceinline__ float sigmoid_t(float z) {
-  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-z));
-  else return sigmoid_f(z);
-}
-template <typename T>
-__device__ __forceinline__ float exp_t(float z) {
-  if constexpr (sizeof(T) == 2) return __expf(z);
-  else return expf(z);
-}
-template <typename T>
-__device__ __forceinline__ float decay_t(float raw, float A) {
-  return exp_t<T>(A * softplus_f(raw));
-}
-
-// Convolution + silu of one channel for the block's tokens; rows in front of the sequence come from its history. KC 0: any
-// number of taps (taps of a channel ws_stride apart).
+// Convolution + silu of one channel for the block's tokens; rows in front of the sequence come from its history (rows hs
+// apart). KC 0: any number of taps (taps of a channel ws_stride apart).
 template <typename T, int KC>
-__device__ __forceinline__ void conv_block(const T* x, long ld, const float* hist, const float* w, int ws_stride, int taps,
-                                           const Block& b, float (&y)[BT]) {
+__device__ __forceinline__ void conv_block(const T* x, long ld, const float* hist, long hs, const float* w, int ws_stride, int taps,
+                                           const DeltaBlock& b, float (&y)[BT]) {
   if constexpr (KC > 0) {
     float u[KC - 1 + BT];
 #pragma unroll
     for (int i = 0; i < KC - 1 + BT; ++i) {
       const int s = b.t0 - (KC - 1) + i;
-      u[i] = s >= b.seq0 ? (i - (KC - 1) < b.n ? ld_f(x + long(s) * ld) : 0.f) : hist[(KC - 1) + (s - b.seq0)];
+      u[i] = s >= b.seq0 ? (i - (KC - 1) < b.n ? ld_f(x + long(s) * ld) : 0.f) : hist[((KC - 1) + (s - b.seq0)) * hs];
     }
 #pragma unroll
     for (int t = 0; t < BT; ++t) {
@@ -94,26 +57,11 @@ __device__ __forceinline__ void conv_block(const T* x, long ld, const float* his
       float acc = 0.f;
       for (int j = 0; j < taps && t < b.n; ++j) {
         const int s = b.t0 + t - (taps - 1) + j;
-        acc = fmaf(w[j * ws_stride], s >= b.seq0 ? ld_f(x + long(s) * ld) : hist[(taps - 1) + (s - b.seq0)], acc);
+        acc = fmaf(w[j * ws_stride], s >= b.seq0 ? ld_f(x + long(s) * ld) : hist[((taps - 1) + (s - b.seq0)) * hs], acc);
       }
       y[t] = silu_t<T>(acc);
     }
   }
-}
-
-// Sum over the warp of 32 values per lane; lane L gets value L.
-__device__ __forceinline__ float transpose_sum(float (&v)[32]) {
-  const int lane = threadIdx.x & 31;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const bool up = lane & o;
-#pragma unroll
-    for (int i = 0; i < o; ++i) {
-      const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
-      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-    }
-  }
-  return v[0];
 }
 
 constexpr int PREP_BLOCKS = 4;           // blocks per warp
@@ -126,9 +74,9 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const ChannelDeltaArgs 
   const int hk = h / (a.H / a.G), lane = threadIdx.x & 31;
   const int q0 = hk * DK, k0 = a.G * DK + hk * DK, v0 = 2 * a.G * DK + h * DV, C = 2 * a.G * DK + a.H * DV;
   for (int i = threadIdx.x; i < W * taps; i += 128) {
-    const int c = i / taps, j = i % taps;
+    const int c = i % W, j = i / W;
     const int ch = c < DK ? q0 + c : c < 2 * DK ? k0 + c - DK : v0 + c - 2 * DK;
-    w_s[j * W + c] = a.conv_w[long(ch) * taps + j];
+    w_s[i] = a.conv_w[long(j) * C + ch];
   }
   griddep_wait();
   griddep_launch();
@@ -140,10 +88,10 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const ChannelDeltaArgs 
   const T* ap = static_cast<const T*>(a.a) + long(h) * DK;
   const int blk0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * PREP_BLOCKS;
   for (int blk = blk0; blk < min(n_blocks, blk0 + PREP_BLOCKS); ++blk) {
-    Block b;
-    if (!find_block(a.cu, a.n_seqs, lo, hi, blk, b)) continue;
+    DeltaBlock b;
+    if (!find_block<BT>(a.cu, a.n_seqs, lo, hi, blk, b)) continue;
     const float* hist = a.conv_state + long(a.slots[b.seq]) * C * (taps - 1);
-    float* r = rec + (long(blk) * a.H + h) * record_floats(DKP, DVP);
+    float* r = rec + (long(h) * n_blocks + blk) * record_floats(DKP, DVP);
     float q[NC][BT], k[NC][BT], g[NC][BT], s[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) s[i] = 0.f;
@@ -151,8 +99,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const ChannelDeltaArgs 
     for (int i = 0; i < NC; ++i) {
       const int c = lane + 32 * i;
       if (c < DK) {
-        conv_block<T, KC>(x + q0 + c, a.ld, hist + long(q0 + c) * (taps - 1), w_s + c, W, taps, b, q[i]);
-        conv_block<T, KC>(x + k0 + c, a.ld, hist + long(k0 + c) * (taps - 1), w_s + DK + c, W, taps, b, k[i]);
+        conv_block<T, KC>(x + q0 + c, a.ld, hist + q0 + c, C, w_s + c, W, taps, b, q[i]);
+        conv_block<T, KC>(x + k0 + c, a.ld, hist + k0 + c, C, w_s + DK + c, W, taps, b, k[i]);
         const float db = a.dt_bias[long(h) * DK + c];
 #pragma unroll
         for (int t = 0; t < BT; ++t) {
@@ -239,7 +187,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const ChannelDeltaArgs 
     float* rv = r + NVEC * DKP + NSCAL;
     for (int c = lane; c < DVP; c += 32) {
       float v[BT] = {0.f, 0.f, 0.f, 0.f};
-      if (c < DV) conv_block<T, KC>(x + v0 + c, a.ld, hist + long(v0 + c) * (taps - 1), w_s + 2 * DK + c, W, taps, b, v);
+      if (c < DV) conv_block<T, KC>(x + v0 + c, a.ld, hist + v0 + c, C, w_s + 2 * DK + c, W, taps, b, v);
 #pragma unroll
       for (int t = 0; t < BT; ++t) rv[t * DVP + c] = v[t];
     }
@@ -311,7 +259,7 @@ __device__ __forceinline__ void store_state(float* col, int r, int DK, const uin
 
 // grid (H * column tiles, sequences), 160 threads: warps 0..3 own four columns each, warp 4 copies the records.
 template <typename T, int NI>
-__global__ void __launch_bounds__(160) delta_scan_kernel(const ChannelDeltaArgs a, int lo, int hi, const float* rec, int* status) {
+__global__ void __launch_bounds__(160) delta_scan_kernel(const ChannelDeltaArgs a, int lo, int hi, int n_blocks, const float* rec, int* status) {
   constexpr int DKP = 32 * NI;
   constexpr int HEAD = NVEC * DKP + NSCAL;               // floats of a record that every column tile reads
   constexpr int STAGE = HEAD + BT * COLS;
@@ -337,8 +285,8 @@ __global__ void __launch_bounds__(160) delta_scan_kernel(const ChannelDeltaArgs 
   const int slot = a.slots[seq];
   if (s1 <= s0 || slot < 0) return;
   const int n_blk = (s1 - s0 + BT - 1) / BT;
-  const float* r0 = rec + (long((s0 - lo) / BT + seq) * a.H + h) * record_floats(DKP, DVP);
-  const long pitch = long(a.H) * record_floats(DKP, DVP);
+  const long pitch = record_floats(DKP, DVP);
+  const float* r0 = rec + (long(h) * n_blocks + (s0 - lo) / BT + seq) * pitch;
   if (warp == 4) {
     if (lane == 0) {
       int i = 0;
@@ -466,11 +414,11 @@ __global__ void __launch_bounds__(128) delta_history_kernel(const ChannelDeltaAr
   if (c >= C) return;
   const int t0 = a.cu[seq], t1 = a.cu[seq + 1];
   if (t1 <= t0 || a.slots[seq] < 0) return;
-  float* st = a.conv_state + (long(a.slots[seq]) * C + c) * K1;
+  float* st = a.conv_state + long(a.slots[seq]) * C * K1 + c;
   const T* x = static_cast<const T*>(a.qkv) + c;
   for (int j = 0; j < K1; ++j) {           // position j takes what was behind it: never read after written
     const int s = t1 - K1 + j;
-    st[j] = s >= t0 ? ld_f(x + long(s) * a.ld) : st[K1 + (s - t0)];
+    st[long(j) * C] = s >= t0 ? ld_f(x + long(s) * a.ld) : st[long(K1 + (s - t0)) * C];
   }
 }
 
@@ -514,15 +462,15 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
     const int c = channel(i);
     const bool own = hpg == 1 || i >= 2 * DK;
     const float xv = ld_f(x + c);
-    float* hc = hist + long(c) * K1;
-    const float* wc = a.conv_w + long(c) * a.KC;
-    float acc = wc[K1] * xv;
+    float* hc = hist + c;
+    const float* wc = a.conv_w + c;
+    float acc = wc[long(K1) * C] * xv;
     for (int j = 0; j < K1; ++j) {
-      const float hv = hc[j];
-      acc = fmaf(wc[j], hv, acc);
-      if (own && j > 0) hc[j - 1] = hv;
+      const float hv = hc[long(j) * C];
+      acc = fmaf(wc[long(j) * C], hv, acc);
+      if (own && j > 0) hc[long(j - 1) * C] = hv;
     }
-    if (own && K1 > 0) hc[K1 - 1] = xv;
+    if (own && K1 > 0) hc[long(K1 - 1) * C] = xv;
     const float y = silu_t<T>(acc);
     if (i < DK) { gq[i] = y; qq = fmaf(y, y, qq); }
     else if (i < 2 * DK) { ks[i - DK] = y; kk = fmaf(y, y, kk); }
@@ -544,9 +492,9 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
       __threadfence();
       for (int i = threadIdx.x; i < 2 * DK; i += 256) {
         const int c = channel(i);
-        float* hc = hist + long(c) * K1;
-        for (int j = 0; j + 1 < K1; ++j) hc[j] = __ldcg(&hc[j + 1]);
-        hc[K1 - 1] = ld_f(x + c);
+        float* hc = hist + c;
+        for (int j = 0; j + 1 < K1; ++j) hc[long(j) * C] = __ldcg(&hc[long(j + 1) * C]);
+        hc[long(K1 - 1) * C] = ld_f(x + c);
       }
     }
   }
@@ -688,7 +636,7 @@ int prep_t(const ChannelDeltaArgs& a, int lo, int hi, int n_blocks, float* rec, 
 }
 
 template <typename T, int NI>
-int scan_t(const ChannelDeltaArgs& a, int lo, int hi, const float* rec, int* status, cudaStream_t s) {
+int scan_t(const ChannelDeltaArgs& a, int lo, int hi, int n_blocks, const float* rec, int* status, cudaStream_t s) {
   const int smem = STAGES * (NVEC * 32 * NI + NSCAL + BT * COLS) * 4;
   auto kfn = delta_scan_kernel<T, NI>;
   static bool attr = false;
@@ -696,7 +644,7 @@ int scan_t(const ChannelDeltaArgs& a, int lo, int hi, const float* rec, int* sta
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return 1;
     attr = true;
   }
-  return launch_pdl(kfn, dim3(a.H * (pad_dv(a.DV) / COLS), a.n_seqs), dim3(160), smem, s, a, lo, hi, rec, status) != cudaSuccess;
+  return launch_pdl(kfn, dim3(a.H * (pad_dv(a.DV) / COLS), a.n_seqs), dim3(160), smem, s, a, lo, hi, n_blocks, rec, status) != cudaSuccess;
 }
 
 template <typename T>
@@ -711,12 +659,17 @@ int scan_all(const ChannelDeltaArgs& a, float* rec, long rec_floats, int* status
     const int nb = (hi - lo) / BT + a.n_seqs;
     int rc = 1;
 #define LB_NI(N_) \
-  if (DKP == 32 * N_) rc = prep_t<T, N_>(a, lo, hi, nb, rec, s) || scan_t<T, N_>(a, lo, hi, rec, status, s);
+  if (DKP == 32 * N_) rc = prep_t<T, N_>(a, lo, hi, nb, rec, s) || scan_t<T, N_>(a, lo, hi, nb, rec, status, s);
     LB_NI(1) LB_NI(2) LB_NI(4) LB_NI(8)
 #undef LB_NI
     if (rc) return 1;
     lo = hi;
   }
+  return 0;
+}
+
+template <typename T>
+int history_t(const ChannelDeltaArgs& a, cudaStream_t s) {
   if (a.write_state && a.KC > 1)
     return launch_pdl(delta_history_kernel<T>, dim3((2 * a.G * a.DK + a.H * a.DV + 127) / 128, a.n_seqs), dim3(128), 0, s, a) !=
            cudaSuccess;
@@ -756,12 +709,19 @@ bool shape_ok(const ChannelDeltaArgs& a) {
 
 }  // namespace
 
-long channel_delta_record_floats(int H, int DK, int DV) { return record_floats(pad_dk(DK), pad_dv(DV)) * H; }
+long channel_delta_record_floats(int H, int DK, int DV, bool f32) {
+  // per four tokens; records of eight tokens count half
+  const long four = record_floats(pad_dk(DK), pad_dv(DV)) * H;
+  return f32 || DK > 128 ? four : max(four, (channel_delta_mma_floats(H, DK, DV) + 1) / 2);
+}
 
 int channel_delta_launch(const ChannelDeltaArgs& a, float* rec, long rec_floats, int* status, bool f32, cudaStream_t s) {
   if (a.n_seqs <= 0 || a.T <= 0) return 0;
   if (!shape_ok(a) || (reinterpret_cast<uintptr_t>(rec) & 127) || (reinterpret_cast<uintptr_t>(a.state) & 15)) return 1;
-  return f32 ? scan_all<float>(a, rec, rec_floats, status, s) : scan_all<__nv_bfloat16>(a, rec, rec_floats, status, s);
+  if (f32) return scan_all<float>(a, rec, rec_floats, status, s) || history_t<float>(a, s);
+  const int rc = channel_delta_mma_ok(a) ? channel_delta_mma_launch(a, rec, rec_floats, status, s)
+                                         : scan_all<__nv_bfloat16>(a, rec, rec_floats, status, s);
+  return rc || history_t<__nv_bfloat16>(a, s);
 }
 
 int channel_delta_decode_launch(const ChannelDeltaArgs& a, const void* gate, long ldg, const float* norm_w, float eps,

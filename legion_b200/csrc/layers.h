@@ -148,8 +148,8 @@ int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld,
 struct QkvConvArgs {
   const void* x; long ld;          // [T, Hq * DK | Hkv * DK | Hkv * DV]
   const float* in_b;               // [columns]; the history holds x + in_b
-  const float* conv_w; int KC;     // [columns, KC]; nullptr: none
-  float* conv_state;               // [slots, columns, KC - 1]
+  const float* conv_w; int KC;     // [KC, columns]; nullptr: none
+  float* conv_state;               // [slots, KC - 1, columns]
   const int* cu; const int* state_slots; int n_seqs;
   const float* qw; const float* kw; int norm_all; float eps;   // weights [DK], or [Hq * DK] / [Hkv * DK] with norm_all
   const float* cos_sin; int rot; int rot_half;                 // [positions, rot]; rot_half: column i turns with i + rot / 2
@@ -165,7 +165,7 @@ int qkv_conv_append_launch(QkvConvArgs a, bool f32, cudaStream_t s);
 // Gated delta rule with a decay per key channel (channel_delta.cu)
 struct ChannelDeltaArgs {
   const void* qkv; long ld;        // [T, G * DK | G * DK | H * DV] in front of the convolution
-  const float* conv_w; int KC; float* conv_state;              // [columns, KC], [slots, columns, KC - 1]
+  const float* conv_w; int KC; float* conv_state;              // [KC, columns], [slots, KC - 1, columns]
   const void* a; long lda;         // [T, H * DK]: decay exp(A softplus(a + dt_bias))
   const float* A; const float* dt_bias;                        // [H], [H * DK]
   const void* b; long ldb;         // [T, H]: beta = sigmoid(b)
@@ -177,7 +177,7 @@ struct ChannelDeltaArgs {
   int write_state;
 };
 // floats of scratch per four tokens (and per sequence); rec: 128-byte aligned, for at least n_seqs + 1 of them
-long channel_delta_record_floats(int H, int DK, int DV);
+long channel_delta_record_floats(int H, int DK, int DV, bool f32);
 int channel_delta_launch(const ChannelDeltaArgs& a, float* rec, long rec_floats, int* status, bool f32, cudaStream_t s);
 // One decode step with the norm per head (times norm_w, times sigmoid(gate)) behind it; ctr: [n_seqs, G] zeroed arrival
 // counters, left zero

@@ -85,7 +85,7 @@ def load(ck, device, dtype) -> "tuple[ModelConfig, Dict[str, torch.Tensor]]":
             w[f"{p}.mix.in"], w[f"{p}.attn.in_b"] = cat(f"{b}.q", f"{b}.k", f"{b}.v"), cat(f"{b}.q.b", f"{b}.k.b", f"{b}.v.b")
             w[f"{p}.attn.q_norm"], w[f"{p}.attn.k_norm"] = get(f"{b}.q.norm"), get(f"{b}.k.norm")
             if m.conv:
-                w[f"{p}.attn.conv_w"] = cat(f"{b}.q.conv", f"{b}.k.conv", f"{b}.v.conv")
+                w[f"{p}.attn.conv_w"] = cat(f"{b}.q.conv", f"{b}.k.conv", f"{b}.v.conv").t()
             w[f"{p}.attn.o"] = get(f"{b}.o")
         else:
             col = m.in_columns()
@@ -94,7 +94,7 @@ def load(ck, device, dtype) -> "tuple[ModelConfig, Dict[str, torch.Tensor]]":
                 t = get(f"{b}.{part}")
                 rows[col[part]:col[part] + t.shape[0]] = t
             w[f"{p}.cd.in"] = rows
-            w[f"{p}.cd.conv_w"] = cat(f"{b}.q.conv", f"{b}.k.conv", f"{b}.v.conv")
+            w[f"{p}.cd.conv_w"] = cat(f"{b}.q.conv", f"{b}.k.conv", f"{b}.v.conv").t()
             w[f"{p}.cd.low"] = torch.cat([F.pad(t, (0, m.rank - t.shape[1])) for t in (get(f"{b}.a2"), get(f"{b}.g2"))], 0)
             w[f"{p}.cd.A"] = -torch.exp(get(f"{b}.A_log").double())
             w[f"{p}.cd.dt_bias"], w[f"{p}.cd.norm"], w[f"{p}.cd.out"] = get(f"{b}.dt_bias"), get(f"{b}.norm"), get(f"{b}.o")

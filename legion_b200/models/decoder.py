@@ -173,7 +173,7 @@ class StatePool:
                     continue
                 if r.kind == "channel_delta":
                     self.ssm[il] = torch.zeros(n_slots, r.heads, r.vdim, r.dim, device=device, dtype=torch.float32)
-                    self.conv[il] = torch.zeros(n_slots, 2 * r.kv_heads * r.dim + r.heads * r.vdim, r.conv - 1, device=device,
+                    self.conv[il] = torch.zeros(n_slots, r.conv - 1, 2 * r.kv_heads * r.dim + r.heads * r.vdim, device=device,
                                                 dtype=torch.float32)
                     continue
                 if r.kind == "rglru":

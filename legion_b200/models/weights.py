@@ -165,7 +165,7 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
     elif m.kind == "channel_delta":
         nk, nv = m.kv_heads * m.dim, m.heads * m.vdim
         s[f"{p}.cd.in"] = (m.in_columns()["end"], H)                            # q | k | v | b | a1 | g1
-        s[f"{p}.cd.conv_w"] = (2 * nk + nv, m.conv)
+        s[f"{p}.cd.conv_w"] = (m.conv, 2 * nk + nv)                             # oldest token first
         s[f"{p}.cd.low"] = (m.heads * m.dim + nv, m.rank)                       # decay | output gate, from a1 and g1
         s[f"{p}.cd.A"] = (m.heads,)
         s[f"{p}.cd.dt_bias"] = (m.heads * m.dim,)
@@ -183,7 +183,7 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
             if a.bias:
                 s[f"{p}.attn.in_b"] = (rows,)
             if a.conv:
-                s[f"{p}.attn.conv_w"] = (rows, a.conv)
+                s[f"{p}.attn.conv_w"] = (a.conv, rows)                          # oldest token first
             s[f"{p}.attn.o"] = (H, a.heads * a.vdim)
         if r is not None:
             inner, conv_c = r.heads * r.vdim, r.heads * r.vdim + 2 * r.groups * r.state

@@ -289,16 +289,16 @@ def causal_conv1d_silu(x, w, bias, conv_state, cu_seq, slots, write_state: bool 
 
 def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout,
                     positions, slots, k_cache, v_cache, heads: int, write_state: bool = True):
-    """``proj`` [T, q | k | v]: bias, short convolution with carried history, norm of q and k over each head or the whole,
+    """``proj`` [T, q | k | v]: bias, short convolution (conv_w [taps, columns]) with carried history [slots, taps - 1, columns], norm of q and k over each head or the whole,
     rotation, k and v to their cache cells. Everything behind the projection is optional (None). Returns q [T, heads, dk]
     in the activation type; the values between are float32."""
     n_kv, dk, dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
     T, nq, nk = proj.shape[0], heads * dk, n_kv * dk
     u = proj.float() if in_b is None else proj.float() + in_b
-    if conv_w is not None and conv_w.shape[1] == 1:
-        u = u * conv_w[:, 0]
+    if conv_w is not None and conv_w.shape[0] == 1:
+        u = u * conv_w[0]
     elif conv_w is not None:
-        u = causal_conv1d_silu(u, conv_w, None, conv_state, cu_seq, state_slots, write_state, None, False)
+        u = causal_conv1d_silu(u, conv_w.t(), None, conv_state.transpose(1, 2), cu_seq, state_slots, write_state, None, False)
     q, k, v = u[:, :nq], u[:, nq:nq + nk], u[:, nq + nk:nq + nk + n_kv * dv]
     if q_norm is not None and norm_over == "all":
         q, k = _norm32(q, q_norm, eps, 0.0), _norm32(k, k_norm, eps, 0.0)
@@ -316,11 +316,12 @@ def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm,
 
 def channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_seq, slots, H: int, G: int, dk: int, dv: int,
                   write_state: bool = True):
-    """Gated delta rule with a decay per key channel. ``qkv`` [T, q | k | v] in front of the short convolution, ``a_raw``
+    """Gated delta rule with a decay per key channel. ``qkv`` [T, q | k | v] in front of the short convolution (conv_w
+    [taps, columns], history [slots, taps - 1, columns]), ``a_raw``
     [T, H * dk] and ``b_raw`` [T, H] before their activations, state [slots, H, dv, dk] float32. Per head
     S = g S (key channels), S += k (beta (v - S^T k))^T, o = S^T q. Returns o [T, H * dv]."""
     T = qkv.shape[0]
-    u = causal_conv1d_silu(qkv, conv_w, None, conv_state, cu_seq, slots, write_state).float()
+    u = causal_conv1d_silu(qkv, conv_w.t(), None, conv_state.transpose(1, 2), cu_seq, slots, write_state).float()
     unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)                  # noqa: E731
     q = unit(u[:, :G * dk].reshape(T, G, dk)).repeat_interleave(H // G, 1) * dk ** -0.5
     k = unit(u[:, G * dk:2 * G * dk].reshape(T, G, dk)).repeat_interleave(H // G, 1)

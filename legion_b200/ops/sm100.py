@@ -1794,10 +1794,10 @@ def channel_delta(qkv, conv_w, conv_state, a_raw, A, dt_bias, b_raw, state, cu_s
     if T == 0:
         return out
     ws = Workspace.get(qkv.device)
-    per = C.channel_delta_record_floats(H, dk, dv)
-    need = (T + 3) // 4 + n                        # records of the whole step
+    per = C.channel_delta_record_floats(H, dk, dv, qkv.dtype == torch.float32)
+    need = (T + 3) // 4 + 2 * n + 2                # records of the whole step
     if write_state:                                # a long step may run in slices of at least 64 tokens
-        need = min(need, max(DELTA_SCRATCH // (4 * per), n + 16))
+        need = min(need, max(DELTA_SCRATCH // (4 * per), 2 * n + 18))
     rec = ws._cache.get("channel_delta_rec")
     if rec is None or rec.numel() < need * per:
         rec = ws._cache["channel_delta_rec"] = torch.empty(need * per, dtype=torch.float32, device=qkv.device)

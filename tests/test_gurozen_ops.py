@@ -150,7 +150,7 @@ def test_projected_rows_on_their_way_to_the_cache(device, dtype, H, G, dk, dv, K
     for name, cuts in CUTS.items():
         kc = torch.full((60, page, G, dk), 7.0, dtype=dtype, device=device)
         vc = torch.full((60, page, G, dv), 7.0, dtype=dtype, device=device)
-        hist = torch.full((6, C, K - 1), 9.0, device=device)
+        hist = torch.full((6, K - 1, C), 9.0, device=device)
         hist[SLOTS] = 0.0
         cell = lambda i, t: (i * 13 + 3) * page + t                         # noqa: E731
         got = [[] for _ in LENS]
@@ -158,7 +158,7 @@ def test_projected_rows_on_their_way_to_the_cache(device, dtype, H, G, dk, dv, K
             x = dev(torch.cat([xs[i][a:a + c] for i, a, c in step]))
             pos = i32([t for _, a, c in step for t in range(a, a + c)], device)
             slots = torch.tensor([cell(i, t) for i, a, c in step for t in range(a, a + c)], device=device)
-            q = ops.qkv_conv_append(x, dev(b), dev(w), hist if K > 1 else None, bounds(step, device),
+            q = ops.qkv_conv_append(x, dev(b), dev(w.t().contiguous()), hist if K > 1 else None, bounds(step, device),
                                     i32([SLOTS[i] for i, _, _ in step], device), dev(qn), dev(kn), "all", 1e-5, cs, "half", pos,
                                     slots, kc, vc, H, max_len=max(c for _, _, c in step))
             at = 0
@@ -171,7 +171,7 @@ def test_projected_rows_on_their_way_to_the_cache(device, dtype, H, G, dk, dv, K
             close(kc.view(-1, G, dk)[rows], want[i][1], dtype)
             close(vc.view(-1, G, dv)[rows], want[i][2], dtype)
             if K > 1 and n >= K - 1:
-                close(hist[SLOTS[i]].t(), (d(xs[i]) + d(b))[n - K + 1:], torch.float32)
+                close(hist[SLOTS[i]], (d(xs[i]) + d(b))[n - K + 1:], torch.float32)
         used = torch.zeros(60 * page, dtype=torch.bool)
         used[[cell(i, t) for i, n in enumerate(LENS) for t in range(n)]] = True
         assert bool((kc.view(-1, G, dk)[~used.to(device)] == 7).all()) and bool((vc.view(-1, G, dv)[~used.to(device)] == 7).all())
@@ -204,10 +204,10 @@ def test_projected_rows_with_other_options(device, dtype, layout):
     live = [20 + i for i in range(T) if i != 3]
     close(vc.view(-1, G, dv)[live], d(x)[[i for i in range(T) if i != 3], (H + G) * dk:].view(-1, G, dv), dtype)
     assert not vc.view(-1, G, dv)[23].any() and not kc.view(-1, G, dk)[23].any()
-    hist = rnd(2, x.shape[1], 2, seed=8, device=device)
+    hist = rnd(2, 2, x.shape[1], seed=8, device=device)
     keep = hist.clone()
     for n in (1, 5):
-        ops.qkv_conv_append(dev(x)[:n], None, rnd(x.shape[1], 3, seed=9, device=device), hist, i32([0, n], device), i32([1], device),
+        ops.qkv_conv_append(dev(x)[:n], None, rnd(3, x.shape[1], seed=9, device=device), hist, i32([0, n], device), i32([1], device),
                             None, None, "all", 1e-5, None, "half", i32(range(n), device), slots[:n], kc, vc, H, write_state=False,
                             max_len=n)
     assert torch.equal(hist, keep)
@@ -287,18 +287,18 @@ DELTA = [(6, 3, 40, 24, 4), (2, 2, 128, 128, 4), (1, 1, 13, 19, 1), (4, 1, 64, 7
 def test_channel_delta_prompts_portions_and_decode(device, dtype, H, G, dk, dv, K):
     xs, As, Bs, w, A, bias, want = delta_case(H, G, dk, dv, K, dtype)
     dev = lambda t: t.to(device)                                            # noqa: E731
-    C = w.shape[0]
+    C, wt = w.shape[0], w.t().contiguous()
     norm, eps = 1 + rnd(dv, seed=7, k=0.2), 1e-5
     gates = [rnd(n, H * dv, seed=300 + n, dtype=dtype) for n in LENS]
     for name, cuts in CUTS.items():
-        hist, state = torch.full((6, C, K - 1), 9.0, device=device), torch.full((6, H, dv, dk), 9.0, device=device)
+        hist, state = torch.full((6, K - 1, C), 9.0, device=device), torch.full((6, H, dv, dk), 9.0, device=device)
         hist[SLOTS], state[SLOTS] = 0.0, 0.0
         got = [[] for _ in LENS]
         for step in portions(LENS, cuts):
             cat = lambda ts: dev(torch.cat([ts[i][a:a + c] for i, a, c in step]))                            # noqa: E731
             wide = torch.cat([cat(xs), cat(Bs)], 1)                         # column slices of one projection
             ml = max(c for _, _, c in step)
-            args = (wide[:, :C], dev(w), hist, cat(As), dev(A), dev(bias), wide[:, C:], state, bounds(step, device),
+            args = (wide[:, :C], dev(wt), hist, cat(As), dev(A), dev(bias), wide[:, C:], state, bounds(step, device),
                     i32([SLOTS[i] for i, _, _ in step], device), H, G, dk, dv)
             if ml == 1 and device != "cpu":
                 y = ops.sm100.channel_delta_decode(*args, cat(gates), dev(norm), eps)
@@ -323,8 +323,8 @@ def test_channel_delta_without_writing_the_state(device, dtype):
     H, G, dk, dv, K = 2, 1, 32, 24, 3
     xs, As, Bs, w, A, bias, want = delta_case(H, G, dk, dv, K, dtype, [30])
     dev = lambda t: t.to(device)                                            # noqa: E731
-    hist, state = torch.zeros(2, w.shape[0], K - 1, device=device), torch.zeros(2, H, dv, dk, device=device)
-    o = ops.channel_delta(dev(xs[0]), dev(w), hist, dev(As[0]), dev(A), dev(bias), dev(Bs[0]), state, i32([0, 30], device),
+    hist, state = torch.zeros(2, K - 1, w.shape[0], device=device), torch.zeros(2, H, dv, dk, device=device)
+    o = ops.channel_delta(dev(xs[0]), dev(w.t().contiguous()), hist, dev(As[0]), dev(A), dev(bias), dev(Bs[0]), state, i32([0, 30], device),
                           i32([1], device), H, G, dk, dv, write_state=False, max_len=30)
     close(o, want[0][0].reshape(30, -1), dtype)
     assert not state.any() and not hist.any()
@@ -339,19 +339,19 @@ def test_channel_delta_in_slices(dtype, H, G, dk, dv, K, monkeypatch):
     xs, As, Bs, w, A, bias, want = delta_case(H, G, dk, dv, K, dtype, lens)
     dev = lambda t: t.cuda()                                                # noqa: E731
     ws = ops.sm100.Workspace.get(torch.device("cuda", torch.cuda.current_device()))
-    for room in (1, 40 * 4 * ops.sm100.ext().channel_delta_record_floats(H, dk, dv)):
+    for room in (1, 40 * 4 * ops.sm100.ext().channel_delta_record_floats(H, dk, dv, dtype == torch.float32)):
         monkeypatch.setattr(ops.sm100, "DELTA_SCRATCH", room)
         ws._cache.pop("channel_delta_rec", None)
-        hist, state = torch.zeros(6, w.shape[0], K - 1).cuda(), torch.zeros(6, H, dv, dk).cuda()
+        hist, state = torch.zeros(6, K - 1, w.shape[0]).cuda(), torch.zeros(6, H, dv, dk).cuda()
         cu = i32([0] + torch.tensor(lens).cumsum(0).tolist(), "cuda")
-        o = ops.channel_delta(dev(torch.cat(xs)), dev(w), hist, dev(torch.cat(As)), dev(A), dev(bias), dev(torch.cat(Bs)), state, cu,
+        o = ops.channel_delta(dev(torch.cat(xs)), dev(w.t().contiguous()), hist, dev(torch.cat(As)), dev(A), dev(bias), dev(torch.cat(Bs)), state, cu,
                               i32([3, 0, 5, 1, 2], "cuda"), H, G, dk, dv, max_len=333)
         for i, (s, n) in enumerate(zip((3, 0, 5, 1, 2), lens)):
             at = sum(lens[:i])
             close(o[at:at + n], want[i][0].reshape(n, -1), dtype)
             close(state[s].transpose(1, 2), want[i][1], dtype, 2e-5, 2e-3)
             if n >= K - 1:
-                close(hist[s].t(), d(xs[i])[n - K + 1:], torch.float32)
+                close(hist[s], d(xs[i])[n - K + 1:], torch.float32)
         ws._cache.pop("channel_delta_rec", None)
     status_ok("cuda:0")
 
@@ -368,9 +368,9 @@ def test_channel_delta_slow_and_instant_decays(device, dtype, raw, first):
     x[0, dk] = 40.0                                                         # but the first token writes channel 0
     x[:, 2 * dk:] = 2.0
     a, b = torch.full((n, dk), raw), torch.full((n, 1), 30.0)
-    w = torch.ones(x.shape[1], 1)
+    w = torch.ones(1, x.shape[1])
     dev = lambda t: t.to(dtype).to(device)                                  # noqa: E731
-    state, hist = torch.zeros(1, 1, dv, dk, device=device), torch.zeros(1, x.shape[1], 0, device=device)
+    state, hist = torch.zeros(1, 1, dv, dk, device=device), torch.zeros(1, 0, x.shape[1], device=device)
     out = []
     cuts = [400, 1, 1, 98]
     for c in range(len(cuts)):
