@@ -423,28 +423,45 @@ __global__ void __launch_bounds__(128) delta_history_kernel(const ChannelDeltaAr
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// Decode: one CTA per (head, sequence), one token per sequence. The state loads are issued in front of the wait for the
-// projections (nothing of this step writes them). q / k channels may serve several heads: the last of them to have read the
+// Decode: one CTA per (head, sequence), one token per sequence. q / k channels may serve several heads: the last of them to have read the
 // old history (an arrival counter per sequence and key head) replaces it.
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int DEC_IT = 4;                // column groups of a warp whose loads are in flight together
 
-template <typename T, int NI>
+template <typename T, int NI, int KC>
 __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArgs a, const T* gate, long ldg, const float* norm_w,
                                                            float eps, unsigned int* ctr) {
-  constexpr int DKP = 32 * NI;
+  constexpr int DKP = 32 * NI, K1C = KC > 0 ? KC - 1 : 0;
   extern __shared__ float sm[];          // g k | g q | g | k [DKP each] | v [DV] | o [DV]
   __shared__ float red[3][8];
   __shared__ int s_last;
   const int DK = a.DK, DV = a.DV, H = a.H, G = a.G, hpg = H / G;
   const int h = blockIdx.x, n = blockIdx.y, hk = h / hpg;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7, tid = threadIdx.x;
   const int slot = a.slots[n];
   float* gk = sm, *gq = sm + DKP, *gs = sm + 2 * DKP, *ks = sm + 3 * DKP, *vs = sm + 4 * DKP, *os = vs + DV;
   float* state = a.state + (long(slot < 0 ? 0 : slot) * H + h) * DV * DK;
   const int n_it = (DV + 31) / 32;       // groups of 32 columns
+  const int K1 = a.KC - 1, C = 2 * G * DK + H * DV, W = 2 * DK + DV;
+  float* hist = a.conv_state + long(slot < 0 ? 0 : slot) * C * K1;
+  auto channel = [&](int i) { return i < DK ? hk * DK + i : i < 2 * DK ? G * DK + hk * DK + i - DK : 2 * G * DK + h * DV + i - 2 * DK; };
+  // Nothing of this step writes weights, state or history in front of this launch: their loads go out before the wait for
+  // the projections (the first two turns of the convolution's loop, all of the decay's and the norm's for usual sizes).
   uint64_t S[DEC_IT][2 * NI];
   auto column = [&](int it) { return it * 32 + warp * 4 + (lane >> 3); };
+  float tw[2][K1C + 1], th[2][K1C > 0 ? K1C : 1];
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int i = tid + 256 * e;
+    if (KC > 0 && i < W) {
+      const int c = channel(i);
+#pragma unroll
+      for (int j = 0; j <= K1C; ++j) tw[e][j] = a.conv_w[long(j) * C + c];
+#pragma unroll
+      for (int j = 0; j < K1C; ++j) th[e][j] = hist[long(j) * C + c];
+    }
+  }
+  const float db = tid < DK ? a.dt_bias[long(h) * DK + tid] : 0.f, Ah = a.A[h], nw = tid < DV ? norm_w[tid] : 0.f;
   if (slot >= 0) {
 #pragma unroll
     for (int it = 0; it < DEC_IT; ++it)
@@ -453,28 +470,57 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
   griddep_wait();
   griddep_launch();
   if (slot < 0) return;
-  const int K1 = a.KC - 1, C = 2 * G * DK + H * DV;
   const T* x = static_cast<const T*>(a.qkv) + long(n) * a.ld;
-  float* hist = a.conv_state + long(slot) * C * K1;
-  auto channel = [&](int i) { return i < DK ? hk * DK + i : i < 2 * DK ? G * DK + hk * DK + i - DK : 2 * G * DK + h * DV + i - 2 * DK; };
+  const T* ap = static_cast<const T*>(a.a) + long(n) * a.lda + long(h) * DK;
+  const T* gr = gate + long(n) * ldg + long(h) * DV;
+  float tx[2];
+#pragma unroll
+  for (int e = 0; e < 2; ++e) tx[e] = tid + 256 * e < W ? ld_f(x + channel(tid + 256 * e)) : 0.f;
+  const float ta = tid < DK ? ld_f(ap + tid) : 0.f, tg = tid < DV ? ld_f(gr + tid) : 0.f;
+  const float beta = sigmoid_t<T>(ld_f(static_cast<const T*>(a.b) + long(n) * a.ldb + h));
   float qq = 0.f, kk = 0.f;
-  for (int i = threadIdx.x; i < 2 * DK + DV; i += 256) {
+  auto one = [&](int i, float xv, const float* w, const float* hv) {       // a channel: convolution, silu, history
     const int c = channel(i);
     const bool own = hpg == 1 || i >= 2 * DK;
-    const float xv = ld_f(x + c);
     float* hc = hist + c;
-    const float* wc = a.conv_w + c;
-    float acc = wc[long(K1) * C] * xv;
-    for (int j = 0; j < K1; ++j) {
-      const float hv = hc[long(j) * C];
-      acc = fmaf(wc[long(j) * C], hv, acc);
-      if (own && j > 0) hc[long(j - 1) * C] = hv;
+    float acc;
+    if constexpr (KC > 0) {
+      acc = w[K1C] * xv;
+#pragma unroll
+      for (int j = 0; j < K1C; ++j) acc = fmaf(w[j], hv[j], acc);
+      if (own) {
+#pragma unroll
+        for (int j = 1; j < K1C; ++j) hc[long(j - 1) * C] = hv[j];
+        if (K1C > 0) hc[long(K1C - 1) * C] = xv;
+      }
+    } else {
+      const float* wc = a.conv_w + c;
+      acc = wc[long(K1) * C] * xv;
+      for (int j = 0; j < K1; ++j) {
+        const float v = hc[long(j) * C];
+        acc = fmaf(wc[long(j) * C], v, acc);
+        if (own && j > 0) hc[long(j - 1) * C] = v;
+      }
+      if (own && K1 > 0) hc[long(K1 - 1) * C] = xv;
     }
-    if (own && K1 > 0) hc[long(K1 - 1) * C] = xv;
     const float y = silu_t<T>(acc);
     if (i < DK) { gq[i] = y; qq = fmaf(y, y, qq); }
     else if (i < 2 * DK) { ks[i - DK] = y; kk = fmaf(y, y, kk); }
     else vs[i - 2 * DK] = y;
+  };
+#pragma unroll
+  for (int e = 0; e < 2; ++e)
+    if (tid + 256 * e < W) one(tid + 256 * e, tx[e], tw[e], th[e]);
+  for (int i = tid + 512; i < W; i += 256) {
+    float w[K1C + 1], hv[K1C > 0 ? K1C : 1];
+    if constexpr (KC > 0) {
+      const int c = channel(i);
+#pragma unroll
+      for (int j = 0; j <= K1C; ++j) w[j] = a.conv_w[long(j) * C + c];
+#pragma unroll
+      for (int j = 0; j < K1C; ++j) hv[j] = hist[long(j) * C + c];
+    }
+    one(i, ld_f(x + channel(i)), w, hv);
   }
   qq = warp_sum_f(qq);
   kk = warp_sum_f(kk);
@@ -501,13 +547,12 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
   qq = kk = 0.f;
 #pragma unroll
   for (int w = 0; w < 8; ++w) { qq += red[0][w]; kk += red[1][w]; }
-  const float rq = a.scale / sqrtf(qq + a.l2_eps), rk = 1.f / sqrtf(kk + a.l2_eps), Ah = a.A[h];
-  const T* ap = static_cast<const T*>(a.a) + long(n) * a.lda + long(h) * DK;
+  const float rq = a.scale / sqrtf(qq + a.l2_eps), rk = 1.f / sqrtf(kk + a.l2_eps);
   float kq = 0.f;
   for (int c = threadIdx.x; c < DKP; c += 256) {
     float g = 1.f, kv = 0.f, qv = 0.f;
     if (c < DK) {
-      g = decay_t<T>(ld_f(ap + c) + a.dt_bias[long(h) * DK + c], Ah);
+      g = decay_t<T>(ta + db, Ah);        // (256 channels at most: one turn)
       kv = ks[c] * rk;
       qv = gq[c] * rq;
     }
@@ -519,7 +564,6 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
   }
   kq = warp_sum_f(kq);
   if (lane == 0) red[2][warp] = kq;
-  const float beta = sigmoid_t<T>(ld_f(static_cast<const T*>(a.b) + long(n) * a.ldb + h));
   __syncthreads();
   kq = 0.f;
 #pragma unroll
@@ -587,9 +631,9 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const ChannelDeltaArg
 #pragma unroll
   for (int w = 0; w < 8; ++w) oo += red[0][w];
   const float inv = 1.f / sqrtf(oo / float(DV) + eps);
-  const T* gr = gate + long(n) * ldg + long(h) * DV;
   T* out = static_cast<T*>(a.out) + long(n) * a.ldo + long(h) * DV;
-  for (int c = threadIdx.x; c < DV; c += 256) st_f(out + c, os[c] * inv * norm_w[c] * sigmoid_t<T>(ld_f(gr + c)));
+  if (tid < DV) st_f(out + tid, os[tid] * inv * nw * sigmoid_t<T>(tg));
+  for (int c = tid + 256; c < DV; c += 256) st_f(out + c, os[c] * inv * norm_w[c] * sigmoid_t<T>(ld_f(gr + c)));
 }
 
 // RMS norm of each head, times w, times sigmoid(gate): one warp per (row, head)
@@ -682,12 +726,18 @@ int decode_t(const ChannelDeltaArgs& a, const void* gate, long ldg, const float*
   const int DKP = pad_dk(a.DK);
   const size_t smem = size_t(4 * DKP + 2 * a.DV) * 4;
   if (smem > 48 * 1024) return 1;
-#define LB_NI(N_)                                                                                                             \
-  if (DKP == 32 * N_)                                                                                                         \
-    return launch_pdl(delta_decode_kernel<T, N_>, dim3(a.H, a.n_seqs), dim3(256), smem, s, a, static_cast<const T*>(gate), ldg, \
-                      norm_w, eps, ctr) != cudaSuccess;
+#define LB_K(N_, K_)                                                                                                          \
+  return launch_pdl(delta_decode_kernel<T, N_, K_>, dim3(a.H, a.n_seqs), dim3(256), smem, s, a, static_cast<const T*>(gate), ldg, \
+                    norm_w, eps, ctr) != cudaSuccess;
+#define LB_NI(N_)               \
+  if (DKP == 32 * N_) {         \
+    if (a.KC == 4) { LB_K(N_, 4) } \
+    if (a.KC == 3) { LB_K(N_, 3) } \
+    LB_K(N_, 0)                 \
+  }
   LB_NI(1) LB_NI(2) LB_NI(4) LB_NI(8)
 #undef LB_NI
+#undef LB_K
   return 1;
 }
 

@@ -11,12 +11,12 @@
 namespace lb {
 namespace {
 
-constexpr int PROMPT_TOK = 8;
+constexpr int PROMPT_TOK = 4;
 
 // TOK: most tokens of a CTA; VEC: columns per thread and turn; KC 0: any number of taps
 template <typename T, int KC, int TOK, int VEC>
-__global__ void __launch_bounds__(TOK == 1 ? 1024 : 256) qkv_conv_kernel(const QkvConvArgs a) {
-  extern __shared__ float y_s[];                   // [tok][nq + nk]
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_conv_kernel(const QkvConvArgs a) {
+  extern __shared__ __align__(16) float y_s[];     // [tok][nq + nk], then [tok][heads]
   __shared__ float red[2][TOK][32];
   griddep_wait();
   griddep_launch();
@@ -141,75 +141,91 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256) qkv_conv_kernel(const Q
       }
   }
   __syncthreads();
-  // a warp per (token, head); a lane takes PV neighbouring pairs
-  constexpr int PV = VEC == 1 ? 1 : 2;
+  // 1 / root mean square per (token, head)
   const int heads = a.Hq + a.Hkv, half = a.rot / 2;
-  for (int i = warp; i < nt * heads; i += n_warps) {
-    const int t = i / heads, h = i % heads;
-    const bool is_q = h < a.Hq;
-    const float* v = y_s + t * N + h * a.DK;
-    const float* nw = is_q ? a.qw : a.kw;
-    float inv = 1.f;
-    if (nw) {
-      float ss = 0.f;
-      int n = a.DK;
-      if (a.norm_all) {
-        n = is_q ? nq : nk;
-        ss = warp_sum_f(lane < n_warps ? red[is_q ? 0 : 1][t][lane] : 0.f);
-        nw += (is_q ? h : h - a.Hq) * a.DK;
-      } else {
-        for (int d = lane; d < a.DK; d += 32) ss = fmaf(v[d], v[d], ss);
-        ss = warp_sum_f(ss);
-      }
-      inv = 1.f / sqrtf(ss / float(n) + a.eps);
+  float* inv_s = y_s + tok * N;                    // [tok][heads]
+  if (a.qw && a.norm_all) {
+    for (int i = warp; i < 2 * nt; i += n_warps) {
+      const int t = i >> 1, k = i & 1;
+      const float ss = warp_sum_f(lane < n_warps ? red[k][t][lane] : 0.f);
+      const float inv = 1.f / sqrtf(ss / float(k ? nk : nq) + a.eps);
+      for (int h = (k ? a.Hq : 0) + lane; h < (k ? heads : a.Hq); h += 32) inv_s[t * heads + h] = inv;
     }
+    __syncthreads();
+  } else if (a.qw) {
+    for (int i = warp; i < nt * heads; i += n_warps) {
+      const float* v = y_s + (i / heads) * N + (i % heads) * a.DK;
+      float ss = 0.f;
+      for (int d = lane; d < a.DK; d += 32) ss = fmaf(v[d], v[d], ss);
+      ss = warp_sum_f(ss);
+      if (lane == 0) inv_s[i] = 1.f / sqrtf(ss / float(a.DK) + a.eps);
+    }
+    __syncthreads();
+  }
+  // norm and rotation: PV neighbouring pairs of columns per thread and turn (columns past the rotated ones pass in pairs too)
+  constexpr int PV = VEC == 1 ? 1 : 2;
+  const bool wide = PV == 2 && a.rot_half && half % 2 == 0;
+  const int step = wide ? 2 : 1, odd = a.DK & 1;
+  const int per = ((a.DK + odd) / 2) / step;       // turns per head
+  auto item = [&](int i) {
+    const int th = i / per, e = (i - th * per) * step, t = th / heads, h = th - t * heads;
+    const bool is_q = h < a.Hq;
     T* dst;
     if (is_q) {
       dst = static_cast<T*>(a.q_out) + (long(t0 + t) * a.Hq + h) * a.DK;
     } else {
       const long cell = a.slots[t0 + t];
-      if (cell < 0) continue;
+      if (cell < 0) return;
       dst = static_cast<T*>(a.k_cache) + cell * a.k_cell + long(h - a.Hq) * a.DK;
     }
-    const float* cs = a.cos_sin ? a.cos_sin + long(a.positions[t0 + t]) * a.rot : nullptr;
-    if (PV == 2 && a.rot_half && half % 2 == 0) {
-      auto two = [&](int d, float (&o)[2]) {
-        const float2 f = *reinterpret_cast<const float2*>(v + d);
-        o[0] = f.x * inv;
-        o[1] = f.y * inv;
-        if (nw) {
-          o[0] *= nw[d];
-          o[1] *= nw[d + 1];
-        }
-      };
-      auto put = [&](int d, float p, float q) {
-        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(p, q);
-        else *reinterpret_cast<float2*>(dst + d) = make_float2(p, q);
-      };
-      for (int p = 2 * lane; p < half; p += 64) {
-        float f[2], g[2];
-        two(p, f);
-        two(p + half, g);
-        const float2 c = *reinterpret_cast<const float2*>(cs + p), s = *reinterpret_cast<const float2*>(cs + half + p);
-        put(p, f[0] * c.x - g[0] * s.x, f[1] * c.y - g[1] * s.y);
-        put(p + half, g[0] * c.x + f[0] * s.x, g[1] * c.y + f[1] * s.y);
+    const float* v = y_s + t * N + h * a.DK;
+    const float* nw = is_q ? a.qw : a.kw;
+    const float inv = nw ? inv_s[t * heads + h] : 1.f;
+    if (nw && a.norm_all) nw += (is_q ? h : h - a.Hq) * a.DK;
+    const bool turn = e < half;
+    // columns of the pair(s): rotated ones half a rotation (or one column) apart, the others side by side
+    const int i0 = turn ? (a.rot_half ? e : 2 * e) : 2 * e, i1 = turn ? (a.rot_half ? e + half : 2 * e + 1) : 2 * e + step;
+    if (wide) {
+      float2 f = *reinterpret_cast<const float2*>(v + i0), g = *reinterpret_cast<const float2*>(v + i1);
+      f.x *= inv; f.y *= inv; g.x *= inv; g.y *= inv;
+      if (nw) {
+        const float2 wf = *reinterpret_cast<const float2*>(nw + i0), wg = *reinterpret_cast<const float2*>(nw + i1);
+        f.x *= wf.x; f.y *= wf.y; g.x *= wg.x; g.y *= wg.y;
       }
-      for (int d = 2 * half + 2 * lane; d < a.DK; d += 64) {
-        float f[2];
-        two(d, f);
-        put(d, f[0], f[1]);
+      if (turn) {
+        const float* cs = a.cos_sin + long(a.positions[t0 + t]) * a.rot;
+        const float2 c = *reinterpret_cast<const float2*>(cs + e), s = *reinterpret_cast<const float2*>(cs + half + e);
+        const float2 p = make_float2(f.x * c.x - g.x * s.x, f.y * c.y - g.y * s.y);
+        g = make_float2(g.x * c.x + f.x * s.x, g.y * c.y + f.y * s.y);
+        f = p;
       }
-      continue;
+      if constexpr (sizeof(T) == 2) {
+        *reinterpret_cast<uint32_t*>(dst + i0) = pack_bf16x2(f.x, f.y);
+        *reinterpret_cast<uint32_t*>(dst + i1) = pack_bf16x2(g.x, g.y);
+      } else {
+        *reinterpret_cast<float2*>(dst + i0) = f;
+        *reinterpret_cast<float2*>(dst + i1) = g;
+      }
+      return;
     }
-    for (int p = lane; p < half; p += 32) {
-      const int i0 = a.rot_half ? p : 2 * p, i1 = a.rot_half ? p + half : 2 * p + 1;
-      const float f = v[i0] * inv * (nw ? nw[i0] : 1.f), g = v[i1] * inv * (nw ? nw[i1] : 1.f);
-      const float c = cs[p], s = cs[half + p];
-      st_f(dst + i0, f * c - g * s);
-      st_f(dst + i1, g * c + f * s);
+    float f = v[i0] * inv * (nw ? nw[i0] : 1.f), g = i1 < a.DK ? v[i1] * inv * (nw ? nw[i1] : 1.f) : 0.f;
+    if (turn) {
+      const float* cs = a.cos_sin + long(a.positions[t0 + t]) * a.rot;
+      const float c = cs[e], s = cs[half + e], p = f * c - g * s;
+      g = g * c + f * s;
+      f = p;
     }
-    for (int d = 2 * half + lane; d < a.DK; d += 32) st_f(dst + d, v[d] * inv * (nw ? nw[d] : 1.f));
-  }
+    st_f(dst + i0, f);
+    if (i1 < a.DK) st_f(dst + i1, g);
+  };
+  const int total = nt * heads * per;
+  int i = threadIdx.x;
+  if constexpr (TOK > 1)
+    for (; i + 3 * int(blockDim.x) < total; i += 4 * blockDim.x) {
+#pragma unroll
+      for (int u = 0; u < 4; ++u) item(i + u * blockDim.x);
+    }
+  for (; i < total; i += blockDim.x) item(i);
 }
 
 template <typename T>
@@ -231,7 +247,7 @@ __global__ void __launch_bounds__(128) qkv_history_kernel(const QkvConvArgs a) {
 template <typename T, int TOK, int VEC>
 int launch_v(const QkvConvArgs& a, cudaStream_t s) {
   const int taps = a.conv_w ? a.KC : 1, C = (a.Hq + a.Hkv) * a.DK + a.Hkv * a.DV;
-  const int smem = (a.Hq + a.Hkv) * a.DK * 4 * a.tok;
+  const int smem = (a.Hq + a.Hkv) * (a.DK + 1) * 4 * a.tok;
   const dim3 grid(a.one ? a.n_seqs : a.T / a.tok + a.n_seqs);
   const int nt = TOK == 1 ? min(1024, max(64, (C / VEC + 31) / 32 * 32)) : 256;
 #define LB_KC(K_)                                                                                                            \
@@ -252,7 +268,7 @@ template <typename T>
 int launch_t(const QkvConvArgs& a, cudaStream_t s) {
   auto al = [](const void* p, size_t n) { return reinterpret_cast<uintptr_t>(p) % n == 0; };
   const bool vec = a.DK % 4 == 0 && a.DV % 4 == 0 && a.ld % 4 == 0 && al(a.x, 4 * sizeof(T)) && al(a.in_b, 16) && al(a.conv_w, 16) &&
-                   al(a.conv_state, 16) && al(a.v_cache, 4 * sizeof(T)) && al(a.k_cache, 8) && al(a.q_out, 8) && al(a.cos_sin, 8);
+                   al(a.conv_state, 16) && al(a.v_cache, 4 * sizeof(T)) && al(a.k_cache, 8) && al(a.q_out, 8) && al(a.cos_sin, 8) && al(a.qw, 8) && al(a.kw, 8);
   const int rc = a.tok == 1 ? (vec ? launch_v<T, 1, 4>(a, s) : launch_v<T, 1, 1>(a, s))
                             : (vec ? launch_v<T, PROMPT_TOK, 4>(a, s) : launch_v<T, PROMPT_TOK, 1>(a, s));
   if (rc) return rc;
@@ -268,7 +284,7 @@ int launch_t(const QkvConvArgs& a, cudaStream_t s) {
 int qkv_conv_append_launch(QkvConvArgs a, bool f32, cudaStream_t s) {
   if (a.T <= 0 || a.n_seqs <= 0) return 0;
   if (a.Hkv <= 0 || a.Hq % a.Hkv || a.rot % 2 || a.rot > a.DK || a.rot < 0 || (a.conv_w && a.KC < 1) || a.n_seqs > 65535) return 1;
-  const long row = long(a.Hq + a.Hkv) * a.DK * 4;
+  const long row = long(a.Hq + a.Hkv) * (a.DK + 1) * 4;
   if (row > 200 * 1024) return 1;
   a.tok = a.max_len <= 1 ? 1 : PROMPT_TOK;
   a.one = a.max_len <= 1 && a.T == a.n_seqs;
