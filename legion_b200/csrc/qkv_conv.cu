@@ -18,6 +18,34 @@ template <typename T, int KC, int TOK, int VEC>
 __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_conv_kernel(const QkvConvArgs a) {
   extern __shared__ __align__(16) float y_s[];     // [tok][nq + nk], then [tok][heads]
   __shared__ float red[2][TOK][32];
+  const int nq = a.Hq * a.DK, nk = a.Hkv * a.DK, nv = a.Hkv * a.DV, C = nq + nk + nv, N = nq + nk;
+  const int taps = a.conv_w ? a.KC : 1, K1 = taps - 1;
+  // A step with one token per sequence: what the projection in front of this launch does not write is on its way before the
+  // wait (bias, taps and history of the thread's first columns, the token's position and cell).
+  constexpr bool EARLY = TOK == 1 && KC > 1;
+  constexpr int EK = EARLY ? KC : 1;
+  const bool early = EARLY && a.one;
+  float eb[VEC], ew[EK][VEC], eh[EK][VEC];
+  int pos1 = 0;
+  long cell1 = -1;
+  if constexpr (EARLY) {
+    const int c = threadIdx.x * VEC;
+    if (early && c < C) {
+      const float* h = a.conv_state + long(a.state_slots[blockIdx.x]) * K1 * C + c;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) eb[j] = 0.f;
+      if (a.in_b) ld_vec<VEC>(a.in_b + c, eb);
+#pragma unroll
+      for (int k = 0; k < KC; ++k) ld_vec<VEC>(a.conv_w + long(k) * C + c, ew[k]);
+#pragma unroll
+      for (int k = 0; k < KC - 1; ++k) ld_vec<VEC>(h + long(k) * C, eh[k]);
+    }
+    if (early) {
+      const int t = a.cu[blockIdx.x];
+      pos1 = a.positions[t];
+      cell1 = a.slots[t];
+    }
+  }
   griddep_wait();
   griddep_launch();
   const int tok = a.tok;
@@ -38,9 +66,8 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
   }
   if (t0 >= s1) return;
   const int nt = min(tok, s1 - t0);
-  const int nq = a.Hq * a.DK, nk = a.Hkv * a.DK, nv = a.Hkv * a.DV, C = nq + nk + nv, N = nq + nk;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
-  const int taps = a.conv_w ? a.KC : 1, K1 = taps - 1;
+  if (TOK == 1 && !early) { pos1 = a.positions[t0]; cell1 = a.slots[t0]; }
   const bool update = a.write_state && a.max_len <= 1 && K1 > 0;
   const T* x = static_cast<const T*>(a.x);
   float* hist = K1 > 0 ? a.conv_state + long(a.state_slots[seq]) * K1 * C : nullptr;
@@ -48,10 +75,11 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
 #pragma unroll
   for (int t = 0; t < TOK; ++t) sq[t] = sk[t] = 0.f;
   for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+    const bool have = early && c == int(threadIdx.x) * VEC;
     float b[VEC], y[TOK][VEC];
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) b[j] = 0.f;
-    if (a.in_b) ld_vec<VEC>(a.in_b + c, b);
+    for (int j = 0; j < VEC; ++j) b[j] = have ? eb[j] : 0.f;
+    if (a.in_b && !have) ld_vec<VEC>(a.in_b + c, b);
     if constexpr (KC > 0) {
       float u[KC - 1 + TOK][VEC], w[KC][VEC];
 #pragma unroll
@@ -64,6 +92,9 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
           ld_vec<VEC>(x + long(s) * a.ld + c, u[i]);
 #pragma unroll
           for (int j = 0; j < VEC; ++j) u[i][j] += b[j];
+        } else if (have) {
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) u[i][j] = eh[i < EK ? i : 0][j];
         } else {
           ld_vec<VEC>(hist + long(K1 + (s - s0)) * C + c, u[i]);
         }
@@ -73,6 +104,9 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
         if (KC == 1 && !a.conv_w) {
 #pragma unroll
           for (int j = 0; j < VEC; ++j) w[k][j] = 1.f;
+        } else if (have) {
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) w[k][j] = ew[k < EK ? k : 0][j];
         } else {
           ld_vec<VEC>(a.conv_w + long(k) * C + c, w[k]);
         }
@@ -127,7 +161,7 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
 #pragma unroll
       for (int t = 0; t < TOK; ++t)
         if (t < nt) {
-          const long cell = a.slots[t0 + t];
+          const long cell = TOK == 1 ? cell1 : long(a.slots[t0 + t]);
           if (cell >= 0) st_vec<VEC>(static_cast<T*>(a.v_cache) + cell * a.v_cell + (c - N), y[t]);
         }
     }
@@ -144,7 +178,11 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
   // 1 / root mean square per (token, head)
   const int heads = a.Hq + a.Hkv, half = a.rot / 2;
   float* inv_s = y_s + tok * N;                    // [tok][heads]
-  if (a.qw && a.norm_all) {
+  float inv_q = 1.f, inv_k = 1.f;
+  if (TOK == 1 && a.qw && a.norm_all) {            // every warp adds up for itself
+    inv_q = 1.f / sqrtf(warp_sum_f(lane < n_warps ? red[0][0][lane] : 0.f) / float(nq) + a.eps);
+    inv_k = 1.f / sqrtf(warp_sum_f(lane < n_warps ? red[1][0][lane] : 0.f) / float(nk) + a.eps);
+  } else if (a.qw && a.norm_all) {
     for (int i = warp; i < 2 * nt; i += n_warps) {
       const int t = i >> 1, k = i & 1;
       const float ss = warp_sum_f(lane < n_warps ? red[k][t][lane] : 0.f);
@@ -174,13 +212,13 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
     if (is_q) {
       dst = static_cast<T*>(a.q_out) + (long(t0 + t) * a.Hq + h) * a.DK;
     } else {
-      const long cell = a.slots[t0 + t];
+      const long cell = TOK == 1 ? cell1 : long(a.slots[t0 + t]);
       if (cell < 0) return;
       dst = static_cast<T*>(a.k_cache) + cell * a.k_cell + long(h - a.Hq) * a.DK;
     }
     const float* v = y_s + t * N + h * a.DK;
     const float* nw = is_q ? a.qw : a.kw;
-    const float inv = nw ? inv_s[t * heads + h] : 1.f;
+    const float inv = !nw ? 1.f : TOK == 1 && a.norm_all ? (is_q ? inv_q : inv_k) : inv_s[t * heads + h];
     if (nw && a.norm_all) nw += (is_q ? h : h - a.Hq) * a.DK;
     const bool turn = e < half;
     // columns of the pair(s): rotated ones half a rotation (or one column) apart, the others side by side
@@ -193,7 +231,7 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
         f.x *= wf.x; f.y *= wf.y; g.x *= wg.x; g.y *= wg.y;
       }
       if (turn) {
-        const float* cs = a.cos_sin + long(a.positions[t0 + t]) * a.rot;
+        const float* cs = a.cos_sin + long(TOK == 1 ? pos1 : a.positions[t0 + t]) * a.rot;
         const float2 c = *reinterpret_cast<const float2*>(cs + e), s = *reinterpret_cast<const float2*>(cs + half + e);
         const float2 p = make_float2(f.x * c.x - g.x * s.x, f.y * c.y - g.y * s.y);
         g = make_float2(g.x * c.x + f.x * s.x, g.y * c.y + f.y * s.y);
@@ -210,7 +248,7 @@ __global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, TOK == 1 ? 1 : 4) qkv_c
     }
     float f = v[i0] * inv * (nw ? nw[i0] : 1.f), g = i1 < a.DK ? v[i1] * inv * (nw ? nw[i1] : 1.f) : 0.f;
     if (turn) {
-      const float* cs = a.cos_sin + long(a.positions[t0 + t]) * a.rot;
+      const float* cs = a.cos_sin + long(TOK == 1 ? pos1 : a.positions[t0 + t]) * a.rot;
       const float c = cs[e], s = cs[half + e], p = f * c - g * s;
       g = g * c + f * s;
       f = p;
