@@ -201,7 +201,9 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
 constexpr int ROUTE_LSTR = 64 * 512;          // floats between the logit planes of two K splits
 constexpr int ROUTE_MAX_KSPLIT = 4;
 
-template <int MAXE>
+// EXT: weights by the sum + 1e-20 (renorm 2) and the shared expert as several groups; a variant of its own, since the launch
+// is latency and code it skips still costs instruction fetches.
+template <int MAXE, bool EXT>
 __global__ void __launch_bounds__(512) moe_route_small_kernel(
     const __nv_bfloat16* __restrict__ x, long ldx, const float* __restrict__ norm_w, float eps, float w_offset,
     __nv_bfloat16* __restrict__ x_normed, long ldn, const __nv_bfloat16* __restrict__ w, long ldw, int H,
@@ -468,7 +470,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) wsum += __shfl_xor_sync(0xffffffffu, wsum, o);
       if (lane < k) {
-        if (renorm) w = w / (renorm == 2 ? wsum + 1e-20f : fmaxf(wsum, 6.1e-5f));
+        if (renorm) w = w / (EXT && renorm == 2 ? wsum + 1e-20f : fmaxf(wsum, 6.1e-5f));
         ids[t * k + lane] = my_id;
         wts[t * k + lane] = w * route_scale;
       }
@@ -478,7 +480,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
   // ---- dense routing tables, indexed by local expert: rows e * bn + t of the intermediate belong to expert e and
   // token t. Each token CTA writes its token's column of out_rows / tok_scale (pair index t * k + c where the
   // token chose the expert, -1 elsewhere) and marks the experts it chose as active.
-  const int P = T * k, kp = k + shared_rows;
+  const int P = T * k, kp = EXT ? k + shared_rows : k;
   for (int t = blockIdx.x; t < T; t += gridDim.x) {
     s_chosen[tid] = -1;
     __syncthreads();
@@ -497,12 +499,12 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
         active[local] = 1;
       }
     }
-    if (tid < shared_rows || (shared_slot && tid == 0)) {
+    if ((EXT && tid < shared_rows) || (shared_slot && tid == 0)) {
       // the shared expert (stacked behind this rank's routed experts as group n_local) is used by every token:
       // its output rows are the pairs P .. P + T - 1, weighted by the sigmoid of its gate (or 1)
       // (shared_rows: the shared expert as that many groups, its output rows behind the token's own pairs)
-      const int slot = n_local + (shared_rows ? tid : 0);
-      out_rows[slot * bn + t] = shared_rows ? t * kp + k + tid : P + t;
+      const int slot = n_local + (EXT && shared_rows ? tid : 0);
+      out_rows[slot * bn + t] = EXT && shared_rows ? t * kp + k + tid : P + t;
       float gl = 0.f;
       if (sh_gate_w)
         for (int sp = 0; sp < ksplit; ++sp) gl += __ldcg(&sh_logit[sp * 64 + t]);
@@ -540,11 +542,17 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
     tile_ntok[slot] = T;
   }
   if (tid == 0) {
-    const int n_shared = shared_rows ? shared_rows : (shared_slot ? 1 : 0);
-    for (int i = 0; i < n_shared; ++i) {
+    int n_shared = shared_slot ? 1 : 0;
+    if constexpr (EXT) n_shared = shared_rows ? shared_rows : n_shared;
+    auto tile = [&](int i) {
       tile_group[n_active + i] = n_local + i;
       slot_base[n_active + i] = (n_local + i) * bn;
       tile_ntok[n_active + i] = T;
+    };
+    if constexpr (EXT) {
+      for (int i = 0; i < n_shared; ++i) tile(i);
+    } else {
+      if (shared_slot) tile(0);
     }
     const int n_slots = n_active + n_shared;
     meta[0] = n_slots;
@@ -575,23 +583,23 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
   if (size_t(tpp) * Hs * 2 > 200 * 1024) return 1;
   const int smem = tpp * Hs * 2;
   const int grid = ((E + (sh_gate_w ? 1 : 0) + epc - 1) / epc) * ksplit;
-#define LB_ROUTE(MAXE)                                                                                              \
+#define LB_ROUTE(MAXE, EXT)                                                                                         \
   {                                                                                                                 \
     static int smem_set = 0;                                                                                        \
+    auto kfn = moe_route_small_kernel<MAXE, EXT>;                                                                   \
     if (smem > smem_set) {                                                                                          \
-      if (cudaFuncSetAttribute(moe_route_small_kernel<MAXE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=  \
-          cudaSuccess)                                                                                              \
-        return 1;                                                                                                   \
+      if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return 1;    \
       smem_set = smem;                                                                                              \
     }                                                                                                               \
-    launch_pdl(moe_route_small_kernel<MAXE>, dim3(grid), dim3(512), smem, s, xb, ldx, norm_w, eps, w_offset, xn,   \
+    launch_pdl(kfn, dim3(grid), dim3(512), smem, s, xb, ldx, norm_w, eps, w_offset, xn,                             \
                ldn, wb, ldw, H, logits, bias, E, k, mode, renorm, route_scale, n_group, topk_group, group_top, ids, wts, T, \
                bn, tile_group, slot_base, tile_ntok, meta, out_rows, tok_scale, done_ctr, e_lo, n_local, sg,        \
-               sh_logit, shared_slot, shared_rows, epc, tpp, ksplit, status, active);                                                    \
+               sh_logit, shared_slot, shared_rows, epc, tpp, ksplit, status, active);                               \
   }
-  if (E <= 128) LB_ROUTE(128)
-  else if (E <= 256) LB_ROUTE(256)
-  else LB_ROUTE(512)
+  const bool ext = shared_rows > 0 || renorm == 2;
+  if (E <= 128) { if (ext) LB_ROUTE(128, true) else LB_ROUTE(128, false) }
+  else if (E <= 256) { if (ext) LB_ROUTE(256, true) else LB_ROUTE(256, false) }
+  else { if (ext) LB_ROUTE(512, true) else LB_ROUTE(512, false) }
 #undef LB_ROUTE
   return cudaGetLastError() != cudaSuccess;
 }
