@@ -27,7 +27,7 @@ NVCC_FLAGS = [
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
 PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any",
-           "channel_delta", "channel_delta_mma", "qkv_conv"}
+           "channel_delta", "channel_delta_mma", "qkv_conv", "depth_step", "forget_scan", "forget_scan_sm100"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:
@@ -64,7 +64,7 @@ CORE = {"gemm_sm100", "sgemm", "elementwise", "sampling", "spec", "tmap", "logit
 _ATTN = {"attn_prefill_sm100", "attn_decode_sm100", "attn_decode", "attn_general"}
 _SCAN = {"linear_scan", "linear_scan_sm100", "conv1d", "conv_any"}
 KIND_KERNELS = {
-    "attn": _ATTN, "lightning": _SCAN, "ssd": _SCAN, "parallel": _ATTN | _SCAN,
+    "attn": _ATTN, "lightning": _SCAN, "ssd": _SCAN, "hgrn2": {"forget_scan", "forget_scan_sm100"},
     "latent": {"attn_mla_sm100", "latent_attn", "attn_prefill_sm100", "attn_decode", "attn_general"},
     "rglru": {"diag_scan", "conv1d", "conv_any"},
     "channel_delta": {"channel_delta", "channel_delta_mma"},
@@ -75,7 +75,10 @@ def kernels_of(cfg) -> set:
     """Source files (without suffix) a ``ModelConfig`` needs beside ``CORE``."""
     if cfg.layers is None:
         return _ATTN | {"moe", "attn_mla_sm100"}
-    need = set().union(*(KIND_KERNELS[x.mixer.kind] for x in cfg.layers)) | {"resid_step" if cfg.sandwich_norm else "hyper"}
+    parts = [m for x in cfg.layers for m in ((x.mixer.left, x.mixer.right) if x.mixer.kind == "parallel" else (x.mixer,))]
+    need = set().union(*(KIND_KERNELS[m.kind] for m in parts)) | {"resid_step" if cfg.sandwich_norm else "hyper"}
+    if cfg.parallel_sublayers:
+        need |= {"depth_step"}
     if any(a is not None and not a.direct() for a in map(cfg.attn_spec, range(cfg.n_layer))):
         need |= {"qkv_conv"}
     return need | {"moe"} if cfg.n_expert else need

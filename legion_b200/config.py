@@ -31,6 +31,9 @@ class AttnSpec:
     conv: int = 0                      # taps of the short convolution (0: none)
     rot: Optional["RotarySpec"] = None
     softcap: float = 0.0               # cap * tanh(score / cap)
+    keep_first: int = 0                # with a window: this many first tokens of the sequence stay visible
+    sink: bool = False                 # a learned number per head whose exponential joins the softmax's denominator
+    gate: str = "none"                 # head: each head's output times the sigmoid of one more row of the projection
     kind: str = "attn"
 
     def direct(self) -> bool:
@@ -61,10 +64,20 @@ class SsdSpec:
 
 
 @dataclass
+class Hgrn2Spec:
+    """HGRN2: a matrix state per head whose rows keep the share f of themselves and take 1 - f of the value, f a vector over
+    the key channels held above a learned lower bound; silu on q, an RMS norm per head behind the state."""
+    heads: int
+    dim: int                           # query / forget-gate head size
+    vdim: int
+    kind: str = "hgrn2"
+
+
+@dataclass
 class ParallelSpec:
     """Two mixers side by side over the same input: left_scale * left + right_scale * right."""
     left: AttnSpec
-    right: SsdSpec
+    right: object                      # SsdSpec | Hgrn2Spec
     left_scale: float = 1.0
     right_scale: float = 1.0
     kind: str = "parallel"
@@ -156,6 +169,7 @@ class LoopSpec:
 class DenseSpec:
     ff: int
     act: str = "silu"                  # xielu: un-gated, with two learned numbers per layer
+    bias: bool = False                 # of all projections
     kind: str = "dense"
 
     def gated(self) -> bool:
@@ -168,7 +182,8 @@ class MoeSpec:
     top: int
     ff: int
     act: str = "silu"
-    router: str = "softmax"            # softmax | sigmoid | softmax_bias (selection by softmax score + correction)
+    router: str = "softmax"            # softmax | biased_softmax (a bias on the logits) | sigmoid | softmax_bias (selection
+                                       # by softmax score + correction)
     correction: bool = False
     renorm: object = True              # chosen weights divided by their sum (held away from zero); "sum": by the plain sum
     scale: float = 1.0                 # ... and multiplied by this
@@ -196,7 +211,7 @@ class LayerSpec:
 
 _SPECS = {c.__dataclass_fields__["kind"].default: c
           for c in (AttnSpec, LightningSpec, SsdSpec, ParallelSpec, RotarySpec, LatentSpec, RgLruSpec, ChannelDeltaSpec, LoopSpec,
-                    DenseSpec, MoeSpec)}
+                    Hgrn2Spec, DenseSpec, MoeSpec)}
 
 
 def spec_from(d):
@@ -321,6 +336,10 @@ class ModelConfig:
     residual_mult: float = 1.0
     embed_norm: bool = False           # the embedding rows pass the model's norm first
     loop: Optional[LoopSpec] = None    # ``layers`` then has one entry per layer run (``LoopSpec.expand``)
+    # with ``layers`` and one stream: both sublayers of a layer read one norm of the residual, x + mixer(h) + ffn(h)
+    parallel_sublayers: bool = False
+    residual_gate: bool = False        # ... each result times the sigmoid of a projection (with bias) of h, column by column
+    depth_average: bool = False        # ... and the next layer reads a learned sum of the embedding and all results so far
     # multi-token prediction
     mtp_layers: int = 0
     # weights
@@ -332,6 +351,9 @@ class ModelConfig:
             self.layers, self.loop = [spec_from(x) for x in self.layers], spec_from(self.loop)
             self.n_layer = len(self.layers)
             self.layer_kinds = [x.mixer.kind for x in self.layers]
+            if not self.parallel_sublayers and (self.residual_gate or self.depth_average
+                                                or any(getattr(x.mlp, "bias", False) for x in self.layers)):
+                raise ValueError("residual gates, depth averages and feed-forward biases come with parallel sublayers")
             attn = [a for a in (self.attn_spec(il) for il in range(self.n_layer)) if a is not None]
             lat = [x.mixer for x in self.layers if isinstance(x.mixer, LatentSpec)]
             if lat:
@@ -371,9 +393,34 @@ class ModelConfig:
     def recurrent_spec(self, il: int):
         """The part of layer il that carries a recurrent state, of a stack with specifications."""
         m = self.layers[il].mixer
-        if isinstance(m, (LightningSpec, SsdSpec, RgLruSpec, ChannelDeltaSpec)):
+        if isinstance(m, (LightningSpec, SsdSpec, RgLruSpec, ChannelDeltaSpec, Hgrn2Spec)):
             return m
         return m.right if isinstance(m, ParallelSpec) else None
+
+    def mix_columns(self, il: int) -> dict:
+        """First column of each part of the stacked input projection ``mix.in``, and its width (``end``): q | k | v | head
+        gates of the attention part, the columns of the recurrent part, the residual gates of both sublayers. Parts behind
+        q | k | v of an attention part start on 16-byte boundaries, except the state-space columns (``ssd``)."""
+        up8 = lambda n: -(-n // 8) * 8                               # noqa: E731
+        a, r, col, n = self.attn_spec(il), self.recurrent_spec(il), {}, 0
+        if a is not None:
+            for part, w in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+                col[part], n = n, n + w
+            if a.gate == "head":
+                col["g"] = up8(n)
+                n = col["g"] + a.heads
+        if r is not None and r.kind == "ssd":
+            col["ssd"] = n
+            n += 2 * r.heads * r.vdim + 2 * r.groups * r.state + r.heads
+        elif r is not None and r.kind == "hgrn2":
+            for part, w in (("rq", r.heads * r.dim), ("rf", r.heads * r.dim), ("rv", r.heads * r.vdim)):
+                col[part] = up8(n)
+                n = col[part] + w
+        for part in ("rg1", "rg2")[:0 if not self.residual_gate else 1 if self.layers[il].mlp is None else 2]:
+            col[part] = up8(n)
+            n = col[part] + self.hidden
+        col["end"] = up8(n) if "rq" in col or "rg1" in col or "g" in col else n
+        return col
 
     def attn_history(self, il: int):
         """(tokens, channels) of the projected q, k and v that the short convolution of an attention layer keeps, or None."""
@@ -388,6 +435,11 @@ class ModelConfig:
         if r is None:
             return 0
         return r.width if r.kind == "rglru" else r.heads * r.vdim * (r.state if r.kind == "ssd" else r.dim)
+
+    def merged_output(self, il: int) -> bool:
+        """Whether the mixer's parts share one output projection ``mix.o`` over their concatenated columns."""
+        r = self.recurrent_spec(il)
+        return r is not None and r.kind == "hgrn2"
 
     # layer runs of a looped stack: caches and states belong to a run, weights to a layer
     def weight_layer(self, il: int) -> int:

@@ -18,8 +18,11 @@
 // a time. Every warpgroup of every split writes one partial (2 x splits per head); the splits of a (sequence,
 // kv head) group count themselves in when their partials are visible and the last one merges them into the
 // output, so there is no combine launch. Split count is a launch constant, lengths and tables are data.
+// A variant of its own (EXT) has sinks (joined in the merge), first tokens that stay visible behind a window (their tiles
+// come ahead of the window's), a sigmoid gate per head and an output scale and pitch.
 //
 // Counterpart in the reference: src/cuda/paged_attn/common.cuh (paged_decode, paged_combine).
+#include "attn_extra.h"
 #include "common.cuh"
 #include "kernels.h"
 #include "tmap.cuh"
@@ -56,7 +59,10 @@ struct DecodeTcArgs {
   __nv_bfloat16* out;   // [B, Hq, dv]
   int* group_ctr;  // [B * gridDim.x] arrival counters of the splits, zero on entry, left zero on exit
   int* status;
+  AttnExtra x;
 };
+
+enum : int { ATTN_PLAIN = 0, ATTN_CAP = 1, ATTN_EXT = 2 };
 
 template <int DK, int DV>
 struct DecodeTcCfg {
@@ -83,12 +89,13 @@ struct DecodeTcCfg {
 // TMEM round trip of the rescale leaves the per-tile critical path.
 static constexpr float DEC_RESCALE_LOG2 = 8.f;
 
-// CAP: the scores pass a soft cap on their way out of tensor memory
-template <int DK, int DV, bool CAP>
+// ATTN_CAP: the scores pass a soft cap on their way out of tensor memory; ATTN_EXT: AttnExtra
+template <int DK, int DV, int MODE>
 __global__ void __launch_bounds__(320, 1)
 paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const DecodeTcArgs a) {
   using Cfg = DecodeTcCfg<DK, DV>;
+  constexpr bool CAP = MODE == ATTN_CAP, EXT = MODE == ATTN_EXT;
   constexpr int NQ = Cfg::NQ, BKV = Cfg::BKV, HALVES = Cfg::HALVES, MT = Cfg::MT;
   constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ uint8_t smem_raw[];
@@ -127,11 +134,13 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int ctx = a.ctx_lens[b];
   const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
   const int blk_first = start / BKV;
-  const int n_units = (ctx + BKV - 1) / BKV - blk_first;
+  const int n_keep = EXT ? min((a.x.keep + BKV - 1) / BKV, blk_first) : 0;    // tiles of kept tokens in front of the window's
+  const int n_units = n_keep + (ctx + BKV - 1) / BKV - blk_first;
   const int units_per = (n_units + a.n_splits - 1) / a.n_splits;
-  const int blk_lo = blk_first + split * units_per;
+  const int blk_lo = blk_first - n_keep + split * units_per;                 // (counted as if the kept tiles led up to the window)
   const int blk_hi = min((ctx + BKV - 1) / BKV, blk_lo + units_per);
   const int n_blk = max(0, blk_hi - blk_lo);
+  auto blk_of = [&](int i) { return EXT && blk_lo + i < blk_first ? blk_lo + i - (blk_first - n_keep) : blk_lo + i; };
   const int head0 = kvh * G + g0;
 
   if (threadIdx.x == 0) *abort_flag = 0;
@@ -187,7 +196,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       for (int i = 0; ok && i < n_blk; ++i) {
         const int slot = i % tiles_per_fill;
         if (slot == 0) {
-          const int pidx = (blk_lo + i) * ppb + lane;
+          const int pidx = EXT ? blk_of(i + lane / ppb) * ppb + lane % ppb : (blk_lo + i) * ppb + lane;
           pg_reg = (long(pidx) * a.page < ctx) ? bt[pidx] : bt[0];
         }
         const int ks = i % KS, vs = i % VS;
@@ -307,8 +316,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           tmem_ld16(my_S, r);
           tmem_ld_wait();
         }
-        const int tok = (blk_lo + i) * BKV + tl;
-        const bool valid = tok >= start && tok < ctx;
+        const int tok = blk_of(i) * BKV + tl;
+        const bool valid = (tok >= start || (EXT && tok < a.x.keep)) && tok < ctx;
         // Only the gn real heads are processed (the MMA's N is padded to 16). The common case needs no column
         // maxima at all: as long as no score exceeds its column's reference maximum by more than the rescale
         // threshold, the probabilities are taken relative to the (stale) reference. The "any score over"
@@ -472,6 +481,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     for (int sidx = lane; sidx < ns; sidx += 32) mm = fmaxf(mm, s_w[q * ns + sidx]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+    if (EXT && a.x.sink) mm = fmaxf(mm, a.x.sink[head0 + q]);
     float ll = 0.f;
     for (int sidx = lane; sidx < ns; sidx += 32) {
       const float m = s_w[q * ns + sidx];
@@ -482,6 +492,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, o);
+    if (EXT && a.x.sink) ll += __expf(a.x.sink[head0 + q] - mm);
     if (lane == 0) s_l[q] = ll;
   }
   __syncthreads();
@@ -494,6 +505,13 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (wgt != 0.f) o += wgt * __ldcg(&a.o_part[(row0 + sidx) * D + d]);
     }
     const float ll = s_l[q];
+    if constexpr (EXT) {
+      float f = ll > 0.f ? a.x.out_scale / ll : 0.f;
+      if (a.x.gate)
+        f /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.x.gate)[b * a.x.ld_gate + head0 + q]));
+      a.out[b * a.x.ldo + (head0 + q) * D + d] = __float2bfloat16(o * f);
+      continue;
+    }
     a.out[(long(b) * a.Hq + head0 + q) * D + d] = __float2bfloat16(ll > 0.f ? o / ll : 0.f);
   }
 }
@@ -501,11 +519,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 namespace {
 thread_local char g_dec_err[256];
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, int MODE>
 int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const DecodeTcArgs& a,
                      dim3 grid, cudaStream_t s) {
   using Cfg = DecodeTcCfg<DK, DV>;
-  auto kfn = paged_decode_tc_kernel<DK, DV, CAP>;
+  auto kfn = paged_decode_tc_kernel<DK, DV, MODE>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -531,7 +549,7 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
                            long v_cell, const int* block_table, int table_width, int page, const int* ctx_lens,
                            float scale, float softcap, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits,
                            float* o_part, float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status,
-                           cudaStream_t s) {
+                           cudaStream_t s, const AttnExtra& x) {
   if (B <= 0) return 0;
   if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || k_cell % 8 || v_cell % 8 || page <= 0 ||
       128 % page != 0 || page % 8 != 0 || Hq % Hkv)
@@ -560,10 +578,17 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   }
   a.o_part = o_part; a.ml_part = ml_part; a.status = status; a.dv = dv;
   a.out = static_cast<__nv_bfloat16*>(out); a.group_ctr = group_ctr;
+  a.x = x;
+  if (x.on && (cap || x.keep < 0)) {
+    snprintf(g_dec_err, sizeof(g_dec_err), "decode attention: sinks, kept tokens and gates come without a soft cap");
+    return 1;
+  }
   dim3 grid(Hkv * gtiles, B, n_splits);
 #define LB_DIM(K_, V_)                                                                                    \
   if (DK == K_ && DV == V_)                                                                               \
-    return cap ? launch_decode_tc<K_, V_, true>(tq, tk, tv, a, grid, s) : launch_decode_tc<K_, V_, false>(tq, tk, tv, a, grid, s);
+    return x.on  ? launch_decode_tc<K_, V_, ATTN_EXT>(tq, tk, tv, a, grid, s)                             \
+           : cap ? launch_decode_tc<K_, V_, ATTN_CAP>(tq, tk, tv, a, grid, s)                             \
+                 : launch_decode_tc<K_, V_, ATTN_PLAIN>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64) LB_DIM(128, 128) LB_DIM(256, 256) LB_DIM(64, 128) LB_DIM(64, 256) LB_DIM(128, 64) LB_DIM(128, 256)
   LB_DIM(256, 64) LB_DIM(256, 128) LB_DIM(64, 192) LB_DIM(128, 192) LB_DIM(256, 192)
 #undef LB_DIM

@@ -2,6 +2,7 @@
 // units. The tcgen05 kernels (attn_prefill_sm100.cu, attn_decode_sm100.cu) take the bf16 shapes; this file serves fp32
 // models and head widths those do not cover.
 #include "act_type.cuh"
+#include "attn_extra.h"
 #include "common.cuh"
 #include "layers.h"
 
@@ -66,7 +67,7 @@ template <typename T, int NV>
 __global__ void __launch_bounds__(128) paged_attn_general_kernel(
     const T* __restrict__ q, long q_row, const T* __restrict__ k_cache, const T* __restrict__ v_cache, long k_cell, long v_cell,
     const int* __restrict__ cu_q, const int* __restrict__ ctx_lens, const int* __restrict__ block_table, int table_width,
-    int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, float cap, int window, T* __restrict__ out) {
+    int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, float cap, int window, T* __restrict__ out, const AttnExtra x) {
   extern __shared__ float q_sm[];
   griddep_wait();
   griddep_launch();
@@ -87,14 +88,20 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
   __syncwarp();
   const int* bt = block_table + long(seq) * table_width;
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int skip = lo - min(x.keep, lo);             // tokens between the kept first ones and the window
   float m = -INFINITY, l = 0.f, acc[NV];
+  if (x.sink) {                                      // as if a key with this score and no value had been seen
+    m = x.sink[h];
+    l = 1.f;
+  }
 #pragma unroll
   for (int j = 0; j < NV; ++j) acc[j] = 0.f;
-  for (int k0 = lo; k0 <= pos; k0 += 32) {
-    const int key = k0 + lane;
+  const int last = pos - skip;                       // places of the visible tokens: 0 .. last
+  for (int k0 = 0; k0 <= last; k0 += 32) {
+    const int place = k0 + lane, key = place < lo - skip ? place : place + skip;
     long cell = 0;
     float s = -INFINITY;
-    if (key <= pos) {
+    if (place <= last) {
       cell = long(bt[key / page]) * page + key % page;
       const T* kr = k_cache + cell * k_cell + long(kvh) * DK;
       float a0 = 0.f, a1 = 0.f;
@@ -111,13 +118,13 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     const float mn = fmaxf(m, mx);
-    const float p = key <= pos ? expf(s - mn) : 0.f;
+    const float p = place <= last ? expf(s - mn) : 0.f;
     const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
     m = mn;
     l = l * alpha + warp_sum_f(p);
 #pragma unroll
     for (int j = 0; j < NV; ++j) acc[j] *= alpha;
-    const int n = min(32, pos - k0 + 1);
+    const int n = min(32, last - k0 + 1);
     for (int i = 0; i < n; ++i) {
       const float pi = __shfl_sync(0xffffffffu, p, i);
       const long ci = __shfl_sync(0xffffffffu, cell, i);
@@ -129,18 +136,20 @@ __global__ void __launch_bounds__(128) paged_attn_general_kernel(
       }
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float f = l > 0.f ? x.out_scale / l : 0.f;
+  if (x.gate) f *= sigmoid_f(ld_f(static_cast<const T*>(x.gate) + t * x.ld_gate + h));
+  T* orow = x.on ? out + t * x.ldo + long(h) * DV : out + (long(t) * Hq + h) * DV;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int d = lane + 32 * j;
-    if (d < DV) st_f(out + (long(t) * Hq + h) * DV + d, acc[j] * inv);
+    if (d < DV) st_f(orow + d, acc[j] * f);
   }
 }
 
 template <typename T>
 int attn_t(const void* q, long q_row, const void* k, const void* v, long k_cell, long v_cell, const int* cu_q, const int* ctx_lens,
            const int* bt, int tw, int page, int n_seqs, int nT, int Hq, int Hkv, int DK, int DV, float scale, float cap,
-           int window, void* out, cudaStream_t s) {
+           int window, void* out, const AttnExtra& x, cudaStream_t s) {
   const long warps = long(nT) * Hq;
   const dim3 grid(unsigned((warps + 3) / 4));
   const size_t smem = size_t(4) * DK * 4;
@@ -149,7 +158,7 @@ int attn_t(const void* q, long q_row, const void* k, const void* v, long k_cell,
   if (DV <= 32 * N)                                                                                                    \
     return launch_pdl(paged_attn_general_kernel<T, N>, grid, dim3(128), smem, s, static_cast<const T*>(q), q_row,      \
                       static_cast<const T*>(k), static_cast<const T*>(v), k_cell, v_cell, cu_q, ctx_lens, bt, tw,      \
-                      page, n_seqs, nT, Hq, Hkv, DK, DV, scale, cap, window, static_cast<T*>(out)) != cudaSuccess;
+                      page, n_seqs, nT, Hq, Hkv, DK, DV, scale, cap, window, static_cast<T*>(out), x) != cudaSuccess;
   LB_NV(2) LB_NV(4) LB_NV(8) LB_NV(16) LB_NV(32)
 #undef LB_NV
   return 1;
@@ -175,13 +184,13 @@ int qkv_norm_append_launch(const void* q, const void* k, const void* v, long ld,
 int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
                               int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, float softcap, int window,
-                              void* out, bool f32, cudaStream_t s) {
+                              void* out, bool f32, cudaStream_t s, const AttnExtra& x) {
   if (T <= 0 || n_seqs <= 0) return 0;
-  if (page <= 0 || Hkv <= 0 || Hq % Hkv) return 1;
+  if (page <= 0 || Hkv <= 0 || Hq % Hkv || x.keep < 0) return 1;
   return f32 ? attn_t<float>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page, n_seqs,
-                             T, Hq, Hkv, DK, DV, scale, softcap, window, out, s)
+                             T, Hq, Hkv, DK, DV, scale, softcap, window, out, x, s)
              : attn_t<__nv_bfloat16>(q, q_row, k_cache, v_cache, k_cell, v_cell, cu_q, ctx_lens, block_table, table_width, page,
-                                     n_seqs, T, Hq, Hkv, DK, DV, scale, softcap, window, out, s);
+                                     n_seqs, T, Hq, Hkv, DK, DV, scale, softcap, window, out, x, s);
 }
 
 }  // namespace lb

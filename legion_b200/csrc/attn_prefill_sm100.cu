@@ -16,9 +16,12 @@
 // comparisons on blocks that are entirely visible, and rescales O only when the row maximum grew by more than
 // 2^8 (probabilities are then relative to a slightly stale maximum).
 // Sequence lengths, query offsets and block tables are data; the grid is (q tiles, heads, seqs).
+// A variant of its own (EXT) has sinks, first tokens that stay visible behind a window (their blocks come ahead of the
+// window's), a sigmoid gate per head and an output scale and pitch; a sink is the running softmax's initial state.
 //
 // Counterparts in the reference: src/cuda/sm80/paged_attn.cuh (paged_prefill_mma, split verify),
 // src/cuda/sm90/paged_attn_wgmma.cu.
+#include "attn_extra.h"
 #include "common.cuh"
 #include "kernels.h"
 #include "tmap.cuh"
@@ -96,7 +99,10 @@ struct PrefillArgs {
   __nv_bfloat16* out;      // [T, Hq, dv]
   int dk, dv;              // head sizes: at most the template's; the tensor maps end there and TMA fills zeros
   int* status;
+  AttnExtra x;
 };
+
+enum : int { ATTN_PLAIN = 0, ATTN_CAP = 1, ATTN_EXT = 2 };
 
 template <int N>
 struct IntC { static constexpr int value = N; };
@@ -119,12 +125,13 @@ struct PrefillCfg {
   static constexpr int TMEM_COLS = TMEM_RAW <= 128 ? 128 : (TMEM_RAW <= 256 ? 256 : 512);
 };
 
-// CAP: the scores pass a soft cap on their way out of tensor memory
-template <int DK, int DV, int BKV, bool CAP>
+// ATTN_CAP: the scores pass a soft cap on their way out of tensor memory; ATTN_EXT: AttnExtra
+template <int DK, int DV, int BKV, int MODE>
 __global__ void __launch_bounds__(160, (DK <= 128 && DV <= 128 && BKV == 64) ? 2 : 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const PrefillArgs a) {
   using Cfg = PrefillCfg<DK, DV, BKV>;
+  constexpr bool CAP = MODE == ATTN_CAP, EXT = MODE == ATTN_EXT;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw;
   if (smem_u32(smem_raw) & 1023u) {       // swizzled tiles need 1024-byte alignment; uniform per CTA, before any barrier
@@ -194,7 +201,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (a.window > 0) kv_lo = max(0, pos0 - a.window + 1);
   const int blk_lo = kv_lo / BKV;
   const int blk_hi = (kv_hi + BKV - 1) / BKV;                     // exclusive
-  const int n_blk = blk_hi - blk_lo;
+  // blocks of kept first tokens that lie in front of the window's
+  const int n_keep = EXT ? min((a.x.keep + BKV - 1) / BKV, blk_lo) : 0;
+  const int n_blk = n_keep + blk_hi - blk_lo;
+  auto blk_of = [&](int i) { return EXT && i < n_keep ? i : blk_lo - n_keep + i; };
   const int* bt = a.block_table + long(seq) * a.table_width;
   const int pages_per_blk = BKV / a.page;
 
@@ -224,10 +234,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
       for (int h = 0; h < Cfg::HALVES; ++h)
         tma_load_3d(q_s + h * (128 * 128), &tmQ, q_full, h * 64, head, q0 + tile_row0);
-      load_k(blk_lo, 0);
-      if (n_blk > 1) load_k(blk_lo + 1, 1);
-      load_v(blk_lo, 0);
-      if (n_blk > 1) load_v(blk_lo + 1, 1);
+      load_k(blk_of(0), 0);
+      if (n_blk > 1) load_k(blk_of(1), 1);
+      load_v(blk_of(0), 0);
+      if (n_blk > 1) load_v(blk_of(1), 1);
       constexpr uint32_t idesc_s = umma_idesc(128, BKV, 1, 1, 0, 0);
       constexpr uint32_t idesc_o = umma_idesc(128, DV, 1, 1, 0, 1);  // B (= V) is MN-major
       bool ok = mbar_wait(q_full, 0, abort_flag);
@@ -258,7 +268,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (ok && n_blk > 0) ok = issue_s(0);
       for (int i = 0; ok && i < n_blk; ++i) {
         // K stage (i + 2) % 3 held block i - 1, whose scores the softmax has consumed (p_ready(i - 1) was seen)
-        if (i + 2 < n_blk) load_k(blk_lo + i + 2, (i + 2) % 3);
+        if (i + 2 < n_blk) load_k(blk_of(i + 2), (i + 2) % 3);
         // the next block's scores, one block ahead of the softmax: buffer (i + 1) & 1 held S(i - 1), read and done
         if (i + 1 < n_blk && !issue_s(i + 1)) break;
         if (i >= 1 && i + 1 < n_blk) {
@@ -266,7 +276,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           if (!mbar_wait(&o_done[(i - 1) & 1], uint32_t((i - 1) >> 1) & 1u, abort_flag)) {
             *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_EMPTY | SITE_PREFILL_ATTN); break;
           }
-          load_v(blk_lo + i + 1, (i + 1) & 1);
+          load_v(blk_of(i + 1), (i + 1) & 1);
         }
         if (!mbar_wait(&p_ready[i & 1], uint32_t(i >> 1) & 1u, abort_flag)) {
           *abort_flag = 1; atomicCAS(a.status, 0, ST_TIMEOUT_FLAG | SITE_PREFILL_ATTN); break;
@@ -293,6 +303,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const bool row_ok = row < rows_here;
     const uint32_t lane_off = uint32_t(warp * 32) << 16;
     float m = -INFINITY, l = 0.f;
+    if (EXT && a.x.sink) {                 // as if a key with this score and no value had been seen
+      m = a.x.sink[head] * 1.4426950408889634f;
+      l = 1.f;
+    }
     bool ok = true;
     for (int i = 0; i < n_blk; ++i) {
       if (!__all_sync(0xffffffffu, mbar_wait(&s_full[i & 1], uint32_t(i >> 1) & 1u, abort_flag))) {
@@ -300,13 +314,15 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       tc_fence_after();
       const uint32_t tmem_Si = tmem_S + uint32_t(i & 1) * BKV;
-      const int key0 = (blk_lo + i) * BKV;
+      const int key0 = blk_of(i) * BKV;
       int hi = a.causal ? min(ctx, qpos + 1) : ctx;   // exclusive key bound for this row
       int lo = (a.window > 0) ? max(0, qpos - a.window + 1) : 0;
       if (!row_ok) { hi = 0; lo = 0; }
       // blocks entirely inside every row's visible range need no per-element mask (all interior blocks of a
       // causal prompt): uniform over the CTA
-      const bool full_blk = a.window == 0 && rows_here == 128 && key0 + BKV <= (a.causal ? min(ctx, pos0 + 1) : ctx);
+      const bool full_blk = (a.window == 0 || (EXT && (key0 > last_pos - a.window || key0 + BKV <= a.x.keep))) &&
+                            rows_here == 128 && key0 + BKV <= (a.causal ? min(ctx, pos0 + 1) : ctx);
+      auto seen = [&](int key) { return (key >= lo || (EXT && key < a.x.keep)) && key < hi; };
       float alpha = 1.f;
       float sum = 0.f;
       if (BKV <= 64) {
@@ -336,7 +352,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
           for (int j = 0; j < BKV; ++j) {
             const int key = key0 + j;
-            if (key >= lo && key < hi) mx = fmaxf(mx, __uint_as_float(r[j]));
+            if (seen(key)) mx = fmaxf(mx, __uint_as_float(r[j]));
           }
         }
         const float m_blk = mx * a.scale_log2;
@@ -372,8 +388,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             float p0 = exp2f(fmaf(__uint_as_float(r[j]), a.scale_log2, neg_m));
             float p1 = exp2f(fmaf(__uint_as_float(r[j + 1]), a.scale_log2, neg_m));
             const int key = key0 + j;
-            if (!(key >= lo && key < hi)) p0 = 0.f;
-            if (!(key + 1 >= lo && key + 1 < hi)) p1 = 0.f;
+            if (!seen(key)) p0 = 0.f;
+            if (!seen(key + 1)) p1 = 0.f;
             // sum what the tensor core will see (bf16-rounded) to keep numerator and denominator consistent
             const __nv_bfloat162 bb = __floats2bfloat162_rn(p0, p1);
             const float2 f = __bfloat1622float2(bb);
@@ -395,7 +411,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int key = key0 + c + j;
-            if (full_blk || (key >= lo && key < hi)) mx = fmaxf(mx, __uint_as_float(r[j]));
+            if (full_blk || seen(key)) mx = fmaxf(mx, __uint_as_float(r[j]));
           }
         }
         const float m_blk = mx * a.scale_log2;
@@ -415,8 +431,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             float p0 = exp2f(fmaf(__uint_as_float(r[j]), a.scale_log2, neg_m));
             float p1 = exp2f(fmaf(__uint_as_float(r[j + 1]), a.scale_log2, neg_m));
             const int key = key0 + c + j;
-            if (!full_blk && !(key >= lo && key < hi)) p0 = 0.f;
-            if (!full_blk && !(key + 1 >= lo && key + 1 < hi)) p1 = 0.f;
+            if (!full_blk && !seen(key)) p0 = 0.f;
+            if (!full_blk && !seen(key + 1)) p1 = 0.f;
             const __nv_bfloat162 bb = __floats2bfloat162_rn(p0, p1);
             const float2 f = __bfloat1622float2(bb);
             sum += f.x + f.y;
@@ -463,8 +479,15 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     if (ok) {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* orow = a.out + (long(q0 + tile_row0 + row) * a.Hq + head) * a.dv;
+      if constexpr (EXT) {
+        const long t = q0 + tile_row0 + row;
+        orow = a.out + t * a.x.ldo + head * a.dv;
+        inv *= a.x.out_scale;
+        if (a.x.gate && row_ok)
+          inv /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.x.gate)[t * a.x.ld_gate + head]));
+      }
 #pragma unroll 1
       for (int c = 0; c < DV; c += 32) {
         uint32_t r[32];
@@ -501,12 +524,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 namespace {
 thread_local char g_attn_err[256];
 
-template <int DK, int DV, int BKV, bool CAP = false>
+template <int DK, int DV, int BKV, int MODE = ATTN_PLAIN>
 int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const PrefillArgs& a,
                    dim3 grid, cudaStream_t s) {
   using Cfg = PrefillCfg<DK, DV, BKV>;
-  static_assert(!CAP || BKV <= 64, "the soft cap is applied to a row of scores in registers");
-  auto kfn = prefill_attn_kernel<DK, DV, BKV, CAP>;
+  static_assert(MODE != ATTN_CAP || BKV <= 64, "the soft cap is applied to a row of scores in registers");
+  auto kfn = prefill_attn_kernel<DK, DV, BKV, MODE>;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(kfn, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess) {
@@ -530,11 +553,11 @@ const char* prefill_attn_last_error() { return g_attn_err; }
 int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                         long v_cell, const int* cu_q, const int* ctx_lens, const int* block_table, int table_width,
                         int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, float softcap,
-                        int window, int causal, void* out, int* status, cudaStream_t s) {
+                        int window, int causal, void* out, int* status, cudaStream_t s, const AttnExtra& x) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
   const int DK = dk <= 64 ? 64 : (dk <= 128 ? 128 : 256), DV = dv <= 64 ? 64 : (dv <= 128 ? 128 : (dv <= 192 ? 192 : 256));
   const bool cap = softcap > 0.f;
-  const int BKV = (DK >= 128 || DV >= 128 || cap) ? 64 : 128;
+  const int BKV = (DK >= 128 || DV >= 128 || cap || x.on) ? 64 : 128;
   if (page <= 0 || BKV % page != 0 || page % 8 != 0) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: page size %d must be a multiple of 8 dividing %d",
              page, BKV);
@@ -546,6 +569,10 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
   }
   // q viewed as [T, Hq, dk]; caches as [cells, Hkv, dk | dv] with cell pitches in elements. A box that reaches past the
   // head size reads zeros there, so head sizes between the template sizes need no padding in memory.
+  if (x.on && (cap || x.keep < 0 || x.ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15))) {
+    snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention: sinks and gates come without a soft cap, 16-byte aligned output rows");
+    return 1;
+  }
   const CUtensorMap* tq = tmap_3d(q, uint64_t(dk), uint64_t(Hq), uint64_t(T), uint64_t(dk) * 2,
                                   uint64_t(Hq) * dk * 2, 64, 1, 128, TM_BF16, true);
   const CUtensorMap* tk = tmap_3d(k_cache, uint64_t(dk), uint64_t(Hkv), uint64_t(n_cells), uint64_t(dk) * 2,
@@ -564,10 +591,13 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
     a.scale_log2 = 2.f * 1.4426950408889634f * softcap;
   }
   a.out = static_cast<__nv_bfloat16*>(out); a.dk = dk; a.dv = dv; a.status = status;
+  a.x = x;
   dim3 grid((max_q_len + 127) / 128, Hq, n_seqs);
 #define LB_DIM(K_, V_, B_)                                                                   \
   if (DK == K_ && DV == V_)                                                                  \
-    return cap ? launch_prefill<K_, V_, 64, true>(tq, tk, tv, a, grid, s) : launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
+    return x.on  ? launch_prefill<K_, V_, 64, ATTN_EXT>(tq, tk, tv, a, grid, s)               \
+           : cap ? launch_prefill<K_, V_, 64, ATTN_CAP>(tq, tk, tv, a, grid, s)               \
+                 : launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
   LB_DIM(64, 64, 128) LB_DIM(128, 128, 64) LB_DIM(256, 256, 64)
   LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64)
   LB_DIM(64, 192, 64) LB_DIM(128, 192, 64) LB_DIM(256, 192, 64) LB_DIM(256, 128, 64)

@@ -43,7 +43,7 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
            const OptT& ws, const OptT& counters, Tensor& status, const OptT& tile_group, const OptT& tile_tok0,
            const OptT& tile_ntok, const OptT& meta, int64_t max_tiles, int64_t rows_per_group, int64_t n_tok,
            std::vector<int64_t> out_peer, const OptT& tile_out0, const OptT& w_scales, const OptT& w_gscale,
-           int64_t x_group_col, int64_t k_override, int64_t act, const OptT& xielu, bool relu2) {
+           int64_t x_group_col, int64_t k_override, int64_t act, const OptT& xielu, bool relu2, const OptT& bias) {
   const bool fp4 = w_scales.has_value();     // w = NVFP4 codes [rows, K/2] uint8, w_scales = e4m3 bytes [rows, K/16]
   if (fp4) {
     TORCH_CHECK(w.scalar_type() == at::kByte && w_scales->is_contiguous() && w_scales->element_size() == 1 &&
@@ -85,6 +85,11 @@ void wgemm(const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, 
     h.xielu = xielu->data_ptr<float>();
   }
   h.relu2 = relu2;
+  if (bias.has_value()) {
+    TORCH_CHECK(dual && bias->scalar_type() == at::kFloat && bias->is_cuda() && bias->is_contiguous() && bias->numel() == 2 * n_feat,
+                "wgemm: float32 biases of gate and up");
+    h.bias = bias->data_ptr<float>();
+  }
   h.tile_group = optp<int>(tile_group); h.tile_tok0 = optp<int>(tile_tok0); h.tile_ntok = optp<int>(tile_ntok);
   h.n_tiles_dev = optp<int>(meta);
   h.tile_out0 = optp<int>(tile_out0);
@@ -365,6 +370,70 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(rc == 0, "paged_decode: unsupported shape or launch failure (", rc, ")");
 }
 
+// Sinks, kept first tokens, output gate, scale and pitch: out is [T, >= Hq * DV], rows may lie apart
+lb::AttnExtra attn_extra(const OptT& sink, int64_t keep, const OptT& gate, double out_scale, const Tensor& out, int64_t T,
+                         int64_t Hq, int64_t DV) {
+  lb::AttnExtra x;
+  x.on = 1;
+  check_bf16(out, "out");
+  TORCH_CHECK(out.dim() == 2 && out.size(0) == T && out.size(1) == Hq * DV, "attention: out [T, heads * value head size]");
+  if (sink.has_value()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->is_contiguous() && sink->numel() == Hq,
+                "attention: sinks are float32 [heads]");
+    x.sink = sink->data_ptr<float>();
+  }
+  if (gate.has_value()) {
+    check_bf16(*gate, "gate");
+    TORCH_CHECK(gate->dim() == 2 && gate->size(0) == T && gate->size(1) == Hq, "attention: gate [T, heads]");
+    x.gate = gate->data_ptr();
+    x.ld_gate = gate->stride(0);
+  }
+  TORCH_CHECK(keep >= 0, "attention: kept tokens");
+  x.keep = int(keep); x.out_scale = float(out_scale); x.ldo = out.stride(0);
+  return x;
+}
+
+void paged_decode_ext(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_table,
+                      const Tensor& ctx_lens, double scale, int64_t window, int64_t n_splits, Tensor& o_part, Tensor& ml_part,
+                      Tensor& out, Tensor& status, Tensor& counters, int64_t keep, const OptT& sink, const OptT& gate,
+                      double out_scale) {
+  check_bf16(q, "q");
+  c10::cuda::CUDAGuard guard(q.device());
+  const int B = int(q.size(0)), Hq = int(q.size(1)), D = int(q.size(2)), DV = int(v_cache.size(-1));
+  const int page = int(k_cache.size(-3)), Hkv = int(k_cache.size(-2));
+  TORCH_CHECK(k_cache.size(-1) == D && v_cache.size(-2) == Hkv && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                  q.is_contiguous() && ctx_lens.numel() == B, "paged_decode_ext: shapes");
+  TORCH_CHECK(o_part.numel() >= int64_t(B) * Hq * n_splits * 2 * DV && ml_part.numel() >= int64_t(B) * Hq * n_splits * 4,
+              "paged_decode_ext: partial buffers too small");
+  const auto x = attn_extra(sink, keep, gate, out_scale, out, B, Hq, DV);
+  const int rc = lb::paged_decode_tc_launch(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), k_cache.numel() / (long(Hkv) * D),
+                                            long(Hkv) * D, long(Hkv) * DV, block_table.data_ptr<int>(),
+                                            int(block_table.size(1)), page, ctx_lens.data_ptr<int>(), float(scale), 0.f,
+                                            int(window), B, Hq, Hkv, D, DV, int(n_splits), o_part.data_ptr<float>(),
+                                            ml_part.data_ptr<float>(), out.data_ptr(), counters.data_ptr<int>(),
+                                            int(counters.numel()), reinterpret_cast<int*>(status.data_ptr()), cur_stream(), x);
+  TORCH_CHECK(rc == 0, rc < 0 ? "paged_decode_ext: shape outside the tensor-core kernel" : lb::paged_decode_tc_last_error());
+}
+
+void prefill_attn_ext(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q, const Tensor& ctx_lens,
+                      const Tensor& block_table, int64_t max_q_len, double scale, int64_t window, Tensor& out, Tensor& status,
+                      int64_t keep, const OptT& sink, const OptT& gate, double out_scale) {
+  check_bf16(q, "q");
+  c10::cuda::CUDAGuard guard(q.device());
+  const long T = q.size(0);
+  const int Hq = int(q.size(1)), D = int(q.size(2)), DV = int(v_cache.size(-1));
+  const int page = int(k_cache.size(-3)), Hkv = int(k_cache.size(-2));
+  TORCH_CHECK(k_cache.size(-1) == D && v_cache.size(-2) == Hkv && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                  q.is_contiguous() && cu_q.numel() == ctx_lens.numel() + 1, "prefill_attn_ext: shapes");
+  const auto x = attn_extra(sink, keep, gate, out_scale, out, T, Hq, DV);
+  const int rc = lb::prefill_attn_launch(q.data_ptr(), T, k_cache.data_ptr(), v_cache.data_ptr(), k_cache.numel() / (long(Hkv) * D),
+                                         long(Hkv) * D, long(Hkv) * DV, cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(),
+                                         block_table.data_ptr<int>(), int(block_table.size(1)), page, int(ctx_lens.numel()),
+                                         int(max_q_len), Hq, Hkv, D, DV, float(scale), 0.f, int(window), 1, out.data_ptr(),
+                                         reinterpret_cast<int*>(status.data_ptr()), cur_stream(), x);
+  TORCH_CHECK(rc == 0, lb::prefill_attn_last_error());
+}
+
 void prefill_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
                   const Tensor& ctx_lens, const Tensor& block_table, int64_t max_q_len, double scale, int64_t window,
                   bool causal, Tensor& out, Tensor& status, double softcap) {
@@ -612,7 +681,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         pybind11::arg("n_tok"), pybind11::arg("out_peer"), pybind11::arg("tile_out0") = pybind11::none(),
         pybind11::arg("w_scales") = pybind11::none(), pybind11::arg("w_gscale") = pybind11::none(),
         pybind11::arg("x_group_col") = 0, pybind11::arg("k_override") = 0, pybind11::arg("act") = 0,
-        pybind11::arg("xielu") = pybind11::none(), pybind11::arg("relu2") = false);
+        pybind11::arg("xielu") = pybind11::none(), pybind11::arg("relu2") = false, pybind11::arg("bias") = pybind11::none());
   m.def("wgemm_fp8", &wgemm_fp8);
   m.def("wgemm_fp8_q", &wgemm_fp8_q);
   m.def("wgemm_allreduce", &wgemm_allreduce);
@@ -624,6 +693,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("embed", &embed);
   m.def("paged_decode", &paged_decode);      // softcap > 0: scores become softcap * tanh(score / softcap)
   m.def("prefill_attn", &prefill_attn);
+  m.def("paged_decode_ext", &paged_decode_ext);
+  m.def("prefill_attn_ext", &prefill_attn_ext);
   m.def("mla_attn", &mla_attn);
   m.def("mla_prep", &mla_prep);
   m.def("router_topk", &router_topk, pybind11::arg("logits"), pybind11::arg("bias"), pybind11::arg("k"),

@@ -251,6 +251,115 @@ void bind_layers(pybind11::module_& m) {
     c10::cuda::CUDAGuard guard(x_out.device());
     TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "prenorm_step: rows of at most 51200 columns", cuda_error());
   });
+  m.def("depth_step", [](const Tensor& x, Tensor& x_out, const OptT& hist, int64_t layer, bool keep, const Tensor& y1,
+                         const OptT& g1, const OptT& b1, const OptT& y2, int64_t y2_rows, const OptT& g2, const OptT& b2,
+                         const OptT& y2_b, const OptT& coef, const Tensor& norm_w, double eps, double w_offset, Tensor& h,
+                         const OptT& rows) {
+    const bool f32 = is_f32(h, "h");
+    same(y1, f32, "y1");
+    const int64_t T = x.size(0), H = x.size(1), R = h.size(0);
+    TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && x.scalar_type() == at::kFloat && x_out.is_contiguous() && x_out.dim() == 2 &&
+                    x_out.scalar_type() == at::kFloat && x_out.size(0) == R && x_out.size(1) == H && h.size(1) == H &&
+                    y1.dim() == 2 && y1.size(0) == T && y1.size(1) == H, "depth_step: x, y1 [rows, width], x_out and h alike");
+    lb::DepthStepArgs a{};
+    a.x = x.data_ptr<float>(); a.x_out = x_out.data_ptr<float>();
+    a.y1 = y1.data_ptr(); a.ldy1 = y1.stride(0); a.y2_rows = 1;
+    if (hist.has_value()) {
+      TORCH_CHECK(hist->is_contiguous() && hist->scalar_type() == at::kFloat && hist->dim() == 3 && hist->size(0) > layer + 1 &&
+                      hist->size(1) == T && hist->size(2) == H && layer >= 0 && coef.has_value(), "depth_step: hist [layers + 1, rows, width]");
+      f32c(*coef, layer + 2, "depth average");
+      a.hist = hist->data_ptr<float>(); a.hist_stride = T * H; a.n_hist = int(layer + 1);
+      a.coef = coef->data_ptr<float>();
+      if (keep) a.hist_out = hist->data_ptr<float>() + (layer + 1) * T * H;
+    }
+    if (y2.has_value()) {
+      same(*y2, f32, "y2");
+      TORCH_CHECK(y2->dim() == 2 && y2->size(1) == H && y2_rows >= 1 && y2->size(0) >= T * y2_rows, "depth_step: y2 [rows * y2_rows, width]");
+      a.y2 = y2->data_ptr(); a.ldy2 = y2->stride(0); a.y2_rows = int(y2_rows);
+      if (y2_b.has_value()) {
+        f32c(*y2_b, H, "feed-forward bias");
+        a.y2_b = y2_b->data_ptr<float>();
+      }
+    }
+    auto gate = [&](const OptT& g, const OptT& b, const void*& gp, const float*& bp) {
+      if (!g.has_value()) return;
+      same(*g, f32, "gate");
+      TORCH_CHECK(b.has_value() && g->dim() == 2 && g->size(0) == T && g->size(1) == H && (!a.ldg || a.ldg == g->stride(0)),
+                  "depth_step: gates [rows, width] of one projection, with bias");
+      f32c(*b, H, "gate bias");
+      gp = g->data_ptr(); bp = b->data_ptr<float>(); a.ldg = g->stride(0);
+    };
+    gate(g1, b1, a.g1, a.b1);
+    if (y2.has_value()) gate(g2, b2, a.g2, a.b2);
+    if (rows.has_value()) {
+      TORCH_CHECK(rows->scalar_type() == at::kLong && rows->is_contiguous() && rows->numel() == R && x_out.data_ptr() != x.data_ptr(),
+                  "depth_step: int64 rows, an output of their own");
+      a.rows = reinterpret_cast<const long*>(rows->data_ptr());
+    } else {
+      TORCH_CHECK(R == T, "depth_step: a row per token");
+    }
+    f32c(norm_w, H, "norm_w");
+    a.norm_w = norm_w.data_ptr<float>(); a.eps = float(eps); a.w_offset = float(w_offset);
+    a.h = h.data_ptr(); a.ldh = h.stride(0); a.n_rows = int(R); a.H = int(H);
+    c10::cuda::CUDAGuard guard(x.device());
+    TORCH_CHECK(lb::depth_step_launch(a, f32, cur_stream()) == 0, "depth_step: rows of at most 25600 columns", cuda_error());
+  });
+  auto forget_args = [](const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_b, const Tensor& lower, Tensor& state,
+                        const Tensor& cu, const Tensor& slots, int64_t H, int64_t N, int64_t P, const Tensor& norm_w, double eps,
+                        double scale, Tensor& out, bool write_state) {
+    const bool f32 = is_f32(q, "q");
+    same(f, f32, "f");
+    same(v, f32, "v");
+    same(out, f32, "out");
+    const int64_t T = q.size(0);
+    TORCH_CHECK(q.dim() == 2 && f.dim() == 2 && v.dim() == 2 && out.dim() == 2 && q.size(1) == H * N && f.size(1) == H * N &&
+                    v.size(1) == H * P && out.size(1) == H * P && f.size(0) == T && v.size(0) == T && out.size(0) == T,
+                "forget scan: q, f [T, H * N], v and out [T, H * P]");
+    f32c(f_b, H * N, "forget bias");
+    f32c(lower, H * N, "lower bounds");
+    f32c(norm_w, P, "norm weight");
+    TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == H &&
+                    state.size(2) == P && state.size(3) == N, "forget scan: state [slots, H, P, N] float32");
+    TORCH_CHECK(cu.scalar_type() == at::kInt && slots.scalar_type() == at::kInt && cu.numel() == slots.numel() + 1,
+                "forget scan: int32 sequence bounds and slots");
+    lb::ForgetScanArgs a{};
+    a.q = q.data_ptr(); a.ldq = q.stride(0); a.f = f.data_ptr(); a.ldf = f.stride(0); a.v = v.data_ptr(); a.ldv = v.stride(0);
+    a.f_b = f_b.data_ptr<float>(); a.lower = lower.data_ptr<float>(); a.state = state.data_ptr<float>();
+    a.cu = cu.data_ptr<int>(); a.slots = slots.data_ptr<int>();
+    a.n_seqs = int(slots.numel()); a.T = int(T); a.H = int(H); a.N = int(N); a.P = int(P);
+    a.norm_w = norm_w.data_ptr<float>(); a.eps = float(eps); a.scale = float(scale);
+    a.out = out.data_ptr(); a.ldo = out.stride(0); a.write_state = write_state;
+    return a;
+  };
+  m.def("forget_scan", [forget_args](const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_b, const Tensor& lower,
+                                     Tensor& state, const Tensor& cu, const Tensor& slots, int64_t H, int64_t N, int64_t P,
+                                     const Tensor& norm_w, double eps, double scale, Tensor& out, bool write_state,
+                                     int64_t max_tokens) {
+    auto a = forget_args(q, f, v, f_b, lower, state, cu, slots, H, N, P, norm_w, eps, scale, out, write_state);
+    a.max_tokens = int(max_tokens);
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::forget_scan_launch(a, q.scalar_type() == at::kFloat, cur_stream()) == 0,
+                "forget scan: key heads of at most 512 columns, value heads of at most 4096", cuda_error());
+  });
+  m.def("forget_chunk_ok", [](int64_t N, int64_t P) { return lb::forget_chunk_ok(int(N), int(P)); });
+  m.def("forget_chunk_scratch_bytes", [](int64_t n_chunks, int64_t H, int64_t N, int64_t P) {
+    return int64_t(lb::forget_chunk_scratch_bytes(int(n_chunks), int(H), int(N), int(P)));
+  });
+  m.def("forget_chunk", [forget_args](const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_b, const Tensor& lower,
+                                      Tensor& state, const Tensor& cu, const Tensor& slots, int64_t H, int64_t N, int64_t P,
+                                      const Tensor& norm_w, double eps, double scale, Tensor& out, bool write_state,
+                                      const Tensor& tab, int64_t n_chunks, Tensor& scratch, Tensor& status) {
+    auto a = forget_args(q, f, v, f_b, lower, state, cu, slots, H, N, P, norm_w, eps, scale, out, write_state);
+    TORCH_CHECK(q.scalar_type() == at::kBFloat16, "forget_chunk: bf16 activations");
+    TORCH_CHECK(tab.scalar_type() == at::kInt && tab.is_contiguous() && tab.numel() >= 3 * n_chunks + 2 * a.n_seqs, "forget_chunk: chunk tables");
+    TORCH_CHECK(scratch.is_contiguous() && size_t(scratch.numel() * scratch.element_size()) >=
+                    lb::forget_chunk_scratch_bytes(int(n_chunks), int(H), int(N), int(P)), "forget_chunk: scratch");
+    const int* t = tab.data_ptr<int>();
+    c10::cuda::CUDAGuard guard(q.device());
+    TORCH_CHECK(lb::forget_chunk_launch(a, t, t + n_chunks, int(n_chunks), t + 3 * n_chunks, t + 3 * n_chunks + a.n_seqs,
+                                        scratch.data_ptr(), reinterpret_cast<int*>(status.data_ptr()), cur_stream()) == 0,
+                "forget_chunk: heads of at most 128 columns", cuda_error());
+  });
   m.def("qkv_conv_append", [](const Tensor& x, const OptT& in_b, const OptT& conv_w, const OptT& conv_state, const Tensor& cu,
                               const Tensor& state_slots, const OptT& qw, const OptT& kw, bool norm_all, double eps,
                               const OptT& cos_sin, bool rot_half, const Tensor& positions, const Tensor& slots, Tensor& q_out,
@@ -356,7 +465,7 @@ void bind_layers(pybind11::module_& m) {
   m.def("sgemm", [](const Tensor& w, const Tensor& x, Tensor& out, const OptT& residual, const OptT& tok_scale,
                     const OptT& out_rows, int64_t n_feat, bool dual, int64_t dual_offset, int64_t act,
                     const OptT& tile_group, const OptT& tile_tok0, const OptT& tile_ntok, const OptT& meta,
-                    int64_t max_tiles, int64_t rows_per_group, int64_t n_tok, const OptT& act_ab) {
+                    int64_t max_tiles, int64_t rows_per_group, int64_t n_tok, const OptT& act_ab, const OptT& bias) {
     const bool f32 = is_f32(x, "x");
     same(w, f32, "w");
     TORCH_CHECK(w.dim() == 2 && x.dim() == 2 && out.dim() == 2 && w.size(1) == x.size(1), "sgemm: K mismatch");
@@ -374,13 +483,22 @@ void bind_layers(pybind11::module_& m) {
     a.tok_scale = optp<float>(tok_scale); a.out_rows = optp<int>(out_rows);
     a.T = int(n_tok); a.K = int(x.size(1)); a.N = int(n_feat);
     a.dual = dual; a.dual_offset = dual_offset; a.act = int(act); a.act_ab = optp<float>(act_ab);
+    if (bias.has_value()) {
+      TORCH_CHECK(dual && !tile_group.has_value(), "sgemm: biases of an ungrouped gate/up product");
+      f32c(*bias, 2 * n_feat, "bias");
+      a.bias = bias->data_ptr<float>();
+    }
     a.tile_group = optp<int>(tile_group); a.tile_tok0 = optp<int>(tile_tok0); a.tile_ntok = optp<int>(tile_ntok);
     a.n_tiles = optp<int>(meta); a.max_tiles = int(max_tiles); a.rows_per_group = rows_per_group;
     TORCH_CHECK(!a.tile_group || (a.tile_tok0 && a.tile_ntok && a.n_tiles), "sgemm: incomplete tile tables");
     TORCH_CHECK(a.tile_group || x.size(0) >= n_tok, "sgemm: too few rows");
     c10::cuda::CUDAGuard guard(x.device());
     TORCH_CHECK(lb::sgemm_launch(a, f32, cur_stream()) == 0, "sgemm failed", cuda_error());
-  });
+  }, pybind11::arg("w"), pybind11::arg("x"), pybind11::arg("out"), pybind11::arg("residual"), pybind11::arg("tok_scale"),
+     pybind11::arg("out_rows"), pybind11::arg("n_feat"), pybind11::arg("dual"), pybind11::arg("dual_offset"), pybind11::arg("act"),
+     pybind11::arg("tile_group"), pybind11::arg("tile_tok0"), pybind11::arg("tile_ntok"), pybind11::arg("meta"),
+     pybind11::arg("max_tiles"), pybind11::arg("rows_per_group"), pybind11::arg("n_tok"), pybind11::arg("act_ab"),
+     pybind11::arg("bias") = pybind11::none());
   m.def("qkv_norm_append", [](const Tensor& q, const Tensor& k, const Tensor& v, const OptT& qw, const OptT& kw, double eps,
                               const Tensor& slots, Tensor& q_out, Tensor& k_cache, Tensor& v_cache) {
     const bool f32 = is_f32(q, "q");
@@ -406,14 +524,30 @@ void bind_layers(pybind11::module_& m) {
   });
   m.def("paged_attn_general", [](const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu_q,
                                  const Tensor& ctx_lens, const Tensor& block_table, double scale, int64_t window,
-                                 Tensor& out, double softcap) {
+                                 Tensor& out, double softcap, int64_t keep, const OptT& sink, const OptT& gate, double out_scale) {
     const bool f32 = is_f32(q, "q");
     same(k_cache, f32, "k_cache");
     same(v_cache, f32, "v_cache");
     same(out, f32, "out");
     const int64_t T = q.size(0), Hq = q.size(1), DK = q.size(2), Hkv = k_cache.size(-2), DV = v_cache.size(-1);
-    TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() &&
-                    k_cache.size(-1) == DK && out.size(0) == T && out.size(1) == Hq && out.size(2) == DV,
+    lb::AttnExtra x;
+    if (out.dim() == 2) {              // rows may lie apart; sinks, kept first tokens, output gate and scale
+      TORCH_CHECK(out.size(0) == T && out.size(1) == Hq * DV && keep >= 0, "paged_attn_general: out [T, heads * value head size]");
+      x.on = 1; x.keep = int(keep); x.out_scale = float(out_scale); x.ldo = out.stride(0);
+      if (sink.has_value()) {
+        f32c(*sink, Hq, "sinks");
+        x.sink = sink->data_ptr<float>();
+      }
+      if (gate.has_value()) {
+        same(*gate, f32, "gate");
+        TORCH_CHECK(gate->size(0) == T && gate->size(1) == Hq, "paged_attn_general: gate [T, heads]");
+        x.gate = gate->data_ptr(); x.ld_gate = gate->stride(0);
+      }
+    } else {
+      TORCH_CHECK(out.dim() == 3 && out.is_contiguous() && out.size(0) == T && out.size(1) == Hq && out.size(2) == DV && !keep &&
+                      !sink.has_value() && !gate.has_value() && out_scale == 1., "paged_attn_general: out [T, heads, size]");
+    }
+    TORCH_CHECK(q.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.size(-1) == DK,
                 "paged_attn_general: shapes");
     TORCH_CHECK(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_table.scalar_type() == at::kInt &&
                     cu_q.numel() == ctx_lens.numel() + 1 && block_table.stride(1) == 1, "paged_attn_general: int32 tables");
@@ -422,9 +556,12 @@ void bind_layers(pybind11::module_& m) {
                                               cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), block_table.data_ptr<int>(),
                                               int(block_table.stride(0)), int(k_cache.size(-3)), int(ctx_lens.numel()),
                                               int(T), int(Hq), int(Hkv), int(DK), int(DV), float(scale), float(softcap),
-                                              int(window), out.data_ptr(), f32, cur_stream()) == 0,
+                                              int(window), out.data_ptr(), f32, cur_stream(), x) == 0,
                 "paged_attn_general: value heads of at most 1024 columns, key heads of at most 2560", cuda_error());
-  });
+  }, pybind11::arg("q"), pybind11::arg("k_cache"), pybind11::arg("v_cache"), pybind11::arg("cu_q"), pybind11::arg("ctx_lens"),
+     pybind11::arg("block_table"), pybind11::arg("scale"), pybind11::arg("window"), pybind11::arg("out"), pybind11::arg("softcap"),
+     pybind11::arg("keep") = 0, pybind11::arg("sink") = pybind11::none(), pybind11::arg("gate") = pybind11::none(),
+     pybind11::arg("out_scale") = 1.);
   m.def("linear_scan", [](const Tensor& q, const Tensor& k, const Tensor& v, bool silu_in, const OptT& decay, const OptT& dt,
                           const OptT& dt_bias, const OptT& A, const OptT& D, const OptT& z, Tensor& state, const Tensor& cu,
                           const Tensor& slots, int64_t H, int64_t G, int64_t N, int64_t P, Tensor& out, bool write_state,

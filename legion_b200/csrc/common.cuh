@@ -33,6 +33,9 @@ enum : int {
   SITE_CHUNK_SCORES = 5 << 8,
   SITE_CHUNK_OUTPUT = 6 << 8,
   SITE_DELTA_SCAN = 7 << 8,
+  SITE_FORGET_STATES = 8 << 8,
+  SITE_FORGET_LEVEL = 9 << 8,
+  SITE_FORGET_OUTPUT = 10 << 8,
 };
 
 // Default deadline for in-kernel waits, in nanoseconds of %globaltimer.

@@ -121,10 +121,11 @@ __device__ __forceinline__ float gate_act(float v, int act) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
 }
 
-// UNARY: the output passes xIELU with the two numbers of WgemmArgs::xielu, or max(., 0)^2. Variants of their own, as is the
+// UNARY: the output passes xIELU with the two numbers of WgemmArgs::xielu, or max(., 0)^2; UN_BIAS: gate and up get their
+// biases (DUAL). Variants of their own, as is the
 // lookahead of output rows for wide token tiles: decode-sized launches run the epilogue once, and code they skip still
 // costs them instruction fetches.
-enum : int { UN_NONE = 0, UN_XIELU = 1, UN_RELU2 = 2 };
+enum : int { UN_NONE = 0, UN_XIELU = 1, UN_RELU2 = 2, UN_BIAS = 3 };
 template <int BN, bool DUAL, bool OUT_F32, bool WFP4, bool WFP8 = false, int UNARY = UN_NONE>
 __global__ void __launch_bounds__(WFP4 ? 448 : 192, 1)
 wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
@@ -587,6 +588,15 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
               if (DUAL) u[j] *= gs1;
             }
           }
+          if constexpr (UNARY == UN_BIAS) {
+            const int feat = it.feat0 + row;
+            const float bg = feat < a.n_feat ? a.bias[feat] : 0.f, bu = feat < a.n_feat ? a.bias[a.n_feat + feat] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              g[j] += bg;
+              u[j] += bu;
+            }
+          }
           if constexpr (UNARY == UN_RELU2) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
@@ -939,7 +949,7 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
   }
   a.tile_group = h.tile_group; a.tile_tok0 = h.tile_tok0; a.tile_out0 = h.tile_out0; a.tile_ntok = h.tile_ntok; a.n_tiles_dev = h.n_tiles_dev;
   a.n_tok_tiles_max = h.n_tok_tiles_max;
-  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act; a.xielu = h.xielu;
+  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act; a.xielu = h.xielu; a.bias = h.bias;
   a.x_group_col = h.x_group_col;
   // (a last K tile that reaches into the next group's columns meets weights that TMA filled with zeros)
   if (h.x_group_col != 0 && (h.x_group_col % 8 != 0 || h.K % 8 != 0 || fp8 || fp4 || !h.tile_group)) {
@@ -962,6 +972,10 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
     snprintf(g_gemm_err, sizeof(g_gemm_err), "wgemm: unary activations come with bf16 weights and bf16 output, one weight tile");
     return 1;
   }
+  if (h.bias && (!h.dual || fp4 || fp8 || h.out_f32 || h.tile_group)) {
+    snprintf(g_gemm_err, sizeof(g_gemm_err), "wgemm: biases come with ungrouped bf16 gate/up weights and bf16 output");
+    return 1;
+  }
   const int num_kb = fp8 ? h.K / 128 : (h.K + BK - 1) / BK;
   if (a.split_k > num_kb) a.split_k = num_kb;
   while (a.split_k > 1 && (a.split_k - 1) * ((num_kb + a.split_k - 1) / a.split_k) >= num_kb) --a.split_k;
@@ -979,6 +993,9 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
     if (fp4) return launch<BN_, DUAL_, false, true>(tmW, tmX, tmS, a, grid, stream);            \
     if (fp8) {                                                                                  \
       if constexpr (BN_ <= 64) return launch<BN_, DUAL_, false, false, true>(tmW, tmX, tmS, a, grid, stream); \
+    }                                                                                           \
+    if constexpr (DUAL_) {                                                                      \
+      if (h.bias) return launch<BN_, true, false, false, false, UN_BIAS>(tmW, tmX, tmS, a, grid, stream); \
     }                                                                                           \
     if constexpr (!DUAL_) {                                                                     \
       if (h.xielu) return launch<BN_, false, false, false, false, UN_XIELU>(tmW, tmX, tmS, a, grid, stream); \

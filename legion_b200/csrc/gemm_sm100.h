@@ -62,6 +62,7 @@ struct WgemmArgs {
   int dual_offset;                // DUAL: rows from a feature's gate row to its up row
   int act;                        // DUAL: activation of the gate, 0 = silu, 1 = gelu (tanh form)
   const float* xielu;             // not DUAL, xIELU variant: its two numbers (act_type.cuh)
+  const float* bias;              // DUAL, bias variant: added to gate (n_feat numbers) and up (the same, behind them)
   int split_k;
   int vec_ok;                     // output rows may be written as aligned 16-byte vectors
   float* ws;                      // split-K partials
@@ -90,6 +91,7 @@ struct WgemmHost {
   int bn; bool dual; int act;
   const float* xielu;             // not dual: the output passes xIELU with these two numbers (null: not)
   bool relu2;                     // not dual: the output is max(., 0)^2
+  const float* bias;              // dual: [2 * n_feat] added to gate and up ahead of the activation (null: none)
   const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles_dev;
   const int* tile_out0;
   int n_tok_tiles_max;

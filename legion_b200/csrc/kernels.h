@@ -3,6 +3,8 @@
 #pragma once
 #include <cuda_runtime.h>
 
+#include "attn_extra.h"
+
 namespace lb {
 
 int rmsnorm_launch(const void* x, long ldx, const void* res_in, long ldri, void* res_out, long ldro, const float* w,
@@ -34,13 +36,13 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
                            long v_cell, const int* block_table, int table_width, int page, const int* ctx_lens,
                            float scale, float softcap, int window, int B, int Hq, int Hkv, int dk, int dv, int n_splits,
                            float* o_part, float* ml_part, void* out, int* group_ctr, int n_group_ctr, int* status,
-                           cudaStream_t s);
+                           cudaStream_t s, const AttnExtra& x = AttnExtra{});
 const char* paged_decode_tc_last_error();
 
 int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* v_cache, long n_cells, long k_cell,
                         long v_cell, const int* cu_q, const int* ctx_lens, const int* block_table, int table_width,
                         int page, int n_seqs, int max_q_len, int Hq, int Hkv, int dk, int dv, float scale, float softcap,
-                        int window, int causal, void* out, int* status, cudaStream_t s);
+                        int window, int causal, void* out, int* status, cudaStream_t s, const AttnExtra& x = AttnExtra{});
 const char* prefill_attn_last_error();
 
 // Latent attention (absorbed form) over the paged latent cache: attn_mla_sm100.cu

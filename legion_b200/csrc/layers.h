@@ -5,6 +5,8 @@
 #include <cuda_runtime.h>
 #include <stddef.h>
 
+#include "attn_extra.h"
+
 namespace lb {
 
 // Hyper-connections with static weights (hyper.cu). X [rows, S, H] fp32.
@@ -27,6 +29,24 @@ struct HyperArgs {
   int rows, S, H;
 };
 int hyper_launch(const HyperArgs& a, bool f32, cudaStream_t s);
+
+// Parallel sublayers on one fp32 residual, with gates and depth average (depth_step.cu).
+struct DepthStepArgs {
+  const float* x;                  // [T, H] the layer's input
+  float* x_out;                    // [n_rows, H] the next one's (may be x without rows)
+  const float* hist; long hist_stride; int n_hist;   // X_0 .. X_(n_hist - 1), hist_stride floats apart; nullptr: no average
+  float* hist_out;                 // [T, H] takes the layer's result; nullptr: not kept
+  const float* coef;               // [n_hist + 1]
+  const void* y1; long ldy1;       // mixer output, activation type
+  const void* y2; long ldy2; int y2_rows; const float* y2_b;   // feed-forward output, the sum of y2_rows consecutive rows
+                                   // (nullptr: none), and its bias
+  const void* g1; const void* g2; long ldg; const float* b1; const float* b2;   // gates before bias and sigmoid; nullptr: open
+  const float* norm_w; float eps, w_offset;
+  void* h; long ldh;               // [n_rows, H]
+  const long* rows;                // tokens whose next input is wanted; nullptr: all
+  int n_rows, H;
+};
+int depth_step_launch(const DepthStepArgs& a, bool f32, cudaStream_t s);
 
 // One fp32 residual between grouped norms, with the next sublayer's input convolution (resid_step.cu).
 struct ResidStepArgs {
@@ -132,6 +152,7 @@ struct SgemmArgs {
   int dual; long dual_offset; int act;   // act(gate) * up, rows dual_offset apart; act 0 silu, 1 gelu (tanh), 2 relu^2
                                          // (no up), 3 xIELU (no up) with act_ab
   const float* act_ab;             // [2]
+  const float* bias;               // dual: [2 * N] added to gate and up ahead of the activation
   int heads; long x_head_col, out_head_col;  // heads > 1: head z reads x columns from z * x_head_col and weight rows from
                                              // z * rows_per_group, and writes output columns from z * out_head_col
   const int* tile_group; const int* tile_tok0; const int* tile_ntok; const int* n_tiles; int max_tiles;
@@ -191,7 +212,7 @@ int head_norm_gate_launch(const void* o, long ldo, const void* gate, long ldg, c
 int paged_attn_general_launch(const void* q, long q_row, const void* k_cache, const void* v_cache, long k_cell, long v_cell,
                               const int* cu_q, const int* ctx_lens, const int* block_table, int table_width, int page,
                               int n_seqs, int T, int Hq, int Hkv, int DK, int DV, float scale, float softcap, int window,
-                              void* out, bool f32, cudaStream_t s);
+                              void* out, bool f32, cudaStream_t s, const AttnExtra& x = AttnExtra{});
 
 // Decayed outer-product state S_t = a_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (linear_scan.cu, linear_scan_sm100.cu).
 struct LinScanArgs {
@@ -220,6 +241,26 @@ size_t linear_chunk_scratch_bytes(int n_chunks, int H, int N, int P);
 int linear_chunk_launch(const LinScanArgs& a, const int* chunk_t0, const int* chunk_n, const int* chunk_seq,
                         int n_chunks, const int* seq_chunk0, const int* seq_nchunk, void* scratch, int* status,
                         cudaStream_t s);
+
+// HGRN2 (forget_scan.cu, forget_scan_sm100.cu): F = lower + (1 - lower) sigmoid(f + f_b), S_t = diag(F_t) S_(t-1) +
+// (1 - F_t) v_t^T, o_t = S_t^T silu(q_t), out = o / rms(o) * norm_w * scale per head.
+struct ForgetScanArgs {
+  const void* q; const void* f; const void* v; long ldq, ldf, ldv;   // [T, H * N], [T, H * N], [T, H * P]
+  const float* f_b; const float* lower;   // [H * N]
+  float* state;                    // [slots, H, P, N]
+  const int* cu; const int* slots;
+  int n_seqs, T, H, N, P;
+  const float* norm_w; float eps, scale;
+  void* out; long ldo;             // [T, H * P]
+  int write_state;
+  int max_tokens;                  // forget_scan: sequences with more tokens are left alone (0: all run)
+};
+int forget_scan_launch(const ForgetScanArgs& a, bool f32, cudaStream_t s);
+// Chunked form on tcgen05 (bf16), chunk tables as of linear_chunk_launch; scratch: forget_chunk_scratch_bytes, 256-byte aligned
+bool forget_chunk_ok(int N, int P);
+size_t forget_chunk_scratch_bytes(int n_chunks, int H, int N, int P);
+int forget_chunk_launch(const ForgetScanArgs& a, const int* chunk_t0, const int* chunk_n, int n_chunks, const int* seq_chunk0,
+                        const int* seq_nchunk, void* scratch, int* status, cudaStream_t s);
 
 // One decode step of a Mamba-2 mixer: convolution with history update, step size, state update, skip and gate.
 struct SsdDecodeArgs {

@@ -16,6 +16,7 @@ namespace lb {
 // mode 1: sigmoid scores, selection by score + bias, optional group-limited routing (n_group groups,
 // keep topk_group groups ranked by the sum of their group_top (1 or 2) best biased scores), weights = unbiased
 // scores of the chosen experts, renormalised and multiplied by route_scale. mode 2: as mode 1 with softmax scores.
+// mode 3: as mode 0 with the bias added to the logits.
 // renorm 1: by the sum of the chosen weights, held away from zero; 2: by the sum + 1e-20.
 template <int MAXE>
 __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, const float* __restrict__ bias, int E,
@@ -24,12 +25,15 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
                                                 float* __restrict__ wts, int t, int* sm_ids = nullptr, float* sm_wts = nullptr) {
   constexpr int PER = MAXE / 32;
   const int lane = threadIdx.x & 31;
+  const bool logit_bias = mode == 3;
+  if (logit_bias) mode = 0;
   float sc[PER], sel[PER];
   float mx = -INFINITY;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
     sc[j] = (e < E) ? __ldcg(logits + t * ldl + e) : -INFINITY;   // L2 read: the row may come from other CTAs
+    if (logit_bias && e < E) sc[j] += bias[e];
     mx = fmaxf(mx, sc[j]);
   }
   float inv_sum = 1.f;
@@ -147,7 +151,7 @@ __device__ __forceinline__ void router_topk_row(const float* logits, long ldl, c
   // weights of the chosen experts from their logits (lane i < k holds choice i)
   float w = 0.f;
   if (lane < k) {
-    const float l = __ldcg(logits + t * ldl + my_id);
+    const float l = __ldcg(logits + t * ldl + my_id) + (logit_bias ? bias[my_id] : 0.f);
     if (mode == 0) w = renorm ? l : __expf(l - mx) * inv_sum;
     else if (mode == 2) w = __expf(l - mx) * inv_sum;
     else w = 1.f / (1.f + __expf(-l));
@@ -201,8 +205,8 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
 constexpr int ROUTE_LSTR = 64 * 512;          // floats between the logit planes of two K splits
 constexpr int ROUTE_MAX_KSPLIT = 4;
 
-// EXT: weights by the sum + 1e-20 (renorm 2) and the shared expert as several groups; a variant of its own, since the launch
-// is latency and code it skips still costs instruction fetches.
+// EXT: weights by the sum + 1e-20 (renorm 2), the shared expert as several groups, a bias on the logits (mode 3); a variant of
+// its own, since the launch is latency and code it skips still costs instruction fetches.
 template <int MAXE, bool EXT>
 __global__ void __launch_bounds__(512) moe_route_small_kernel(
     const __nv_bfloat16* __restrict__ x, long ldx, const float* __restrict__ norm_w, float eps, float w_offset,
@@ -225,6 +229,8 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
   griddep_launch();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nv = H / 8;
+  const bool logit_bias = EXT && mode == 3;
+  if (logit_bias) mode = 0;
 
   // K split: CTA (rg, ks) owns router rows rg * epc .. and columns ks * H / ksplit .. of them; the partial logits of
   // the splits land in separate planes (LSTR floats apart) and are added in a fixed order by whoever reads them
@@ -375,6 +381,7 @@ __global__ void __launch_bounds__(512) moe_route_small_kernel(
     if (e < E) {
       l = __ldcg(logits + long(t) * E + e);
       for (int sp = 1; sp < ksplit; ++sp) l += __ldcg(logits + long(sp) * ROUTE_LSTR + long(t) * E + e);
+      if (EXT && logit_bias) l += bias[e];
     }
     s_logit[e] = l;
     float mxv = 0.f, inv_sum = 1.f;
@@ -569,6 +576,7 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
   if (T <= 0) return 0;
   if (k > 32 || E > 512 || n_group > 32 || H % 8 || T > 64 || T * k > 1024 || T > bn || shared_rows < 0 || shared_rows > 64)
     return 1;
+  if (mode == 3 && !bias) return 1;
   if (sh_gate_w && (!sh_logit || !(shared_slot || shared_rows))) return 1;
   auto sg = static_cast<const __nv_bfloat16*>(sh_gate_w);
   auto xb = static_cast<const __nv_bfloat16*>(x);
@@ -596,7 +604,7 @@ int moe_route_small_launch(const void* x, long ldx, const float* norm_w, float e
                bn, tile_group, slot_base, tile_ntok, meta, out_rows, tok_scale, done_ctr, e_lo, n_local, sg,        \
                sh_logit, shared_slot, shared_rows, epc, tpp, ksplit, status, active);                               \
   }
-  const bool ext = shared_rows > 0 || renorm == 2;
+  const bool ext = shared_rows > 0 || renorm == 2 || mode == 3;
   if (E <= 128) { if (ext) LB_ROUTE(128, true) else LB_ROUTE(128, false) }
   else if (E <= 256) { if (ext) LB_ROUTE(256, true) else LB_ROUTE(256, false) }
   else { if (ext) LB_ROUTE(512, true) else LB_ROUTE(512, false) }
@@ -608,7 +616,7 @@ int router_topk_launch(const float* logits, long ldl, const float* bias, int E, 
                        float route_scale, int n_group, int topk_group, int group_top, int* ids, float* wts, float* gate,
                        int T, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (k > 32 || E > 512 || n_group > 32) return 1;
+  if (k > 32 || E > 512 || n_group > 32 || (mode == 3 && !bias)) return 1;
   const int blocks = (T * 32 + 127) / 128;
   if (E <= 128)
     router_topk_kernel<128><<<blocks, 128, 0, s>>>(logits, ldl, bias, E, k, mode, renorm, route_scale, n_group,

@@ -97,7 +97,8 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const SgemmArgs a) {
       const int n = n0 + fm + j;
       if (n >= a.N) continue;
       float v = acc[0][i][j];
-      if constexpr (DUAL) v = act_of<T>(v, a.act) * acc[1][i][j];
+      if constexpr (DUAL) v = a.bias ? act_of<T>(v + a.bias[n], a.act) * (acc[1][i][j] + a.bias[a.N + n])
+                                     : act_of<T>(v, a.act) * acc[1][i][j];
       else if (a.act == 2) { v = fmaxf(v, 0.f); v *= v; }
       else if (a.act == 3) v = xielu_f(v, a.act_ab[0], a.act_ab[1]);
       v *= sc;

@@ -3,7 +3,8 @@
 ``config.json`` ``model_type`` selects the mapper: ``qwen3`` / ``qwen3_moe`` / ``llama`` / ``mistral``,
 ``qwen3_next`` / ``qwen3_5`` / ``qwen3_5_moe`` (hybrid Gated DeltaNet), ``deepseek_v3`` (MLA), ``gemma4`` /
 ``gemma4_text`` (``hf_gemma4``), ``nemotron_h`` (``hf_nemotron``); ``architecture: Nisasun`` (``nisasun``),
-``architecture: Pemezen`` (``pemezen``), ``architecture: Gurozen`` (``gurozen``).
+``architecture: Pemezen`` (``pemezen``), ``architecture: Gurozen`` (``gurozen``),
+``architecture: Mananex`` (``mananex``).
 Transforms applied while loading the Qwen3.5 family (``src/hf/qwen35.rs:6-20`` in the reference):
 ``A_log -> -exp(A_log)``; RMSNorm weights stored as (w - 1) get +1 (all but the DeltaNet output norm);
 fused ``in_proj_qkvz`` / ``in_proj_ba`` are de-interleaved per key head; conv1d ``[C, 1, k]`` is squeezed;
@@ -20,7 +21,7 @@ import torch
 
 from ..config import ModelConfig
 from ..models.weights import is_fp32_weight, weight_shapes
-from . import gurozen, hf_gemma4, hf_nemotron, nisasun, pemezen
+from . import gurozen, hf_gemma4, hf_nemotron, mananex, nisasun, pemezen
 from . import quant_formats as qf
 from .safetensors_io import Checkpoint, save_file
 
@@ -38,6 +39,8 @@ def config_from_hf(c: dict) -> ModelConfig:
         return pemezen.config_from_json(c)
     if gurozen.is_gurozen(c):
         return gurozen.config_from_json(c)
+    if mananex.is_mananex(c):
+        return mananex.config_from_json(c)
     c = dict(c.get("text_config") or c)
     mt = c.get("model_type", "llama")
     n_head = c["num_attention_heads"]
@@ -239,6 +242,9 @@ def load_hf(path: str, device="cpu", dtype=torch.float32, keep_quant: bool = Fal
         return cfg, w, ck
     if gurozen.is_gurozen(ck.config):
         cfg, w = gurozen.load(ck, torch.device(device), dtype)
+        return cfg, w, ck
+    if mananex.is_mananex(ck.config):
+        cfg, w = mananex.load(ck, torch.device(device), dtype)
         return cfg, w, ck
     cfg = config_from_hf(ck.config)
     src = _Source(ck, torch.device(device), dtype)

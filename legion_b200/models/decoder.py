@@ -180,7 +180,7 @@ class StatePool:
                     self.ssm[il] = torch.zeros(n_slots, r.width, device=device, dtype=torch.float32)
                     self.conv[il] = torch.zeros(n_slots, r.width, r.conv - 1, device=device, dtype=torch.float32)
                     continue
-                N = r.dim if r.kind == "lightning" else r.state
+                N = r.state if r.kind == "ssd" else r.dim
                 # state[head, value column, key column]
                 self.ssm[il] = torch.zeros(n_slots, r.heads, r.vdim, N, device=device, dtype=torch.float32)
                 if r.kind == "ssd":
@@ -982,8 +982,9 @@ class Decoder:
         return out
 
     # ------------------------------------------------------------------ stacks with layer specifications
-    def _softmax_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache, st: StatePool):
-        """Attention part of a layer; ``proj`` starts with its q | k | v columns. Returns (output, columns used)."""
+    def _softmax_heads(self, p: str, il: int, proj, b: StepBatch, kv: KvCache, st: StatePool, scale: float = 1.0, out=None):
+        """Attention part of a layer in front of its output projection; ``proj`` starts with its q | k | v columns. Returns
+        [T, heads * vdim] times ``scale``, in ``out`` when given."""
         cfg, w, a = self.cfg, self.w, self.cfg.attn_spec(il)
         nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
         if a.direct():
@@ -997,9 +998,29 @@ class Decoder:
                                     self.rotary_table(a.rot) if a.rot is not None else None,
                                     a.rot.layout if a.rot is not None else "half", b.positions, b.slots, kv.k[il], kv.v[il],
                                     a.heads, write_state=b.write_state, max_len=b.max_q_len)
+        g = cfg.mix_columns(il)["g"] if a.gate == "head" else 0
         o = ops.paged_attention(q, kv.k[il], kv.v[il], b.block_table, b.ctx_lens, b.cu_q, b.max_q_len, a.scale,
-                                window=a.window, max_ctx=b.max_ctx or None, softcap=a.softcap)
-        return ops.linear(o.reshape(o.shape[0], -1), w[f"{p}.attn.o"]), nq + nk + nv
+                                window=a.window, max_ctx=b.max_ctx or None, softcap=a.softcap, keep_first=a.keep_first,
+                                sink=w.get(f"{p}.attn.sink"), gate=proj[:, g:g + a.heads] if g else None, out_scale=scale,
+                                out=out)
+        return o.reshape(o.shape[0], -1)
+
+    def _softmax_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache, st: StatePool):
+        return ops.linear(self._softmax_heads(p, il, proj, b, kv, st), self.w[f"{p}.attn.o"])
+
+    def _merged_mixer(self, p: str, il: int, proj, b: StepBatch, kv: KvCache, st: StatePool):
+        """HGRN2, alone or beside attention: both parts write their scaled columns of one tensor, one output projection."""
+        cfg, w, m, a, r = self.cfg, self.w, self.cfg.layers[il].mixer, self.cfg.attn_spec(il), self.cfg.recurrent_spec(il)
+        ls, rs = (m.left_scale, m.right_scale) if m.kind == "parallel" else (1.0, 1.0)
+        nl, col = a.heads * a.vdim if a is not None else 0, cfg.mix_columns(il)
+        o = torch.empty(proj.shape[0], nl + r.heads * r.vdim, dtype=proj.dtype, device=proj.device)
+        if a is not None:
+            self._softmax_heads(p, il, proj, b, kv, st, ls, o[:, :nl])
+        part = lambda n, width: proj[:, col[n]:col[n] + width]                                # noqa: E731
+        ops.forget_scan(part("rq", r.heads * r.dim), part("rf", r.heads * r.dim), part("rv", r.heads * r.vdim), w[f"{p}.hg.f_b"],
+                        w[f"{p}.hg.lower"], st.ssm[il], b.cu_q, b.state_slots, r.heads, r.dim, r.vdim, w[f"{p}.hg.norm"],
+                        cfg.rms_eps, rs, write_state=b.write_state, max_len=b.max_q_len, cu_host=b.cu_q_host, out=o[:, nl:])
+        return ops.linear(o, w[f"{p}.mix.o"])
 
     def _ssd_mixer(self, p: str, il: int, proj, b: StepBatch, st: StatePool):
         """Mamba-2 part of a layer; ``proj`` holds its z | x | B | C | dt columns. Decode steps run convolution, state
@@ -1122,17 +1143,20 @@ class Decoder:
         proj = ops.linear(h, self.w[f"{p}.mix.in"])
         if m.kind == "ssd":
             return [(self._ssd_mixer(p, il, proj, b, st), 1.0)]
-        left, used = self._softmax_mixer(p, il, proj, b, kv, st)
+        if self.cfg.merged_output(il):
+            return [(self._merged_mixer(p, il, proj, b, kv, st), 1.0)]
+        left = self._softmax_mixer(p, il, proj, b, kv, st)
         if m.kind == "attn":
             return [(left, 1.0)]
-        return [(left, m.left_scale), (self._ssd_mixer(p, il, proj[:, used:], b, st), m.right_scale)]
+        return [(left, m.left_scale), (self._ssd_mixer(p, il, proj[:, self.cfg.mix_columns(il)["ssd"]:], b, st), m.right_scale)]
 
     def _spec_ffn(self, p: str, il: int, h):
         w, f = self.w, self.cfg.layers[il].mlp
         if f.kind == "dense" and not f.gated():
             return [(ops.linear(ops.up_act(h, w[f"{p}.mlp.up"], w[f"{p}.mlp.act"]), w[f"{p}.mlp.down"]), 1.0)]
         if f.kind == "dense":
-            return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act), w[f"{p}.mlp.down"]), 1.0)]
+            return [(ops.linear(ops.gate_up_act(h, w[f"{p}.mlp.gate_up"], f.ff, f.act, w.get(f"{p}.mlp.gate_up_b")),
+                                w[f"{p}.mlp.down"]), 1.0)]       # (a bias of the down projection joins in the step behind)
         up, down, E = w[f"{p}.moe.gate_up"], w[f"{p}.moe.down"], f.experts
         routing = ops.router(h, w[f"{p}.moe.router"], f.top, f.router, f.renorm, f.scale, w.get(f"{p}.moe.router_bias"),
                              f.n_group, f.keep_group, n_local=E, group_top=f.group_top, gate_row=f.shared_gate,
@@ -1245,6 +1269,41 @@ class Decoder:
             if b.capture_layers and il in b.capture_layers and (last or subs[i + 1][0] != il):
                 captures[il] = x.clone()
         hidden = h if b.logit_rows is None else h.index_select(0, b.logit_rows)
+        out = StepOutput(hidden=hidden, captures=captures)
+        if want_logits:
+            out.logits = self.logits(hidden)
+        self.pctx.end_step()
+        return out
+
+    def _forward_parallel(self, b: StepBatch, kv: KvCache, st: Optional[StatePool], want_logits: bool) -> StepOutput:
+        """Forward pass of a stack with layer specifications whose sublayers read one norm side by side, on one fp32 residual.
+        Behind a layer one launch gates and adds both results, sums up the depth average and norms the next input."""
+        cfg, w = self.cfg, self.w
+        H, eps, off, L = cfg.hidden, cfg.rms_eps, cfg.norm_offset, cfg.n_layer
+        table, ids = (w["tok_embd"], b.token_ids) if b.embeds is None else (b.embeds, None)
+        x, hist, h = ops.depth_start(table, ids, L, w["l0.attn_norm"], eps, off, cfg.depth_average)
+        captures: Dict[int, torch.Tensor] = {}
+        rows = b.logit_rows                           # behind the last layer only the wanted rows go on
+        for il, spec in enumerate(cfg.layers):
+            p, last = f"l{cfg.weight_layer(il)}", il + 1 == L
+            capture = bool(b.capture_layers) and il in b.capture_layers
+            g1 = b1 = g2 = b2 = y2 = None
+            proj, col = ops.linear(h, w[f"{p}.mix.in"]), cfg.mix_columns(il)
+            y1 = self._merged_mixer(p, il, proj, b, kv, st) if cfg.merged_output(il) else self._softmax_mixer(p, il, proj, b, kv, st)
+            if spec.mlp is not None:
+                y2 = self._spec_ffn(p, il, h)[0][0]
+            if cfg.residual_gate:
+                g1, b1 = proj[:, col["rg1"]:col["rg1"] + H], w[f"{p}.rg_b"][:H]
+                if y2 is not None:
+                    g2, b2 = proj[:, col["rg2"]:col["rg2"] + H], w[f"{p}.rg_b"][H:]
+            keep = None
+            if last and not capture:
+                keep, rows = rows, None
+            x, h = ops.depth_step(x, hist, il, y1, g1, b1, y2, g2, b2, w.get(f"{p}.mlp.down_b"), w.get(f"{p}.dwa"),
+                                  w["output_norm"] if last else w[f"l{cfg.weight_layer(il + 1)}.attn_norm"], eps, off, keep)
+            if capture:
+                captures[il] = x.clone()
+        hidden = h if rows is None else h.index_select(0, rows)
         out = StepOutput(hidden=hidden, captures=captures)
         if want_logits:
             out.logits = self.logits(hidden)
@@ -1500,6 +1559,8 @@ class Decoder:
         if self.cfg.layers is not None:
             if self.cfg.sandwich_norm:
                 return self._forward_sandwich(b, kv, st, want_logits)
+            if self.cfg.parallel_sublayers:
+                return self._forward_parallel(b, kv, st, want_logits)
             if self.cfg.hyper_mode == "static":
                 return self._forward_streams(b, kv, st, want_logits)
             return self._forward_prenorm(b, kv, st, want_logits)

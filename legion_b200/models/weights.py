@@ -135,12 +135,16 @@ def _ffn_shapes(cfg: ModelConfig, p: str, moe: bool, s: Dict[str, Tuple[int, ...
 
 def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
     """A layer of a stack with specifications (``ModelConfig.layers``). What reads the mixer's input is one stacked
-    projection: ``lin.qkvg`` (linear attention: q | k | v | gate), ``mix.in`` (q | k | v of the attention part, then
-    z | x | B | C | dt of the state-space part), ``cd.in`` (``ChannelDeltaSpec.in_columns``)."""
+    projection: ``lin.qkvg`` (linear attention: q | k | v | gate), ``mix.in`` (``ModelConfig.mix_columns``; z | x | B | C | dt
+    of a state-space part), ``cd.in`` (``ChannelDeltaSpec.in_columns``)."""
     p, H, spec = f"l{cfg.weight_layer(il)}", cfg.hidden, cfg.layers[il]
     s: Dict[str, Tuple[int, ...]] = {f"{p}.attn_norm": (H,)}
-    if spec.mlp is not None:
+    if spec.mlp is not None and not cfg.parallel_sublayers:
         s[f"{p}.ffn_norm"] = (H,)
+    if cfg.residual_gate:
+        s[f"{p}.rg_b"] = (H if spec.mlp is None else 2 * H,)                    # mixer | feed-forward
+    if cfg.depth_average:
+        s[f"{p}.dwa"] = (il + 2,)                       # embedding output, results of layers 0 .. il
     m = spec.mixer
     if m.kind == "lightning":
         s[f"{p}.lin.qkvg"] = (2 * m.heads * (m.dim + m.vdim), H)
@@ -172,10 +176,10 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
         s[f"{p}.cd.norm"] = (m.vdim,)
         s[f"{p}.cd.out"] = (H, nv)
     else:
-        a, r = cfg.attn_spec(il), cfg.recurrent_spec(il)
-        rows = 0
+        a, r, merged = cfg.attn_spec(il), cfg.recurrent_spec(il), cfg.merged_output(il)
+        out_cols = 0
         if a is not None:
-            rows += (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim
+            rows = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim
             if a.qk_norm:
                 whole = a.norm_over == "all"
                 s[f"{p}.attn.q_norm"] = (a.heads * a.dim if whole else a.dim,)
@@ -184,17 +188,25 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
                 s[f"{p}.attn.in_b"] = (rows,)
             if a.conv:
                 s[f"{p}.attn.conv_w"] = (a.conv, rows)                          # oldest token first
-            s[f"{p}.attn.o"] = (H, a.heads * a.vdim)
-        if r is not None:
+            if a.sink:
+                s[f"{p}.attn.sink"] = (a.heads,)
+            out_cols += a.heads * a.vdim
+            if not merged:
+                s[f"{p}.attn.o"] = (H, out_cols)
+        if merged:
+            s[f"{p}.hg.f_b"] = (r.heads * r.dim,)
+            s[f"{p}.hg.lower"] = (r.heads * r.dim,)
+            s[f"{p}.hg.norm"] = (r.vdim,)
+            s[f"{p}.mix.o"] = (H, out_cols + r.heads * r.vdim)
+        elif r is not None:
             inner, conv_c = r.heads * r.vdim, r.heads * r.vdim + 2 * r.groups * r.state
-            rows += inner + conv_c + r.heads
             s[f"{p}.ssm.conv_w"] = (conv_c, r.conv)
             s[f"{p}.ssm.conv_b"] = (conv_c,)
             for leaf in ("A", "D", "dt_bias"):
                 s[f"{p}.ssm.{leaf}"] = (r.heads,)
             s[f"{p}.ssm.norm"] = (inner,)
             s[f"{p}.ssm.out"] = (H, inner)
-        s[f"{p}.mix.in"] = (rows, H)
+        s[f"{p}.mix.in"] = (cfg.mix_columns(il)["end"], H)
     n = cfg.hyper_streams
     if cfg.sandwich_norm:
         for which in ("attn", "ffn")[:1 if spec.mlp is None else 2]:
@@ -211,7 +223,7 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
     if f.kind == "moe":
         n = f.experts + f.shared_slots()
         s[f"{p}.moe.router"] = (f.experts + int(f.shared_gate), H)              # its last row gates the shared expert
-        if f.correction:
+        if f.correction or f.router == "biased_softmax":
             s[f"{p}.moe.router_bias"] = (f.experts,)
         s[f"{p}.moe.gate_up"] = (n, 2 * f.ff if f.gated() else f.ff, H)
         s[f"{p}.moe.down"] = (n, H, f.ff)
@@ -222,6 +234,8 @@ def spec_layer_shapes(cfg: ModelConfig, il: int) -> Dict[str, Tuple[int, ...]]:
     else:
         s[f"{p}.mlp.gate_up"] = (2 * f.ff, H)
         s[f"{p}.mlp.down"] = (H, f.ff)
+        if f.bias:
+            s[f"{p}.mlp.gate_up_b"], s[f"{p}.mlp.down_b"] = (2 * f.ff,), (H,)
     return s
 
 
@@ -311,7 +325,8 @@ def is_fp32_weight(name: str) -> bool:
     return leaf.endswith("norm") or leaf in ("A", "D", "dt_bias", "conv_w", "conv_b", "router_bias", "hc_f", "hc_scale",
                                              "hc_base", "hcg_norm", "hcg_down", "hcg_up", "hcg_inject", "router_scale",
                                              "out_scale", "st_in", "st_out", "st_mix", "in_b", "gates_b", "log_decay",
-                                             "act", "attn_taps", "ffn_taps")
+                                             "act", "attn_taps", "ffn_taps", "sink", "f_b", "lower", "rg_b", "dwa",
+                                             "gate_up_b", "down_b")
 
 
 def layer_of(name: str) -> Optional[int]:
@@ -352,7 +367,14 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=torch.float32, seed: in
             t = (2 * torch.log(0.9 + 0.099 * torch.rand(shp, generator=g))).to(device)
         elif leaf == "act":               # xIELU: softplus(p), 1/2 + softplus(q)
             t = torch.tensor([0.8, 1.3], device=device)
-        elif leaf in ("dt_bias", "conv_b", "router_bias", "in_b", "gates_b"):
+        elif leaf == "lower":             # lower bounds of forget gates
+            t = (0.9 * torch.rand(shp, generator=g)).to(device)
+        elif leaf == "dwa":               # near the plain residual: most weight on the last result
+            t = (torch.randn(shp, generator=g) * 0.05).to(device)
+            t[-1] += 1.0
+        elif leaf in ("rg_b", "f_b"):     # gates open, memories long
+            t = (1.5 + torch.randn(shp, generator=g)).to(device)
+        elif leaf in ("dt_bias", "conv_b", "router_bias", "in_b", "gates_b", "gate_up_b", "down_b", "sink"):
             t = (torch.randn(shp, generator=g) * 0.1).to(device)
         elif leaf in ("st_in", "st_out", "st_mix"):
             n = shp[0]                    # near the plain residual: the streams' mean in, every stream gets the output

@@ -34,7 +34,10 @@ def linear(x, w, residual=None, out_dtype=None, out=None, tok_scale=None):
     return y
 
 
-def gate_up_act(x, w_gate_up, n_ff, act="silu"):
+def gate_up_act(x, w_gate_up, n_ff, act="silu", bias=None):
+    """act(x Wg^T + bg) * (x Wu^T + bu); ``bias`` float32 [bg | bu], optional."""
+    if bias is not None and _cuda(x):
+        return _sm.gate_up_act(x, w_gate_up, n_ff, act=act, bias=bias)
     if _cuda(x):
         if act == "silu" or (act == "gelu_tanh" and isinstance(w_gate_up, torch.Tensor)):
             return _sm.gate_up_act(x, w_gate_up, n_ff, act=act)
@@ -42,7 +45,7 @@ def gate_up_act(x, w_gate_up, n_ff, act="silu"):
         out = torch.empty(x.shape[0], n_ff, dtype=torch.bfloat16, device=x.device)
         _sm.ext().glu(h, out, n_ff, {"gelu_tanh": 1, "relu2": 2}[act])
         return out
-    return _ref.gate_up_act(x, w_gate_up, n_ff, act)
+    return _ref.gate_up_act(x, w_gate_up, n_ff, act, bias)
 
 
 def rmsnorm(x, w, eps, w_offset=0.0, residual=None):
@@ -71,10 +74,24 @@ def apply_output_gate(attn, gate, n_q, d):
 
 
 def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, max_q_len, scale, window=0, causal=True,
-                    decode_splits=None, max_ctx=None, softcap=0.0):
+                    decode_splits=None, max_ctx=None, softcap=0.0, keep_first=0, sink=None, gate=None, out_scale=1.0, out=None):
     """Varlen paged attention; ``max_q_len == 1`` selects the flash-decoding kernel on CUDA. fp32 caches and head sizes
     the tensor-core kernels do not take run on the general kernel (causal only). ``softcap`` > 0: scores become
-    softcap * tanh(score / softcap)."""
+    softcap * tanh(score / softcap). ``keep_first``: first tokens that stay visible behind the window; ``sink`` [Hq]
+    float32: exp(sink) joins the softmax's denominator; ``gate`` [T, Hq]: each head's output times its sigmoid; ``out_scale``
+    multiplies the output; ``out`` [T, Hq * Dv] (rows may lie apart) takes it."""
+    if keep_first or sink is not None or gate is not None or out is not None or out_scale != 1.0:
+        if not causal or softcap:
+            raise NotImplementedError("sinks, kept first tokens and output gates come with causal attention without a soft cap")
+        if _cuda(q):
+            return _sm.attention_ext(q, k_cache, v_cache, block_table, ctx_lens, cu_q, max_q_len, scale, window, keep_first,
+                                     sink, gate, out_scale, out, decode_splits, max_ctx)
+        o = _ref.paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, sinks=sink,
+                                 keep_first=keep_first, gate=gate, out_scale=out_scale)
+        if out is None:
+            return o
+        out.copy_(o.reshape(out.shape))
+        return out
     if _cuda(q):
         if not _sm.attn_tc_ok(q, k_cache, v_cache):
             return _sm.paged_attn_general(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window, causal,
@@ -281,6 +298,37 @@ def head_norm_gate(o, gate, w, eps, heads):
         return _sm.head_norm_gate(o, gate, w, eps, heads)
     return _ref.gated_rmsnorm(o.view(o.shape[0], heads, -1), gate.reshape(o.shape[0], heads, -1), w, eps,
                               "sigmoid").reshape(o.shape)
+
+
+def depth_start(table, ids, layers: int, norm_w, eps, w_offset=0.0, average=True):
+    """Start of a stack with parallel sublayers: x = embedding rows (``ids`` None: rows are given). Returns (x [T, H] float32,
+    hist [layers + 1, T, H] float32 with x as its first entry, or None without depth averages, norm of x)."""
+    T = table.shape[0] if ids is None else ids.numel()
+    hist = torch.empty(layers + 1 if average else 1, T, table.shape[1], dtype=torch.float32, device=table.device)
+    if _cuda(table):
+        _, h = _sm.prenorm_step(None, (), 1.0, norm_w, eps, w_offset, None, start=(table, ids, None), x_out=hist[0])
+    else:
+        x, h = _ref.prenorm_start(table if ids is None else table[ids.long()], None, norm_w, eps, w_offset)
+        hist[0] = x
+    return hist[0], hist if average else None, h
+
+
+def depth_step(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset=0.0, rows=None):
+    """Behind a layer with parallel sublayers (see ``reference.depth_step``), one launch; ``y2`` may be a
+    ops.sm100.PendingCombine."""
+    f = _sm.depth_step if _cuda(x) else _ref.depth_step
+    return f(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset, rows)
+
+
+def forget_scan(q, f, v, f_b, lower, state, cu_seq, slots, H, N, P, norm_w, eps, scale=1.0, write_state=True, max_len=None,
+                cu_host=None, out=None):
+    """HGRN2 state with the norm per head behind it (see ``reference.forget_scan``); ``out`` [T, H * P] may have rows that lie
+    apart."""
+    args = (q, f, v, f_b, lower, state, cu_seq, slots, H, N, P, norm_w, eps, scale, write_state)
+    if _cuda(q):
+        return _sm.forget_scan(*args, max_len=max_len, cu_host=cu_host, out=out)
+    y = _ref.forget_scan(*args)
+    return y if out is None else out.copy_(y)
 
 
 def resid_start(table, ids, embed_scale, norm_w, groups, eps, conv=None, max_len=None):

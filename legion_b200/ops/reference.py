@@ -33,9 +33,11 @@ def linear(x, w, residual=None, out_dtype=None):
     return y.to(out_dtype or x.dtype)
 
 
-def gate_up_act(x, w_gate_up, n_ff: int, act: str = "silu"):
+def gate_up_act(x, w_gate_up, n_ff: int, act: str = "silu", bias=None):
     """w_gate_up rows: [gate(n_ff) | up(n_ff)]; returns act(gate) * up."""
     h = x.float() @ w_gate_up.float().t()
+    if bias is not None:
+        h = h + bias
     if w_gate_up.shape[0] == n_ff:            # un-gated FFN (squared ReLU): only the up projection exists
         return activation(h, act).to(x.dtype)
     g, u = h[:, :n_ff], h[:, n_ff:2 * n_ff]
@@ -169,9 +171,11 @@ def _gather_kv(cache, table_row, n_tokens):
 
 
 def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, window: int = 0, causal: bool = True,
-                    sinks=None, softcap: float = 0.0):
+                    sinks=None, softcap: float = 0.0, keep_first: int = 0, gate=None, out_scale: float = 1.0):
     """Varlen paged attention. q: [T, Hq, D]; sequence i owns query rows cu_q[i]:cu_q[i+1], which are the
-    LAST rows of its ctx_lens[i] cached tokens. Returns [T, Hq, Dv] (values may have a head size of their own)."""
+    LAST rows of its ctx_lens[i] cached tokens. Returns [T, Hq, Dv] (values may have a head size of their own).
+    ``keep_first``: first tokens that a window leaves visible; ``sinks`` [Hq]: exp(sink) joins the denominator; the output
+    times ``out_scale`` and, with ``gate`` [T, Hq], times its sigmoid."""
     T, Hq, D = q.shape
     Hkv = k_cache.shape[2]
     G = Hq // Hkv
@@ -195,7 +199,7 @@ def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, win
         if causal:
             mask &= kpos <= qpos
         if window > 0:
-            mask &= kpos > qpos - window
+            mask &= (kpos > qpos - window) | (kpos < keep_first)
         s = s.masked_fill(~mask[None], float("-inf"))
         if sinks is not None:
             s = torch.cat([s, sinks.float().view(Hq, 1, 1).expand(Hq, q1 - q0, 1)], dim=-1)
@@ -203,19 +207,23 @@ def paged_attention(q, k_cache, v_cache, block_table, ctx_lens, cu_q, scale, win
         else:
             p = torch.softmax(s, dim=-1)
         p = torch.nan_to_num(p)
-        out[q0:q1] = torch.einsum("hqk,khd->qhd", p, v).to(q.dtype)
+        o = torch.einsum("hqk,khd->qhd", p, v) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].float()).unsqueeze(2)
+        out[q0:q1] = o.to(q.dtype)
     return out
 
 
 def router_topk(logits, k: int, mode: str = "softmax", renorm: bool = True, route_scale: float = 1.0, bias=None,
                 n_group: int = 1, topk_group: int = 1, group_top: int = 2):
     """Returns (ids [T, k] int32, weights [T, k] float32); ties go to the lower expert id. ``renorm``: True holds the sum
-    of the chosen weights away from zero, "sum" divides by it as it is. ``softmax_bias``: selection
+    of the chosen weights away from zero, "sum" divides by it as it is. ``biased_softmax``: the bias joins the logits;
+    ``softmax_bias``: selection
     by softmax score + bias, like the sigmoid mode; ``group_top``: how many scores a group's rank sums up."""
     lf = logits.float()
     T, E = lf.shape
-    if mode == "softmax":
-        scores = torch.softmax(lf, dim=-1)
+    if mode in ("softmax", "biased_softmax"):
+        scores = torch.softmax(lf if mode == "softmax" else lf + bias.float(), dim=-1)
         sel = scores.clone()
     else:
         scores = torch.softmax(lf, dim=-1) if mode == "softmax_bias" else torch.sigmoid(lf)
@@ -471,6 +479,49 @@ def prenorm_step(x, terms, mult: float, norm_w, eps: float, w_offset: float, dty
     if terms:
         x = x + mult * sum(c * t.float() for t, c in terms)
     return x, None if norm_w is None else _norm32(x, norm_w, eps, w_offset).to(dtype)
+
+
+def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps: float, w_offset: float, rows=None):
+    """Behind layer ``i`` of a stack with parallel sublayers: X = x + sigmoid(g1 + b1) y1 + sigmoid(g2 + b2) (y2 + y2_b) (no
+    gate without ``g1``; ``y2`` may be None). With ``hist`` [layers + 1, T, H] float32 (the embedding output and the layers'
+    results) X becomes its entry i + 1 and the next input is the sum of coef[j] * hist[j] for j = 0 .. i + 1. Returns that
+    and its norm, of the given ``rows`` only when there are any."""
+    open_ = lambda g, b: 1.0 if g is None else torch.sigmoid(g.float() + b)                # noqa: E731
+    X = x + open_(g1, b1) * y1.float()
+    if y2 is not None:
+        f = y2.float() if y2_b is None else y2.float() + y2_b
+        X = X + open_(g2, b2) * f
+    if hist is not None:
+        hist[i + 1] = X
+        X = torch.einsum("j,jth->th", coef, hist[:i + 2])
+    if rows is not None:
+        X = X.index_select(0, rows)
+    return X, _norm32(X, norm_w, eps, w_offset).to(y1.dtype)
+
+
+def forget_scan(q, f, v, f_b, lower, state, cu_seq, slots, H: int, N: int, P: int, norm_w, eps: float, scale: float = 1.0,
+                write_state: bool = True):
+    """HGRN2: with F = lower + (1 - lower) sigmoid(f + f_b) per key channel, S_t = diag(F_t) S_(t-1) + (1 - F_t) v_t^T and
+    o_t = S_t^T silu(q_t); q, f [T, H * N], v [T, H * P], state [slots, H, P, N] float32. Returns the RMS norm of each
+    head's o times norm_w [P] times ``scale``, [T, H * P]."""
+    T = q.shape[0]
+    z = f.float() + f_b
+    keep = (lower + (1 - lower) * torch.sigmoid(z)).view(T, H, N)
+    write = ((1 - lower) * torch.sigmoid(-z)).view(T, H, N)
+    qf, vf = F.silu(q.float()).view(T, H, N), v.float().view(T, H, P)
+    out = torch.zeros(T, H, P)
+    for i in range(len(slots)):
+        t0, t1, s = int(cu_seq[i]), int(cu_seq[i + 1]), int(slots[i])
+        if t1 <= t0:
+            continue
+        S = state[s].clone()
+        for t in range(t0, t1):
+            S = S * keep[t].unsqueeze(1) + vf[t].unsqueeze(2) * write[t].unsqueeze(1)
+            out[t] = torch.einsum("hpn,hn->hp", S, qf[t])
+        if write_state:
+            state[s] = S
+    out = _norm32(out, norm_w, eps, 0.0) * scale
+    return out.reshape(T, H * P).to(q.dtype)
 
 
 def xielu(z, ab):

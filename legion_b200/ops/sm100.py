@@ -593,7 +593,7 @@ def _linear_fp8(x, w: "Fp8Weight", residual, out, dual: bool, n_feat: int):
     return out
 
 
-ROUTER_MODES = {"softmax": 0, "sigmoid": 1, "softmax_bias": 2}
+ROUTER_MODES = {"softmax": 0, "sigmoid": 1, "softmax_bias": 2, "biased_softmax": 3}
 RENORM = {False: 0, True: 1, "sum": 2}       # see config.MoeSpec.renorm
 GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
 
@@ -605,14 +605,14 @@ def tma_ok(*ts) -> bool:
 
 
 def sgemm(x, w, residual=None, out=None, out_dtype=None, dual: bool = False, n_ff: int = 0, act: str = "silu",
-          act_ab=None, unary: Optional[str] = None, tok_scale=None):
+          act_ab=None, unary: Optional[str] = None, tok_scale=None, bias=None):
     """x @ w^T in fp32 arithmetic on the FMA units: fp32 models and shapes outside the tcgen05 GEMM's alignment rules.
     ``dual``: act(x Wg^T) * (x Wu^T) with Wg = w[:n_ff], Wu = w[n_ff:]."""
     T, N = x.shape[0], (n_ff if dual else w.shape[0])
     if out is None:
         out = torch.empty(T, N, dtype=out_dtype or x.dtype, device=x.device)
     ext().sgemm(w, x, out, residual, tok_scale, None, N, dual, n_ff if dual else 0,
-                3 if act_ab is not None else GATE_ACTS[unary] if unary else GATE_ACTS[act] if dual else 0, None, None, None, None, 0, 0, T, act_ab)
+                3 if act_ab is not None else GATE_ACTS[unary] if unary else GATE_ACTS[act] if dual else 0, None, None, None, None, 0, 0, T, act_ab, bias)
     return out
 
 
@@ -663,11 +663,14 @@ def linear(x, w, residual=None, out=None, out_dtype=torch.bfloat16, split_k: Opt
     return out
 
 
-def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[int] = None, act: str = "silu"):
-    """act(x @ Wg^T) * (x @ Wu^T) with Wg = w_gate_up[:n_ff], Wu = w_gate_up[n_ff:] (GELU: bf16 weights only)."""
+def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[int] = None, act: str = "silu", bias=None):
+    """act(x @ Wg^T) * (x @ Wu^T) with Wg = w_gate_up[:n_ff], Wu = w_gate_up[n_ff:] (GELU and ``bias``, float32 [bg | bu] added
+    ahead of the activation: bf16 and fp32 weights only)."""
     C = ext()
     if isinstance(w_gate_up, torch.Tensor) and isinstance(x, torch.Tensor) and not tma_ok(x, w_gate_up):
-        return sgemm(x, w_gate_up, None, out, None, True, n_ff, act)
+        return sgemm(x, w_gate_up, None, out, None, True, n_ff, act, bias=bias)
+    if bias is not None and not isinstance(w_gate_up, torch.Tensor):
+        raise ValueError("biases run in the epilogue of bf16 and fp32 weights")
     if isinstance(x, Fp8Act) and not isinstance(w_gate_up, Fp8Weight):
         x = x.x
     T, K = x.shape
@@ -691,7 +694,7 @@ def gate_up_act(x, w_gate_up, n_ff: int, out=None, bn=None, split_k: Optional[in
     q = isinstance(w_gate_up, QWeight)
     C.wgemm(w_gate_up.codes if q else w_gate_up, x, out, None, None, None, n_ff, True, n_ff, bn, sk,
             ws.splitk if sk > 1 else None, ws.counters if sk > 1 else None, ws.status, None, None, None, None, 0, 0, T,
-            [], None, w_gate_up.scales if q else None, w_gate_up.gscale if q else None, 0, 0, GATE_ACTS[act])
+            [], None, w_gate_up.scales if q else None, w_gate_up.gscale if q else None, 0, 0, GATE_ACTS[act], bias=bias)
     return out
 
 
@@ -778,6 +781,39 @@ def prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, sc
     ws = Workspace.get(q.device)
     C.prefill_attn(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, causal, out, ws.status,
                    float(softcap))
+    return out
+
+
+def attention_ext(q, k_cache, v_cache, block_table, ctx_lens, cu_q, max_q_len, scale, window=0, keep_first=0, sink=None, gate=None,
+                  out_scale=1.0, out=None, n_splits=None, max_ctx=None):
+    """Paged causal attention with sinks, first tokens that stay visible behind the window, a gate per head, an output scale
+    and output rows that may lie apart ([T, heads * value head size])."""
+    C = ext()
+    T, Hq, _ = q.shape
+    Hkv, D = k_cache.shape[2], v_cache.shape[3]
+    if out is None:
+        out = torch.empty(T, Hq * D, dtype=q.dtype, device=q.device)
+    if T == 0:
+        return out
+    aligned = out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0
+    if not (attn_tc_ok(q, k_cache, v_cache) and aligned):
+        C.paged_attn_general(q, k_cache, v_cache, cu_q, ctx_lens, block_table, scale, window, out, 0.0, keep_first, sink, gate,
+                             out_scale)
+        return out
+    ws = Workspace.get(q.device)
+    if max_q_len > 1:
+        C.prefill_attn_ext(q, k_cache, v_cache, cu_q, ctx_lens, block_table, max_q_len, scale, window, out, ws.status, keep_first,
+                           sink, gate, out_scale)
+        return out
+    if n_splits is None:
+        span = max_ctx or block_table.shape[1] * k_cache.shape[1]
+        if window > 0:
+            span = min(span, window + 128 + -(-keep_first // 128) * 128)       # tiles that can hold visible tokens
+        n_splits = decode_splits(T, Hkv, (Hq // Hkv + 15) // 16, span, D)
+    o_part = ws.buf("dec_o", (T * Hq * n_splits * 2 * D,), torch.float32)
+    ml_part = ws.buf("dec_ml", (T * Hq * n_splits * 2 * 2,), torch.float32)
+    C.paged_decode_ext(q, k_cache, v_cache, block_table, ctx_lens, scale, window, n_splits, o_part, ml_part, out, ws.status,
+                       ws.counters, keep_first, sink, gate, out_scale)
     return out
 
 
@@ -1748,7 +1784,7 @@ def hyper_step(X, terms, mix, out_w, in_w, norm_w, eps, w_offset=0.0):
     return X, h
 
 
-def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None, dtype=None):
+def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None, dtype=None, x_out=None):
     """x (fp32 [T, H]) updated in place by mult * (sum of scale * tensor over ``terms``), and its norm in the activation type
     (``norm_w`` None: none); ``raw`` takes x itself in the activation type. ``start`` = (embedding table, ids or None, norm
     weight or None) begins a step. Returns (x, norm)."""
@@ -1757,7 +1793,7 @@ def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None
     if start is not None:
         table, ids, pre_w = start
         T = table.shape[0] if ids is None else ids.numel()
-        x, dtype = torch.empty(T, table.shape[1], dtype=torch.float32, device=table.device), table.dtype
+        x, dtype = torch.empty(T, table.shape[1], dtype=torch.float32, device=table.device) if x_out is None else x_out, table.dtype
     (y0, c0), (y1, c1) = (list(terms) + [(None, 0.0), (None, 0.0)])[:2]
     rows = 1
     if isinstance(y0, PendingCombine):
@@ -1766,6 +1802,22 @@ def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None
     if x.shape[0]:
         ext().prenorm_step(x_in, x, table, ids, pre_w, y0, c0 * mult, rows, y1, c1 * mult, norm_w, eps, w_offset, h, raw)
     return x, h
+
+
+def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset=0.0, rows=None):
+    """``reference.depth_step`` in one launch (``csrc/depth_step.cu``). ``x`` is updated in place unless it is an entry of
+    ``hist`` or only ``rows`` are wanted; the last layer's result is not kept."""
+    y2_rows = 1
+    if isinstance(y2, PendingCombine):
+        y2_rows, y2 = y2.rows, y2.y
+    n = x.shape[0] if rows is None else rows.numel()
+    own = rows is not None or (hist is not None and x.data_ptr() == hist.data_ptr())
+    x_out = torch.empty(n, x.shape[1], dtype=torch.float32, device=x.device) if own else x
+    h = torch.empty(n, x.shape[1], dtype=y1.dtype, device=x.device)
+    if n:
+        ext().depth_step(x, x_out, hist, i, hist is not None and i + 2 < hist.shape[0], y1, g1, b1, y2, y2_rows, g2, b2, y2_b, coef,
+                         norm_w, eps, w_offset, h, rows)
+    return x_out, h
 
 
 def qkv_conv_append(proj, in_b, conv_w, conv_state, cu_seq, state_slots, q_norm, k_norm, norm_over, eps, rot, layout, positions,
@@ -1885,6 +1937,35 @@ def linear_scan(q, k, v, state, cu_seq, slots, H, G, N, P, decay=None, silu_in=F
     if scratch is None or scratch.numel() < need:
         scratch = ws._cache["linear_chunk_scratch"] = torch.empty(need, dtype=torch.uint8, device=q.device)
     C.linear_chunk(*args, tab, n_chunks, scratch, ws.status)
+    return out
+
+
+def forget_scan(q, f, v, f_b, lower, state, cu_seq, slots, H, N, P, norm_w, eps, scale=1.0, write_state=True, max_len=None,
+                cu_host=None, out=None, chunked=None):
+    """HGRN2 state over the step's tokens with the norm per head behind it, state [slots, H, P, N] fp32 updated in place. bf16
+    prompts run in 128-token chunks on the tensor cores (``csrc/forget_scan_sm100.cu``), decode rows, short portions and fp32
+    on the streaming kernel (``csrc/forget_scan.cu``). ``chunked`` forces the choice."""
+    C = ext()
+    if out is None:
+        out = torch.empty(q.shape[0], H * P, dtype=q.dtype, device=q.device)
+    args = (q, f, v, f_b, lower, state, cu_seq, slots, H, N, P, norm_w, float(eps), float(scale), out, bool(write_state))
+    if chunked is None:
+        chunked = (q.dtype == torch.bfloat16 and cu_host is not None and (max_len or 0) >= LINEAR_CHUNK_MIN
+                   and C.forget_chunk_ok(N, P))
+    if not chunked:
+        C.forget_scan(*args, 0)
+        return out
+    ws = Workspace.get(q.device)
+    tab, n_chunks, short = _linear_chunk_tables(ws, cu_host if cu_host is not None else cu_seq.tolist(), q.device)
+    if short or n_chunks == 0:           # single tokens and the like beside prompts
+        C.forget_scan(*args, LINEAR_CHUNK_SHORT)
+    if n_chunks == 0:
+        return out
+    need = C.forget_chunk_scratch_bytes(n_chunks, H, N, P)
+    scratch = ws._cache.get("linear_chunk_scratch")
+    if scratch is None or scratch.numel() < need:
+        scratch = ws._cache["linear_chunk_scratch"] = torch.empty(need, dtype=torch.uint8, device=q.device)
+    C.forget_chunk(*args, tab, n_chunks, scratch, ws.status)
     return out
 
 
