@@ -19,6 +19,9 @@ Configurations (``--config``):
   14 Gurozen at 4B parameters in bf16 (24 layer runs: delta-rule layers with a decay per key channel and soft-capped
      attention in turn, dense and 32-expert feed-forward parts); compared with 7.
   15 the same at 13B (20 layer runs, 4096 columns); compared with 9.
+  16 Mananex at 4B parameters in bf16 (24 layers: windowed attention with sinks beside HGRN2, both sublayers on one norm,
+     depth averages, dense and 32-expert feed-forward parts); compared with 6.
+  17 the same at 13B (20 layers, 4096 columns); compared with 8.
 The ONE parsed number (``value``) is decode tokens/s at 16 users of the selected configuration; the other rows of
 the grid (1 and 64 users, 32K prefill) are under ``extra``.
 
@@ -112,6 +115,8 @@ CONFIGS = {
     13: dict(model="mla-7b", prompt_len=2048, weights="bf16", dtype="bf16"),
     14: dict(model="gurozen-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
     15: dict(model="gurozen-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    16: dict(model="mananex-4b", prompt_len=2048, weights="bf16", dtype="bf16"),
+    17: dict(model="mananex-13b", prompt_len=2048, weights="bf16", dtype="bf16"),
 }
 
 

@@ -827,7 +827,47 @@ def gurozen_13b() -> ModelConfig:
     return _gurozen(20, 4096, 32, 12288, 3072)
 
 
+def tiny_mananex() -> "ModelConfig":
+    """Mananex in miniature: windowed attention with a sink, kept first tokens and head gates beside an HGRN2 state in every
+    layer, both sublayers on one norm, gated residuals, depth averages, dense parts with biases, softmax-routed experts with a
+    logit bias, one layer without feed-forward part. Sizes differ from layer to layer."""
+    def mixer(heads, kv, dim, vdim, window, keep, rot, h, d, v, ls, rs):
+        return ParallelSpec(AttnSpec(heads, kv, dim, vdim, dim ** -0.5, window=window, keep_first=keep, qk_norm=False,
+                                     rot=RotarySpec(rot, 1e4), sink=True, gate="head"), Hgrn2Spec(h, d, v), ls, rs)
+    return ModelConfig(
+        arch="mananex", hidden=144, vocab=512, rms_eps=1e-5, norm_offset=1.0, tie_embeddings=True, parallel_sublayers=True,
+        residual_gate=True, depth_average=True,
+        layers=[LayerSpec(mixer(6, 2, 32, 48, 40, 3, 24, 3, 40, 56, 0.7, 0.8), DenseSpec(200, bias=True)),
+                LayerSpec(mixer(4, 4, 48, 24, 75, 5, 48, 5, 24, 32, 1.1, 0.5), MoeSpec(10, 3, 56, router="biased_softmax")),
+                LayerSpec(mixer(2, 1, 64, 64, 130, 1, 16, 2, 64, 40, 0.4, 1.2), None),
+                LayerSpec(mixer(3, 1, 40, 32, 17, 2, 8, 1, 72, 80, 0.9, 0.6), MoeSpec(6, 2, 40, router="biased_softmax"))])
+
+
+def _mananex(n_layer: int, hidden: int, heads: int, ff: int, expert_ff: int) -> ModelConfig:
+    """Attention of ``heads`` query heads with window 1024 beside as many HGRN2 heads, dense and 32-expert feed-forward parts
+    in turn."""
+    layers = []
+    for il in range(n_layer):
+        mixer = ParallelSpec(AttnSpec(heads, heads // 4, 128, 128, 128 ** -0.5, window=1024, keep_first=4, qk_norm=False,
+                                      rot=RotarySpec(64, 1e6), sink=True, gate="head"), Hgrn2Spec(heads, 128, 128), 0.5, 0.5)
+        layers.append(LayerSpec(mixer, MoeSpec(32, 4, expert_ff, router="biased_softmax") if il % 2 else DenseSpec(ff, bias=True)))
+    return ModelConfig(arch="mananex", hidden=hidden, vocab=65536, rms_eps=1e-5, norm_offset=1.0, tie_embeddings=True,
+                       parallel_sublayers=True, residual_gate=True, depth_average=True, layers=layers)
+
+
+def mananex_4b() -> ModelConfig:
+    """Mananex with layers the size of a small production model (random weights; speed measurements)."""
+    return _mananex(24, 2048, 16, 6144, 1024)
+
+
+def mananex_13b() -> ModelConfig:
+    return _mananex(20, 4096, 32, 12288, 2048)
+
+
 PRESETS = {
+    "tiny-mananex": tiny_mananex,
+    "mananex-4b": mananex_4b,
+    "mananex-13b": mananex_13b,
     "tiny-gurozen": tiny_gurozen,
     "gurozen-4b": gurozen_4b,
     "gurozen-13b": gurozen_13b,

@@ -24,7 +24,7 @@ BUCKETS = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256)
 
 class _Entry:
     __slots__ = ("graph", "B", "W", "pack_h", "pack_d", "batch", "picks", "picks_h", "logits", "n_ints", "arange",
-                 "bt_key", "pack_np", "all_picks", "all_picks_h", "logits_local")
+                 "bt_key", "pack_np", "all_picks", "all_picks_h", "logits_local", "parts")
 
 
 class DecodeGraphs:
@@ -124,6 +124,7 @@ class DecodeGraphs:
                     write_state=True, cu_q_host=list(range(n + 1)),
                     decode_splits=ops.sm100.decode_splits(n, Hkv, (G + 15) // 16, eng.cfg.ctx_size)), lo, hi))
             e.logits = torch.empty(B, eng.mcfg.vocab, dtype=torch.float32, device=dev)
+        e.parts = parts           # the lanes' own tensors (sequence bounds) live as long as the graph that reads them
         WS = ops.sm100.Workspace
 
         def run_lane(i):
