@@ -627,6 +627,95 @@ def bench_delta(rows):
             del up, dn
 
 
+def bench_forget(rows):
+    """Mananex: HGRN2 state, rotation and append, windowed attention with sinks, kept first tokens and head gates, gated residual
+    with depth average, biased gate / up and routing, each beside the like kernel of the other families. frac_hbm: bytes that
+    must move once; frac_tc: FLOPs over measured cuBLAS bf16 (attention, products)."""
+    from legion_b200.ops import sm100
+    hbm, tf, src = peaks()
+    f = lambda *s: (torch.randn(*s, device="cuda") * 0.5).bfloat16()                 # noqa: E731
+
+    def row(kernel, n, L, ms, byts=None, flops=None):
+        r = dict(kernel=kernel, n_seq=n, L=L, us=round(ms * 1e3, 2), peaks=src)
+        if byts:
+            r["frac_hbm"] = round(byts / ms / 1e6 / hbm, 3)
+        if flops:
+            r["frac_tc"] = round(flops / ms / 1e9 / tf, 3)
+        rows.append(r)
+        print(r, flush=True)
+    H, G, D, W, window = 16, 4, 128, 2048, 1024
+    one, zero = torch.ones(H * D, device="cuda"), torch.zeros(H * D, device="cuda")
+    for n, L in (CASE["attn"] or ((1, 1), (16, 1), (64, 1), (1, 8192), (4, 2048))):
+        T = n * L
+        cu, cu_host = torch.arange(0, T + 1, L, device="cuda", dtype=torch.int32), list(range(0, T + 1, L))
+        slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        tm = timeit if L > 1 else timeit_graph
+        # HGRN2, 16 heads of 128 x 128
+        proj, st, low = f(T, 4 * H * D), torch.zeros(n, H, D, D, device="cuda"), torch.rand(H * D, device="cuda") * 0.9
+        q, k, v, g = (proj[:, i * H * D:(i + 1) * H * D] for i in range(4))
+        byts = T * 4 * H * D * 2 + st.numel() * 8
+        row("forget_scan 16x128x128 (norm included)", n, L, tm(lambda: sm100.forget_scan(
+            q, k, v, one, low, st, cu, slots, H, D, D, one[:D], 1e-6, max_len=L, cu_host=cu_host)), byts)
+        dec = torch.full((H,), 0.99, device="cuda")
+        scan = lambda: sm100.linear_scan(q, k, v, st, cu, slots, H, H, D, D, decay=dec, silu_in=True, max_len=L, cu_host=cu_host)  # noqa: E731
+        row("linear_scan constant decay, same size", n, L, tm(scan), byts)
+        o = scan()
+        row("group_norm_gate 2048 behind it", n, L, tm(lambda: sm100.group_norm_gate(o, g, one, 1e-5)), T * H * D * 6)
+        cw, hist = torch.randn(4, 3 * H * D, device="cuda"), torch.zeros(n, 3, 3 * H * D, device="cuda")
+        args = (f(T, 3 * H * D), cw, hist, k, -one[:H], zero, f(T, H), st, cu, slots, H, H, D, D)
+        if L == 1:
+            row("channel_delta_decode, same size (convolution, norm and gate included)", n, L,
+                tm(lambda: sm100.channel_delta_decode(*args, g, one[:D], 1e-6)), byts + hist.numel() * 8)
+        else:
+            row("channel_delta, same size (convolution included)", n, L, tm(lambda: sm100.channel_delta(*args, max_len=L)), byts)
+        # attention: 16 query heads over 4 kv heads of 128, window 1024
+        page, ctx = 64, max(L, 2048)
+        nb = ctx // page
+        kc, vc = f(n * nb, page, G, D), f(n * nb, page, G, D)
+        bt = torch.arange(n * nb, device="cuda", dtype=torch.int32).view(n, nb)
+        pos = torch.arange(ctx - L, ctx, device="cuda", dtype=torch.int32).repeat(n)
+        cells = (bt.long()[:, :, None] * page + torch.arange(page, device="cuda")).view(n, -1)[:, ctx - L:].reshape(-1).contiguous()
+        qkv, cs = f(T, (H + 2 * G) * D), torch.randn(ctx, 64, device="cuda")
+        row("rotation and append 16/4 heads of 128", n, L, tm(lambda: sm100.qkv_conv_append(
+            qkv, None, None, None, cu, slots, None, None, "head", 1e-6, cs, "pairs", pos, cells, kc, vc, H, max_len=L)), T * qkv.shape[1] * 4)
+        row("qk_norm_rope_append, same size", n, L, tm(lambda: sm100.qk_norm_rope_append(
+            qkv, H, G, D, one[:D], one[:D], 1e-6, 0.0, cs, 64, pos, cells, kc, vc)), T * qkv.shape[1] * 4)
+        qq, cl, gate = f(T, H, D), torch.full((n,), ctx, device="cuda", dtype=torch.int32), f(T, H)
+        ext = lambda: sm100.attention_ext(qq, kc, vc, bt, cl, cu, L, D ** -0.5, window, 4, zero[:H], gate, 0.5, max_ctx=ctx)   # noqa: E731
+        if L == 1:
+            kv = n * min(ctx, window) * G * D * 4
+            row(f"windowed attention, sink and head gate, decode at {ctx}", n, L, tm(ext), kv)
+            row(f"windowed attention, decode at {ctx}", n, L, tm(lambda: sm100.paged_decode(
+                qq, kc, vc, bt, cl, D ** -0.5, window, max_ctx=ctx)), kv)
+        else:
+            flops = n * (L - window / 2) * window * H * D * 4
+            row("windowed attention, sink and head gate, prompt", n, L, tm(ext), flops=flops)
+            row("windowed attention, prompt", n, L, tm(lambda: sm100.prefill_attn(qq, kc, vc, cu, cl, bt, L, D ** -0.5, window)), flops=flops)
+        # residual with gates and depth average behind layers 0, 11 and 22 of 24
+        hist = torch.randn(25, T, W, device="cuda") if T <= 64 else torch.zeros(25, T, W, device="cuda")
+        x, y, p2, nw = torch.randn(T, W, device="cuda"), f(T, W), f(T, 2 * W), torch.zeros(W, device="cuda")
+        for i in (0, 11, 22):
+            row(f"depth_step 2048, {i + 2} terms", n, L, tm(lambda: sm100.depth_step(
+                x, hist, i, y, p2[:, :W], nw, y, p2[:, W:], nw, nw, one[:i + 2], nw, 1e-6, 1.0)), T * W * (4 * (i + 4) + 10))
+        del hist
+        X, mix = torch.randn(T, 4, W, device="cuda"), torch.eye(4, device="cuda")
+        row("hyper_step 4x2048", n, L, tm(lambda: sm100.hyper_step(X, [(y, 1.0)], mix, one[:4], one[:4], nw, 1e-5, 1.0)), T * W * 36)
+        row("prenorm_step 2048", n, L, tm(lambda: sm100.prenorm_step(x, [(y, 1.0)], 0.5, nw, 1e-6, 1.0, dtype=torch.bfloat16)), T * W * 12)
+        # feed-forward parts
+        gu, ff = f(2 * 6144, W), 6144
+        gb = torch.zeros(2 * ff, device="cuda")
+        for name, b in (("gate / up 6144 with biases", gb), ("gate / up 6144", None)):
+            row(name, n, L, tm(lambda: sm100.gate_up_act(y, gu, ff, bias=b)), gu.numel() * 2 + T * (W + ff) * 2, 2.0 * T * gu.numel())
+        rw, up, dn = f(32, W), f(32, 2 * 1024, W), f(32, W, 1024)
+        rb = torch.zeros(32, device="cuda")
+        seen = 32 * (1 - (1 - 4 / 32) ** T)
+        for name, mode, b in (("router with logit bias + experts", "biased_softmax", rb), ("router + experts", "softmax", None)):
+            def experts():
+                r = sm100.router(y, rw, 4, mode, True, 1.0, b, n_local=32)
+                return sm100.moe_experts(y, r.ids, r.wts, up, dn, 1024, 0, routing=r, defer_combine="pairs")
+            row(name, n, L, tm(experts), seen * (up[0].numel() + dn[0].numel()) * 2 + T * W * 12, 8.0 * T * (up[0].numel() + dn[0].numel()))
+
+
 class Batch:
     """The fields of a step that a planner reads."""
 
@@ -816,7 +905,7 @@ def main(argv=None):
     if a.gemm:
         CASE["gemm"] = [tuple(int(y) for y in x.split("x")) for x in a.gemm.split(",")]
     rows = []
-    table = {"delta": bench_delta, "resid": bench_resid, "diag": bench_diag, "latent": bench_latent, "linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
+    table = {"forget": bench_forget, "delta": bench_delta, "resid": bench_resid, "diag": bench_diag, "latent": bench_latent, "linear": bench_linear, "hyper": bench_hyper, "attn_sizes": bench_attn_sizes, "moe_nv4": bench_moe_nv4, "gdn": bench_gdn, "moe_fp8": bench_moe_fp8, "mla": bench_mla, "moe_nvfp4": bench_moe_nvfp4, "layer_parts": bench_layer_parts, "decode_pages": bench_decode_pages, "gemm": bench_gemm, "moe": bench_moe, "decode_attn": bench_decode_attn, "prefill_attn": bench_prefill_attn}
     for name in a.only.split(","):
         table[name](rows)
     from legion_b200.ops.sm100 import Workspace

@@ -27,7 +27,7 @@ NVCC_FLAGS = [
 ]
 # sources whose arithmetic serves fp32 models too: exact division, square root and exponentials, no flush to zero
 PRECISE = {"hyper", "sgemm", "attn_general", "linear_scan", "resid_step", "latent_attn", "diag_scan", "logits", "conv_any",
-           "channel_delta", "channel_delta_mma", "qkv_conv", "depth_step", "forget_scan", "forget_scan_sm100"}
+           "channel_delta", "channel_delta_mma", "qkv_conv", "depth_step", "forget_scan"}
 
 
 def _cu_flags(src: Path, verbose: bool) -> list[str]:

@@ -11,13 +11,14 @@
 // are read) and, inside blocks of 8 tokens, from inner products on FMA units. All products of gates run forward in time, each
 // factor at most 1: no quotient and no logarithm of a gate appears, and gates near 0 and near 1 keep their accuracy.
 //
-// A thread owns two neighbouring channels of 16 tokens; what a level or the carry needs from other segments of the same channels
-// are their total products, shared once. The state between chunks stays fp32; whatever enters a contraction beside the bf16
+// A thread owns two neighbouring channels of a segment of tokens; what a level or the carry needs from other segments of the same
+// channels are their total products, shared once. The state between chunks stays fp32; whatever enters a contraction beside the bf16
 // projections and the activated queries (decayed writes, A, the state) is split into two bf16 terms, so it contributes with
 // about 16 bits. The norm per head ends the OUTPUT kernel.
 #include "act_type.cuh"
 #include "common.cuh"
 #include "layers.h"
+#include "state_cols.cuh"
 
 namespace lb {
 namespace {
@@ -26,14 +27,6 @@ constexpr int C = 128;                    // tokens per chunk
 constexpr int HALF = C * 128;             // bytes of one 64-column half of a 128-row tile
 constexpr int SEG = 16, SEGS = C / SEG;   // tokens of a thread, segments of a chunk
 
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
-      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
-      "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // A operand (bf16 pairs in 32-bit cells, row = lane) from tensor memory
 __device__ __forceinline__ void umma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc,
@@ -55,7 +48,12 @@ struct ForgetChunkArgs {
   int* status;
 };
 
-__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float sigmoid_fast(float z) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return r;
+}
 
 __device__ __forceinline__ float2 bf2(uint32_t u) {
   return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
@@ -290,85 +288,51 @@ __global__ void __launch_bounds__(256) forget_carry_kernel(const ForgetChunkArgs
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// OUTPUT
+// OUTPUT: a thread owns two neighbouring channels of 8 tokens, with -(1 - F) in registers: a product moves on by one fused
+// multiply-add. The code of a level is the same for all of them (a loop, so that it stays in the instruction cache).
 // ---------------------------------------------------------------------------------------------------------------
-// One level: halves of S tokens. Rows of a right half get their decayed queries in the q tile, rows of a left half their
-// decayed writes in the k tiles; the other rows of either tile are not read back.
-template <int S, int PAIRS>
-__device__ __forceinline__ void build_level(const float2 (&q)[SEG], const float2 (&w)[SEG], const float2* g_s, int p, int seg,
-                                            uint8_t* q_s, uint8_t* kh_s, uint8_t* kl_s) {
-  auto put_q = [&](int i, float2 m) {
-    *reinterpret_cast<uint32_t*>(q_s + pair_off(seg * SEG + i, p)) = pack_bf16x2(q[i].x * m.x, q[i].y * m.y);
-  };
-  auto put_k = [&](int i, float2 m) {
-    const int off = pair_off(seg * SEG + i, p);
-    uint32_t hi, lo;
-    split2(w[i].x * m.x, w[i].y * m.y, hi, lo);
-    *reinterpret_cast<uint32_t*>(kh_s + off) = hi;
-    *reinterpret_cast<uint32_t*>(kl_s + off) = lo;
-  };
-  if constexpr (S >= SEG) {
-    constexpr int HS = S / SEG;             // segments of a half
-    const int at = seg % HS, half0 = seg - at;
-    if ((seg / HS) & 1) {
-      float2 m = totals<PAIRS>(g_s, p, half0, seg);
-#pragma unroll
-      for (int i = 0; i < SEG; ++i) {
-        m.x *= 1.f - w[i].x;
-        m.y *= 1.f - w[i].y;
-        put_q(i, m);
-      }
-    } else {
-      float2 m = totals<PAIRS>(g_s, p, seg + 1, half0 + HS);
-#pragma unroll
-      for (int i = SEG - 1; i >= 0; --i) {
-        put_k(i, m);
-        m.x *= 1.f - w[i].x;
-        m.y *= 1.f - w[i].y;
-      }
-    }
-  } else {
-#pragma unroll
-    for (int b = 0; b < SEG; b += 2 * S) {
-      float2 m = make_float2(1.f, 1.f);
-#pragma unroll
-      for (int i = b + S - 1; i >= b; --i) {
-        put_k(i, m);
-        m.x *= 1.f - w[i].x;
-        m.y *= 1.f - w[i].y;
-      }
-      m = make_float2(1.f, 1.f);
-#pragma unroll
-      for (int i = b + S; i < b + 2 * S; ++i) {
-        m.x *= 1.f - w[i].x;
-        m.y *= 1.f - w[i].y;
-        put_q(i, m);
-      }
-    }
-  }
+constexpr int OSEG = 8, OSEGS = C / OSEG;
+constexpr int imax(int a, int b) { return a > b ? a : b; }
+
+// Levels: q tile | high parts | remainders. Beside them first 1 - F (fp32) and the queries' projections (bf16) by token for the blocks of 8,
+// later the values and the state in front of the chunk.
+template <int NH, int PH>
+struct OutSmem {
+  static constexpr int TILES = 3 * NH * HALF;
+  static constexpr int SHALF = PH * 64 * 128;                 // bytes of one 64-column half of the state tile
+  static constexpr int SHARE = imax(PH * HALF + 2 * NH * SHALF, NH * 64 * C * 4 + NH * HALF);
+  static constexpr int BYTES = TILES + SHARE + OSEGS * NH * 32 * 8 + C * 8 * 4 + NH * 4 * C * 4 + 1024 + 128;
+  static_assert(BYTES <= 227 * 1024, "shared memory budget");
+};
+
+__device__ __forceinline__ void tmem_ld8(uint32_t taddr, uint32_t (&r)[8]) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+               : "r"(taddr) : "memory");
+}
+__device__ __forceinline__ void tmem_st4(uint32_t taddr, const uint32_t (&r)[4]) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x4.b32 [%0], {%1, %2, %3, %4};"
+               ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
 }
 
 template <int NH, int PH>
-constexpr int output_smem() {
-  return (3 * NH + PH) * HALF + 2 * NH * (PH * 64 * 128) + SEGS * NH * 32 * 8 + NH * C * 8 * 4 + 2 * NH * C * 4 + 1024 + 128;
-}
-
-template <int NH, int PH>
-__global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const ForgetChunkArgs a) {
-  constexpr int NT = NH * 256, PAIRS = NH * 32, WGS = NT / 128;
-  constexpr int PW = PH * 64;
-  constexpr int SHALF = PW * 128;           // bytes of one 64-column half of the state tile
+__global__ void __launch_bounds__(NH * 512, 1) forget_output_kernel(const ForgetChunkArgs a) {
+  using Sm = OutSmem<NH, PH>;
+  constexpr int NT = NH * 512, PAIRS = NH * 32, WGS = NT / 128, PW = PH * 64, SHALF = Sm::SHALF;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* q_s = smem;
   uint8_t* kh_s = q_s + NH * HALF;
   uint8_t* kl_s = kh_s + NH * HALF;
-  uint8_t* v_s = kl_s + NH * HALF;
+  uint8_t* share = smem + Sm::TILES;
+  float* nw_s = reinterpret_cast<float*>(share);                         // [C][NH * 64] -(1 - F)
+  uint32_t* qb_s = reinterpret_cast<uint32_t*>(share + NH * 64 * C * 4); // [C][PAIRS] queries before silu, pairs of bf16
+  uint8_t* v_s = share;
   uint8_t* sh_s = v_s + PH * HALF;
   uint8_t* sl_s = sh_s + NH * SHALF;
-  float2* g_s = reinterpret_cast<float2*>(sl_s + NH * SHALF);            // [SEGS][PAIRS] totals
-  float* diag_s = reinterpret_cast<float*>(g_s + SEGS * PAIRS);          // [NH][C][8] A inside blocks of 8, a plane per 64 channels
-  float* red_s = diag_s + NH * C * 8;                                    // [WGS][C] sums of squares
+  uint64_t* g_s = reinterpret_cast<uint64_t*>(share + Sm::SHARE);        // [OSEGS][PAIRS] products of the segments' gates
+  float* diag_s = reinterpret_cast<float*>(g_s + OSEGS * PAIRS);         // [C][8] A inside blocks of 8
+  float* red_s = diag_s + C * 8;                                         // [WGS][C] sums of squares
   uint64_t* bars = reinterpret_cast<uint64_t*>(red_s + WGS * C);         // [4] levels, [1] output
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -388,30 +352,102 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
   griddep_wait();
   griddep_launch();
   const int t0 = a.chunk_t0[chunk], nval = a.chunk_n[chunk];
-  float2 q[SEG], w[SEG];
+  uint64_t q[OSEG], nw[OSEG];
   {
-    const auto* qp = static_cast<const __nv_bfloat16*>(L.q) + long(t0 + seg * SEG) * L.ldq + long(h) * L.N;
-    uint32_t raw[SEG];
+    const long row0 = t0 + seg * OSEG;
+    const auto* qp = static_cast<const __nv_bfloat16*>(L.q) + row0 * L.ldq + long(h) * L.N;
+    const auto* fp = static_cast<const __nv_bfloat16*>(L.f) + row0 * L.ldf + long(h) * L.N;
+    uint32_t rq[OSEG], rf[OSEG];
 #pragma unroll
-    for (int i = 0; i < SEG; ++i) raw[i] = seg * SEG + i < nval ? ld_pair(qp + i * L.ldq, 2 * p, L.N, a.pair_q) : 0u;
-    load_writes(a, h, t0, nval, p, seg, w);
-#pragma unroll
-    for (int i = 0; i < SEG; ++i) {
-      const float2 z = bf2(raw[i]);
-      q[i] = make_float2(z.x * sigmoid_fast(z.x), z.y * sigmoid_fast(z.y));
+    for (int i = 0; i < OSEG; ++i) {
+      const bool in = seg * OSEG + i < nval;
+      rq[i] = in ? ld_pair(qp + i * L.ldq, 2 * p, L.N, a.pair_q) : 0u;
+      rf[i] = in ? ld_pair(fp + i * L.ldf, 2 * p, L.N, a.pair_f) : 0u;
     }
+    float2 b = make_float2(0.f, 0.f), open = b;               // bias, 1 - lower (0 past the head's channels)
+    if (2 * p < L.N) { b.x = L.f_b[h * L.N + 2 * p]; open.x = 1.f - L.lower[h * L.N + 2 * p]; }
+    if (2 * p + 1 < L.N) { b.y = L.f_b[h * L.N + 2 * p + 1]; open.y = 1.f - L.lower[h * L.N + 2 * p + 1]; }
+    uint64_t g = p2(1.f, 1.f);
+#pragma unroll
+    for (int i = 0; i < OSEG; ++i) {
+      const int t = seg * OSEG + i;
+      const float2 z = bf2(rq[i]), e = bf2(rf[i]);
+      const float qx = z.x * sigmoid_fast(z.x), qy = z.y * sigmoid_fast(z.y);
+      q[i] = p2(qx, qy);
+      nw[i] = t < nval ? p2(-open.x * sigmoid_fast(-(e.x + b.x)), -open.y * sigmoid_fast(-(e.y + b.y))) : 0ull;
+      g = fma2(nw[i], g, g);
+      *reinterpret_cast<uint64_t*>(nw_s + t * (NH * 64) + 2 * p) = nw[i];
+      qb_s[t * PAIRS + p] = rq[i];
+    }
+    g_s[seg * PAIRS + p] = g;
   }
-  g_s[seg * PAIRS + p] = total_of(w);
   __syncthreads();
   const uint32_t tmem = *tmem_slot;
   // high parts and remainders of A (bf16 pairs), two level accumulators, the output
   const uint32_t tm_hi = tmem, tm_lo = tmem + 64, tm_d = tmem + 128, tm_o = tmem + 384;
-  const uint32_t qa = smem_u32(q_s), kh = smem_u32(kh_s), kl = smem_u32(kl_s), va = smem_u32(v_s);
+  const uint32_t qa = smem_u32(q_s), kh = smem_u32(kh_s), kl = smem_u32(kl_s);
   const int wq = warp & 3, wg = warp >> 2;                // 32 tokens (rows of tensor memory), warpgroup
   const uint32_t lane_off = uint32_t(wq * 32) << 16;
+  const uint32_t tile0 = (p >> 5) * HALF + seg * OSEG * 128 + ((p & 31) >> 2) * 16 + (p & 3) * 4;   // token 0 of the segment
+  auto at = [&](int i) { return (tile0 ^ (i << 4)) + i * 128; };          // (swizzle: 16-byte chunk xor token mod 8)
+  auto product = [&](int lo, int hi) {                    // of the gates of segments lo .. hi - 1
+    uint64_t m = p2(1.f, 1.f);
+#pragma unroll 1
+    for (int s = lo; s < hi; ++s) m = mul2(m, g_s[s * PAIRS + p]);
+    return m;
+  };
+  auto put_queries = [&](uint64_t m) {                    // decayed from the front of the segment on, m in front of it
+#pragma unroll
+    for (int i = 0; i < OSEG; ++i) {
+      m = fma2(nw[i], m, m);
+      float x, y;
+      u2(mul2(q[i], m), x, y);
+      *reinterpret_cast<uint32_t*>(q_s + at(i)) = pack_bf16x2(x, y);
+    }
+  };
   bool ok = true;
-  // products of a level, once all its rows are in place
-  auto level_mma = [&](int lv) {
+  auto wait = [&](int bar, int site) {                    // one warp polls; the barrier behind it is the others' wait
+    if (warp == 0) {
+      if (!mbar_wait(&bars[bar], 0, abort_flag)) {
+        *abort_flag = 1;
+        atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | site);
+      }
+      __syncwarp();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    ok = ok && !*abort_flag;
+  };
+  // eight columns of A from column c on: high parts and remainders into tensor memory
+  auto store8 = [&](int c, const float (&x)[8]) {
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) split2(x[2 * j], x[2 * j + 1], hi[j], lo[j]);
+    tmem_st4(tm_hi + lane_off + c / 2, hi);
+    tmem_st4(tm_lo + lane_off + c / 2, lo);
+  };
+
+#pragma unroll 1
+  for (int lv = 0; lv < 4; ++lv) {
+    // halves of 8, 4, 2, 1 segments: rows of a right half get their decayed queries in the q tile, rows of a left half their
+    // decayed writes in the k tiles; the other rows of either tile are not read back
+    const int hs = 8 >> lv, half0 = seg & ~(hs - 1);
+    if (seg & hs) {
+      put_queries(product(half0, seg));
+    } else {
+      uint64_t m = product(seg + 1, half0 + hs);
+#pragma unroll
+      for (int i = OSEG - 1; i >= 0; --i) {
+        float x, y;
+        uint32_t hi, lo;
+        u2(mul2(nw[i], m), x, y);
+        split2(-x, -y, hi, lo);
+        *reinterpret_cast<uint32_t*>(kh_s + at(i)) = hi;
+        *reinterpret_cast<uint32_t*>(kl_s + at(i)) = lo;
+        m = fma2(nw[i], m, m);
+      }
+    }
     fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
@@ -428,177 +464,134 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
       umma_commit(&bars[lv]);
     }
     __syncwarp();
-  };
-  auto level_wait = [&](int lv) {
-    if (!mbar_wait(&bars[lv], 0, abort_flag)) {
-      *abort_flag = 1;
-      atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_FORGET_LEVEL);
-      ok = false;
-    }
-    __syncwarp();
-    tc_fence_after();
-  };
-  // 32 columns of A (group g) of the warp's rows, high parts and remainders, into tensor memory
-  auto store_group = [&](int g, const float (&x)[32]) {
-    uint32_t hi[16], lo[16];
+    if (lv == 0) {
+      // blocks of 8 tokens: a warp takes the tokens of one place in several blocks, CG lanes share a token's channels
+      constexpr int CG = NH * 4, TPW = 32 / CG;
+      const int i8 = warp & 7, t = ((warp >> 3) * TPW + lane / CG) * 8 + i8, cg = lane % CG;
+      uint64_t qv[8], D[8];
 #pragma unroll
-    for (int j = 0; j < 16; ++j) split2(x[2 * j], x[2 * j + 1], hi[j], lo[j]);
-    tmem_st16(tm_hi + lane_off + g * 16, hi);
-    tmem_st16(tm_lo + lane_off + g * 16, lo);
-  };
-  auto copy_group = [&](int g, int lv) {
-    uint32_t r[32];
-    float x[32];
-    tmem_ld32(tm_d + (lv & 1) * 128 + lane_off + g * 32, r);
-    tmem_ld_wait();
-#pragma unroll
-    for (int j = 0; j < 32; ++j) x[j] = __uint_as_float(r[j]);
-    store_group(g, x);
-  };
-  const int diag_wg = wq % WGS;                           // the warpgroup that puts this warp's diagonal group together
-
-  build_level<64, PAIRS>(q, w, g_s, p, seg, q_s, kh_s, kl_s);
-  level_mma(0);
-  load_values<PH, NT>(a, h, t0, nval, v_s);
-  // blocks of 8 tokens: A_ij summed over the thread's channels, then over the warp's
-#pragma unroll
-  for (int b = 0; b < SEG; b += 8) {
-    float2 c[8];                                          // decayed writes of the block's tokens, as token i sees them
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      float s[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        s[j] = 0.f;
-        if (j < i) {
-          c[j].x *= 1.f - w[b + i].x;
-          c[j].y *= 1.f - w[b + i].y;
-        }
-        if (j == i) c[j] = w[b + i];
-        if (j <= i) s[j] = fmaf(q[b + i].x, c[j].x, q[b + i].y * c[j].y);
+      for (int k = 0; k < 4; ++k) {
+        const uint2 u = *reinterpret_cast<const uint2*>(qb_s + t * PAIRS + 2 * (cg + CG * k));
+        const float2 x = bf2(u.x), y = bf2(u.y);
+        qv[2 * k] = p2(x.x * sigmoid_fast(x.x), x.y * sigmoid_fast(x.y));
+        qv[2 * k + 1] = p2(y.x * sigmoid_fast(y.x), y.y * sigmoid_fast(y.y));
+        D[2 * k] = D[2 * k + 1] = p2(1.f, 1.f);
       }
+#pragma unroll 1
+      for (int j = i8; j >= 0; --j) {
+        const float* wr = nw_s + (t - i8 + j) * (NH * 64) + 4 * cg;
+        uint64_t acc = 0ull;
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1) {                   // lane l gets sum l & 7 of four lanes each
-        const bool up = lane & o;
-#pragma unroll
-        for (int j = 0; j < o; ++j) {
-          const float send = up ? s[j] : s[j + o], keep = up ? s[j + o] : s[j];
-          s[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        for (int k = 0; k < 4; ++k) {
+          uint64_t w0, w1;
+          ld4(wr + 4 * CG * k, w0, w1);
+          acc = fma2(mul2(w0, D[2 * k]), qv[2 * k], acc);
+          acc = fma2(mul2(w1, D[2 * k + 1]), qv[2 * k + 1], acc);
+          D[2 * k] = fma2(w0, D[2 * k], D[2 * k]);
+          D[2 * k + 1] = fma2(w1, D[2 * k + 1], D[2 * k + 1]);
         }
+        float x, y;
+        u2(acc, x, y);
+        x += y;
+#pragma unroll
+        for (int o = CG / 2; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+        if (cg == 0) diag_s[t * 8 + j] = -x;
       }
-      s[0] += __shfl_xor_sync(0xffffffffu, s[0], 8);
-      s[0] += __shfl_xor_sync(0xffffffffu, s[0], 16);
-      if (lane < 8) diag_s[((NH == 2 ? (warp & 1) : 0) * C + seg * SEG + b + i) * 8 + lane] = s[0];
-    }
-  }
-  level_wait(0);
-  __syncthreads();                                        // the tiles are free again
-  build_level<32, PAIRS>(q, w, g_s, p, seg, q_s, kh_s, kl_s);
-  level_mma(1);
-  // groups of columns 0 .. 63 for the rows of the right half; what lies above the diagonal is zero
+    } else if (lv == 1) {
+      load_values<PH, NT>(a, h, t0, nval, v_s);           // (1 - F and the queries by token have been read)
+#pragma unroll 1
+      for (int c = wg * 16; c < C; c += WGS * 16)
+#pragma unroll 1
+        for (int e = c; e < c + 16; e += 8) {
+          float x[8];
+          if (wq >= 2 && c < 64) {                        // rows of the right half, columns of the left one
+            uint32_t r[8];
+            tmem_ld8(tm_d + lane_off + e, r);
+            tmem_ld_wait();
 #pragma unroll
-  for (int g = 0; g < 4; ++g) {
-    if (g % WGS != wg) continue;
-    if (g < 2 && wq >= 2) copy_group(g, 0);
-    if (g > wq) {
-      const float zero[32] = {};
-      store_group(g, zero);
-    }
-  }
-  level_wait(1);
-  __syncthreads();
-  build_level<16, PAIRS>(q, w, g_s, p, seg, q_s, kh_s, kl_s);
-  level_mma(2);
-  if ((wq == 1 && wg == 0) || (wq == 3 && wg == 2 % WGS)) copy_group(wq - 1, 1);
-  // the state in front of the chunk, high parts and remainders
-  {
-    const float* S0 = a.dS + (long(chunk) * L.H + h) * L.P * L.N;
-    constexpr int IT = PW * NH * 8 / NT;
-    auto put = [&](int row, int c8, const float (&v)[8]) {
-      const int off = (c8 >> 3) * SHALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4);
-      uint4 hi, lo;
-      split2(v[0], v[1], hi.x, lo.x);
-      split2(v[2], v[3], hi.y, lo.y);
-      split2(v[4], v[5], hi.z, lo.z);
-      split2(v[6], v[7], hi.w, lo.w);
-      *reinterpret_cast<uint4*>(sh_s + off) = hi;
-      *reinterpret_cast<uint4*>(sl_s + off) = lo;
-    };
+            for (int j = 0; j < 8; ++j) x[j] = __uint_as_float(r[j]);
+            store8(e, x);
+          } else if (c / 32 > wq) {                       // above the diagonal
 #pragma unroll
-    for (int i = 0; i < IT; ++i) {
-      const int e = threadIdx.x + NT * i, row = e / (NH * 8), c8 = e % (NH * 8), col = c8 * 8;
-      float v[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] = 0.f;
-      if (row < L.P) {
-        if (L.N % 8 == 0) {
-          if (col < L.N) {
-            const float4* src = reinterpret_cast<const float4*>(S0 + long(row) * L.N + col);
-            const float4 f0 = src[0], f1 = src[1];
-            v[0] = f0.x; v[1] = f0.y; v[2] = f0.z; v[3] = f0.w;
-            v[4] = f1.x; v[5] = f1.y; v[6] = f1.z; v[7] = f1.w;
+            for (int j = 0; j < 8; ++j) x[j] = 0.f;
+            store8(e, x);
           }
-        } else {
-#pragma unroll
-          for (int j = 0; j < 8; ++j)
-            if (col + j < L.N) v[j] = S0[long(row) * L.N + col + j];
         }
+    } else if (lv == 2) {
+      // the state in front of the chunk, high parts and remainders
+      const float* S0 = a.dS + (long(chunk) * L.H + h) * L.P * L.N;
+      constexpr int IT = PW * NH * 8 / NT;
+#pragma unroll
+      for (int i = 0; i < IT; ++i) {
+        const int e = threadIdx.x + NT * i, row = e / (NH * 8), c8 = e % (NH * 8), col = c8 * 8;
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = 0.f;
+        if (row < L.P) {
+          if (L.N % 8 == 0) {
+            if (col < L.N) {
+              const float4* src = reinterpret_cast<const float4*>(S0 + long(row) * L.N + col);
+              const float4 f0 = src[0], f1 = src[1];
+              v[0] = f0.x; v[1] = f0.y; v[2] = f0.z; v[3] = f0.w;
+              v[4] = f1.x; v[5] = f1.y; v[6] = f1.z; v[7] = f1.w;
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              if (col + j < L.N) v[j] = S0[long(row) * L.N + col + j];
+          }
+        }
+        const int off = (c8 >> 3) * SHALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4);
+        uint4 hi, lo;
+        split2(v[0], v[1], hi.x, lo.x);
+        split2(v[2], v[3], hi.y, lo.y);
+        split2(v[4], v[5], hi.z, lo.z);
+        split2(v[6], v[7], hi.w, lo.w);
+        *reinterpret_cast<uint4*>(sh_s + off) = hi;
+        *reinterpret_cast<uint4*>(sl_s + off) = lo;
       }
-      put(row, c8, v);
-    }
-  }
-  level_wait(2);
-  float x16[16];                                          // columns 0 .. 15 of the diagonal group, for its lower half
-  if (wg == diag_wg) {
-    uint32_t r[16];
-    tmem_ld16(tm_d + lane_off + wq * 32, r);
-    tmem_ld_wait();
+#pragma unroll 1
+      for (int c = wg * 16; c < C; c += WGS * 16)
+        if ((wq & 1) && c / 32 == wq - 1) {               // the second 32 rows of either half against the first
+#pragma unroll 1
+          for (int e = c; e < c + 16; e += 8) {
+            uint32_t r[8];
+            float x[8];
+            tmem_ld8(tm_d + 128 + lane_off + e, r);
+            tmem_ld_wait();
 #pragma unroll
-    for (int j = 0; j < 16; ++j) x16[j] = __uint_as_float(r[j]);
+            for (int j = 0; j < 8; ++j) x[j] = __uint_as_float(r[j]);
+            store8(e, x);
+          }
+        }
+    }
+    wait(lv, SITE_FORGET_LEVEL);                          // the tiles are free, accumulators two levels back have been read
   }
-  __syncthreads();
-  build_level<8, PAIRS>(q, w, g_s, p, seg, q_s, kh_s, kl_s);
-  level_mma(3);
-  level_wait(3);
-  if (wg == diag_wg) {
-    uint32_t r[32];
-    float x[32];
-    tmem_ld32(tm_d + 128 + lane_off + wq * 32, r);
-    tmem_ld_wait();
-    const int blk = lane >> 3;                            // block of 8 tokens inside the group
-    const float* dr = diag_s + (wq * 32 + lane) * 8;
-    float d[8];
-    {
-      const float4 d0 = *reinterpret_cast<const float4*>(dr), d1 = *reinterpret_cast<const float4*>(dr + 4);
-      d[0] = d0.x; d[1] = d0.y; d[2] = d0.z; d[3] = d0.w;
-      d[4] = d1.x; d[5] = d1.y; d[6] = d1.z; d[7] = d1.w;
-      if constexpr (NH == 2) {
-        const float4 e0 = *reinterpret_cast<const float4*>(dr + C * 8), e1 = *reinterpret_cast<const float4*>(dr + C * 8 + 4);
-        d[0] += e0.x; d[1] += e0.y; d[2] += e0.z; d[3] += e0.w;
-        d[4] += e1.x; d[5] += e1.y; d[6] += e1.z; d[7] += e1.w;
+  put_queries(product(0, seg));                           // decayed from the chunk's first token on
+  // the 32 columns on the diagonal: levels of 16 and of 8 and the blocks of 8
+#pragma unroll 1
+  for (int c = wg * 16; c < C; c += WGS * 16)
+    if (c / 32 == wq) {
+#pragma unroll 1
+      for (int e = c; e < c + 16; e += 8) {
+        const int cb = (e >> 3) & 3, blk = lane >> 3;     // blocks of 8 of the columns and of the lane's token
+        uint32_t r16[8], r8[8];
+        tmem_ld8(tm_d + lane_off + e, r16);
+        tmem_ld8(tm_d + 128 + lane_off + e, r8);
+        const float4 d0 = *reinterpret_cast<const float4*>(diag_s + (wq * 32 + lane) * 8);
+        const float4 d1 = *reinterpret_cast<const float4*>(diag_s + (wq * 32 + lane) * 8 + 4);
+        const float d[8] = {d0.x, d0.y, d0.z, d0.w, d1.x, d1.y, d1.z, d1.w};
+        tmem_ld_wait();
+        float x[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          x[j] = cb == blk                       ? (j <= (lane & 7) ? d[j] : 0.f)
+                 : !(cb & 1) && blk == cb + 1    ? __uint_as_float(r8[j])
+                 : cb < 2 && blk >= 2            ? __uint_as_float(r16[j])
+                                                 : 0.f;
+        store8(e, x);
       }
     }
-#pragma unroll
-    for (int c = 0; c < 32; ++c) {
-      const int cb = c >> 3;
-      float v = 0.f;
-      if (cb == blk) v = (c & 7) <= (lane & 7) ? d[c & 7] : 0.f;
-      else if ((cb == 0 && blk == 1) || (cb == 2 && blk == 3)) v = __uint_as_float(r[c]);
-      else if (cb < 2 && blk >= 2) v = x16[c & 15];
-      x[c] = v;
-    }
-    store_group(wq, x);
-  }
-  __syncthreads();                                        // the q tile is free
-  {
-    float2 m = totals<PAIRS>(g_s, p, 0, seg);             // queries decayed from the chunk's first token on
-#pragma unroll
-    for (int i = 0; i < SEG; ++i) {
-      m.x *= 1.f - w[i].x;
-      m.y *= 1.f - w[i].y;
-      *reinterpret_cast<uint32_t*>(q_s + pair_off(seg * SEG + i, p)) = pack_bf16x2(q[i].x * m.x, q[i].y * m.y);
-    }
-  }
   tmem_st_wait();
   fence_proxy_async_smem();
   tc_fence_before();
@@ -607,7 +600,7 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
   if (threadIdx.x == 0) {
     constexpr uint32_t idesc_x = umma_idesc(128, PW, 1, 1, 0, 0);
     constexpr uint32_t idesc_o = umma_idesc(128, PW, 1, 1, 0, 1);
-    const uint32_t sh = smem_u32(sh_s), sl = smem_u32(sl_s);
+    const uint32_t sh = smem_u32(sh_s), sl = smem_u32(sl_s), va = smem_u32(v_s);
 #pragma unroll
     for (int k = 0; k < NH * 4; ++k) {
       const uint64_t ad = umma_desc_k_sw128(qa + (k >> 2) * HALF + (k & 3) * 32);
@@ -624,31 +617,21 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
     umma_commit(&bars[4]);
   }
   __syncwarp();
-  if (!mbar_wait(&bars[4], 0, abort_flag)) {
-    *abort_flag = 1;
-    atomicCAS(a.status, 0, ST_TIMEOUT_TMEM_FULL | SITE_FORGET_OUTPUT);
-    ok = false;
-  }
-  __syncwarp();
-  tc_fence_after();
-  // norm over the head's value columns (those past P are zeros): 32 columns per warp, sums joined through shared memory
+  wait(4, SITE_FORGET_OUTPUT);
+  // norm over the head's value columns (those past P are zeros): 16 columns per warp and turn, sums joined in shared memory
   const int row = wq * 32 + lane;
-  constexpr int GROUPS = PW / 32, PER = (GROUPS + WGS - 1) / WGS;        // column groups, and of them per warpgroup
-  float y[PER][32];
+  constexpr int GROUPS = PW / 16, PER = (GROUPS + WGS - 1) / WGS;        // column groups, and of them per warpgroup
+  uint32_t y[PER][16];
   float ss = 0.f;
-  const bool all_ok = __all_sync(0xffffffffu, ok);
+  const bool all_ok = ok;                                 // (the same for the whole CTA)
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int g = wg + i * WGS;
     if (all_ok && g < GROUPS) {
-      uint32_t r[32];
-      tmem_ld32(tm_o + lane_off + g * 32, r);
+      tmem_ld16(tm_o + lane_off + g * 16, y[i]);
       tmem_ld_wait();
 #pragma unroll
-      for (int j = 0; j < 32; ++j) {
-        y[i][j] = __uint_as_float(r[j]);
-        ss = fmaf(y[i][j], y[i][j], ss);
-      }
+      for (int j = 0; j < 16; ++j) ss = fmaf(__uint_as_float(y[i][j]), __uint_as_float(y[i][j]), ss);
     }
   }
   red_s[wg * C + row] = ss;
@@ -664,12 +647,12 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
       const int g = wg + i * WGS;
       if (g >= GROUPS) continue;
 #pragma unroll
-      for (int j = 0; j < 32; j += 8) {
-        const int col = g * 32 + j;
+      for (int j = 0; j < 16; j += 8) {
+        const int col = g * 16 + j;
         if (col >= L.P) continue;
         float z[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) z[e] = col + e < L.P ? y[i][j + e] * inv * __ldg(L.norm_w + col + e) : 0.f;
+        for (int e = 0; e < 8; ++e) z[e] = col + e < L.P ? __uint_as_float(y[i][j + e]) * inv * __ldg(L.norm_w + col + e) : 0.f;
         if (a.vec_o) {
           *reinterpret_cast<uint4*>(orow + col) = make_uint4(pack_bf16x2(z[0], z[1]), pack_bf16x2(z[2], z[3]),
                                                              pack_bf16x2(z[4], z[5]), pack_bf16x2(z[6], z[7]));
@@ -691,8 +674,7 @@ __global__ void __launch_bounds__(NH * 256, 1) forget_output_kernel(const Forget
 
 template <int NH, int PH>
 int launch_np(const ForgetChunkArgs& a, int n_chunks, const int* seq_chunk0, const int* seq_nchunk, cudaStream_t s) {
-  constexpr int SA = states_smem<NH, PH>(), SC = output_smem<NH, PH>();
-  static_assert(SC <= 227 * 1024, "shared memory budget");
+  constexpr int SA = states_smem<NH, PH>(), SC = OutSmem<NH, PH>::BYTES;
   auto ks = forget_states_kernel<NH, PH>;
   auto ko = forget_output_kernel<NH, PH>;
   static bool attr = false;
@@ -711,7 +693,7 @@ int launch_np(const ForgetChunkArgs& a, int n_chunks, const int* seq_chunk0, con
   if ((vec == 4 ? launch_pdl(forget_carry_kernel<4>, gc, dim3(256), 0, s, a, seq_chunk0, seq_nchunk)
                 : launch_pdl(forget_carry_kernel<1>, gc, dim3(256), 0, s, a, seq_chunk0, seq_nchunk)) != cudaSuccess)
     return 1;
-  return launch_pdl(ko, grid, dim3(NH * 256), SC, s, a) != cudaSuccess;
+  return launch_pdl(ko, grid, dim3(NH * 512), SC, s, a) != cudaSuccess;
 }
 
 }  // namespace

@@ -3,7 +3,8 @@
 // v to the paged cache. A CTA takes a few consecutive tokens of one sequence, so taps are read once for all of them and a
 // norm over all heads stays inside it; q and k wait in shared memory in fp32 for their norms, v goes straight to its cell.
 // Decode steps have a CTA per token with a thread per four columns and update the history here; prompts leave that to a
-// second small launch, since other CTAs may still read the old one.
+// second small launch, since other CTAs may still read the old one. Rows that are only rotated (neighbouring columns) and
+// appended have a form of their own: nothing passes between threads, so each takes eight columns of a token.
 #include "act_type.cuh"
 #include "common.cuh"
 #include "layers.h"
@@ -282,6 +283,68 @@ __global__ void __launch_bounds__(128) qkv_history_kernel(const QkvConvArgs a) {
   }
 }
 
+template <typename T>
+__device__ __forceinline__ void ld8(const T* p, float (&v)[8]) {
+  float a[4], b[4];
+  if constexpr (sizeof(T) == 2) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      v[2 * j] = __uint_as_float(w[j] << 16);
+      v[2 * j + 1] = __uint_as_float(w[j] & 0xffff0000u);
+    }
+  } else {
+    ld_f4(p, a);
+    ld_f4(p + 4, b);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { v[j] = a[j]; v[4 + j] = b[j]; }
+  }
+}
+template <typename T>
+__device__ __forceinline__ void st8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                              pack_bf16x2(v[6], v[7]));
+  } else {
+    st_f4(p, {v[0], v[1], v[2], v[3]});
+    st_f4(p + 4, {v[4], v[5], v[6], v[7]});
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_rotate_kernel(const QkvConvArgs a) {
+  const int nq = a.Hq * a.DK, nk = a.Hkv * a.DK, per = (nq + nk + a.Hkv * a.DV) / 8;
+  const long i = long(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= long(a.T) * per) return;
+  const int t = int(i / per), c = int(i % per) * 8, d = c < nq + nk ? c % a.DK : a.rot;
+  // positions, cells and the table are not written by the projection in front of this launch
+  const long cell = c < nq ? 0 : a.slots[t];
+  float cs[4], sn[4];
+  const bool turn = d < a.rot;
+  if (turn) {
+    const float* row = a.cos_sin + long(a.positions[t]) * a.rot + d / 2;
+    ld_f4(row, cs);
+    ld_f4(row + a.rot / 2, sn);
+  }
+  griddep_wait();
+  griddep_launch();
+  if (cell < 0) return;
+  float v[8];
+  ld8(static_cast<const T*>(a.x) + t * a.ld + c, v);
+  if (turn) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float f = v[2 * j], g = v[2 * j + 1];
+      v[2 * j] = f * cs[j] - g * sn[j];
+      v[2 * j + 1] = g * cs[j] + f * sn[j];
+    }
+  }
+  if (c < nq) st8(static_cast<T*>(a.q_out) + long(t) * nq + c, v);
+  else if (c < nq + nk) st8(static_cast<T*>(a.k_cache) + cell * a.k_cell + (c - nq), v);
+  else st8(static_cast<T*>(a.v_cache) + cell * a.v_cell + (c - nq - nk), v);
+}
+
 template <typename T, int TOK, int VEC>
 int launch_v(const QkvConvArgs& a, cudaStream_t s) {
   const int taps = a.conv_w ? a.KC : 1, C = (a.Hq + a.Hkv) * a.DK + a.Hkv * a.DV;
@@ -305,6 +368,11 @@ int launch_v(const QkvConvArgs& a, cudaStream_t s) {
 template <typename T>
 int launch_t(const QkvConvArgs& a, cudaStream_t s) {
   auto al = [](const void* p, size_t n) { return reinterpret_cast<uintptr_t>(p) % n == 0; };
+  if (!a.in_b && !a.conv_w && !a.qw && (a.rot == 0 || (!a.rot_half && al(a.cos_sin, 16))) && a.rot % 8 == 0 && a.DK % 8 == 0 &&
+      a.DV % 8 == 0 && a.ld % 8 == 0 && al(a.x, 16) && al(a.q_out, 16) && al(a.k_cache, 16) && al(a.v_cache, 16)) {
+    const long n = long(a.T) * (((a.Hq + a.Hkv) * a.DK + a.Hkv * a.DV) / 8);
+    return launch_pdl(qkv_rotate_kernel<T>, dim3(unsigned((n + 255) / 256)), dim3(256), 0, s, a) != cudaSuccess;
+  }
   const bool vec = a.DK % 4 == 0 && a.DV % 4 == 0 && a.ld % 4 == 0 && al(a.x, 4 * sizeof(T)) && al(a.in_b, 16) && al(a.conv_w, 16) &&
                    al(a.conv_state, 16) && al(a.v_cache, 4 * sizeof(T)) && al(a.k_cache, 8) && al(a.q_out, 8) && al(a.cos_sin, 8) && al(a.qw, 8) && al(a.kw, 8);
   const int rc = a.tok == 1 ? (vec ? launch_v<T, 1, 4>(a, s) : launch_v<T, 1, 1>(a, s))

@@ -296,9 +296,14 @@ def test_sampled_generation_on_gpu():
 
 
 @gpu
+@pytest.mark.parametrize("branches,lanes", [(3, 2), (0, 2), (0, 1)])
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
-def test_many_sequences_decode_together(models, dtype):
-    """More decoded sequences than one routing tile holds; two lanes of the captured step from 64 rows on."""
+def test_many_sequences_decode_together(models, dtype, branches, lanes, monkeypatch):
+    """More decoded sequences than one routing tile holds, with sublayers on branches of the captured step, as two lanes of it,
+    and in a row."""
+    from legion_b200.ops import sm100
+    monkeypatch.setitem(sm100.TUNE, "parallel_branches", branches)
+    monkeypatch.setitem(sm100.TUNE, "decode_lanes", lanes)
     cfg, w, path = models.get("mixed", dtype)
     n = 70
     seqs = {f"q{i}": nc.tokens(cfg, 9 + i % 5, 200 + i) for i in range(n)}
