@@ -691,12 +691,16 @@ def bench_forget(rows):
             flops = n * (L - window / 2) * window * H * D * 4
             row("windowed attention, sink and head gate, prompt", n, L, tm(ext), flops=flops)
             row("windowed attention, prompt", n, L, tm(lambda: sm100.prefill_attn(qq, kc, vc, cu, cl, bt, L, D ** -0.5, window)), flops=flops)
-        # residual with gates and depth average behind layers 0, 11 and 22 of 24
-        hist = torch.randn(25, T, W, device="cuda") if T <= 64 else torch.zeros(25, T, W, device="cuda")
+        # residual with gates and depth average: four layers from the 1st, 13th and 21st of 24 on
+        hist = sm100.DepthHistory(torch.zeros(25, T, W, device="cuda"))
         x, y, p2, nw = torch.randn(T, W, device="cuda"), f(T, W), f(T, 2 * W), torch.zeros(W, device="cuda")
-        for i in (0, 11, 22):
-            row(f"depth_step 2048, {i + 2} terms", n, L, tm(lambda: sm100.depth_step(
-                x, hist, i, y, p2[:, :W], nw, y, p2[:, W:], nw, nw, one[:i + 2], nw, 1e-6, 1.0)), T * W * (4 * (i + 4) + 10))
+        co = [torch.ones(26, device="cuda") for _ in range(4)]
+
+        def four(i):
+            for j in range(i, i + 4):
+                sm100.depth_step(x, hist, j, y, p2[:, :W], nw, y, p2[:, W:], nw, nw, co[:4 - (j - i)], nw, 1e-6, 1.0)
+        for i in (0, 12, 20):
+            row(f"depth_step 2048, behind layers {i} .. {i + 3}, each", n, L, tm(lambda: four(i)) / 4, T * W * (i + 22 - (i == 20) + 10))
         del hist
         X, mix = torch.randn(T, 4, W, device="cuda"), torch.eye(4, device="cuda")
         row("hyper_step 4x2048", n, L, tm(lambda: sm100.hyper_step(X, [(y, 1.0)], mix, one[:4], one[:4], nw, 1e-5, 1.0)), T * W * 36)

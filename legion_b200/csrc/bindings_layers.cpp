@@ -251,10 +251,12 @@ void bind_layers(pybind11::module_& m) {
     c10::cuda::CUDAGuard guard(x_out.device());
     TORCH_CHECK(lb::hyper_launch(a, f32, cur_stream()) == 0, "prenorm_step: rows of at most 51200 columns", cuda_error());
   });
-  m.def("depth_step", [](const Tensor& x, Tensor& x_out, const OptT& hist, int64_t layer, bool keep, const Tensor& y1,
-                         const OptT& g1, const OptT& b1, const OptT& y2, int64_t y2_rows, const OptT& g2, const OptT& b2,
-                         const OptT& y2_b, const OptT& coef, const Tensor& norm_w, double eps, double w_offset, Tensor& h,
-                         const OptT& rows) {
+  // first: index of the first earlier result to sum up (those before it are in `part`); coefs: of this layer and, for the sums
+  // that `ahead` takes, of the layers behind it
+  m.def("depth_step", [](const Tensor& x, Tensor& x_out, const OptT& hist, int64_t layer, int64_t first, const OptT& part, bool keep,
+                         const Tensor& y1, const OptT& g1, const OptT& b1, const OptT& y2, int64_t y2_rows, const OptT& g2,
+                         const OptT& b2, const OptT& y2_b, const std::vector<Tensor>& coefs, const OptT& ahead,
+                         const Tensor& norm_w, double eps, double w_offset, Tensor& h, const OptT& rows) {
     const bool f32 = is_f32(h, "h");
     same(y1, f32, "y1");
     const int64_t T = x.size(0), H = x.size(1), R = h.size(0);
@@ -266,11 +268,26 @@ void bind_layers(pybind11::module_& m) {
     a.y1 = y1.data_ptr(); a.ldy1 = y1.stride(0); a.y2_rows = 1;
     if (hist.has_value()) {
       TORCH_CHECK(hist->is_contiguous() && hist->scalar_type() == at::kFloat && hist->dim() == 3 && hist->size(0) > layer + 1 &&
-                      hist->size(1) == T && hist->size(2) == H && layer >= 0 && coef.has_value(), "depth_step: hist [layers + 1, rows, width]");
-      f32c(*coef, layer + 2, "depth average");
-      a.hist = hist->data_ptr<float>(); a.hist_stride = T * H; a.n_hist = int(layer + 1);
-      a.coef = coef->data_ptr<float>();
+                      hist->size(1) == T && hist->size(2) == H && layer >= 0 && first >= 0 && first <= layer + 1 && !coefs.empty(),
+                  "depth_step: hist [layers + 1, rows, width]");
+      a.hist = hist->data_ptr<float>() + first * T * H; a.hist_stride = T * H; a.n_hist = int(layer + 1 - first);
+      f32c(coefs[0], layer + 2, "depth average");
+      a.coef = coefs[0].data_ptr<float>() + first;
       if (keep) a.hist_out = hist->data_ptr<float>() + (layer + 1) * T * H;
+      if (part.has_value()) {
+        f32c(*part, T * H, "partial sum");
+        a.part = part->data_ptr<float>();
+      }
+      if (ahead.has_value()) {
+        a.n_ahead = int(coefs.size()) - 1;
+        TORCH_CHECK(a.n_ahead <= lb::DEPTH_AHEAD && first == 0, "depth_step: sums ahead");
+        f32c(*ahead, a.n_ahead * T * H, "sums ahead");
+        a.ahead_out = ahead->data_ptr<float>();
+        for (int s = 0; s < a.n_ahead; ++s) {
+          f32c(coefs[s + 1], layer + 2, "depth average");
+          a.ahead_coef[s] = coefs[s + 1].data_ptr<float>();
+        }
+      }
     }
     if (y2.has_value()) {
       same(*y2, f32, "y2");

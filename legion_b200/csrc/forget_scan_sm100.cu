@@ -44,7 +44,7 @@ struct ForgetChunkArgs {
   const int* chunk_t0; const int* chunk_n;
   float* dS;                              // [chunks, H, P, N]: chunk contributions, then the state in front of each chunk
   float* gC;                              // [chunks, H, N]: product of the chunk's gates
-  int pair_q, pair_f, vec_v, vec_o;       // 4-byte pairs / 16-byte vectors are aligned
+  int vec_q, vec_f, vec_v, vec_o;         // 16-byte vectors are aligned
   int* status;
 };
 
@@ -59,13 +59,38 @@ __device__ __forceinline__ float2 bf2(uint32_t u) {
   return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
 }
 // columns c, c + 1 of a row (zero from `width` on)
-__device__ __forceinline__ uint32_t ld_pair(const __nv_bfloat16* row, int c, int width, bool pair) {
-  if (pair && c + 1 < width) return __ldg(reinterpret_cast<const unsigned int*>(row + c));
+__device__ __forceinline__ uint32_t ld_pair(const __nv_bfloat16* row, int c, int width) {
   uint32_t u = 0;
   if (c < width) u = __bfloat16_as_ushort(row[c]);
   if (c + 1 < width) u |= uint32_t(__bfloat16_as_ushort(row[c + 1])) << 16;
   return u;
 }
+// 16 bytes global -> shared, zeros without `in`
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool in) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+// A chunk's rows of a head, W8 * 8 columns (zeros past `width` and past its tokens), by asynchronous copies where rows are
+// aligned; off(row, 8-column piece): byte offset of a piece.
+template <int W8, int NT, typename Off>
+__device__ __forceinline__ void stage_rows(uint8_t* dst, const __nv_bfloat16* src, long ld, int width, int nval, bool vec, Off off) {
+#pragma unroll
+  for (int i = 0; i < C * W8 / NT; ++i) {
+    const int e = threadIdx.x + NT * i, row = e / W8, c8 = e % W8;
+    const bool in = row < nval && c8 * 8 < width;
+    const __nv_bfloat16* r = src + (in ? row * ld + c8 * 8 : 0);
+    uint8_t* to = dst + off(row, c8);
+    if (vec) {
+      cp_async16(to, r, in);
+    } else {
+      uint32_t u[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) u[j] = in ? ld_pair(r, 2 * j, width - c8 * 8) : 0u;
+      *reinterpret_cast<uint4*>(to) = make_uint4(u[0], u[1], u[2], u[3]);
+    }
+  }
+}
+__device__ __forceinline__ int tile_off(int row, int c8) { return (c8 >> 3) * HALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4); }
 // byte offset of column pair p of a row in a K-major tile of 64-column halves, 128-byte swizzle
 __device__ __forceinline__ int pair_off(int row, int p) {
   return (p >> 5) * HALF + row * 128 + ((((p & 31) >> 2) ^ (row & 7)) << 4) + (p & 3) * 4;
@@ -77,20 +102,17 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   lo = pack_bf16x2(x - f.x, y - f.y);
 }
 
-// What a thread writes per token of its segment: 1 - F of its two channels (0 past the chunk's tokens).
-__device__ __forceinline__ void load_writes(const ForgetChunkArgs& a, int h, int t0, int nval, int p, int seg, float2 (&w)[SEG]) {
+// What a thread writes per token of its segment: 1 - F of its two channels (0 past the chunk's tokens); f_s: the staged rows.
+__device__ __forceinline__ void load_writes(const ForgetChunkArgs& a, const uint32_t* f_s, int pairs, int h, int nval, int p, int seg,
+                                            float2 (&w)[SEG]) {
   const ForgetScanArgs& L = a.L;
   const int c = 2 * p;
-  const auto* fp = static_cast<const __nv_bfloat16*>(L.f) + long(t0 + seg * SEG) * L.ldf + long(h) * L.N;
-  uint32_t raw[SEG];
-#pragma unroll
-  for (int i = 0; i < SEG; ++i) raw[i] = seg * SEG + i < nval ? ld_pair(fp + i * L.ldf, c, L.N, a.pair_f) : 0u;
   float2 b = make_float2(0.f, 0.f), open = b;               // bias, 1 - lower (0 past the head's channels)
   if (c < L.N) { b.x = L.f_b[h * L.N + c]; open.x = 1.f - L.lower[h * L.N + c]; }
   if (c + 1 < L.N) { b.y = L.f_b[h * L.N + c + 1]; open.y = 1.f - L.lower[h * L.N + c + 1]; }
 #pragma unroll
   for (int i = 0; i < SEG; ++i) {
-    const float2 z = bf2(raw[i]);
+    const float2 z = bf2(f_s[(seg * SEG + i) * pairs + p]);
     const bool in = seg * SEG + i < nval;
     w[i].x = in ? open.x * sigmoid_fast(-(z.x + b.x)) : 0.f;
     w[i].y = in ? open.y * sigmoid_fast(-(z.y + b.y)) : 0.f;
@@ -114,31 +136,12 @@ __device__ __forceinline__ float2 totals(const float2* g_s, int p, int lo, int h
   return m;
 }
 
-// Values of the chunk as a tile [128 tokens][PH * 64 columns]
+// Values of the chunk as a tile [128 tokens][PH * 64 columns] (asynchronous copies: wait for them)
 template <int PH, int NT>
 __device__ __forceinline__ void load_values(const ForgetChunkArgs& a, int h, int t0, int nval, uint8_t* dst) {
   const ForgetScanArgs& L = a.L;
-  const auto* vp = static_cast<const __nv_bfloat16*>(L.v) + long(t0) * L.ldv + long(h) * L.P;
-  constexpr int IT = C * PH * 8 / NT;
-  uint4 raw[IT];
-#pragma unroll
-  for (int i = 0; i < IT; ++i) {
-    const int e = threadIdx.x + NT * i, row = e / (PH * 8), c = (e % (PH * 8)) * 8;
-    raw[i] = make_uint4(0u, 0u, 0u, 0u);
-    if (row >= nval || c >= L.P) continue;
-    const __nv_bfloat16* src = vp + long(row) * L.ldv;
-    if (a.vec_v) {
-      raw[i] = __ldg(reinterpret_cast<const uint4*>(src + c));
-    } else {
-      raw[i].x = ld_pair(src, c, L.P, false); raw[i].y = ld_pair(src, c + 2, L.P, false);
-      raw[i].z = ld_pair(src, c + 4, L.P, false); raw[i].w = ld_pair(src, c + 6, L.P, false);
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < IT; ++i) {
-    const int e = threadIdx.x + NT * i, row = e / (PH * 8), c8 = e % (PH * 8);
-    *reinterpret_cast<uint4*>(dst + (c8 >> 3) * HALF + row * 128 + (((c8 & 7) ^ (row & 7)) << 4)) = raw[i];
-  }
+  stage_rows<PH * 8, NT>(dst, static_cast<const __nv_bfloat16*>(L.v) + long(t0) * L.ldv + long(h) * L.P, L.ldv, L.P, nval, a.vec_v,
+                         tile_off);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -151,7 +154,7 @@ template <int NH, int PH>
 __global__ void __launch_bounds__(NH * 256) forget_states_kernel(const ForgetChunkArgs a) {
   constexpr int NT = NH * 256, PAIRS = NH * 32;
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);   // (an offset: the address space stays known)
   uint8_t* v_s = smem;
   uint8_t* kh_s = v_s + PH * HALF;
   uint8_t* kl_s = kh_s + NH * HALF;
@@ -175,10 +178,14 @@ __global__ void __launch_bounds__(NH * 256) forget_states_kernel(const ForgetChu
   griddep_wait();
   griddep_launch();
   const int t0 = a.chunk_t0[chunk], nval = a.chunk_n[chunk];
+  stage_rows<NH * 8, NT>(kl_s, static_cast<const __nv_bfloat16*>(L.f) + long(t0) * L.ldf + long(h) * L.N, L.ldf, L.N, nval, a.vec_f,
+                         [](int row, int c8) { return row * (NH * 128) + c8 * 16; });
   load_values<PH, NT>(a, h, t0, nval, v_s);
   {
+    cp_async_wait();
+    __syncthreads();
     float2 w[SEG];
-    load_writes(a, h, t0, nval, p, seg, w);
+    load_writes(a, reinterpret_cast<const uint32_t*>(kl_s), PAIRS, h, nval, p, seg, w);
     g_s[seg * PAIRS + p] = total_of(w);
     __syncthreads();
     float2 m = totals<PAIRS>(g_s, p, seg + 1, SEGS);
@@ -320,7 +327,7 @@ __global__ void __launch_bounds__(NH * 512, 1) forget_output_kernel(const Forget
   using Sm = OutSmem<NH, PH>;
   constexpr int NT = NH * 512, PAIRS = NH * 32, WGS = NT / 128, PW = PH * 64, SHALF = Sm::SHALF;
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);   // (an offset: the address space stays known)
   uint8_t* q_s = smem;
   uint8_t* kh_s = q_s + NH * HALF;
   uint8_t* kl_s = kh_s + NH * HALF;
@@ -354,30 +361,27 @@ __global__ void __launch_bounds__(NH * 512, 1) forget_output_kernel(const Forget
   const int t0 = a.chunk_t0[chunk], nval = a.chunk_n[chunk];
   uint64_t q[OSEG], nw[OSEG];
   {
-    const long row0 = t0 + seg * OSEG;
-    const auto* qp = static_cast<const __nv_bfloat16*>(L.q) + row0 * L.ldq + long(h) * L.N;
-    const auto* fp = static_cast<const __nv_bfloat16*>(L.f) + row0 * L.ldf + long(h) * L.N;
-    uint32_t rq[OSEG], rf[OSEG];
-#pragma unroll
-    for (int i = 0; i < OSEG; ++i) {
-      const bool in = seg * OSEG + i < nval;
-      rq[i] = in ? ld_pair(qp + i * L.ldq, 2 * p, L.N, a.pair_q) : 0u;
-      rf[i] = in ? ld_pair(fp + i * L.ldf, 2 * p, L.N, a.pair_f) : 0u;
-    }
+    auto rows = [](int row, int c8) { return row * (NH * 128) + c8 * 16; };
+    stage_rows<NH * 8, NT>(reinterpret_cast<uint8_t*>(qb_s), static_cast<const __nv_bfloat16*>(L.q) + long(t0) * L.ldq + long(h) * L.N,
+                           L.ldq, L.N, nval, a.vec_q, rows);
+    stage_rows<NH * 8, NT>(kh_s, static_cast<const __nv_bfloat16*>(L.f) + long(t0) * L.ldf + long(h) * L.N, L.ldf, L.N, nval, a.vec_f,
+                           rows);
     float2 b = make_float2(0.f, 0.f), open = b;               // bias, 1 - lower (0 past the head's channels)
     if (2 * p < L.N) { b.x = L.f_b[h * L.N + 2 * p]; open.x = 1.f - L.lower[h * L.N + 2 * p]; }
     if (2 * p + 1 < L.N) { b.y = L.f_b[h * L.N + 2 * p + 1]; open.y = 1.f - L.lower[h * L.N + 2 * p + 1]; }
+    cp_async_wait();
+    __syncthreads();
+    const uint32_t* f_s = reinterpret_cast<const uint32_t*>(kh_s);
     uint64_t g = p2(1.f, 1.f);
 #pragma unroll
     for (int i = 0; i < OSEG; ++i) {
       const int t = seg * OSEG + i;
-      const float2 z = bf2(rq[i]), e = bf2(rf[i]);
+      const float2 z = bf2(qb_s[t * PAIRS + p]), e = bf2(f_s[t * PAIRS + p]);
       const float qx = z.x * sigmoid_fast(z.x), qy = z.y * sigmoid_fast(z.y);
       q[i] = p2(qx, qy);
       nw[i] = t < nval ? p2(-open.x * sigmoid_fast(-(e.x + b.x)), -open.y * sigmoid_fast(-(e.y + b.y))) : 0ull;
       g = fma2(nw[i], g, g);
       *reinterpret_cast<uint64_t*>(nw_s + t * (NH * 64) + 2 * p) = nw[i];
-      qb_s[t * PAIRS + p] = rq[i];
     }
     g_s[seg * PAIRS + p] = g;
   }
@@ -593,6 +597,7 @@ __global__ void __launch_bounds__(NH * 512, 1) forget_output_kernel(const Forget
       }
     }
   tmem_st_wait();
+  cp_async_wait();                                        // the values
   fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
@@ -715,8 +720,8 @@ int forget_chunk_launch(const ForgetScanArgs& L, const int* chunk_t0, const int*
   a.dS = static_cast<float*>(scratch);
   a.gC = a.dS + size_t(n_chunks) * L.H * L.N * L.P;
   auto al = [](const void* p, long ld, int w, int n) { return reinterpret_cast<uintptr_t>(p) % (2 * n) == 0 && ld % n == 0 && w % n == 0; };
-  a.pair_q = al(L.q, L.ldq, L.N, 2);
-  a.pair_f = al(L.f, L.ldf, L.N, 2);
+  a.vec_q = al(L.q, L.ldq, L.N, 8);
+  a.vec_f = al(L.f, L.ldf, L.N, 8);
   a.vec_v = al(L.v, L.ldv, L.P, 8);
   a.vec_o = al(L.out, L.ldo, L.P, 8);
   if (L.N <= 64) return L.P <= 64 ? launch_np<1, 1>(a, n_chunks, seq_chunk0, seq_nchunk, s)

@@ -31,12 +31,16 @@ struct HyperArgs {
 int hyper_launch(const HyperArgs& a, bool f32, cudaStream_t s);
 
 // Parallel sublayers on one fp32 residual, with gates and depth average (depth_step.cu).
+constexpr int DEPTH_AHEAD = 3;     // layers for which a pass over all earlier results sums up ahead
 struct DepthStepArgs {
   const float* x;                  // [T, H] the layer's input
   float* x_out;                    // [n_rows, H] the next one's (may be x without rows)
-  const float* hist; long hist_stride; int n_hist;   // X_0 .. X_(n_hist - 1), hist_stride floats apart; nullptr: no average
+  const float* hist; long hist_stride; int n_hist;   // earlier results to sum up, hist_stride floats apart
+  const float* part;               // [T, H] sum of those before them; nullptr: none
   float* hist_out;                 // [T, H] takes the layer's result; nullptr: not kept
-  const float* coef;               // [n_hist + 1]
+  const float* coef;               // [n_hist + 1] of hist's results and of the layer's own; nullptr: no average
+  int n_ahead; float* ahead_out;   // [n_ahead] tensors [T, H], hist_stride apart: the same sums with other coefficients
+  const float* ahead_coef[DEPTH_AHEAD];
   const void* y1; long ldy1;       // mixer output, activation type
   const void* y2; long ldy2; int y2_rows; const float* y2_b;   // feed-forward output, the sum of y2_rows consecutive rows
                                    // (nullptr: none), and its bias

@@ -1342,7 +1342,8 @@ class Decoder:
             keep = None
             if last and not capture:
                 keep, rows = rows, None
-            x, h = ops.depth_step(x, hist, il, y1, g1, b1, y2, g2, b2, w.get(f"{p}.mlp.down_b"), w.get(f"{p}.dwa"),
+            coefs = [w[f"l{j}.dwa"] for j in range(il, min(L, il + 1 + ops.sm100.DEPTH_AHEAD))] if hist is not None else None
+            x, h = ops.depth_step(x, hist, il, y1, g1, b1, y2, g2, b2, w.get(f"{p}.mlp.down_b"), coefs,
                                   w["output_norm"] if last else w[f"l{cfg.weight_layer(il + 1)}.attn_norm"], eps, off, keep)
             if capture:
                 captures[il] = x.clone()

@@ -302,7 +302,7 @@ def head_norm_gate(o, gate, w, eps, heads):
 
 def depth_start(table, ids, layers: int, norm_w, eps, w_offset=0.0, average=True):
     """Start of a stack with parallel sublayers: x = embedding rows (``ids`` None: rows are given). Returns (x [T, H] float32,
-    hist [layers + 1, T, H] float32 with x as its first entry, or None without depth averages, norm of x)."""
+    ops.sm100.DepthHistory with x as its first entry, or None without depth averages, norm of x)."""
     T = table.shape[0] if ids is None else ids.numel()
     hist = torch.empty(layers + 1 if average else 1, T, table.shape[1], dtype=torch.float32, device=table.device)
     if _cuda(table):
@@ -310,14 +310,14 @@ def depth_start(table, ids, layers: int, norm_w, eps, w_offset=0.0, average=True
     else:
         x, h = _ref.prenorm_start(table if ids is None else table[ids.long()], None, norm_w, eps, w_offset)
         hist[0] = x
-    return hist[0], hist if average else None, h
+    return hist[0], _sm.DepthHistory(hist) if average else None, h
 
 
-def depth_step(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset=0.0, rows=None):
+def depth_step(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coefs, norm_w, eps, w_offset=0.0, rows=None):
     """Behind a layer with parallel sublayers (see ``reference.depth_step``), one launch; ``y2`` may be a
     ops.sm100.PendingCombine."""
     f = _sm.depth_step if _cuda(x) else _ref.depth_step
-    return f(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset, rows)
+    return f(x, hist, i, y1, g1, b1, y2, g2, b2, y2_b, coefs, norm_w, eps, w_offset, rows)
 
 
 def forget_scan(q, f, v, f_b, lower, state, cu_seq, slots, H, N, P, norm_w, eps, scale=1.0, write_state=True, max_len=None,

@@ -481,19 +481,20 @@ def prenorm_step(x, terms, mult: float, norm_w, eps: float, w_offset: float, dty
     return x, None if norm_w is None else _norm32(x, norm_w, eps, w_offset).to(dtype)
 
 
-def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps: float, w_offset: float, rows=None):
+def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coefs, norm_w, eps: float, w_offset: float, rows=None):
     """Behind layer ``i`` of a stack with parallel sublayers: X = x + sigmoid(g1 + b1) y1 + sigmoid(g2 + b2) (y2 + y2_b) (no
-    gate without ``g1``; ``y2`` may be None). With ``hist`` [layers + 1, T, H] float32 (the embedding output and the layers'
-    results) X becomes its entry i + 1 and the next input is the sum of coef[j] * hist[j] for j = 0 .. i + 1. Returns that
-    and its norm, of the given ``rows`` only when there are any."""
+    gate without ``g1``; ``y2`` may be None). With ``hist`` (``hist.X`` [layers + 1, T, H] float32: the embedding output and the
+    layers' results) X becomes its entry i + 1 and the next input is the sum of coefs[0][j] * hist.X[j] for j = 0 .. i + 1
+    (``coefs``: of layer i, then of the layers behind it). Returns that and its norm, of the given ``rows`` only when there are
+    any."""
     open_ = lambda g, b: 1.0 if g is None else torch.sigmoid(g.float() + b)                # noqa: E731
     X = x + open_(g1, b1) * y1.float()
     if y2 is not None:
         f = y2.float() if y2_b is None else y2.float() + y2_b
         X = X + open_(g2, b2) * f
     if hist is not None:
-        hist[i + 1] = X
-        X = torch.einsum("j,jth->th", coef, hist[:i + 2])
+        hist.X[i + 1] = X
+        X = torch.einsum("j,jth->th", coefs[0], hist.X[:i + 2])
     if rows is not None:
         X = X.index_select(0, rows)
     return X, _norm32(X, norm_w, eps, w_offset).to(y1.dtype)

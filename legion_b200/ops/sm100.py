@@ -1804,19 +1804,42 @@ def prenorm_step(x, terms, mult, norm_w, eps, w_offset=0.0, raw=None, start=None
     return x, h
 
 
-def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coef, norm_w, eps, w_offset=0.0, rows=None):
+DEPTH_AHEAD = 3              # layers for which a pass over all earlier results sums up ahead (csrc/layers.h)
+
+
+class DepthHistory:
+    """The embedding output and the results of the layers, [layers + 1, T, H] float32, and the sums over them that a pass of
+    ``depth_step`` left for the layers behind it."""
+    __slots__ = ("X", "ahead")
+
+    def __init__(self, X):
+        self.X, self.ahead = X, None
+
+
+def depth_step(x, hist, i: int, y1, g1, b1, y2, g2, b2, y2_b, coefs, norm_w, eps, w_offset=0.0, rows=None):
     """``reference.depth_step`` in one launch (``csrc/depth_step.cu``). ``x`` is updated in place unless it is an entry of
-    ``hist`` or only ``rows`` are wanted; the last layer's result is not kept."""
+    ``hist`` or only ``rows`` are wanted; the last layer's result is not kept. One layer in ``DEPTH_AHEAD`` + 1 reads all
+    earlier results, and sums them up for the layers behind it too."""
     y2_rows = 1
     if isinstance(y2, PendingCombine):
         y2_rows, y2 = y2.rows, y2.y
     n = x.shape[0] if rows is None else rows.numel()
-    own = rows is not None or (hist is not None and x.data_ptr() == hist.data_ptr())
+    own = rows is not None or (hist is not None and x.data_ptr() == hist.X.data_ptr())
     x_out = torch.empty(n, x.shape[1], dtype=torch.float32, device=x.device) if own else x
     h = torch.empty(n, x.shape[1], dtype=y1.dtype, device=x.device)
-    if n:
-        ext().depth_step(x, x_out, hist, i, hist is not None and i + 2 < hist.shape[0], y1, g1, b1, y2, y2_rows, g2, b2, y2_b, coef,
-                         norm_w, eps, w_offset, h, rows)
+    if n == 0:
+        return x_out, h
+    X = part = ahead = None
+    first, keep, r = 0, False, i % (DEPTH_AHEAD + 1)
+    if hist is not None:
+        X = hist.X
+        keep = i + 2 < X.shape[0]
+        if r:
+            part, first, coefs = hist.ahead[r - 1], i - r + 2, coefs[:1]
+        elif len(coefs) > 1:
+            ahead = hist.ahead = torch.empty(len(coefs) - 1, *x.shape, dtype=torch.float32, device=x.device)
+    ext().depth_step(x, x_out, X, i, first, part, keep, y1, g1, b1, y2, y2_rows, g2, b2, y2_b, coefs or [], ahead, norm_w, eps,
+                     w_offset, h, rows)
     return x_out, h
 
 

@@ -327,9 +327,9 @@ def test_single_writes_show_at_every_distance(H, N, P):
 # ------------------------------------------------------------------------------------------- residual, gates, depth average
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("W", [64, 90, 2048, 5000])
-@pytest.mark.parametrize("T", [1, 37])
+@pytest.mark.parametrize("T", [1, 37, 400])
 def test_gated_residual_and_depth_average(device, dtype, W, T):
-    eps, L = 1e-5, 6
+    eps, L = 1e-5, 10
     dev = lambda t: t.to(device)                                            # noqa: E731
     emb = rnd(40, W, seed=1, dtype=dtype)
     ids = torch.randint(0, 40, (T,), generator=torch.Generator().manual_seed(2)).int()
@@ -337,13 +337,13 @@ def test_gated_residual_and_depth_average(device, dtype, W, T):
     for average, gated in ((True, True), (True, False), (False, True)):
         x, hist, h = ops.depth_start(dev(emb), dev(ids), L, dev(n0), eps, 1.0, average)
         wx = d(emb)[ids.long()]
-        outputs = [wx]
+        outputs, all_coef = [wx], [rnd(i + 2, seed=60 + i, k=0.6) for i in range(L)]
         assert (hist is not None) == average
         close(h, oracle.model_norm(wx, d(n0), eps), dtype)
         for i in range(L):
             proj = rnd(T, 2 * W + 24, seed=10 + i, dtype=dtype)
             y1, y2, bias = rnd(T, W, seed=20 + i, dtype=dtype), rnd(T, W, seed=30 + i, dtype=dtype), rnd(W, seed=40 + i)
-            gb, coef, nw = rnd(2 * W, seed=50 + i), rnd(i + 2, seed=60 + i), rnd(W, seed=70 + i, k=0.3)
+            gb, coef, nw = rnd(2 * W, seed=50 + i), all_coef[i], rnd(W, seed=70 + i, k=0.3)
             has_ff, has_bias, last = i != 2, i % 2 == 0, i + 1 == L
             rows = torch.tensor([T - 1, 0, T - 1]) if last else None
             g1, g2 = proj[:, 8:8 + W], proj[:, 16 + W:16 + 2 * W]
@@ -363,7 +363,7 @@ def test_gated_residual_and_depth_average(device, dtype, W, T):
             x, h = ops.depth_step(x, hist, i, dev(y1), pd[:, 8:8 + W] if gated else None, dev(gb)[:W] if gated else None,
                                   y2_dev if has_ff else None, pd[:, 16 + W:16 + 2 * W] if gated and has_ff else None,
                                   dev(gb)[W:] if gated and has_ff else None, dev(bias) if has_bias else None,
-                                  dev(coef) if average else None, dev(nw), eps, 1.0, dev(rows) if last else None)
+                                  [dev(c) for c in all_coef[i:i + 4]] if average else None, dev(nw), eps, 1.0, dev(rows) if last else None)
             if last:
                 wx = wx[rows]
             close(x, wx, torch.float32, 5e-6 if dtype == torch.float32 else 5e-5)
