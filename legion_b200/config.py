@@ -455,6 +455,11 @@ class ModelConfig:
         n = 0 if lo is None else lo.stop - lo.start
         return n > 0 and lo.start <= il < lo.start + n * lo.times and (il - lo.start) % n == 0
 
+    def stream_rows(self) -> int:
+        """float32 rows of the residual's width that a step keeps per token until its end: with depth averages the embedding
+        output, every layer's result and the sums made ahead."""
+        return self.n_layer + 1 + 3 if self.depth_average else 0
+
     def conv_inputs(self, il: int) -> List[str]:
         """Sublayers of layer il whose input passes a short convolution (``input_conv``)."""
         if self.layers is None or self.input_conv < 1:

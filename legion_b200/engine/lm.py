@@ -266,7 +266,8 @@ class LmEngine(Engine):
             del sp
         free, total = torch.cuda.mem_get_info(dev)
         m = self.mcfg
-        ws = mp.workspace_reserve(m.hidden, m.vocab, c.max_batch_tokens, c.max_seqs, m.n_expert, m.top_k, m.expert_ff)
+        ws = mp.workspace_reserve(m.hidden, m.vocab, c.max_batch_tokens, c.max_seqs, m.n_expert, m.top_k, m.expert_ff,
+                                  m.stream_rows())
         auto = c.kv_cache_tokens is not None and c.kv_cache_tokens < 0
         asked = 0 if auto else n_blocks * c.block_size
         plan = mp.fit(total, free, torch.cuda.memory_allocated(dev), bpb, c.block_size, state_bytes, ws, c.max_seqs,

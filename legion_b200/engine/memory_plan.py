@@ -51,16 +51,17 @@ class MemoryPlan:
 
 
 def workspace_reserve(hidden: int, vocab: int, max_batch_tokens: int, max_seqs: int, n_expert: int, top_k: int,
-                      expert_ff: int) -> int:
+                      expert_ff: int, stream_rows: int = 0) -> int:
     """Bytes a step needs beside weights and pools: activations of the widest layer for a full batch, the logits of
     every sequence, the expert-sorted copies of a prompt-sized MoE step, split-K and attention workspaces, and the
-    private pools of the captured decode graphs (one per batch bucket)."""
+    private pools of the captured decode graphs (one per batch bucket). ``stream_rows``: float32 rows of the residual's width
+    that a step keeps per token (``ModelConfig.stream_rows``)."""
     T = max_batch_tokens
     act = T * hidden * 2 * 12                                  # residual, normed, projections, attention output ...
     moe = T * max(1, top_k) * (hidden + expert_ff) * 2 * 2 if n_expert else 0
     logits = max_seqs * vocab * 4 * 3
     fixed = (64 + 32 + 256) << 20                              # split-K, attention partials, graph pools
-    return int(act + moe + logits + fixed)
+    return int(act + moe + logits + fixed + T * hidden * 4 * stream_rows)
 
 
 def fit(total_bytes: int, free_bytes: int, weights_bytes: int, bytes_per_block: int, block_size: int,

@@ -14,6 +14,7 @@ import mananex_oracle as oracle
 import nisasun_case as nc
 from legion_b200.config import DenseSpec, LayerSpec, MoeSpec, PRESETS, Hgrn2Spec, ModelConfig
 from legion_b200.engine.lm import EngineConfig, LmEngine, build_engine
+from legion_b200.engine.memory_plan import workspace_reserve
 from legion_b200.engine.replay import TraceReplay, replay_engine
 from legion_b200.engine.types import GenerateRequest, SamplingParams
 from legion_b200.hw.gpu import model_bytes_per_step
@@ -91,6 +92,9 @@ def test_registry_and_config_round_trip():
     assert list(col) == ["q", "k", "v", "g", "rq", "rf", "rv", "rg1", "rg2", "end"]
     assert all(v % 8 == 0 for v in col.values()) and col["g"] == 3 * 40 + 40 + 32 and col["rq"] == col["g"] + 8
     assert model_bytes_per_step(c, 4, 100)["total_bytes"] > 0
+    assert c.stream_rows() == 8 and PRESETS["tiny-gurozen"]().stream_rows() == 0
+    reserve = [workspace_reserve(144, 512, 1000, 4, 0, 0, 0, n) for n in (0, c.stream_rows())]
+    assert reserve[1] - reserve[0] == 1000 * 144 * 4 * 8
     with pytest.raises(ValueError, match="parallel sublayers"):
         ModelConfig(layers=[LayerSpec(Hgrn2Spec(1, 8, 8), DenseSpec(8, bias=True))])
 

@@ -245,12 +245,10 @@ CUTS = {"whole": [[300]] * 4, "tokens": [[1]] * 4, "twos": [[2]] * 4,
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("H,N,P", HEADS)
-@pytest.mark.parametrize("cuts", list(CUTS))
+@pytest.mark.parametrize("H,N,P,cuts", [(*s, c) for s in HEADS for c in ("whole", "mixed")]
+                         + [(*s, c) for s in HEADS[:4] for c in ("tokens", "twos")])
 def test_forget_scan_in_portions(device, dtype, H, N, P, cuts):
     """Unequal sequences in portions of every size, states in slots that others used, outputs beside other columns."""
-    if cuts in ("tokens", "twos") and (H, N, P) not in HEADS[:4]:
-        pytest.skip("covered by the first sizes")
     eps, scale = 1e-5, 0.8
     qs, fs, vs, b, lower, nw = forget_case(dtype, H, N, P, LENS)
     want = [forget_expected(q, f, v, b, lower, nw, H, N, P, eps, scale) for q, f, v in zip(qs, fs, vs)]
@@ -385,13 +383,11 @@ def test_biases_of_the_gated_feed_forward_part(device, dtype, T, K, ff):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("T", [1, 13, 64, 65, 200])
-@pytest.mark.parametrize("W,ff,E,top", [(96, 56, 6, 3), (256, 64, 8, 2), (90, 27, 3, 1), (64, 40, 4, 4), (4096, 16, 140, 6)])
+@pytest.mark.parametrize("T,W,ff,E,top", [(t, *s) for t in (1, 13, 64, 65, 200) for s in (
+    (96, 56, 6, 3), (256, 64, 8, 2), (90, 27, 3, 1), (64, 40, 4, 4))] + [(1, 4096, 16, 140, 6), (13, 4096, 16, 140, 6)])
 def test_experts_behind_a_router_with_a_logit_bias(device, dtype, T, W, ff, E, top):
     """Through the model's own feed-forward function. The bias decides choices (some experts lead by it alone) and weights."""
     from legion_b200.models.decoder import Decoder
-    if E > 100 and T > 13:
-        pytest.skip("wide model: decode-sized steps")
     x = rnd(T, W, seed=1, dtype=dtype)
     ow = {"m.router": rnd(E, W, seed=2, dtype=dtype, k=2 * W ** -0.5), "m.router.b": rnd(E, seed=3, k=2.0)}
     for e in range(E):
