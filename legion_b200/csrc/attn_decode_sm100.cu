@@ -59,10 +59,7 @@ struct DecodeTcArgs {
   __nv_bfloat16* out;   // [B, Hq, dv]
   int* group_ctr;  // [B * gridDim.x] arrival counters of the splits, zero on entry, left zero on exit
   int* status;
-  AttnExtra x;
 };
-
-enum : int { ATTN_PLAIN = 0, ATTN_CAP = 1, ATTN_EXT = 2 };
 
 template <int DK, int DV>
 struct DecodeTcCfg {
@@ -93,9 +90,15 @@ static constexpr float DEC_RESCALE_LOG2 = 8.f;
 template <int DK, int DV, int MODE>
 __global__ void __launch_bounds__(320, 1)
 paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                       const __grid_constant__ CUtensorMap tmV, const DecodeTcArgs a) {
+                       const __grid_constant__ CUtensorMap tmV, const DecodeTcArgs a, const AttnExtraArg<MODE> x) {
   using Cfg = DecodeTcCfg<DK, DV>;
   constexpr bool CAP = MODE == ATTN_CAP, EXT = MODE == ATTN_EXT;
+  int keep = 0;                                          // first tokens that stay visible behind the window
+  const float* sink = nullptr;
+  if constexpr (EXT) {
+    keep = x.keep;
+    sink = x.sink;
+  }
   constexpr int NQ = Cfg::NQ, BKV = Cfg::BKV, HALVES = Cfg::HALVES, MT = Cfg::MT;
   constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ uint8_t smem_raw[];
@@ -134,7 +137,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int ctx = a.ctx_lens[b];
   const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
   const int blk_first = start / BKV;
-  const int n_keep = EXT ? min((a.x.keep + BKV - 1) / BKV, blk_first) : 0;    // tiles of kept tokens in front of the window's
+  const int n_keep = EXT ? min((keep + BKV - 1) / BKV, blk_first) : 0;    // tiles of kept tokens in front of the window's
   const int n_units = n_keep + (ctx + BKV - 1) / BKV - blk_first;
   const int units_per = (n_units + a.n_splits - 1) / a.n_splits;
   const int blk_lo = blk_first - n_keep + split * units_per;                 // (counted as if the kept tiles led up to the window)
@@ -317,7 +320,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           tmem_ld_wait();
         }
         const int tok = blk_of(i) * BKV + tl;
-        const bool valid = (tok >= start || (EXT && tok < a.x.keep)) && tok < ctx;
+        const bool valid = (tok >= start || (EXT && tok < keep)) && tok < ctx;
         // Only the gn real heads are processed (the MMA's N is padded to 16). The common case needs no column
         // maxima at all: as long as no score exceeds its column's reference maximum by more than the rescale
         // threshold, the probabilities are taken relative to the (stale) reference. The "any score over"
@@ -481,7 +484,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     for (int sidx = lane; sidx < ns; sidx += 32) mm = fmaxf(mm, s_w[q * ns + sidx]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
-    if (EXT && a.x.sink) mm = fmaxf(mm, a.x.sink[head0 + q]);
+    if (EXT && sink) mm = fmaxf(mm, sink[head0 + q]);
     float ll = 0.f;
     for (int sidx = lane; sidx < ns; sidx += 32) {
       const float m = s_w[q * ns + sidx];
@@ -492,7 +495,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, o);
-    if (EXT && a.x.sink) ll += __expf(a.x.sink[head0 + q] - mm);
+    if (EXT && sink) ll += __expf(sink[head0 + q] - mm);
     if (lane == 0) s_l[q] = ll;
   }
   __syncthreads();
@@ -506,10 +509,10 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
     const float ll = s_l[q];
     if constexpr (EXT) {
-      float f = ll > 0.f ? a.x.out_scale / ll : 0.f;
-      if (a.x.gate)
-        f /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.x.gate)[b * a.x.ld_gate + head0 + q]));
-      a.out[b * a.x.ldo + (head0 + q) * D + d] = __float2bfloat16(o * f);
+      float f = ll > 0.f ? x.out_scale / ll : 0.f;
+      if (x.gate)
+        f /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(x.gate)[b * x.ld_gate + head0 + q]));
+      a.out[b * x.ldo + (head0 + q) * D + d] = __float2bfloat16(o * f);
       continue;
     }
     a.out[(long(b) * a.Hq + head0 + q) * D + d] = __float2bfloat16(ll > 0.f ? o / ll : 0.f);
@@ -521,7 +524,7 @@ thread_local char g_dec_err[256];
 
 template <int DK, int DV, int MODE>
 int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const DecodeTcArgs& a,
-                     dim3 grid, cudaStream_t s) {
+                     dim3 grid, cudaStream_t s, const AttnExtra& x) {
   using Cfg = DecodeTcCfg<DK, DV>;
   auto kfn = paged_decode_tc_kernel<DK, DV, MODE>;
   static bool attr = false;
@@ -532,7 +535,9 @@ int launch_decode_tc(const CUtensorMap* tq, const CUtensorMap* tk, const CUtenso
     }
     attr = true;
   }
-  launch_pdl(kfn, grid, dim3(320), Cfg::SMEM, s, *tq, *tk, *tv, a);
+  AttnExtraArg<MODE> xa;
+  if constexpr (MODE == ATTN_EXT) xa = AttnExtraArg<MODE>(x);
+  launch_pdl(kfn, grid, dim3(320), Cfg::SMEM, s, *tq, *tk, *tv, a, xa);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     snprintf(g_dec_err, sizeof(g_dec_err), "decode attention launch: %s", cudaGetErrorString(e));
@@ -578,7 +583,6 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   }
   a.o_part = o_part; a.ml_part = ml_part; a.status = status; a.dv = dv;
   a.out = static_cast<__nv_bfloat16*>(out); a.group_ctr = group_ctr;
-  a.x = x;
   if (x.on && (cap || x.keep < 0)) {
     snprintf(g_dec_err, sizeof(g_dec_err), "decode attention: sinks, kept tokens and gates come without a soft cap");
     return 1;
@@ -586,9 +590,9 @@ int paged_decode_tc_launch(const void* q, const void* k_cache, const void* v_cac
   dim3 grid(Hkv * gtiles, B, n_splits);
 #define LB_DIM(K_, V_)                                                                                    \
   if (DK == K_ && DV == V_)                                                                               \
-    return x.on  ? launch_decode_tc<K_, V_, ATTN_EXT>(tq, tk, tv, a, grid, s)                             \
-           : cap ? launch_decode_tc<K_, V_, ATTN_CAP>(tq, tk, tv, a, grid, s)                             \
-                 : launch_decode_tc<K_, V_, ATTN_PLAIN>(tq, tk, tv, a, grid, s);
+    return x.on  ? launch_decode_tc<K_, V_, ATTN_EXT>(tq, tk, tv, a, grid, s, x)                             \
+           : cap ? launch_decode_tc<K_, V_, ATTN_CAP>(tq, tk, tv, a, grid, s, x)                             \
+                 : launch_decode_tc<K_, V_, ATTN_PLAIN>(tq, tk, tv, a, grid, s, x);
   LB_DIM(64, 64) LB_DIM(128, 128) LB_DIM(256, 256) LB_DIM(64, 128) LB_DIM(64, 256) LB_DIM(128, 64) LB_DIM(128, 256)
   LB_DIM(256, 64) LB_DIM(256, 128) LB_DIM(64, 192) LB_DIM(128, 192) LB_DIM(256, 192)
 #undef LB_DIM

@@ -13,4 +13,14 @@ struct AttnExtra {
   long ldo = 0;                    // elements between output rows
 };
 
+// Modes of the tensor-core attention kernels; only ATTN_EXT carries the optional parts among its arguments.
+enum : int { ATTN_PLAIN = 0, ATTN_CAP = 1, ATTN_EXT = 2 };
+template <int MODE>
+struct AttnExtraArg {};
+template <>
+struct AttnExtraArg<ATTN_EXT> : AttnExtra {
+  AttnExtraArg() = default;
+  explicit AttnExtraArg(const AttnExtra& x) : AttnExtra(x) {}
+};
+
 }  // namespace lb

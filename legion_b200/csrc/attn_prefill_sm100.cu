@@ -99,10 +99,7 @@ struct PrefillArgs {
   __nv_bfloat16* out;      // [T, Hq, dv]
   int dk, dv;              // head sizes: at most the template's; the tensor maps end there and TMA fills zeros
   int* status;
-  AttnExtra x;
 };
-
-enum : int { ATTN_PLAIN = 0, ATTN_CAP = 1, ATTN_EXT = 2 };
 
 template <int N>
 struct IntC { static constexpr int value = N; };
@@ -129,9 +126,11 @@ struct PrefillCfg {
 template <int DK, int DV, int BKV, int MODE>
 __global__ void __launch_bounds__(160, (DK <= 128 && DV <= 128 && BKV == 64) ? 2 : 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                    const __grid_constant__ CUtensorMap tmV, const PrefillArgs a) {
+                    const __grid_constant__ CUtensorMap tmV, const PrefillArgs a, const AttnExtraArg<MODE> x) {
   using Cfg = PrefillCfg<DK, DV, BKV>;
   constexpr bool CAP = MODE == ATTN_CAP, EXT = MODE == ATTN_EXT;
+  int keep = 0;                           // first tokens that stay visible behind the window
+  if constexpr (EXT) keep = x.keep;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw;
   if (smem_u32(smem_raw) & 1023u) {       // swizzled tiles need 1024-byte alignment; uniform per CTA, before any barrier
@@ -202,7 +201,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const int blk_lo = kv_lo / BKV;
   const int blk_hi = (kv_hi + BKV - 1) / BKV;                     // exclusive
   // blocks of kept first tokens that lie in front of the window's
-  const int n_keep = EXT ? min((a.x.keep + BKV - 1) / BKV, blk_lo) : 0;
+  const int n_keep = EXT ? min((keep + BKV - 1) / BKV, blk_lo) : 0;
   const int n_blk = n_keep + blk_hi - blk_lo;
   auto blk_of = [&](int i) { return EXT && i < n_keep ? i : blk_lo - n_keep + i; };
   const int* bt = a.block_table + long(seq) * a.table_width;
@@ -303,9 +302,11 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const bool row_ok = row < rows_here;
     const uint32_t lane_off = uint32_t(warp * 32) << 16;
     float m = -INFINITY, l = 0.f;
-    if (EXT && a.x.sink) {                 // as if a key with this score and no value had been seen
-      m = a.x.sink[head] * 1.4426950408889634f;
-      l = 1.f;
+    if constexpr (EXT) {
+      if (x.sink) {                        // as if a key with this score and no value had been seen
+        m = x.sink[head] * 1.4426950408889634f;
+        l = 1.f;
+      }
     }
     bool ok = true;
     for (int i = 0; i < n_blk; ++i) {
@@ -320,9 +321,9 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (!row_ok) { hi = 0; lo = 0; }
       // blocks entirely inside every row's visible range need no per-element mask (all interior blocks of a
       // causal prompt): uniform over the CTA
-      const bool full_blk = (a.window == 0 || (EXT && (key0 > last_pos - a.window || key0 + BKV <= a.x.keep))) &&
+      const bool full_blk = (a.window == 0 || (EXT && (key0 > last_pos - a.window || key0 + BKV <= keep))) &&
                             rows_here == 128 && key0 + BKV <= (a.causal ? min(ctx, pos0 + 1) : ctx);
-      auto seen = [&](int key) { return (key >= lo || (EXT && key < a.x.keep)) && key < hi; };
+      auto seen = [&](int key) { return (key >= lo || (EXT && key < keep)) && key < hi; };
       float alpha = 1.f;
       float sum = 0.f;
       if (BKV <= 64) {
@@ -483,10 +484,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       __nv_bfloat16* orow = a.out + (long(q0 + tile_row0 + row) * a.Hq + head) * a.dv;
       if constexpr (EXT) {
         const long t = q0 + tile_row0 + row;
-        orow = a.out + t * a.x.ldo + head * a.dv;
-        inv *= a.x.out_scale;
-        if (a.x.gate && row_ok)
-          inv /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.x.gate)[t * a.x.ld_gate + head]));
+        orow = a.out + t * x.ldo + head * a.dv;
+        inv *= x.out_scale;
+        if (x.gate && row_ok)
+          inv /= 1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(x.gate)[t * x.ld_gate + head]));
       }
 #pragma unroll 1
       for (int c = 0; c < DV; c += 32) {
@@ -526,7 +527,7 @@ thread_local char g_attn_err[256];
 
 template <int DK, int DV, int BKV, int MODE = ATTN_PLAIN>
 int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const PrefillArgs& a,
-                   dim3 grid, cudaStream_t s) {
+                   dim3 grid, cudaStream_t s, const AttnExtra& x) {
   using Cfg = PrefillCfg<DK, DV, BKV>;
   static_assert(MODE != ATTN_CAP || BKV <= 64, "the soft cap is applied to a row of scores in registers");
   auto kfn = prefill_attn_kernel<DK, DV, BKV, MODE>;
@@ -538,7 +539,9 @@ int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorM
     }
     attr = true;
   }
-  kfn<<<grid, 160, Cfg::SMEM, s>>>(*tq, *tk, *tv, a);
+  AttnExtraArg<MODE> xa;
+  if constexpr (MODE == ATTN_EXT) xa = AttnExtraArg<MODE>(x);
+  kfn<<<grid, 160, Cfg::SMEM, s>>>(*tq, *tk, *tv, a, xa);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     snprintf(g_attn_err, sizeof(g_attn_err), "prefill attention launch: %s", cudaGetErrorString(e));
@@ -591,13 +594,12 @@ int prefill_attn_launch(const void* q, long T, const void* k_cache, const void* 
     a.scale_log2 = 2.f * 1.4426950408889634f * softcap;
   }
   a.out = static_cast<__nv_bfloat16*>(out); a.dk = dk; a.dv = dv; a.status = status;
-  a.x = x;
   dim3 grid((max_q_len + 127) / 128, Hq, n_seqs);
 #define LB_DIM(K_, V_, B_)                                                                   \
   if (DK == K_ && DV == V_)                                                                  \
-    return x.on  ? launch_prefill<K_, V_, 64, ATTN_EXT>(tq, tk, tv, a, grid, s)               \
-           : cap ? launch_prefill<K_, V_, 64, ATTN_CAP>(tq, tk, tv, a, grid, s)               \
-                 : launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s);
+    return x.on  ? launch_prefill<K_, V_, 64, ATTN_EXT>(tq, tk, tv, a, grid, s, x)               \
+           : cap ? launch_prefill<K_, V_, 64, ATTN_CAP>(tq, tk, tv, a, grid, s, x)               \
+                 : launch_prefill<K_, V_, B_>(tq, tk, tv, a, grid, s, x);
   LB_DIM(64, 64, 128) LB_DIM(128, 128, 64) LB_DIM(256, 256, 64)
   LB_DIM(64, 128, 64) LB_DIM(64, 256, 64) LB_DIM(128, 64, 64) LB_DIM(128, 256, 64) LB_DIM(256, 64, 64)
   LB_DIM(64, 192, 64) LB_DIM(128, 192, 64) LB_DIM(256, 192, 64) LB_DIM(256, 128, 64)

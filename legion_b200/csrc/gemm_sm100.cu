@@ -121,7 +121,7 @@ __device__ __forceinline__ float gate_act(float v, int act) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
 }
 
-// UNARY: the output passes xIELU with the two numbers of WgemmArgs::xielu, or max(., 0)^2; UN_BIAS: gate and up get their
+// UNARY: the output passes xIELU with its two WgemmArgs::numbers, or max(., 0)^2; UN_BIAS: gate and up get their
 // biases (DUAL). Variants of their own, as is the
 // lookahead of output rows for wide token tiles: decode-sized launches run the epilogue once, and code they skip still
 // costs them instruction fetches.
@@ -590,7 +590,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
           }
           if constexpr (UNARY == UN_BIAS) {
             const int feat = it.feat0 + row;
-            const float bg = feat < a.n_feat ? a.bias[feat] : 0.f, bu = feat < a.n_feat ? a.bias[a.n_feat + feat] : 0.f;
+            const float bg = feat < a.n_feat ? a.numbers[feat] : 0.f, bu = feat < a.n_feat ? a.numbers[a.n_feat + feat] : 0.f;
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               g[j] += bg;
@@ -605,7 +605,7 @@ wgemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CU
             }
           }
           if constexpr (UNARY == UN_XIELU) {
-            const float xi_a = a.xielu[0], xi_b = a.xielu[1];
+            const float xi_a = a.numbers[0], xi_b = a.numbers[1];
 #pragma unroll
             for (int j = 0; j < 32; ++j) g[j] = xielu_fast(g[j], xi_a, xi_b);
           }
@@ -949,7 +949,7 @@ int wgemm_launch(const WgemmHost& h, cudaStream_t stream) {
   }
   a.tile_group = h.tile_group; a.tile_tok0 = h.tile_tok0; a.tile_out0 = h.tile_out0; a.tile_ntok = h.tile_ntok; a.n_tiles_dev = h.n_tiles_dev;
   a.n_tok_tiles_max = h.n_tok_tiles_max;
-  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act; a.xielu = h.xielu; a.bias = h.bias;
+  a.rows_per_group = h.rows_per_group; a.dual_offset = h.dual_offset; a.act = h.act; a.numbers = h.bias ? h.bias : h.xielu;
   a.x_group_col = h.x_group_col;
   // (a last K tile that reaches into the next group's columns meets weights that TMA filled with zeros)
   if (h.x_group_col != 0 && (h.x_group_col % 8 != 0 || h.K % 8 != 0 || fp8 || fp4 || !h.tile_group)) {

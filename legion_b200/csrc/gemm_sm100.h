@@ -61,8 +61,8 @@ struct WgemmArgs {
                                   //   projections read their head's slice of a [tokens, heads * width] tensor in place)
   int dual_offset;                // DUAL: rows from a feature's gate row to its up row
   int act;                        // DUAL: activation of the gate, 0 = silu, 1 = gelu (tanh form)
-  const float* xielu;             // not DUAL, xIELU variant: its two numbers (act_type.cuh)
-  const float* bias;              // DUAL, bias variant: added to gate (n_feat numbers) and up (the same, behind them)
+  const float* numbers;           // xIELU variant: its two numbers (act_type.cuh); bias variant (DUAL): added to gate (n_feat
+                                  //   numbers) and up (the same, behind them)
   int split_k;
   int vec_ok;                     // output rows may be written as aligned 16-byte vectors
   float* ws;                      // split-K partials
