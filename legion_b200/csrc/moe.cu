@@ -688,41 +688,48 @@ __global__ void __launch_bounds__(512) moe_scan_kernel(const int* __restrict__ c
   }
   if (e == 0) offsets[n_local] = s_off[n_local];
 }
-// pass 3: one CTA per local expert writes its pairs, in pair order, at its offset.
-__global__ void __launch_bounds__(256) moe_fill_kernel(const int* __restrict__ ids, const float* __restrict__ wts,
-                                                       int n_pairs, int k, int e_lo, const int* __restrict__ offsets,
-                                                       int* __restrict__ sorted_token, int* __restrict__ sorted_pair,
-                                                       float* __restrict__ sorted_w) {
+// pass 3: one CTA per local expert writes its pairs, in pair order, at its offset. A thread looks at FILL consecutive pairs per
+// turn, so that the barriers of the running count come once per several thousand pairs.
+constexpr int FILL = 8;
+__global__ void __launch_bounds__(1024) moe_fill_kernel(const int* __restrict__ ids, const float* __restrict__ wts,
+                                                        int n_pairs, int k, int e_lo, const int* __restrict__ offsets,
+                                                        int* __restrict__ sorted_token, int* __restrict__ sorted_pair,
+                                                        float* __restrict__ sorted_w) {
   const int e = e_lo + blockIdx.x;
-  const int base0 = offsets[blockIdx.x];
-  __shared__ int warp_tot[8];
-  __shared__ int running;
-  if (threadIdx.x == 0) running = 0;
-  __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int p0 = 0; p0 < n_pairs; p0 += 256) {
-    const int p = p0 + threadIdx.x;
-    const bool hit = p < n_pairs && ids[p] == e;
-    const unsigned bal = __ballot_sync(0xffffffffu, hit);
-    const int before = __popc(bal & ((1u << lane) - 1));
-    if (lane == 0) warp_tot[warp] = __popc(bal);
-    __syncthreads();
-    int wbase = 0;
-    for (int w = 0; w < warp; ++w) wbase += warp_tot[w];
-    const int base = running;
-    if (hit) {
-      const int dst = base0 + base + wbase + before;
-      sorted_token[dst] = p / k;
-      sorted_pair[dst] = p;
-      sorted_w[dst] = wts[p];
+  int base = offsets[blockIdx.x];
+  __shared__ int warp_tot[2][32];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  int turn = 0;
+  for (int p0 = 0; p0 < n_pairs; p0 += blockDim.x * FILL, turn ^= 1) {
+    const int p = p0 + threadIdx.x * FILL;
+    unsigned hits = 0;
+#pragma unroll
+    for (int j = 0; j < FILL; ++j)
+      if (p + j < n_pairs && ids[p + j] == e) hits |= 1u << j;
+    int incl = __popc(hits);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int n = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += n;
     }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-      int t = 0;
-      for (int w = 0; w < 8; ++w) t += warp_tot[w];
-      running = base + t;
+    if (lane == 31) warp_tot[turn][warp] = incl;
+    __syncthreads();                        // (the next turn writes the other row: no second barrier)
+    int mine = lane < n_warps ? warp_tot[turn][lane] : 0, before = lane < warp ? mine : 0;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      mine += __shfl_xor_sync(0xffffffffu, mine, o);
+      before += __shfl_xor_sync(0xffffffffu, before, o);
     }
-    __syncthreads();
+    int dst = base + before + incl - __popc(hits);
+    base += mine;
+    while (hits) {
+      const int q = p + __ffs(hits) - 1;
+      hits &= hits - 1;
+      sorted_token[dst] = q / k;
+      sorted_pair[dst] = q;
+      sorted_w[dst] = wts[q];
+      ++dst;
+    }
   }
 }
 
@@ -733,7 +740,7 @@ int moe_plan_launch(const int* ids, const float* wts, int n_tokens, int k, int e
   const int n_pairs = n_tokens * k;
   moe_count_kernel<<<n_local, 256, 0, s>>>(ids, n_pairs, e_lo, counts);
   moe_scan_kernel<<<1, 512, 0, s>>>(counts, n_local, bn, offsets, tile_group, tile_tok0, tile_ntok, max_tiles, meta);
-  moe_fill_kernel<<<n_local, 256, 0, s>>>(ids, wts, n_pairs, k, e_lo, offsets, sorted_token, sorted_pair, sorted_w);
+  moe_fill_kernel<<<n_local, n_pairs > 2048 ? 1024 : 256, 0, s>>>(ids, wts, n_pairs, k, e_lo, offsets, sorted_token, sorted_pair, sorted_w);
   return cudaGetLastError() != cudaSuccess;
 }
 
