@@ -94,7 +94,7 @@ def test_rotated_rows_on_their_way_to_the_cache(device, dtype, H, G, dk, dv, dim
     assert torch.equal(d(v_dev).view(-1, G, dv), want_vc)
 
 
-@pytest.mark.parametrize("dims,base", [(2, 10.0), (16, 1e6), (24, 1e4), (128, 5e5)])
+@pytest.mark.parametrize("dims,base", [(2, 10.0), (16, 2e5), (24, 1e4), (128, 1e6)])
 def test_rotation_frequencies(dims, base):
     from legion_b200.models.decoder import Decoder
     dec = Decoder.__new__(Decoder)
@@ -171,7 +171,7 @@ def test_sink_attention_with_kept_first_tokens(device, dtype, H, G, dk, dv, wind
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("window,keep,far", [(72, 4, 500), (64, 1, 320), (128, 130, 700), (200, 64, 513), (1, 2, 130)])
+@pytest.mark.parametrize("window,keep,far", [(75, 3, 500), (64, 1, 320), (128, 130, 700), (200, 64, 513), (1, 2, 130)])
 def test_edges_of_the_window_and_of_the_kept_tokens(device, dtype, window, keep, far):
     """One key stands out for every query: it must show just inside the window and among the kept first tokens, and be gone
     right behind either edge; as a single decoded token, as the last of a portion of two, and inside longer portions."""
